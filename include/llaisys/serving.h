@@ -1,5 +1,5 @@
 /*
- * llaisys C ABI -- iteration-level ("continuous") batching engine over a Qwen2 model and its paged KV cache.
+ * llaisys C ABI -- iteration-level ("continuous") batching engine over a model and its cache.
  *
  * New: the reference describes a multi-user service with a request queue, continuous batching and a KV-cache pool with
  * prefix matching as future work (reference: README.md:415-424) and has no code for it. Status codes as in paged_kv.h.
@@ -9,7 +9,7 @@
 #ifndef LLAISYS_SERVING_H
 #define LLAISYS_SERVING_H
 
-#include "models/qwen2.h"
+#include "models/model.h"
 
 #ifdef __cplusplus
 extern "C" {
@@ -25,9 +25,9 @@ struct LlaisysEngineEvent {
 };
 
 /* max_batch requests per step; at most max_tokens_per_step tokens per step (one per decoding request first, prompt
- * chunks of at most prefill_chunk tokens per request with the rest). llaisysQwen2ModelConfigureCache must have sized
+ * chunks of at most prefill_chunk tokens per request with the rest). llaisysModelConfigureCache must have sized
  * the model's cache: its max_seqs bounds the live requests, its pages bound what can be admitted. */
-LLAISYS_API int llaisysEngineCreate(struct LlaisysEngine **engine_out, struct LlaisysQwen2Model *model, size_t max_batch,
+LLAISYS_API int llaisysEngineCreate(struct LlaisysEngine **engine_out, struct LlaisysModel *model, size_t max_batch,
                                     size_t max_tokens_per_step, size_t prefill_chunk);
 LLAISYS_API void llaisysEngineDestroy(struct LlaisysEngine *engine);
 /* Queues a request (first come, first served). end_token < 0 = the model's. A request is admitted to the running set

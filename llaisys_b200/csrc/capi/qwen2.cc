@@ -3,38 +3,12 @@
 #include "llaisys/models/qwen2.h"
 #include "llaisys/paged_kv.h"
 
-#include "../models/qwen2.hpp"
+#include "model_handle.hpp"
 
 #include <iostream>
 
-#include "qwen2_handle.hpp"
-
-namespace llaisys::kernels {
-void set_last_error(const std::string &msg);
-}
-
-namespace {
-template <typename F>
-int guarded(F &&body) {
-    try {
-        body();
-        return LLAISYS_OK;
-    } catch (const llaisys::kv::StatusError &e) {
-        llaisys::kernels::set_last_error(e.what());
-        return e.code;
-    } catch (const std::invalid_argument &e) {
-        llaisys::kernels::set_last_error(e.what());
-        return LLAISYS_E_INVALID;
-    } catch (const std::exception &e) {
-        llaisys::kernels::set_last_error(e.what());
-        return LLAISYS_E_DEVICE;
-    }
-}
-int null_model() {
-    llaisys::kernels::set_last_error("qwen2: null model handle");
-    return LLAISYS_E_INVALID;
-}
-} // namespace
+using llaisys::capi::guarded;
+using llaisys::capi::null_model;
 
 extern "C" {
 
@@ -78,9 +52,9 @@ int llaisysQwen2ModelSetAllReduceNccl(LlaisysQwen2Model *model, const void *uniq
         return null_model();
     }
     return guarded([&] {
-        llaisys::core::context().setDevice(model->impl.deviceType(), model->impl.deviceId());
-        model->impl.setCollective(
-            llaisys::comm::Collective::nccl(unique_id_128_bytes, model->impl.tpRank(), model->impl.tpWorld()));
+        llaisys::core::context().setDevice(model->qwen2().deviceType(), model->qwen2().deviceId());
+        model->qwen2().setCollective(
+            llaisys::comm::Collective::nccl(unique_id_128_bytes, model->qwen2().tpRank(), model->qwen2().tpWorld()));
     });
 }
 
@@ -89,52 +63,52 @@ int llaisysQwen2ModelSetAllReduceCallback(LlaisysQwen2Model *model, llaisysAllRe
         return null_model();
     }
     return guarded([&] {
-        model->impl.setCollective(llaisys::comm::Collective::callback(fn, user, model->impl.tpRank(), model->impl.tpWorld()));
+        model->qwen2().setCollective(llaisys::comm::Collective::callback(fn, user, model->qwen2().tpRank(), model->qwen2().tpWorld()));
     });
 }
 
 void llaisysQwen2ModelDestroy(LlaisysQwen2Model *model) { delete model; }
 
-LlaisysQwen2Weights *llaisysQwen2ModelWeights(LlaisysQwen2Model *model) { return model ? model->impl.weights() : nullptr; }
+LlaisysQwen2Weights *llaisysQwen2ModelWeights(LlaisysQwen2Model *model) { return model ? model->qwen2().weights() : nullptr; }
 
 int64_t llaisysQwen2ModelInfer(LlaisysQwen2Model *model, int64_t *token_ids, size_t ntoken) {
     // legacy convention: misuse throws through the C frame
-    return model->impl.infer(token_ids, ntoken);
+    return model->impl->infer(token_ids, ntoken);
 }
 
 int llaisysQwen2ModelConfigureCache(LlaisysQwen2Model *model, size_t max_seqs, size_t max_tokens) {
-    return model ? guarded([&] { model->impl.configureCache(max_seqs, max_tokens); }) : null_model();
+    return model ? guarded([&] { model->impl->configureCache(max_seqs, max_tokens); }) : null_model();
 }
 int llaisysQwen2ModelSeqAdd(LlaisysQwen2Model *model, int32_t *seq_out) {
     if (model == nullptr || seq_out == nullptr) {
         return null_model();
     }
-    return guarded([&] { *seq_out = model->impl.seqAdd(); });
+    return guarded([&] { *seq_out = model->impl->seqAdd(); });
 }
 int llaisysQwen2ModelSeqAddWithPrefix(LlaisysQwen2Model *model, const int64_t *tokens, size_t n, int32_t *seq_out,
                                       size_t *matched_out) {
     if (model == nullptr || seq_out == nullptr || matched_out == nullptr) {
         return null_model();
     }
-    return guarded([&] { *seq_out = model->impl.seqAddWithPrefix(tokens, n, matched_out); });
+    return guarded([&] { *seq_out = model->impl->seqAddWithPrefix(tokens, n, matched_out); });
 }
 int llaisysQwen2ModelSeqFree(LlaisysQwen2Model *model, int32_t seq) {
-    return model ? guarded([&] { model->impl.seqFree(seq); }) : null_model();
+    return model ? guarded([&] { model->impl->seqFree(seq); }) : null_model();
 }
 int llaisysQwen2ModelReset(LlaisysQwen2Model *model) {
-    return model ? guarded([&] { model->impl.reset(); }) : null_model();
+    return model ? guarded([&] { model->impl->reset(); }) : null_model();
 }
 int llaisysQwen2ModelStep(LlaisysQwen2Model *model, const int32_t *seq_ids, const int32_t *n_tokens, size_t n_seqs,
                           const int64_t *tokens, int64_t *next_out) {
-    return model ? guarded([&] { model->impl.step(seq_ids, n_tokens, n_seqs, tokens, next_out); }) : null_model();
+    return model ? guarded([&] { model->impl->step(seq_ids, n_tokens, n_seqs, tokens, next_out); }) : null_model();
 }
 int llaisysQwen2ModelDecodeLoop(LlaisysQwen2Model *model, const int32_t *seq_ids, size_t n_seqs, const int64_t *first_tokens,
                                 size_t n_steps, int64_t *tokens_out) {
-    return model ? guarded([&] { model->impl.decodeLoop(seq_ids, n_seqs, first_tokens, n_steps, tokens_out); }) : null_model();
+    return model ? guarded([&] { model->impl->decodeLoop(seq_ids, n_seqs, first_tokens, n_steps, tokens_out); }) : null_model();
 }
 int llaisysQwen2ModelLastLogits(LlaisysQwen2Model *model, float *out_host, size_t capacity_floats) {
-    return model ? guarded([&] { model->impl.lastLogits(out_host, capacity_floats); }) : null_model();
+    return model ? guarded([&] { model->impl->lastLogits(out_host, capacity_floats); }) : null_model();
 }
-double llaisysQwen2ModelLastLoopMs(LlaisysQwen2Model *model) { return model ? model->impl.lastLoopMs() : 0.0; }
+double llaisysQwen2ModelLastLoopMs(LlaisysQwen2Model *model) { return model ? model->impl->lastLoopMs() : 0.0; }
 
 } // extern "C"

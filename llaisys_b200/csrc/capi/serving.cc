@@ -3,45 +3,27 @@
 #include "llaisys/paged_kv.h"
 
 #include "../serve/engine.hpp"
-#include "qwen2_handle.hpp"
-
-namespace llaisys::kernels {
-void set_last_error(const std::string &msg);
-}
+#include "model_handle.hpp"
 
 struct LlaisysEngine {
     llaisys::serve::Engine impl;
-    LlaisysEngine(llaisys::models::Qwen2 &model, const llaisys::serve::EngineConfig &cfg) : impl(model, cfg) {}
+    LlaisysEngine(llaisys::models::Decoder &model, const llaisys::serve::EngineConfig &cfg) : impl(model, cfg) {}
 };
 
 static_assert(sizeof(LlaisysEngineEvent) == sizeof(llaisys::serve::Event), "event layouts must agree");
 
 namespace {
-template <typename F>
-int guarded(F &&body) {
-    try {
-        body();
-        return LLAISYS_OK;
-    } catch (const llaisys::kv::StatusError &e) {
-        llaisys::kernels::set_last_error(e.what());
-        return e.code;
-    } catch (const std::invalid_argument &e) {
-        llaisys::kernels::set_last_error(e.what());
-        return LLAISYS_E_INVALID;
-    } catch (const std::exception &e) {
-        llaisys::kernels::set_last_error(e.what());
-        return LLAISYS_E_DEVICE;
-    }
-}
 int null_handle() {
     llaisys::kernels::set_last_error("engine: null handle");
     return LLAISYS_E_INVALID;
 }
 } // namespace
 
+using llaisys::capi::guarded;
+
 extern "C" {
 
-int llaisysEngineCreate(LlaisysEngine **engine_out, LlaisysQwen2Model *model, size_t max_batch, size_t max_tokens_per_step,
+int llaisysEngineCreate(LlaisysEngine **engine_out, LlaisysModel *model, size_t max_batch, size_t max_tokens_per_step,
                         size_t prefill_chunk) {
     if (engine_out == nullptr || model == nullptr) {
         return null_handle();
@@ -51,7 +33,7 @@ int llaisysEngineCreate(LlaisysEngine **engine_out, LlaisysQwen2Model *model, si
         cfg.max_batch = max_batch;
         cfg.max_tokens_per_step = max_tokens_per_step;
         cfg.prefill_chunk = prefill_chunk;
-        *engine_out = new LlaisysEngine(model->impl, cfg);
+        *engine_out = new LlaisysEngine(*model->impl, cfg);
     });
 }
 void llaisysEngineDestroy(LlaisysEngine *engine) { delete engine; }

@@ -7,6 +7,12 @@
 #include <cstddef>
 #include <cstdint>
 
+#ifdef __CUDACC__
+#define LLAISYS_ARGS_FN __host__ __device__
+#else
+#define LLAISYS_ARGS_FN
+#endif
+
 namespace llaisys::kernels {
 
 // Where the K and V rows of a sequence live. One description covers both layouts on the path:
@@ -26,7 +32,14 @@ struct KVView {
     int32_t page_size = 16;
     int32_t num_pages = 0; // physical pages addressable through this view (bounds check)
     int32_t nkvh = 0;
-    int32_t d = 0;
+    int32_t d = 0; // elements of a K row (and of a V row unless v_d says otherwise)
+    // V rows of another shape than K rows (0 = the same): used by the generic attention and the norm + append kernel; every
+    // other kernel needs equal shapes.
+    int32_t v_d = 0;
+    int64_t v_head_stride = 0, v_token_stride = 0;
+    LLAISYS_ARGS_FN int32_t vDim() const { return v_d ? v_d : d; }
+    LLAISYS_ARGS_FN int64_t vHeadStride() const { return v_d ? v_head_stride : head_stride; }
+    LLAISYS_ARGS_FN int64_t vTokenStride() const { return v_d ? v_token_stride : token_stride; }
     // Optional TMA view of the same memory (page pools only): a 128-byte tensor-map blob in HOST memory over the
     // whole multi-layer pool, and the index of this layer's page 0 in it (layer * num_pages).
     // Launch append / decode with programmatic stream serialisation: the kernel's set-up and its first K/V copies may
@@ -56,6 +69,7 @@ struct AttnBatch {
     int32_t max_q_len = 1;
     int32_t max_kv_len = 0;
     int32_t nh = 0;
+    int32_t window = 0; // > 0: a query at position i sees keys j with 0 <= i - j < window; 0: all earlier keys
 };
 
 // Output selection: `out` [total_q, nh, d] in the KV dtype, or `part` float [total_q, nh, d + 2] holding the
@@ -63,6 +77,10 @@ struct AttnBatch {
 struct AttnOut {
     void *out = nullptr;
     float *part = nullptr;
+    // out only: every (row, head) of the normalised output is multiplied by row_scale[row * nh + h] (an output gate), and
+    // row r starts at out + r * row_stride elements (0 = packed rows of nh * d)
+    const float *row_scale = nullptr;
+    int64_t row_stride = 0;
     const struct PeerSink *peers = nullptr; // decode over a page pool only: partial rows go to exchange slots instead
 };
 
@@ -87,6 +105,48 @@ struct AttnScratch {
     int32_t *counters = nullptr;  // int32 [counters_len], all zero between launches
     size_t counters_len = 0;
     int32_t *error_flag = nullptr; // set non-zero when a kernel skipped an out-of-range page / position
+};
+
+// K1c: what enters attention without positions, fused: from a packed projection row [.. q | k | v .. gate ..] the per-head
+// RMS norm of q and k (one weight of `d` for all heads), k and v into their page slots, q to a packed tensor, and the
+// output gate of every head turned into a factor for the attention kernel's epilogue.
+struct NormAppendArgs {
+    const void *proj = nullptr; // [n_rows, row_stride] elements of the cache's dtype
+    int64_t row_stride = 0;
+    int64_t q_at = 0, k_at = 0, v_at = 0, gate_at = 0; // first element of each part in a row; gate_at < 0: no gate
+    const void *q_norm = nullptr, *k_norm = nullptr;   // [d], cache dtype; null = no norm
+    float eps = 0.f;
+    void *q_out = nullptr;      // [n_rows, nh, d]
+    float *row_scale = nullptr; // [n_rows, nh] = gate_scale * sigmoid(gate)
+    float gate_scale = 1.f;
+    const int32_t *seq_ids = nullptr, *positions = nullptr; // per row, on the device
+    size_t n_rows = 0;
+    int32_t nh = 0;
+};
+
+// Gated linear attention over one packed projection (per head a state S [dk, dv], decayed per key channel):
+//   S_t = diag(a_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T (q_scale q_t),  a_t = exp(log_sigmoid(W_a2 z_t + b) / tau)
+//   out_t = out_scale * rms_norm(o_t, norm) * silu(g_t)
+// q, k: heads x dk; v, g, out: heads x dv; z: the low-rank half of the decay projection, `rank` numbers shared by all heads.
+struct GatedLinearArgs {
+    const void *proj = nullptr; // [n_rows, row_stride], model dtype
+    int64_t row_stride = 0;
+    int64_t q_at = 0, k_at = 0, v_at = 0, g_at = 0, z_at = 0;
+    const void *decay_w = nullptr; // [heads * dk, rank], model dtype
+    const void *decay_b = nullptr; // [heads * dk]
+    const void *norm_w = nullptr;  // [dv]
+    float tau = 1.f, q_scale = 1.f, eps = 0.f, out_scale = 1.f;
+    int32_t heads = 0, dk = 0, dv = 0, rank = 0;
+    float *state = nullptr; // slot s, head h: state + s * slot_stride + h * dk * dv, row-major [dk, dv]
+    int64_t slot_stride = 0;
+    // the batch: sequence i owns rows [q_starts[i], q_starts[i + 1]) and state slot seq_ids[i]; kv_lens[i] tokens after the
+    // step (a sequence whose first token is in the step starts from zero)
+    const int32_t *seq_ids = nullptr, *q_starts = nullptr, *kv_lens = nullptr;
+    int32_t n_seqs = 0, n_rows = 0, max_q_len = 0;
+    void *out = nullptr; // row r, head h: out + r * out_stride + h * dv, model dtype
+    int64_t out_stride = 0;
+    float *raw = nullptr;   // scratch [n_rows, heads * dv]
+    float *decay = nullptr; // scratch [n_rows, heads * dk]
 };
 
 using stream_t = void *;

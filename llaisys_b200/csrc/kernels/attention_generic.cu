@@ -1,4 +1,4 @@
-// Generic attention over a paged or contiguous K/V view: any of F32 / F16 / BF16, head_dim <= 256, any GQA
+// Generic attention over a paged or contiguous K/V view: any of F32 / F16 / BF16, V rows of up to 256, any GQA
 // ratio, any page size, decode or ragged causal chunks.
 //
 // One CTA of four warps per (query row, query head). Keys are dealt to warps in blocks of 32; inside a warp
@@ -23,12 +23,13 @@ constexpr int kMaxDimsPerLane = 8; // head_dim <= 256
 template <typename T>
 __global__ void __launch_bounds__(kWarps * 32)
     attention_generic_kernel(KVView kv, AttnBatch batch, const T *__restrict__ q, float scale, T *__restrict__ out,
-                             float *__restrict__ part, int32_t *error_flag) {
+                             float *__restrict__ part, const float *__restrict__ row_scale, int64_t out_stride,
+                             int32_t *error_flag) {
     extern __shared__ float smem[];
-    const int d = kv.d;
+    const int d = kv.d, dv = kv.vDim();
     float *q_s = smem;                    // [d] query, pre-multiplied by scale
-    float *acc_s = smem + d;              // [kWarps][d]
-    float *m_s = acc_s + kWarps * d;      // [kWarps]
+    float *acc_s = smem + d;              // [kWarps][dv]
+    float *m_s = acc_s + kWarps * dv;     // [kWarps]
     float *l_s = m_s + kWarps;            // [kWarps]
 
     const int row = blockIdx.x;
@@ -58,6 +59,7 @@ __global__ void __launch_bounds__(kWarps * 32)
     const int kv_len = batch.kv_lens ? batch.kv_lens[seq] : batch.const_kv_len;
     int visible = kv_len - q_len + t + 1; // causal offset: query t sees keys j <= t + (kv_len - q_len)
     visible = visible < 0 ? 0 : (visible > kv_len ? kv_len : visible);
+    const int first = batch.window > 0 ? max(0, visible - batch.window) : 0; // the query sits at position visible - 1
     const int seq_row = batch.seq_ids ? batch.seq_ids[seq] : seq;
     const int kvh = h / (batch.nh / kv.nkvh);
 
@@ -68,7 +70,7 @@ __global__ void __launch_bounds__(kWarps * 32)
     __syncthreads();
 
     const T *k_base = static_cast<const T *>(kv.k_base) + int64_t(kvh) * kv.head_stride;
-    const T *v_base = static_cast<const T *>(kv.v_base) + int64_t(kvh) * kv.head_stride;
+    const T *v_base = static_cast<const T *>(kv.v_base) + int64_t(kvh) * kv.vHeadStride();
 
     float m = -INFINITY, l = 0.f;
     float acc[kMaxDimsPerLane];
@@ -77,10 +79,10 @@ __global__ void __launch_bounds__(kWarps * 32)
         acc[i] = 0.f;
     }
 
-    for (int base = warp * 32; base < visible; base += kWarps * 32) {
+    for (int base = first + warp * 32; base < visible; base += kWarps * 32) {
         const int j = base + lane;
         bool valid = j < visible;
-        int64_t row_off = 0;
+        int64_t row_off = 0, v_off = 0;
         if (valid) {
             const int blk = j / kv.page_size;
             int page = blk;
@@ -92,6 +94,7 @@ __global__ void __launch_bounds__(kWarps * 32)
                 valid = false;
             } else {
                 row_off = int64_t(page) * kv.page_stride + int64_t(j - blk * kv.page_size) * kv.token_stride;
+                v_off = int64_t(page) * kv.page_stride + int64_t(j - blk * kv.page_size) * kv.vTokenStride();
             }
         }
         float s = -INFINITY;
@@ -128,7 +131,7 @@ __global__ void __launch_bounds__(kWarps * 32)
         const int n_here = min(32, visible - base);
         for (int jj = 0; jj < n_here; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
-            const int64_t off = __shfl_sync(0xffffffffu, row_off, jj);
+            const int64_t off = __shfl_sync(0xffffffffu, v_off, jj);
             if (pj == 0.f) {
                 continue; // skipped page or underflow (warp-uniform)
             }
@@ -136,7 +139,7 @@ __global__ void __launch_bounds__(kWarps * 32)
 #pragma unroll
             for (int i = 0; i < kMaxDimsPerLane; ++i) {
                 const int dim = lane + 32 * i;
-                if (dim < d) {
+                if (dim < dv) {
                     acc[i] = fmaf(pj, to_f32(v_row[dim]), acc[i]);
                 }
             }
@@ -151,8 +154,8 @@ __global__ void __launch_bounds__(kWarps * 32)
 #pragma unroll
     for (int i = 0; i < kMaxDimsPerLane; ++i) {
         const int dim = lane + 32 * i;
-        if (dim < d) {
-            acc_s[warp * d + dim] = acc[i];
+        if (dim < dv) {
+            acc_s[warp * dv + dim] = acc[i];
         }
     }
     __syncthreads();
@@ -170,22 +173,23 @@ __global__ void __launch_bounds__(kWarps * 32)
     }
     const float inv_l = l_all > 0.f ? 1.f / l_all : 0.f;
     const int64_t o_row = int64_t(row) * batch.nh + h;
-    for (int dim = threadIdx.x; dim < d; dim += blockDim.x) {
+    const float gate = row_scale != nullptr ? row_scale[o_row] : 1.f;
+    for (int dim = threadIdx.x; dim < dv; dim += blockDim.x) {
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) {
-            o += acc_s[w * d + dim] * w_scale[w];
+            o += acc_s[w * dv + dim] * w_scale[w];
         }
         o *= inv_l;
         if (part != nullptr) {
-            part[o_row * (d + 2) + dim] = o;
+            part[o_row * (dv + 2) + dim] = o;
         } else {
-            out[o_row * d + dim] = from_f32<T>(o);
+            out[int64_t(row) * out_stride + int64_t(h) * dv + dim] = from_f32<T>(o * gate);
         }
     }
     if (part != nullptr && threadIdx.x == 0) {
-        part[o_row * (d + 2) + d] = m_all;
-        part[o_row * (d + 2) + d + 1] = l_all;
+        part[o_row * (dv + 2) + dv] = m_all;
+        part[o_row * (dv + 2) + dv + 1] = l_all;
     }
 }
 
@@ -193,9 +197,11 @@ template <typename T>
 void launch(cudaStream_t s, const KVView &kv, const AttnBatch &batch, const void *q, float scale, const AttnOut &out,
             int32_t *error_flag) {
     const dim3 grid(unsigned(batch.total_q), unsigned(batch.nh));
-    const size_t smem = (size_t(kv.d) * (1 + kWarps) + 2 * kWarps) * sizeof(float);
+    const size_t smem = (size_t(kv.d) + size_t(kv.vDim()) * kWarps + 2 * kWarps) * sizeof(float);
     attention_generic_kernel<T><<<grid, kWarps * 32, smem, s>>>(kv, batch, static_cast<const T *>(q), scale,
-                                                                static_cast<T *>(out.out), out.part, error_flag);
+                                                                static_cast<T *>(out.out), out.part, out.row_scale,
+                                                                out.row_stride ? out.row_stride : int64_t(batch.nh) * kv.vDim(),
+                                                                error_flag);
 }
 
 } // namespace
@@ -205,7 +211,8 @@ void attention_generic(stream_t stream, llaisysDataType_t dtype, const KVView &k
     if (batch.total_q <= 0 || batch.nh <= 0) {
         return;
     }
-    CHECK_ARGUMENT(kv.d > 0 && kv.d <= 32 * kMaxDimsPerLane, "attention: head_dim must be in [1, 256]");
+    CHECK_ARGUMENT(kv.d > 0 && kv.d <= 8192 && kv.vDim() > 0 && kv.vDim() <= 32 * kMaxDimsPerLane,
+                   "attention: V rows must have 1 to 256 elements, K rows at most 8192");
     CHECK_ARGUMENT(kv.nkvh > 0 && batch.nh % kv.nkvh == 0, "attention: nh must be a multiple of nkvh");
     CHECK_ARGUMENT(batch.nh <= 65535, "attention: too many heads for one launch");
     auto s = static_cast<cudaStream_t>(stream);

@@ -82,6 +82,33 @@ void paged_rope_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
                        const void *bias, const int32_t *seq_ids, const int32_t *positions, int32_t n_rows, int32_t nh,
                        float theta, int32_t max_blocks, int32_t *error_flag);
 
+// K1c (see NormAppendArgs); same addressing and flags as K1.
+void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const NormAppendArgs &args,
+                       int32_t max_blocks, int32_t *error_flag);
+
+// Gated linear attention (see GatedLinearArgs). decode: one token per sequence, everything in one launch. chunk: ragged
+// runs of tokens.
+void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args);
+void gated_linear_chunk(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args);
+
+// ---- operators of a residual stream kept in f32 (x float [rows, d]) around dtype activations ----
+// x[r, :] = scale * w[tokens[r], :]; copy (may be null): the same rounded to dtype, row r at copy + r * copy_stride
+void embed_scaled(stream_t stream, llaisysDataType_t dtype, float *x, void *copy, int64_t copy_stride, const int64_t *tokens,
+                  const void *w, float scale, size_t rows, size_t d, size_t vocab);
+// out[r, :] = dtype(x[r, :]), row r at out + r * out_stride
+void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const float *x, size_t rows, size_t d);
+// out[i, :] = rms_norm(x[r, :]) * w with r = row_index[i] (null: r = i), f32 arithmetic, one rounding
+void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
+                     const void *w, float eps, size_t rows, size_t d);
+// out (f32) = alpha * in . W^T (+ out when accumulate): a projection into the stream, or logits
+void linear_f32(stream_t stream, llaisysDataType_t dtype, float *out, const void *in, const void *weight, size_t m, size_t n,
+                size_t k, bool accumulate, float alpha = 1.f);
+// v = max(v, 0)^2 in place
+void relu_squared(stream_t stream, llaisysDataType_t dtype, void *v, size_t n);
+// logits = cap * tanh(logits / cap) in place (cap <= 0: unchanged) and the row-wise argmax of the result, one launch;
+// scratch as argmax_rows_split
+void softcap_argmax(stream_t stream, float *logits, float cap, int64_t *idx_out, size_t rows, size_t n, void *scratch);
+
 // K5: tokens [0, n_tokens) of table row seq_row -> k_out, v_out [n_tokens, nkvh, d].
 void paged_gather(stream_t stream, size_t elem_size, const KVView &kv, int32_t seq_row, int32_t n_tokens,
                   void *k_out, void *v_out, int32_t *error_flag);

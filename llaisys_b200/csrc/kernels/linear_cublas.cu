@@ -68,6 +68,33 @@ cublasHandle_t handle_for_current_device() {
     return h;
 }
 
+cudaDataType cuda_type(llaisysDataType_t dtype) {
+    switch (dtype) {
+    case LLAISYS_DTYPE_F32:
+        return CUDA_R_32F;
+    case LLAISYS_DTYPE_F16:
+        return CUDA_R_16F;
+    case LLAISYS_DTYPE_BF16:
+        return CUDA_R_16BF;
+    default:
+        EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
+    }
+}
+
+// Row-major out[M, N] = alpha in[M, K] . W[N, K]^T + beta out, f32 accumulation (f32 operands in true f32: no TF32 mode is
+// ever set on the handle). Column-major this is out^T[N, M] = W^T(as stored)[K, N]^T . in^T[K, M].
+void gemm(stream_t stream, llaisysDataType_t dtype, llaisysDataType_t out_dtype, void *out, const void *in, const void *weight,
+          size_t m, size_t n, size_t k, float alpha, float beta) {
+    ASSERT(cublas_api().ok, "linear on NVIDIA needs cuBLAS (libcublas.so.12 was not found)");
+    const cudaDataType type = cuda_type(dtype), out_type = cuda_type(out_dtype);
+    cublasHandle_t h = handle_for_current_device();
+    cublasStatus_t st = cublas_api().set_stream(h, static_cast<cudaStream_t>(stream));
+    ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasSetStream failed with status " << int(st));
+    st = cublas_api().gemm_ex(h, CUBLAS_OP_T, CUBLAS_OP_N, int(n), int(m), int(k), &alpha, weight, type, int(k), in, type,
+                              int(k), &beta, out, out_type, int(n), CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
+    ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasGemmEx failed with status " << int(st));
+}
+
 std::atomic<int> g_linear_policy{0};
 
 } // namespace
@@ -100,32 +127,19 @@ void linear(stream_t stream, llaisysDataType_t dtype, void *out, const void *in,
         }
         return;
     }
-    ASSERT(cublas_api().ok, "linear on NVIDIA needs cuBLAS (libcublas.so.12 was not found)");
-    cudaDataType type;
-    switch (dtype) {
-    case LLAISYS_DTYPE_F32:
-        type = CUDA_R_32F;
-        break;
-    case LLAISYS_DTYPE_F16:
-        type = CUDA_R_16F;
-        break;
-    case LLAISYS_DTYPE_BF16:
-        type = CUDA_R_16BF;
-        break;
-    default:
-        EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
-    }
-    cublasHandle_t h = handle_for_current_device();
-    cublasStatus_t st = cublas_api().set_stream(h, static_cast<cudaStream_t>(stream));
-    ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasSetStream failed with status " << int(st));
-    // Row-major out[M, N] = in[M, K] . W[N, K]^T is column-major out^T[N, M] = W^T(as stored)[K, N]^T . in^T[K, M].
-    const float alpha = 1.f, beta = accumulate ? 1.f : 0.f; // accumulate: out += in . W^T, one rounding of the sum
-    st = cublas_api().gemm_ex(h, CUBLAS_OP_T, CUBLAS_OP_N, int(n), int(m), int(k), &alpha, weight, type, int(k), in, type,
-                              int(k), &beta, out, type, int(n), CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
-    ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasGemmEx failed with status " << int(st));
+    // accumulate: out += in . W^T, one rounding of the sum
+    gemm(stream, dtype, dtype, out, in, weight, m, n, k, 1.f, accumulate ? 1.f : 0.f);
     if (bias != nullptr) {
         bias_add(stream, dtype, out, bias, m, n);
     }
+}
+
+void linear_f32(stream_t stream, llaisysDataType_t dtype, float *out, const void *in, const void *weight, size_t m, size_t n,
+                size_t k, bool accumulate, float alpha) {
+    if (m == 0 || n == 0) {
+        return;
+    }
+    gemm(stream, dtype, LLAISYS_DTYPE_F32, out, in, weight, m, n, k, alpha, accumulate ? 1.f : 0.f);
 }
 
 } // namespace llaisys::kernels

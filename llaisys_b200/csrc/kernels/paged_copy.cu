@@ -308,6 +308,111 @@ __global__ void paged_rope_append_kernel(unsigned char *__restrict__ k_pool, uns
     }
 }
 
+// K1c: one warp per (row, head) over the nh query, nkvh key and nkvh value heads of a projection row. Query and key heads
+// are divided by their root mean square and weighted; the warp of a query head also turns that head's gate into the factor
+// the attention kernel applies. f32 arithmetic, one rounding.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+    paged_norm_append_kernel(unsigned char *__restrict__ k_pool, unsigned char *__restrict__ v_pool, NormAppendArgs a,
+                             const int32_t *__restrict__ table, CopyGeom g, int32_t d, int32_t dv, int64_t v_head_stride_b,
+                             int64_t v_token_stride_b, int32_t max_blocks, int32_t *error_flag) {
+    using P = Pack<T, VEC>;
+    asm volatile("griddepcontrol.wait;\n" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    const int32_t heads = a.nh + 2 * g.nkvh;
+    const int64_t item = (int64_t(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
+    const int lane = threadIdx.x & 31;
+    if (item >= int64_t(a.n_rows) * heads) {
+        return;
+    }
+    const int64_t row = item / heads;
+    const int32_t head = int32_t(item - row * heads);
+    const bool is_q = head < a.nh, is_v = head >= a.nh + g.nkvh;
+    const T *proj = static_cast<const T *>(a.proj) + row * a.row_stride;
+    const int32_t kvh = is_v ? head - a.nh - g.nkvh : head - a.nh;
+    const T *src = proj + (is_q ? a.q_at + int64_t(head) * d : (is_v ? a.v_at + int64_t(kvh) * dv : a.k_at + int64_t(kvh) * d));
+    const int32_t n = is_v ? dv : d;
+    const T *w = static_cast<const T *>(is_q ? a.q_norm : a.k_norm);
+    float inv = 1.f;
+    if (is_v) {
+        w = nullptr;
+    } else if (w != nullptr) {
+        float ss = 0.f;
+        for (int32_t i = lane * VEC; i < n; i += 32 * VEC) {
+            const P x = *reinterpret_cast<const P *>(src + i);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                ss = fmaf(to_f32(x.v[e]), to_f32(x.v[e]), ss);
+            }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        }
+        inv = rsqrtf(ss / float(n) + a.eps);
+    }
+    T *dst;
+    if (is_q) {
+        dst = static_cast<T *>(a.q_out) + (row * a.nh + head) * d;
+        if (lane == 0 && a.row_scale != nullptr) {
+            a.row_scale[row * a.nh + head] =
+                a.gate_at < 0 ? a.gate_scale : a.gate_scale / (1.f + expf(-to_f32(proj[a.gate_at + head])));
+        }
+    } else {
+        int32_t page, slot;
+        if (!resolve_slot(table, g, a.seq_ids[row], a.positions[row], max_blocks, error_flag, page, slot)) {
+            return;
+        }
+        const int64_t off = int64_t(page) * g.page_stride_b +
+                            (is_v ? int64_t(kvh) * v_head_stride_b + int64_t(slot) * v_token_stride_b
+                                  : int64_t(kvh) * g.head_stride_b + int64_t(slot) * g.token_stride_b);
+        dst = reinterpret_cast<T *>((is_v ? v_pool : k_pool) + off);
+    }
+    for (int32_t i = lane * VEC; i < n; i += 32 * VEC) {
+        P x = *reinterpret_cast<const P *>(src + i);
+        if (w != nullptr) {
+            const P ww = *reinterpret_cast<const P *>(w + i);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                x.v[e] = from_f32<T>(to_f32(x.v[e]) * inv * to_f32(ww.v[e]));
+            }
+        }
+        *reinterpret_cast<P *>(dst + i) = x;
+    }
+}
+
+template <typename T>
+void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &a, int32_t max_blocks, int32_t *error_flag) {
+    CopyGeom g{};
+    g.page_stride_b = kv.page_stride * int64_t(sizeof(T));
+    g.head_stride_b = kv.head_stride * int64_t(sizeof(T));
+    g.token_stride_b = kv.token_stride * int64_t(sizeof(T));
+    g.nkvh = kv.nkvh;
+    g.page_size = kv.page_size;
+    g.num_pages = kv.num_pages;
+    g.table_stride = kv.table_stride;
+    constexpr int kVec = 4;
+    auto aligned = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const int32_t d = kv.d, dv = kv.vDim();
+    const bool wide = d % kVec == 0 && dv % kVec == 0 && a.row_stride % kVec == 0 && a.q_at % kVec == 0 && a.k_at % kVec == 0 &&
+                      a.v_at % kVec == 0 && aligned(a.proj) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out);
+    const int64_t warps = int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh);
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(unsigned((warps + 7) / 8));
+    cfg.blockDim = dim3(256);
+    cfg.stream = s;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = 1;
+    auto kernel = wide ? paged_norm_append_kernel<T, kVec> : paged_norm_append_kernel<T, 1>;
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, static_cast<unsigned char *>(kv.k_base),
+                                          static_cast<unsigned char *>(kv.v_base), NormAppendArgs(a), kv.block_table, g, d, dv,
+                                          kv.vHeadStride() * int64_t(sizeof(T)), kv.vTokenStride() * int64_t(sizeof(T)),
+                                          max_blocks, error_flag));
+}
+
 template <typename T>
 void launch_rope_append(cudaStream_t s, const KVView &kv, void *q_out, const void *qkv, const void *bias,
                         const int32_t *seq_ids, const int32_t *positions, int32_t n_rows, int32_t nh, float theta,
@@ -451,6 +556,28 @@ void paged_rope_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
         EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
     }
     check_launch("paged_rope_append");
+}
+
+void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const NormAppendArgs &args,
+                       int32_t max_blocks, int32_t *error_flag) {
+    if (args.n_rows == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    switch (dtype) {
+    case LLAISYS_DTYPE_F32:
+        launch_norm_append<float>(s, kv, args, max_blocks, error_flag);
+        break;
+    case LLAISYS_DTYPE_F16:
+        launch_norm_append<__half>(s, kv, args, max_blocks, error_flag);
+        break;
+    case LLAISYS_DTYPE_BF16:
+        launch_norm_append<__nv_bfloat16>(s, kv, args, max_blocks, error_flag);
+        break;
+    default:
+        EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
+    }
+    check_launch("paged_norm_append");
 }
 
 } // namespace llaisys::kernels

@@ -1,0 +1,315 @@
+// Operators of a decoder whose residual stream stays in f32 between layers: the embedding with its scale, the norm that
+// turns stream rows into activations, the cast that feeds the stream to a projection, the squared-relu activation and the
+// soft cap of the logits with the greedy choice behind it. All HBM-bound, one pass over their data.
+#include "device_utils.cuh"
+#include "kernels.hpp"
+#include "mma_utils.cuh"
+
+#include <utility>
+
+namespace llaisys::kernels {
+
+namespace {
+
+template <typename T, int N>
+struct alignas(sizeof(T) * N) Vec {
+    T v[N];
+};
+
+// Programmatic launch: every kernel below waits for its predecessor before it touches anything, then lets its successor be
+// scheduled, so that a launch hides under the kernel before it (see rms_norm_vec_kernel).
+template <typename... KArgs, typename... Args>
+void launch_programmatic(void (*kernel)(KArgs...), dim3 grid, unsigned block, cudaStream_t s, Args &&...args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(block);
+    cfg.stream = s;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = 1;
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, KArgs(std::forward<Args>(args))...));
+}
+
+template <typename T, int VEC>
+__global__ void embed_scaled_kernel(float *__restrict__ x, T *__restrict__ copy, int64_t copy_stride,
+                                    const int64_t *__restrict__ tokens, const T *__restrict__ w, float scale, int32_t d,
+                                    int64_t vocab) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    int64_t tok = tokens[row];
+    tok = tok < 0 || tok >= vocab ? 0 : tok; // validated on the host; never read out of range here
+    const T *src = w + tok * d;
+    for (int32_t i = int32_t(threadIdx.x) * VEC; i < d; i += int32_t(blockDim.x) * VEC) {
+        const Vec<T, VEC> in = *reinterpret_cast<const Vec<T, VEC> *>(src + i);
+        Vec<float, VEC> f;
+        Vec<T, VEC> c;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            f.v[e] = to_f32(in.v[e]) * scale;
+            c.v[e] = from_f32<T>(f.v[e]);
+        }
+        *reinterpret_cast<Vec<float, VEC> *>(x + row * d + i) = f;
+        if (copy != nullptr) {
+            *reinterpret_cast<Vec<T, VEC> *>(copy + row * copy_stride + i) = c;
+        }
+    }
+}
+
+template <typename T, int VEC>
+__global__ void stream_cast_kernel(T *__restrict__ out, int64_t out_stride, const float *__restrict__ x, int32_t d) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    for (int32_t i = int32_t(threadIdx.x) * VEC; i < d; i += int32_t(blockDim.x) * VEC) {
+        const Vec<float, VEC> in = *reinterpret_cast<const Vec<float, VEC> *>(x + row * d + i);
+        Vec<T, VEC> c;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            c.v[e] = from_f32<T>(in.v[e]);
+        }
+        *reinterpret_cast<Vec<T, VEC> *>(out + row * out_stride + i) = c;
+    }
+}
+
+// One CTA per row; the first PER_THREAD pieces of a thread stay in registers between the two passes, what a very long row
+// has beyond them is read again.
+template <typename T, int VEC, int PER_THREAD>
+__global__ void stream_rms_norm_kernel(T *__restrict__ out, const float *__restrict__ x, const int64_t *__restrict__ row_index,
+                                       const T *__restrict__ w, float eps, int32_t d) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    using F = Vec<float, VEC>;
+    const int64_t row = row_index != nullptr ? row_index[blockIdx.x] : int64_t(blockIdx.x);
+    const float *src = x + row * d;
+    const int32_t n_vec = d / VEC;
+    F held[PER_THREAD];
+    float ss = 0.f;
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * int32_t(blockDim.x);
+        if (i < n_vec) {
+            held[r] = *reinterpret_cast<const F *>(src + int64_t(i) * VEC);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                ss = fmaf(held[r].v[e], held[r].v[e], ss);
+            }
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * int32_t(blockDim.x); i < n_vec; i += int32_t(blockDim.x)) {
+        const F f = *reinterpret_cast<const F *>(src + int64_t(i) * VEC);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            ss = fmaf(f.v[e], f.v[e], ss);
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    }
+    __shared__ float s_part[32];
+    if ((threadIdx.x & 31) == 0) {
+        s_part[threadIdx.x >> 5] = ss;
+    }
+    __syncthreads();
+    float tot = 0.f;
+    for (int i = 0; i < int(blockDim.x >> 5); ++i) {
+        tot += s_part[i]; // every thread sums the few partials in the same order
+    }
+    const float inv = rsqrtf(tot / float(d) + eps);
+    T *dst = out + int64_t(blockIdx.x) * d;
+    auto store = [&](int32_t i, const F &f) {
+        const Vec<T, VEC> ww = *reinterpret_cast<const Vec<T, VEC> *>(w + int64_t(i) * VEC);
+        Vec<T, VEC> o;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            o.v[e] = from_f32<T>(f.v[e] * inv * to_f32(ww.v[e]));
+        }
+        *reinterpret_cast<Vec<T, VEC> *>(dst + int64_t(i) * VEC) = o;
+    };
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * int32_t(blockDim.x);
+        if (i < n_vec) {
+            store(i, held[r]);
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * int32_t(blockDim.x); i < n_vec; i += int32_t(blockDim.x)) {
+        store(i, *reinterpret_cast<const F *>(src + int64_t(i) * VEC));
+    }
+}
+
+template <typename T, int VEC>
+__global__ void relu_squared_kernel(T *__restrict__ v, size_t n_vec) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    using P = Vec<T, VEC>;
+    const size_t stride = size_t(gridDim.x) * blockDim.x;
+    for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < n_vec; i += stride) {
+        P p = reinterpret_cast<const P *>(v)[i];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float f = fmaxf(to_f32(p.v[e]), 0.f);
+            p.v[e] = from_f32<T>(f * f);
+        }
+        reinterpret_cast<P *>(v)[i] = p;
+    }
+}
+
+// The split argmax of ops_misc.cu with the soft cap applied on the way: a row's CTAs fold (value, index) into one 64-bit
+// key, the last of them to arrive writes the index and leaves key and counter zero.
+__global__ void softcap_argmax_kernel(float *__restrict__ logits, float cap, int64_t *__restrict__ idx_out, size_t n,
+                                      unsigned long long *__restrict__ keys, unsigned *__restrict__ counters) {
+    const size_t row_i = blockIdx.y;
+    float *row = logits + row_i * n;
+    const size_t chunk = (n + gridDim.x - 1) / gridDim.x;
+    const size_t lo = size_t(blockIdx.x) * chunk, hi = lo + chunk < n ? lo + chunk : n;
+    unsigned long long best = 0;
+    for (size_t i = lo + threadIdx.x; i < hi; i += blockDim.x) {
+        float v = row[i];
+        if (cap > 0.f) {
+            v = cap * tanhf(v / cap);
+            row[i] = v;
+        }
+        if (v == v) { // NaN never wins
+            const unsigned b = __float_as_uint(v);
+            const unsigned ord = (b & 0x80000000u) ? ~b : (b | 0x80000000u);
+            const unsigned long long key =
+                (static_cast<unsigned long long>(ord) << 32) | static_cast<unsigned long long>(0xffffffffu - unsigned(i));
+            best = key > best ? key : best;
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const unsigned long long other = __shfl_xor_sync(0xffffffffu, best, o);
+        best = other > best ? other : best;
+    }
+    __shared__ unsigned long long s_best[32];
+    if ((threadIdx.x & 31) == 0) {
+        s_best[threadIdx.x >> 5] = best;
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        for (int i = 1; i < int(blockDim.x >> 5); ++i) {
+            best = s_best[i] > best ? s_best[i] : best;
+        }
+        atomicMax(keys + row_i, best);
+        __threadfence();
+        if (atomicAdd(counters + row_i, 1u) == gridDim.x - 1) {
+            __threadfence();
+            const unsigned long long win = atomicExch(keys + row_i, 0ull);
+            counters[row_i] = 0u;
+            idx_out[row_i] = win == 0ull ? 0 : int64_t(0xffffffffu - unsigned(win & 0xffffffffull));
+        }
+    }
+}
+
+unsigned block_for(size_t n_vec, size_t per_thread) {
+    const size_t want = (n_vec + per_thread - 1) / per_thread;
+    const size_t block = (want + 31) / 32 * 32;
+    return unsigned(block < 64 ? 64 : (block > 1024 ? 1024 : block));
+}
+bool aligned16(const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
+
+template <typename F>
+void dispatch(llaisysDataType_t dtype, F &&body) {
+    switch (dtype) {
+    case LLAISYS_DTYPE_F32:
+        body(float{});
+        break;
+    case LLAISYS_DTYPE_F16:
+        body(__half{});
+        break;
+    case LLAISYS_DTYPE_BF16:
+        body(__nv_bfloat16{});
+        break;
+    default:
+        EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
+    }
+}
+
+} // namespace
+
+void embed_scaled(stream_t stream, llaisysDataType_t dtype, float *x, void *copy, int64_t copy_stride, const int64_t *tokens,
+                  const void *w, float scale, size_t rows, size_t d, size_t vocab) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        const bool wide = d % 4 == 0 && copy_stride % 4 == 0 && aligned16(x) && aligned16(w) && (copy == nullptr || aligned16(copy));
+        auto kernel = wide ? embed_scaled_kernel<T, 4> : embed_scaled_kernel<T, 1>;
+        launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, x, static_cast<T *>(copy), copy_stride,
+                            tokens, static_cast<const T *>(w), scale, int32_t(d), int64_t(vocab));
+    });
+    check_launch("embed_scaled");
+}
+
+void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const float *x, size_t rows, size_t d) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        const bool wide = d % 4 == 0 && out_stride % 4 == 0 && aligned16(x) && aligned16(out);
+        auto kernel = wide ? stream_cast_kernel<T, 4> : stream_cast_kernel<T, 1>;
+        launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, static_cast<T *>(out), out_stride, x,
+                            int32_t(d));
+    });
+    check_launch("stream_cast");
+}
+
+void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
+                     const void *w, float eps, size_t rows, size_t d) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        const bool wide = d % 4 == 0 && aligned16(x) && aligned16(out) && aligned16(w);
+        auto kernel = wide ? stream_rms_norm_kernel<T, 4, 4> : stream_rms_norm_kernel<T, 1, 4>;
+        launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, static_cast<T *>(out), x, row_index,
+                            static_cast<const T *>(w), eps, int32_t(d));
+    });
+    check_launch("stream_rms_norm");
+}
+
+void relu_squared(stream_t stream, llaisysDataType_t dtype, void *v, size_t n) {
+    if (n == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        constexpr int kVec = 16 / int(sizeof(T));
+        const bool wide = n % kVec == 0 && aligned16(v);
+        const size_t n_vec = wide ? n / kVec : n;
+        const size_t want = (n_vec + 255) / 256, cap = 148 * 16;
+        auto kernel = wide ? relu_squared_kernel<T, kVec> : relu_squared_kernel<T, 1>;
+        launch_programmatic(kernel, dim3(unsigned(want < cap ? want : cap)), 256u, s, static_cast<T *>(v), n_vec);
+    });
+    check_launch("relu_squared");
+}
+
+void softcap_argmax(stream_t stream, float *logits, float cap, int64_t *idx_out, size_t rows, size_t n, void *scratch) {
+    if (rows == 0 || n == 0) {
+        return;
+    }
+    CHECK_ARGUMENT(n < 0xffffffffull && rows <= 65535, "softcap_argmax: rows too many or too long");
+    auto s = static_cast<cudaStream_t>(stream);
+    auto *keys = static_cast<unsigned long long *>(scratch);
+    auto *counters = reinterpret_cast<unsigned *>(keys + rows);
+    size_t splits = (n + 4095) / 4096;
+    const size_t cap_splits = (148 * 8 + rows - 1) / rows;
+    splits = splits > cap_splits ? cap_splits : splits;
+    const dim3 grid{static_cast<unsigned>(splits), static_cast<unsigned>(rows), 1u};
+    softcap_argmax_kernel<<<grid, 256, 0, s>>>(logits, cap, idx_out, n, keys, counters);
+    check_launch("softcap_argmax");
+}
+
+} // namespace llaisys::kernels

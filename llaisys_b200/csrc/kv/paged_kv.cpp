@@ -34,6 +34,8 @@ template <typename... Args>
     } while (0)
 
 constexpr size_t kMaxInt32 = size_t(std::numeric_limits<int32_t>::max());
+// A window no sequence can outgrow is no window.
+int32_t windowOf(const AttnOptions &opt) { return opt.window < kMaxInt32 ? int32_t(opt.window) : 0; }
 constexpr size_t kMaxDecodeSeqs = 1024; // sequences per launch of the TMA decode kernel
 
 } // namespace
@@ -43,17 +45,35 @@ constexpr size_t kMaxDecodeSeqs = 1024; // sequences per launch of the TMA decod
 PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
     KV_REQUIRE(cfg.dtype == LLAISYS_DTYPE_F32 || cfg.dtype == LLAISYS_DTYPE_F16 || cfg.dtype == LLAISYS_DTYPE_BF16,
                LLAISYS_E_INVALID, "paged KV: dtype must be F32, F16 or BF16");
-    KV_REQUIRE(cfg.nlayer > 0 && cfg.num_pages > 0 && cfg.page_size > 0 && cfg.nkvh > 0 && cfg.head_dim > 0 &&
-                   cfg.max_seqs > 0 && cfg.max_pages_per_seq > 0,
+    KV_REQUIRE(cfg.nlayer > 0 && cfg.num_pages > 0 && cfg.page_size > 0 && cfg.max_seqs > 0 && cfg.max_pages_per_seq > 0,
                LLAISYS_E_INVALID, "paged KV: every size must be positive");
     KV_REQUIRE(cfg.num_pages <= kMaxInt32 && cfg.max_seqs <= kMaxInt32 && cfg.max_pages_per_seq <= kMaxInt32 &&
                    cfg.page_size * cfg.max_pages_per_seq <= kMaxInt32,
                LLAISYS_E_INVALID, "paged KV: sizes must fit 32-bit indices");
     _elem = utils::dsize(cfg.dtype);
-    KV_REQUIRE((cfg.head_dim * _elem) % 16 == 0, LLAISYS_E_INVALID,
-               "paged KV: a head row (head_dim * element size) must be a multiple of 16 bytes");
-    _page_elems = 2 * cfg.nkvh * cfg.page_size * cfg.head_dim;
-    _layer_bytes = cfg.num_pages * _page_elems * _elem;
+    const size_t align = 16 / _elem;
+    if (_cfg.layers.empty()) {
+        KV_REQUIRE((cfg.head_dim * _elem) % 16 == 0, LLAISYS_E_INVALID,
+                   "paged KV: a head row (head_dim * element size) must be a multiple of 16 bytes");
+        _cfg.layers.assign(cfg.nlayer, KVLayerShape{cfg.nkvh, cfg.head_dim, cfg.head_dim});
+    }
+    KV_REQUIRE(_cfg.layers.size() == cfg.nlayer, LLAISYS_E_INVALID, "paged KV: one shape per layer");
+    size_t pool_bytes = 0, max_kvh = 0;
+    for (const KVLayerShape &shape : _cfg.layers) {
+        KV_REQUIRE(shape.nkvh > 0 && shape.k_dim > 0 && shape.v_dim > 0, LLAISYS_E_INVALID, "paged KV: every size must be positive");
+        Layer l;
+        l.nkvh = shape.nkvh;
+        l.k_dim = shape.k_dim;
+        l.v_dim = shape.v_dim;
+        l.k_row = (l.k_dim + align - 1) / align * align;
+        l.v_row = (l.v_dim + align - 1) / align * align;
+        l.page_elems = l.nkvh * cfg.page_size * (l.k_row + l.v_row);
+        l.offset = pool_bytes;
+        l.bytes = cfg.num_pages * l.page_elems * _elem;
+        pool_bytes += (l.bytes + 255) / 256 * 256;
+        max_kvh = std::max(max_kvh, l.nkvh);
+        _layers.push_back(l);
+    }
 
     auto &ctx = core::context();
     KV_REQUIRE(cfg.device_type == LLAISYS_DEVICE_CPU || cfg.device_type == LLAISYS_DEVICE_NVIDIA, LLAISYS_E_INVALID,
@@ -64,7 +84,7 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
     ctx.setDevice(cfg.device_type, cfg.device_id);
     auto &rt = ctx.runtime();
 
-    _pool = rt.allocateDeviceStorage(cfg.nlayer * _layer_bytes);
+    _pool = rt.allocateDeviceStorage(pool_bytes);
     _table_dev = rt.allocateDeviceStorage(cfg.max_seqs * cfg.max_pages_per_seq * sizeof(int32_t));
     _error_dev = rt.allocateDeviceStorage(sizeof(int32_t));
     // Pages start zeroed: tokens past a sequence's length are never read as data, but a tile load may touch
@@ -75,22 +95,29 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
         kernels::fill_zero(rt.stream(), _table_dev->memory(), _table_dev->size());
         kernels::fill_zero(rt.stream(), _error_dev->memory(), _error_dev->size());
         rt.synchronize();
-        if (_elem == 2 && cfg.head_dim == 128 && cfg.page_size == 16) {
-            // one row of 128 elements per (layer, page, K|V, kv-head, slot)
-            const uint64_t rows = uint64_t(cfg.nlayer) * cfg.num_pages * 2 * cfg.nkvh * cfg.page_size;
-            _has_tma = kernels::make_kv_tensor_map(_tma_desc, _pool->memory(), rows, uint32_t(cfg.nkvh), cfg.dtype) == 0;
-            _has_tma_tile =
-                kernels::make_kv_tile_tensor_map(_tma_tile_desc, _pool->memory(), rows, uint32_t(cfg.nkvh), cfg.dtype) == 0;
-            // These pools are served by the TMA decode kernel and the tcgen05 chunk kernel and by nothing else: a pool
+        bool any_tma = false;
+        for (Layer &l : _layers) {
+            if (_elem != 2 || l.k_dim != 128 || l.v_dim != 128 || cfg.page_size != 16) {
+                continue;
+            }
+            // one row of 128 elements per (page, K|V, kv-head, slot)
+            const uint64_t rows = uint64_t(cfg.num_pages) * 2 * l.nkvh * cfg.page_size;
+            std::byte *base = _pool->memory() + l.offset;
+            l.has_tma = kernels::make_kv_tensor_map(l.tma_desc, base, rows, uint32_t(l.nkvh), cfg.dtype) == 0 &&
+                        kernels::make_kv_tile_tensor_map(l.tma_tile_desc, base, rows, uint32_t(l.nkvh), cfg.dtype) == 0;
+            // These layers are served by the TMA decode kernel and the tcgen05 chunk kernel and by nothing else: a pool
             // they cannot address is refused here, not quietly handed to a slower kernel later.
-            KV_REQUIRE(_has_tma && _has_tma_tile, LLAISYS_E_DEVICE,
+            KV_REQUIRE(l.has_tma, LLAISYS_E_DEVICE,
                        "paged KV: no TMA tensor map for this pool (cuTensorMapEncodeTiled unavailable, or more than 2^31 "
                        "rows of 128 elements)");
+            any_tma = true;
+        }
+        if (any_tma) {
             // Workspace of both kernels, for the largest call this cache can take (a decode call is cut into launches
             // of at most kMaxDecodeSeqs sequences; the chunk kernel's need does not depend on the batch).
             size_t floats = 0, counters = 0, f2 = 0, c2 = 0;
             const size_t seqs = std::min(cfg.max_seqs, kMaxDecodeSeqs);
-            kernels::attention_decode_split_scratch(int32_t(seqs), int32_t(8 * cfg.nkvh), int32_t(cfg.nkvh), 128,
+            kernels::attention_decode_split_scratch(int32_t(seqs), int32_t(8 * max_kvh), int32_t(max_kvh), 128,
                                                     int32_t(cfg.page_size * cfg.max_pages_per_seq), &floats, &counters);
             kernels::attention_prefill_tc_scratch(&f2, &c2);
             _partials_floats = std::max(floats, f2);
@@ -367,10 +394,10 @@ int32_t PagedKV::seqFork(int32_t parent, size_t n_tokens) {
         const int32_t src = prow[full], dst = takePage();
         _page_ref[dst] = 1;
         crow[cs.n_pages++] = dst;
-        const size_t page_bytes = _page_elems * _elem;
         auto &rt = enter();
-        for (size_t l = 0; l < _cfg.nlayer; ++l) {
-            std::byte *base = _pool->memory() + l * _layer_bytes;
+        for (const Layer &l : _layers) {
+            const size_t page_bytes = l.page_elems * _elem;
+            std::byte *base = _pool->memory() + l.offset;
             if (onDevice()) {
                 rt.api()->memcpy_async(base + size_t(dst) * page_bytes, base + size_t(src) * page_bytes, page_bytes,
                                        LLAISYS_MEMCPY_D2D, rt.stream());
@@ -407,32 +434,45 @@ void PagedKV::checkLayer(size_t layer) const {
     KV_REQUIRE(layer < _cfg.nlayer, LLAISYS_E_INVALID, "paged KV: layer ", layer, " out of range (", _cfg.nlayer, ")");
 }
 
+void PagedKV::requireEqualRows(size_t layer, const char *what) const {
+    KV_REQUIRE(_layers[layer].k_dim == _layers[layer].v_dim && _layers[layer].k_dim == _layers[layer].k_row, LLAISYS_E_UNSUPPORTED,
+               "paged KV ", what, ": this layer's K and V rows differ in length or are padded");
+}
+
+void PagedKV::requirePlain(size_t layer, const AttnOptions &opt) const {
+    requireEqualRows(layer, "attention on the CPU");
+    KV_REQUIRE(opt.window == 0 && opt.row_scale == nullptr && opt.row_stride == 0, LLAISYS_E_UNSUPPORTED,
+               "paged attention: windows and output scales on NVIDIA caches only");
+}
+
 std::byte *PagedKV::poolData(size_t layer) const {
     checkLayer(layer);
-    return _pool->memory() + layer * _layer_bytes;
+    return _pool->memory() + _layers[layer].offset;
 }
 
 kernels::KVView PagedKV::view(size_t layer) const {
+    const Layer &l = _layers[layer];
     kernels::KVView v;
     v.k_base = poolData(layer);
-    v.v_base = poolData(layer) + _cfg.nkvh * _cfg.page_size * _cfg.head_dim * _elem;
-    v.page_stride = int64_t(_page_elems);
-    v.head_stride = int64_t(_cfg.page_size * _cfg.head_dim);
-    v.token_stride = int64_t(_cfg.head_dim);
+    v.v_base = poolData(layer) + l.nkvh * _cfg.page_size * l.k_row * _elem;
+    v.page_stride = int64_t(l.page_elems);
+    v.head_stride = int64_t(_cfg.page_size * l.k_row);
+    v.token_stride = int64_t(l.k_row);
     v.block_table = blockTableData();
     v.table_stride = int32_t(_cfg.max_pages_per_seq);
     v.page_size = int32_t(_cfg.page_size);
     v.num_pages = int32_t(_cfg.num_pages);
-    v.nkvh = int32_t(_cfg.nkvh);
-    v.d = int32_t(_cfg.head_dim);
-    v.overlap_launch = _overlap;
-    if (_has_tma_tile) {
-        v.tma_tile_desc = _tma_tile_desc;
-        v.tma_page0 = int64_t(layer) * int64_t(_cfg.num_pages);
+    v.nkvh = int32_t(l.nkvh);
+    v.d = int32_t(l.k_dim);
+    if (l.v_dim != l.k_dim) {
+        v.v_d = int32_t(l.v_dim);
+        v.v_head_stride = int64_t(_cfg.page_size * l.v_row);
+        v.v_token_stride = int64_t(l.v_row);
     }
-    if (_has_tma) {
-        v.tma_desc = _tma_desc;
-        v.tma_page0 = int64_t(layer) * int64_t(_cfg.num_pages);
+    v.overlap_launch = _overlap;
+    if (l.has_tma) {
+        v.tma_tile_desc = l.tma_tile_desc;
+        v.tma_desc = l.tma_desc;
     }
     return v;
 }
@@ -522,6 +562,7 @@ void PagedKV::appendDev(size_t layer, const void *k_rows, const void *v_rows, co
         return;
     }
     KV_REQUIRE(k_rows && v_rows && seq_ids_dev && positions_dev, LLAISYS_E_INVALID, "paged KV append: null argument");
+    requireEqualRows(layer, "append");
     const kernels::KVView v = view(layer);
     if (!onDevice()) {
         const int err = cpu::paged_append(_elem, v, k_rows, v_rows, seq_ids_dev, positions_dev, int32_t(n_rows),
@@ -543,11 +584,12 @@ void PagedKV::ropeAppendDev(size_t layer, void *q_out, const void *qkv, const vo
                             const int32_t *positions_dev, size_t n_rows, size_t nh, float theta, llaisysStream_t stream) {
     checkLayer(layer);
     KV_REQUIRE(n_rows <= kMaxInt32 && nh > 0 && nh <= 4096, LLAISYS_E_INVALID, "paged KV rope append: bad sizes");
-    KV_REQUIRE(_cfg.head_dim % 2 == 0, LLAISYS_E_INVALID, "paged KV rope append: head_dim must be even");
+    KV_REQUIRE(_layers[layer].k_dim % 2 == 0, LLAISYS_E_INVALID, "paged KV rope append: head_dim must be even");
     if (n_rows == 0) {
         return;
     }
     KV_REQUIRE(q_out && qkv && seq_ids_dev && positions_dev, LLAISYS_E_INVALID, "paged KV rope append: null argument");
+    requireEqualRows(layer, "rope append");
     const kernels::KVView v = view(layer);
     if (!onDevice()) {
         const int err = cpu::paged_rope_append(_cfg.dtype, v, q_out, qkv, bias, seq_ids_dev, positions_dev, int32_t(n_rows),
@@ -566,12 +608,29 @@ void PagedKV::ropeAppendDev(size_t layer, void *q_out, const void *qkv, const vo
 #endif
 }
 
+void PagedKV::normAppendDev(size_t layer, const kernels::NormAppendArgs &args, llaisysStream_t stream) {
+    checkLayer(layer);
+    KV_REQUIRE(args.n_rows <= kMaxInt32 && args.nh > 0 && args.nh <= 4096, LLAISYS_E_INVALID, "paged KV norm append: bad sizes");
+    if (args.n_rows == 0) {
+        return;
+    }
+    KV_REQUIRE(onDevice(), LLAISYS_E_UNSUPPORTED, "paged KV norm append: NVIDIA caches only");
+#ifdef ENABLE_NVIDIA_API
+    enter();
+    kernels::paged_norm_append(stream, _cfg.dtype, view(layer), args, int32_t(_cfg.max_pages_per_seq),
+                               reinterpret_cast<int32_t *>(_error_dev->memory()));
+#else
+    (void)stream;
+    fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
+#endif
+}
+
 void PagedKV::decodeDev(size_t layer, void *out, float *part, const void *q, const int32_t *seq_ids_dev,
                         const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len, size_t nh, float scale,
-                        llaisysStream_t stream) {
+                        llaisysStream_t stream, const AttnOptions &opt) {
     checkLayer(layer);
-    KV_REQUIRE(nh > 0 && nh % _cfg.nkvh == 0, LLAISYS_E_INVALID, "paged attention: nh = ", nh,
-               " is not a multiple of nkvh = ", _cfg.nkvh);
+    KV_REQUIRE(nh > 0 && nh % _layers[layer].nkvh == 0, LLAISYS_E_INVALID, "paged attention: nh = ", nh,
+               " is not a multiple of nkvh = ", _layers[layer].nkvh);
     KV_REQUIRE(n_seqs <= kMaxInt32 && max_kv_len <= _cfg.page_size * _cfg.max_pages_per_seq, LLAISYS_E_INVALID,
                "paged attention: batch or context too large for this cache");
     if (n_seqs == 0) {
@@ -579,16 +638,18 @@ void PagedKV::decodeDev(size_t layer, void *out, float *part, const void *q, con
     }
     KV_REQUIRE((out != nullptr) != (part != nullptr), LLAISYS_E_INVALID, "paged attention: exactly one output");
     KV_REQUIRE(q && seq_ids_dev && kv_lens_dev, LLAISYS_E_INVALID, "paged attention: null argument");
+    KV_REQUIRE(part == nullptr || (opt.row_scale == nullptr && opt.row_stride == 0), LLAISYS_E_INVALID,
+               "paged attention: partial results take neither an output scale nor a row stride");
     launchDecode(layer, out, part, q, nullptr, nullptr, seq_ids_dev, kv_lens_dev, n_seqs, max_kv_len, nh, scale, stream,
-                 _overlap);
+                 _overlap, nullptr, nullptr, nullptr, opt);
 }
 
 void PagedKV::decodeStepDev(size_t layer, void *out, const void *q, const void *k_new, const void *v_new,
                             const int32_t *seq_ids_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len,
                             size_t nh, float scale, llaisysStream_t stream) {
     checkLayer(layer);
-    KV_REQUIRE(nh > 0 && nh % _cfg.nkvh == 0, LLAISYS_E_INVALID, "paged decode step: nh = ", nh,
-               " is not a multiple of nkvh = ", _cfg.nkvh);
+    KV_REQUIRE(nh > 0 && nh % _layers[layer].nkvh == 0, LLAISYS_E_INVALID, "paged decode step: nh = ", nh,
+               " is not a multiple of nkvh = ", _layers[layer].nkvh);
     KV_REQUIRE(n_seqs <= kMaxInt32 && max_kv_len <= _cfg.page_size * _cfg.max_pages_per_seq, LLAISYS_E_INVALID,
                "paged decode step: batch or context too large for this cache");
     if (n_seqs == 0) {
@@ -606,7 +667,7 @@ void PagedKV::decodeStepDev(size_t layer, void *out, const void *q, const void *
         decodeDev(layer, out, nullptr, q, seq_ids_dev, kv_lens_dev, n_seqs, max_kv_len, nh, scale, nullptr);
         return;
     }
-    KV_REQUIRE(fastShape() && nh / _cfg.nkvh <= 8, LLAISYS_E_UNSUPPORTED,
+    KV_REQUIRE(fastShape(layer) && nh / _layers[layer].nkvh <= 8, LLAISYS_E_UNSUPPORTED,
                "paged decode step: the one-launch step needs a 16-bit pool with head_dim 128, 16-token pages and at most 8 "
                "query heads per kv head; use llaisysPagedKVAppendDev + llaisysPagedAttentionDecodeDev");
     launchDecode(layer, out, nullptr, q, k_new, v_new, seq_ids_dev, kv_lens_dev, n_seqs, max_kv_len, nh, scale, stream,
@@ -617,12 +678,12 @@ void PagedKV::decodeSplitDev(size_t layer, const void *q, const int32_t *seq_ids
                              size_t n_seqs, size_t max_kv_len, size_t nh, float scale, const kernels::PeerSink &peers,
                              llaisysStream_t stream) {
     checkLayer(layer);
-    KV_REQUIRE(nh > 0 && nh % _cfg.nkvh == 0, LLAISYS_E_INVALID, "split decode: nh = ", nh, " is not a multiple of nkvh = ",
-               _cfg.nkvh);
+    KV_REQUIRE(nh > 0 && nh % _layers[layer].nkvh == 0, LLAISYS_E_INVALID, "split decode: nh = ", nh, " is not a multiple of nkvh = ",
+               _layers[layer].nkvh);
     KV_REQUIRE(n_seqs >= 1 && n_seqs <= kMaxDecodeSeqs && max_kv_len <= _cfg.page_size * _cfg.max_pages_per_seq,
                LLAISYS_E_INVALID, "split decode: 1 to 1024 sequences per call, context within the cache's tables");
     KV_REQUIRE(q && seq_ids_dev && kv_lens_dev, LLAISYS_E_INVALID, "split decode: null argument");
-    KV_REQUIRE(onDevice() && fastShape() && nh / _cfg.nkvh <= 8, LLAISYS_E_UNSUPPORTED,
+    KV_REQUIRE(onDevice() && fastShape(layer) && nh / _layers[layer].nkvh <= 8, LLAISYS_E_UNSUPPORTED,
                "split decode with the exchange in the kernel needs a 16-bit device pool, head_dim 128, 16-token pages");
     launchDecode(layer, nullptr, nullptr, q, nullptr, nullptr, seq_ids_dev, kv_lens_dev, n_seqs, max_kv_len, nh, scale, stream,
                  _overlap, &peers);
@@ -633,10 +694,10 @@ void PagedKV::decodeSplitDev(size_t layer, const void *q, const int32_t *seq_ids
 void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, const void *k_new, const void *v_new,
                            const int32_t *seq_ids_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len,
                            size_t nh, float scale, llaisysStream_t stream, bool overlap, const kernels::PeerSink *peers,
-                           const int32_t *host_seq_ids, const int32_t *host_kv_lens) {
+                           const int32_t *host_seq_ids, const int32_t *host_kv_lens, const AttnOptions &opt) {
     kernels::KVView v = view(layer);
     v.overlap_launch = overlap;
-    const size_t d = _cfg.head_dim;
+    const size_t d = _layers[layer].k_dim, out_row = opt.row_stride ? opt.row_stride : nh * _layers[layer].v_dim;
     for (size_t at = 0; at < n_seqs; at += kMaxDecodeSeqs) {
         kernels::AttnBatch b;
         b.seq_ids = seq_ids_dev ? seq_ids_dev + at : nullptr;
@@ -649,12 +710,16 @@ void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, 
         b.max_q_len = 1;
         b.max_kv_len = int32_t(max_kv_len);
         b.nh = int32_t(nh);
+        b.window = windowOf(opt);
         kernels::AttnOut o;
-        o.out = out ? static_cast<std::byte *>(out) + at * nh * d * _elem : nullptr;
+        o.out = out ? static_cast<std::byte *>(out) + at * out_row * _elem : nullptr;
+        o.row_scale = opt.row_scale ? opt.row_scale + at * nh : nullptr;
+        o.row_stride = int64_t(opt.row_stride);
         o.part = part ? part + at * nh * (d + 2) : nullptr;
         o.peers = peers;
         const std::byte *q_at = static_cast<const std::byte *>(q) + at * nh * d * _elem;
         if (!onDevice()) {
+            requirePlain(layer, opt);
             const int err = cpu::attention(_cfg.dtype, v, b, q_at, scale, o);
             *reinterpret_cast<int32_t *>(_error_dev->memory()) |= err;
             _last_kernel = LLAISYS_KERNEL_CPU;
@@ -664,7 +729,7 @@ void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, 
 #ifdef ENABLE_NVIDIA_API
         enter();
         if (k_new != nullptr) {
-            const size_t row_bytes = _cfg.nkvh * d * _elem;
+            const size_t row_bytes = _layers[layer].nkvh * d * _elem;
             const char *why = nullptr;
             if (kernels::attention_decode_tma(stream, _cfg.dtype, v, b, q_at, scale, o, scratch(),
                                               static_cast<const std::byte *>(k_new) + at * row_bytes,
@@ -687,10 +752,11 @@ void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, 
 
 void PagedKV::prefillDev(size_t layer, void *out, const void *q, const int32_t *seq_ids_dev,
                          const int32_t *q_starts_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t total_q,
-                         size_t max_q_len, size_t max_kv_len, size_t nh, float scale, llaisysStream_t stream) {
+                         size_t max_q_len, size_t max_kv_len, size_t nh, float scale, llaisysStream_t stream,
+                         const AttnOptions &opt) {
     checkLayer(layer);
-    KV_REQUIRE(nh > 0 && nh % _cfg.nkvh == 0, LLAISYS_E_INVALID, "paged attention: nh = ", nh,
-               " is not a multiple of nkvh = ", _cfg.nkvh);
+    KV_REQUIRE(nh > 0 && nh % _layers[layer].nkvh == 0, LLAISYS_E_INVALID, "paged attention: nh = ", nh,
+               " is not a multiple of nkvh = ", _layers[layer].nkvh);
     KV_REQUIRE(n_seqs <= kMaxInt32 && total_q <= kMaxInt32 && max_kv_len <= _cfg.page_size * _cfg.max_pages_per_seq,
                LLAISYS_E_INVALID, "paged attention: batch or context too large for this cache");
     if (n_seqs == 0 || total_q == 0) {
@@ -708,9 +774,13 @@ void PagedKV::prefillDev(size_t layer, void *out, const void *q, const int32_t *
     b.max_q_len = int32_t(max_q_len);
     b.max_kv_len = int32_t(max_kv_len);
     b.nh = int32_t(nh);
+    b.window = windowOf(opt);
     kernels::AttnOut o;
     o.out = out;
+    o.row_scale = opt.row_scale;
+    o.row_stride = int64_t(opt.row_stride);
     if (!onDevice()) {
+        requirePlain(layer, opt);
         const int err = cpu::attention(_cfg.dtype, v, b, q, scale, o);
         *reinterpret_cast<int32_t *>(_error_dev->memory()) |= err;
         _last_kernel = LLAISYS_KERNEL_CPU;
@@ -760,6 +830,7 @@ void PagedKV::gather(size_t layer, int32_t seq, size_t n_tokens, void *k_out, vo
         return;
     }
     KV_REQUIRE(k_out && v_out, LLAISYS_E_INVALID, "paged KV gather: null output");
+    requireEqualRows(layer, "gather");
     flush();
     const kernels::KVView v = view(layer);
     if (!onDevice()) {
@@ -810,8 +881,8 @@ void PagedKV::decodeStepHost(size_t layer, void *out_host, const void *q_host, c
     }
     KV_REQUIRE(out_host && q_host && k_new_host && v_new_host && seq_ids && kv_lens, LLAISYS_E_INVALID,
                "paged decode step: null argument");
-    KV_REQUIRE(nh > 0 && nh % _cfg.nkvh == 0, LLAISYS_E_INVALID, "paged attention: nh = ", nh,
-               " is not a multiple of nkvh = ", _cfg.nkvh);
+    KV_REQUIRE(nh > 0 && nh % _layers[layer].nkvh == 0, LLAISYS_E_INVALID, "paged attention: nh = ", nh,
+               " is not a multiple of nkvh = ", _layers[layer].nkvh);
     KV_REQUIRE(n_seqs <= _cfg.max_seqs, LLAISYS_E_INVALID, "paged decode step: more rows than the cache has sequences");
     size_t max_kv = 0;
     std::vector<int32_t> &pos = _step_positions;
@@ -840,7 +911,7 @@ void PagedKV::decodeStepHost(size_t layer, void *out_host, const void *q_host, c
         return;
     }
     auto &rt = enter();
-    const size_t q_bytes = n_seqs * nh * _cfg.head_dim * _elem, kv_bytes = n_seqs * _cfg.nkvh * _cfg.head_dim * _elem;
+    const size_t q_bytes = n_seqs * nh * _layers[layer].k_dim * _elem, kv_bytes = n_seqs * _layers[layer].nkvh * _layers[layer].k_dim * _elem;
     const size_t need = 2 * q_bytes + 2 * kv_bytes; // q | out | k | v, each a multiple of 16 bytes
     if (need > _step_cap) {
         _step_cap = need * 2;
@@ -850,7 +921,7 @@ void PagedKV::decodeStepHost(size_t layer, void *out_host, const void *q_host, c
     const auto *api = rt.api();
     llaisysStream_t stream = rt.stream();
 #ifdef ENABLE_NVIDIA_API
-    if (fastShape() && nh / _cfg.nkvh <= 8) {
+    if (fastShape(layer) && nh / _layers[layer].nkvh <= 8) {
         // Two launches and no copy-engine transfer when the caller's buffers are page-locked and mapped (each small
         // copy costs more in set-up than in transfer): a copy kernel brings q to the device -- q is read by every CTA
         // that works on its sequence, so it is not left in host memory -- and the one-launch step reads each new K/V row
@@ -979,7 +1050,7 @@ namespace {
 // call to the generic kernel behind the caller's back.
 bool fast_shape(llaisysDataType_t dtype, const kernels::KVView &view, const kernels::AttnBatch &batch) {
     return (dtype == LLAISYS_DTYPE_BF16 || dtype == LLAISYS_DTYPE_F16) && view.d == 128 && view.page_size == 16 &&
-           view.nkvh > 0 && batch.nh % view.nkvh == 0 && batch.nh / view.nkvh <= 8;
+           view.vDim() == 128 && view.nkvh > 0 && batch.nh % view.nkvh == 0 && batch.nh / view.nkvh <= 8;
 }
 } // namespace
 
@@ -987,7 +1058,7 @@ int run_attention_nvidia(llaisysStream_t stream, llaisysDataType_t dtype, const 
                          const kernels::AttnBatch &batch, const void *q, float scale, const kernels::AttnOut &out,
                          const kernels::AttnScratch &scratch) {
     const bool one_query_each = batch.q_starts == nullptr && batch.const_q_len == 1;
-    const bool fast = fast_shape(dtype, view, batch);
+    const bool fast = fast_shape(dtype, view, batch) && batch.window == 0 && out.row_scale == nullptr && out.row_stride == 0;
     int used = LLAISYS_KERNEL_GENERIC;
     if (fast && one_query_each && view.block_table != nullptr && batch.kv_lens != nullptr) {
         // a page pool: the TMA kernel, or nothing

@@ -23,12 +23,26 @@ struct StatusError : std::runtime_error {
     StatusError(int code_, const std::string &what) : std::runtime_error(what), code(code_) {}
 };
 
+// Geometry of one layer's K/V rows.
+struct KVLayerShape {
+    size_t nkvh = 0, k_dim = 0, v_dim = 0;
+};
+
+// What a layer's attention adds to plain causal attention.
+struct AttnOptions {
+    size_t window = 0;                 // sliding window in tokens, the query's own included; 0 = none
+    const float *row_scale = nullptr;  // device, [rows, nh]: factor on every head's output
+    size_t row_stride = 0;             // elements between output rows; 0 = packed
+};
+
 struct PagedKVConfig {
     llaisysDeviceType_t device_type = LLAISYS_DEVICE_CPU;
     int device_id = 0;
     llaisysDataType_t dtype = LLAISYS_DTYPE_BF16;
     size_t nlayer = 1, num_pages = 0, page_size = 16, nkvh = 0, head_dim = 0;
     size_t max_seqs = 0, max_pages_per_seq = 0;
+    // one entry per layer when layers differ (or V rows are not as long as K rows): nkvh / head_dim above are ignored then
+    std::vector<KVLayerShape> layers;
 };
 
 class PagedKV {
@@ -69,7 +83,7 @@ public:
 
     // ---- device-side views ----
     std::byte *poolData(size_t layer) const;
-    size_t layerBytes() const { return _layer_bytes; }
+    size_t layerBytes() const { return _layers[0].bytes; } // of layer 0; all layers' when they have one shape
     const int32_t *blockTableData() const { return reinterpret_cast<const int32_t *>(_table_dev->memory()); }
     void setLaunchOverlap(bool enable) { _overlap = enable; }
     // LLAISYS_KERNEL_* id of the kernel that served this cache's most recent attention call
@@ -99,7 +113,7 @@ public:
                        const int32_t *positions_dev, size_t n_rows, size_t nh, float theta, llaisysStream_t stream);
     void decodeDev(size_t layer, void *out, float *part, const void *q, const int32_t *seq_ids_dev,
                    const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len, size_t nh, float scale,
-                   llaisysStream_t stream);
+                   llaisysStream_t stream, const AttnOptions &opt = {});
     // One decode step in one launch: row i of k_new / v_new becomes token kv_lens[i] - 1 of sequence i, then attention of
     // q[i] over the kv_lens[i] tokens. Device caches: 16-bit, head_dim 128, page 16 pools only (the TMA decode kernel).
     void decodeStepDev(size_t layer, void *out, const void *q, const void *k_new, const void *v_new,
@@ -107,12 +121,14 @@ public:
                        float scale, llaisysStream_t stream);
     // Partial decode of this cache's slice of a KV-range split, its rows stored by the decode kernel itself into slot
     // `rank` of every rank's exchange buffer and this rank's flag stamped there when the last row is out. TMA pools only.
-    bool canPushPartials(size_t nh) const { return onDevice() && fastShape() && nh % _cfg.nkvh == 0 && nh / _cfg.nkvh <= 8; }
+    bool canPushPartials(size_t nh) const { return onDevice() && fastShape(0) && nh % _cfg.nkvh == 0 && nh / _cfg.nkvh <= 8; }
     void decodeSplitDev(size_t layer, const void *q, const int32_t *seq_ids_dev, const int32_t *kv_lens_dev, size_t n_seqs,
                         size_t max_kv_len, size_t nh, float scale, const kernels::PeerSink &peers, llaisysStream_t stream);
     void prefillDev(size_t layer, void *out, const void *q, const int32_t *seq_ids_dev, const int32_t *q_starts_dev,
                     const int32_t *kv_lens_dev, size_t n_seqs, size_t total_q, size_t max_q_len, size_t max_kv_len,
-                    size_t nh, float scale, llaisysStream_t stream);
+                    size_t nh, float scale, llaisysStream_t stream, const AttnOptions &opt = {});
+    // Per-head RMS norm of q and k, then append: see kernels::paged_norm_append. Device caches only.
+    void normAppendDev(size_t layer, const kernels::NormAppendArgs &args, llaisysStream_t stream);
 
 private:
     struct Seq {
@@ -139,20 +155,34 @@ private:
     const Seq &liveSeq(int32_t seq) const;
     void markDirty(int32_t seq, int32_t lo, int32_t hi);
     void checkLayer(size_t layer) const;
+    void requireEqualRows(size_t layer, const char *what) const; // K and V rows of one length, unpadded
+    void requirePlain(size_t layer, const AttnOptions &opt) const;
     kernels::KVView view(size_t layer) const;
     core::Runtime &enter() const;                   // make the cache's device current on this thread
     int32_t *stage(const int32_t *const *arrays, const size_t *lens, size_t n_arrays); // host arrays -> device
     kernels::AttnScratch scratch() const;
     // 16-bit, head_dim 128, 16-token pages on a device: the shapes the TMA decode and tcgen05 chunk kernels serve
-    bool fastShape() const { return _has_tma; }
+    bool fastShape(size_t layer) const { return _layers[layer].has_tma; }
     void launchDecode(size_t layer, void *out, float *part, const void *q, const void *k_new, const void *v_new,
                       const int32_t *seq_ids_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len, size_t nh,
                       float scale, llaisysStream_t stream, bool overlap, const kernels::PeerSink *peers = nullptr,
-                      const int32_t *host_seq_ids = nullptr, const int32_t *host_kv_lens = nullptr);
+                      const int32_t *host_seq_ids = nullptr, const int32_t *host_kv_lens = nullptr,
+                      const AttnOptions &opt = {});
     bool onDevice() const { return _cfg.device_type != LLAISYS_DEVICE_CPU; }
 
     PagedKVConfig _cfg;
-    size_t _elem = 0, _page_elems = 0, _layer_bytes = 0;
+    size_t _elem = 0;
+    // Geometry of one layer in the pool. Rows are padded to whole 16-byte pieces (k_row, v_row elements).
+    struct Layer {
+        size_t nkvh = 0, k_dim = 0, v_dim = 0, k_row = 0, v_row = 0;
+        size_t page_elems = 0; // K and V of one page
+        size_t offset = 0, bytes = 0; // of the layer's pages in the pool
+        // TMA view of the layer's pages (NVIDIA, 16-bit, K and V rows of 128, page 16 only)
+        alignas(64) unsigned char tma_desc[128] = {};      // decode: box = K and V of a page
+        alignas(64) unsigned char tma_tile_desc[256] = {}; // prefill, two maps: box = one half-tile (K); box = one tile as two halves (V)
+        bool has_tma = false;
+    };
+    std::vector<Layer> _layers;
 
     // block manager
     std::vector<int32_t> _free_pages; // stack; back() is handed out next
@@ -179,10 +209,6 @@ private:
     uint32_t _seen_epoch = 0;
     const void *_host_stage_alias = nullptr; // device-side address of _host_stage (mapped page-locked memory)
 
-    // TMA view of the pool (NVIDIA, 16-bit, head_dim 128, page 16 only); _has_tma is false otherwise
-    alignas(64) unsigned char _tma_desc[128] = {};      // decode: box = K and V of a page
-    alignas(64) unsigned char _tma_tile_desc[256] = {}; // prefill, two maps: box = one half-tile (K); box = one tile as two halves (V)
-    bool _has_tma = false, _has_tma_tile = false;
     bool _overlap = false; // launch append / decode with programmatic stream serialisation
     int _last_kernel = 0;
 };

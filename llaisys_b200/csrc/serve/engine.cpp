@@ -11,12 +11,12 @@ namespace {
 constexpr size_t kPage = 16;
 } // namespace
 
-Engine::Engine(models::Qwen2 &model, const EngineConfig &cfg) : _model_ptr(&model), _cfg(cfg) {
+Engine::Engine(models::Decoder &model, const EngineConfig &cfg) : _model_ptr(&model), _cfg(cfg) {
     if (cfg.max_batch == 0 || cfg.max_tokens_per_step == 0 || cfg.prefill_chunk == 0) {
         fail(LLAISYS_E_INVALID, "engine: limits must be positive");
     }
     if (model.maxTokensPerSeq() == 0) {
-        fail(LLAISYS_E_INVALID, "engine: configure the model's cache first (llaisysQwen2ModelConfigureCache)");
+        fail(LLAISYS_E_INVALID, "engine: configure the model's cache first (llaisysModelConfigureCache)");
     }
     model.addObserver(this);
 }
@@ -40,7 +40,7 @@ void Engine::modelDestroyed() {
     _waiting.clear();
 }
 
-models::Qwen2 &Engine::model() {
+models::Decoder &Engine::model() {
     if (_model_ptr == nullptr) {
         fail(LLAISYS_E_INVALID, "engine: its model has been destroyed");
     }
@@ -59,7 +59,7 @@ int64_t Engine::submit(const int64_t *prompt, size_t n_prompt, size_t max_new_to
         fail(LLAISYS_E_INVALID, "engine: prompt + max_new_tokens exceed the cache's maximum sequence length");
     }
     for (size_t i = 0; i < n_prompt; ++i) {
-        if (prompt[i] < 0 || size_t(prompt[i]) >= model().meta().voc) {
+        if (prompt[i] < 0 || size_t(prompt[i]) >= model().vocab()) {
             fail(LLAISYS_E_INVALID, "engine: token id out of range");
         }
     }
@@ -67,7 +67,7 @@ int64_t Engine::submit(const int64_t *prompt, size_t n_prompt, size_t max_new_to
     r.id = _next_id++;
     r.prompt.assign(prompt, prompt + n_prompt);
     r.max_new = max_new_tokens;
-    r.end_token = end_token < 0 ? model().meta().end_token : end_token;
+    r.end_token = end_token < 0 ? model().endToken() : end_token;
     _waiting.push_back(std::move(r));
     return _waiting.back().id;
 }

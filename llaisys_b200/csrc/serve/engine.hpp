@@ -1,4 +1,4 @@
-// Iteration-level ("continuous") batching over one Qwen2 model and its paged KV cache: requests join a queue at any
+// Iteration-level ("continuous") batching over one model and its cache: requests join a queue at any
 // time; every step() forms one batch out of the running requests -- one token for each request that is decoding, the
 // next chunk of the prompt for each that is still prefilling -- runs it as ONE model step, and hands the unfinished
 // requests back. A request is admitted when the pool can hold its prompt and everything it may generate, so a running
@@ -6,7 +6,7 @@
 // New code: the reference describes this service as future work (README.md:415-424).
 #pragma once
 
-#include "../models/qwen2.hpp"
+#include "../models/decoder.hpp"
 
 #include <deque>
 #include <vector>
@@ -28,7 +28,7 @@ struct Event {
 
 class Engine : private models::ModelObserver {
 public:
-    Engine(models::Qwen2 &model, const EngineConfig &cfg);
+    Engine(models::Decoder &model, const EngineConfig &cfg);
     ~Engine();
     Engine(const Engine &) = delete;
     Engine &operator=(const Engine &) = delete;
@@ -60,9 +60,9 @@ private:
     void admit();
     void finish(size_t running_index);
     void modelDestroyed() override; // the model went first: forget it, every later call fails cleanly
-    models::Qwen2 &model();
+    models::Decoder &model();
 
-    models::Qwen2 *_model_ptr;
+    models::Decoder *_model_ptr;
     EngineConfig _cfg;
     std::deque<Request> _waiting;
     std::vector<Request> _running;

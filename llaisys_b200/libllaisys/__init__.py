@@ -110,6 +110,31 @@ class LlaisysQwen2Weights(Structure):
             "mlp_norm_w", "mlp_gate_w", "mlp_up_w", "mlp_down_w")]
 
 
+class LlaisysWindowAttentionMeta(Structure):
+    """struct LlaisysWindowAttentionMeta (include/llaisys/models/vozozen.h)."""
+    _fields_ = [("heads", c_size_t), ("kv_heads", c_size_t), ("dim", c_size_t), ("vdim", c_size_t), ("window", c_size_t),
+                ("scale", c_float)]
+
+
+class LlaisysGatedLinearMeta(Structure):
+    """struct LlaisysGatedLinearMeta (include/llaisys/models/vozozen.h)."""
+    _fields_ = [("heads", c_size_t), ("dim", c_size_t), ("vdim", c_size_t), ("rank", c_size_t), ("tau", c_float)]
+
+
+class LlaisysVozozenLayerMeta(Structure):
+    """struct LlaisysVozozenLayerMeta (include/llaisys/models/vozozen.h)."""
+    _fields_ = [("left", LlaisysWindowAttentionMeta), ("right", LlaisysGatedLinearMeta), ("left_scale", c_float),
+                ("right_scale", c_float), ("ff", c_size_t)]
+
+
+class LlaisysVozozenMeta(Structure):
+    """struct LlaisysVozozenMeta (include/llaisys/models/vozozen.h)."""
+    _fields_ = [("dtype", llaisysDataType_t), ("nlayer", c_size_t), ("layers", POINTER(LlaisysVozozenLayerMeta)),
+                ("width", c_size_t), ("voc", c_size_t), ("maxseq", c_size_t), ("embed_scale", c_float), ("eps", c_float),
+                ("logit_softcap", c_float), ("loop_start", c_size_t), ("loop_stop", c_size_t), ("loop_times", c_size_t),
+                ("end_token", c_int64)]
+
+
 class LlaisysEngineEvent(Structure):
     """struct LlaisysEngineEvent (include/llaisys/serving.h)."""
     _fields_ = [("request", c_int64), ("token", c_int64), ("finished", c_int32), ("reserved", c_int32)]
@@ -233,6 +258,28 @@ PROTOTYPES: dict[str, tuple] = {
     "llaisysNcclUniqueId": (c_int, [c_void_p]),
     "llaisysQwen2ModelSetAllReduceNccl": (c_int, [_MODEL, c_void_p]),
     "llaisysQwen2ModelSetAllReduceCallback": (c_int, [_MODEL, ALL_REDUCE_FN, c_void_p]),
+    # include/llaisys/models/model.h
+    "llaisysModelDestroy": (None, [_MODEL]),
+    "llaisysModelVocab": (c_size_t, [_MODEL]),
+    "llaisysModelLoadTensor": (c_int, [_MODEL, c_char_p, llaisysDataType_t, POINTER(c_size_t), c_size_t, c_void_p,
+                                       POINTER(c_int)]),
+    "llaisysModelMissingTensors": (c_size_t, [_MODEL, c_char_p, c_size_t]),
+    "llaisysModelConfigureCache": (c_int, [_MODEL, c_size_t, c_size_t, c_size_t]),
+    "llaisysModelSeqAdd": (c_int, [_MODEL, _I32P]),
+    "llaisysModelSeqAddWithPrefix": (c_int, [_MODEL, POINTER(c_int64), c_size_t, _I32P, POINTER(c_size_t)]),
+    "llaisysModelSeqFree": (c_int, [_MODEL, c_int32]),
+    "llaisysModelFreePages": (c_size_t, [_MODEL]),
+    "llaisysModelInfer": (c_int, [_MODEL, POINTER(c_int64), c_size_t, POINTER(c_int64)]),
+    "llaisysModelReset": (c_int, [_MODEL]),
+    "llaisysModelStep": (c_int, [_MODEL, _I32P, _I32P, c_size_t, POINTER(c_int64), POINTER(c_int64)]),
+    "llaisysModelStepRows": (c_int, [_MODEL, _I32P, _I32P, c_size_t, POINTER(c_int64), _I32P, c_size_t, POINTER(c_int64)]),
+    "llaisysModelDecodeLoop": (c_int, [_MODEL, _I32P, c_size_t, POINTER(c_int64), c_size_t, POINTER(c_int64)]),
+    "llaisysModelLastLogits": (c_int, [_MODEL, POINTER(c_float), c_size_t]),
+    "llaisysModelLastLoopMs": (c_double, [_MODEL]),
+    # include/llaisys/models/vozozen.h
+    "llaisysVozozenModelCreate": (_MODEL, [POINTER(LlaisysVozozenMeta), llaisysDeviceType_t, c_int]),
+    "llaisysVozozenModelRecordStream": (c_int, [_MODEL, c_int]),
+    "llaisysVozozenModelLayerStream": (c_int, [_MODEL, POINTER(c_float), c_size_t, POINTER(c_size_t)]),
     # include/llaisys/serving.h
     "llaisysEngineCreate": (c_int, [POINTER(c_void_p), _MODEL, c_size_t, c_size_t, c_size_t]),
     "llaisysEngineDestroy": (None, [c_void_p]),
@@ -276,5 +323,6 @@ LIB_LLAISYS = load_shared_library()
 __all__ = [
     "LIB_LLAISYS", "PROTOTYPES", "LlaisysRuntimeAPI", "llaisysStream_t", "llaisysTensor_t", "llaisysPagedKV_t",
     "llaisysDataType_t", "DataType", "llaisysDeviceType_t", "DeviceType", "llaisysMemcpyKind_t", "MemcpyKind",
-    "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent", "ALL_REDUCE_FN",
+    "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent",
+    "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
 ]

@@ -8,18 +8,14 @@ generate() follows the Hugging Face convention the reference's test compares aga
 from __future__ import annotations
 
 import ctypes
-import itertools
 import json
-from ctypes import c_float, c_int, c_int32, c_int64
+from ctypes import c_int
 from pathlib import Path
-from typing import Mapping, Sequence
-
-import numpy as np
+from typing import Mapping
 
 from ..libllaisys import LIB_LLAISYS, DataType, DeviceType, LlaisysQwen2Meta
 from ..paged_kv import _check
-
-_TORCH_DTYPE_NAMES = {"bfloat16": DataType.BF16, "float16": DataType.F16, "float32": DataType.F32}
+from .base import DTYPE_NAMES, CausalLM
 
 
 def _torch_dtype(dtype: DataType):
@@ -27,7 +23,7 @@ def _torch_dtype(dtype: DataType):
     return {DataType.BF16: torch.bfloat16, DataType.F16: torch.float16, DataType.F32: torch.float32}[dtype]
 
 
-class Qwen2:
+class Qwen2(CausalLM):
     def __init__(self, model_path=None, device: DeviceType = DeviceType.CPU, *, device_id: int = 0,
                  config: Mapping | None = None, state_dict: Mapping | None = None, dtype: DataType | None = None,
                  max_seq_len: int | None = None, tp_group=None):
@@ -40,7 +36,7 @@ class Qwen2:
         if config is None:
             raise ValueError("Qwen2 needs a checkpoint directory or a config")
         if dtype is None:
-            dtype = _TORCH_DTYPE_NAMES.get(str(config.get("torch_dtype", config.get("dtype", "bfloat16"))), DataType.BF16)
+            dtype = DTYPE_NAMES.get(str(config.get("torch_dtype", config.get("dtype", "bfloat16"))), DataType.BF16)
         nh = int(config["num_attention_heads"])
         hs = int(config["hidden_size"])
         eos = config.get("eos_token_id", -1)
@@ -53,6 +49,7 @@ class Qwen2:
             maxseq=int(max_seq_len or config.get("max_position_embeddings", 4096)),
             voc=int(config["vocab_size"]), epsilon=float(config.get("rms_norm_eps", 1e-6)),
             theta=float(config.get("rope_theta", 10000.0)), end_token=int(-1 if eos is None else eos))
+        self.vocab, self.max_seq, self.end_token = int(self.meta.voc), int(self.meta.maxseq), int(self.meta.end_token)
         self.dtype = dtype
         self.device = device
         self.device_id = device_id
@@ -192,114 +189,3 @@ class Qwen2:
         buf = (ctypes.c_size_t * ndim)()
         LIB_LLAISYS.tensorGetShape(handle, buf)
         return tuple(buf)
-
-    def close(self) -> None:
-        if getattr(self, "_model", None):
-            LIB_LLAISYS.llaisysQwen2ModelDestroy(self._model)
-            self._model = None
-
-    def __del__(self):
-        self.close()
-
-    # ---- the reference's call: one prompt in, prompt + completion out ----------------------------------------------------
-
-    def generate(self, inputs: Sequence[int], max_new_tokens: int | None = None, top_k: int = 1, top_p: float = 0.8,
-                 temperature: float = 0.8, seed: int | None = None) -> list[int]:
-        """Greedy when top_k == 1 (the argmax is taken on the device); otherwise temperature / top-k / top-p sampling
-        on the host from the step's logits. Stops after max_new_tokens or at the model's end token (kept in the
-        output, as Hugging Face's generate does)."""
-        inputs = [int(t) for t in inputs]
-        if not inputs:
-            return []
-        if max_new_tokens is None:
-            max_new_tokens = max(0, int(self.meta.maxseq) - len(inputs))
-        _check(LIB_LLAISYS.llaisysQwen2ModelReset(self._model))
-        rng = np.random.default_rng(seed)
-        out = list(inputs)
-        feed = inputs
-        for _ in range(max_new_tokens):
-            arr = (c_int64 * len(feed))(*feed)
-            token = int(LIB_LLAISYS.llaisysQwen2ModelInfer(self._model, arr, len(feed)))
-            if top_k != 1:
-                token = self._sample(self.last_logits()[0], top_k, top_p, temperature, rng)
-            out.append(token)
-            if token == self.meta.end_token:
-                break
-            feed = [token]
-        return out
-
-    @staticmethod
-    def _sample(logits: np.ndarray, top_k: int, top_p: float, temperature: float, rng) -> int:
-        scores = logits.astype(np.float64) / max(float(temperature), 1e-6)
-        order = np.argsort(-scores, kind="stable")
-        if top_k and top_k > 0:
-            order = order[:top_k]
-        probs = np.exp(scores[order] - scores[order[0]])
-        probs /= probs.sum()
-        if 0.0 < top_p < 1.0:
-            keep = int(np.searchsorted(np.cumsum(probs), top_p, side="left")) + 1
-            order, probs = order[:keep], probs[:keep] / probs[:keep].sum()
-        return int(order[rng.choice(len(order), p=probs)])
-
-    # ---- batched sequences ----------------------------------------------------------------------------------------------
-
-    def configure_cache(self, max_seqs: int, max_tokens: int) -> None:
-        _check(LIB_LLAISYS.llaisysQwen2ModelConfigureCache(self._model, max_seqs, max_tokens))
-
-    def add_seq(self) -> int:
-        seq = c_int32(-1)
-        _check(LIB_LLAISYS.llaisysQwen2ModelSeqAdd(self._model, ctypes.byref(seq)))
-        return seq.value
-
-    def add_seq_with_prefix(self, tokens: Sequence[int]) -> tuple[int, int]:
-        """New sequence that reuses cached K/V of earlier sequences starting with the same tokens (whole pages, leaving
-        at least one token to run). -> (sequence id, tokens already covered); feed tokens[covered:] to step()."""
-        arr = np.ascontiguousarray(tokens, dtype=np.int64)
-        seq, matched = c_int32(-1), ctypes.c_size_t(0)
-        _check(LIB_LLAISYS.llaisysQwen2ModelSeqAddWithPrefix(self._model, arr.ctypes.data_as(ctypes.POINTER(c_int64)),
-                                                             arr.size, ctypes.byref(seq), ctypes.byref(matched)))
-        return seq.value, int(matched.value)
-
-    def free_seq(self, seq: int) -> None:
-        _check(LIB_LLAISYS.llaisysQwen2ModelSeqFree(self._model, seq))
-
-    def step(self, seq_ids: Sequence[int], tokens: Sequence[Sequence[int]]) -> list[int]:
-        """Appends tokens[i] to sequence seq_ids[i] (any mix of prefill chunks and single decode tokens) and returns
-        the greedy next token of every sequence."""
-        n = len(seq_ids)
-        if len(tokens) != n:
-            raise ValueError("one token list per sequence")
-        ids = np.ascontiguousarray(seq_ids, dtype=np.int32)
-        # (one pass over the token lists: building an array per sequence and concatenating them cost more than the
-        # library call's own host work in a 64-sequence decode step)
-        counts = np.fromiter(map(len, tokens), dtype=np.int32, count=n)
-        flat = np.fromiter(itertools.chain.from_iterable(tokens), dtype=np.int64, count=int(counts.sum()))
-        nxt = np.zeros(n, dtype=np.int64)
-        _check(LIB_LLAISYS.llaisysQwen2ModelStep(
-            self._model, ids.ctypes.data_as(ctypes.POINTER(c_int32)), counts.ctypes.data_as(ctypes.POINTER(c_int32)), n,
-            flat.ctypes.data_as(ctypes.POINTER(c_int64)), nxt.ctypes.data_as(ctypes.POINTER(c_int64))))
-        return nxt.tolist()
-
-    def decode_loop(self, seq_ids: Sequence[int], first_tokens: Sequence[int], n_steps: int) -> np.ndarray:
-        """n_steps greedy steps with the loop state kept on the device; returns int64 [n_steps, n_seqs]."""
-        n = len(seq_ids)
-        ids = np.ascontiguousarray(seq_ids, dtype=np.int32)
-        first = np.ascontiguousarray(first_tokens, dtype=np.int64)
-        if first.shape != (n,):
-            raise ValueError("one first token per sequence")
-        out = np.zeros((n_steps, n), dtype=np.int64)
-        _check(LIB_LLAISYS.llaisysQwen2ModelDecodeLoop(
-            self._model, ids.ctypes.data_as(ctypes.POINTER(c_int32)), n, first.ctypes.data_as(ctypes.POINTER(c_int64)),
-            n_steps, out.ctypes.data_as(ctypes.POINTER(c_int64))))
-        return out
-
-    def last_logits(self, n_seqs: int = 1) -> np.ndarray:
-        """float32 [n_seqs, voc] logits of the most recent step (n_seqs = that step's sequence count)."""
-        out = np.zeros((n_seqs, int(self.meta.voc)), dtype=np.float32)
-        _check(LIB_LLAISYS.llaisysQwen2ModelLastLogits(self._model, out.ctypes.data_as(ctypes.POINTER(c_float)), out.size))
-        return out
-
-    @property
-    def last_loop_ms(self) -> float:
-        """Device milliseconds per decode step of the last decode_loop()."""
-        return float(LIB_LLAISYS.llaisysQwen2ModelLastLoopMs(self._model))
