@@ -5,12 +5,9 @@
 #include "../models/qwen2.hpp"
 #include "../models/vozozen.hpp"
 
-#include <memory>
-#include <string>
+#include "status.hpp"
 
-namespace llaisys::kernels {
-void set_last_error(const std::string &msg);
-}
+#include <memory>
 
 struct LlaisysModel {
     explicit LlaisysModel(std::unique_ptr<llaisys::models::Decoder> decoder) : impl(std::move(decoder)) {}
@@ -24,24 +21,6 @@ struct LlaisysQwen2Model : LlaisysModel {
 };
 
 namespace llaisys::capi {
-
-// Runs `body`; every failure becomes a status code plus a thread-local message (llaisysGetLastError).
-template <typename F>
-int guarded(F &&body) {
-    try {
-        body();
-        return LLAISYS_OK;
-    } catch (const kv::StatusError &e) {
-        kernels::set_last_error(e.what());
-        return e.code;
-    } catch (const std::invalid_argument &e) {
-        kernels::set_last_error(e.what());
-        return LLAISYS_E_INVALID;
-    } catch (const std::exception &e) {
-        kernels::set_last_error(e.what());
-        return LLAISYS_E_DEVICE;
-    }
-}
 
 inline int null_model() {
     kernels::set_last_error("model: null handle or argument");

@@ -6,17 +6,12 @@
 #include "../core/core.hpp"
 
 #include "../cpu/cpu_kernels.hpp"
-#include "../kv/paged_kv.hpp"
+#include "paged_kv_handle.hpp"
 #ifdef ENABLE_NVIDIA_API
 #include "../kernels/kernels.hpp"
 #endif
 
 #include <string>
-
-struct LlaisysPagedKV {
-    llaisys::kv::PagedKV impl;
-    explicit LlaisysPagedKV(const llaisys::kv::PagedKVConfig &cfg) : impl(cfg) {}
-};
 
 namespace {
 

@@ -147,6 +147,9 @@ struct GatedLinearArgs {
     int64_t out_stride = 0;
     float *raw = nullptr;   // scratch [n_rows, heads * dv]
     float *decay = nullptr; // scratch [n_rows, heads * dk]
+    // scratch for cutting long runs into segments that run in parallel (gated_linear_segment_floats); null: never cut
+    float *segments = nullptr;
+    size_t segment_floats = 0;
 };
 
 using stream_t = void *;

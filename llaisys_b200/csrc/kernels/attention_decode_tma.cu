@@ -31,6 +31,7 @@
 
 #include <cuda.h>
 
+#include <algorithm>
 #include <cstring>
 #include <mutex>
 #include <type_traits>
@@ -85,6 +86,11 @@ struct TmaDecodeParams {
     char *pool_k;                           // K tile of (page 0, kv-head 0) of this layer
     long long page_stride_b, head_stride_b; // bytes between pages / kv-heads
     long long v_offset_b;                   // V tile - K tile of the same (page, kv-head)
+    // windowed instantiation: keys j >= kv_len - window take part (window > 0; as long as the cache's tables = none), output
+    // rows of a sequence lie out_stride elements apart and row r is multiplied by row_scale[r] (null: 1)
+    int32_t window;
+    long long out_stride;
+    const float *row_scale;
     // KV-range split across GPUs (exchange instantiation; out null, part = PeerSink::rows): a pair's finished rows
     // (o, m, l) are written locally like any partial output, and the epilogue warp of the CTA that finished them then
     // stores every value, together with the step number, as one 8-byte word into slot `rank` of EVERY rank's exchange
@@ -164,6 +170,9 @@ __device__ __forceinline__ int seq_kv_len(const int32_t *kv_lens, int max_tokens
     return min(max(kv_lens[s], 0), max_tokens);
 }
 
+// First page of the window of a sequence's newest token (windowed instantiation).
+__device__ __forceinline__ int first_page(const TmaDecodeParams &p, int kv_len) { return max(kv_len - p.window, 0) / kPage; }
+
 __device__ __forceinline__ Segment next_segment(Cursor &c, const int *cum, const TmaDecodeParams &p, const int32_t *kv_lens) {
     Segment sg;
     sg.s = c.s;
@@ -187,6 +196,12 @@ __device__ __forceinline__ Segment next_segment(Cursor &c, const int *cum, const
     return sg;
 }
 
+// Windowed instantiation: a sequence's output row and its heads' factors (heads are then rows of kD within it).
+__device__ __forceinline__ void *win_out(const TmaDecodeParams &p, int s) { return static_cast<char *>(p.out) + s * p.out_stride * 2; }
+__device__ __forceinline__ const float *win_scale(const TmaDecodeParams &p, int s) {
+    return p.row_scale != nullptr ? p.row_scale + (long long)s * p.nh : nullptr;
+}
+
 // Polls a barrier phase; gives up after kWaitLimit polls or when another warp of the CTA already gave up.
 __device__ __forceinline__ bool wait_or_abort(uint32_t bar, uint32_t parity, volatile int *abort_flag) {
     for (uint32_t i = 0; i < kWaitLimit; ++i) {
@@ -207,7 +222,10 @@ __device__ __forceinline__ bool wait_or_abort(uint32_t bar, uint32_t parity, vol
 // kShare: launches with few pairs for their grid, whose pairs can be in many pieces, carry the shared merge (all five
 // warps of the last-arriving CTA); the others do not even contain its code -- this kernel's timing moves by a
 // microsecond with what is compiled around its hot loop.
-template <bool kBf16, bool kXchg, bool kShare>
+// kWin: sliding window, output row stride and output factor per head -- an instantiation of its own for the same reason.
+// The pages below a sequence's window are not part of the line at all: page indices of a segment count from the first
+// page the window reaches.
+template <bool kBf16, bool kXchg, bool kShare, bool kWin>
 __global__ void __launch_bounds__(kThreads, kCtasPerSm)
     paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ InlineIndex ix,
                             TmaDecodeParams p) {
@@ -244,7 +262,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
     // -- page counts and block-table rows of all sequences: ONE round trip to global memory by all threads, then the
     //    prefix sums (warp 0, in place) --------------------------------------------------------------------------
     for (int s = tid; s < p.n_seqs; s += kThreads) {
-        cum[s + 1] = (seq_kv_len(kv_lens, p.max_tokens, s) + kPage - 1) / kPage;
+        const int len = seq_kv_len(kv_lens, p.max_tokens, s);
+        cum[s + 1] = (len + kPage - 1) / kPage - (kWin ? first_page(p, len) : 0);
         rows[s] = seq_ids ? seq_ids[s] : s;
     }
     if (warp == kProducerWarp && lane == 0) {
@@ -309,7 +328,7 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                         p.part[row * (kD + 2) + kD + 1] = 0.f;
                     }
                 } else {
-                    store_out<kBf16>(p.out, row * kD + tid, 0.f);
+                    store_out<kBf16>(p.out, kWin ? s * p.out_stride + (row - (long long)s * p.nh) * kD + tid : row * kD + tid, 0.f);
                 }
             }
         }
@@ -350,7 +369,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
             if (sg.n <= 0) {
                 break; // inconsistent lengths: the consumers flag it
             }
-            const long long tbase = (long long)rows[sg.s] * p.table_stride + sg.j0;
+            const int page0_seg = kWin ? first_page(p, sg.kv_len) + sg.j0 : sg.j0; // the segment's first page in the sequence
+            const long long tbase = (long long)rows[sg.s] * p.table_stride + page0_seg;
             // first page the kernel before this one on the stream may still be writing: the one holding token kv_len - 2
             const int guard_page = (max(sg.kv_len, 2) - 2) / kPage;
             for (int base = 0; base < sg.n && !dead; base += kIssueLanes) {
@@ -361,7 +381,7 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 // page order, so every wait ends. No more lanes than ring slots take part in a round: two lanes
                 // on one slot would wait for consecutive phases of the same barrier, and a parity wait cannot tell
                 // phase k + 1 from phase k - 1.
-                if (!waited && sg.j0 + min(base + kIssueLanes, sg.n) > guard_page) {
+                if (!waited && page0_seg + min(base + kIssueLanes, sg.n) > guard_page) {
                     // these copies reach the sequence's newest rows, which may come from the previous kernel on the
                     // stream (everything before it was there long ago)
                     grid_dependency_wait();
@@ -483,11 +503,21 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                         }
                         __syncwarp();
                     }
-                    warp_merge_finish<kBf16>(stash, kMergeWarps, p.group, lane, p.out, p.part, row0);
+                    if constexpr (kWin) {
+                        warp_merge_finish<kBf16>(stash, kMergeWarps, p.group, lane, win_out(p, sg.s), nullptr,
+                                                 (long long)sg.kvh * p.group, win_scale(p, sg.s));
+                    } else {
+                        warp_merge_finish<kBf16>(stash, kMergeWarps, p.group, lane, p.out, p.part, row0);
+                    }
                   }
                 }
                 if (!shared_merge) {
-                    warp_combine_partials<kBf16>(first, expected, p.group, lane, p.out, p.part, row0);
+                    if constexpr (kWin) {
+                        warp_combine_partials<kBf16>(first, expected, p.group, lane, win_out(p, sg.s), nullptr,
+                                                     (long long)sg.kvh * p.group, win_scale(p, sg.s));
+                    } else {
+                        warp_combine_partials<kBf16>(first, expected, p.group, lane, p.out, p.part, row0);
+                    }
                 }
                 if constexpr (kXchg) {
                     __syncwarp(); // the lanes' stores of the merged rows come before the loads that send them
@@ -557,7 +587,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
         }
         // fused step: index in this segment of the pair's last page, which receives the new row; the warp that will
         // take that page fetches the row (K: lanes 0-15, V: lanes 16-31, 16 bytes each) and the page index now
-        const int new_i = p.k_new != nullptr ? (cum[sg.s + 1] - cum[sg.s]) - 1 - sg.j0 : -1;
+        const int seg_page0 = kWin ? first_page(p, sg.kv_len) + sg.j0 : sg.j0;
+        const int new_i = !kWin && p.k_new != nullptr ? (cum[sg.s + 1] - cum[sg.s]) - 1 - sg.j0 : -1;
         const bool brings_new = new_i >= 0 && new_i < sg.n && new_i % kConsumerWarps == warp;
         const uint32_t my_stage = stage_u32 + warp * kStageBytes;
         if (brings_new) {
@@ -583,7 +614,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 break;
             }
             const uint32_t tile = ring_u32 + slot * kSlotBytes;
-            const int n_valid = min(kPage, sg.kv_len - (sg.j0 + i) * kPage);
+            const int n_valid = min(kPage, sg.kv_len - (seg_page0 + i) * kPage);
+            const int n_before = kWin ? sg.kv_len - p.window - (seg_page0 + i) * kPage : 0; // tokens of the page below the window
             const bool patch = brings_new && i == new_i;
             if (patch) {
                 // the new row: over slot n_valid - 1 of the tile (swizzled like the TMA copy) and into the page itself
@@ -627,7 +659,7 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 mma_16816<kBf16>(sc, a, qf[ks][0], qf[ks][1]);
             }
             // online softmax in the log2 domain; this thread holds tokens g, g + 8 for heads 2*q4, 2*q4 + 1
-            const bool ok_lo = g < n_valid, ok_hi = g + 8 < n_valid;
+            const bool ok_lo = g < n_valid && (!kWin || g >= n_before), ok_hi = g + 8 < n_valid && (!kWin || g + 8 >= n_before);
             const float t0 = ok_lo ? sc[0] * p.scale_log2 : -INFINITY;
             const float t1 = ok_lo ? sc[1] * p.scale_log2 : -INFINITY;
             const float t2 = ok_hi ? sc[2] * p.scale_log2 : -INFINITY;
@@ -742,7 +774,12 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                         p.part[row * (kD + 2) + kD + 1] = l_all;
                     }
                 } else {
-                    store_out<kBf16>(p.out, row * kD + dim, o * inv);
+                    if constexpr (kWin) {
+                        store_out<kBf16>(p.out, sg.s * p.out_stride + (long long)(sg.kvh * p.group + h) * kD + dim,
+                                         o * inv * (p.row_scale != nullptr ? p.row_scale[row] : 1.f));
+                    } else {
+                        store_out<kBf16>(p.out, row * kD + dim, o * inv);
+                    }
                 }
             } else {
                 slot_out[h * kPartStride + dim] = o; // un-normalised, relative to m_all
@@ -809,7 +846,7 @@ size_t smem_bytes(int group, int n_seqs) {
            size_t(2 * n_seqs + 1) * sizeof(int) + 16 + size_t(kConsumerWarps) * kStageBytes;
 }
 
-template <bool kBf16, bool kXchg, bool kShare>
+template <bool kBf16, bool kXchg, bool kShare, bool kWin>
 void launch(cudaStream_t s, const CUtensorMap &tmap, const InlineIndex &ix, const TmaDecodeParams &p, int grid, size_t smem,
             bool overlap) {
     static std::once_flag once[64];
@@ -819,8 +856,8 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const InlineIndex &ix, cons
         int optin = 0;
         LLAISYS_CUDA_CHECK(cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev));
         cudaFuncAttributes attr{};
-        LLAISYS_CUDA_CHECK(cudaFuncGetAttributes(&attr, paged_decode_tma_kernel<kBf16, kXchg, kShare>));
-        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tma_kernel<kBf16, kXchg, kShare>,
+        LLAISYS_CUDA_CHECK(cudaFuncGetAttributes(&attr, paged_decode_tma_kernel<kBf16, kXchg, kShare, kWin>));
+        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tma_kernel<kBf16, kXchg, kShare, kWin>,
                                                 cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                 optin - int(attr.sharedSizeBytes)));
     });
@@ -834,7 +871,7 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const InlineIndex &ix, cons
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = overlap ? 1 : 0;
-    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_decode_tma_kernel<kBf16, kXchg, kShare>, tmap, ix, p));
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_decode_tma_kernel<kBf16, kXchg, kShare, kWin>, tmap, ix, p));
 }
 
 } // namespace
@@ -904,7 +941,14 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
         return -1;
     }
     const int group = batch.nh / kv.nkvh;
-    const int grid = decode_grid_size(batch.n_seqs, kv.nkvh, batch.max_kv_len);
+    const bool windowed = batch.window > 0 || out.row_scale != nullptr || out.row_stride != 0;
+    if (windowed && (out.out == nullptr || out.peers != nullptr || k_new != nullptr)) {
+        reason = "a window or an output scale goes with plain decode into an output tensor only";
+        return -1;
+    }
+    // (a window reaches at most window + page - 1 tokens' worth of pages)
+    const int grid = decode_grid_size(batch.n_seqs, kv.nkvh,
+                                      batch.window > 0 ? std::min(batch.max_kv_len, batch.window + kPage - 1) : batch.max_kv_len);
     const size_t n_pairs = size_t(batch.n_seqs) * kv.nkvh;
     if (scratch.partials == nullptr || scratch.counters == nullptr || scratch.error_flag == nullptr ||
         scratch.partials_floats < (size_t(grid) * (1 + kMergeWarps) + n_pairs) * group * kPartStride ||
@@ -948,6 +992,9 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
     p.page_stride_b = kv.page_stride * 2;
     p.head_stride_b = kv.head_stride * 2;
     p.v_offset_b = static_cast<char *>(kv.v_base) - static_cast<char *>(kv.k_base);
+    p.window = batch.window > 0 ? batch.window : p.max_tokens;
+    p.out_stride = out.row_stride != 0 ? out.row_stride : (long long)batch.nh * kD;
+    p.row_scale = out.row_scale;
     p.xchg = PeerSink{};
     if (out.peers != nullptr) {
         p.xchg = *out.peers;
@@ -966,13 +1013,22 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
     const bool xchg = out.peers != nullptr;
     // pairs can be in kSharedMergeFrom pieces or more only where the grid has that many CTAs per pair
     const bool share = size_t(grid) >= n_pairs * size_t(kSharedMergeFrom - 1);
-    auto go = [&](auto bf, auto xc, auto sh) {
-        launch<decltype(bf)::value, decltype(xc)::value, decltype(sh)::value>(s, tmap, ix, p, grid, smem, kv.overlap_launch);
+    auto go = [&](auto bf, auto xc, auto sh, auto wi) {
+        launch<decltype(bf)::value, decltype(xc)::value, decltype(sh)::value, decltype(wi)::value>(s, tmap, ix, p, grid, smem,
+                                                                                                   kv.overlap_launch);
     };
-    auto pick_share = [&](auto bf, auto xc) {
-        share ? go(bf, xc, std::true_type{}) : go(bf, xc, std::false_type{});
+    auto pick_share = [&](auto bf, auto xc, auto wi) {
+        share ? go(bf, xc, std::true_type{}, wi) : go(bf, xc, std::false_type{}, wi);
     };
-    auto pick_xchg = [&](auto bf) { xchg ? pick_share(bf, std::true_type{}) : pick_share(bf, std::false_type{}); };
+    auto pick_xchg = [&](auto bf) {
+        if (xchg) {
+            pick_share(bf, std::true_type{}, std::false_type{});
+        } else if (windowed) {
+            pick_share(bf, std::false_type{}, std::true_type{});
+        } else {
+            pick_share(bf, std::false_type{}, std::false_type{});
+        }
+    };
     bf16 ? pick_xchg(std::true_type{}) : pick_xchg(std::false_type{});
     check_launch("paged_decode_tma");
     return 0;

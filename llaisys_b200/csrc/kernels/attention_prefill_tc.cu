@@ -127,6 +127,11 @@ struct PrefillParams {
     int32_t *error_flag;
     float *partials;   // [2 * gridDim.x][kPartialFloats]
     int32_t *counters; // [gridDim.x], zero between launches
+    // windowed instantiation: query t sees keys j > t + off - window; rows of out lie out_stride elements apart and head h
+    // of row r is multiplied by row_scale[r * nh + h] (null: 1)
+    int32_t window;
+    long long out_stride;
+    const float *row_scale;
     int32_t out_wide;  // out is 32-byte aligned: rows are stored 32 bytes (a whole sector) per instruction
 };
 
@@ -134,6 +139,7 @@ struct PrefillParams {
 
 struct SeqGeom {
     int q_start, q_len, kv_len, off, n_qb;
+    int window; // 0: none
 };
 
 __device__ __forceinline__ SeqGeom seq_geom(const PrefillParams &p, int a) {
@@ -149,12 +155,20 @@ __device__ __forceinline__ SeqGeom seq_geom(const PrefillParams &p, int a) {
     }
     g.off = g.kv_len - g.q_len; // query t sees keys j <= t + off
     g.n_qb = (g.q_len + kBlockM - 1) / kBlockM;
+    g.window = p.window;
     return g;
 }
 
 // keys any row of row block qb can see, and the 64-key blocks that hold them
 __device__ __forceinline__ int tile_kv_hi(const SeqGeom &g, int qb) { return min(g.kv_len, qb * kBlockM + kBlockM + g.off); }
-__device__ __forceinline__ int tile_blocks(const SeqGeom &g, int qb) { return (tile_kv_hi(g, qb) + kBlockN - 1) / kBlockN; }
+// first 64-key block that any row of the row block sees: 0, or where the window of the block's first row begins (its blocks
+// are counted from there)
+__device__ __forceinline__ int tile_first(const SeqGeom &g, int qb) {
+    return g.window > 0 ? max(qb * kBlockM + g.off - g.window + 1, 0) / kBlockN : 0;
+}
+__device__ __forceinline__ int tile_blocks(const SeqGeom &g, int qb) {
+    return (tile_kv_hi(g, qb) + kBlockN - 1) / kBlockN - tile_first(g, qb);
+}
 
 // units of the line that a sequence takes: per tile its blocks, then kTileCost units that stand for no block
 __device__ __forceinline__ int seq_blocks(const PrefillParams &p, const SeqGeom &g) {
@@ -175,7 +189,8 @@ struct Walker {
 
 struct Fragment {
     int a, qb, h;
-    int b0, b1;     // key blocks [b0, b1) of the tile
+    int b0, b1;     // key blocks [b0, b1) of the tile, counted from `first`
+    int first;      // the tile's first key block (tile_first)
     int tile_nblk;  // blocks of the whole tile
     int tile_begin; // index on the line of the tile's block 0
 };
@@ -211,6 +226,7 @@ __device__ __forceinline__ bool locate(const PrefillParams &p, Walker &w, int &p
         f.h = h;
         f.b0 = b0;
         f.tile_nblk = nb;
+        f.first = tile_first(w.g, qb);
         f.b1 = min(nb, b0 + (piece_end - pos));
         f.tile_begin = pos - b0;
         return true;
@@ -249,7 +265,9 @@ __device__ __forceinline__ void add2(float &s0, float &s1, float a0, float a1) {
         : "f"(a0), "f"(a1));
 }
 
-template <bool kBf16>
+// kWin: sliding window, output row stride and output factor; a separate instantiation, so that the plain kernel's loops
+// carry nothing of it.
+template <bool kBf16, bool kWin>
 __global__ void __launch_bounds__(kThreads, 2)
     paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ CUtensorMap tmap_v,
                             PrefillParams p) {
@@ -280,7 +298,9 @@ __global__ void __launch_bounds__(kThreads, 2)
         for (int a = tid; a < p.n_seqs; a += kThreads) {
             const SeqGeom g = seq_geom(p, a);
             mine += seq_blocks(p, g);
-            mine_max = max(mine_max, g.n_qb > 0 ? tile_blocks(g, g.n_qb - 1) : 0);
+            for (int qb = g.window > 0 ? 0 : g.n_qb - 1; qb >= 0 && qb < g.n_qb; ++qb) { // (without a window the last is longest)
+                mine_max = max(mine_max, tile_blocks(g, qb));
+            }
         }
 #pragma unroll
         for (int d = 16; d > 0; d >>= 1) {
@@ -448,14 +468,14 @@ __global__ void __launch_bounds__(kThreads, 2)
                 }
                 return idx < n_pages ? p.block_table[tbase + idx] : 0;
             };
-            int group = load_group(f.b0), next_group = load_group(f.b0 + 8);
+            int group = load_group(f.first + f.b0), next_group = load_group(f.first + f.b0 + 8);
             for (int i = 0; i < n && alive; ++i) {
                 const int gi = done + i, st = gi & 1;
-                const int first = (f.b0 + i) * kPagesPerBlock;
+                const int first = (f.first + f.b0 + i) * kPagesPerBlock;
                 const int n_pg = min(kPagesPerBlock, n_pages - first);
                 if (i > 0 && (i & 7) == 0) {
                     group = next_group;
-                    next_group = load_group(f.b0 + i + 8);
+                    next_group = load_group(f.first + f.b0 + i + 8);
                 }
                 int page = __shfl_sync(0xffffffffu, group, (i & 7) * kPagesPerBlock + (lane & (kPagesPerBlock - 1)));
                 if (lane < n_pg && !p.contiguous && (page < 0 || page >= p.num_pages)) {
@@ -598,8 +618,9 @@ __global__ void __launch_bounds__(kThreads, 2)
                 }
                 tc_fence_after();
                 const uint32_t tmem_s = tmem_base + lane_base + kColS + buf * kBlockN;
-                const int j0 = (f.b0 + i) * kBlockN;
+                const int j0 = ((kWin ? f.first : 0) + f.b0 + i) * kBlockN;
                 const int n_ok = min(min(last_visible, g.kv_len - 1) - j0 + 1, kBlockN); // visible columns are [0, n_ok)
+                const int n_lo = kWin ? last_visible - p.window + 1 - j0 : 0; // columns below n_lo lie before the row's window
                 uint32_t sr[kBlockN / 32][32];
 #pragma unroll
                 for (int c = 0; c < kBlockN / 32; ++c) {
@@ -610,12 +631,12 @@ __global__ void __launch_bounds__(kThreads, 2)
                 // Otherwise the hidden scores become -inf and take the same path: 2^(-inf * scale - m) = 0. (A scale
                 // that is not positive takes the slow path further down.)
                 const bool plain = p.scale_log2 > 0.f;
-                if (plain && !__all_sync(0xffffffffu, n_ok >= kBlockN)) {
+                if (plain && !__all_sync(0xffffffffu, n_ok >= kBlockN && (!kWin || n_lo <= 0))) {
 #pragma unroll
                     for (int c = 0; c < kBlockN / 32; ++c) {
 #pragma unroll
                         for (int k = 0; k < 32; ++k) {
-                            sr[c][k] = c * 32 + k < n_ok ? sr[c][k] : 0xff800000u;
+                            sr[c][k] = c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo) ? sr[c][k] : 0xff800000u;
                         }
                     }
                 }
@@ -639,7 +660,7 @@ __global__ void __launch_bounds__(kThreads, 2)
                     for (int c = 0; c < kBlockN / 32; ++c) {
 #pragma unroll
                         for (int k = 0; k < 32; ++k) {
-                            if (c * 32 + k < n_ok) {
+                            if (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo)) {
                                 mx8[k & 7] = fmaxf(mx8[k & 7], __uint_as_float(sr[c][k]) * p.scale_log2);
                             }
                         }
@@ -687,8 +708,8 @@ __global__ void __launch_bounds__(kThreads, 2)
 #pragma unroll
                         for (int k = 0; k < 32; k += 2) {
                             const float p0 =
-                                (c * 32 + k < n_ok) ? fast_exp2(fmaf(__uint_as_float(sr[c][k]), p.scale_log2, neg_m)) : 0.f;
-                            const float p1 = (c * 32 + k + 1 < n_ok)
+                                (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo)) ? fast_exp2(fmaf(__uint_as_float(sr[c][k]), p.scale_log2, neg_m)) : 0.f;
+                            const float p1 = (c * 32 + k + 1 < n_ok && (!kWin || c * 32 + k + 1 >= n_lo))
                                                  ? fast_exp2(fmaf(__uint_as_float(sr[c][k + 1]), p.scale_log2, neg_m))
                                                  : 0.f;
                             l0 += p0;
@@ -751,7 +772,8 @@ __global__ void __launch_bounds__(kThreads, 2)
             }
             tc_fence_after();
             const bool whole = f.b0 == 0 && f.b1 == f.tile_nblk;
-            char *out_row = static_cast<char *>(p.out) + ((long long)(g.q_start + t) * p.nh + f.h) * (kD * 2);
+            char *out_row = static_cast<char *>(p.out) + (kWin ? (long long)(g.q_start + t) * p.out_stride * 2 + f.h * (kD * 2)
+                                                               : ((long long)(g.q_start + t) * p.nh + f.h) * (kD * 2));
             bool store_rows = whole, staged = false;
             float w_own = 1.f, l_all = l, m_all = m_used;
             float w_oth[4] = {0.f, 0.f, 0.f, 0.f}; // staged merge: weights of the other fragments, in the order of their CTAs
@@ -879,7 +901,10 @@ __global__ void __launch_bounds__(kThreads, 2)
                 }
             }
             if (store_rows && (staged || !dead)) {
-                const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+                float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+                if (kWin && p.row_scale != nullptr && t < g.q_len) {
+                    inv *= p.row_scale[(long long)(g.q_start + t) * p.nh + f.h];
+                }
 #pragma unroll
                 for (int c4 = 0; c4 < 4; ++c4) {
                     if (staged && c4 > 0 && c4 % chunks_per_trip == 0) {
@@ -1060,13 +1085,13 @@ int prefill_slots() {
     return n;
 }
 
-template <bool kBf16>
+template <bool kBf16, bool kWin>
 void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, const PrefillParams &p, int grid, bool overlap) {
     static std::once_flag once[64];
     int dev = 0;
     LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
     std::call_once(once[dev & 63], [] {
-        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_prefill_tc_kernel<kBf16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_prefill_tc_kernel<kBf16, kWin>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                 int(kSmemBytes)));
     });
     cudaLaunchConfig_t cfg{};
@@ -1079,7 +1104,7 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, 
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = overlap ? 1 : 0;
-    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_prefill_tc_kernel<kBf16>, tmap, tmap_v, p));
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_prefill_tc_kernel<kBf16, kWin>, tmap, tmap_v, p));
 }
 
 } // namespace
@@ -1220,7 +1245,14 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
         reinterpret_cast<uintptr_t>(scratch.partials) % 16 != 0) {
         return -1;
     }
-    p.out_wide = reinterpret_cast<uintptr_t>(out.out) % 32 == 0 ? 1 : 0;
+    const bool windowed = batch.window > 0 || out.row_scale != nullptr || out.row_stride != 0;
+    if ((windowed && !paged) || out.row_stride % 8 != 0) {
+        return -1;
+    }
+    p.window = windowed && batch.window <= 0 ? kv.table_stride * kPage : batch.window; // (a factor alone: a window nothing outgrows)
+    p.out_stride = out.row_stride != 0 ? out.row_stride : (long long)batch.nh * kD;
+    p.row_scale = out.row_scale;
+    p.out_wide = reinterpret_cast<uintptr_t>(out.out) % 32 == 0 && p.out_stride % 16 == 0 ? 1 : 0;
     p.partials = scratch.partials;
     p.counters = scratch.counters;
     CUtensorMap tmap, tmap_v;
@@ -1232,10 +1264,12 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
         return -1;
     }
     auto s = static_cast<cudaStream_t>(stream);
-    if (bf16) {
-        launch<true>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
+    if (windowed) {
+        bf16 ? launch<true, true>(s, tmap, tmap_v, p, grid, kv.overlap_launch)
+             : launch<false, true>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
     } else {
-        launch<false>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
+        bf16 ? launch<true, false>(s, tmap, tmap_v, p, grid, kv.overlap_launch)
+             : launch<false, false>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
     }
     check_launch("paged_prefill_tc");
     return 0;

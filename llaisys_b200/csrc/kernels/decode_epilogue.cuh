@@ -192,16 +192,16 @@ __device__ __forceinline__ void warp_merge_parts(MergeState<kHeads> &st, const f
 }
 
 // Normalises a finished merge and stores it: rows of the K/V dtype into `out`, or (part != nullptr) rows of d + 2
-// floats (o, m in natural-log units, l).
+// floats (o, m in natural-log units, l). scale (null: none): a factor per output row of `out`.
 template <bool kBf16, int kHeads>
 __device__ __forceinline__ void warp_merge_store(const MergeState<kHeads> &st, int group, int lane, void *out, float *part,
-                                                 long long out_row0) {
+                                                 long long out_row0, const float *scale = nullptr) {
     constexpr int kD = 128, kOutStride = kD + 2;
 #pragma unroll
     for (int h = 0; h < kHeads; ++h) {
         if (h < group) {
             const long long row = out_row0 + h;
-            const float inv = st.l[h] > 0.f ? 1.f / st.l[h] : 0.f;
+            const float inv = (st.l[h] > 0.f ? 1.f / st.l[h] : 0.f) * (scale != nullptr ? scale[row] : 1.f);
             const float r[4] = {st.o[h].x * inv, st.o[h].y * inv, st.o[h].z * inv, st.o[h].w * inv};
             if (part != nullptr) {
 #pragma unroll
@@ -241,23 +241,23 @@ __device__ __forceinline__ void warp_merge_stash(const MergeState<kHeads> &st, i
 
 template <bool kBf16, int kHeads, int kParts>
 __device__ __forceinline__ void warp_combine_impl(const float *first, int expected, int group, int lane, void *out,
-                                                  float *part, long long out_row0) {
+                                                  float *part, long long out_row0, const float *scale) {
     MergeState<kHeads> st;
     st.clear();
     warp_merge_parts<kHeads, kParts, false>(st, first, expected, 0, 1, group, lane);
     __syncwarp(); // every lane has consumed its loads: `part` may lie over the partials just read
-    warp_merge_store<kBf16, kHeads>(st, group, lane, out, part, out_row0);
+    warp_merge_store<kBf16, kHeads>(st, group, lane, out, part, out_row0, scale);
 }
 
 template <bool kBf16>
 __device__ __forceinline__ void warp_combine_partials(const float *first, int expected, int group, int lane, void *out,
-                                                      float *part, long long out_row0) {
+                                                      float *part, long long out_row0, const float *scale = nullptr) {
     if (group <= 4) {
-        warp_combine_impl<kBf16, 4, 4>(first, expected, group, lane, out, part, out_row0);
+        warp_combine_impl<kBf16, 4, 4>(first, expected, group, lane, out, part, out_row0, scale);
     } else if (group <= 6) {
-        warp_combine_impl<kBf16, 6, 4>(first, expected, group, lane, out, part, out_row0);
+        warp_combine_impl<kBf16, 6, 4>(first, expected, group, lane, out, part, out_row0, scale);
     } else {
-        warp_combine_impl<kBf16, 8, 2>(first, expected, group, lane, out, part, out_row0);
+        warp_combine_impl<kBf16, 8, 2>(first, expected, group, lane, out, part, out_row0, scale);
     }
 }
 
@@ -291,22 +291,22 @@ __device__ __forceinline__ void warp_merge_share(const float *first, int expecte
 
 template <bool kBf16>
 __device__ __forceinline__ void warp_merge_finish(const float *stash, int n_warps, int group, int lane, void *out, float *part,
-                                                  long long out_row0) {
+                                                  long long out_row0, const float *scale = nullptr) {
     if (group <= 4) {
         MergeState<4> st;
         st.clear();
         warp_merge_parts<4, 4, false>(st, stash, n_warps, 0, 1, group, lane);
-        warp_merge_store<kBf16, 4>(st, group, lane, out, part, out_row0);
+        warp_merge_store<kBf16, 4>(st, group, lane, out, part, out_row0, scale);
     } else if (group <= 6) {
         MergeState<6> st;
         st.clear();
         warp_merge_parts<6, 4, false>(st, stash, n_warps, 0, 1, group, lane);
-        warp_merge_store<kBf16, 6>(st, group, lane, out, part, out_row0);
+        warp_merge_store<kBf16, 6>(st, group, lane, out, part, out_row0, scale);
     } else {
         MergeState<8> st;
         st.clear();
         warp_merge_parts<8, 2, false>(st, stash, n_warps, 0, 1, group, lane);
-        warp_merge_store<kBf16, 8>(st, group, lane, out, part, out_row0);
+        warp_merge_store<kBf16, 8>(st, group, lane, out, part, out_row0, scale);
     }
 }
 

@@ -332,4 +332,6 @@ void gated_linear_chunk(stream_t stream, llaisysDataType_t dtype, const GatedLin
     check_launch("gated_linear_chunk");
 }
 
+size_t gated_linear_segment_floats(llaisysDataType_t, size_t, size_t, size_t, size_t, size_t) { return 0; }
+
 } // namespace llaisys::kernels

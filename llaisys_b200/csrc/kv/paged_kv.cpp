@@ -34,8 +34,10 @@ template <typename... Args>
     } while (0)
 
 constexpr size_t kMaxInt32 = size_t(std::numeric_limits<int32_t>::max());
-// A window no sequence can outgrow is no window.
-int32_t windowOf(const AttnOptions &opt) { return opt.window < kMaxInt32 ? int32_t(opt.window) : 0; }
+// A window longer than any sequence of the cache is cut to what a sequence can hold.
+int32_t windowOf(const PagedKVConfig &cfg, const AttnOptions &opt) {
+    return int32_t(std::min(opt.window, cfg.page_size * cfg.max_pages_per_seq));
+}
 constexpr size_t kMaxDecodeSeqs = 1024; // sequences per launch of the TMA decode kernel
 
 } // namespace
@@ -710,7 +712,7 @@ void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, 
         b.max_q_len = 1;
         b.max_kv_len = int32_t(max_kv_len);
         b.nh = int32_t(nh);
-        b.window = windowOf(opt);
+        b.window = windowOf(_cfg, opt);
         kernels::AttnOut o;
         o.out = out ? static_cast<std::byte *>(out) + at * out_row * _elem : nullptr;
         o.row_scale = opt.row_scale ? opt.row_scale + at * nh : nullptr;
@@ -774,7 +776,7 @@ void PagedKV::prefillDev(size_t layer, void *out, const void *q, const int32_t *
     b.max_q_len = int32_t(max_q_len);
     b.max_kv_len = int32_t(max_kv_len);
     b.nh = int32_t(nh);
-    b.window = windowOf(opt);
+    b.window = windowOf(_cfg, opt);
     kernels::AttnOut o;
     o.out = out;
     o.row_scale = opt.row_scale;
@@ -1058,7 +1060,7 @@ int run_attention_nvidia(llaisysStream_t stream, llaisysDataType_t dtype, const 
                          const kernels::AttnBatch &batch, const void *q, float scale, const kernels::AttnOut &out,
                          const kernels::AttnScratch &scratch) {
     const bool one_query_each = batch.q_starts == nullptr && batch.const_q_len == 1;
-    const bool fast = fast_shape(dtype, view, batch) && batch.window == 0 && out.row_scale == nullptr && out.row_stride == 0;
+    const bool fast = fast_shape(dtype, view, batch);
     int used = LLAISYS_KERNEL_GENERIC;
     if (fast && one_query_each && view.block_table != nullptr && batch.kv_lens != nullptr) {
         // a page pool: the TMA kernel, or nothing

@@ -135,6 +135,26 @@ class LlaisysVozozenMeta(Structure):
                 ("end_token", c_int64)]
 
 
+class LlaisysNormAppend(Structure):
+    """struct LlaisysNormAppend (include/llaisys/mixers.h)."""
+    _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("k_at", c_int64), ("v_at", c_int64),
+                ("gate_at", c_int64), ("q_norm", c_void_p), ("k_norm", c_void_p), ("eps", c_float), ("gate_scale", c_float),
+                ("q_out", c_void_p), ("row_scale", c_void_p), ("seq_ids_dev", c_void_p), ("positions_dev", c_void_p),
+                ("n_rows", c_size_t), ("nh", c_size_t)]
+
+
+class LlaisysGatedLinear(Structure):
+    """struct LlaisysGatedLinear (include/llaisys/mixers.h)."""
+    _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("k_at", c_int64), ("v_at", c_int64),
+                ("g_at", c_int64), ("z_at", c_int64), ("decay_w", c_void_p), ("decay_b", c_void_p), ("norm_w", c_void_p),
+                ("tau", c_float), ("q_scale", c_float), ("eps", c_float), ("out_scale", c_float), ("heads", c_size_t),
+                ("dk", c_size_t), ("dv", c_size_t), ("rank", c_size_t), ("state", c_void_p), ("slot_stride", c_int64),
+                ("seq_ids_dev", c_void_p), ("q_starts_dev", c_void_p), ("kv_lens_dev", c_void_p), ("n_seqs", c_size_t),
+                ("n_rows", c_size_t), ("max_q_len", c_size_t), ("out", c_void_p), ("out_stride", c_int64),
+                ("scratch_raw", c_void_p), ("scratch_decay", c_void_p), ("scratch_segments", c_void_p),
+                ("scratch_segment_floats", c_size_t)]
+
+
 class LlaisysEngineEvent(Structure):
     """struct LlaisysEngineEvent (include/llaisys/serving.h)."""
     _fields_ = [("request", c_int64), ("token", c_int64), ("finished", c_int32), ("reserved", c_int32)]
@@ -258,6 +278,17 @@ PROTOTYPES: dict[str, tuple] = {
     "llaisysNcclUniqueId": (c_int, [c_void_p]),
     "llaisysQwen2ModelSetAllReduceNccl": (c_int, [_MODEL, c_void_p]),
     "llaisysQwen2ModelSetAllReduceCallback": (c_int, [_MODEL, ALL_REDUCE_FN, c_void_p]),
+    # include/llaisys/mixers.h
+    "llaisysPagedKVCreateLayers": (c_int, [POINTER(_KV), llaisysDeviceType_t, c_int, llaisysDataType_t, c_size_t,
+                                           POINTER(c_size_t), POINTER(c_size_t), POINTER(c_size_t), c_size_t, c_size_t,
+                                           c_size_t, c_size_t]),
+    "llaisysPagedKVNormAppendDev": (c_int, [_KV, c_size_t, POINTER(LlaisysNormAppend), llaisysStream_t]),
+    "llaisysPagedAttentionOptDev": (c_int, [_KV, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t,
+                                            c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, c_void_p, c_size_t,
+                                            llaisysStream_t]),
+    "llaisysGatedLinearDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysGatedLinear), c_int,
+                                      llaisysStream_t]),
+    "llaisysGatedLinearSegmentFloats": (c_size_t, [llaisysDataType_t, c_size_t, c_size_t, c_size_t, c_size_t, c_size_t]),
     # include/llaisys/models/model.h
     "llaisysModelDestroy": (None, [_MODEL]),
     "llaisysModelVocab": (c_size_t, [_MODEL]),
@@ -324,5 +355,5 @@ __all__ = [
     "LIB_LLAISYS", "PROTOTYPES", "LlaisysRuntimeAPI", "llaisysStream_t", "llaisysTensor_t", "llaisysPagedKV_t",
     "llaisysDataType_t", "DataType", "llaisysDeviceType_t", "DeviceType", "llaisysMemcpyKind_t", "MemcpyKind",
     "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent",
-    "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
+    "LlaisysNormAppend", "LlaisysGatedLinear", "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
 ]

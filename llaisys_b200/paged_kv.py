@@ -14,7 +14,8 @@ from typing import Sequence
 
 import numpy as np
 
-from .libllaisys import LIB_LLAISYS, DataType, DeviceType, Status, llaisysPagedKV_t
+from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysGatedLinear, LlaisysNormAppend, Status,
+                         llaisysPagedKV_t)
 from .runtime import _addr
 
 _I32P = ctypes.POINTER(c_int32)
@@ -259,6 +260,54 @@ class PagedKVCache:
         _check(LIB_LLAISYS.llaisysPagedAttentionPrefillDev(self._kv, layer, _addr(out), _addr(q), _addr(seq_ids_dev),
                                                            _addr(q_starts_dev), _addr(kv_lens_dev), n_seqs, total_q,
                                                            max_q_len, max_kv_len, nh, scale, stream))
+
+
+    # ---- windows, output factors, layers of their own shape (include/llaisys/mixers.h) ----
+    @classmethod
+    def with_layers(cls, num_pages: int, layers: Sequence[tuple[int, int, int]], *, page_size: int = 16,
+                    dtype: DataType = DataType.BF16, device: DeviceType = DeviceType.NVIDIA, device_id: int = 0,
+                    max_seqs: int = 64, max_pages_per_seq: int | None = None) -> "PagedKVCache":
+        """Cache with one (nkvh, k_dim, v_dim) per layer."""
+        self = cls.__new__(cls)
+        self._kv = None
+        self.max_pages_per_seq = max_pages_per_seq or num_pages
+        handle = llaisysPagedKV_t()
+        cols = [(ctypes.c_size_t * len(layers))(*[layer[i] for layer in layers]) for i in range(3)]
+        _check(LIB_LLAISYS.llaisysPagedKVCreateLayers(byref(handle), int(device), device_id, int(dtype), len(layers), *cols,
+                                                      num_pages, page_size, max_seqs, self.max_pages_per_seq))
+        self._kv = handle
+        return self
+
+    def norm_append_dev(self, layer: int, stream, **fields) -> None:
+        """Per-head norm of q and k, append of k and v, gates to factors; fields of LlaisysNormAppend (buffers may be
+        tensors)."""
+        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev"}
+        args = LlaisysNormAppend(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+        _check(LIB_LLAISYS.llaisysPagedKVNormAppendDev(self._kv, layer, byref(args), stream))
+
+    def attention_dev(self, layer: int, out, q, seq_ids_dev, q_starts_dev, kv_lens_dev, *, n_seqs: int, total_q: int,
+                      max_q_len: int, max_kv_len: int, nh: int, scale: float, stream, window: int = 0, row_scale=None,
+                      row_stride: int = 0) -> None:
+        """Decode (q_starts_dev None) or ragged chunks, with a sliding window, a factor per (row, head) and an output row
+        stride."""
+        _check(LIB_LLAISYS.llaisysPagedAttentionOptDev(
+            self._kv, layer, _addr(out), _addr(q), _addr(seq_ids_dev), None if q_starts_dev is None else _addr(q_starts_dev),
+            _addr(kv_lens_dev), n_seqs, total_q, max_q_len, max_kv_len, nh, scale, window,
+            None if row_scale is None else _addr(row_scale), row_stride, stream))
+
+
+def gated_linear_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
+    """Gated linear attention on device buffers; fields of LlaisysGatedLinear (include/llaisys/mixers.h), buffers may be
+    tensors."""
+    pointers = {"proj", "decay_w", "decay_b", "norm_w", "state", "seq_ids_dev", "q_starts_dev", "kv_lens_dev", "out",
+                "scratch_raw", "scratch_decay", "scratch_segments"}
+    args = LlaisysGatedLinear(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+    _check(LIB_LLAISYS.llaisysGatedLinearDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
+
+
+def gated_linear_segment_floats(dtype: DataType, heads: int, dk: int, dv: int, n_seqs: int, max_q_len: int) -> int:
+    """Size of scratch_segments for a chunk call of these sizes."""
+    return int(LIB_LLAISYS.llaisysGatedLinearSegmentFloats(int(dtype), heads, dk, dv, n_seqs, max_q_len))
 
 
 def lse_merge(out, parts, n_parts: int, n_rows: int, head_dim: int, *, dtype: DataType,

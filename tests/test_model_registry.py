@@ -1,0 +1,201 @@
+"""Host side of the model package: the class a config selects, configurations and their weights, the safetensors reader, the
+trace protocol and the command line. No GPU."""
+import io
+import json
+import struct
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import llaisys_b200 as llaisys
+from llaisys_b200 import trace
+from llaisys_b200.models import Qwen2, Vozozen, load_model, model_class
+from llaisys_b200.models import vozozen as vz
+from llaisys_b200.models.weights import SafetensorsFile, checkpoint_files
+from oracle import vozozen as oracle
+from tests import vozozen_cases as cases
+
+
+def write_safetensors(path, tensors):
+    header, blob = {"__metadata__": {"format": "pt"}}, b""
+    for name, a in tensors.items():
+        kind = {np.dtype(np.uint16): "BF16", np.dtype(np.float32): "F32", np.dtype(np.int32): "I32"}[a.dtype]
+        header[name] = {"dtype": kind, "shape": list(a.shape), "data_offsets": [len(blob), len(blob) + a.nbytes]}
+        blob += a.tobytes()
+    text = json.dumps(header).encode()
+    path.write_bytes(struct.pack("<Q", len(text)) + text + blob)
+
+
+def test_class_by_config():
+    assert model_class({"architecture": "Vozozen"}) is Vozozen
+    assert model_class({"architectures": ["Qwen2ForCausalLM"], "model_type": "qwen2"}) is Qwen2
+    assert model_class({"model_type": "qwen2"}) is Qwen2
+    with pytest.raises(ValueError, match="Mamba"):
+        model_class({"architecture": "Mamba"})
+
+
+def test_qwen2_checkpoint_through_the_registry(tmp_path):
+    """A directory with config.json and safetensors becomes a running model (CPU) without naming its class."""
+    import safetensors.torch
+    from tests.test_qwen2_model import hf_greedy, hf_model
+
+    cfg, hf = hf_model(seed=5)
+    (tmp_path / "config.json").write_text(json.dumps({**cfg, "model_type": "qwen2", "dtype": "float32"}))
+    state = {k: v.contiguous().clone() for k, v in hf.state_dict().items()}
+    safetensors.torch.save_file(state, str(tmp_path / "model.safetensors"))
+    model = load_model(tmp_path, llaisys.DeviceType.CPU)
+    assert isinstance(model, Qwen2)
+    assert model.generate([3, 1, 4], max_new_tokens=5) == hf_greedy(hf, [3, 1, 4], 5)
+    # logits at chosen rows, and a pool smaller than slots x length, on the shared step
+    model.configure_cache(2, 64, 64)
+    assert model.free_pages == 4
+    toks = list(range(20))
+    got = model.step_rows([model.add_seq()], [toks], [4, 19])
+    with torch.no_grad():
+        want = hf(torch.tensor([toks])).logits[0, [4, 19]].float().numpy()
+    assert np.abs(got - want).max() < 2e-4
+
+
+def test_safetensors_reader(tmp_path):
+    a = np.arange(6, dtype=np.float32).reshape(2, 3)
+    b = cases.bf16_words(np.array([1.0, -2.5, 3.14159], dtype=np.float32))
+    c = np.array([7, 8], dtype=np.int32)
+    write_safetensors(tmp_path / "x.safetensors", {"a": a, "b": b, "c": c})
+    f = SafetensorsFile(tmp_path / "x.safetensors")
+    assert f.names() == ["a", "b", "c"] and f.shape("a") == (2, 3) and f.dtype("b") == "BF16"
+    assert np.array_equal(f.array("a"), a) and np.array_equal(f.array("b"), b) and np.array_equal(f.array("c"), c)
+    assert oracle.to_f64(f.array("b"))[1] == -2.5
+    (tmp_path / "short.safetensors").write_bytes(b"abc")
+    with pytest.raises(ValueError):
+        SafetensorsFile(tmp_path / "short.safetensors")
+    with pytest.raises(FileNotFoundError):
+        list(checkpoint_files(tmp_path / "nowhere"))
+
+
+@pytest.mark.parametrize("name", sorted(cases.CASES))
+def test_configuration_reaches_the_library(name):
+    cfg, ranks = cases.CASES[name]
+    meta = vz.build_meta(cfg, ranks, llaisys.DataType.BF16)
+    assert meta.nlayer == len(cfg["layers"]) and meta.width == cfg["width"] and meta.voc == cfg["vocab"]
+    for i, entry in enumerate(cfg["layers"]):
+        got, left, right = meta.layers[i], entry["mixer"]["left"], entry["mixer"]["right"]
+        assert (got.left.heads, got.left.kv_heads, got.left.dim, got.left.vdim, got.left.window) == (
+            left["heads"], left["kv_heads"], left["dim"], left["vdim"], left["mask"]["size"])
+        assert (got.right.heads, got.right.dim, got.right.vdim, got.right.rank) == (
+            right["heads"], right["dim"], right["vdim"], ranks[i])
+        assert got.right.tau == pytest.approx(right["tau"]) and got.left.scale == pytest.approx(left["scale"])
+        assert got.left_scale == pytest.approx(entry["mixer"]["left_scale"])
+        assert got.right_scale == pytest.approx(entry["mixer"]["right_scale"])
+        assert got.ff == (entry["mlp"]["ff"] if entry["mlp"] else 0)
+    assert meta.logit_softcap == pytest.approx(cfg["logit_softcap"]) and meta.eps == pytest.approx(cfg["norm"]["eps"])
+    assert meta.embed_scale == pytest.approx(cfg["embedding"]["scale"])
+    loop = cfg["loop"]
+    assert (meta.loop_start, meta.loop_stop, meta.loop_times) == ((loop["start"], loop["stop"], loop["times"]) if loop else (0, 0, 0))
+
+
+def test_unknown_parts_of_a_configuration_are_refused():
+    cfg, ranks = cases.case("looped")[0], cases.CASES["looped"][1]
+    cfg["layers"][0]["type"] = "serial"
+    with pytest.raises(ValueError, match="serial"):
+        vz.build_meta(cfg, ranks, llaisys.DataType.BF16)
+    cfg = cases.case("looped")[0]
+    cfg["layers"][0]["mlp"]["kind"] = "experts"
+    with pytest.raises(ValueError, match="experts"):
+        vz.build_meta(cfg, ranks, llaisys.DataType.BF16)
+
+
+def test_no_host_stand_in():
+    cfg, w = cases.case("looped")
+    with pytest.raises(RuntimeError, match="NVIDIA"):
+        Vozozen(config=cfg, state_dict=w, device=llaisys.DeviceType.CPU)
+    with pytest.raises(ValueError, match="a1"):
+        Vozozen(config=cfg, state_dict={k: v for k, v in w.items() if not k.endswith("a1")}, device=llaisys.DeviceType.CPU)
+
+
+def test_oracle_mechanisms_agree_with_closed_forms():
+    """The plain functions the device is compared with, on cases whose answers are known."""
+    torch.manual_seed(0)
+    q, k, v = (torch.randn(12, 2, 4, dtype=torch.float64) for _ in range(3))
+    ones = torch.ones(12, 2, 4, dtype=torch.float64)
+    out, S = oracle.gated_linear(q, k, v, ones)  # no decay: plain sums of outer products
+    want = torch.stack([sum((q[t, 1] @ k[s, 1]) * v[s, 1] for s in range(t + 1)) for t in range(12)])
+    assert torch.allclose(out[:, 1], want) and torch.allclose(S[0], torch.einsum("td,te->de", k[:, 0], v[:, 0]))
+    assert torch.allclose(oracle.key_decay(torch.tensor([0.0]).double(), 1.0), torch.tensor([0.5]).double())
+    assert torch.allclose(oracle.window_attention(q, k, v, 1.0, 1), v)  # each token sees itself only
+    full = torch.nn.functional.scaled_dot_product_attention(*(x.transpose(0, 1) for x in (q, k, v)), is_causal=True, scale=0.7)
+    assert torch.allclose(oracle.window_attention(q, k, v, 0.7, 12), full.transpose(0, 1))
+    cfg = cases.CASES["looped"][0]
+    assert oracle.run_order(cfg) == [(0, False), (1, True), (2, False), (1, True), (2, False)]
+
+
+class FakeModel:
+    """Stands in for a model: counts slots and 'logits' = (sequence, position, token)."""
+    vocab = 3
+
+    def configure_cache(self, seqs, tokens, pool):
+        self.sizes, self.free, self.len = (seqs, tokens, pool), list(range(seqs)), {}
+
+    def add_seq(self):
+        s = self.free.pop()
+        self.len[s] = 0
+        return s
+
+    def free_seq(self, s):
+        self.free.append(s)
+
+    def step_rows(self, seqs, tokens, rows):
+        assert len(set(seqs)) == len(seqs)
+        flat = []
+        for s, toks in zip(seqs, tokens):
+            for t in toks:
+                flat.append((s, self.len[s], t))
+                self.len[s] += 1
+        return np.array([flat[r] for r in rows], dtype=np.float32).reshape(len(rows), 3)
+
+
+def test_trace_runner_slots_and_rows():
+    model = FakeModel()
+    runner = trace.TraceRunner(model, 640)
+    assert model.sizes == (trace.MAX_LIVE, 640, 640)
+    a = runner.step([{"id": "x", "tokens": [5, 6, 7], "want": [2]}, {"id": "y", "tokens": [9], "want": [0]}])
+    assert a[:, 1:].tolist() == [[2, 7], [0, 9]]
+    b = runner.step([{"id": "y", "tokens": [1, 2], "want": []}], ["x"])
+    assert b.shape == (0, 3) and len(model.free) == trace.MAX_LIVE - 1
+    c = runner.step([{"id": "x", "tokens": [4], "want": [0]}, {"id": "y", "tokens": [3], "want": [0]}], ["x", "y"])
+    assert c[:, 1:].tolist() == [[0, 4], [3, 3]] and len(model.free) == trace.MAX_LIVE
+
+
+def test_trace_main_protocol(tmp_path, monkeypatch, capsys):
+    import llaisys_b200.models as models
+
+    monkeypatch.setattr(models, "load_model", lambda path, dtype: FakeModel())
+    lines = [{"step": 0, "entries": [{"id": "q", "tokens": [1, 2], "want": [1, 0]}], "end": []},
+             {"step": 1, "entries": [{"id": "q", "tokens": [2], "want": []}], "end": ["q"]}]
+    monkeypatch.setattr(sys, "stdin", io.StringIO("\n".join(map(json.dumps, lines)) + "\n"))
+    rc = trace.main(["--model", "m", "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "64"])
+    assert rc == 0 and capsys.readouterr().out.split("\n")[:2] == ["done 0", "done 1"]
+    got = np.fromfile(tmp_path / "0.f32", dtype="<f4").reshape(2, 3)
+    assert got[:, 1:].tolist() == [[1, 2], [0, 1]] and not (tmp_path / "1.f32").exists()
+
+
+def test_command_line_generates(tmp_path, capsys):
+    """python -m llaisys_b200 generate, on a Qwen2 checkpoint (CPU): several prompts through the batching engine."""
+    import safetensors.torch
+    from llaisys_b200.cli import main
+    from tests.test_qwen2_model import hf_greedy, hf_model
+
+    cfg, hf = hf_model(seed=6)
+    (tmp_path / "config.json").write_text(json.dumps({**cfg, "model_type": "qwen2"}))
+    safetensors.torch.save_file({k: v.contiguous().clone() for k, v in hf.state_dict().items()}, str(tmp_path / "model.safetensors"))
+    assert main(["info", "--model", str(tmp_path)]) == 0
+    assert "Qwen2" in capsys.readouterr().out
+    assert main(["generate", "--model", str(tmp_path), "--device", "cpu", "--dtype", "float32", "--max-new-tokens", "4",
+                 "--prompt", "3,1,4", "--prompt", "1,5,9,2,6"]) == 0
+    out = [json.loads(line) for line in capsys.readouterr().out.strip().split("\n")]
+    for row, p in zip(out, ([3, 1, 4], [1, 5, 9, 2, 6])):
+        assert row["prompt"] == p and row["tokens"] == hf_greedy(hf, p, 4)[len(p):]
+    assert main(["generate", "--model", str(tmp_path), "--device", "cpu", "--dtype", "float32", "--max-new-tokens", "3",
+                 "--prompt", "7", "--top-k", "4", "--seed", "2"]) == 0
+    assert len(json.loads(capsys.readouterr().out)["tokens"]) == 3
