@@ -76,9 +76,8 @@ struct LlaisysGatedLinear {
 };
 LLAISYS_API int llaisysGatedLinearDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype,
                                       const struct LlaisysGatedLinear *args, int decode, llaisysStream_t stream);
-/* Floats of scratch_segments for a call of these sizes (0: such a call is never cut). */
-LLAISYS_API size_t llaisysGatedLinearSegmentFloats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv, size_t n_seqs,
-                                                   size_t max_q_len);
+/* Floats of scratch_segments that serve every call of these sizes (0: such calls are never cut). */
+LLAISYS_API size_t llaisysGatedLinearSegmentFloats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
 
 #ifdef __cplusplus
 }

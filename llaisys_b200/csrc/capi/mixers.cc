@@ -152,12 +152,11 @@ int llaisysGatedLinearDev(llaisysDeviceType_t device_type, int device_id, llaisy
     });
 }
 
-size_t llaisysGatedLinearSegmentFloats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv, size_t n_seqs,
-                                       size_t max_q_len) {
+size_t llaisysGatedLinearSegmentFloats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv) {
 #ifdef ENABLE_NVIDIA_API
-    return llaisys::kernels::gated_linear_segment_floats(dtype, heads, dk, dv, n_seqs, max_q_len);
+    return llaisys::kernels::gated_linear_segment_floats(dtype, heads, dk, dv);
 #else
-    (void)dtype, (void)heads, (void)dk, (void)dv, (void)n_seqs, (void)max_q_len;
+    (void)dtype, (void)heads, (void)dk, (void)dv;
     return 0;
 #endif
 }

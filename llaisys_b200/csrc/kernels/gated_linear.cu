@@ -2,8 +2,10 @@
 //   * decode: one token per sequence, everything from the projection row to the gated, normed output in one launch. A CTA
 //     owns one (sequence, head): it reads that head's f32 state once, updates it and writes it back -- HBM-bound,
 //     2 * dk * dv * 4 bytes per head.
+//     In a batch of runs the same kernel serves the sequences that bring a single token.
 //   * recurrent: runs of tokens, one after the other in f32 with the state in registers. A CTA owns 16 value columns of one
 //     (sequence, head). Exact in the order of the definition.
+//     (The third form, runs on the tensor cores, is gated_linear_chunk.cu; bf16 models run that one.)
 // All arithmetic of the recurrence, the decay and the norm is f32.
 #include "device_utils.cuh"
 #include "gated_linear.cuh"
@@ -32,11 +34,15 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_linear_decode_kernel(Gat
     const int tid = int(threadIdx.x);
     const int64_t slot = a.seq_ids[i];
     const bool fresh = a.kv_lens[i] == 1;
+    const int row_i = a.q_starts != nullptr ? a.q_starts[i] : i;
     grid_dependency_wait();
     grid_launch_dependents();
+    if (a.q_starts != nullptr && a.q_starts[i + 1] - row_i != 1) {
+        return; // a run of tokens (or none): another kernel's
+    }
 
     float *state = a.state + slot * a.slot_stride + int64_t(head) * a.dk * a.dv;
-    const T *row = static_cast<const T *>(a.proj) + int64_t(i) * a.row_stride;
+    const T *row = static_cast<const T *>(a.proj) + int64_t(row_i) * a.row_stride;
     for (int r = tid; r < a.rank; r += kDecodeThreads) {
         s_z[r] = to_f32(row[a.z_at + r]);
     }
@@ -118,7 +124,7 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_linear_decode_kernel(Gat
         tot += s_red[w];
     }
     const float inv = rsqrtf(tot / float(a.dv) + a.eps) * a.out_scale;
-    T *out = static_cast<T *>(a.out) + int64_t(i) * a.out_stride + int64_t(head) * a.dv;
+    T *out = static_cast<T *>(a.out) + int64_t(row_i) * a.out_stride + int64_t(head) * a.dv;
     const T *w = static_cast<const T *>(a.norm_w);
     for (int c = tid; c < a.dv; c += kDecodeThreads) {
         const float g = to_f32(row[a.g_at + int64_t(head) * a.dv + c]);
@@ -282,13 +288,7 @@ void check_args(const GatedLinearArgs &a) {
     CHECK_ARGUMENT(int64_t(a.n_seqs) * a.heads <= 0x7fffffff, "gated linear attention: too many (sequence, head) pairs");
 }
 
-} // namespace
-
-void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &a) {
-    if (a.n_seqs == 0) {
-        return;
-    }
-    check_args(a);
+void single_tokens(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &a) {
     auto s = static_cast<cudaStream_t>(stream);
     dispatch(dtype, [&](auto tag) {
         using T = decltype(tag);
@@ -312,6 +312,18 @@ void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLi
         auto kernel = wide ? gated_linear_decode_kernel<T, 4> : gated_linear_decode_kernel<T, 1>;
         LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, GatedLinearArgs(a), int(col_groups)));
     });
+}
+
+} // namespace
+
+void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args) {
+    if (args.n_seqs == 0) {
+        return;
+    }
+    check_args(args);
+    GatedLinearArgs a = args;
+    a.q_starts = nullptr; // row i is sequence i's
+    single_tokens(stream, dtype, a);
     check_launch("gated_linear_decode");
 }
 
@@ -322,16 +334,26 @@ void gated_linear_chunk(stream_t stream, llaisysDataType_t dtype, const GatedLin
     check_args(a);
     CHECK_ARGUMENT(a.raw != nullptr && a.decay != nullptr, "gated linear attention: scratch missing");
     auto s = static_cast<cudaStream_t>(stream);
-    dispatch(dtype, [&](auto tag) {
+    auto finish = [&](auto tag) {
         using T = decltype(tag);
-        gated_linear_decay_kernel<T><<<unsigned(a.n_rows), 128, size_t(a.rank) * sizeof(float), s>>>(a);
-        recurrent<T>(s, a);
         const int64_t items = int64_t(a.n_rows) * a.heads;
         gated_linear_out_kernel<T><<<unsigned((items + 7) / 8), 256, 0, s>>>(a);
-    });
+    };
+    if (gated_linear_tiles_apply(dtype, a)) {
+        gated_linear_tiles(stream, a);
+        if (a.dv > 128) {
+            finish(__nv_bfloat16{}); // (rows of single tokens hold nothing yet: the next kernel writes them)
+        }
+        single_tokens(stream, dtype, a);
+    } else {
+        dispatch(dtype, [&](auto tag) {
+            using T = decltype(tag);
+            gated_linear_decay_kernel<T><<<unsigned(a.n_rows), 128, size_t(a.rank) * sizeof(float), s>>>(a);
+            recurrent<T>(s, a);
+            finish(tag);
+        });
+    }
     check_launch("gated_linear_chunk");
 }
-
-size_t gated_linear_segment_floats(llaisysDataType_t, size_t, size_t, size_t, size_t, size_t) { return 0; }
 
 } // namespace llaisys::kernels

@@ -90,8 +90,8 @@ void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
 // runs of tokens.
 void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args);
 void gated_linear_chunk(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args);
-// Floats of GatedLinearArgs::segments for a chunk call of these sizes; 0 = such a call is never cut.
-size_t gated_linear_segment_floats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv, size_t n_seqs, size_t max_q_len);
+// Floats of GatedLinearArgs::segments that serve every chunk call of these sizes; 0 = such calls are never cut.
+size_t gated_linear_segment_floats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
 
 // ---- operators of a residual stream kept in f32 (x float [rows, d]) around dtype activations ----
 // x[r, :] = scale * w[tokens[r], :]; copy (may be null): the same rounded to dtype, row r at copy + r * copy_stride

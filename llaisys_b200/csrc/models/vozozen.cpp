@@ -237,7 +237,7 @@ void Vozozen::ensureActivations(size_t n_tokens, size_t n_out) {
     const size_t W = _meta.width;
     if (n_tokens > _ws_tokens) {
         ++_generation;
-        size_t proj = 0, q = 0, heads = 0, mix = 0, raw = 0, decay = 0, ff = 0;
+        size_t proj = 0, q = 0, heads = 0, mix = 0, raw = 0, decay = 0, ff = 0, segments = 0;
         for (const Layer &l : _layers) {
             proj = std::max(proj, l.n_proj);
             q = std::max(q, l.meta.left.heads * l.meta.left.dim);
@@ -246,6 +246,10 @@ void Vozozen::ensureActivations(size_t n_tokens, size_t n_out) {
             raw = std::max(raw, l.meta.right.heads * l.meta.right.vdim);
             decay = std::max(decay, l.meta.right.heads * l.meta.right.dim);
             ff = std::max(ff, l.meta.ff);
+#ifdef ENABLE_NVIDIA_API
+            segments = std::max(segments, kernels::gated_linear_segment_floats(_dtype, l.meta.right.heads, l.meta.right.dim,
+                                                                               l.meta.right.vdim));
+#endif
         }
         _x = rt.allocateDeviceStorage(n_tokens * W * sizeof(float));
         _pass_in = rt.allocateDeviceStorage(n_tokens * 2 * W * _elem);
@@ -256,6 +260,9 @@ void Vozozen::ensureActivations(size_t n_tokens, size_t n_out) {
         _mix = rt.allocateDeviceStorage(n_tokens * mix * _elem);
         _raw = rt.allocateDeviceStorage(n_tokens * raw * sizeof(float));
         _decay = rt.allocateDeviceStorage(n_tokens * decay * sizeof(float));
+        if (segments != 0 && !_segments) {
+            _segments = rt.allocateDeviceStorage(segments * sizeof(float));
+        }
         _u = rt.allocateDeviceStorage(n_tokens * std::max<size_t>(ff, 1) * _elem);
 #ifdef ENABLE_NVIDIA_API
         // the padding columns between and behind the two sides meet zero weights: they only have to be finite
@@ -324,6 +331,8 @@ void Vozozen::forward(const StepArrays &a, const StepShape &s) {
         g.out_stride = int64_t(l.n_mix);
         g.raw = reinterpret_cast<float *>(_raw->memory());
         g.decay = reinterpret_cast<float *>(_decay->memory());
+        g.segments = _segments ? reinterpret_cast<float *>(_segments->memory()) : nullptr;
+        g.segment_floats = _segments ? _segments->size() / sizeof(float) : 0;
         if (s.decode_only) {
             kernels::gated_linear_decode(_stream, _dtype, g);
         } else {

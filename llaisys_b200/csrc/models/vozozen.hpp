@@ -65,7 +65,7 @@ private:
     std::vector<core::storage_t> _weight_blocks;
     std::byte *_embed = nullptr, *_loop_in = nullptr, *_final_norm = nullptr, *_head = nullptr;
 
-    core::storage_t _x, _pass_in, _h, _proj, _q, _row_scale, _mix, _raw, _decay, _u, _h_out;
+    core::storage_t _x, _pass_in, _h, _proj, _q, _row_scale, _mix, _raw, _decay, _segments, _u, _h_out;
     bool _record = false;
     std::vector<float> _recorded;
 };

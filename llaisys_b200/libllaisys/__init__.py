@@ -288,7 +288,7 @@ PROTOTYPES: dict[str, tuple] = {
                                             llaisysStream_t]),
     "llaisysGatedLinearDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysGatedLinear), c_int,
                                       llaisysStream_t]),
-    "llaisysGatedLinearSegmentFloats": (c_size_t, [llaisysDataType_t, c_size_t, c_size_t, c_size_t, c_size_t, c_size_t]),
+    "llaisysGatedLinearSegmentFloats": (c_size_t, [llaisysDataType_t, c_size_t, c_size_t, c_size_t]),
     # include/llaisys/models/model.h
     "llaisysModelDestroy": (None, [_MODEL]),
     "llaisysModelVocab": (c_size_t, [_MODEL]),

@@ -305,9 +305,9 @@ def gated_linear_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 
     _check(LIB_LLAISYS.llaisysGatedLinearDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
 
 
-def gated_linear_segment_floats(dtype: DataType, heads: int, dk: int, dv: int, n_seqs: int, max_q_len: int) -> int:
-    """Size of scratch_segments for a chunk call of these sizes."""
-    return int(LIB_LLAISYS.llaisysGatedLinearSegmentFloats(int(dtype), heads, dk, dv, n_seqs, max_q_len))
+def gated_linear_segment_floats(dtype: DataType, heads: int, dk: int, dv: int) -> int:
+    """Size of scratch_segments for chunk calls of these sizes (0: they are never cut)."""
+    return int(LIB_LLAISYS.llaisysGatedLinearSegmentFloats(int(dtype), heads, dk, dv))
 
 
 def lse_merge(out, parts, n_parts: int, n_rows: int, head_dim: int, *, dtype: DataType,

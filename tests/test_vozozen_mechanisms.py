@@ -247,7 +247,7 @@ class Gla:
         out = torch.full((rows, self.out_width), 5.0, dtype=self.dtype, device="cuda")
         raw = torch.empty(rows, self.heads * self.dv, device="cuda")
         decay = torch.empty(rows, self.heads * self.dk, device="cuda")
-        n_seg = llaisys.gated_linear_segment_floats(LL[self.dtype], self.heads, self.dk, self.dv, len(who), max(counts))
+        n_seg = llaisys.gated_linear_segment_floats(LL[self.dtype], self.heads, self.dk, self.dv)
         seg = torch.full((n_seg,), float("nan"), device="cuda") if n_seg and segments else None
         torch.cuda.synchronize()
         llaisys.gated_linear_dev(
