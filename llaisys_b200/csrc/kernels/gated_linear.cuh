@@ -14,8 +14,8 @@ struct alignas(sizeof(T) * N) Pieces {
 __device__ __forceinline__ float silu(float g) { return g / (1.f + expf(-g)); }
 // log(1 / (1 + exp(-z))) = min(z, 0) - log(1 + x), x = exp(-|z|) in (0, 1]; log(1 + x) = 2 artanh(s) with s = x / (2 + x) <= 1/3
 // by the odd power series of artanh up to s^13 (the first term left out is below 1e-8 of the sum).
-__device__ __forceinline__ float log_sigmoid(float z) {
-    const float x = expf(-fabsf(z)), s = __fdividef(x, 2.f + x), s2 = s * s;
+__device__ __forceinline__ float log_sigmoid_of(float z, float x) {
+    const float s = __fdividef(x, 2.f + x), s2 = s * s;
     float p = 1.f / 13.f;
     p = fmaf(p, s2, 1.f / 11.f);
     p = fmaf(p, s2, 1.f / 9.f);
@@ -25,6 +25,7 @@ __device__ __forceinline__ float log_sigmoid(float z) {
     p = fmaf(p, s2, 1.f);
     return fminf(z, 0.f) - 2.f * s * p;
 }
+__device__ __forceinline__ float log_sigmoid(float z) { return log_sigmoid_of(z, expf(-fabsf(z))); }
 
 // log a_t of key channel c of `head`: log_sigmoid(W_a2[h dk + c, :] . z + b[h dk + c]) / tau, z [rank] in shared memory
 template <typename T>
