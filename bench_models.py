@@ -1,0 +1,304 @@
+"""bench.py --workload vozozen: the Vozozen design beside Qwen2 at equal size, one GPU.
+
+Two parts, one JSON line:
+  models   prefill and decode throughput of whole models with random weights. Equal size: the same width, query and kv heads,
+           layers and vocabulary, and an MLP of as many parameters (Vozozen's has two matrices, so its inner size is 1.5 times
+           Qwen2's three). Vozozen's second mixer (gated linear attention) comes on top.
+  kernels  every new kernel alone next to the like kernel of Qwen2, each as a fraction of its own roofline: CUDA graphs of
+           launches over rotating buffers larger than L2, the median of the replays.
+"""
+from __future__ import annotations
+
+import json
+import statistics
+
+import numpy as np
+
+SIZES = {
+    "1.5B-like": dict(width=1536, heads=12, kv_heads=2, gla_heads=6, ff=8960, layers=8, vocab=32768, window=1024),
+    "8B-like": dict(width=4096, heads=32, kv_heads=8, gla_heads=16, ff=14336, layers=4, vocab=32768, window=1024),
+}
+D = 128
+PREFILL = {"one prompt of 8192": [8192], "eight prompts of 1024": [1024] * 8}
+DECODE_SEQS, DECODE_CTX, DECODE_STEPS = 64, 2048, 64
+
+
+def vozozen_config(s: dict) -> dict:
+    mixer = {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "mask": {"size": s["window"]},
+                      "scale": D ** -0.5},
+             "right": {"heads": s["gla_heads"], "dim": D, "vdim": D, "tau": 16.0}, "left_scale": 0.7, "right_scale": 0.7}
+    layer = {"type": "parallel", "mixer": mixer, "mlp": {"kind": "dense", "ff": s["ff"] * 3 // 2}}
+    return {"architecture": "Vozozen", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "loop": None, "layers": [layer] * s["layers"]}
+
+
+def qwen2_config(s: dict) -> dict:
+    return {"hidden_size": s["width"], "num_attention_heads": s["heads"], "num_key_value_heads": s["kv_heads"], "head_dim": D,
+            "intermediate_size": s["ff"], "num_hidden_layers": s["layers"], "vocab_size": s["vocab"], "rms_norm_eps": 1e-6,
+            "rope_theta": 1e6}
+
+
+def build_model(torch, llaisys, family: str, s: dict):
+    """-> the model, bytes of weights a decode step reads, parameters of the matrices applied to every token"""
+    if family == "qwen2":
+        from bench import qwen2_random_weights
+
+        cfg = qwen2_config(s)
+        model = llaisys.models.Qwen2(config=cfg, device=llaisys.DeviceType.NVIDIA, dtype=llaisys.DataType.BF16,
+                                     max_seq_len=DECODE_CTX + 256)
+        total = per_token = 0
+        for name, value in qwen2_random_weights(cfg, 4, "cuda"):
+            model.load_tensor(name, value)
+            if "embed_tokens" not in name:
+                total += value.numel() * 2
+                per_token += value.numel() if value.ndim == 2 and name != "lm_head.weight" else 0
+        return model, total, per_token
+    from llaisys_b200.models.vozozen import weight_shapes
+
+    cfg = vozozen_config(s)
+    g = torch.Generator(device="cuda").manual_seed(4)
+    weights, total, per_token = {}, 0, 0
+    for name, shape in weight_shapes(cfg, [16] * s["layers"]).items():
+        if name.endswith(("norm", "norm1", "norm2")):
+            w = torch.ones(shape)
+        elif name.endswith("a2.b"):
+            w = torch.full(shape, 3.0)
+        else:
+            w = torch.randn(shape, generator=g, device="cuda") * 0.02
+        weights[name] = w.bfloat16().cpu().view(torch.int16).numpy().view(np.uint16)
+        if name != "embed":
+            total += w.numel() * 2
+            per_token += w.numel() if w.ndim == 2 and name != "head" else 0
+    model = llaisys.models.Vozozen(config=cfg, state_dict=weights, dtype=llaisys.DataType.BF16)
+    return model, total, per_token
+
+
+def visible(n: int, window: int | None) -> int:
+    """(query, key) pairs of a causal run of n tokens from an empty cache"""
+    full = n * (n + 1) // 2
+    return full if window is None or window >= n else full - (n - window) * (n - window + 1) // 2
+
+
+def prefill_flops(family: str, s: dict, lens: list[int], per_token: int) -> float:
+    tokens = sum(lens)
+    flops = 2.0 * tokens * per_token + 2.0 * len(lens) * s["vocab"] * s["width"]
+    window = s["window"] if family == "vozozen" else None
+    flops += s["layers"] * s["heads"] * 4.0 * D * sum(visible(n, window) for n in lens)
+    if family == "vozozen":
+        flops += s["layers"] * s["gla_heads"] * tokens * 4.0 * D * D  # state update and read-out
+    return flops
+
+
+def measure_model(torch, llaisys, stream, family: str, s: dict, repeats: int) -> dict:
+    from bench import _peaks
+
+    hbm, _, sustained, kind = _peaks()
+    model, weight_bytes, per_token = build_model(torch, llaisys, family, s)
+    model.configure_cache(DECODE_SEQS, max(8192, DECODE_CTX + 2 * DECODE_STEPS), DECODE_SEQS * (DECODE_CTX + 2 * DECODE_STEPS + 16))
+    rng = np.random.default_rng(0)
+    rec = {"parameters_per_token": per_token, "prefill": {}, "decode": {}}
+    for what, lens in PREFILL.items():
+        prompts = [rng.integers(0, s["vocab"], n).tolist() for n in lens]
+        times = []
+        for r in range(3 + repeats):
+            seqs = [model.add_seq() for _ in lens]
+            a, b = (torch.cuda.Event(enable_timing=True) for _ in range(2))
+            a.record(stream)
+            model.step(seqs, prompts)
+            b.record(stream)
+            b.synchronize()
+            if r >= 3:
+                times.append(a.elapsed_time(b))
+            for q in seqs:
+                model.free_seq(q)
+        ms, flops = statistics.median(times), prefill_flops(family, s, lens, per_token)
+        rec["prefill"][what] = {"tokens_per_s": sum(lens) * 1e3 / ms, "ms": ms, "ms_min": min(times), "ms_max": max(times),
+                                "tflops": flops / ms / 1e9, "frac_of_sustained_gemm": flops / ms / 1e9 / sustained}
+    seqs = [model.add_seq() for _ in range(DECODE_SEQS)]
+    nxt = []
+    for i in range(0, DECODE_SEQS, 4):
+        nxt += model.step(seqs[i:i + 4], [rng.integers(0, s["vocab"], DECODE_CTX).tolist() for _ in range(4)])
+    nxt = model.decode_loop(seqs, nxt, 8)[-1].tolist()
+    model.decode_loop(seqs, nxt, DECODE_STEPS + 1)
+    ms = model.last_loop_ms
+    keys = min(DECODE_CTX + DECODE_STEPS // 2, s["window"]) if family == "vozozen" else DECODE_CTX + DECODE_STEPS // 2
+    kv = s["layers"] * DECODE_SEQS * keys * s["kv_heads"] * 2 * D * 2
+    state = 2 * s["layers"] * DECODE_SEQS * s["gla_heads"] * D * D * 4 if family == "vozozen" else 0
+    moved = weight_bytes + kv + state
+    rec["decode"] = {"tokens_per_s": DECODE_SEQS * 1e3 / ms, "ms_per_step": ms, "bytes": {"weights": weight_bytes, "kv": kv, "state": state},
+                     "gb_per_s": moved / ms / 1e6, "frac_of_copy": moved / ms / 1e6 / hbm, "peak_kind": kind}
+    model.close()
+    return rec
+
+
+# ---- kernels ----------------------------------------------------------------------------------------------------------------
+
+
+class Kernels:
+    """Timed launches of single kernels on the library's stream."""
+
+    def __init__(self, torch, llaisys, stream, repeats: int):
+        from bench import _peaks
+
+        self.torch, self.ll, self.stream, self.repeats = torch, llaisys, stream, repeats
+        self.cs = llaisys.context_stream()
+        self.hbm, self.burst, _, self.kind = _peaks()
+        self.gen = torch.Generator(device="cuda").manual_seed(1)
+
+    def rand(self, *shape, scale=1.0):
+        return (self.torch.randn(*shape, generator=self.gen, device="cuda") * scale).bfloat16()
+
+    def i32(self, values):
+        return self.torch.tensor(values, dtype=self.torch.int32, device="cuda")
+
+    def time(self, launch, per_graph: int = 8) -> float:
+        """Median microseconds per launch(i)"""
+        from bench import replay_times
+
+        torch = self.torch
+        for i in range(3):
+            launch(i)
+        self.stream.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph, stream=self.stream):
+            for i in range(per_graph):
+                launch(i)
+        return statistics.median(replay_times(torch, self.stream, graph, self.repeats)) * 1e3 / per_graph
+
+    def memory(self, us: float, nbytes: int) -> dict:
+        return {"us": us, "bytes": nbytes, "tb_per_s": nbytes / us / 1e6, "frac": nbytes / us / 1e3 / self.hbm, "of": f"{self.kind} copy"}
+
+    def tensor(self, us: float, flops: float) -> dict:
+        return {"us": us, "tflops": flops / us / 1e6, "frac": flops / us / 1e6 / self.burst, "of": f"{self.kind} burst bf16 GEMM"}
+
+    def attention(self, heads: int, kv_heads: int, window: int, layers: int = 3) -> dict:
+        """Decode over 64 sequences and one chunk of 8192 tokens, with the window and without one at equal visible keys /
+        at full length; the position-wise kernel in front of each."""
+        torch, ll = self.torch, self.ll
+        out = {}
+        n_seqs, ctx, rows = 64, 2 * window, 8192
+        pages = max(n_seqs * ctx, rows) // 16
+        cache = ll.PagedKVCache(pages, kv_heads, D, nlayer=layers, dtype=ll.DataType.BF16, device=ll.DeviceType.NVIDIA,
+                                max_seqs=n_seqs, max_pages_per_seq=max(ctx, rows) // 16)
+        seqs = [cache.add_seq() for _ in range(n_seqs)]
+        for q in seqs:
+            cache.reserve(q, ctx)
+        cache.flush()
+        cache.set_launch_overlap(True)
+        width = (heads + 2 * kv_heads) * D
+        for layer in range(layers):  # every page holds something
+            for lo in range(0, n_seqs, 8):
+                part = seqs[lo:lo + 8]
+                ids, pos = self.i32([q for q in part for _ in range(ctx)]), self.i32(list(range(ctx)) * len(part))
+                k, v = self.rand(len(part) * ctx, kv_heads, D), self.rand(len(part) * ctx, kv_heads, D)
+                cache.append_dev(layer, k, v, ids, pos, len(part) * ctx, self.cs)
+                self.stream.synchronize()
+        q, o = self.rand(n_seqs, heads, D), self.rand(n_seqs, heads, D)
+        factor = torch.rand(n_seqs, heads, device="cuda")
+        ids, full, short = self.i32(seqs), self.i32([ctx] * n_seqs), self.i32([window] * n_seqs)
+        kv_bytes = n_seqs * window * kv_heads * 2 * D * 2 + 2 * n_seqs * heads * D * 2
+        common = dict(n_seqs=n_seqs, nh=heads, scale=D ** -0.5, stream=self.cs)
+        us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, None, full, total_q=n_seqs, max_q_len=1, max_kv_len=ctx,
+                                                     window=window, row_scale=factor, **common))
+        out["decode attention, window"] = self.memory(us, kv_bytes)
+        us = self.time(lambda i: cache.decode_dev(i % layers, o, q, ids, short, n_seqs, window, heads, D ** -0.5, self.cs))
+        out["decode attention, Qwen2, as many keys"] = self.memory(us, kv_bytes)
+
+        qn, kn = self.rand(D), self.rand(D)
+        wide = width + heads  # the gate behind q | k | v
+        for n in (n_seqs, rows):
+            if n == rows:
+                for s in seqs:
+                    cache.free_seq(s)
+                long = cache.add_seq()
+                cache.reserve(long, rows)
+                cache.flush()
+                ids_n, pos_n = self.i32([long] * rows), self.i32(list(range(rows)))
+            else:
+                ids_n, pos_n = ids, self.i32([ctx - 1] * n_seqs)
+            proj = [self.rand(n, (wide + 7) // 8 * 8) for _ in range(layers)]
+            qo, fac = self.rand(n, heads, D), torch.empty(n, heads, device="cuda")
+            moved = n * (2 * width * 2 + heads * 6)
+            us = self.time(lambda i: cache.norm_append_dev(
+                i % layers, self.cs, proj=proj[i % layers], row_stride=proj[0].shape[1], q_at=0, k_at=heads * D,
+                v_at=(heads + kv_heads) * D, gate_at=width, q_norm=qn, k_norm=kn, eps=1e-6, gate_scale=0.7, q_out=qo, row_scale=fac,
+                seq_ids_dev=ids_n, positions_dev=pos_n, n_rows=n, nh=heads))
+            out[f"norm + append, {n} rows"] = self.memory(us, moved)
+            packed = [self.rand(n, width) for _ in range(layers)]
+            bias = self.rand(width)
+            us = self.time(lambda i: self._rope_append(cache, i % layers, qo, packed[i % layers], bias, ids_n, pos_n, n, heads))
+            out[f"rope + append, Qwen2, {n} rows"] = self.memory(us, n * 2 * width * 2)
+        q, o = self.rand(rows, heads, D), self.rand(rows, heads, D)
+        factor = torch.rand(rows, heads, device="cuda")
+        ids, starts, lens = self.i32([long]), self.i32([0, rows]), self.i32([rows])
+        common = dict(n_seqs=1, total_q=rows, max_q_len=rows, max_kv_len=rows, nh=heads, scale=D ** -0.5, stream=self.cs)
+        us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, lens, window=window, row_scale=factor, **common))
+        out["chunk attention, window, 8192 tokens"] = self.tensor(us, 4.0 * D * heads * visible(rows, window))
+        us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, lens, **common))
+        out["chunk attention, Qwen2, 8192 tokens"] = self.tensor(us, 4.0 * D * heads * visible(rows, None))
+        cache.check()
+        cache.close()
+        return out
+
+    def _rope_append(self, cache, layer, qo, packed, bias, ids, pos, n, heads):
+        lib = self.ll.libllaisys.LIB_LLAISYS
+        rc = lib.llaisysPagedKVRopeAppendDev(cache._kv, layer, qo.data_ptr(), packed.data_ptr(), bias.data_ptr(), ids.data_ptr(),
+                                             pos.data_ptr(), n, heads, 1e6, self.cs)
+        assert rc == 0
+
+    def gated_linear(self, heads: int, lens: list[int], rank: int = 16, copies: int = 3) -> dict:
+        torch, ll = self.torch, self.ll
+        decode, rows, n = max(lens) == 1, sum(lens), heads * D
+        at = dict(q_at=0, k_at=n, v_at=2 * n, g_at=3 * n, z_at=4 * n)
+        width = 4 * n + rank
+        copies = copies if decode or rows * width * 2 < 300e6 else 2
+        proj = [self.rand(rows, width, scale=0.7) for _ in range(copies)]
+        state = [torch.zeros(len(lens), heads * D * D, device="cuda") for _ in range(copies)]
+        w, b, norm = self.rand(n, rank, scale=0.3), self.rand(n) + 3, self.rand(D)
+        out = self.rand(rows, n)
+        raw = torch.empty(4, device="cuda")  # (the tensor-core form uses neither scratch at 128 value columns)
+        floats = ll.gated_linear_segment_floats(ll.DataType.BF16, heads, D, D)
+        seg = torch.empty(floats, device="cuda")
+        ids, starts = self.i32(list(range(len(lens)))), self.i32([0, *np.cumsum(lens).tolist()])
+        kv = self.i32([x + 100 for x in lens])
+        us = self.time(lambda i: ll.gated_linear_dev(
+            ll.DataType.BF16, decode=decode, stream=self.cs, proj=proj[i % copies], row_stride=width, **at, decay_w=w, decay_b=b,
+            norm_w=norm, tau=16.0, q_scale=D ** -0.5, eps=1e-6, out_scale=0.7, heads=heads, dk=D, dv=D, rank=rank,
+            state=state[i % copies], slot_stride=heads * D * D, seq_ids_dev=ids, q_starts_dev=starts, kv_lens_dev=kv,
+            n_seqs=len(lens), n_rows=rows, max_q_len=max(lens), out=out, out_stride=n, scratch_raw=raw, scratch_decay=raw,
+            scratch_segments=seg, scratch_segment_floats=floats))
+        rec = self.memory(us, rows * (width + n) * 2 + 2 * len(lens) * heads * D * D * 4)
+        if not decode:
+            rec["f32_tflops_of_the_recurrence"] = rows * heads * 4.0 * D * D / us / 1e6
+        return rec
+
+
+def run(args) -> None:
+    from bench import ClockSampler, _init_device
+
+    torch, llaisys, rank, local_rank, world, _ = _init_device()
+    if world != 1:
+        raise SystemExit("--workload vozozen runs on one GPU")
+    handle = llaisys.context_stream()
+    stream = torch.cuda.ExternalStream(int(getattr(handle, "value", handle)))
+    repeats = 10 if args.repeats == 100 else max(3, args.repeats)
+    models, kernels = {}, {}
+    with ClockSampler(local_rank) as clocks:
+        for name, s in SIZES.items():
+            models[name] = {"size": s, **{f: measure_model(torch, llaisys, stream, f, s, repeats) for f in ("vozozen", "qwen2")}}
+            k = Kernels(torch, llaisys, stream, max(30, repeats))
+            kernels[name] = k.attention(s["heads"], s["kv_heads"], s["window"])
+            kernels[name]["gated linear decode, 64 sequences"] = k.gated_linear(s["gla_heads"], [1] * 64)
+            kernels[name]["gated linear chunk, one run of 8192"] = k.gated_linear(s["gla_heads"], [8192])
+            kernels[name]["gated linear chunk, eight runs of 1024"] = k.gated_linear(s["gla_heads"], [1024] * 8)
+    value = models["8B-like"]["vozozen"]["decode"]["tokens_per_s"]
+    print(json.dumps({
+        "metric": "decode tokens/s (Vozozen, 8B-like layers, greedy)", "value": value, "unit": "tokens/s", "n_gpus": 1,
+        "steps": DECODE_STEPS, "warmup": 8, "ms_per_step": models["8B-like"]["vozozen"]["decode"]["ms_per_step"],
+        "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic (random weights, random-token prompts)",
+        "config": {"workload": "vozozen", "decode": f"{DECODE_SEQS} sequences, {DECODE_CTX}-token prompts", "prefill": list(PREFILL),
+                   "l2": "weights, caches and rotated kernel buffers are larger than L2"},
+        "models": models, "kernels": kernels, "clocks": clocks.summary(),
+        "timing": "CUDA events: prefill around step(), decode around the library's graph replays, kernels around graph replays (median)",
+    }), flush=True)

@@ -153,6 +153,7 @@ __device__ __forceinline__ SeqGeom seq_geom(const PrefillParams &p, int a) {
         g.q_len = p.q_starts[a + 1] - g.q_start;
         g.kv_len = min(max(p.kv_lens[a], g.q_len), p.table_stride * kPage);
     }
+    g.q_len = min(g.q_len, g.kv_len); // (a chunk longer than the tables can hold: flagged elsewhere, never off the end here)
     g.off = g.kv_len - g.q_len; // query t sees keys j <= t + off
     g.n_qb = (g.q_len + kBlockM - 1) / kBlockM;
     g.window = p.window;
@@ -172,9 +173,20 @@ __device__ __forceinline__ int tile_blocks(const SeqGeom &g, int qb) {
 
 // units of the line that a sequence takes: per tile its blocks, then kTileCost units that stand for no block
 __device__ __forceinline__ int seq_blocks(const PrefillParams &p, const SeqGeom &g) {
-    int per_head = 0;
-    for (int qb = 0; qb < g.n_qb; ++qb) {
-        per_head += tile_blocks(g, qb) + kTileCost;
+    // the sum of tile_blocks over the row blocks in closed form (a loop over them, three times per CTA in front of all work,
+    // was a large part of a launch over one long chunk): row block qb < n - 1 ends at key (qb + 1) 128 + off, the last one at
+    // kv_len; blocks before the window are 2 qb + floor((off - window + 1) / 64) where that is not negative
+    static_assert(kBlockM == 2 * kBlockN, "row blocks advance two key blocks");
+    const int n = g.n_qb;
+    if (n == 0) {
+        return 0;
+    }
+    int per_head = (n - 1) * n + (n - 1) * ((g.off + kBlockN - 1) / kBlockN) + (g.kv_len + kBlockN - 1) / kBlockN + n * kTileCost;
+    if (g.window > 0) {
+        const int a = g.off - g.window + 1, q0 = a >= 0 ? 0 : (-a + kBlockM - 1) / kBlockM;
+        if (q0 < n) {
+            per_head -= (n - 1) * n - (q0 - 1) * q0 + (n - q0) * (a >> 6); // (an arithmetic shift: floor)
+        }
     }
     return per_head * p.nh;
 }
@@ -185,6 +197,8 @@ struct Walker {
     int seq_begin; // index on the line of its first block
     int n_blocks;  // its blocks (all heads)
     SeqGeom g;
+    int qb, qb_begin; // a row block at or before the last position asked for, and its first unit inside the sequence: positions
+                      // only move forward, so a search starts here instead of at row block 0
 };
 
 struct Fragment {
@@ -204,14 +218,17 @@ __device__ __forceinline__ bool locate(const PrefillParams &p, Walker &w, int &p
             ++w.a;
             w.g = seq_geom(p, w.a);
             w.n_blocks = seq_blocks(p, w.g);
+            w.qb = w.qb_begin = 0;
         }
-        int x = pos - w.seq_begin;
-        int qb = 0, nb = tile_blocks(w.g, 0);
+        int x = pos - w.seq_begin - w.qb_begin;
+        int qb = w.qb, nb = tile_blocks(w.g, qb);
         while (x >= (nb + kTileCost) * p.nh && qb + 1 < w.g.n_qb) {
             x -= (nb + kTileCost) * p.nh;
+            w.qb_begin += (nb + kTileCost) * p.nh;
             ++qb;
             nb = tile_blocks(w.g, qb);
         }
+        w.qb = qb;
         const int h = min(x / (nb + kTileCost), p.nh - 1);
         const int b0 = x - h * (nb + kTileCost);
         if (b0 >= nb + kTileCost) {
@@ -298,9 +315,9 @@ __global__ void __launch_bounds__(kThreads, 2)
         for (int a = tid; a < p.n_seqs; a += kThreads) {
             const SeqGeom g = seq_geom(p, a);
             mine += seq_blocks(p, g);
-            for (int qb = g.window > 0 ? 0 : g.n_qb - 1; qb >= 0 && qb < g.n_qb; ++qb) { // (without a window the last is longest)
-                mine_max = max(mine_max, tile_blocks(g, qb));
-            }
+            // (with a window: what a tile can reach, it only sizes the pieces)
+            const int reach = g.window > 0 ? (g.window + kBlockM - 1 + kBlockN - 1) / kBlockN + 1 : 1 << 30;
+            mine_max = max(mine_max, g.n_qb > 0 ? min((g.kv_len + kBlockN - 1) / kBlockN, reach) : 0);
         }
 #pragma unroll
         for (int d = 16; d > 0; d >>= 1) {
@@ -365,6 +382,7 @@ __global__ void __launch_bounds__(kThreads, 2)
     walker.seq_begin = s_sched[13];
     walker.g = seq_geom(p, walker.a);
     walker.n_blocks = seq_blocks(p, walker.g);
+    walker.qb = walker.qb_begin = 0;
     Fragment first_fragment;
     Walker first_walker = walker;
     {

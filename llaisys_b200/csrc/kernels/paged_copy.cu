@@ -381,6 +381,87 @@ __global__ void __launch_bounds__(256)
     }
 }
 
+// The same for head rows of at most 32 16-byte pieces: `lanes` (a power of two) neighbouring lanes share a head row, one
+// piece each, which stays in registers between the norm and the store; a thread keeps kItems rows in flight.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+    paged_norm_append_pieces_kernel(unsigned char *__restrict__ k_pool, unsigned char *__restrict__ v_pool, NormAppendArgs a,
+                                    const int32_t *__restrict__ table, CopyGeom g, int32_t d, int32_t dv, int64_t v_head_stride_b,
+                                    int64_t v_token_stride_b, int32_t lanes, int32_t max_blocks, int32_t *error_flag) {
+    using P = Pack<T, VEC>;
+    constexpr int kItems = 2;
+    asm volatile("griddepcontrol.wait;\n" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    const int32_t heads = a.nh + 2 * g.nkvh, total = int32_t(a.n_rows) * heads;
+    const int32_t per_block = int32_t(blockDim.x) / lanes;
+    const int32_t item0 = int32_t(blockIdx.x) * per_block * kItems + int32_t(threadIdx.x) / lanes;
+    const int32_t piece = int32_t(threadIdx.x) % lanes, at = piece * VEC;
+    P x[kItems];
+    int32_t row[kItems], head[kItems];
+    bool holds[kItems];
+    float ss[kItems];
+#pragma unroll
+    for (int u = 0; u < kItems; ++u) {
+        const int32_t item = item0 + u * per_block;
+        row[u] = item / heads;
+        head[u] = item - row[u] * heads;
+        const bool is_q = head[u] < a.nh, is_v = head[u] >= a.nh + g.nkvh;
+        holds[u] = item < total && at < (is_v ? dv : d);
+        if (holds[u]) {
+            const int64_t part = is_q ? a.q_at + int64_t(head[u]) * d
+                                      : (is_v ? a.v_at + int64_t(head[u] - a.nh - g.nkvh) * dv : a.k_at + int64_t(head[u] - a.nh) * d);
+            x[u] = *reinterpret_cast<const P *>(static_cast<const T *>(a.proj) + int64_t(row[u]) * a.row_stride + part + at);
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < kItems; ++u) {
+        ss[u] = 0.f;
+        if (holds[u]) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                ss[u] = fmaf(to_f32(x[u].v[e]), to_f32(x[u].v[e]), ss[u]);
+            }
+        }
+        for (int o = lanes / 2; o > 0; o >>= 1) {
+            ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o);
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < kItems; ++u) {
+        if (!holds[u]) {
+            continue;
+        }
+        const bool is_q = head[u] < a.nh, is_v = head[u] >= a.nh + g.nkvh;
+        const T *w = is_v ? nullptr : static_cast<const T *>(is_q ? a.q_norm : a.k_norm);
+        if (w != nullptr) {
+            const float inv = rsqrtf(ss[u] / float(d) + a.eps);
+            const P ww = *reinterpret_cast<const P *>(w + at);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                x[u].v[e] = from_f32<T>(to_f32(x[u].v[e]) * inv * to_f32(ww.v[e]));
+            }
+        }
+        if (is_q) {
+            *reinterpret_cast<P *>(static_cast<T *>(a.q_out) + (int64_t(row[u]) * a.nh + head[u]) * d + at) = x[u];
+            if (piece == 0 && a.row_scale != nullptr) {
+                const T *proj = static_cast<const T *>(a.proj) + int64_t(row[u]) * a.row_stride;
+                a.row_scale[int64_t(row[u]) * a.nh + head[u]] =
+                    a.gate_at < 0 ? a.gate_scale : a.gate_scale / (1.f + expf(-to_f32(proj[a.gate_at + head[u]])));
+            }
+            continue;
+        }
+        int32_t page, slot;
+        if (!resolve_slot(table, g, a.seq_ids[row[u]], a.positions[row[u]], max_blocks, error_flag, page, slot)) {
+            continue;
+        }
+        const int32_t kvh = is_v ? head[u] - a.nh - g.nkvh : head[u] - a.nh;
+        const int64_t off = int64_t(page) * g.page_stride_b +
+                            (is_v ? int64_t(kvh) * v_head_stride_b + int64_t(slot) * v_token_stride_b
+                                  : int64_t(kvh) * g.head_stride_b + int64_t(slot) * g.token_stride_b);
+        *reinterpret_cast<P *>((is_v ? v_pool : k_pool) + off + int64_t(at) * int64_t(sizeof(T))) = x[u];
+    }
+}
+
 template <typename T>
 void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &a, int32_t max_blocks, int32_t *error_flag) {
     CopyGeom g{};
@@ -406,6 +487,23 @@ void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = 1;
+    constexpr int kPiece = 16 / int(sizeof(T));
+    const int32_t longest = d > dv ? d : dv;
+    // (small calls are latency-bound: there the kernel with a warp per head row has the shorter chain)
+    if (a.n_rows > 1024 && d % kPiece == 0 && dv % kPiece == 0 && longest <= 32 * kPiece && a.row_stride % kPiece == 0 && a.q_at % kPiece == 0 &&
+        a.k_at % kPiece == 0 && a.v_at % kPiece == 0 && wide && int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh) < (int64_t(1) << 31)) {
+        int32_t lanes = 1;
+        while (lanes * kPiece < longest) {
+            lanes *= 2;
+        }
+        const int64_t per_block = 2 * (256 / lanes);
+        cfg.gridDim = dim3(unsigned((warps + per_block - 1) / per_block)); // (`warps` = head rows)
+        LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_norm_append_pieces_kernel<T, kPiece>, static_cast<unsigned char *>(kv.k_base),
+                                              static_cast<unsigned char *>(kv.v_base), NormAppendArgs(a), kv.block_table, g, d, dv,
+                                              kv.vHeadStride() * int64_t(sizeof(T)), kv.vTokenStride() * int64_t(sizeof(T)), lanes,
+                                              max_blocks, error_flag));
+        return;
+    }
     auto kernel = wide ? paged_norm_append_kernel<T, kVec> : paged_norm_append_kernel<T, 1>;
     LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, static_cast<unsigned char *>(kv.k_base),
                                           static_cast<unsigned char *>(kv.v_base), NormAppendArgs(a), kv.block_table, g, d, dv,

@@ -157,16 +157,17 @@ def test_window_over_a_long_sequence_on_the_fast_kernels(cuda_device):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("d,dv", [(64, 64), (20, 12), (128, 128), (13, 9)])
-def test_norm_append(cuda_device, dtype, d, dv):
+@pytest.mark.parametrize("d,dv", [(64, 64), (20, 12), (128, 128), (13, 9), (24, 40), (256, 8)])
+@pytest.mark.parametrize("rows", [37, 1100])
+def test_norm_append(cuda_device, dtype, d, dv, rows):
     """q and k per head over their own root mean square, gates to factors, v untouched; k and v arrive in their pages."""
-    nh, nkvh, rows, eps = 4, 2, 37, 1e-3
+    nh, nkvh, eps = 4, 2, 1e-3
     g = torch.Generator().manual_seed(d)
-    cache = llaisys.PagedKVCache.with_layers(8, [(1, 8, 8), (nkvh, d, dv)], dtype=LL[dtype], max_seqs=2)
+    cache = llaisys.PagedKVCache.with_layers(rows // 16 + 3, [(1, 8, 8), (nkvh, d, dv)], dtype=LL[dtype], max_seqs=2)
     seq = cache.add_seq()
     cache.reserve(seq, rows)
     cache.flush()
-    width = nh * d + nkvh * d + nkvh * dv + nh + 3
+    width = (nh * d + nkvh * d + nkvh * dv + nh + 10) // 8 * 8
     proj = (torch.randn(rows, width, generator=g) * 0.3).to(dtype)
     qn, kn = ((1 + 0.3 * torch.randn(d, generator=g)).to(dtype) for _ in range(2))
     q_out = torch.zeros(rows, nh, d, dtype=dtype, device="cuda")
@@ -184,7 +185,7 @@ def test_norm_append(cuda_device, dtype, d, dv):
     gates = p[:, (nh + nkvh) * d + nkvh * dv:][:, :nh]
     assert (factor.cpu().double() - 0.37 * torch.sigmoid(gates)).abs().max().item() <= 1e-6
     # k and v as attention sees them: a query of one huge coordinate picks one key, whose value comes back
-    for row in (0, 15, 16, 36):
+    for row in (0, 15, 16, rows - 1):
         q = torch.zeros(1, nh, d, dtype=dtype)
         out = torch.zeros(1, nh, dv, dtype=dtype, device="cuda")
         cache.attention_dev(1, out, q.cuda(), i32([seq]), None, i32([row + 1]), n_seqs=1, total_q=1, max_q_len=1,
