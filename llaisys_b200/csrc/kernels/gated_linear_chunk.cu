@@ -593,11 +593,22 @@ __global__ void gated_linear_scan_kernel(GatedLinearArgs a, int segs, int seg_le
     const int n = (len + seg_len - 1) / seg_len, d = int(e / a.dv);
     float *slot = a.segments + (int64_t(i) * a.heads + head) * segs * stride;
     float s = a.kv_lens[i] == len ? 0.f : a.state[int64_t(a.seq_ids[i]) * a.slot_stride + int64_t(head) * size + e];
-    for (int j = 0; j < n; ++j) {
-        float *p = slot + j * stride;
-        const float add = j + 1 < n ? p[e] : 0.f, decay = j + 1 < n ? ex2(p[size + d]) : 0.f;
-        p[e] = s;
-        s = fmaf(s, decay, add);
+    constexpr int kAtOnce = 8; // segments fetched together: the sums are a chain, the loads are not
+    for (int j0 = 0; j0 < n; j0 += kAtOnce) {
+        float add[kAtOnce], decay[kAtOnce];
+#pragma unroll
+        for (int u = 0; u < kAtOnce; ++u) {
+            const bool used = j0 + u + 1 < n; // (nothing starts from what the last segment leaves)
+            add[u] = used ? slot[(j0 + u) * stride + e] : 0.f;
+            decay[u] = used ? slot[(j0 + u) * stride + size + d] : 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < kAtOnce; ++u) {
+            if (j0 + u < n) {
+                slot[(j0 + u) * stride + e] = s;
+                s = fmaf(s, ex2(decay[u]), add[u]);
+            }
+        }
     }
 }
 
