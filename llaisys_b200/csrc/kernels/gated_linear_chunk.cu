@@ -52,7 +52,7 @@ struct ChunkSmem { // byte offsets
     static constexpr int kA = kQh + (kOperands > kOutputs ? kOperands : kOutputs); // scores high, low [64][64] bf16, swizzled
     static constexpr int kG = kA + 2 * kTile * kTile * 2;       // output gates of the tile [64][DV] bf16
     static constexpr int kPart = kG + kTile * DV * 2;           // decay sums of the token parts [4][DK] f32
-    static constexpr int kRef = kPart + 4 * DK * 4;             // per channel: the reference m, and the factors' exponents of S
+    static constexpr int kRef = kPart + 4 * DK * 4;             // per channel: the reference m, and the factors of S
     static constexpr int kIn = kRef + DK * 4;                   // on the way into its frame
     static constexpr int kOut = kIn + DK * 4;                   // and out of it
     static constexpr int kZ = kOut + DK * 4;                    // low-rank decay inputs [64][rank, padded to 16] bf16
@@ -61,10 +61,11 @@ struct ChunkSmem { // byte offsets
 __device__ __forceinline__ uint32_t swz(int row, int chunk, int row_bytes) { // 16-byte chunk `chunk` of row `row`
     return uint32_t(row * row_bytes + ((chunk ^ (row & 7)) << 4));
 }
-// x0, x1 as packed bf16 (x0 low half) and what is left of them after that rounding
+// x0, x1 as two packed pairs of bf16 (x0 in the low half): their upper halves as they are, and the rest rounded
 __device__ __forceinline__ void split2(float x0, float x1, uint32_t &hi, uint32_t &lo) {
-    hi = pack2<true>(x0, x1);
-    lo = pack2<true>(x0 - __uint_as_float(hi << 16), x1 - __uint_as_float(hi & 0xffff0000u));
+    const uint32_t u0 = __float_as_uint(x0), u1 = __float_as_uint(x1);
+    hi = __byte_perm(u0, u1, 0x7632);
+    lo = pack2<true>(x0 - __uint_as_float(u0 & 0xffff0000u), x1 - __uint_as_float(u1 & 0xffff0000u));
 }
 // 2^x without `volatile` (free to be interleaved); ex2(-inf) = 0
 __device__ __forceinline__ float ex2(float x) {
@@ -291,8 +292,8 @@ __global__ void __launch_bounds__(DV * 4)
                 auto set = [&](int stop) {
                     const float ref = s_b[b_at((p0 + stop - 1) / 2, tid)], last_sum = s_b[b_at(stop - 1, tid)];
                     s_ref[tid] = ref;
-                    s_in[tid] = ref - base;
-                    s_out[tid] = last_sum - ref;
+                    s_in[tid] = ex2(ref - base);
+                    s_out[tid] = ex2(last_sum - ref);
                     return last_sum - base;
                 };
                 float total = 0.f;
@@ -364,7 +365,7 @@ __global__ void __launch_bounds__(DV * 4)
             // ---- S^ = 2^m S ------------------------------------------------------------------------------------------
 #pragma unroll
             for (int nt = 0; nt < kNt; ++nt) {
-                const float f0 = ex2(s_in[d0 + nt * 8 + 2 * q4]), f1 = ex2(s_in[d0 + nt * 8 + 2 * q4 + 1]);
+                const float f0 = s_in[d0 + nt * 8 + 2 * q4], f1 = s_in[d0 + nt * 8 + 2 * q4 + 1];
                 s[nt][0] *= f0;
                 s[nt][1] *= f1;
                 s[nt][2] *= f0;
@@ -462,7 +463,7 @@ __global__ void __launch_bounds__(DV * 4)
             }
 #pragma unroll
             for (int nt = 0; nt < kNt; ++nt) {
-                const float f0 = ex2(s_out[d0 + nt * 8 + 2 * q4]), f1 = ex2(s_out[d0 + nt * 8 + 2 * q4 + 1]);
+                const float f0 = s_out[d0 + nt * 8 + 2 * q4], f1 = s_out[d0 + nt * 8 + 2 * q4 + 1];
                 s[nt][0] *= f0;
                 s[nt][1] *= f1;
                 s[nt][2] *= f0;
