@@ -11,9 +11,9 @@ from oracle import vozozen as oracle
 from tests import vozozen_cases as cases
 
 pytestmark = pytest.mark.gpu
-DT = {"f32": llaisys.DataType.F32, "bf16": llaisys.DataType.BF16}
+DT = {"f32": llaisys.DataType.F32, "f16": llaisys.DataType.F16, "bf16": llaisys.DataType.BF16}
 # relative rms error of a row of logits (mean taken off): float32 rounding; bfloat16 rounding through a few layers
-TOL = {"f32": 2e-5, "bf16": 0.06}
+TOL = {"f32": 2e-5, "f16": 0.01, "bf16": 0.06}
 
 
 def make(cfg, w, dtype):
@@ -41,7 +41,7 @@ def ready(request, cuda_device):
     return request.param, cfg, w, toks, logits, streams
 
 
-@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("dtype", ["f32", "f16", "bf16"])
 def test_whole_prompt_and_every_layer(ready, dtype):
     name, cfg, w, toks, logits, streams = ready
     model = make(cfg, w, dtype)
