@@ -1,7 +1,8 @@
 /*
  * llaisys C ABI -- token mixers beyond plain causal attention, on device buffers and an explicit stream: caches whose
- * layers differ in shape, attention with a sliding window and an output factor per head, the position-free norm + append
- * in front of it, and gated linear attention with recurrent state. NVIDIA devices. No counterpart in the reference.
+ * layers differ in shape, attention with a sliding window (that can keep a sequence's first tokens) and an output factor per
+ * head, the norm / rotation + append in front of it, gated linear attention and the gated delta rule with recurrent state.
+ * NVIDIA devices. No counterpart in the reference.
  * Status codes as in paged_kv.h; as for every ...Dev call there: no host validation of index arrays, no staging copy.
  */
 #ifndef LLAISYS_MIXERS_H
@@ -23,7 +24,8 @@ LLAISYS_API int llaisysPagedKVCreateLayers(llaisysPagedKV_t *kv_out, llaisysDevi
 /* One projection row per token, [n_rows, row_stride] of the cache's dtype, holding q [nh, k_dim] at element q_at, k
  * [nkvh, k_dim] at k_at, v [nkvh, v_dim] at v_at and (gate_at >= 0) one gate number per query head. q and k heads are
  * divided by their root mean square (eps inside the root) and weighted with q_norm / k_norm [k_dim] (NULL: left as they
- * are); q goes to q_out [n_rows, nh, k_dim], k and v to token positions[i] of sequence seq_ids[i], and row_scale
+ * are); then, with rot_dims > 0, dims i and i + rot_dims / 2 (i < rot_dims / 2) of each turn by the angle whose cosine and
+ * sine are rot_table[row][i] (llaisysRotaryTableDev); q goes to q_out [n_rows, nh, k_dim], k and v to token positions[i] of sequence seq_ids[i], and row_scale
  * [n_rows, nh] (NULL: none) becomes gate_scale * sigmoid(gate) -- gate_scale alone without a gate. */
 struct LlaisysNormAppend {
     const void *proj;
@@ -33,20 +35,24 @@ struct LlaisysNormAppend {
     void *q_out;
     float *row_scale;
     const int32_t *seq_ids_dev, *positions_dev;
-    size_t n_rows, nh;
+    size_t n_rows, nh, rot_dims;
+    const float *rot_table; /* [n_rows, rot_dims / 2, 2] */
 };
+/* table[row, i] = (cos, sin)(positions[row] * freq[i]), i < half, all on the device */
+LLAISYS_API int llaisysRotaryTableDev(llaisysDeviceType_t device_type, int device_id, float *table, const int32_t *positions_dev,
+                                      const float *freq_dev, size_t n_rows, size_t half, llaisysStream_t stream);
 LLAISYS_API int llaisysPagedKVNormAppendDev(llaisysPagedKV_t kv, size_t layer, const struct LlaisysNormAppend *args,
                                             llaisysStream_t stream);
 
 /* Attention over the pages with options. q_starts_dev NULL: one query per sequence (total_q = n_seqs); else ragged chunks as
- * in llaisysPagedAttentionPrefillDev. window > 0: the query at position i sees keys j with 0 <= i - j < window.
- * row_scale [total_q, nh] (device, may be NULL) multiplies every head's output; row r of out starts at r * row_stride
+ * in llaisysPagedAttentionPrefillDev. window > 0: the query at position i sees keys j <= i with i - j < window or
+ * j < keep_first. row_scale [total_q, nh] (device, may be NULL) multiplies every head's output; row r of out starts at r * row_stride
  * elements (0: packed rows of nh * v_dim). */
 LLAISYS_API int llaisysPagedAttentionOptDev(llaisysPagedKV_t kv, size_t layer, void *out, const void *q,
                                             const int32_t *seq_ids_dev, const int32_t *q_starts_dev, const int32_t *kv_lens_dev,
                                             size_t n_seqs, size_t total_q, size_t max_q_len, size_t max_kv_len, size_t nh,
-                                            float scale, size_t window, const float *row_scale, size_t row_stride,
-                                            llaisysStream_t stream);
+                                            float scale, size_t window, size_t keep_first, const float *row_scale,
+                                            size_t row_stride, llaisysStream_t stream);
 
 /* Gated linear attention. Per head, with state S [dk, dv] in f32 (row-major, slot s of the sequence in seq_ids at
  * state + s * slot_stride + head * dk * dv):
@@ -78,6 +84,48 @@ LLAISYS_API int llaisysGatedLinearDev(llaisysDeviceType_t device_type, int devic
                                       const struct LlaisysGatedLinear *args, int decode, llaisysStream_t stream);
 /* Floats of scratch_segments that serve every call of these sizes (0: such calls are never cut). */
 LLAISYS_API size_t llaisysGatedLinearSegmentFloats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
+
+/* Gated delta rule. q, k (kv_heads x dk) and v (heads x dv) of a projection row pass a causal convolution over time of `taps`
+ * taps per channel (conv_q, conv_k, conv_v [channels, taps], the last tap is the current token's, zeros before a sequence's
+ * start), then silu; q and k of a head become x / sqrt(sum(x^2) + unit_eps), q also times q_scale. Head h reads q/k head
+ * h / (heads / kv_heads). Per head, with state S [dk, dv] in f32:
+ *     S' = diag(g_t) S_{t-1},  u_t = beta_t (v_t - S'^T k_t),  S_t = S' + k_t u_t^T,  o_t = S_t^T q_t
+ *     beta_t = sigmoid(b_t),   g_t = exp(-exp(a_log_h) * softplus(x_t + dt_bias))
+ *     out_t = o_t / sqrt(mean(o_t^2) + eps) * norm_w * (gate_silu ? silu : sigmoid)(gate_t)
+ * x_t: with decay_w NULL one number per head, at element a_at of the row (dt_bias [heads]); else one per head and key channel,
+ * decay_w z_t with decay_w [heads * dk, rank] (rows decay_ld apart) and z_t the `rank` numbers at a_at (dt_bias [heads * dk]).
+ * b_t: heads numbers at b_at. gate: heads x dv at gate + r * gate_stride. All but state and scratch are of `dtype`.
+ * state: slot s of a sequence holds [heads][dk][dv], then the convolutions' inputs [taps][2 kv_heads dk + heads dv] (position p
+ * at p mod taps); llaisysGatedDeltaSizes gives its floats. Sequences, rows and `decode` as for LlaisysGatedLinear. scratch
+ * (16-byte aligned) is needed by chunks (decode = 0); with scratch_segments long runs are cut into segments that run in
+ * parallel. */
+struct LlaisysGatedDelta {
+    const void *proj;
+    int64_t row_stride, q_at, k_at, v_at, b_at, a_at;
+    const void *conv_q, *conv_k, *conv_v;
+    const void *decay_w;
+    int64_t decay_ld;
+    const void *a_log, *dt_bias, *norm_w, *gate;
+    int64_t gate_stride;
+    int gate_silu;
+    float q_scale, eps, unit_eps;
+    size_t taps, heads, kv_heads, dk, dv, rank;
+    float *state;
+    int64_t slot_stride;
+    const int32_t *seq_ids_dev, *q_starts_dev, *kv_lens_dev;
+    size_t n_seqs, n_rows, max_q_len;
+    void *out;
+    int64_t out_stride;
+    float *scratch;
+    size_t scratch_floats;
+    float *scratch_segments;
+    size_t scratch_segment_floats;
+};
+LLAISYS_API int llaisysGatedDeltaDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype,
+                                     const struct LlaisysGatedDelta *args, int decode, llaisysStream_t stream);
+/* Floats of a sequence's state, of `scratch` for n_rows rows and of `scratch_segments` (any pointer may be NULL). */
+LLAISYS_API void llaisysGatedDeltaSizes(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t kv_heads, size_t dk, size_t dv,
+                                        size_t taps, size_t *state_floats, size_t *scratch_floats, size_t *segment_floats);
 
 #ifdef __cplusplus
 }

@@ -55,6 +55,12 @@ LLAISYS_API int llaisysModelDecodeLoop(struct LlaisysModel *model, const int32_t
 LLAISYS_API int llaisysModelLastLogits(struct LlaisysModel *model, float *out_host, size_t capacity_floats);
 LLAISYS_API double llaisysModelLastLoopMs(struct LlaisysModel *model);
 
+/* Development aid, for models with an f32 residual stream: copies the stream after every layer run of the next steps to host
+ * memory, [runs, rows, width]. Takes effect until called again; LLAISYS_E_INVALID from LayerStream when the last step was not
+ * recorded. */
+LLAISYS_API int llaisysModelRecordStream(struct LlaisysModel *model, int enable);
+LLAISYS_API int llaisysModelLayerStream(struct LlaisysModel *model, float *out_host, size_t capacity_floats, size_t *floats_out);
+
 #ifdef __cplusplus
 }
 #endif

@@ -49,11 +49,6 @@ struct LlaisysVozozenMeta {
 /* NULL on failure (message on stderr and in llaisysGetLastError). */
 LLAISYS_API struct LlaisysModel *llaisysVozozenModelCreate(const struct LlaisysVozozenMeta *meta, llaisysDeviceType_t device,
                                                            int device_id);
-/* Development aid: copies the f32 residual stream after every layer run of the next steps to host memory. Takes effect
- * until called again; LLAISYS_E_INVALID from LayerStream when the last step was not recorded. */
-LLAISYS_API int llaisysVozozenModelRecordStream(struct LlaisysModel *model, int enable);
-LLAISYS_API int llaisysVozozenModelLayerStream(struct LlaisysModel *model, float *out_host, size_t capacity_floats,
-                                               size_t *floats_out);
 
 #ifdef __cplusplus
 }

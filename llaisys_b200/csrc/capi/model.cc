@@ -1,4 +1,5 @@
 // extern "C" thunks of the generic model API and of the families that have no older ABI of their own.
+#include "llaisys/models/doderax.h"
 #include "llaisys/models/model.h"
 #include "llaisys/models/vozozen.h"
 #include "llaisys/paged_kv.h"
@@ -10,6 +11,18 @@
 
 using llaisys::capi::guarded;
 using llaisys::capi::null_model;
+
+template <typename Model, typename Meta>
+static LlaisysModel *create_model(const char *function, const Meta *meta, llaisysDeviceType_t device, int device_id) {
+    LlaisysModel *model = nullptr;
+    const int rc = meta == nullptr ? null_model()
+                                   : guarded([&] { model = new LlaisysModel(std::make_unique<Model>(*meta, device, device_id)); });
+    if (rc != LLAISYS_OK) {
+        std::cerr << "[ERROR] " << function << ": " << llaisysGetLastError() << std::endl;
+        return nullptr;
+    }
+    return model;
+}
 
 extern "C" {
 
@@ -81,30 +94,17 @@ int llaisysModelLastLogits(LlaisysModel *model, float *out_host, size_t capacity
 double llaisysModelLastLoopMs(LlaisysModel *model) { return model ? model->impl->lastLoopMs() : 0.0; }
 
 LlaisysModel *llaisysVozozenModelCreate(const LlaisysVozozenMeta *meta, llaisysDeviceType_t device, int device_id) {
-    LlaisysModel *model = nullptr;
-    const int rc = meta == nullptr ? null_model() : guarded([&] {
-        model = new LlaisysModel(std::make_unique<llaisys::models::Vozozen>(*meta, device, device_id));
-    });
-    if (rc != LLAISYS_OK) {
-        std::cerr << "[ERROR] llaisysVozozenModelCreate: " << llaisysGetLastError() << std::endl;
-        return nullptr;
-    }
-    return model;
+    return create_model<llaisys::models::Vozozen>("llaisysVozozenModelCreate", meta, device, device_id);
+}
+LlaisysModel *llaisysDoderaxModelCreate(const LlaisysDoderaxMeta *meta, llaisysDeviceType_t device, int device_id) {
+    return create_model<llaisys::models::Doderax>("llaisysDoderaxModelCreate", meta, device, device_id);
 }
 
-static llaisys::models::Vozozen &vozozen(LlaisysModel *model) {
-    auto *v = dynamic_cast<llaisys::models::Vozozen *>(model->impl.get());
-    if (v == nullptr) {
-        throw llaisys::kv::StatusError(LLAISYS_E_INVALID, "model: not a vozozen model");
-    }
-    return *v;
+int llaisysModelRecordStream(LlaisysModel *model, int enable) {
+    return model ? guarded([&] { model->impl->recordStream(enable != 0); }) : null_model();
 }
-int llaisysVozozenModelRecordStream(LlaisysModel *model, int enable) {
-    return model ? guarded([&] { vozozen(model).recordStream(enable != 0); }) : null_model();
-}
-int llaisysVozozenModelLayerStream(LlaisysModel *model, float *out_host, size_t capacity_floats, size_t *floats_out) {
-    return model && floats_out ? guarded([&] { *floats_out = vozozen(model).layerStream(out_host, capacity_floats); })
-                               : null_model();
+int llaisysModelLayerStream(LlaisysModel *model, float *out_host, size_t capacity_floats, size_t *floats_out) {
+    return model && floats_out ? guarded([&] { *floats_out = model->impl->layerStream(out_host, capacity_floats); }) : null_model();
 }
 
 } // extern "C"

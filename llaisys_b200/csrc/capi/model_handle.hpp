@@ -2,6 +2,7 @@
 // either.
 #pragma once
 
+#include "../models/doderax.hpp"
 #include "../models/qwen2.hpp"
 #include "../models/vozozen.hpp"
 

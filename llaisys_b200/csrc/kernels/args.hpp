@@ -70,6 +70,7 @@ struct AttnBatch {
     int32_t max_kv_len = 0;
     int32_t nh = 0;
     int32_t window = 0; // > 0: a query at position i sees keys j with 0 <= i - j < window; 0: all earlier keys
+    int32_t keep_first = 0; // with a window: keys j < keep_first stay visible behind it (j <= i)
 };
 
 // Output selection: `out` [total_q, nh, d] in the KV dtype, or `part` float [total_q, nh, d + 2] holding the
@@ -107,15 +108,19 @@ struct AttnScratch {
     int32_t *error_flag = nullptr; // set non-zero when a kernel skipped an out-of-range page / position
 };
 
-// K1c: what enters attention without positions, fused: from a packed projection row [.. q | k | v .. gate ..] the per-head
-// RMS norm of q and k (one weight of `d` for all heads), k and v into their page slots, q to a packed tensor, and the
-// output gate of every head turned into a factor for the attention kernel's epilogue.
+// K1c: what enters attention, fused: from a packed projection row [.. q | k | v .. gate ..] the per-head RMS norm of q and k
+// (one weight of `d` for all heads), the rotation of their first rot_dims dimensions, k and v into their page slots, q to a
+// packed tensor, and the output gate of every head turned into a factor for the attention kernel's epilogue. Norm, rotation
+// and gate are optional.
 struct NormAppendArgs {
     const void *proj = nullptr; // [n_rows, row_stride] elements of the cache's dtype
     int64_t row_stride = 0;
     int64_t q_at = 0, k_at = 0, v_at = 0, gate_at = 0; // first element of each part in a row; gate_at < 0: no gate
     const void *q_norm = nullptr, *k_norm = nullptr;   // [d], cache dtype; null = no norm
     float eps = 0.f;
+    // dims i and i + rot_dims / 2 (i < rot_dims / 2) turn by the angle whose (cos, sin) is rot_table[row][i] (rotary_table)
+    int32_t rot_dims = 0;
+    const float *rot_table = nullptr; // [n_rows, rot_dims / 2, 2]
     void *q_out = nullptr;      // [n_rows, nh, d]
     float *row_scale = nullptr; // [n_rows, nh] = gate_scale * sigmoid(gate)
     float gate_scale = 1.f;
@@ -150,6 +155,45 @@ struct GatedLinearArgs {
     // scratch for cutting long runs into segments that run in parallel (gated_linear_segment_floats); null: never cut
     float *segments = nullptr;
     size_t segment_floats = 0;
+};
+
+// Gated delta rule over one packed projection. q, k (kv_heads x dk) and v (heads x dv) pass a causal convolution of `taps` taps
+// per channel and silu; q and k become unit vectors x / sqrt(sum x^2 + unit_eps), q times q_scale; head h reads q/k head
+// h / (heads / kv_heads). Per head a state S [dk, dv]:
+//   S' = diag(g_t) S_{t-1},  u_t = beta_t (v_t - S'^T k_t),  S_t = S' + k_t u_t^T,  o_t = S_t^T q_t
+//   beta_t = sigmoid(b_t),  log g_t = -exp(A_log_h) softplus(x_t + dt_bias)
+// x_t: one number per head (decay_w null: at a_at of the row), or per head and key channel, decay_w z_t with the `rank` numbers
+// z_t at a_at. out_t = rms_norm(o_t, norm) * gate(y_t), y_t heads x dv at `gate`.
+struct GatedDeltaArgs {
+    const void *proj = nullptr; // [n_rows, row_stride], model dtype
+    int64_t row_stride = 0;
+    int64_t q_at = 0, k_at = 0, v_at = 0, b_at = 0, a_at = 0;
+    const void *conv_q = nullptr, *conv_k = nullptr, *conv_v = nullptr; // [channels, taps]; the last tap is the current token's
+    int32_t taps = 0;
+    const void *decay_w = nullptr; // [heads * dk, rank], rows decay_ld apart; null: one decay per head
+    int64_t decay_ld = 0;
+    const void *a_log = nullptr;   // [heads]
+    const void *dt_bias = nullptr; // [heads] or [heads * dk]
+    const void *norm_w = nullptr;  // [dv]
+    const void *gate = nullptr;    // row r, head h: gate + r * gate_stride + h * dv
+    int64_t gate_stride = 0;
+    int32_t gate_silu = 0;         // 1: silu(y), 0: sigmoid(y)
+    float q_scale = 1.f, eps = 0.f, unit_eps = 1e-6f;
+    int32_t heads = 0, kv_heads = 0, dk = 0, dv = 0, rank = 0;
+    // slot s: the heads' matrices [heads][dk][dv], then convolution inputs [taps][2 kv_heads dk + heads dv]: position p at
+    // p mod taps
+    float *state = nullptr;
+    int64_t slot_stride = 0;
+    // the batch, as in GatedLinearArgs
+    const int32_t *seq_ids = nullptr, *q_starts = nullptr, *kv_lens = nullptr;
+    int32_t n_seqs = 0, n_rows = 0, max_q_len = 0;
+    void *out = nullptr; // row r, head h: out + r * out_stride + h * dv, model dtype
+    int64_t out_stride = 0;
+    float *scratch = nullptr; // chunk only, 16-byte aligned (gated_delta_scratch_floats)
+    size_t scratch_floats = 0;
+    float *segments = nullptr; // see gated_delta_segment_floats; null: never cut
+    size_t segment_floats = 0;
+    LLAISYS_ARGS_FN int32_t channels() const { return 2 * kv_heads * dk + heads * dv; }
 };
 
 using stream_t = void *;

@@ -86,9 +86,9 @@ struct TmaDecodeParams {
     char *pool_k;                           // K tile of (page 0, kv-head 0) of this layer
     long long page_stride_b, head_stride_b; // bytes between pages / kv-heads
     long long v_offset_b;                   // V tile - K tile of the same (page, kv-head)
-    // windowed instantiation: keys j >= kv_len - window take part (window > 0; as long as the cache's tables = none), output
+    // windowed instantiation: keys j >= kv_len - window and j < keep_first take part (window > 0; as long as the cache's tables = none), output
     // rows of a sequence lie out_stride elements apart and row r is multiplied by row_scale[r] (null: 1)
-    int32_t window;
+    int32_t window, keep_first;
     long long out_stride;
     const float *row_scale;
     // KV-range split across GPUs (exchange instantiation; out null, part = PeerSink::rows): a pair's finished rows
@@ -170,8 +170,12 @@ __device__ __forceinline__ int seq_kv_len(const int32_t *kv_lens, int max_tokens
     return min(max(kv_lens[s], 0), max_tokens);
 }
 
-// First page of the window of a sequence's newest token (windowed instantiation).
-__device__ __forceinline__ int first_page(const TmaDecodeParams &p, int kv_len) { return max(kv_len - p.window, 0) / kPage; }
+// Windowed instantiation: a sequence's pages on the line are [0, kept_pages) and those from the window of its newest token on;
+// `gap_pages` lie between. Page i of the line is page i or i + gap_pages of the sequence.
+__device__ __forceinline__ int kept_pages(const TmaDecodeParams &p) { return (p.keep_first + kPage - 1) / kPage; }
+__device__ __forceinline__ int gap_pages(const TmaDecodeParams &p, int kv_len) {
+    return max(max(kv_len - p.window, 0) / kPage - kept_pages(p), 0);
+}
 
 __device__ __forceinline__ Segment next_segment(Cursor &c, const int *cum, const TmaDecodeParams &p, const int32_t *kv_lens) {
     Segment sg;
@@ -223,8 +227,8 @@ __device__ __forceinline__ bool wait_or_abort(uint32_t bar, uint32_t parity, vol
 // warps of the last-arriving CTA); the others do not even contain its code -- this kernel's timing moves by a
 // microsecond with what is compiled around its hot loop.
 // kWin: sliding window, output row stride and output factor per head -- an instantiation of its own for the same reason.
-// The pages below a sequence's window are not part of the line at all: page indices of a segment count from the first
-// page the window reaches.
+// The pages between a sequence's kept first tokens and its window are not part of the line at all: page indices of a segment
+// count without them.
 template <bool kBf16, bool kXchg, bool kShare, bool kWin>
 __global__ void __launch_bounds__(kThreads, kCtasPerSm)
     paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ InlineIndex ix,
@@ -263,7 +267,7 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
     //    prefix sums (warp 0, in place) --------------------------------------------------------------------------
     for (int s = tid; s < p.n_seqs; s += kThreads) {
         const int len = seq_kv_len(kv_lens, p.max_tokens, s);
-        cum[s + 1] = (len + kPage - 1) / kPage - (kWin ? first_page(p, len) : 0);
+        cum[s + 1] = (len + kPage - 1) / kPage - (kWin ? gap_pages(p, len) : 0);
         rows[s] = seq_ids ? seq_ids[s] : s;
     }
     if (warp == kProducerWarp && lane == 0) {
@@ -369,8 +373,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
             if (sg.n <= 0) {
                 break; // inconsistent lengths: the consumers flag it
             }
-            const int page0_seg = kWin ? first_page(p, sg.kv_len) + sg.j0 : sg.j0; // the segment's first page in the sequence
-            const long long tbase = (long long)rows[sg.s] * p.table_stride + page0_seg;
+            const int kept = kWin ? kept_pages(p) : 0, gap = kWin ? gap_pages(p, sg.kv_len) : 0;
+            const long long tbase = (long long)rows[sg.s] * p.table_stride;
             // first page the kernel before this one on the stream may still be writing: the one holding token kv_len - 2
             const int guard_page = (max(sg.kv_len, 2) - 2) / kPage;
             for (int base = 0; base < sg.n && !dead; base += kIssueLanes) {
@@ -381,7 +385,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 // page order, so every wait ends. No more lanes than ring slots take part in a round: two lanes
                 // on one slot would wait for consecutive phases of the same barrier, and a parity wait cannot tell
                 // phase k + 1 from phase k - 1.
-                if (!waited && page0_seg + min(base + kIssueLanes, sg.n) > guard_page) {
+                const int line_end = sg.j0 + min(base + kIssueLanes, sg.n);
+                if (!waited && line_end + (line_end > kept ? gap : 0) > guard_page) {
                     // these copies reach the sequence's newest rows, which may come from the previous kernel on the
                     // stream (everything before it was there long ago)
                     grid_dependency_wait();
@@ -390,7 +395,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 const bool active = lane < kIssueLanes && base + lane < sg.n;
                 int ok = 1;
                 if (active) {
-                    int page = p.block_table[tbase + base + lane];
+                    const int line_page = sg.j0 + base + lane;
+                    int page = p.block_table[tbase + line_page + (kWin && line_page >= kept ? gap : 0)];
                     if (page < 0 || page >= p.num_pages) {
                         atomicOr(p.error_flag, kErrBadPage);
                         page = 0;
@@ -587,7 +593,7 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
         }
         // fused step: index in this segment of the pair's last page, which receives the new row; the warp that will
         // take that page fetches the row (K: lanes 0-15, V: lanes 16-31, 16 bytes each) and the page index now
-        const int seg_page0 = kWin ? first_page(p, sg.kv_len) + sg.j0 : sg.j0;
+        const int kept = kWin ? kept_pages(p) : 0, gap = kWin ? gap_pages(p, sg.kv_len) : 0;
         const int new_i = !kWin && p.k_new != nullptr ? (cum[sg.s + 1] - cum[sg.s]) - 1 - sg.j0 : -1;
         const bool brings_new = new_i >= 0 && new_i < sg.n && new_i % kConsumerWarps == warp;
         const uint32_t my_stage = stage_u32 + warp * kStageBytes;
@@ -614,8 +620,10 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 break;
             }
             const uint32_t tile = ring_u32 + slot * kSlotBytes;
-            const int n_valid = min(kPage, sg.kv_len - (seg_page0 + i) * kPage);
-            const int n_before = kWin ? sg.kv_len - p.window - (seg_page0 + i) * kPage : 0; // tokens of the page below the window
+            const int token0 = (sg.j0 + i + (kWin && sg.j0 + i >= kept ? gap : 0)) * kPage; // the page's first token
+            const int n_valid = min(kPage, sg.kv_len - token0);
+            // tokens of the page below the window, and how many of those are kept all the same
+            const int n_before = kWin ? sg.kv_len - p.window - token0 : 0, n_kept = kWin ? p.keep_first - token0 : 0;
             const bool patch = brings_new && i == new_i;
             if (patch) {
                 // the new row: over slot n_valid - 1 of the tile (swizzled like the TMA copy) and into the page itself
@@ -659,7 +667,8 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 mma_16816<kBf16>(sc, a, qf[ks][0], qf[ks][1]);
             }
             // online softmax in the log2 domain; this thread holds tokens g, g + 8 for heads 2*q4, 2*q4 + 1
-            const bool ok_lo = g < n_valid && (!kWin || g >= n_before), ok_hi = g + 8 < n_valid && (!kWin || g + 8 >= n_before);
+            const bool ok_lo = g < n_valid && (!kWin || g >= n_before || g < n_kept);
+            const bool ok_hi = g + 8 < n_valid && (!kWin || g + 8 >= n_before || g + 8 < n_kept);
             const float t0 = ok_lo ? sc[0] * p.scale_log2 : -INFINITY;
             const float t1 = ok_lo ? sc[1] * p.scale_log2 : -INFINITY;
             const float t2 = ok_hi ? sc[2] * p.scale_log2 : -INFINITY;
@@ -946,9 +955,10 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
         reason = "a window or an output scale goes with plain decode into an output tensor only";
         return -1;
     }
-    // (a window reaches at most window + page - 1 tokens' worth of pages)
+    // (a window reaches at most window + page - 1 tokens' worth of pages, the kept tokens keep_first + page - 1)
+    const int64_t reach = int64_t(batch.window) + batch.keep_first + (batch.keep_first > 0 ? 2 : 1) * (kPage - 1);
     const int grid = decode_grid_size(batch.n_seqs, kv.nkvh,
-                                      batch.window > 0 ? std::min(batch.max_kv_len, batch.window + kPage - 1) : batch.max_kv_len);
+                                      batch.window > 0 ? int(std::min<int64_t>(batch.max_kv_len, reach)) : batch.max_kv_len);
     const size_t n_pairs = size_t(batch.n_seqs) * kv.nkvh;
     if (scratch.partials == nullptr || scratch.counters == nullptr || scratch.error_flag == nullptr ||
         scratch.partials_floats < (size_t(grid) * (1 + kMergeWarps) + n_pairs) * group * kPartStride ||
@@ -993,6 +1003,7 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
     p.head_stride_b = kv.head_stride * 2;
     p.v_offset_b = static_cast<char *>(kv.v_base) - static_cast<char *>(kv.k_base);
     p.window = batch.window > 0 ? batch.window : p.max_tokens;
+    p.keep_first = batch.window > 0 ? batch.keep_first : 0;
     p.out_stride = out.row_stride != 0 ? out.row_stride : (long long)batch.nh * kD;
     p.row_scale = out.row_scale;
     p.xchg = PeerSink{};

@@ -59,7 +59,9 @@ __global__ void __launch_bounds__(kWarps * 32)
     const int kv_len = batch.kv_lens ? batch.kv_lens[seq] : batch.const_kv_len;
     int visible = kv_len - q_len + t + 1; // causal offset: query t sees keys j <= t + (kv_len - q_len)
     visible = visible < 0 ? 0 : (visible > kv_len ? kv_len : visible);
-    const int first = batch.window > 0 ? max(0, visible - batch.window) : 0; // the query sits at position visible - 1
+    // keys that are seen: [0, kept) and [kept + gap, visible); the query sits at position visible - 1
+    const int first = batch.window > 0 ? max(0, visible - batch.window) : 0;
+    const int kept = min(batch.keep_first, first), gap = first - kept;
     const int seq_row = batch.seq_ids ? batch.seq_ids[seq] : seq;
     const int kvh = h / (batch.nh / kv.nkvh);
 
@@ -79,9 +81,10 @@ __global__ void __launch_bounds__(kWarps * 32)
         acc[i] = 0.f;
     }
 
-    for (int base = first + warp * 32; base < visible; base += kWarps * 32) {
-        const int j = base + lane;
-        bool valid = j < visible;
+    const int n_keys = visible - gap;
+    for (int base = warp * 32; base < n_keys; base += kWarps * 32) {
+        const int j = base + lane + (base + lane >= kept ? gap : 0);
+        bool valid = base + lane < n_keys;
         int64_t row_off = 0, v_off = 0;
         if (valid) {
             const int blk = j / kv.page_size;
@@ -128,7 +131,7 @@ __global__ void __launch_bounds__(kWarps * 32)
         for (int i = 0; i < kMaxDimsPerLane; ++i) {
             acc[i] *= alpha;
         }
-        const int n_here = min(32, visible - base);
+        const int n_here = min(32, n_keys - base);
         for (int jj = 0; jj < n_here; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
             const int64_t off = __shfl_sync(0xffffffffu, v_off, jj);

@@ -127,9 +127,9 @@ struct PrefillParams {
     int32_t *error_flag;
     float *partials;   // [2 * gridDim.x][kPartialFloats]
     int32_t *counters; // [gridDim.x], zero between launches
-    // windowed instantiation: query t sees keys j > t + off - window; rows of out lie out_stride elements apart and head h
+    // windowed instantiation: query t sees keys j > t + off - window and j < keep_first; rows of out lie out_stride elements apart and head h
     // of row r is multiplied by row_scale[r * nh + h] (null: 1)
-    int32_t window;
+    int32_t window, keep_first;
     long long out_stride;
     const float *row_scale;
     int32_t out_wide;  // out is 32-byte aligned: rows are stored 32 bytes (a whole sector) per instruction
@@ -139,7 +139,8 @@ struct PrefillParams {
 
 struct SeqGeom {
     int q_start, q_len, kv_len, off, n_qb;
-    int window; // 0: none
+    int window;      // 0: none
+    int kept_blocks; // 64-key blocks that hold the first tokens a window keeps
 };
 
 __device__ __forceinline__ SeqGeom seq_geom(const PrefillParams &p, int a) {
@@ -157,25 +158,26 @@ __device__ __forceinline__ SeqGeom seq_geom(const PrefillParams &p, int a) {
     g.off = g.kv_len - g.q_len; // query t sees keys j <= t + off
     g.n_qb = (g.q_len + kBlockM - 1) / kBlockM;
     g.window = p.window;
+    g.kept_blocks = (p.keep_first + kBlockN - 1) / kBlockN;
     return g;
 }
 
 // keys any row of row block qb can see, and the 64-key blocks that hold them
 __device__ __forceinline__ int tile_kv_hi(const SeqGeom &g, int qb) { return min(g.kv_len, qb * kBlockM + kBlockM + g.off); }
-// first 64-key block that any row of the row block sees: 0, or where the window of the block's first row begins (its blocks
-// are counted from there)
-__device__ __forceinline__ int tile_first(const SeqGeom &g, int qb) {
-    return g.window > 0 ? max(qb * kBlockM + g.off - g.window + 1, 0) / kBlockN : 0;
+// key blocks that no row of the row block sees, between the blocks of the kept first tokens and the one where the window of
+// the block's first row begins; a tile's blocks are counted without them
+__device__ __forceinline__ int tile_gap(const SeqGeom &g, int qb) {
+    return g.window > 0 ? max(qb * kBlockM + g.off - g.window + 1 - g.kept_blocks * kBlockN, 0) / kBlockN : 0;
 }
 __device__ __forceinline__ int tile_blocks(const SeqGeom &g, int qb) {
-    return (tile_kv_hi(g, qb) + kBlockN - 1) / kBlockN - tile_first(g, qb);
+    return (tile_kv_hi(g, qb) + kBlockN - 1) / kBlockN - tile_gap(g, qb);
 }
 
 // units of the line that a sequence takes: per tile its blocks, then kTileCost units that stand for no block
 __device__ __forceinline__ int seq_blocks(const PrefillParams &p, const SeqGeom &g) {
     // the sum of tile_blocks over the row blocks in closed form (a loop over them, three times per CTA in front of all work,
     // was a large part of a launch over one long chunk): row block qb < n - 1 ends at key (qb + 1) 128 + off, the last one at
-    // kv_len; blocks before the window are 2 qb + floor((off - window + 1) / 64) where that is not negative
+    // kv_len; blocks in front of the window are 2 qb + floor((off - window + 1) / 64), less the kept ones, where that is not negative
     static_assert(kBlockM == 2 * kBlockN, "row blocks advance two key blocks");
     const int n = g.n_qb;
     if (n == 0) {
@@ -183,7 +185,7 @@ __device__ __forceinline__ int seq_blocks(const PrefillParams &p, const SeqGeom 
     }
     int per_head = (n - 1) * n + (n - 1) * ((g.off + kBlockN - 1) / kBlockN) + (g.kv_len + kBlockN - 1) / kBlockN + n * kTileCost;
     if (g.window > 0) {
-        const int a = g.off - g.window + 1, q0 = a >= 0 ? 0 : (-a + kBlockM - 1) / kBlockM;
+        const int a = g.off - g.window + 1 - g.kept_blocks * kBlockN, q0 = a >= 0 ? 0 : (-a + kBlockM - 1) / kBlockM;
         if (q0 < n) {
             per_head -= (n - 1) * n - (q0 - 1) * q0 + (n - q0) * (a >> 6); // (an arithmetic shift: floor)
         }
@@ -203,8 +205,8 @@ struct Walker {
 
 struct Fragment {
     int a, qb, h;
-    int b0, b1;     // key blocks [b0, b1) of the tile, counted from `first`
-    int first;      // the tile's first key block (tile_first)
+    int b0, b1;     // key blocks [b0, b1) of the tile, counted without its gap
+    int gap;        // tile_gap
     int tile_nblk;  // blocks of the whole tile
     int tile_begin; // index on the line of the tile's block 0
 };
@@ -243,7 +245,7 @@ __device__ __forceinline__ bool locate(const PrefillParams &p, Walker &w, int &p
         f.h = h;
         f.b0 = b0;
         f.tile_nblk = nb;
-        f.first = tile_first(w.g, qb);
+        f.gap = tile_gap(w.g, qb);
         f.b1 = min(nb, b0 + (piece_end - pos));
         f.tile_begin = pos - b0;
         return true;
@@ -316,7 +318,7 @@ __global__ void __launch_bounds__(kThreads, 2)
             const SeqGeom g = seq_geom(p, a);
             mine += seq_blocks(p, g);
             // (with a window: what a tile can reach, it only sizes the pieces)
-            const int reach = g.window > 0 ? (g.window + kBlockM - 1 + kBlockN - 1) / kBlockN + 1 : 1 << 30;
+            const int reach = g.window > 0 ? (g.window + kBlockM - 1 + kBlockN - 1) / kBlockN + 1 + g.kept_blocks : 1 << 30;
             mine_max = max(mine_max, g.n_qb > 0 ? min((g.kv_len + kBlockN - 1) / kBlockN, reach) : 0);
         }
 #pragma unroll
@@ -479,21 +481,23 @@ __global__ void __launch_bounds__(kThreads, 2)
             // current one is requested a whole group early: a table load issued when its block is due costs more than
             // a block takes (measured: about 1300 clocks between a V tile and the next K tile, on the critical path
             // of every block).
+            auto key_block = [&](int b) { return kWin && b >= walker.g.kept_blocks ? b + f.gap : b; };
             auto load_group = [&](int blk0) {
-                const int idx = blk0 * kPagesPerBlock + lane;
+                const int idx = kWin ? key_block(blk0 + lane / kPagesPerBlock) * kPagesPerBlock + lane % kPagesPerBlock
+                                     : blk0 * kPagesPerBlock + lane;
                 if (p.contiguous) {
                     return idx; // block b of the tensor is its tokens [64 b, 64 b + 64)
                 }
                 return idx < n_pages ? p.block_table[tbase + idx] : 0;
             };
-            int group = load_group(f.first + f.b0), next_group = load_group(f.first + f.b0 + 8);
+            int group = load_group(f.b0), next_group = load_group(f.b0 + 8);
             for (int i = 0; i < n && alive; ++i) {
                 const int gi = done + i, st = gi & 1;
-                const int first = (f.first + f.b0 + i) * kPagesPerBlock;
+                const int first = key_block(f.b0 + i) * kPagesPerBlock;
                 const int n_pg = min(kPagesPerBlock, n_pages - first);
                 if (i > 0 && (i & 7) == 0) {
                     group = next_group;
-                    next_group = load_group(f.first + f.b0 + i + 8);
+                    next_group = load_group(f.b0 + i + 8);
                 }
                 int page = __shfl_sync(0xffffffffu, group, (i & 7) * kPagesPerBlock + (lane & (kPagesPerBlock - 1)));
                 if (lane < n_pg && !p.contiguous && (page < 0 || page >= p.num_pages)) {
@@ -636,9 +640,10 @@ __global__ void __launch_bounds__(kThreads, 2)
                 }
                 tc_fence_after();
                 const uint32_t tmem_s = tmem_base + lane_base + kColS + buf * kBlockN;
-                const int j0 = ((kWin ? f.first : 0) + f.b0 + i) * kBlockN;
+                const int j0 = (f.b0 + i + (kWin && f.b0 + i >= g.kept_blocks ? f.gap : 0)) * kBlockN;
                 const int n_ok = min(min(last_visible, g.kv_len - 1) - j0 + 1, kBlockN); // visible columns are [0, n_ok)
-                const int n_lo = kWin ? last_visible - p.window + 1 - j0 : 0; // columns below n_lo lie before the row's window
+                const int n_lo = kWin ? last_visible - p.window + 1 - j0 : 0; // columns below n_lo lie before the row's window,
+                const int n_kept = kWin ? p.keep_first - j0 : 0;              // those below n_kept are seen all the same
                 uint32_t sr[kBlockN / 32][32];
 #pragma unroll
                 for (int c = 0; c < kBlockN / 32; ++c) {
@@ -649,12 +654,12 @@ __global__ void __launch_bounds__(kThreads, 2)
                 // Otherwise the hidden scores become -inf and take the same path: 2^(-inf * scale - m) = 0. (A scale
                 // that is not positive takes the slow path further down.)
                 const bool plain = p.scale_log2 > 0.f;
-                if (plain && !__all_sync(0xffffffffu, n_ok >= kBlockN && (!kWin || n_lo <= 0))) {
+                if (plain && !__all_sync(0xffffffffu, n_ok >= kBlockN && (!kWin || n_lo <= 0 || n_kept >= kBlockN))) {
 #pragma unroll
                     for (int c = 0; c < kBlockN / 32; ++c) {
 #pragma unroll
                         for (int k = 0; k < 32; ++k) {
-                            sr[c][k] = c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo) ? sr[c][k] : 0xff800000u;
+                            sr[c][k] = c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo || c * 32 + k < n_kept) ? sr[c][k] : 0xff800000u;
                         }
                     }
                 }
@@ -678,7 +683,7 @@ __global__ void __launch_bounds__(kThreads, 2)
                     for (int c = 0; c < kBlockN / 32; ++c) {
 #pragma unroll
                         for (int k = 0; k < 32; ++k) {
-                            if (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo)) {
+                            if (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo || c * 32 + k < n_kept)) {
                                 mx8[k & 7] = fmaxf(mx8[k & 7], __uint_as_float(sr[c][k]) * p.scale_log2);
                             }
                         }
@@ -726,8 +731,8 @@ __global__ void __launch_bounds__(kThreads, 2)
 #pragma unroll
                         for (int k = 0; k < 32; k += 2) {
                             const float p0 =
-                                (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo)) ? fast_exp2(fmaf(__uint_as_float(sr[c][k]), p.scale_log2, neg_m)) : 0.f;
-                            const float p1 = (c * 32 + k + 1 < n_ok && (!kWin || c * 32 + k + 1 >= n_lo))
+                                (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo || c * 32 + k < n_kept)) ? fast_exp2(fmaf(__uint_as_float(sr[c][k]), p.scale_log2, neg_m)) : 0.f;
+                            const float p1 = (c * 32 + k + 1 < n_ok && (!kWin || c * 32 + k + 1 >= n_lo || c * 32 + k + 1 < n_kept))
                                                  ? fast_exp2(fmaf(__uint_as_float(sr[c][k + 1]), p.scale_log2, neg_m))
                                                  : 0.f;
                             l0 += p0;
@@ -1268,6 +1273,7 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
         return -1;
     }
     p.window = windowed && batch.window <= 0 ? kv.table_stride * kPage : batch.window; // (a factor alone: a window nothing outgrows)
+    p.keep_first = batch.window > 0 ? batch.keep_first : 0;
     p.out_stride = out.row_stride != 0 ? out.row_stride : (long long)batch.nh * kD;
     p.row_scale = out.row_scale;
     p.out_wide = reinterpret_cast<uintptr_t>(out.out) % 32 == 0 && p.out_stride % 16 == 0 ? 1 : 0;

@@ -10,7 +10,7 @@ namespace llaisys::kernels {
 namespace {
 
 // After a greedy step: feed the chosen tokens back as the next inputs, log them, advance positions and lengths.
-__global__ void advance_decode_state_kernel(int64_t *__restrict__ tokens, const int64_t *__restrict__ next,
+__global__ void advance_decode_state_kernel(int64_t *__restrict__ tokens, int64_t *__restrict__ prev, const int64_t *__restrict__ next,
                                             int64_t *__restrict__ pos64, int32_t *__restrict__ pos32,
                                             int32_t *__restrict__ kv_lens, int64_t *__restrict__ log,
                                             int32_t *__restrict__ step_counter, int n) {
@@ -18,6 +18,7 @@ __global__ void advance_decode_state_kernel(int64_t *__restrict__ tokens, const 
     const int step = *step_counter;
     if (i < n) {
         const int64_t t = next[i];
+        prev[i] = tokens[i];
         tokens[i] = t;
         log[int64_t(step) * n + i] = t;
         pos64[i] += 1;
@@ -31,10 +32,10 @@ __global__ void bump_counter_kernel(int32_t *counter) { *counter += 1; }
 
 } // namespace
 
-void advance_decode_state(stream_t stream, int64_t *tokens, const int64_t *next, int64_t *pos64, int32_t *pos32,
+void advance_decode_state(stream_t stream, int64_t *tokens, int64_t *prev, const int64_t *next, int64_t *pos64, int32_t *pos32,
                           int32_t *kv_lens, int64_t *log, int32_t *step_counter, int n) {
     auto s = static_cast<cudaStream_t>(stream);
-    advance_decode_state_kernel<<<(n + 255) / 256, 256, 0, s>>>(tokens, next, pos64, pos32, kv_lens, log, step_counter, n);
+    advance_decode_state_kernel<<<(n + 255) / 256, 256, 0, s>>>(tokens, prev, next, pos64, pos32, kv_lens, log, step_counter, n);
     bump_counter_kernel<<<1, 1, 0, s>>>(step_counter);
     check_launch("advance_decode_state");
 }

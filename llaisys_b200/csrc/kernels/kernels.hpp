@@ -32,9 +32,10 @@ void argmax_rows(stream_t stream, llaisysDataType_t dtype, int64_t *idx_out, voi
                  size_t n);
 void embedding(stream_t stream, size_t elem_size, void *out, const int64_t *index, const void *weight, size_t n, size_t d,
                size_t vocab);
-// accumulate: out += in . W^T (the residual add of a decoder block folded into the projection; one rounding of the sum)
+// accumulate: out += in . W^T (the residual add of a decoder block folded into the projection; one rounding of the sum).
+// in_stride, out_stride: elements between rows of `in` and `out` (0: packed rows of k and n)
 void linear(stream_t stream, llaisysDataType_t dtype, void *out, const void *in, const void *weight, const void *bias,
-            size_t m, size_t n, size_t k, bool accumulate = false);
+            size_t m, size_t n, size_t k, bool accumulate = false, size_t in_stride = 0, size_t out_stride = 0);
 // K6: the tcgen05 weight-streaming kernel behind linear() for at most 128 rows of 16-bit activations (K a multiple of 64,
 // N a multiple of 64, not vocabulary-sized). False = shape not covered, nothing launched. overlap: programmatic launch
 // (the weight stream starts under the previous kernel's tail). linear_tc_status synchronises the stream and returns (and
@@ -58,7 +59,7 @@ void rope(stream_t stream, llaisysDataType_t dtype, void *out, const void *in, c
 void swiglu(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate, const void *up, size_t n);
 
 // Device-resident decode loop support: state hand-over between steps, CUDA graph capture / replay, event timing.
-void advance_decode_state(stream_t stream, int64_t *tokens, const int64_t *next, int64_t *pos64, int32_t *pos32,
+void advance_decode_state(stream_t stream, int64_t *tokens, int64_t *prev, const int64_t *next, int64_t *pos64, int32_t *pos32,
                           int32_t *kv_lens, int64_t *log, int32_t *step_counter, int n);
 void graph_capture_begin(stream_t stream);
 void *graph_capture_end(stream_t stream); // instantiated executable graph
@@ -86,6 +87,16 @@ void paged_rope_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
 void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const NormAppendArgs &args,
                        int32_t max_blocks, int32_t *error_flag);
 
+// Gated delta rule (see GatedDeltaArgs). decode: one token per sequence, everything in one launch. chunk: ragged runs of
+// tokens.
+void gated_delta_decode(stream_t stream, llaisysDataType_t dtype, const GatedDeltaArgs &args);
+void gated_delta_chunk(stream_t stream, llaisysDataType_t dtype, const GatedDeltaArgs &args);
+// Floats of one sequence's state: the matrices of all heads, then the newest `taps` inputs of the short convolutions.
+size_t gated_delta_state_floats(size_t heads, size_t kv_heads, size_t dk, size_t dv, size_t taps);
+// Floats of GatedDeltaArgs::scratch for n_rows rows, and of GatedDeltaArgs::segments (0: chunk calls are never cut).
+size_t gated_delta_scratch_floats(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t kv_heads, size_t dk, size_t dv);
+size_t gated_delta_segment_floats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
+
 // Gated linear attention (see GatedLinearArgs). decode: one token per sequence, everything in one launch. chunk: ragged
 // runs of tokens.
 void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args);
@@ -97,16 +108,30 @@ size_t gated_linear_segment_floats(llaisysDataType_t dtype, size_t heads, size_t
 // x[r, :] = scale * w[tokens[r], :]; copy (may be null): the same rounded to dtype, row r at copy + r * copy_stride
 void embed_scaled(stream_t stream, llaisysDataType_t dtype, float *x, void *copy, int64_t copy_stride, const int64_t *tokens,
                   const void *w, float scale, size_t rows, size_t d, size_t vocab);
+// x[r, :] = w[tokens[r], :] + pairs[b, :] with b = (prev[r] * mul_prev + tokens[r] * mul_cur) mod buckets, or b = buckets where
+// prev[r] < 0 (no token before this one); pairs has buckets + 1 rows
+void embed_pairs(stream_t stream, llaisysDataType_t dtype, float *x, const int64_t *tokens, const int64_t *prev, const void *w,
+                 const void *pairs, int64_t mul_prev, int64_t mul_cur, int64_t buckets, size_t rows, size_t d, size_t vocab);
 // out[r, :] = dtype(x[r, :]), row r at out + r * out_stride
 void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const float *x, size_t rows, size_t d);
-// out[i, :] = rms_norm(x[r, :]) * w with r = row_index[i] (null: r = i), f32 arithmetic, one rounding
+// out[i, :] = rms_norm(x[r, :]) * (offset + w) with r = row_index[i] (null: r = i), f32 arithmetic, one rounding. offset 1: a
+// weight stored around zero
 void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
-                     const void *w, float eps, size_t rows, size_t d);
+                     const void *w, float eps, size_t rows, size_t d, float offset = 0.f);
 // out (f32) = alpha * in . W^T (+ out when accumulate): a projection into the stream, or logits
 void linear_f32(stream_t stream, llaisysDataType_t dtype, float *out, const void *in, const void *weight, size_t m, size_t n,
-                size_t k, bool accumulate, float alpha = 1.f);
+                size_t k, bool accumulate, float alpha = 1.f, size_t in_stride = 0);
 // v = max(v, 0)^2 in place
 void relu_squared(stream_t stream, llaisysDataType_t dtype, void *v, size_t n);
+// out = gelu(in), tanh form, [rows, n] each with its own row stride (elements)
+void gelu_tanh(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const void *in, int64_t in_stride,
+               size_t rows, size_t n);
+// x += scale * (rms_norm(a) * wa + rms_norm(b) * wb), a and b f32 [rows, d] like x; h (may be null) = dtype(rms_norm(x) *
+// (offset + w)) of the new x, the norm that comes next
+void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const float *a, const void *wa, const float *b,
+                       const void *wb, float scale, float eps, void *h, const void *w, float offset, size_t rows, size_t d);
+// table[r, i] = (cos, sin)(positions[r] * freq[i]), i < half
+void rotary_table(stream_t stream, float *table, const int32_t *positions, const float *freq, size_t rows, size_t half);
 // logits = cap * tanh(logits / cap) in place (cap <= 0: unchanged) and the row-wise argmax of the result, one launch;
 // scratch as argmax_rows_split
 void softcap_argmax(stream_t stream, float *logits, float cap, int64_t *idx_out, size_t rows, size_t n, void *scratch);

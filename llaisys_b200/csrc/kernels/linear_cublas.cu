@@ -84,14 +84,14 @@ cudaDataType cuda_type(llaisysDataType_t dtype) {
 // Row-major out[M, N] = alpha in[M, K] . W[N, K]^T + beta out, f32 accumulation (f32 operands in true f32: no TF32 mode is
 // ever set on the handle). Column-major this is out^T[N, M] = W^T(as stored)[K, N]^T . in^T[K, M].
 void gemm(stream_t stream, llaisysDataType_t dtype, llaisysDataType_t out_dtype, void *out, const void *in, const void *weight,
-          size_t m, size_t n, size_t k, float alpha, float beta) {
+          size_t m, size_t n, size_t k, size_t in_stride, size_t out_stride, float alpha, float beta) {
     ASSERT(cublas_api().ok, "linear on NVIDIA needs cuBLAS (libcublas.so.12 was not found)");
     const cudaDataType type = cuda_type(dtype), out_type = cuda_type(out_dtype);
     cublasHandle_t h = handle_for_current_device();
     cublasStatus_t st = cublas_api().set_stream(h, static_cast<cudaStream_t>(stream));
     ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasSetStream failed with status " << int(st));
     st = cublas_api().gemm_ex(h, CUBLAS_OP_T, CUBLAS_OP_N, int(n), int(m), int(k), &alpha, weight, type, int(k), in, type,
-                              int(k), &beta, out, out_type, int(n), CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
+                              int(in_stride), &beta, out, out_type, int(out_stride), CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
     ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasGemmEx failed with status " << int(st));
 }
 
@@ -108,10 +108,12 @@ bool set_linear_policy(int policy) {
 }
 
 void linear(stream_t stream, llaisysDataType_t dtype, void *out, const void *in, const void *weight, const void *bias,
-            size_t m, size_t n, size_t k, bool accumulate) {
+            size_t m, size_t n, size_t k, bool accumulate, size_t in_stride, size_t out_stride) {
     if (m == 0 || n == 0) {
         return;
     }
+    in_stride = in_stride == 0 ? k : in_stride;
+    out_stride = out_stride == 0 ? n : out_stride;
     // Decode-sized calls may take the hand-written streaming kernel (skinny_gemm_tc.cu). Measured on B200 against cuBLAS
     // (graph replays, weights rotated beyond L2): it wins where the activations are a small fraction of the traffic and K is
     // long enough to split over a cluster (8 x 8960 -> 1536: 12.5 vs 17.2 us); at 64 rows every CTA re-reads the
@@ -120,7 +122,7 @@ void linear(stream_t stream, llaisysDataType_t dtype, void *out, const void *in,
     const int policy = g_linear_policy.load(std::memory_order_relaxed);
     const bool force_tc = policy == 1, never_tc = policy == 2;
     const bool prefer_tc = m <= 16 && k >= 4096;
-    if (!never_tc && (force_tc || prefer_tc) && m <= 128 &&
+    if (!never_tc && (force_tc || prefer_tc) && m <= 128 && in_stride == k && out_stride == n &&
         linear_tc(stream, dtype, out, in, weight, m, n, k, accumulate, false)) {
         if (bias != nullptr) {
             bias_add(stream, dtype, out, bias, m, n);
@@ -128,18 +130,19 @@ void linear(stream_t stream, llaisysDataType_t dtype, void *out, const void *in,
         return;
     }
     // accumulate: out += in . W^T, one rounding of the sum
-    gemm(stream, dtype, dtype, out, in, weight, m, n, k, 1.f, accumulate ? 1.f : 0.f);
+    gemm(stream, dtype, dtype, out, in, weight, m, n, k, in_stride, out_stride, 1.f, accumulate ? 1.f : 0.f);
     if (bias != nullptr) {
+        ASSERT(out_stride == n, "linear: a bias goes with packed output rows");
         bias_add(stream, dtype, out, bias, m, n);
     }
 }
 
 void linear_f32(stream_t stream, llaisysDataType_t dtype, float *out, const void *in, const void *weight, size_t m, size_t n,
-                size_t k, bool accumulate, float alpha) {
+                size_t k, bool accumulate, float alpha, size_t in_stride) {
     if (m == 0 || n == 0) {
         return;
     }
-    gemm(stream, dtype, LLAISYS_DTYPE_F32, out, in, weight, m, n, k, alpha, accumulate ? 1.f : 0.f);
+    gemm(stream, dtype, LLAISYS_DTYPE_F32, out, in, weight, m, n, k, in_stride == 0 ? k : in_stride, n, alpha, accumulate ? 1.f : 0.f);
 }
 
 } // namespace llaisys::kernels

@@ -308,6 +308,51 @@ __global__ void paged_rope_append_kernel(unsigned char *__restrict__ k_pool, uns
     }
 }
 
+// Elements [at, at + VEC) of a q or k head row after norm (inv, w; w null: none) and rotation: the partners across the rotated
+// range are read from the row itself. VEC divides rot_dims / 2, so a piece lies in one half.
+template <typename T, int VEC>
+__device__ __forceinline__ Pack<T, VEC> norm_rotate(Pack<T, VEC> x, const T *src, int32_t at, float inv, const T *w,
+                                                    const NormAppendArgs &a, int64_t row) {
+    using P = Pack<T, VEC>;
+    const int32_t half = a.rot_dims / 2;
+    const bool turns = at < a.rot_dims;
+    if (w == nullptr && !turns) {
+        return x;
+    }
+    float f[VEC];
+    auto normed = [&](const P &v, int32_t from, float (&y)[VEC]) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            y[e] = to_f32(v.v[e]);
+        }
+        if (w != nullptr) {
+            const P ww = *reinterpret_cast<const P *>(w + from);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                y[e] = y[e] * inv * to_f32(ww.v[e]);
+            }
+        }
+    };
+    normed(x, at, f);
+    if (turns) {
+        const bool first = at < half;
+        const int32_t other = first ? at + half : at - half, angle = first ? at : other;
+        float g[VEC];
+        normed(*reinterpret_cast<const P *>(src + other), other, g);
+        const float2 *cs = reinterpret_cast<const float2 *>(a.rot_table) + row * half + angle;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float2 t = cs[e];
+            f[e] = first ? f[e] * t.x - g[e] * t.y : f[e] * t.x + g[e] * t.y;
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+        x.v[e] = from_f32<T>(f[e]);
+    }
+    return x;
+}
+
 // K1c: one warp per (row, head) over the nh query, nkvh key and nkvh value heads of a projection row. Query and key heads
 // are divided by their root mean square and weighted; the warp of a query head also turns that head's gate into the factor
 // the attention kernel applies. f32 arithmetic, one rounding.
@@ -370,12 +415,8 @@ __global__ void __launch_bounds__(256)
     }
     for (int32_t i = lane * VEC; i < n; i += 32 * VEC) {
         P x = *reinterpret_cast<const P *>(src + i);
-        if (w != nullptr) {
-            const P ww = *reinterpret_cast<const P *>(w + i);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) {
-                x.v[e] = from_f32<T>(to_f32(x.v[e]) * inv * to_f32(ww.v[e]));
-            }
+        if (!is_v) {
+            x = norm_rotate<T, VEC>(x, src, i, inv, w, a, row);
         }
         *reinterpret_cast<P *>(dst + i) = x;
     }
@@ -432,14 +473,11 @@ __global__ void __launch_bounds__(256)
             continue;
         }
         const bool is_q = head[u] < a.nh, is_v = head[u] >= a.nh + g.nkvh;
-        const T *w = is_v ? nullptr : static_cast<const T *>(is_q ? a.q_norm : a.k_norm);
-        if (w != nullptr) {
-            const float inv = rsqrtf(ss[u] / float(d) + a.eps);
-            const P ww = *reinterpret_cast<const P *>(w + at);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) {
-                x[u].v[e] = from_f32<T>(to_f32(x[u].v[e]) * inv * to_f32(ww.v[e]));
-            }
+        if (!is_v) {
+            const T *src = static_cast<const T *>(a.proj) + int64_t(row[u]) * a.row_stride +
+                           (is_q ? a.q_at + int64_t(head[u]) * d : a.k_at + int64_t(head[u] - a.nh) * d);
+            x[u] = norm_rotate<T, VEC>(x[u], src, at, rsqrtf(ss[u] / float(d) + a.eps), static_cast<const T *>(is_q ? a.q_norm : a.k_norm), a,
+                                       row[u]);
         }
         if (is_q) {
             *reinterpret_cast<P *>(static_cast<T *>(a.q_out) + (int64_t(row[u]) * a.nh + head[u]) * d + at) = x[u];
@@ -476,7 +514,8 @@ void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &
     auto aligned = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const int32_t d = kv.d, dv = kv.vDim();
     const bool wide = d % kVec == 0 && dv % kVec == 0 && a.row_stride % kVec == 0 && a.q_at % kVec == 0 && a.k_at % kVec == 0 &&
-                      a.v_at % kVec == 0 && aligned(a.proj) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out);
+                      a.v_at % kVec == 0 && aligned(a.proj) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out) &&
+                      a.rot_dims / 2 % kVec == 0;
     const int64_t warps = int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh);
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(unsigned((warps + 7) / 8));
@@ -491,7 +530,7 @@ void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &
     const int32_t longest = d > dv ? d : dv;
     // (small calls are latency-bound: there the kernel with a warp per head row has the shorter chain)
     if (a.n_rows > 1024 && d % kPiece == 0 && dv % kPiece == 0 && longest <= 32 * kPiece && a.row_stride % kPiece == 0 && a.q_at % kPiece == 0 &&
-        a.k_at % kPiece == 0 && a.v_at % kPiece == 0 && wide && int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh) < (int64_t(1) << 31)) {
+        a.k_at % kPiece == 0 && a.v_at % kPiece == 0 && a.rot_dims / 2 % kPiece == 0 && wide && int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh) < (int64_t(1) << 31)) {
         int32_t lanes = 1;
         while (lanes * kPiece < longest) {
             lanes *= 2;

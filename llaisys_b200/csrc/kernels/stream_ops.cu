@@ -59,6 +59,30 @@ __global__ void embed_scaled_kernel(float *__restrict__ x, T *__restrict__ copy,
 }
 
 template <typename T, int VEC>
+__global__ void embed_pairs_kernel(float *__restrict__ x, const int64_t *__restrict__ tokens, const int64_t *__restrict__ prev,
+                                   const T *__restrict__ w, const T *__restrict__ pairs, int64_t mul_prev, int64_t mul_cur,
+                                   int64_t buckets, int32_t d, int64_t vocab) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    int64_t tok = tokens[row];
+    tok = tok < 0 || tok >= vocab ? 0 : tok; // validated on the host; never read out of range here
+    const int64_t before = prev[row];
+    const int64_t bucket =
+        before < 0 ? buckets : ((before % buckets) * mul_prev + (tok % buckets) * mul_cur) % buckets; // factors below buckets
+    const T *src = w + tok * d, *pair = pairs + bucket * d;
+    for (int32_t i = int32_t(threadIdx.x) * VEC; i < d; i += int32_t(blockDim.x) * VEC) {
+        const Vec<T, VEC> a = *reinterpret_cast<const Vec<T, VEC> *>(src + i), b = *reinterpret_cast<const Vec<T, VEC> *>(pair + i);
+        Vec<float, VEC> f;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            f.v[e] = to_f32(a.v[e]) + to_f32(b.v[e]);
+        }
+        *reinterpret_cast<Vec<float, VEC> *>(x + row * d + i) = f;
+    }
+}
+
+template <typename T, int VEC>
 __global__ void stream_cast_kernel(T *__restrict__ out, int64_t out_stride, const float *__restrict__ x, int32_t d) {
     grid_dependency_wait();
     grid_launch_dependents();
@@ -78,7 +102,7 @@ __global__ void stream_cast_kernel(T *__restrict__ out, int64_t out_stride, cons
 // has beyond them is read again.
 template <typename T, int VEC, int PER_THREAD>
 __global__ void stream_rms_norm_kernel(T *__restrict__ out, const float *__restrict__ x, const int64_t *__restrict__ row_index,
-                                       const T *__restrict__ w, float eps, int32_t d) {
+                                       const T *__restrict__ w, float eps, int32_t d, float offset) {
     grid_dependency_wait();
     grid_launch_dependents();
     using F = Vec<float, VEC>;
@@ -125,7 +149,7 @@ __global__ void stream_rms_norm_kernel(T *__restrict__ out, const float *__restr
         Vec<T, VEC> o;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            o.v[e] = from_f32<T>(f.v[e] * inv * to_f32(ww.v[e]));
+            o.v[e] = from_f32<T>(f.v[e] * inv * (offset + to_f32(ww.v[e])));
         }
         *reinterpret_cast<Vec<T, VEC> *>(dst + int64_t(i) * VEC) = o;
     };
@@ -138,6 +162,148 @@ __global__ void stream_rms_norm_kernel(T *__restrict__ out, const float *__restr
     }
     for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * int32_t(blockDim.x); i < n_vec; i += int32_t(blockDim.x)) {
         store(i, *reinterpret_cast<const F *>(src + int64_t(i) * VEC));
+    }
+}
+
+// Sum over the CTA, the same value for every thread (partials in the same order); `part` holds 32 floats.
+__device__ __forceinline__ float block_sum(float v, float *part) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        v += __shfl_xor_sync(0xffffffffu, v, o);
+    }
+    __syncthreads(); // `part` may still be read by an earlier call
+    if ((threadIdx.x & 31) == 0) {
+        part[threadIdx.x >> 5] = v;
+    }
+    __syncthreads();
+    float tot = 0.f;
+    for (int i = 0; i < int(blockDim.x >> 5); ++i) {
+        tot += part[i];
+    }
+    return tot;
+}
+
+// One CTA per row, like stream_rms_norm_kernel: two norms over the rows of a and b, their sum into the stream, and the norm
+// that follows. The first PER_THREAD pieces of a thread stay in registers.
+template <typename T, int VEC, int PER_THREAD>
+__global__ void stream_add_normed_kernel(float *__restrict__ x, const float *__restrict__ a, const T *__restrict__ wa,
+                                         const float *__restrict__ b, const T *__restrict__ wb, float scale, float eps,
+                                         T *__restrict__ h, const T *__restrict__ w, float offset, int32_t d) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    using F = Vec<float, VEC>;
+    using W = Vec<T, VEC>;
+    __shared__ float s_a[32], s_b[32];
+    const int64_t row = int64_t(blockIdx.x) * d;
+    const int32_t n_vec = d / VEC, step = int32_t(blockDim.x);
+    F ha[PER_THREAD], hb[PER_THREAD];
+    float sa = 0.f, sb = 0.f;
+    auto square = [](const F &f, float &s) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            s = fmaf(f.v[e], f.v[e], s);
+        }
+    };
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * step;
+        if (i < n_vec) {
+            ha[r] = reinterpret_cast<const F *>(a + row)[i];
+            hb[r] = reinterpret_cast<const F *>(b + row)[i];
+            square(ha[r], sa);
+            square(hb[r], sb);
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * step; i < n_vec; i += step) {
+        square(reinterpret_cast<const F *>(a + row)[i], sa);
+        square(reinterpret_cast<const F *>(b + row)[i], sb);
+    }
+    const float ia = rsqrtf(block_sum(sa, s_a) / float(d) + eps) * scale, ib = rsqrtf(block_sum(sb, s_b) / float(d) + eps) * scale;
+    float sx = 0.f;
+    auto add = [&](int32_t i, const F &fa, const F &fb) {
+        F f = reinterpret_cast<const F *>(x + row)[i];
+        const W va = reinterpret_cast<const W *>(wa)[i], vb = reinterpret_cast<const W *>(wb)[i];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            f.v[e] += fa.v[e] * ia * to_f32(va.v[e]) + fb.v[e] * ib * to_f32(vb.v[e]);
+        }
+        square(f, sx);
+        reinterpret_cast<F *>(x + row)[i] = f;
+        return f;
+    };
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * step;
+        if (i < n_vec) {
+            ha[r] = add(i, ha[r], hb[r]); // from here on the new stream
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * step; i < n_vec; i += step) {
+        add(i, reinterpret_cast<const F *>(a + row)[i], reinterpret_cast<const F *>(b + row)[i]);
+    }
+    if (h == nullptr) {
+        return;
+    }
+    const float inv = rsqrtf(block_sum(sx, s_a) / float(d) + eps);
+    auto store = [&](int32_t i, const F &f) {
+        const W ww = reinterpret_cast<const W *>(w)[i];
+        W o;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            o.v[e] = from_f32<T>(f.v[e] * inv * (offset + to_f32(ww.v[e])));
+        }
+        reinterpret_cast<W *>(h + row)[i] = o;
+    };
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * step;
+        if (i < n_vec) {
+            store(i, ha[r]);
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * step; i < n_vec; i += step) {
+        store(i, reinterpret_cast<const F *>(x + row)[i]); // (written by this thread)
+    }
+}
+
+// z / 2 (1 + tanh(y)) = z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
+template <typename T>
+__device__ __forceinline__ float gelu(float z) {
+    const float y2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+    if constexpr (sizeof(T) == 4) {
+        return z / (1.f + expf(-y2));
+    } else {
+        return __fdividef(z, 1.f + __expf(fminf(-y2, 80.f)));
+    }
+}
+
+template <typename T, int VEC>
+__global__ void gelu_tanh_kernel(T *__restrict__ out, int64_t out_stride, const T *__restrict__ in, int64_t in_stride, int32_t n_vec) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    using P = Vec<T, VEC>;
+    const P *src = reinterpret_cast<const P *>(in + int64_t(blockIdx.y) * in_stride);
+    P *dst = reinterpret_cast<P *>(out + int64_t(blockIdx.y) * out_stride);
+    for (int32_t i = int32_t(blockIdx.x) * int32_t(blockDim.x) + int32_t(threadIdx.x); i < n_vec; i += int32_t(gridDim.x) * int32_t(blockDim.x)) {
+        P p = src[i];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            p.v[e] = from_f32<T>(gelu<T>(to_f32(p.v[e])));
+        }
+        dst[i] = p;
+    }
+}
+
+__global__ void rotary_table_kernel(float2 *__restrict__ table, const int32_t *__restrict__ positions, const float *__restrict__ freq,
+                                    int32_t half, int64_t total) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t at = int64_t(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (at < total) {
+        const int64_t row = at / half;
+        float s, c;
+        sincosf(float(positions[row]) * freq[at - row * half], &s, &c);
+        table[at] = make_float2(c, s);
     }
 }
 
@@ -248,6 +414,24 @@ void embed_scaled(stream_t stream, llaisysDataType_t dtype, float *x, void *copy
     check_launch("embed_scaled");
 }
 
+void embed_pairs(stream_t stream, llaisysDataType_t dtype, float *x, const int64_t *tokens, const int64_t *prev, const void *w,
+                 const void *pairs, int64_t mul_prev, int64_t mul_cur, int64_t buckets, size_t rows, size_t d, size_t vocab) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    CHECK_ARGUMENT(buckets > 0 && buckets < (int64_t(1) << 31), "embed_pairs: 1 to 2^31 - 1 buckets");
+    auto s = static_cast<cudaStream_t>(stream);
+    auto mod = [&](int64_t v) { return (v % buckets + buckets) % buckets; };
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        const bool wide = d % 4 == 0 && aligned16(x) && aligned16(w) && aligned16(pairs);
+        auto kernel = wide ? embed_pairs_kernel<T, 4> : embed_pairs_kernel<T, 1>;
+        launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, x, tokens, prev, static_cast<const T *>(w),
+                            static_cast<const T *>(pairs), mod(mul_prev), mod(mul_cur), buckets, int32_t(d), int64_t(vocab));
+    });
+    check_launch("embed_pairs");
+}
+
 void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const float *x, size_t rows, size_t d) {
     if (rows == 0 || d == 0) {
         return;
@@ -264,7 +448,7 @@ void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t ou
 }
 
 void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
-                     const void *w, float eps, size_t rows, size_t d) {
+                     const void *w, float eps, size_t rows, size_t d, float offset) {
     if (rows == 0 || d == 0) {
         return;
     }
@@ -274,9 +458,59 @@ void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const 
         const bool wide = d % 4 == 0 && aligned16(x) && aligned16(out) && aligned16(w);
         auto kernel = wide ? stream_rms_norm_kernel<T, 4, 4> : stream_rms_norm_kernel<T, 1, 4>;
         launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, static_cast<T *>(out), x, row_index,
-                            static_cast<const T *>(w), eps, int32_t(d));
+                            static_cast<const T *>(w), eps, int32_t(d), offset);
     });
     check_launch("stream_rms_norm");
+}
+
+void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const float *a, const void *wa, const float *b,
+                       const void *wb, float scale, float eps, void *h, const void *w, float offset, size_t rows, size_t d) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        const bool wide = d % 4 == 0 && aligned16(x) && aligned16(a) && aligned16(b) && aligned16(wa) && aligned16(wb) && aligned16(h) &&
+                          aligned16(w);
+        auto kernel = wide ? stream_add_normed_kernel<T, 4, 3> : stream_add_normed_kernel<T, 1, 3>;
+        launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, x, a, static_cast<const T *>(wa), b,
+                            static_cast<const T *>(wb), scale, eps, static_cast<T *>(h), static_cast<const T *>(w), offset, int32_t(d));
+    });
+    check_launch("stream_add_normed");
+}
+
+void gelu_tanh(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const void *in, int64_t in_stride,
+               size_t rows, size_t n) {
+    if (rows == 0 || n == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        constexpr int kVec = 16 / int(sizeof(T));
+        const bool wide = n % kVec == 0 && out_stride % kVec == 0 && in_stride % kVec == 0 && aligned16(out) && aligned16(in);
+        const size_t n_vec = wide ? n / kVec : n;
+        auto kernel = wide ? gelu_tanh_kernel<T, kVec> : gelu_tanh_kernel<T, 1>;
+        constexpr size_t kRows = 65535;
+        for (size_t r = 0; r < rows; r += kRows) {
+            const size_t m = rows - r < kRows ? rows - r : kRows;
+            launch_programmatic(kernel, dim3(unsigned((n_vec + 511) / 512), unsigned(m)), 256u, s,
+                                static_cast<T *>(out) + int64_t(r) * out_stride, out_stride,
+                                static_cast<const T *>(in) + int64_t(r) * in_stride, in_stride, int32_t(n_vec));
+        }
+    });
+    check_launch("gelu_tanh");
+}
+
+void rotary_table(stream_t stream, float *table, const int32_t *positions, const float *freq, size_t rows, size_t half) {
+    if (rows == 0 || half == 0) {
+        return;
+    }
+    const int64_t total = int64_t(rows) * int64_t(half);
+    launch_programmatic(rotary_table_kernel, dim3(unsigned((total + 255) / 256)), 256u, static_cast<cudaStream_t>(stream),
+                        reinterpret_cast<float2 *>(table), positions, freq, int32_t(half), total);
+    check_launch("rotary_table");
 }
 
 void relu_squared(stream_t stream, llaisysDataType_t dtype, void *v, size_t n) {

@@ -35,8 +35,10 @@ template <typename... Args>
 
 constexpr size_t kMaxInt32 = size_t(std::numeric_limits<int32_t>::max());
 // A window longer than any sequence of the cache is cut to what a sequence can hold.
-int32_t windowOf(const PagedKVConfig &cfg, const AttnOptions &opt) {
-    return int32_t(std::min(opt.window, cfg.page_size * cfg.max_pages_per_seq));
+void setWindow(kernels::AttnBatch &b, const PagedKVConfig &cfg, const AttnOptions &opt) {
+    const size_t longest = cfg.page_size * cfg.max_pages_per_seq;
+    b.window = int32_t(std::min(opt.window, longest));
+    b.keep_first = opt.window != 0 ? int32_t(std::min(opt.keep_first, longest)) : 0;
 }
 constexpr size_t kMaxDecodeSeqs = 1024; // sequences per launch of the TMA decode kernel
 
@@ -712,7 +714,7 @@ void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, 
         b.max_q_len = 1;
         b.max_kv_len = int32_t(max_kv_len);
         b.nh = int32_t(nh);
-        b.window = windowOf(_cfg, opt);
+        setWindow(b, _cfg, opt);
         kernels::AttnOut o;
         o.out = out ? static_cast<std::byte *>(out) + at * out_row * _elem : nullptr;
         o.row_scale = opt.row_scale ? opt.row_scale + at * nh : nullptr;
@@ -776,7 +778,7 @@ void PagedKV::prefillDev(size_t layer, void *out, const void *q, const int32_t *
     b.max_q_len = int32_t(max_q_len);
     b.max_kv_len = int32_t(max_kv_len);
     b.nh = int32_t(nh);
-    b.window = windowOf(_cfg, opt);
+    setWindow(b, _cfg, opt);
     kernels::AttnOut o;
     o.out = out;
     o.row_scale = opt.row_scale;

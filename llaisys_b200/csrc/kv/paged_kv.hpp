@@ -31,6 +31,7 @@ struct KVLayerShape {
 // What a layer's attention adds to plain causal attention.
 struct AttnOptions {
     size_t window = 0;                 // sliding window in tokens, the query's own included; 0 = none
+    size_t keep_first = 0;             // with a window: the first tokens of a sequence that stay visible behind it
     const float *row_scale = nullptr;  // device, [rows, nh]: factor on every head's output
     size_t row_stride = 0;             // elements between output rows; 0 = packed
 };

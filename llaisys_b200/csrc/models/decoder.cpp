@@ -50,6 +50,9 @@ bool Decoder::loadTensor(const std::string &, llaisysDataType_t, const std::vect
     failModel(LLAISYS_E_UNSUPPORTED, "this model's weights are loaded through their handles");
 }
 
+void Decoder::recordStream(bool) { failModel(LLAISYS_E_UNSUPPORTED, "this model keeps no record of its stream"); }
+size_t Decoder::layerStream(float *, size_t) { failModel(LLAISYS_E_UNSUPPORTED, "this model keeps no record of its stream"); }
+
 void Decoder::dropStepGraphs() {
 #ifdef ENABLE_NVIDIA_API
     for (StepGraph &g : _step_graphs) {
@@ -96,6 +99,7 @@ void Decoder::configureCache(size_t max_seqs, size_t max_tokens, size_t pool_tok
     _cache->setLaunchOverlap(_on_gpu);
     _max_tokens_per_seq = cfg.max_pages_per_seq * kPageSize;
     _seq_len.assign(max_seqs, kNotLive);
+    _seq_last.assign(max_seqs, -1);
     _seq_tokens.assign(max_seqs, {});
 }
 
@@ -112,6 +116,7 @@ int32_t Decoder::seqAdd() {
     }
     const int32_t s = _cache->seqAdd();
     _seq_len[s] = 0;
+    _seq_last[s] = -1;
     _seq_tokens[s].clear();
     return s;
 }
@@ -127,6 +132,7 @@ int32_t Decoder::seqAddWithPrefix(const int64_t *tokens, size_t n, size_t *match
             throw;
         }
         _seq_tokens[s].assign(tokens, tokens + got);
+        _seq_last[s] = got != 0 ? tokens[got - 1] : -1;
     }
     _seq_len[s] = got;
     if (matched != nullptr) {
@@ -145,6 +151,7 @@ void Decoder::seqReserve(int32_t seq, size_t n_tokens) {
 
 // The sequence now holds K/V for n more tokens: remember their ids and publish the pages they completed.
 void Decoder::recordTokens(int32_t seq, const int64_t *tokens, size_t n) {
+    _seq_last[seq] = tokens[n - 1];
     if (_state) {
         return; // pages of a network with recurrent state are not a whole prefix: never shared
     }
@@ -203,8 +210,8 @@ void Decoder::ensureWorkspace(size_t n_tokens, size_t n_seqs, size_t n_out) {
         const std::vector<std::byte> zeros(n_out * 12);
         copyToDevice(_argmax_scratch->memory(), zeros.data(), zeros.size());
     }
-    // tokens, pos64, out_rows, next (int64) then seq32, pos32, kv_lens, seq_list, q_starts (int32), 16-byte aligned
-    const size_t need = align_up(n_tokens * 8, 16) * 2 + align_up(n_out * 8, 16) * 2 + align_up(n_tokens * 4, 16) * 2 +
+    // tokens, pos64, prev, out_rows, next (int64) then seq32, pos32, kv_lens, seq_list, q_starts (int32), 16-byte aligned
+    const size_t need = align_up(n_tokens * 8, 16) * 3 + align_up(n_out * 8, 16) * 2 + align_up(n_tokens * 4, 16) * 2 +
                         align_up(n_seqs * 4, 16) * 2 + align_up((n_seqs + 1) * 4, 16);
     if (need > _meta_bytes) {
         ++_generation;
@@ -224,6 +231,7 @@ Decoder::StepArrays Decoder::carveStepArrays(size_t n_tokens, size_t n_seqs, siz
     std::byte *base = _meta_block->memory();
     a.tokens = reinterpret_cast<int64_t *>(base + take(n_tokens * 8));
     a.pos64 = reinterpret_cast<int64_t *>(base + take(n_tokens * 8));
+    a.prev = reinterpret_cast<int64_t *>(base + take(n_tokens * 8));
     a.out_rows = reinterpret_cast<int64_t *>(base + take(n_out * 8));
     a.next = reinterpret_cast<int64_t *>(base + take(n_out * 8));
     a.seq32 = reinterpret_cast<int32_t *>(base + take(n_tokens * 4));
@@ -324,6 +332,7 @@ void Decoder::stepRows(const int32_t *seq_ids, const int32_t *n_tokens, size_t n
         decode_only = decode_only && n == 1;
         for (size_t t = 0; t < n; ++t, ++row) {
             host(a.tokens)[row] = tokens[row];
+            host(a.prev)[row] = t != 0 ? tokens[row - 1] : _seq_last[seq_ids[i]];
             host(a.pos64)[row] = int64_t(len + t);
             host(a.pos32)[row] = int32_t(len + t);
             host(a.seq32)[row] = seq_ids[i];
@@ -426,6 +435,7 @@ void Decoder::decodeLoop(const int32_t *seq_ids, size_t n_seqs, const int64_t *f
     for (size_t i = 0; i < n_seqs; ++i) {
         const size_t len = seqLen(seq_ids[i]);
         host(a.tokens)[i] = first_tokens[i];
+        host(a.prev)[i] = _seq_last[seq_ids[i]];
         host(a.pos64)[i] = int64_t(len);
         host(a.pos32)[i] = int32_t(len);
         host(a.seq32)[i] = seq_ids[i];
@@ -454,13 +464,14 @@ void Decoder::decodeLoop(const int32_t *seq_ids, size_t n_seqs, const int64_t *f
         forward(a, shape);
 #ifdef ENABLE_NVIDIA_API
         if (_on_gpu) {
-            kernels::advance_decode_state(_stream, a.tokens, a.next, a.pos64, a.pos32, a.kv_lens, log_dev, counter_dev,
+            kernels::advance_decode_state(_stream, a.tokens, a.prev, a.next, a.pos64, a.pos32, a.kv_lens, log_dev, counter_dev,
                                           int(n_seqs));
             return;
         }
 #endif
         int32_t &step = *counter_dev;
         for (size_t i = 0; i < n_seqs; ++i) {
+            a.prev[i] = a.tokens[i];
             a.tokens[i] = a.next[i];
             log_dev[size_t(step) * n_seqs + i] = a.next[i];
             a.pos64[i] += 1;

@@ -50,6 +50,11 @@ public:
     // Names of weights that no loadTensor call has filled yet.
     virtual std::vector<std::string> missingTensors() const { return {}; }
 
+    // Development aid, for models that have it: keep the residual stream after every layer run of the steps that follow;
+    // layerStream gives [runs, rows, width] of the last such step (-> its floats; out_host may be null).
+    virtual void recordStream(bool enable);
+    virtual size_t layerStream(float *out_host, size_t capacity_floats);
+
     // A cache of max_seqs sequences of at most max_tokens tokens each. pool_tokens: how many tokens all live sequences
     // together can hold (whole pages); 0 = max_seqs * max_tokens.
     void configureCache(size_t max_seqs, size_t max_tokens, size_t pool_tokens = 0);
@@ -80,6 +85,7 @@ protected:
     // device pointers of one step's index arrays (all inside _meta_block)
     struct StepArrays {
         int64_t *tokens = nullptr, *pos64 = nullptr, *out_rows = nullptr, *next = nullptr;
+        int64_t *prev = nullptr; // the token before each row's in its sequence, -1 for the first
         int32_t *seq32 = nullptr, *pos32 = nullptr, *kv_lens = nullptr, *q_starts = nullptr, *seq_list = nullptr;
     };
     struct StepShape {
@@ -129,6 +135,7 @@ private:
 
     size_t _max_tokens_per_seq = 0;
     std::vector<size_t> _seq_len; // by sequence id; SIZE_MAX = not live
+    std::vector<int64_t> _seq_last;  // by sequence id: its newest token, -1 when it has none
     std::vector<std::vector<int64_t>> _seq_tokens; // ids of the tokens each sequence holds (keys of the prefix cache)
     int32_t _implicit_seq = -1;
     core::storage_t _meta_block;

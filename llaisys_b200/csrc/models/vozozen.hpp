@@ -9,42 +9,27 @@
 // projection over both sides accumulated into the stream, norm, up, activation, down accumulated into the stream.
 #pragma once
 
-#include "decoder.hpp"
+#include "stream_decoder.hpp"
 #include "llaisys/models/vozozen.h"
 
-#include <map>
-#include <string>
 #include <vector>
 
 namespace llaisys::models {
 
-class Vozozen : public Decoder {
+class Vozozen : public StreamDecoder {
 public:
     Vozozen(const LlaisysVozozenMeta &meta, llaisysDeviceType_t device, int device_id);
 
     size_t vocab() const override { return _meta.voc; }
     size_t maxSeq() const override { return _meta.maxseq; }
     int64_t endToken() const override { return _meta.end_token; }
-    bool loadTensor(const std::string &name, llaisysDataType_t dtype, const std::vector<size_t> &shape, const void *data) override;
-    std::vector<std::string> missingTensors() const override;
-
-    void recordStream(bool enable) { _record = enable; }
-    size_t layerStream(float *out_host, size_t capacity_floats); // -> floats of the last recorded step: [runs, rows, width]
 
 private:
     kv::PagedKVConfig cacheShape() const override;
     std::vector<size_t> stateShape() const override;
     void ensureActivations(size_t n_tokens, size_t n_out) override;
     void forward(const StepArrays &a, const StepShape &s) override;
-    bool graphable() const override { return !_record; }
 
-    // Where a named tensor goes: `rows` x `cols` at (row, col) of a packed matrix with `ld` columns.
-    struct Slot {
-        std::byte *base;
-        size_t row, col, rows, cols, ld;
-        size_t ndim; // of the checkpoint tensor (1: cols == 1 is a vector of `rows`)
-        bool loaded = false;
-    };
     struct Layer {
         LlaisysVozozenLayerMeta meta;
         std::byte *norm1, *norm2, *proj, *out, *up, *down, *q_norm, *k_norm, *decay_w, *decay_b, *gla_norm;
@@ -53,21 +38,13 @@ private:
         size_t right, n_mix; // first column of the right mixer in the mix buffer, columns in all (padded to 8)
     };
 
-    std::byte *matrix(size_t rows, size_t cols); // zeroed, owned by the model
-    void place(const std::string &name, std::byte *base, size_t row, size_t col, size_t rows, size_t cols, size_t ld, size_t ndim = 2);
-    std::byte *vector(const std::string &name, size_t n);
-
     LlaisysVozozenMeta _meta;
     std::vector<Layer> _layers;
     std::vector<size_t> _runs;       // layer of every run, in order
     std::vector<bool> _starts_pass;  // run r is the first of a pass
-    std::map<std::string, Slot> _slots;
-    std::vector<core::storage_t> _weight_blocks;
     std::byte *_embed = nullptr, *_loop_in = nullptr, *_final_norm = nullptr, *_head = nullptr;
 
     core::storage_t _x, _pass_in, _h, _proj, _q, _row_scale, _mix, _raw, _decay, _segments, _u, _h_out;
-    bool _record = false;
-    std::vector<float> _recorded;
 };
 
 } // namespace llaisys::models

@@ -135,12 +135,49 @@ class LlaisysVozozenMeta(Structure):
                 ("end_token", c_int64)]
 
 
+class LlaisysDeltaMixerMeta(Structure):
+    """struct LlaisysDeltaMixerMeta (include/llaisys/models/doderax.h)."""
+    _fields_ = [("heads", c_size_t), ("kv_heads", c_size_t), ("dim", c_size_t), ("vdim", c_size_t), ("taps", c_size_t),
+                ("decay_rank", c_size_t), ("gate_rank", c_size_t)]
+
+
+class LlaisysSinkAttentionMeta(Structure):
+    """struct LlaisysSinkAttentionMeta (include/llaisys/models/doderax.h)."""
+    _fields_ = [("heads", c_size_t), ("kv_heads", c_size_t), ("dim", c_size_t), ("vdim", c_size_t), ("window", c_size_t),
+                ("keep_first", c_size_t), ("rot_dims", c_size_t), ("rot_base", c_double), ("scale", c_float)]
+
+
+class LlaisysDoderaxLayerMeta(Structure):
+    """struct LlaisysDoderaxLayerMeta (include/llaisys/models/doderax.h)."""
+    _fields_ = [("parallel", c_int), ("attn", LlaisysSinkAttentionMeta), ("delta", LlaisysDeltaMixerMeta), ("ff", c_size_t)]
+
+
+class LlaisysDoderaxMeta(Structure):
+    """struct LlaisysDoderaxMeta (include/llaisys/models/doderax.h)."""
+    _fields_ = [("dtype", llaisysDataType_t), ("nlayer", c_size_t), ("layers", POINTER(LlaisysDoderaxLayerMeta)),
+                ("width", c_size_t), ("voc", c_size_t), ("maxseq", c_size_t), ("pair_buckets", c_size_t), ("pair_mul_prev", c_int64),
+                ("pair_mul_cur", c_int64), ("eps", c_float), ("logit_scale", c_float), ("end_token", c_int64)]
+
+
 class LlaisysNormAppend(Structure):
     """struct LlaisysNormAppend (include/llaisys/mixers.h)."""
     _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("k_at", c_int64), ("v_at", c_int64),
                 ("gate_at", c_int64), ("q_norm", c_void_p), ("k_norm", c_void_p), ("eps", c_float), ("gate_scale", c_float),
                 ("q_out", c_void_p), ("row_scale", c_void_p), ("seq_ids_dev", c_void_p), ("positions_dev", c_void_p),
-                ("n_rows", c_size_t), ("nh", c_size_t)]
+                ("n_rows", c_size_t), ("nh", c_size_t), ("rot_dims", c_size_t), ("rot_table", c_void_p)]
+
+
+class LlaisysGatedDelta(Structure):
+    """struct LlaisysGatedDelta (include/llaisys/mixers.h)."""
+    _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("k_at", c_int64), ("v_at", c_int64),
+                ("b_at", c_int64), ("a_at", c_int64), ("conv_q", c_void_p), ("conv_k", c_void_p), ("conv_v", c_void_p),
+                ("decay_w", c_void_p), ("decay_ld", c_int64), ("a_log", c_void_p), ("dt_bias", c_void_p), ("norm_w", c_void_p),
+                ("gate", c_void_p), ("gate_stride", c_int64), ("gate_silu", c_int), ("q_scale", c_float), ("eps", c_float),
+                ("unit_eps", c_float), ("taps", c_size_t), ("heads", c_size_t), ("kv_heads", c_size_t), ("dk", c_size_t),
+                ("dv", c_size_t), ("rank", c_size_t), ("state", c_void_p), ("slot_stride", c_int64), ("seq_ids_dev", c_void_p),
+                ("q_starts_dev", c_void_p), ("kv_lens_dev", c_void_p), ("n_seqs", c_size_t), ("n_rows", c_size_t),
+                ("max_q_len", c_size_t), ("out", c_void_p), ("out_stride", c_int64), ("scratch", c_void_p),
+                ("scratch_floats", c_size_t), ("scratch_segments", c_void_p), ("scratch_segment_floats", c_size_t)]
 
 
 class LlaisysGatedLinear(Structure):
@@ -284,8 +321,13 @@ PROTOTYPES: dict[str, tuple] = {
                                            c_size_t, c_size_t]),
     "llaisysPagedKVNormAppendDev": (c_int, [_KV, c_size_t, POINTER(LlaisysNormAppend), llaisysStream_t]),
     "llaisysPagedAttentionOptDev": (c_int, [_KV, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t,
-                                            c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, c_void_p, c_size_t,
-                                            llaisysStream_t]),
+                                            c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, c_size_t, c_void_p,
+                                            c_size_t, llaisysStream_t]),
+    "llaisysRotaryTableDev": (c_int, [llaisysDeviceType_t, c_int, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t,
+                                      llaisysStream_t]),
+    "llaisysGatedDeltaDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysGatedDelta), c_int,
+                                     llaisysStream_t]),
+    "llaisysGatedDeltaSizes": (None, [llaisysDataType_t] + [c_size_t] * 6 + [POINTER(c_size_t)] * 3),
     "llaisysGatedLinearDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysGatedLinear), c_int,
                                       llaisysStream_t]),
     "llaisysGatedLinearSegmentFloats": (c_size_t, [llaisysDataType_t, c_size_t, c_size_t, c_size_t]),
@@ -307,10 +349,12 @@ PROTOTYPES: dict[str, tuple] = {
     "llaisysModelDecodeLoop": (c_int, [_MODEL, _I32P, c_size_t, POINTER(c_int64), c_size_t, POINTER(c_int64)]),
     "llaisysModelLastLogits": (c_int, [_MODEL, POINTER(c_float), c_size_t]),
     "llaisysModelLastLoopMs": (c_double, [_MODEL]),
+    "llaisysModelRecordStream": (c_int, [_MODEL, c_int]),
+    "llaisysModelLayerStream": (c_int, [_MODEL, POINTER(c_float), c_size_t, POINTER(c_size_t)]),
     # include/llaisys/models/vozozen.h
+    # include/llaisys/models/doderax.h
+    "llaisysDoderaxModelCreate": (_MODEL, [POINTER(LlaisysDoderaxMeta), llaisysDeviceType_t, c_int]),
     "llaisysVozozenModelCreate": (_MODEL, [POINTER(LlaisysVozozenMeta), llaisysDeviceType_t, c_int]),
-    "llaisysVozozenModelRecordStream": (c_int, [_MODEL, c_int]),
-    "llaisysVozozenModelLayerStream": (c_int, [_MODEL, POINTER(c_float), c_size_t, POINTER(c_size_t)]),
     # include/llaisys/serving.h
     "llaisysEngineCreate": (c_int, [POINTER(c_void_p), _MODEL, c_size_t, c_size_t, c_size_t]),
     "llaisysEngineDestroy": (None, [c_void_p]),
@@ -355,5 +399,6 @@ __all__ = [
     "LIB_LLAISYS", "PROTOTYPES", "LlaisysRuntimeAPI", "llaisysStream_t", "llaisysTensor_t", "llaisysPagedKV_t",
     "llaisysDataType_t", "DataType", "llaisysDeviceType_t", "DeviceType", "llaisysMemcpyKind_t", "MemcpyKind",
     "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent",
-    "LlaisysNormAppend", "LlaisysGatedLinear", "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
+    "LlaisysNormAppend", "LlaisysGatedLinear", "LlaisysGatedDelta", "LlaisysDoderaxMeta", "LlaisysDoderaxLayerMeta",
+    "LlaisysSinkAttentionMeta", "LlaisysDeltaMixerMeta", "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
 ]

@@ -1,7 +1,8 @@
 """Model wrappers (reference: python/llaisys/models/__init__.py:1)."""
 from .base import CausalLM
+from .doderax import Doderax
 from .qwen2 import Qwen2
 from .registry import MODELS, load_model, model_class
 from .vozozen import Vozozen
 
-__all__ = ["CausalLM", "Qwen2", "Vozozen", "MODELS", "load_model", "model_class"]
+__all__ = ["CausalLM", "Doderax", "Qwen2", "Vozozen", "MODELS", "load_model", "model_class"]

@@ -6,13 +6,16 @@ from __future__ import annotations
 
 import ctypes
 import itertools
-from ctypes import c_float, c_int32, c_int64
-from typing import Sequence
+import json
+from ctypes import c_float, c_int, c_int32, c_int64, c_size_t
+from pathlib import Path
+from typing import Mapping, Sequence
 
 import numpy as np
 
-from ..libllaisys import LIB_LLAISYS, DataType
-from ..paged_kv import _check
+from ..libllaisys import LIB_LLAISYS, DataType, DeviceType
+from ..paged_kv import LlaisysError, _check
+from .weights import LIBRARY_DTYPE, checkpoint_files
 
 DTYPE_NAMES = {"bfloat16": DataType.BF16, "float16": DataType.F16, "float32": DataType.F32}
 
@@ -161,3 +164,99 @@ class CausalLM:
     def last_loop_ms(self) -> float:
         """Device milliseconds per decode step of the last decode_loop()."""
         return float(LIB_LLAISYS.llaisysModelLastLoopMs(self._model))
+
+
+class NamedWeightsLM(CausalLM):
+    """A family whose weights are loaded by their checkpoint names (llaisysModelLoadTensor) and whose residual stream is f32. It
+    supplies meta_of() and the library's constructor."""
+    create: str          # C function: (meta *, device, device id) -> handle
+
+    def meta_of(self, config: Mapping, shapes: Mapping[str, tuple[int, ...]], dtype: DataType, max_seq_len: int | None):
+        """The C description of a model: `shapes` holds the shapes of the checkpoint's tensors."""
+        raise NotImplementedError
+
+    def __init__(self, model_path=None, device: DeviceType = DeviceType.NVIDIA, *, device_id: int = 0,
+                 config: Mapping | None = None, state_dict: Mapping | None = None, dtype: DataType | None = None,
+                 max_seq_len: int | None = None):
+        """From a checkpoint directory, or from a config and a state dict of numpy arrays (float32, or bfloat16 as its
+        16-bit words) or torch tensors. dtype: of matrix products and activations; bfloat16 when neither this argument nor
+        the config names one."""
+        files = []
+        if model_path is not None:
+            config = json.loads((Path(model_path) / "config.json").read_text())
+            files = list(checkpoint_files(model_path))
+        if config is None:
+            raise ValueError(f"{type(self).__name__} needs a checkpoint directory or a config")
+        if dtype is None:
+            dtype = DTYPE_NAMES.get(str(config.get("torch_dtype", "bfloat16")), DataType.BF16)
+        shapes = {name: f.shape(name) for f in files for name in f.names()}
+        if state_dict is not None:
+            shapes |= {name: tuple(value.shape) for name, value in state_dict.items()}
+        self.config = dict(config)
+        self.meta = self.meta_of(config, shapes, dtype, max_seq_len)
+        self.vocab, self.max_seq, self.end_token = int(self.meta.voc), int(self.meta.maxseq), int(self.meta.end_token)
+        self.dtype, self.device, self.device_id = dtype, device, device_id
+        self._model = getattr(LIB_LLAISYS, self.create)(ctypes.byref(self.meta), int(device), device_id)
+        if not self._model:
+            raise RuntimeError(f"{self.create} failed: " + (LIB_LLAISYS.llaisysGetLastError() or b"").decode())
+        for f in files:
+            for name in f.names():
+                if f.dtype(name) in LIBRARY_DTYPE:
+                    self._load(name, f.array(name), LIBRARY_DTYPE[f.dtype(name)])
+        for name, value in (state_dict or {}).items():
+            self.load_tensor(name, value)
+        first = ctypes.create_string_buffer(256)
+        n_missing = int(LIB_LLAISYS.llaisysModelMissingTensors(self._model, first, len(first)))
+        if n_missing:
+            raise ValueError(f"checkpoint lacks {n_missing} tensors, e.g. {first.value.decode()}")
+
+    def load_tensor(self, name: str, value) -> None:
+        """Copies one weight: a numpy array (float32 / float16, or uint16 holding bfloat16) or a torch tensor."""
+        if not isinstance(value, np.ndarray):
+            import torch
+            host = value.detach().to("cpu").contiguous()
+            if host.dtype == torch.bfloat16:
+                value = host.view(torch.int16).numpy().view(np.uint16)
+            else:
+                value = host.float().numpy()
+        kind = {np.dtype(np.float32): DataType.F32, np.dtype(np.float16): DataType.F16,
+                np.dtype(np.uint16): DataType.BF16}.get(value.dtype)
+        if kind is None:
+            raise ValueError(f"{name}: unsupported array type {value.dtype}")
+        self._load(name, value, kind)
+
+    def _load(self, name: str, array: np.ndarray, kind: DataType) -> None:
+        array = np.ascontiguousarray(array)
+        shape = (c_size_t * array.ndim)(*array.shape)
+        known = c_int(0)
+        try:
+            _check(LIB_LLAISYS.llaisysModelLoadTensor(self._model, name.encode(), int(kind), shape, array.ndim,
+                                                      array.ctypes.data, ctypes.byref(known)))
+        except LlaisysError as err:
+            raise ValueError(str(err)) from err
+
+    # ---- development aid ------------------------------------------------------------------------------------------------
+
+    def record_stream(self, enable: bool = True) -> None:
+        """Keep the residual stream after every layer run of the steps that follow (slow)."""
+        _check(LIB_LLAISYS.llaisysModelRecordStream(self._model, int(enable)))
+
+    def layer_runs(self) -> int:
+        return len(self.config["layers"])
+
+    def layer_stream(self) -> np.ndarray:
+        """float32 [layer runs, rows, width] of the last step."""
+        n = c_size_t(0)
+        _check(LIB_LLAISYS.llaisysModelLayerStream(self._model, None, 0, ctypes.byref(n)))
+        out = np.zeros(n.value, dtype=np.float32)
+        _check(LIB_LLAISYS.llaisysModelLayerStream(self._model, out.ctypes.data_as(ctypes.POINTER(c_float)), out.size,
+                                                   ctypes.byref(n)))
+        return out.reshape(self.layer_runs(), -1, int(self.meta.width))
+
+
+def tensor_rows(shapes: Mapping[str, tuple[int, ...]], names: Sequence[str]) -> list[int]:
+    """First dimension of each named tensor: sizes that only a checkpoint's weights hold."""
+    missing = [n for n in names if n not in shapes]
+    if missing:
+        raise ValueError(f"checkpoint lacks {len(missing)} tensors, e.g. {missing[:3]}")
+    return [int(shapes[n][0]) for n in names]

@@ -8,13 +8,13 @@ memory; index arguments are Python sequences or numpy int32 arrays on the host.
 from __future__ import annotations
 
 import ctypes
-from ctypes import byref, c_int32
+from ctypes import byref, c_int32, c_size_t
 from enum import IntEnum
 from typing import Sequence
 
 import numpy as np
 
-from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysGatedLinear, LlaisysNormAppend, Status,
+from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysGatedDelta, LlaisysGatedLinear, LlaisysNormAppend, Status,
                          llaisysPagedKV_t)
 from .runtime import _addr
 
@@ -279,21 +279,21 @@ class PagedKVCache:
         return self
 
     def norm_append_dev(self, layer: int, stream, **fields) -> None:
-        """Per-head norm of q and k, append of k and v, gates to factors; fields of LlaisysNormAppend (buffers may be
+        """Per-head norm and rotation of q and k, append of k and v, gates to factors; fields of LlaisysNormAppend (buffers may be
         tensors)."""
-        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev"}
+        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev", "rot_table"}
         args = LlaisysNormAppend(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
         _check(LIB_LLAISYS.llaisysPagedKVNormAppendDev(self._kv, layer, byref(args), stream))
 
     def attention_dev(self, layer: int, out, q, seq_ids_dev, q_starts_dev, kv_lens_dev, *, n_seqs: int, total_q: int,
-                      max_q_len: int, max_kv_len: int, nh: int, scale: float, stream, window: int = 0, row_scale=None,
-                      row_stride: int = 0) -> None:
-        """Decode (q_starts_dev None) or ragged chunks, with a sliding window, a factor per (row, head) and an output row
-        stride."""
+                      max_q_len: int, max_kv_len: int, nh: int, scale: float, stream, window: int = 0, keep_first: int = 0,
+                      row_scale=None, row_stride: int = 0) -> None:
+        """Decode (q_starts_dev None) or ragged chunks, with a sliding window that can keep a sequence's first tokens, a factor
+        per (row, head) and an output row stride."""
         _check(LIB_LLAISYS.llaisysPagedAttentionOptDev(
             self._kv, layer, _addr(out), _addr(q), _addr(seq_ids_dev), None if q_starts_dev is None else _addr(q_starts_dev),
             _addr(kv_lens_dev), n_seqs, total_q, max_q_len, max_kv_len, nh, scale, window,
-            None if row_scale is None else _addr(row_scale), row_stride, stream))
+            keep_first, None if row_scale is None else _addr(row_scale), row_stride, stream))
 
 
 def gated_linear_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
@@ -303,6 +303,27 @@ def gated_linear_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 
                 "scratch_raw", "scratch_decay", "scratch_segments"}
     args = LlaisysGatedLinear(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
     _check(LIB_LLAISYS.llaisysGatedLinearDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
+
+
+def gated_delta_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
+    """Gated delta rule on device buffers; fields of LlaisysGatedDelta (include/llaisys/mixers.h), buffers may be tensors."""
+    pointers = {"proj", "conv_q", "conv_k", "conv_v", "decay_w", "a_log", "dt_bias", "norm_w", "gate", "state", "seq_ids_dev",
+                "q_starts_dev", "kv_lens_dev", "out", "scratch", "scratch_segments"}
+    args = LlaisysGatedDelta(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+    _check(LIB_LLAISYS.llaisysGatedDeltaDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
+
+
+def gated_delta_sizes(dtype: DataType, n_rows: int, heads: int, kv_heads: int, dk: int, dv: int, taps: int) -> tuple[int, int, int]:
+    """Floats of a sequence's state, of `scratch` for n_rows rows and of `scratch_segments`."""
+    sizes = [c_size_t(0) for _ in range(3)]
+    LIB_LLAISYS.llaisysGatedDeltaSizes(int(dtype), n_rows, heads, kv_heads, dk, dv, taps, *[byref(s) for s in sizes])
+    return tuple(int(s.value) for s in sizes)
+
+
+def rotary_table_dev(table, positions_dev, freq_dev, n_rows: int, half: int, *, stream, device_id: int = 0) -> None:
+    """table [n_rows, half, 2] = (cos, sin)(position * freq), f32, on the device."""
+    _check(LIB_LLAISYS.llaisysRotaryTableDev(int(DeviceType.NVIDIA), device_id, _addr(table), _addr(positions_dev), _addr(freq_dev),
+                                             n_rows, half, stream))
 
 
 def gated_linear_segment_floats(dtype: DataType, heads: int, dk: int, dv: int) -> int:
