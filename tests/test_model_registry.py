@@ -11,10 +11,13 @@ import torch
 
 import llaisys_b200 as llaisys
 from llaisys_b200 import trace
-from llaisys_b200.models import Qwen2, Vozozen, load_model, model_class
+from llaisys_b200.models import Doderax, Qwen2, Vozozen, load_model, model_class
+from llaisys_b200.models import doderax as dx
 from llaisys_b200.models import vozozen as vz
 from llaisys_b200.models.weights import SafetensorsFile, checkpoint_files
+from oracle import doderax as doderax_oracle
 from oracle import vozozen as oracle
+from tests import doderax_cases
 from tests import vozozen_cases as cases
 
 
@@ -30,6 +33,7 @@ def write_safetensors(path, tensors):
 
 def test_class_by_config():
     assert model_class({"architecture": "Vozozen"}) is Vozozen
+    assert model_class({"architecture": "Doderax"}) is Doderax
     assert model_class({"architectures": ["Qwen2ForCausalLM"], "model_type": "qwen2"}) is Qwen2
     assert model_class({"model_type": "qwen2"}) is Qwen2
     with pytest.raises(ValueError, match="Mamba"):
@@ -104,6 +108,83 @@ def test_unknown_parts_of_a_configuration_are_refused():
     cfg["layers"][0]["mlp"]["kind"] = "experts"
     with pytest.raises(ValueError, match="experts"):
         vz.build_meta(cfg, ranks, llaisys.DataType.BF16)
+
+
+@pytest.mark.parametrize("name", sorted(doderax_cases.CASES))
+def test_doderax_configuration_reaches_the_library(name):
+    cfg, ranks = doderax_cases.CASES[name]
+    shapes = dx.weight_shapes(cfg, ranks)
+    assert dx.low_ranks(cfg, shapes) == ranks
+    meta = dx.build_meta(cfg, ranks, llaisys.DataType.BF16)
+    pairs = cfg["embedding"]["bigram"]
+    assert (meta.nlayer, meta.width, meta.voc) == (len(cfg["layers"]), cfg["width"], cfg["vocab"])
+    assert (meta.pair_buckets, meta.pair_mul_prev, meta.pair_mul_cur) == (pairs["buckets"], pairs["mul_prev"], pairs["mul_cur"])
+    assert meta.eps == pytest.approx(cfg["norm"]["eps"]) and meta.logit_scale == pytest.approx(cfg["logit_scale"])
+    for i, entry in enumerate(cfg["layers"]):
+        got, mixer = meta.layers[i], entry["mixer"]
+        assert got.ff == (entry["mlp"]["ff"] if entry["mlp"] else 0) and bool(got.parallel) == (entry["type"] == "parallel")
+        delta = mixer["right"] if got.parallel else mixer
+        assert (got.delta.heads, got.delta.kv_heads, got.delta.dim, got.delta.vdim, got.delta.taps, got.delta.decay_rank,
+                got.delta.gate_rank) == (*(delta[k] for k in ("heads", "kv_heads", "dim", "vdim", "conv")), *ranks[i])
+        if got.parallel:
+            a, left = got.attn, mixer["left"]
+            assert (a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.keep_first, a.rot_dims) == (
+                left["heads"], left["kv_heads"], left["dim"], left["vdim"], left["mask"]["size"], left["mask"]["keep_first"],
+                left["rot"]["dims"])
+            assert a.rot_base == left["rot"]["base"] and a.scale == pytest.approx(left["scale"])
+
+
+def test_unknown_parts_of_a_doderax_configuration_are_refused():
+    cfg, _ = doderax_cases.case("mixed")
+    ranks = doderax_cases.CASES["mixed"][1]
+    cfg["layers"][0]["type"] = "serial"
+    with pytest.raises(ValueError, match="serial"):
+        dx.build_meta(cfg, ranks, llaisys.DataType.BF16)
+    cfg, w = doderax_cases.case("mixed")
+    cfg["layers"][1]["mlp"]["kind"] = "experts"
+    with pytest.raises(ValueError, match="experts"):
+        dx.build_meta(cfg, ranks, llaisys.DataType.BF16)
+    cfg, w = doderax_cases.case("mixed")
+    with pytest.raises(ValueError, match="l0.mix.a1"):
+        Doderax(config=cfg, state_dict={k: v for k, v in w.items() if k != "l0.mix.a1"}, device=llaisys.DeviceType.CPU)
+    with pytest.raises(RuntimeError, match="NVIDIA"):
+        Doderax(config=cfg, state_dict=w, device=llaisys.DeviceType.CPU)
+
+
+def test_doderax_oracle_mechanisms_agree_with_closed_forms():
+    torch.manual_seed(1)
+    T, H, d, dv = 10, 2, 6, 5
+    q, k, v = torch.randn(T, H, d).double(), torch.nn.functional.normalize(torch.randn(T, H, d).double(), dim=-1), torch.randn(T, H, dv).double()
+    none, one = torch.zeros(T, H, d).double(), torch.ones(T, H).double()
+    # orthogonal keys: nothing to correct, plain sums of outer products
+    basis = torch.eye(d).double()[[0, 1, 2, 3, 4, 5]].unsqueeze(1).expand(d, H, d)
+    _, S = doderax_oracle.delta_rule(q[:d], basis, v[:d], none[:d], one[:d])
+    assert torch.allclose(S, v[:d].transpose(0, 1))
+    # full write strength: the newest key reads its own value back, with any decay
+    log = doderax_oracle.decay_log(torch.tensor(0.3).double(), torch.randn(T, H, d).double())
+    y, S = doderax_oracle.delta_rule(k, k, v, log, one)
+    assert torch.allclose(y, v) and (log < 0).all()
+    # no write strength: the state only decays
+    _, S1 = doderax_oracle.delta_rule(q, k, v, log, 0 * one, state=S)
+    assert torch.allclose(S1, S * torch.exp(log.sum(0)).unsqueeze(2))
+    assert torch.allclose(doderax_oracle.decay_log(torch.zeros(1).double(), torch.zeros(1).double()), -torch.tensor([2.0]).double().log())
+    # rotation: lengths stay, equal distances give equal products, position 0 and the unrotated dims pass
+    x = torch.randn(1, 1, 8).double().expand(9, 1, 8)
+    r = doderax_oracle.rotate(x, 6, 50.0)
+    assert torch.allclose(r.norm(dim=-1), x.norm(dim=-1)) and torch.allclose(r[0], x[0]) and torch.equal(r[..., 6:], x[..., 6:])
+    dots = torch.einsum("ihd,jhd->ij", r, r)
+    assert torch.allclose(dots[2, 0], dots[8, 6])
+    # a window that covers everything, and one of a single token beside kept ones
+    args = q, k, v
+    full = doderax_oracle.sink_attention(*args, 0.7, T, 0)
+    assert torch.allclose(full, doderax_oracle.sink_attention(*args, 0.7, 1, T)) and torch.allclose(full, oracle.window_attention(*args, 0.7, T))
+    assert torch.allclose(doderax_oracle.sink_attention(*args, 0.7, 1, 0), v)
+    w = torch.zeros(3, 4).double()
+    w[:, -1] = 1.0
+    y = torch.randn(7, 3).double()
+    assert torch.allclose(doderax_oracle.short_conv(y, w), oracle.silu(y))
+    assert doderax_oracle.pair_rows([3, 4, 3], {"buckets": 10, "mul_prev": 2, "mul_cur": 5}) == [10, 6, 3]
+    assert torch.allclose(doderax_oracle.gelu(y), torch.nn.functional.gelu(y, approximate="tanh"))
 
 
 def test_no_host_stand_in():

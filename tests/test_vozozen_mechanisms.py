@@ -55,7 +55,7 @@ class Pool:
                                    n_rows=len(ids), nh=1)
         self.cache.check()
 
-    def attend(self, q, q_lens, kv_lens, nh, scale, window, factor, decode):
+    def attend(self, q, q_lens, kv_lens, nh, scale, window, factor, decode, keep_first=0):
         n = len(q_lens)
         rows = sum(q_lens)
         width = nh * self.dv + 24
@@ -63,21 +63,22 @@ class Pool:
         starts = i32([0, *np.cumsum(q_lens).tolist()])
         self.cache.attention_dev(0, out, q.cuda().contiguous(), i32(self.seqs[:n]), None if decode else starts, i32(kv_lens),
                                  n_seqs=n, total_q=rows, max_q_len=max(q_lens), max_kv_len=max(kv_lens), nh=nh, scale=scale,
-                                 stream=stream(), window=window, row_scale=factor.cuda() if factor is not None else None,
+                                 stream=stream(), window=window, keep_first=keep_first, row_scale=factor.cuda() if factor is not None else None,
                                  row_stride=width)
         self.cache.check()
         assert torch.all(out[:, nh * self.dv:] == 7.0), "columns behind the heads were written"
         return out[:, :nh * self.dv].reshape(rows, nh, self.dv).cpu()
 
-    def expect(self, q, q_lens, kv_lens, scale, window, factor):
+    def expect(self, q, q_lens, kv_lens, scale, window, factor, keep_first=0):
         outs, at = [], 0
         for i, (n, kv) in enumerate(zip(q_lens, kv_lens)):
             share = q.shape[1] // self.nkvh
             for t in range(n):
                 last = kv - n + t
                 first = max(0, last - window + 1) if window else 0
-                k = self.k[i][first:last + 1].double().repeat_interleave(share, 1)
-                v = self.v[i][first:last + 1].double().repeat_interleave(share, 1)
+                seen = [*range(min(keep_first, first)), *range(first, last + 1)]
+                k = self.k[i][seen].double().repeat_interleave(share, 1)
+                v = self.v[i][seen].double().repeat_interleave(share, 1)
                 s = torch.einsum("jhd,hd->hj", k, q[at].double()) * scale
                 o = torch.einsum("hj,jhd->hd", s.softmax(-1), v)
                 outs.append(o * (factor[at].double().unsqueeze(1) if factor is not None else 1.0))
