@@ -16,6 +16,7 @@ random permutation of a 16384-page pool):
   config3     chunked prefill: 8 sequences, context ~ U{0..8192}, a 512-token chunk appended and attended causally
   config5     one 131072-token sequence, 28 layers, KV range split over the GPUs, partial results exchanged and merged
   vozozen     the Vozozen design beside Qwen2 at equal size: whole models and single kernels (bench_models.py)
+  doderax     the Doderax design beside Vozozen, in the same way
 The default run (north_star) also measures config2 and config3 in the same process (N = 1: sub-records "config2",
 "config3") and, with N > 1, the KV-range split of config5 in the same process group (sub-record "kv_split"): the one
 mode of this path in which GPUs exchange data.
@@ -1283,7 +1284,7 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=100, help="steps per timed graph replay (the graph is replayed >= 30 times)")
     ap.add_argument("--warmup", type=int, default=20)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="north_star", choices=["north_star", "config2", "config3", "config4", "config5", "copy", "vozozen"])
+    ap.add_argument("--workload", default="north_star", choices=["north_star", "config2", "config3", "config4", "config5", "copy", "vozozen", "doderax"])
     ap.add_argument("--layers", type=int, default=4, help="pools to rotate over between steps (L2 flush)")
     ap.add_argument("--repeats", type=int, default=100, help="replays of the timed graph (at least 30)")
     ap.add_argument("--tp", action="store_true", help="config4 on several GPUs: tensor parallelism instead of sequence sharding")
@@ -1316,7 +1317,7 @@ def main() -> None:
     if args.workload == "copy":
         run_copy_workload(args)
         return
-    if args.workload == "vozozen":
+    if args.workload in ("vozozen", "doderax"):
         import bench_models
 
         bench_models.run(args)

@@ -1,10 +1,12 @@
-"""bench.py --workload vozozen: the Vozozen design beside Qwen2 at equal size, one GPU.
+"""bench.py --workload vozozen | doderax: a design beside its closest relative at equal size, one GPU -- Vozozen beside Qwen2,
+Doderax beside Vozozen.
 
 Two parts, one JSON line:
   models   prefill and decode throughput of whole models with random weights. Equal size: the same width, query and kv heads,
-           layers and vocabulary, and an MLP of as many parameters (Vozozen's has two matrices, so its inner size is 1.5 times
-           Qwen2's three). Vozozen's second mixer (gated linear attention) comes on top.
-  kernels  every new kernel alone next to the like kernel of Qwen2, each as a fraction of its own roofline: CUDA graphs of
+           layers and vocabulary, and an MLP of as many parameters (two matrices have an inner size 1.5 times that of Qwen2's
+           three). Vozozen's second mixer (gated linear attention) comes on top of Qwen2's attention; Doderax has as many heads of
+           the delta rule in every layer, and attention in every other one.
+  kernels  every new kernel alone next to the like kernel of the relative, each as a fraction of its own roofline: CUDA graphs of
            launches over rotating buffers larger than L2, the median of the replays.
 """
 from __future__ import annotations
@@ -21,6 +23,7 @@ SIZES = {
 D = 128
 PREFILL = {"one prompt of 8192": [8192], "eight prompts of 1024": [1024] * 8}
 DECODE_SEQS, DECODE_CTX, DECODE_STEPS = 64, 2048, 64
+KEEP_FIRST, TAPS, LOW_RANK = 64, 4, 128  # Doderax: kept first tokens, convolution taps, ranks of its decay and gate projections
 
 
 def vozozen_config(s: dict) -> dict:
@@ -38,6 +41,23 @@ def qwen2_config(s: dict) -> dict:
             "rope_theta": 1e6}
 
 
+def doderax_config(s: dict) -> dict:
+    def delta(kv_heads):
+        return {"heads": s["gla_heads"], "kv_heads": kv_heads, "dim": D, "vdim": D, "conv": TAPS}
+
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "mask": {"size": s["window"], "keep_first": KEEP_FIRST},
+            "rot": {"dims": D, "base": 1e6}, "scale": D ** -0.5}
+    mlp = {"kind": "dense", "ff": s["ff"] * 3 // 2}
+    layers = [{"type": "channel_delta", "mixer": delta(s["gla_heads"]), "mlp": mlp},
+              {"type": "parallel", "mixer": {"left": left, "right": delta(s["gla_heads"] // 2)}, "mlp": mlp}]
+    return {"architecture": "Doderax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}, "layers": layers * (s["layers"] // 2)}
+
+
+def attention_layers(family: str, s: dict) -> int:
+    return s["layers"] // 2 if family == "doderax" else s["layers"]
+
+
 def build_model(torch, llaisys, family: str, s: dict):
     """-> the model, bytes of weights a decode step reads, parameters of the matrices applied to every token"""
     if family == "qwen2":
@@ -53,39 +73,55 @@ def build_model(torch, llaisys, family: str, s: dict):
                 total += value.numel() * 2
                 per_token += value.numel() if value.ndim == 2 and name != "lm_head.weight" else 0
         return model, total, per_token
-    from llaisys_b200.models.vozozen import weight_shapes
+    if family == "doderax":
+        from llaisys_b200.models.doderax import weight_shapes
 
-    cfg = vozozen_config(s)
+        cfg = doderax_config(s)
+        shapes = weight_shapes(cfg, [(LOW_RANK, LOW_RANK)] * s["layers"])
+    else:
+        from llaisys_b200.models.vozozen import weight_shapes
+
+        cfg = vozozen_config(s)
+        shapes = weight_shapes(cfg, [16] * s["layers"])
     g = torch.Generator(device="cuda").manual_seed(4)
     weights, total, per_token = {}, 0, 0
-    for name, shape in weight_shapes(cfg, [16] * s["layers"]).items():
-        if name.endswith(("norm", "norm1", "norm2")):
+    for name, shape in shapes.items():
+        if name.endswith(("norm", "norm1", "norm2", ".out")):
             w = torch.ones(shape)
-        elif name.endswith("a2.b"):
-            w = torch.full(shape, 3.0)
+        elif name.endswith(("a2.b", "dt_bias")):
+            w = torch.full(shape, 3.0 if family == "vozozen" else -5.0)
+        elif name.endswith("A_log"):
+            w = torch.zeros(shape)
+        elif name.endswith(".conv"):
+            w = torch.randn(shape, generator=g, device="cuda") * 0.5
         else:
             w = torch.randn(shape, generator=g, device="cuda") * 0.02
         weights[name] = w.bfloat16().cpu().view(torch.int16).numpy().view(np.uint16)
-        if name != "embed":
+        if name not in ("embed", "bigram"):
             total += w.numel() * 2
-            per_token += w.numel() if w.ndim == 2 and name != "head" else 0
-    model = llaisys.models.Vozozen(config=cfg, state_dict=weights, dtype=llaisys.DataType.BF16)
+            per_token += w.numel() if w.ndim == 2 and name != "head" and not name.endswith(".conv") else 0
+    cls = llaisys.models.Doderax if family == "doderax" else llaisys.models.Vozozen
+    model = cls(config=cfg, state_dict=weights, dtype=llaisys.DataType.BF16)
     return model, total, per_token
 
 
-def visible(n: int, window: int | None) -> int:
+def visible(n: int, window: int | None, keep: int = 0) -> int:
     """(query, key) pairs of a causal run of n tokens from an empty cache"""
     full = n * (n + 1) // 2
-    return full if window is None or window >= n else full - (n - window) * (n - window + 1) // 2
+    if window is None or window >= n:
+        return full
+    out = n - window  # queries behind a full window; the i-th of them misses i tokens, `keep` of which it sees all the same
+    kept = sum(min(i, keep) for i in range(1, min(out, keep) + 1)) + max(out - keep, 0) * keep
+    return full - out * (out + 1) // 2 + kept
 
 
 def prefill_flops(family: str, s: dict, lens: list[int], per_token: int) -> float:
     tokens = sum(lens)
     flops = 2.0 * tokens * per_token + 2.0 * len(lens) * s["vocab"] * s["width"]
-    window = s["window"] if family == "vozozen" else None
-    flops += s["layers"] * s["heads"] * 4.0 * D * sum(visible(n, window) for n in lens)
-    if family == "vozozen":
-        flops += s["layers"] * s["gla_heads"] * tokens * 4.0 * D * D  # state update and read-out
+    window, keep = (None if family == "qwen2" else s["window"]), (KEEP_FIRST if family == "doderax" else 0)
+    flops += attention_layers(family, s) * s["heads"] * 4.0 * D * sum(visible(n, window, keep) for n in lens)
+    if family != "qwen2":  # state update and read-out, and the delta rule's correction
+        flops += s["layers"] * s["gla_heads"] * tokens * (6.0 if family == "doderax" else 4.0) * D * D
     return flops
 
 
@@ -121,9 +157,11 @@ def measure_model(torch, llaisys, stream, family: str, s: dict, repeats: int) ->
     nxt = model.decode_loop(seqs, nxt, 8)[-1].tolist()
     model.decode_loop(seqs, nxt, DECODE_STEPS + 1)
     ms = model.last_loop_ms
-    keys = min(DECODE_CTX + DECODE_STEPS // 2, s["window"]) if family == "vozozen" else DECODE_CTX + DECODE_STEPS // 2
-    kv = s["layers"] * DECODE_SEQS * keys * s["kv_heads"] * 2 * D * 2
-    state = 2 * s["layers"] * DECODE_SEQS * s["gla_heads"] * D * D * 4 if family == "vozozen" else 0
+    keys = DECODE_CTX + DECODE_STEPS // 2
+    if family != "qwen2":
+        keys = min(keys, s["window"] + (KEEP_FIRST if family == "doderax" else 0))
+    kv = attention_layers(family, s) * DECODE_SEQS * keys * s["kv_heads"] * 2 * D * 2
+    state = 2 * s["layers"] * DECODE_SEQS * s["gla_heads"] * D * D * 4 if family != "qwen2" else 0
     moved = weight_bytes + kv + state
     rec["decode"] = {"tokens_per_s": DECODE_SEQS * 1e3 / ms, "ms_per_step": ms, "bytes": {"weights": weight_bytes, "kv": kv, "state": state},
                      "gb_per_s": moved / ms / 1e6, "frac_of_copy": moved / ms / 1e6 / hbm, "peak_kind": kind}
@@ -171,9 +209,9 @@ class Kernels:
     def tensor(self, us: float, flops: float) -> dict:
         return {"us": us, "tflops": flops / us / 1e6, "frac": flops / us / 1e6 / self.burst, "of": f"{self.kind} burst bf16 GEMM"}
 
-    def attention(self, heads: int, kv_heads: int, window: int, layers: int = 3) -> dict:
+    def attention(self, heads: int, kv_heads: int, window: int, layers: int = 3, design: str = "vozozen") -> dict:
         """Decode over 64 sequences and one chunk of 8192 tokens, with the window and without one at equal visible keys /
-        at full length; the position-wise kernel in front of each."""
+        at full length (doderax: with kept first tokens and without); the position-wise kernel in front of each."""
         torch, ll = self.torch, self.ll
         out = {}
         n_seqs, ctx, rows = 64, 2 * window, 8192
@@ -201,8 +239,13 @@ class Kernels:
         us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, None, full, total_q=n_seqs, max_q_len=1, max_kv_len=ctx,
                                                      window=window, row_scale=factor, **common))
         out["decode attention, window"] = self.memory(us, kv_bytes)
-        us = self.time(lambda i: cache.decode_dev(i % layers, o, q, ids, short, n_seqs, window, heads, D ** -0.5, self.cs))
-        out["decode attention, Qwen2, as many keys"] = self.memory(us, kv_bytes)
+        if design == "doderax":
+            us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, None, full, total_q=n_seqs, max_q_len=1, max_kv_len=ctx,
+                                                         window=window, keep_first=KEEP_FIRST, **common))
+            out["decode attention, window and kept tokens"] = self.memory(us, kv_bytes * (window + KEEP_FIRST) // window)
+        else:
+            us = self.time(lambda i: cache.decode_dev(i % layers, o, q, ids, short, n_seqs, window, heads, D ** -0.5, self.cs))
+            out["decode attention, Qwen2, as many keys"] = self.memory(us, kv_bytes)
 
         qn, kn = self.rand(D), self.rand(D)
         wide = width + heads  # the gate behind q | k | v
@@ -224,6 +267,14 @@ class Kernels:
                 v_at=(heads + kv_heads) * D, gate_at=width, q_norm=qn, k_norm=kn, eps=1e-6, gate_scale=0.7, q_out=qo, row_scale=fac,
                 seq_ids_dev=ids_n, positions_dev=pos_n, n_rows=n, nh=heads))
             out[f"norm + append, {n} rows"] = self.memory(us, moved)
+            if design == "doderax":
+                table = torch.rand(n, D // 2, 2, device="cuda")
+                us = self.time(lambda i: cache.norm_append_dev(
+                    i % layers, self.cs, proj=proj[i % layers], row_stride=proj[0].shape[1], q_at=0, k_at=heads * D,
+                    v_at=(heads + kv_heads) * D, gate_at=-1, q_norm=None, k_norm=None, eps=1e-6, gate_scale=1.0, q_out=qo, row_scale=None,
+                    seq_ids_dev=ids_n, positions_dev=pos_n, n_rows=n, nh=heads, rot_dims=D, rot_table=table))
+                out[f"rotation + append, {n} rows"] = self.memory(us, n * (2 * width * 2 + D * 4))
+                continue
             packed = [self.rand(n, width) for _ in range(layers)]
             bias = self.rand(width)
             us = self.time(lambda i: self._rope_append(cache, i % layers, qo, packed[i % layers], bias, ids_n, pos_n, n, heads))
@@ -234,8 +285,12 @@ class Kernels:
         common = dict(n_seqs=1, total_q=rows, max_q_len=rows, max_kv_len=rows, nh=heads, scale=D ** -0.5, stream=self.cs)
         us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, lens, window=window, row_scale=factor, **common))
         out["chunk attention, window, 8192 tokens"] = self.tensor(us, 4.0 * D * heads * visible(rows, window))
-        us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, lens, **common))
-        out["chunk attention, Qwen2, 8192 tokens"] = self.tensor(us, 4.0 * D * heads * visible(rows, None))
+        if design == "doderax":
+            us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, lens, window=window, keep_first=KEEP_FIRST, **common))
+            out["chunk attention, window and kept tokens, 8192 tokens"] = self.tensor(us, 4.0 * D * heads * visible(rows, window, KEEP_FIRST))
+        else:
+            us = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, lens, **common))
+            out["chunk attention, Qwen2, 8192 tokens"] = self.tensor(us, 4.0 * D * heads * visible(rows, None))
         cache.check()
         cache.close()
         return out
@@ -273,31 +328,72 @@ class Kernels:
         return rec
 
 
+    def gated_delta(self, heads: int, kv_heads: int, lens: list[int], rank: int, copies: int = 3) -> dict:
+        """rank 0: one decay per head"""
+        torch, ll = self.torch, self.ll
+        decode, rows, nq, nv = max(lens) == 1, sum(lens), kv_heads * D, heads * D
+        at, width = {}, 0
+        for name, n in (("q", nq), ("k", nq), ("v", nv), ("b", heads), ("a", rank or heads), ("g", nv)):
+            at[name], width = width, width + (n + 7) // 8 * 8
+        copies = copies if decode or rows * width * 2 < 300e6 else 2
+        proj = [self.rand(rows, width, scale=0.7) for _ in range(copies)]
+        floats, n_scratch, n_seg = ll.gated_delta_sizes(ll.DataType.BF16, rows, heads, kv_heads, D, D, TAPS)
+        state = [torch.zeros(len(lens), floats, device="cuda") for _ in range(copies)]
+        conv = {f"conv_{n}": self.rand(m, TAPS, scale=0.5) for n, m in (("q", nq), ("k", nq), ("v", nv))}
+        w = self.rand(nv, rank, scale=0.3) if rank else None
+        bias, a_log, norm = self.rand(nv if rank else heads) - 5, self.rand(heads, scale=0.1), self.rand(D)
+        out, scratch, seg = self.rand(rows, nv), torch.empty(n_scratch, device="cuda"), torch.empty(n_seg, device="cuda")
+        ids, starts = self.i32(list(range(len(lens)))), self.i32([0, *np.cumsum(lens).tolist()])
+        kv = self.i32([x + 100 for x in lens])
+        us = self.time(lambda i: ll.gated_delta_dev(
+            ll.DataType.BF16, decode=decode, stream=self.cs, proj=proj[i % copies], row_stride=width, q_at=at["q"], k_at=at["k"],
+            v_at=at["v"], b_at=at["b"], a_at=at["a"], **conv, decay_w=w, decay_ld=rank, a_log=a_log, dt_bias=bias, norm_w=norm,
+            gate=proj[i % copies].data_ptr() + at["g"] * 2, gate_stride=width, gate_silu=1, q_scale=D ** -0.5, eps=1e-6, unit_eps=1e-6,
+            taps=TAPS, heads=heads, kv_heads=kv_heads, dk=D, dv=D, rank=rank, state=state[i % copies], slot_stride=floats,
+            seq_ids_dev=ids, q_starts_dev=starts, kv_lens_dev=kv, n_seqs=len(lens), n_rows=rows, max_q_len=max(lens), out=out,
+            out_stride=nv, scratch=scratch, scratch_floats=n_scratch, scratch_segments=seg, scratch_segment_floats=n_seg))
+        rec = self.memory(us, rows * (width + nv) * 2 + 2 * len(lens) * floats * 4)
+        if not decode:
+            rec["f32_tflops_of_the_recurrence"] = rows * heads * 6.0 * D * D / us / 1e6
+        return rec
+
+
 def run(args) -> None:
     from bench import ClockSampler, _init_device
 
     torch, llaisys, rank, local_rank, world, _ = _init_device()
     if world != 1:
-        raise SystemExit("--workload vozozen runs on one GPU")
+        raise SystemExit(f"--workload {args.workload} runs on one GPU")
     handle = llaisys.context_stream()
     stream = torch.cuda.ExternalStream(int(getattr(handle, "value", handle)))
     repeats = 10 if args.repeats == 100 else max(3, args.repeats)
+    design = args.workload
+    relative = {"vozozen": "qwen2", "doderax": "vozozen"}[design]
+    chunks = {"one run of 8192": [8192], "eight runs of 1024": [1024] * 8}
     models, kernels = {}, {}
     with ClockSampler(local_rank) as clocks:
         for name, s in SIZES.items():
-            models[name] = {"size": s, **{f: measure_model(torch, llaisys, stream, f, s, repeats) for f in ("vozozen", "qwen2")}}
+            models[name] = {"size": s, **{f: measure_model(torch, llaisys, stream, f, s, repeats) for f in (design, relative)}}
             k = Kernels(torch, llaisys, stream, max(30, repeats))
-            kernels[name] = k.attention(s["heads"], s["kv_heads"], s["window"])
-            kernels[name]["gated linear decode, 64 sequences"] = k.gated_linear(s["gla_heads"], [1] * 64)
-            kernels[name]["gated linear chunk, one run of 8192"] = k.gated_linear(s["gla_heads"], [8192])
-            kernels[name]["gated linear chunk, eight runs of 1024"] = k.gated_linear(s["gla_heads"], [1024] * 8)
-    value = models["8B-like"]["vozozen"]["decode"]["tokens_per_s"]
+            kernels[name] = k.attention(s["heads"], s["kv_heads"], s["window"], design=design)
+            h = s["gla_heads"]
+            kernels[name]["gated linear decode, 64 sequences"] = k.gated_linear(h, [1] * 64)
+            if design == "doderax":
+                kernels[name]["gated delta decode, decay per channel, 64 sequences"] = k.gated_delta(h, h, [1] * 64, 16)
+                kernels[name][f"gated delta decode, decay per channel of rank {LOW_RANK}, 64 sequences"] = k.gated_delta(h, h, [1] * 64, LOW_RANK)
+                kernels[name]["gated delta decode, decay per head, 64 sequences"] = k.gated_delta(h, h // 2, [1] * 64, 0)
+            for what, lens in chunks.items():
+                kernels[name]["gated linear chunk, " + what] = k.gated_linear(h, lens)
+                if design == "doderax":
+                    kernels[name]["gated delta chunk, decay per channel, " + what] = k.gated_delta(h, h, lens, 16)
+                    kernels[name][f"gated delta chunk, decay per channel of rank {LOW_RANK}, " + what] = k.gated_delta(h, h, lens, LOW_RANK)
+                    kernels[name]["gated delta chunk, decay per head, " + what] = k.gated_delta(h, h // 2, lens, 0)
+    decode = models["8B-like"][design]["decode"]
     print(json.dumps({
-        "metric": "decode tokens/s (Vozozen, 8B-like layers, greedy)", "value": value, "unit": "tokens/s", "n_gpus": 1,
-        "steps": DECODE_STEPS, "warmup": 8, "ms_per_step": models["8B-like"]["vozozen"]["decode"]["ms_per_step"],
-        "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
-        "data": "synthetic (random weights, random-token prompts)",
-        "config": {"workload": "vozozen", "decode": f"{DECODE_SEQS} sequences, {DECODE_CTX}-token prompts", "prefill": list(PREFILL),
+        "metric": f"decode tokens/s ({design.capitalize()}, 8B-like layers, greedy)", "value": decode["tokens_per_s"], "unit": "tokens/s",
+        "n_gpus": 1, "steps": DECODE_STEPS, "warmup": 8, "ms_per_step": decode["ms_per_step"], "higher_is_better": True,
+        "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic (random weights, random-token prompts)",
+        "config": {"workload": design, "decode": f"{DECODE_SEQS} sequences, {DECODE_CTX}-token prompts", "prefill": list(PREFILL),
                    "l2": "weights, caches and rotated kernel buffers are larger than L2"},
         "models": models, "kernels": kernels, "clocks": clocks.summary(),
         "timing": "CUDA events: prefill around step(), decode around the library's graph replays, kernels around graph replays (median)",

@@ -37,7 +37,7 @@ namespace {
 constexpr int kTile = 32;
 constexpr float kMaxDecay = 80.f;       // log2 units
 constexpr float kMaxTokenDecay = 160.f; // log2: one token's decay is cut here, where it is zero in f32
-constexpr int kMaxRank = 256;
+constexpr int kMaxRank = 512;
 constexpr int kMaxCtas = 148; // (pairs x segments) of a launch that is cut
 constexpr int kMinSegments = 3; // two passes over the state instead of one: fewer segments do not pay
 constexpr int kAStride = 36;  // floats per column of A
@@ -879,7 +879,7 @@ void gated_delta_tiles(stream_t stream, const GatedDeltaArgs &a) {
     auto aligned = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     CHECK_ARGUMENT(aligned(a.gate) && a.gate_stride % 8 == 0 && aligned(a.out) && a.out_stride % 8 == 0, "gated delta rule: gate and output rows must be 16-byte aligned");
     CHECK_ARGUMENT(a.decay_w == nullptr || (a.rank <= kMaxRank && aligned(a.proj) && a.row_stride % 8 == 0 && a.a_at % 8 == 0),
-                   "gated delta rule: decay inputs must be 16-byte aligned, at most 256 per token");
+                   "gated delta rule: decay inputs must be 16-byte aligned, at most 512 per token");
     const DeltaScratch at = delta_scratch(LLAISYS_DTYPE_BF16, a.n_rows, a.heads, a.kv_heads, a.dk, a.dv);
     const int slices = (a.dv + 127) / 128;
     const int64_t pairs = int64_t(a.n_seqs) * a.heads;
