@@ -21,7 +21,7 @@ namespace llaisys::kernels {
 
 namespace {
 
-constexpr int kDecodeThreads = 256;
+constexpr int kDecodeThreads = 512;
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -47,18 +47,47 @@ __device__ void keep_inputs(const GatedDeltaArgs &a, int head, int64_t slot, int
     }
 }
 
-// thread = (VEC columns, every row_groups-th of the dk rows, NR of them at most)
+// Sum over ranks of w[r] z[r], by the four neighbouring lanes `lane4` = 0 .. 3 of one channel; every one gets the sum.
+template <typename T>
+__device__ __forceinline__ float decay_product(const T *w, const float *z, int rank, bool wide, int lane4) {
+    float acc = 0.f;
+    constexpr int kVec = 16 / int(sizeof(T));
+    if (wide) { // rows of w in whole 16-byte pieces (padding included, which meets zeros in z)
+        using P = Pieces<T, kVec>;
+#pragma unroll 4
+        for (int r = lane4 * kVec; r < rank; r += 4 * kVec) {
+            const P p = *reinterpret_cast<const P *>(w + r);
+#pragma unroll
+            for (int e = 0; e < kVec; ++e) {
+                acc = fmaf(to_f32(p.v[e]), z[r + e], acc);
+            }
+        }
+    } else {
+#pragma unroll 4
+        for (int r = lane4; r < rank; r += 4) {
+            acc = fmaf(to_f32(w[r]), z[r], acc);
+        }
+    }
+    acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+    return acc + __shfl_xor_sync(0xffffffffu, acc, 2);
+}
+
+// thread = (VEC columns, every row_groups-th of the dk rows, NR of them at most). Everything that no kernel of this step writes
+// is fetched before the wait for the previous kernel: the state, the convolutions' earlier inputs and weights.
 template <typename T, int VEC, int NR>
-__global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(GatedDeltaArgs a, int col_groups) {
+__global__ void __launch_bounds__(kDecodeThreads, 2) gated_delta_decode_kernel(GatedDeltaArgs a, int col_groups, int wide_decay) {
     extern __shared__ __align__(16) float smem[];
-    float *s_q = smem;              // [dk] unit vectors
-    float *s_k = s_q + a.dk;        // [dk]
-    float *s_a = s_k + a.dk;        // [dk] decay
-    float *s_v = s_a + a.dk;        // [dv]
-    float *s_o = s_v + a.dv;        // [dv]
-    float *s_z = s_o + a.dv;        // [rank]
-    float *s_part = s_z + a.rank;   // [row groups][columns of a pass]
-    __shared__ float s_red[2][kDecodeThreads / 32];
+    auto up4 = [](int n) { return (n + 3) / 4 * 4; };
+    const int rank_pad = (a.rank + 31) / 32 * 32;
+    float *s_q = smem;                   // [dk] unit vectors
+    float *s_k = s_q + up4(a.dk);        // [dk]
+    float *s_a = s_k + up4(a.dk);        // [dk] decay
+    float *s_v = s_a + up4(a.dk);        // [dv]
+    float *s_o = s_v + up4(a.dv);        // [dv]
+    float *s_z = s_o + up4(a.dv);        // [rank, padded]
+    float *s_u = s_z + rank_pad;         // [columns of a pass]
+    float *s_part = s_u + up4(col_groups * VEC); // [row groups][columns of a pass]
+    __shared__ float s_red[3][kDecodeThreads / 32];
 
     const int head = int(blockIdx.x) % a.heads, i = int(blockIdx.x) / a.heads;
     const int tid = int(threadIdx.x), warp = tid >> 5, lane = tid & 31;
@@ -75,7 +104,6 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(Gate
     }
     const bool fresh = pos == 0;
 
-    // ---- this thread's piece of the state (nothing of it is written by the kernel before this one) ----------------------
     float *state = a.state + slot * a.slot_stride + int64_t(head) * a.dk * a.dv;
     using F = Pieces<float, VEC>;
     const int row_groups = kDecodeThreads / col_groups, cg = tid % col_groups, rg = tid / col_groups;
@@ -95,23 +123,54 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(Gate
         }
     };
     load(cg * VEC);
+
+    // ---- convolutions: channel j of this head's q | k | v ---------------------------------------------------------------
+    const int group = a.heads / a.kv_heads, kvh = head / group, nq = a.kv_heads * a.dk, channels = a.channels();
+    float *ring = delta_ring(a, slot);
+    auto channel = [&](int j) {
+        return j < a.dk ? kvh * a.dk + j : (j < 2 * a.dk ? nq + kvh * a.dk + (j - a.dk) : 2 * nq + head * a.dv + (j - 2 * a.dk));
+    };
+    auto history = [&](int ch, float &w_now) { // what the earlier inputs add to the channel's sum
+        const T *w = delta_taps<T>(a, ch);
+        w_now = to_f32(w[a.taps - 1]);
+        float x[3], y[3], acc = 0.f;
+#pragma unroll
+        for (int b = 1; b <= 3; ++b) {
+            const bool in = b < a.taps && b <= pos;
+            x[b - 1] = in ? ring[int64_t((pos - b) % a.taps) * channels + ch] : 0.f;
+            y[b - 1] = in ? to_f32(w[a.taps - 1 - b]) : 0.f;
+        }
+#pragma unroll
+        for (int b = 0; b < 3; ++b) {
+            acc = fmaf(x[b], y[b], acc);
+        }
+        for (int b = 4; b < a.taps && b <= pos; ++b) {
+            acc = fmaf(ring[int64_t((pos - b) % a.taps) * channels + ch], to_f32(w[a.taps - 1 - b]), acc);
+        }
+        return acc;
+    };
+    const int n_channels = 2 * a.dk + a.dv;
+    float w_now = 0.f, acc_first = tid < n_channels ? history(channel(tid), w_now) : 0.f;
+    const float a_log = to_f32(static_cast<const T *>(a.a_log)[head]);
+    const float norm = tid < a.dv ? to_f32(static_cast<const T *>(a.norm_w)[tid]) : 0.f;
     grid_dependency_wait();
     grid_launch_dependents();
 
-    // ---- convolutions, decay inputs -------------------------------------------------------------------------------------
     const T *row = static_cast<const T *>(a.proj) + int64_t(row_i) * a.row_stride;
-    const int group = a.heads / a.kv_heads, kvh = head / group, nq = a.kv_heads * a.dk, channels = a.channels();
-    float *ring = delta_ring(a, slot);
-    float ss[2] = {0.f, 0.f};
-    for (int j = tid; j < 2 * a.dk + a.dv; j += kDecodeThreads) {
-        const int part = j < a.dk ? 0 : (j < 2 * a.dk ? 1 : 2);
-        const int ch = part == 0 ? kvh * a.dk + j : (part == 1 ? nq + kvh * a.dk + (j - a.dk) : 2 * nq + head * a.dv + (j - 2 * a.dk));
-        const T *w = delta_taps<T>(a, ch);
-        const float now = to_f32(row[delta_input_at(a, ch)]);
-        float acc = now * to_f32(w[a.taps - 1]);
-        for (int b = 1; b < a.taps && b <= pos; ++b) {
-            acc = fmaf(ring[int64_t((pos - b) % a.taps) * channels + ch], to_f32(w[a.taps - 1 - b]), acc);
+    const T *gate = static_cast<const T *>(a.gate) + int64_t(row_i) * a.gate_stride + int64_t(head) * a.dv;
+    const float gate_in = tid < a.dv ? to_f32(gate[tid]) : 0.f;
+    const float beta = sigmoid_of(to_f32(row[a.b_at + head]));
+    if (a.decay_w != nullptr) {
+        for (int r = tid; r < rank_pad; r += kDecodeThreads) {
+            s_z[r] = r < a.rank ? to_f32(row[a.a_at + r]) : 0.f;
         }
+    }
+    float ss[2] = {0.f, 0.f};
+    for (int j = tid; j < n_channels; j += kDecodeThreads) {
+        const int ch = channel(j), part = j < a.dk ? 0 : (j < 2 * a.dk ? 1 : 2);
+        const float now = to_f32(row[delta_input_at(a, ch)]);
+        float acc = j == tid ? acc_first : history(ch, w_now);
+        acc = fmaf(now, w_now, acc);
         if (part == 2 || head % group == 0) {
             ring[int64_t(pos % a.taps) * channels + ch] = now; // (no other CTA reads this place in this launch)
         }
@@ -120,11 +179,6 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(Gate
         ss[0] += part == 0 ? y * y : 0.f;
         ss[1] += part == 1 ? y * y : 0.f;
     }
-    if (a.decay_w != nullptr) {
-        for (int r = tid; r < a.rank; r += kDecodeThreads) {
-            s_z[r] = to_f32(row[a.a_at + r]);
-        }
-    }
     ss[0] = warp_sum(ss[0]);
     ss[1] = warp_sum(ss[1]);
     if (lane == 0) {
@@ -132,33 +186,51 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(Gate
         s_red[1][warp] = ss[1];
     }
     __syncthreads();
-    float unit[2] = {a.unit_eps, a.unit_eps};
-    for (int w = 0; w < kDecodeThreads / 32; ++w) {
-        unit[0] += s_red[0][w];
-        unit[1] += s_red[1][w];
+    if (a.decay_w != nullptr) {
+        const T *w = static_cast<const T *>(a.decay_w) + int64_t(head) * a.dk * a.decay_ld;
+        const T *bias = static_cast<const T *>(a.dt_bias) + int64_t(head) * a.dk;
+        for (int c0 = 0; c0 < a.dk; c0 += kDecodeThreads / 4) { // four lanes per channel
+            const int c = c0 + (tid >> 2), cc = min(c, a.dk - 1);
+            const float x = decay_product(w + int64_t(cc) * a.decay_ld, s_z, a.rank, wide_decay != 0, tid & 3) + to_f32(bias[cc]);
+            if ((tid & 3) == 0 && c < a.dk) {
+                s_a[c] = expf(delta_decay_log(a_log, x));
+            }
+        }
+    } else {
+        const float g = expf(delta_decay_log(a_log, to_f32(row[a.a_at + head]) + to_f32(static_cast<const T *>(a.dt_bias)[head])));
+        for (int c = tid; c < a.dk; c += kDecodeThreads) {
+            s_a[c] = g;
+        }
     }
-    unit[0] = a.q_scale * rsqrtf(unit[0]);
-    unit[1] = rsqrtf(unit[1]);
-    const float a_log = to_f32(static_cast<const T *>(a.a_log)[head]);
-    for (int c = tid; c < a.dk; c += kDecodeThreads) {
-        s_q[c] *= unit[0];
-        s_k[c] *= unit[1];
-        const float x = a.decay_w != nullptr
-                            ? delta_decay_input<T>(a, s_z, head, c)
-                            : to_f32(row[a.a_at + head]) + to_f32(static_cast<const T *>(a.dt_bias)[head]);
-        s_a[c] = expf(delta_decay_log(a_log, x));
+    {
+        float unit[2] = {a.unit_eps, a.unit_eps};
+#pragma unroll
+        for (int w = 0; w < kDecodeThreads / 32; ++w) {
+            unit[0] += s_red[0][w];
+            unit[1] += s_red[1][w];
+        }
+        unit[0] = a.q_scale * rsqrtf(unit[0]);
+        unit[1] = rsqrtf(unit[1]);
+        for (int c = tid; c < a.dk; c += kDecodeThreads) {
+            s_q[c] *= unit[0];
+            s_k[c] *= unit[1];
+        }
     }
-    const float beta = sigmoid_of(to_f32(row[a.b_at + head]));
     __syncthreads();
 
     // ---- the state, as many columns at a time as the CTA's threads cover ------------------------------------------------
     const int pass = col_groups * VEC;
+    float so = 0.f; // squares of this thread's outputs
     for (int base = 0; base < a.dv; base += pass) {
         const int c0 = base + cg * VEC;
         if (base > 0) {
             load(c0);
         }
-        float acc[VEC] = {};
+        F acc;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            acc.v[e] = 0.f;
+        }
 #pragma unroll
         for (int u = 0; u < NR; ++u) {
             const int r = rg + u * row_groups;
@@ -167,26 +239,30 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(Gate
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) {
                     s[u].v[e] *= g;
-                    acc[e] = fmaf(s[u].v[e], k, acc[e]);
+                    acc.v[e] = fmaf(s[u].v[e], k, acc.v[e]);
                 }
             }
         }
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            s_part[rg * pass + cg * VEC + e] = acc[e];
-        }
-        __syncthreads();
-        float w[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            float got = 0.f;
+        F *mine = reinterpret_cast<F *>(s_part + rg * pass + cg * VEC);
+        *mine = acc;
+        auto column = [&](int c) {
+            float sum = 0.f;
+#pragma unroll 8
             for (int g = 0; g < row_groups; ++g) {
-                got += s_part[g * pass + cg * VEC + e];
+                sum += s_part[g * pass + c];
             }
-            w[e] = c0 + e < a.dv ? beta * (s_v[c0 + e] - got) : 0.f;
-            acc[e] = 0.f;
+            return sum;
+        };
+        __syncthreads();
+        for (int c = tid; c < pass; c += kDecodeThreads) {
+            s_u[c] = base + c < a.dv ? beta * (s_v[base + c] - column(c)) : 0.f;
         }
         __syncthreads();
+        const F w = *reinterpret_cast<const F *>(s_u + cg * VEC);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            acc.v[e] = 0.f;
+        }
 #pragma unroll
         for (int u = 0; u < NR; ++u) {
             const int r = rg + u * row_groups;
@@ -194,48 +270,41 @@ __global__ void __launch_bounds__(kDecodeThreads) gated_delta_decode_kernel(Gate
                 const float k = s_k[r], q = s_q[r];
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) {
-                    s[u].v[e] = fmaf(k, w[e], s[u].v[e]);
-                    acc[e] = fmaf(q, s[u].v[e], acc[e]);
+                    s[u].v[e] = fmaf(k, w.v[e], s[u].v[e]);
+                    acc.v[e] = fmaf(q, s[u].v[e], acc.v[e]);
                 }
                 *reinterpret_cast<F *>(state + int64_t(r) * a.dv + c0) = s[u];
             }
         }
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            s_part[rg * pass + cg * VEC + e] = acc[e];
-        }
+        *mine = acc;
         __syncthreads();
         for (int c = tid; c < pass && base + c < a.dv; c += kDecodeThreads) {
-            float o = 0.f;
-            for (int g = 0; g < row_groups; ++g) {
-                o += s_part[g * pass + c];
-            }
+            const float o = column(c);
             s_o[base + c] = o;
+            so = fmaf(o, o, so);
         }
-        __syncthreads();
+        if (base + pass < a.dv) {
+            __syncthreads(); // the next pass writes the partial sums
+        }
     }
 
     // ---- norm, gate ------------------------------------------------------------------------------------------------------
-    float so = 0.f;
-    for (int c = tid; c < a.dv; c += kDecodeThreads) {
-        so = fmaf(s_o[c], s_o[c], so);
-    }
     so = warp_sum(so);
     if (lane == 0) {
-        s_red[0][warp] = so;
+        s_red[2][warp] = so;
     }
     __syncthreads();
     float tot = 0.f;
+#pragma unroll
     for (int w = 0; w < kDecodeThreads / 32; ++w) {
-        tot += s_red[0][w];
+        tot += s_red[2][w];
     }
     const float inv = rsqrtf(tot / float(a.dv) + a.eps);
     T *out = static_cast<T *>(a.out) + int64_t(row_i) * a.out_stride + int64_t(head) * a.dv;
-    const T *gate = static_cast<const T *>(a.gate) + int64_t(row_i) * a.gate_stride + int64_t(head) * a.dv;
-    const T *norm = static_cast<const T *>(a.norm_w);
     for (int c = tid; c < a.dv; c += kDecodeThreads) {
-        const float y = to_f32(gate[c]);
-        out[c] = from_f32<T>(s_o[c] * inv * to_f32(norm[c]) * (a.gate_silu ? silu(y) : sigmoid_of(y)));
+        const float y = c == tid ? gate_in : to_f32(gate[c]);
+        const float w = c == tid ? norm : to_f32(static_cast<const T *>(a.norm_w)[c]);
+        out[c] = from_f32<T>(s_o[c] * inv * w * (a.gate_silu ? silu(y) : sigmoid_of(y)));
     }
 }
 
@@ -244,7 +313,7 @@ constexpr int kStrip = 16, kPrepWarps = 8;
 // One warp per head of q, k or v (and one for write strengths and decays of all heads) over a strip of kStrip rows; a lane owns
 // VEC channels and keeps their newest inputs in registers from row to row (kTaps; 0: any number of taps, inputs read again).
 template <typename T, int VEC, int kTaps>
-__global__ void __launch_bounds__(kPrepWarps * 32) gated_delta_prepare_kernel(GatedDeltaArgs a, DeltaScratch at) {
+__global__ void __launch_bounds__(kPrepWarps * 32, kTaps > 0 ? 4 : 2) gated_delta_prepare_kernel(GatedDeltaArgs a, DeltaScratch at) {
     const int lane = int(threadIdx.x) & 31, unit = int(blockIdx.y) * kPrepWarps + (int(threadIdx.x) >> 5);
     const int r0 = int(blockIdx.x) * kStrip, r1 = min(r0 + kStrip, a.n_rows);
     const int units = 2 * a.kv_heads + a.heads;
@@ -282,10 +351,10 @@ __global__ void __launch_bounds__(kPrepWarps * 32) gated_delta_prepare_kernel(Ga
     const int ch0 = is_v ? 2 * a.kv_heads * a.dk + (unit - 2 * a.kv_heads) * a.dv : unit * a.dk;
     using P = Pieces<T, VEC>;
     T *conv = reinterpret_cast<T *>(a.scratch);
-    float ss[kStrip];
-#pragma unroll
+    __shared__ float s_squares[kPrepWarps][kStrip][32]; // (a thread's own places: no barrier)
+    float *ss = &s_squares[threadIdx.x >> 5][0][lane];
     for (int u = 0; u < kStrip; ++u) {
-        ss[u] = 0.f;
+        ss[u * 32] = 0.f;
     }
     for (int c = lane * VEC; c < size; c += 32 * VEC) {
         const int ch = ch0 + c;
@@ -320,13 +389,60 @@ __global__ void __launch_bounds__(kPrepWarps * 32) gated_delta_prepare_kernel(Ga
             }
         };
         int seq = seq0, start = a.q_starts[seq], stop = a.q_starts[seq + 1];
-        bool refill = true;
+        auto finish = [&](int row, const float (&acc)[VEC]) {
+            P y;
+            float sum = 0.f;
 #pragma unroll
-        for (int u = 0; u < kStrip; ++u) {
-            const int row = r0 + u;
-            if (row >= r1) {
-                break;
+            for (int e = 0; e < VEC; ++e) {
+                y.v[e] = from_f32<T>(std::is_same_v<T, float> ? silu(acc[e]) : __fdividef(acc[e], 1.f + __expf(fminf(-acc[e], 80.f))));
+                sum = fmaf(to_f32(y.v[e]), to_f32(y.v[e]), sum);
             }
+            *reinterpret_cast<P *>(conv + int64_t(row) * at.conv_stride + ch) = y;
+            if (!is_v) {
+                ss[(row - r0) * 32] += sum;
+            }
+        };
+        if constexpr (kTaps > 0) {
+            if (r0 >= start && r0 + kStrip <= stop) { // the strip lies inside one run: all its inputs are asked for eight rows at a time
+                const float *ring = delta_ring(a, a.seq_ids[seq]);
+                const int pos0 = a.kv_lens[seq] - (stop - start);
+#pragma unroll
+                for (int b = 1; b < kTaps; ++b) {
+                    input(r0, b, start, pos0, ring, held[b]);
+                }
+                constexpr int kBatch = kStrip / 2;
+#pragma unroll 1
+                for (int u0 = 0; u0 < kStrip; u0 += kBatch) {
+                    P raw[kBatch];
+#pragma unroll
+                    for (int u = 0; u < kBatch; ++u) {
+                        raw[u] = *reinterpret_cast<const P *>(proj + int64_t(r0 + u0 + u) * a.row_stride + in_at);
+                    }
+#pragma unroll
+                    for (int u = 0; u < kBatch; ++u) {
+                        float acc[VEC];
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) {
+                            held[0][e] = to_f32(raw[u].v[e]);
+                            acc[e] = held[0][e] * taps[0][e];
+#pragma unroll
+                            for (int b = 1; b < kTaps; ++b) {
+                                acc[e] = fmaf(held[b][e], taps[b][e], acc[e]);
+                            }
+#pragma unroll
+                            for (int b = kTaps - 1; b > 0; --b) {
+                                held[b][e] = held[b - 1][e];
+                            }
+                        }
+                        finish(r0 + u0 + u, acc);
+                    }
+                }
+                continue;
+            }
+        }
+        bool refill = true;
+#pragma unroll 1
+        for (int row = r0; row < r1; ++row) {
             while (row >= stop && seq + 1 < a.n_seqs) {
                 ++seq;
                 start = stop;
@@ -373,21 +489,14 @@ __global__ void __launch_bounds__(kPrepWarps * 32) gated_delta_prepare_kernel(Ga
                     }
                 }
             }
-            P y;
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) {
-                y.v[e] = from_f32<T>(std::is_same_v<T, float> ? silu(acc[e]) : __fdividef(acc[e], 1.f + __expf(-acc[e])));
-                ss[u] = fmaf(to_f32(y.v[e]), to_f32(y.v[e]), ss[u]);
-            }
-            *reinterpret_cast<P *>(conv + int64_t(row) * at.conv_stride + ch) = y;
+            finish(row, acc);
         }
     }
     if (is_v) {
         return;
     }
-#pragma unroll
     for (int u = 0; u < kStrip; ++u) {
-        const float tot = warp_sum(ss[u]);
+        const float tot = warp_sum(ss[u * 32]);
         if (lane == u && r0 + u < r1) {
             a.scratch[at.unit + int64_t(r0 + u) * 2 * a.kv_heads + unit] = rsqrtf(tot + a.unit_eps) * (unit < a.kv_heads ? a.q_scale : 1.f);
         }
@@ -584,8 +693,8 @@ void single_tokens(stream_t stream, llaisysDataType_t dtype, const GatedDeltaArg
         using T = decltype(tag);
         const bool wide = a.dv % 4 == 0 && a.slot_stride % 4 == 0 && reinterpret_cast<uintptr_t>(a.state) % 16 == 0;
         const int groups = wide ? a.dv / 4 : a.dv;
-        int row_groups = 1; // at least dk / 16, so that a thread holds at most 16 rows
-        while (row_groups * 16 < a.dk) {
+        int row_groups = 1; // at least dk / 8, so that a thread holds at most 8 rows
+        while (row_groups * 8 < a.dk) {
             row_groups *= 2;
         }
         int col_groups = 1;
@@ -594,11 +703,14 @@ void single_tokens(stream_t stream, llaisysDataType_t dtype, const GatedDeltaArg
         }
         row_groups = kDecodeThreads / col_groups;
         const int nr = (a.dk + row_groups - 1) / row_groups;
-        const size_t floats = 3 * size_t(a.dk) + 2 * size_t(a.dv) + size_t(a.rank) + size_t(kDecodeThreads) * (wide ? 4 : 1);
+        const int vec = wide ? 4 : 1;
+        auto up4 = [](int n) { return size_t(n + 3) / 4 * 4; };
+        const size_t floats = 3 * up4(a.dk) + 2 * up4(a.dv) + size_t(a.rank + 31) / 32 * 32 + up4(col_groups * vec) + size_t(kDecodeThreads) * vec;
+        const bool wide_decay = a.decay_ld * sizeof(T) % 16 == 0 && reinterpret_cast<uintptr_t>(a.decay_w) % 16 == 0;
         cudaLaunchConfig_t cfg{};
         cfg.gridDim = dim3(unsigned(a.n_seqs) * unsigned(a.heads));
         cfg.blockDim = dim3(kDecodeThreads);
-        cfg.dynamicSmemBytes = floats * sizeof(float); // at most 1536 + 4096 + 2048 + 1024 floats
+        cfg.dynamicSmemBytes = floats * sizeof(float); // at most 1536 + 4096 + 2048 + 2048 + 2048 floats
         cfg.stream = s;
         cudaLaunchAttribute attr{};
         attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -607,11 +719,11 @@ void single_tokens(stream_t stream, llaisysDataType_t dtype, const GatedDeltaArg
         cfg.numAttrs = 1;
         auto pick = [&](auto vec) {
             constexpr int V = decltype(vec)::value;
-            return nr <= 4 ? gated_delta_decode_kernel<T, V, 4>
-                           : (nr <= 8 ? gated_delta_decode_kernel<T, V, 8> : gated_delta_decode_kernel<T, V, 16>);
+            return nr <= 2 ? gated_delta_decode_kernel<T, V, 2>
+                           : (nr <= 4 ? gated_delta_decode_kernel<T, V, 4> : gated_delta_decode_kernel<T, V, 8>);
         };
         auto kernel = wide ? pick(std::integral_constant<int, 4>{}) : pick(std::integral_constant<int, 1>{});
-        LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, GatedDeltaArgs(a), int(col_groups)));
+        LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, GatedDeltaArgs(a), int(col_groups), int(wide_decay)));
     });
 }
 

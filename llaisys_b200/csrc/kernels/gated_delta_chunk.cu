@@ -9,6 +9,10 @@
 // forward substitution while the others multiply by the state. The split of the decays, its limit and the PIECES of a tile that
 // decays more strongly are those of gated_linear_chunk.cu.
 //
+// Three barriers of the whole CTA divide a tile: (1) decays and operands of this tile, each warp for its own channels, and what
+// is left to do for the outputs of the tile before; (2) everything that reads the old state, the triangular system beside it;
+// (3) corrections, new state, outputs.
+//
 // Precision: the recurrence is f32. The tensor cores take 16-bit operands, so every f32 operand enters as the sum of two bf16
 // numbers, a product of two such operands as its three leading terms; what is left out is below 2^-16 of a term. Accumulators,
 // the state and the triangular inverse are f32.
@@ -16,8 +20,8 @@
 // A CTA owns up to 128 value columns of one (sequence, head). The transposed state S^T [dv, dk] lives in its warps'
 // accumulators, 16 value rows x half of the key channels each, and doubles as the A operand of both products with it. The two
 // warps of a row block ("half" 0 and 1) sum over different channels; half 0 turns both sums into the right-hand side V - K~ S^,
-// each half solves for one 16-token block of U, and they pass operand fragments to one another through shared memory in
-// register order. The next tile's inputs arrive by cp.async under the current tile's products.
+// each half solves for one 16-token block of U, and they pass operand fragments and sums to one another through shared memory
+// in register order. The next tile's inputs arrive by cp.async under the current tile's products.
 //
 // Few (sequence, head) pairs leave SMs idle, so long runs are cut into SEGMENTS. What a segment does to the state is affine,
 // S_end = M S_start + C: a first launch runs every segment from zero with its values (C) and from the identity without values
@@ -45,30 +49,34 @@ constexpr float kLog2e = 1.4426950408889634f;
 
 template <int DK, int DV>
 struct DeltaSmem { // byte offsets
-    static constexpr int kRowBlocks = DV / 16;
+    static constexpr int kWarps = DV / 8, kRowBlocks = DV / 16;
+    static constexpr int kSplit = kWarps == 16 ? 4 : 2;         // warps per 16 x 16 block of A, each with a share of the channels
     static constexpr int kOperand = 2 * kTile * DK * 2;         // high and low
-    static constexpr int kQ = 0;                                // convolved q, k [32][DK] bf16
+    static constexpr int kQ = 0;                                // convolved q, k [32][DK] bf16, swizzled
     static constexpr int kK = kQ + kTile * DK * 2;
     static constexpr int kV = kK + kTile * DK * 2;              // v, two buffers [32][DV] bf16, swizzled
-    static constexpr int kB = kV + 2 * kTile * DV * 2;          // running sums of the tile's log2 decays [32][DK] f32
+    static constexpr int kB = kV + 2 * kTile * DV * 2;          // running sums of the tile's log2 decays [channels / 8][32][8] f32
     static constexpr int kQh = kB + kTile * DK * 4;             // q^ [32][DK] bf16, swizzled, high and low
     static constexpr int kKh = kQh + kOperand;                  // k^
     static constexpr int kKt = kKh + kOperand;                  // k~
-    static constexpr int kO = kQh;                              // o [half][32][DV] f32 over the operands once they are used up
-    static constexpr int kOutputs = 2 * kTile * DV * 4;
-    static constexpr int kS = kQh + (3 * kOperand > kOutputs ? 3 * kOperand : kOutputs); // q^ . k^ [32][32] bf16, high and low
+    static constexpr int kO = kKt + kOperand;                   // o [32][DV] f32
+    static constexpr int kS = kO + kTile * DV * 4;              // q^ . k^ [32][32] bf16, high and low
     static constexpr int kT = kS + 2 * kTile * kTile * 2;       // (I + A)^-1 diag(beta), the same
-    static constexpr int kA = kT + 2 * kTile * kTile * 2;       // A, column s at kAStride s, f32
-    static constexpr int kInv = kA + kTile * kAStride * 4;      // inverse of the second diagonal block, by columns [16][16] f32
-    static constexpr int kX = kInv + 16 * 16 * 4;               // half 1's S^^T k~: [row block][8-token group][lane] float4
+    static constexpr int kInv = kT + 2 * kTile * kTile * 2;     // inverse of the second diagonal block, by columns [16][16] f32
+    static constexpr int kX = kInv + 16 * 16 * 4;               // half 1's sums: [row block][8-token group][lane] float4
     static constexpr int kF = kX + kRowBlocks * 4 * 512;        // fragments, per row block: [R block 0 | U block 0 | U block 1][high, low][lane]
-    static constexpr int kG = kF + kRowBlocks * 3 * 2 * 512;    // output gates of the tile [32][DV] bf16
+    static constexpr int kFragments = kRowBlocks * 3 * 2 * 512;
+    static constexpr int kA = kF;                               // before them: shares of A, column s at kAStride s, f32
+    static constexpr int kShare = kTile * kAStride * 4;
+    static_assert(kSplit * kShare <= kFragments, "A fits where the fragments come later");
+    static constexpr int kG = kF + kFragments;                  // output gates of the tile [32][DV] bf16
     static constexpr int kScal = kG + kTile * DV * 2;           // per token, two buffers: q factor, k factor, beta, log decay [4][32] f32
-    static constexpr int kPart = kScal + 2 * 4 * kTile * 4;     // decay sums of the token parts [4][DK] f32
-    static constexpr int kRef = kPart + 4 * DK * 4;             // per channel: the reference m, and the factors of S
-    static constexpr int kIn = kRef + DK * 4;                   // on the way into its frame
+    static constexpr int kNorm = kScal + 2 * 4 * kTile * 4;     // output norm [DV] f32
+    static constexpr int kBias = kNorm + DV * 4;                // decay biases [DK] f32
+    static constexpr int kIn = kBias + DK * 4;                  // per channel: the factors of S on the way into the tile's frame
     static constexpr int kOut = kIn + DK * 4;                   // and out of it
-    static constexpr int kZ = kOut + DK * 4;                    // low-rank decay inputs [32][rank, padded to 16] bf16
+    static constexpr int kZ = kOut + DK * 4;                    // low-rank decay inputs [32][rank, padded to 16] bf16, swizzled; then
+                                                                // decay weights as fragments [16 ranks][8 channels][lane] 8 bytes
 };
 
 // 16-byte chunk `chunk` of row `row` of a matrix with 64-byte rows
@@ -85,10 +93,12 @@ __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], con
     mma_bf16(d, ah, bl0, bl1);
 }
 
-// T = (I + A)^-1 diag(beta) of 32 tokens by one warp. A by columns (s_a, below the diagonal; the rest is not read), two diagonal
+// T = (I + A)^-1 diag(beta) of 32 tokens by one warp. A / beta by columns in kSplit shares `share` floats apart (below the diagonal;
+// the rest means nothing), summed into the first; two diagonal
 // blocks of 16 by forward substitution (lane: one column of one block), then T_10 = -T_11 A_10 T_00. high / low: T as two bf16
 // matrices, swizzled; the block above the diagonal is never read.
-__device__ __forceinline__ void invert(const float *s_a, float *s_inv, const float *s_beta, unsigned char *high, int lane) {
+template <int kSplit>
+__device__ __forceinline__ void invert(float *s_a, int share, float *s_inv, const float *s_beta, unsigned char *high, int lane) {
     const int blk = lane >> 4, c = lane & 15;
     auto put = [&](int t, int col, float v) {
         const uint32_t u = __float_as_uint(v);
@@ -96,6 +106,20 @@ __device__ __forceinline__ void invert(const float *s_a, float *s_inv, const flo
         *reinterpret_cast<uint16_t *>(high + at) = uint16_t(u >> 16);
         *reinterpret_cast<__nv_bfloat16 *>(high + kTile * kTile * 2 + at) = __float2bfloat16_rn(v - __uint_as_float(u & 0xffff0000u));
     };
+#pragma unroll
+    for (int u = 0; u < 6; ++u) { // columns 0 .. 15 have eight groups of four rows, columns 16 .. 31 the last four of them
+        const int at = u * 32 + lane, s = at < 128 ? at >> 3 : 16 + ((at - 128) >> 2), t = (at < 128 ? at & 7 : 4 + (at & 3)) * 4;
+        float *p = s_a + s * kAStride + t;
+        float4 v = *reinterpret_cast<const float4 *>(p);
+        const float4 b = *reinterpret_cast<const float4 *>(s_beta + t);
+#pragma unroll
+        for (int w = 1; w < kSplit; ++w) {
+            const float4 more = *reinterpret_cast<const float4 *>(p + w * share);
+            v.x += more.x, v.y += more.y, v.z += more.z, v.w += more.w;
+        }
+        *reinterpret_cast<float4 *>(p) = make_float4(v.x * b.x, v.y * b.y, v.z * b.z, v.w * b.w);
+    }
+    __syncwarp();
     float x[16];
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
@@ -165,17 +189,21 @@ __device__ __forceinline__ void invert(const float *s_a, float *s_inv, const flo
 
 template <int DK, int DV, bool kStateOnly>
 __global__ void __launch_bounds__(DV * 4)
-    gated_delta_tile_kernel(GatedDeltaArgs a, DeltaScratch at, int segs, int seg_len, int dv_slices) {
+    gated_delta_tile_kernel(GatedDeltaArgs a, DeltaScratch at, int segs, int seg_len, int dv_slices, int weights_in_smem) {
     using M = DeltaSmem<DK, DV>;
     constexpr int kThreads = DV * 4, kWarps = DV / 8, kRowBlocks = DV / 16;
-    constexpr int kHalf = DK / 2, kNt = kHalf / 8; // channels of a warp, in 8-channel groups
+    constexpr int kHalf = DK / 2, kNt = kHalf / 8; // channels of a warp in the products with the state, in 8-channel groups
+    constexpr int kChunks = DK / 8;                // 8-channel groups of the decays and operands: one warp each, or two
+    constexpr int kSplit = M::kSplit, kInvWarp = kWarps - 4; // the warp that inverts takes no share of A
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ int s_limit;
     const uint32_t sm = smem_u32(smem);
-    float *s_b = reinterpret_cast<float *>(smem + M::kB), *s_part = reinterpret_cast<float *>(smem + M::kPart);
-    auto b_at = [](int t, int d) { return t * DK + (d ^ (((t >> 1) & 3) << 3)); };
-    float *s_ref = reinterpret_cast<float *>(smem + M::kRef), *s_in = reinterpret_cast<float *>(smem + M::kIn);
-    float *s_out = reinterpret_cast<float *>(smem + M::kOut), *s_a = reinterpret_cast<float *>(smem + M::kA);
+    float *s_b = reinterpret_cast<float *>(smem + M::kB);
+    auto b_at = [](int t, int d) { return (d >> 3) * (kTile * 8) + t * 8 + ((d & 7) ^ (((t >> 2) & 1) << 2)); };
+    float *s_in = reinterpret_cast<float *>(smem + M::kIn), *s_out = reinterpret_cast<float *>(smem + M::kOut);
+    float *s_a = reinterpret_cast<float *>(smem + M::kA), *s_o = reinterpret_cast<float *>(smem + M::kO);
+    float *s_norm = reinterpret_cast<float *>(smem + M::kNorm), *s_bias = reinterpret_cast<float *>(smem + M::kBias);
+    auto o_at = [](int t, int c) { return t * DV + (c ^ (((t >> 1) & 3) << 3)); };
 
     const int tid = int(threadIdx.x), warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, q4 = lane & 3, lr = lane & 7, lm = lane >> 3;
@@ -223,26 +251,36 @@ __global__ void __launch_bounds__(DV * 4)
     const int kvh = head / (a.heads / a.kv_heads), nq = a.kv_heads * a.dk;
     const bool per_channel = a.decay_w != nullptr;
     const int rank_steps = per_channel ? (a.rank + 15) / 16 : 0;
-    // what a warp needs of the decay projection: its 16 channels' biases and weights (the first 16 ranks stay in registers)
-    constexpr int kParts = kWarps / (DK / 16), kPartTiles = 4 / kParts; // token parts of a tile, 8-token groups per part
-    static_assert(kParts >= 1 && kPartTiles >= 1, "decays: a warp has 16 channels of at least 8 tokens");
-    const int ch0 = (warp % (DK / 16)) * 16, part = warp / (DK / 16);
-    auto decay_weights = [&](int ks, uint32_t (&wa)[4]) {
+    // decay weights of 8 channels x 16 ranks as a B fragment: channel 8 c + g, ranks 16 ks + 2 q4 (+ 8), two at a time
+    auto decay_weights = [&](int ks, int c, uint32_t (&wb)[2]) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { // rows ch0 + g (+ 8), ranks 16 ks + 2 q4 (+ 8), two at a time
-            const int d = ch0 + g + 8 * (e & 1), r = ks * 16 + 2 * q4 + 8 * (e >> 1);
+        for (int e = 0; e < 2; ++e) {
+            const int d = c * 8 + g, r = ks * 16 + 2 * q4 + 8 * e;
             const uint16_t *w = reinterpret_cast<const uint16_t *>(a.decay_w) + (int64_t(head) * a.dk + d) * a.decay_ld + r;
-            wa[e] = d < a.dk && r < a.rank ? uint32_t(w[0]) | (r + 1 < a.rank ? uint32_t(w[1]) << 16 : 0u) : 0u;
+            wb[e] = d < a.dk && r < a.rank ? uint32_t(w[0]) | (r + 1 < a.rank ? uint32_t(w[1]) << 16 : 0u) : 0u;
         }
     };
-    uint32_t first_w[4] = {};
-    float bias[2] = {};
+    unsigned char *s_w = smem + M::kZ + kTile * rank_steps * 32 + lane * 8;
+    // place of 16-byte piece `chunk` of a token's decay inputs: eight rows in a row fall on different banks
+    auto z_at = [&](int t, int chunk) {
+        const int key = (rank_steps & 3) == 0 ? t & 7 : ((rank_steps & 1) == 0 ? (t >> 1) & 3 : (t >> 2) & 1);
+        return uint32_t(M::kZ + t * rank_steps * 32 + ((chunk ^ key) << 4));
+    };
     if (per_channel) {
-        decay_weights(0, first_w);
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            const int d = ch0 + g + 8 * h;
-            bias[h] = d < a.dk ? to_f32(static_cast<const __nv_bfloat16 *>(a.dt_bias)[int64_t(head) * a.dk + d]) : 0.f;
+        if (weights_in_smem) {
+            for (int u = warp; u < rank_steps * kChunks; u += kWarps) {
+                uint32_t wb[2];
+                decay_weights(u / kChunks, u % kChunks, wb);
+                *reinterpret_cast<uint2 *>(s_w + u * 256) = make_uint2(wb[0], wb[1]);
+            }
+        }
+        for (int d = tid; d < DK; d += kThreads) {
+            s_bias[d] = d < a.dk ? to_f32(static_cast<const __nv_bfloat16 *>(a.dt_bias)[int64_t(head) * a.dk + d]) : 0.f;
+        }
+    }
+    if (!kStateOnly && dv_slices == 1) {
+        for (int c = tid; c < DV; c += kThreads) {
+            s_norm[c] = c < n_cols ? to_f32(static_cast<const __nv_bfloat16 *>(a.norm_w)[c]) : 0.f;
         }
     }
     const float to_log2 = per_channel ? expf(to_f32(static_cast<const __nv_bfloat16 *>(a.a_log)[head])) * kLog2e : kLog2e;
@@ -252,17 +290,18 @@ __global__ void __launch_bounds__(DV * 4)
             const int t = u / kPieces, c = u - t * kPieces;
             const int bytes = t0 + t < end && c * 8 < a.dk ? 16 : 0;
             const __nv_bfloat16 *src = bytes ? conv + int64_t(t0 + t) * at.conv_stride + int64_t(kvh) * a.dk + c * 8 : conv;
+            const uint32_t to = swz(t, c, DK * 2);
             if (!kStateOnly) {
-                cp_async_16(sm + M::kQ + u * 16, src, bytes);
+                cp_async_16(sm + M::kQ + to, src, bytes);
             }
-            cp_async_16(sm + M::kK + u * 16, bytes ? src + nq : conv, bytes);
+            cp_async_16(sm + M::kK + to, bytes ? src + nq : conv, bytes);
         }
         if (per_channel) {
             const int z_pieces = rank_steps * 2;
             for (int u = tid; u < kTile * z_pieces; u += kThreads) {
                 const int t = u / z_pieces, c = u - t * z_pieces;
                 const int bytes = t0 + t < end ? max(0, min(16, (a.rank - c * 8) * 2)) : 0;
-                cp_async_16(sm + M::kZ + u * 16, bytes ? z_rows + int64_t(t0 + t) * a.row_stride + c * 8 : z_rows, bytes);
+                cp_async_16(sm + z_at(t, c), bytes ? z_rows + int64_t(t0 + t) * a.row_stride + c * 8 : z_rows, bytes);
             }
         }
         if (!identity) {
@@ -296,12 +335,6 @@ __global__ void __launch_bounds__(DV * 4)
             cp_async_commit();
         }
     };
-    constexpr int kPer = DV / 32; // value columns per lane when outputs leave
-    float norm_w[kPer];
-#pragma unroll
-    for (int e = 0; e < kPer; ++e) {
-        norm_w[e] = !kStateOnly && dv_slices == 1 && lane * kPer + e < n_cols ? to_f32(static_cast<const __nv_bfloat16 *>(a.norm_w)[lane * kPer + e]) : 0.f;
-    }
     if (identity) { // no values: both buffers stay zero
         for (int u = tid; u < 2 * kTile * DV / 8; u += kThreads) {
             *reinterpret_cast<uint4 *>(smem + M::kV + u * 16) = make_uint4(0, 0, 0, 0);
@@ -329,6 +362,174 @@ __global__ void __launch_bounds__(DV * 4)
         split2(c1[2], c1[3], hi[3], lo[3]);
     };
 
+    // running sums of the tile's log2 decays for 8 channels, by one warp: W z on the tensor cores (bf16 products in f32 are exact)
+    // or the tokens' own, then a scan along the tokens
+    auto decays = [&](int c, const float *s_scal) {
+        if (per_channel) {
+            float v[4][2]; // tokens 8 j + g, channels 8 c + 2 q4 (+ 1)
+            {
+                float acc[2][4] = {};
+                for (int ks = 0; ks < rank_steps; ++ks) {
+                    uint32_t wb[2];
+                    if (weights_in_smem) {
+                        const uint2 w = *reinterpret_cast<const uint2 *>(s_w + (ks * kChunks + c) * 256);
+                        wb[0] = w.x, wb[1] = w.y;
+                    } else {
+                        decay_weights(ks, c, wb);
+                    }
+#pragma unroll
+                    for (int mt = 0; mt < 2; ++mt) {
+                        uint32_t za[4];
+                        ldmatrix_x4(za, sm + z_at(mt * 16 + lr + 8 * (lm & 1), 2 * ks + (lm >> 1)));
+                        mma_bf16(acc[mt], za, wb[0], wb[1]);
+                    }
+                }
+                const float2 bias = *reinterpret_cast<const float2 *>(s_bias + c * 8 + 2 * q4);
+                const bool real = c * 8 < a.dk; // (channels the model does not have keep factor 1; dk is a multiple of 8)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const float x = acc[j >> 1][2 * (j & 1) + e] + (e == 0 ? bias.x : bias.y);
+                        v[j][e] = real ? fmaxf(log_sigmoid_fast(-x) * to_log2, -kMaxTokenDecay) : 0.f;
+                    }
+                }
+            }
+#pragma unroll
+            for (int off = 1; off < 8; off *= 2) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const float up = __shfl_up_sync(0xffffffffu, v[j][e], off * 4);
+                        v[j][e] += g >= off ? up : 0.f;
+                    }
+                }
+            }
+            float base[2] = {0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                float2 sum;
+                sum.x = v[j][0] + base[0];
+                sum.y = v[j][1] + base[1];
+                *reinterpret_cast<float2 *>(s_b + b_at(8 * j + g, c * 8 + 2 * q4)) = sum;
+                if (j < 3) {
+                    base[0] += __shfl_sync(0xffffffffu, v[j][0], 28 + q4);
+                    base[1] += __shfl_sync(0xffffffffu, v[j][1], 28 + q4);
+                }
+            }
+        } else {
+            float v = fmaxf(s_scal[3 * kTile + lane] * to_log2, -kMaxTokenDecay);
+#pragma unroll
+            for (int off = 1; off < 32; off *= 2) {
+                const float up = __shfl_up_sync(0xffffffffu, v, off);
+                v += lane >= off ? up : 0.f;
+            }
+            const float4 all = make_float4(v, v, v, v);
+            *reinterpret_cast<float4 *>(s_b + b_at(lane, c * 8)) = all;
+            *reinterpret_cast<float4 *>(s_b + b_at(lane, c * 8 + 4)) = all;
+        }
+        __syncwarp();
+    };
+    // q^, k^ and k~ of 8 channels and tokens [p0, p1) (zero elsewhere), by one warp, and the factors of S; -> whether the piece's
+    // decays are within the limit
+    auto operands = [&](int c, int p0, int p1, const float *s_scal) {
+        const int t = lane, mid = (p0 + p1 - 1) / 2;
+        uint4 qh = make_uint4(0, 0, 0, 0), ql = qh, kh = qh, kl = qh, th = qh, tl = qh;
+        const uint32_t to = swz(t, c, DK * 2);
+        if (t >= p0 && t < p1) {
+            const uint4 kw = *reinterpret_cast<const uint4 *>(smem + M::kK + to);
+            uint4 qw = make_uint4(0, 0, 0, 0);
+            if (!kStateOnly) {
+                qw = *reinterpret_cast<const uint4 *>(smem + M::kQ + to);
+            }
+            const float fq = s_scal[t], fk = s_scal[kTile + t];
+            const float4 b0 = *reinterpret_cast<const float4 *>(s_b + b_at(t, c * 8)), b1 = *reinterpret_cast<const float4 *>(s_b + b_at(t, c * 8 + 4));
+            const float4 r0 = *reinterpret_cast<const float4 *>(s_b + b_at(mid, c * 8)), r1 = *reinterpret_cast<const float4 *>(s_b + b_at(mid, c * 8 + 4));
+            auto pair = [&](uint32_t qp, uint32_t kp, float e0, float e1, uint32_t &qhi, uint32_t &qlo, uint32_t &khi, uint32_t &klo, uint32_t &thi,
+                            uint32_t &tlo) {
+                const float f0 = ex2(e0), f1 = ex2(e1), k0 = lo_half(kp) * fk, k1 = hi_half(kp) * fk;
+                if (!kStateOnly) {
+                    split2(lo_half(qp) * fq * f0, hi_half(qp) * fq * f1, qhi, qlo);
+                }
+                split2(k0 * f0, k1 * f1, thi, tlo);
+                split2(k0 * ex2(-e0), k1 * ex2(-e1), khi, klo);
+            };
+            pair(qw.x, kw.x, b0.x - r0.x, b0.y - r0.y, qh.x, ql.x, kh.x, kl.x, th.x, tl.x);
+            pair(qw.y, kw.y, b0.z - r0.z, b0.w - r0.w, qh.y, ql.y, kh.y, kl.y, th.y, tl.y);
+            pair(qw.z, kw.z, b1.x - r1.x, b1.y - r1.y, qh.z, ql.z, kh.z, kl.z, th.z, tl.z);
+            pair(qw.w, kw.w, b1.z - r1.z, b1.w - r1.w, qh.w, ql.w, kh.w, kl.w, th.w, tl.w);
+        }
+        if (!kStateOnly) {
+            *reinterpret_cast<uint4 *>(smem + M::kQh + to) = qh;
+            *reinterpret_cast<uint4 *>(smem + M::kQh + kTile * DK * 2 + to) = ql;
+        }
+        *reinterpret_cast<uint4 *>(smem + M::kKh + to) = kh;
+        *reinterpret_cast<uint4 *>(smem + M::kKh + kTile * DK * 2 + to) = kl;
+        *reinterpret_cast<uint4 *>(smem + M::kKt + to) = th;
+        *reinterpret_cast<uint4 *>(smem + M::kKt + kTile * DK * 2 + to) = tl;
+        bool ok = true;
+        if (lane < 8) {
+            const int d = c * 8 + lane;
+            const float base = p0 > 0 ? s_b[b_at(p0 - 1, d)] : 0.f, ref = s_b[b_at(mid, d)], last_sum = s_b[b_at(p1 - 1, d)];
+            s_in[d] = ex2(ref - base);
+            s_out[d] = ex2(last_sum - ref);
+            ok = last_sum - base >= -kMaxDecay;
+        }
+        return ok;
+    };
+    // norm, gate and store of a finished tile's o [token][value column]
+    auto outputs = [&](int t0, int n) {
+        constexpr int kRows = kTile / kWarps, kPer = DV / 32; // a warp's tokens side by side: their sums and exponentials overlap
+        using F = Pieces<float, kPer>; // (the swizzle moves whole groups of eight columns)
+        using P = Pieces<__nv_bfloat16, kPer>;
+        const int c = lane * kPer;
+        F v[kRows];
+        float ss[kRows];
+#pragma unroll
+        for (int u = 0; u < kRows; ++u) {
+            v[u] = *reinterpret_cast<const F *>(s_o + o_at(warp + u * kWarps, c));
+            ss[u] = 0.f;
+#pragma unroll
+            for (int e = 0; e < kPer; ++e) {
+                ss[u] = fmaf(v[u].v[e], v[u].v[e], ss[u]); // (columns past n_cols are zero)
+            }
+        }
+        if (dv_slices > 1) { // the norm runs over more columns than this CTA has: a kernel of its own finishes
+#pragma unroll
+            for (int u = 0; u < kRows; ++u) {
+                const int t = warp + u * kWarps;
+                if (t < n && c < n_cols) {
+                    *reinterpret_cast<F *>(a.scratch + at.raw + (int64_t(t0 + t) * a.heads + head) * a.dv + col0 + c) = v[u];
+                }
+            }
+            return;
+        }
+#pragma unroll
+        for (int o2 = 16; o2 > 0; o2 >>= 1) {
+#pragma unroll
+            for (int u = 0; u < kRows; ++u) {
+                ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o2);
+            }
+        }
+        const F norm = *reinterpret_cast<const F *>(s_norm + c);
+#pragma unroll
+        for (int u = 0; u < kRows; ++u) {
+            const int t = warp + u * kWarps;
+            const float inv = rsqrtf(ss[u] / float(a.dv) + a.eps);
+            const P gate = *reinterpret_cast<const P *>(smem + M::kG + (t * DV + c) * 2);
+            P y;
+#pragma unroll
+            for (int e = 0; e < kPer; ++e) {
+                const float z = to_f32(gate.v[e]);
+                y.v[e] = __float2bfloat16_rn(v[u].v[e] * inv * norm.v[e] * __fdividef(a.gate_silu ? z : 1.f, 1.f + ex2(fminf(z * -kLog2e, 120.f))));
+            }
+            if (t < n && c < n_cols) { // (n_cols is a multiple of 8)
+                *reinterpret_cast<P *>(static_cast<__nv_bfloat16 *>(a.out) + int64_t(t0 + t) * a.out_stride + int64_t(head) * a.dv + c) = y;
+            }
+        }
+    };
+
     int buf = 0;
     for (int t0 = begin; t0 < end; t0 += kTile, buf ^= 1) {
         const int n = min(kTile, end - t0);
@@ -341,174 +542,90 @@ __global__ void __launch_bounds__(DV * 4)
         }
         cp_async_wait<0>();
         __syncthreads();
-        // ---- running sums of the log2 decays: W z on the tensor cores (16 channels x 8 tokens at a time, bf16 products in f32
-        //      are exact) or the tokens' own, then a scan along the tokens. A warp does 16 channels of one part of the tile. ---
-        {
-            float acc[kPartTiles][4] = {};
-            for (int ks = 0; ks < rank_steps; ++ks) {
-                uint32_t wa[4];
-                if (ks == 0) {
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        wa[e] = first_w[e];
+        bool ok = true;
+        for (int c = warp; c < kChunks; c += kWarps) {
+            decays(c, s_scal);
+            ok = operands(c, 0, n, s_scal) && ok;
+        }
+        if (!kStateOnly && t0 > begin) {
+            outputs(t0 - kTile, kTile);
+        }
+        const bool whole = __syncthreads_and(ok);
+        for (int p0 = 0; p0 < n;) {
+            int p1 = n;
+            if (!whole) { // how many tokens from p0 on go together, and their operands
+                if (tid == 0) {
+                    s_limit = n;
+                }
+                __syncthreads();
+                if (tid < DK) {
+                    const float base = p0 > 0 ? s_b[b_at(p0 - 1, tid)] : 0.f;
+                    int t = p0 + 1; // at least one token
+                    while (t < n && s_b[b_at(t, tid)] - base >= -kMaxDecay) {
+                        ++t;
                     }
-                } else {
-                    decay_weights(ks, wa);
+                    atomicMin(&s_limit, t);
                 }
-#pragma unroll
-                for (int nt = 0; nt < kPartTiles; ++nt) {
-                    const int t = (part * kPartTiles + nt) * 8 + g;
-                    const uint32_t *z = reinterpret_cast<const uint32_t *>(smem + M::kZ + (t * rank_steps + ks) * 32);
-                    mma_bf16(acc[nt], wa, z[q4], z[q4 + 4]);
+                __syncthreads();
+                p1 = s_limit;
+                for (int c = warp; c < kChunks; c += kWarps) {
+                    operands(c, p0, p1, s_scal);
                 }
-            }
-            float carry[2] = {0.f, 0.f};
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int d = ch0 + g + 8 * h;
-#pragma unroll
-                for (int nt = 0; nt < kPartTiles; ++nt) {
-                    const int t = (part * kPartTiles + nt) * 8 + 2 * q4;
-                    float l0 = per_channel ? log_sigmoid_fast(-(acc[nt][2 * h] + bias[h])) : s_scal[3 * kTile + t];
-                    float l1 = per_channel ? log_sigmoid_fast(-(acc[nt][2 * h + 1] + bias[h])) : s_scal[3 * kTile + t + 1];
-                    l0 = fmaxf(l0 * to_log2, -kMaxTokenDecay);
-                    l1 = fmaxf(l1 * to_log2, -kMaxTokenDecay);
-                    float incl = l0 + l1;
-                    const float up1 = __shfl_up_sync(0xffffffffu, incl, 1, 4);
-                    incl += q4 >= 1 ? up1 : 0.f;
-                    const float up2 = __shfl_up_sync(0xffffffffu, incl, 2, 4);
-                    incl += q4 >= 2 ? up2 : 0.f;
-                    const float before = __shfl_up_sync(0xffffffffu, incl, 1, 4);
-                    acc[nt][2 * h] = carry[h] + (q4 >= 1 ? before : 0.f) + l0;
-                    acc[nt][2 * h + 1] = acc[nt][2 * h] + l1;
-                    carry[h] += __shfl_sync(0xffffffffu, incl, 3, 4);
-                }
-                if (kParts > 1 && q4 == 0) {
-                    s_part[part * DK + d] = carry[h];
-                }
-            }
-            if (kParts > 1) {
                 __syncthreads();
             }
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int d = ch0 + g + 8 * h;
-                float base = 0.f;
-                for (int u = 0; u < part; ++u) {
-                    base += s_part[u * DK + d];
-                }
-#pragma unroll
-                for (int nt = 0; nt < kPartTiles; ++nt) {
-                    const int t = (part * kPartTiles + nt) * 8 + 2 * q4;
-                    // (channels the model does not have keep factor 1)
-                    s_b[b_at(t, d)] = d < a.dk ? acc[nt][2 * h] + base : 0.f;
-                    s_b[b_at(t + 1, d)] = d < a.dk ? acc[nt][2 * h + 1] + base : 0.f;
-                }
-            }
-            __syncthreads();
-        }
-        for (int p0 = 0; p0 < n;) {
-            // ---- how many tokens from p0 on go together; the piece's reference and the factors of S -----------------------
-            int p1 = n;
-            {
-                const float base = tid < DK && p0 > 0 ? s_b[b_at(p0 - 1, tid)] : 0.f;
-                auto set = [&](int stop) {
-                    const float ref = s_b[b_at((p0 + stop - 1) / 2, tid)], last_sum = s_b[b_at(stop - 1, tid)];
-                    s_ref[tid] = ref;
-                    s_in[tid] = ex2(ref - base);
-                    s_out[tid] = ex2(last_sum - ref);
-                    return last_sum - base;
-                };
-                float total = 0.f;
-                if (tid < DK) {
-                    total = set(n);
-                }
-                if (!__syncthreads_and(total >= -kMaxDecay)) {
-                    if (tid == 0) {
-                        s_limit = n;
-                    }
-                    __syncthreads();
-                    if (tid < DK && total < -kMaxDecay) {
-                        int t = p0 + 1; // at least one token
-                        while (t < n && s_b[b_at(t, tid)] - base >= -kMaxDecay) {
-                            ++t;
-                        }
-                        atomicMin(&s_limit, t);
-                    }
-                    __syncthreads();
-                    p1 = s_limit;
-                    if (tid < DK) {
-                        set(p1);
-                    }
-                    __syncthreads();
-                }
-            }
-            // ---- q^, k^ and k~, zero outside the piece ---------------------------------------------------------------
-            for (int u = tid; u < kTile * (DK / 8); u += kThreads) {
-                const int t = u / (DK / 8), c = u - t * (DK / 8);
-                uint4 qh = make_uint4(0, 0, 0, 0), ql = qh, kh = qh, kl = qh, th = qh, tl = qh;
-                if (t >= p0 && t < p1) {
-                    const uint4 kw = *reinterpret_cast<const uint4 *>(smem + M::kK + u * 16);
-                    uint4 qw = make_uint4(0, 0, 0, 0);
-                    if (!kStateOnly) {
-                        qw = *reinterpret_cast<const uint4 *>(smem + M::kQ + u * 16);
-                    }
-                    const float fq = s_scal[t], fk = s_scal[kTile + t];
-                    const float4 b0 = *reinterpret_cast<const float4 *>(s_b + b_at(t, c * 8));
-                    const float4 b1 = *reinterpret_cast<const float4 *>(s_b + b_at(t, c * 8) + 4);
-                    const float4 r0 = *reinterpret_cast<const float4 *>(s_ref + c * 8);
-                    const float4 r1 = *reinterpret_cast<const float4 *>(s_ref + c * 8 + 4);
-                    auto pair = [&](uint32_t qp, uint32_t kp, float e0, float e1, uint32_t &qhi, uint32_t &qlo, uint32_t &khi, uint32_t &klo,
-                                    uint32_t &thi, uint32_t &tlo) {
-                        const float f0 = ex2(e0), f1 = ex2(e1), k0 = lo_half(kp) * fk, k1 = hi_half(kp) * fk;
-                        if (!kStateOnly) {
-                            split2(lo_half(qp) * fq * f0, hi_half(qp) * fq * f1, qhi, qlo);
-                        }
-                        split2(k0 * f0, k1 * f1, thi, tlo);
-                        split2(k0 * ex2(-e0), k1 * ex2(-e1), khi, klo);
-                    };
-                    pair(qw.x, kw.x, b0.x - r0.x, b0.y - r0.y, qh.x, ql.x, kh.x, kl.x, th.x, tl.x);
-                    pair(qw.y, kw.y, b0.z - r0.z, b0.w - r0.w, qh.y, ql.y, kh.y, kl.y, th.y, tl.y);
-                    pair(qw.z, kw.z, b1.x - r1.x, b1.y - r1.y, qh.z, ql.z, kh.z, kl.z, th.z, tl.z);
-                    pair(qw.w, kw.w, b1.z - r1.z, b1.w - r1.w, qh.w, ql.w, kh.w, kl.w, th.w, tl.w);
-                }
-                const uint32_t to = swz(t, c, DK * 2);
-                if (!kStateOnly) {
-                    *reinterpret_cast<uint4 *>(smem + M::kQh + to) = qh;
-                    *reinterpret_cast<uint4 *>(smem + M::kQh + kTile * DK * 2 + to) = ql;
-                }
-                *reinterpret_cast<uint4 *>(smem + M::kKh + to) = kh;
-                *reinterpret_cast<uint4 *>(smem + M::kKh + kTile * DK * 2 + to) = kl;
-                *reinterpret_cast<uint4 *>(smem + M::kKt + to) = th;
-                *reinterpret_cast<uint4 *>(smem + M::kKt + kTile * DK * 2 + to) = tl;
-            }
-            __syncthreads();
             if (p1 == n) {
                 load_gates(t0);
             }
             if (p1 == n && t0 + kTile < end) {
                 load_tile(t0 + kTile, buf ^ 1); // q, k and z are used up; v and the scalars go to the other buffer
             }
-            // ---- the 16 x 16 blocks on and below the diagonal of k~ . k^ (warps 0 to 2) and q^ . k^ (warps 3 to 5) -----------
-            if (warp < (kStateOnly ? 3 : 6)) {
-                const bool is_q = warp >= 3;
-                const int w = is_q ? warp - 3 : warp, tb = w > 0, sb = w > 1;
-                float c[6][4] = {}; // three products x two 8-key halves, summed below: six independent chains
+            // ---- the 16 x 16 blocks on and below the diagonal of k~ . k^ (a share of the channels per warp) and q^ . k^ -----------
+            constexpr int kBlockTasks = 3 * kSplit;
+            const int share_of = warp < kInvWarp ? warp : (warp == kInvWarp ? kBlockTasks : warp - 1);
+            const int q_block = kWarps == 16 ? warp - 13 : (warp + 1) % 8;
+            // one 16-channel step of a block: three products x two 8-key halves, six independent chains
+            auto block_step = [&](int operand, int tb, int sb, int ks, float (&c)[6][4]) {
+                const uint32_t qa = sm + operand + swz(tb * 16 + lr + 8 * (lm & 1), 2 * ks + (lm >> 1), DK * 2);
+                const uint32_t ka = sm + M::kKh + swz(sb * 16 + (lm >> 1) * 8 + lr, 2 * ks + (lm & 1), DK * 2);
+                uint32_t ah[4], al[4], bh[4], bl[4];
+                ldmatrix_x4(ah, qa);
+                ldmatrix_x4(bh, ka);
+                ldmatrix_x4(al, qa + kTile * DK * 2);
+                ldmatrix_x4(bl, ka + kTile * DK * 2);
+                mma_bf16(c[0], ah, bh[0], bh[1]);
+                mma_bf16(c[1], ah, bh[2], bh[3]);
+                mma_bf16(c[2], al, bh[0], bh[1]);
+                mma_bf16(c[3], al, bh[2], bh[3]);
+                mma_bf16(c[4], ah, bl[0], bl[1]);
+                mma_bf16(c[5], ah, bl[2], bl[3]);
+            };
+            if (share_of < kBlockTasks) {
+                const int w = share_of / kSplit, part = share_of % kSplit, tb = w > 0, sb = w > 1;
+                constexpr int kSteps = DK / 16 / kSplit;
+                float c[6][4] = {};
+#pragma unroll
+                for (int k1 = 0; k1 < kSteps; ++k1) {
+                    block_step(M::kKt, tb, sb, part * kSteps + k1, c);
+                }
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int t = tb * 16 + g + 8 * (e >> 1), sc = sb * 16 + h * 8 + 2 * q4 + (e & 1);
+                        s_a[part * (M::kShare / 4) + sc * kAStride + t] = c[h][e] + (c[2 + h][e] + c[4 + h][e]);
+                    }
+                }
+                named_barrier_arrive(1, (kBlockTasks + 1) * 32);
+            } else if (warp == kInvWarp) {
+                named_barrier_sync(1, (kBlockTasks + 1) * 32); // A is complete
+                invert<kSplit>(s_a, M::kShare / 4, reinterpret_cast<float *>(smem + M::kInv), s_scal + 2 * kTile, smem + M::kT, lane);
+            }
+            if (!kStateOnly && q_block >= 0 && q_block < 3) {
+                const int tb = q_block > 0, sb = q_block > 1;
+                float c[6][4] = {};
 #pragma unroll
                 for (int ks = 0; ks < DK / 16; ++ks) {
-                    const uint32_t qa = sm + (is_q ? M::kQh : M::kKt) + swz(tb * 16 + lr + 8 * (lm & 1), 2 * ks + (lm >> 1), DK * 2);
-                    const uint32_t ka = sm + M::kKh + swz(sb * 16 + (lm >> 1) * 8 + lr, 2 * ks + (lm & 1), DK * 2);
-                    uint32_t ah[4], al[4], bh[4], bl[4];
-                    ldmatrix_x4(ah, qa);
-                    ldmatrix_x4(bh, ka);
-                    ldmatrix_x4(al, qa + kTile * DK * 2);
-                    ldmatrix_x4(bl, ka + kTile * DK * 2);
-                    mma_bf16(c[0], ah, bh[0], bh[1]);
-                    mma_bf16(c[1], ah, bh[2], bh[3]);
-                    mma_bf16(c[2], al, bh[0], bh[1]);
-                    mma_bf16(c[3], al, bh[2], bh[3]);
-                    mma_bf16(c[4], ah, bl[0], bl[1]);
-                    mma_bf16(c[5], ah, bl[2], bl[3]);
+                    block_step(M::kQh, tb, sb, ks, c);
                 }
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
@@ -517,23 +634,11 @@ __global__ void __launch_bounds__(DV * 4)
                         const int t = tb * 16 + g + 4 * e, sc = sb * 16 + h * 8 + 2 * q4;
                         const float x0 = c[h][e] + (c[2 + h][e] + c[4 + h][e]);
                         const float x1 = c[h][e + 1] + (c[2 + h][e + 1] + c[4 + h][e + 1]);
-                        if (is_q) {
-                            uint32_t hi, lo;
-                            split2(sc <= t ? x0 : 0.f, sc + 1 <= t ? x1 : 0.f, hi, lo);
-                            const uint32_t to = M::kS + swz64(t, sb * 2 + h) + q4 * 4;
-                            *reinterpret_cast<uint32_t *>(smem + to) = hi;
-                            *reinterpret_cast<uint32_t *>(smem + to + kTile * kTile * 2) = lo;
-                        } else {
-                            const float beta = s_scal[2 * kTile + t];
-                            s_a[sc * kAStride + t] = beta * x0; // (on and above the diagonal: not read)
-                            s_a[(sc + 1) * kAStride + t] = beta * x1;
-                        }
-                    }
-                }
-                if (!is_q) {
-                    named_barrier_sync(1, 96); // A is complete
-                    if (warp == 0) {
-                        invert(s_a, reinterpret_cast<float *>(smem + M::kInv), s_scal + 2 * kTile, smem + M::kT, lane);
+                        uint32_t hi, lo;
+                        split2(sc <= t ? x0 : 0.f, sc + 1 <= t ? x1 : 0.f, hi, lo);
+                        const uint32_t to = M::kS + swz64(t, sb * 2 + h) + q4 * 4;
+                        *reinterpret_cast<uint32_t *>(smem + to) = hi;
+                        *reinterpret_cast<uint32_t *>(smem + to + kTile * kTile * 2) = lo;
                     }
                 }
             }
@@ -703,71 +808,33 @@ __global__ void __launch_bounds__(DV * 4)
             p0 = p1;
         }
         if constexpr (!kStateOnly) {
-            // ---- o [token][value column] through shared memory: norm, gate, store ------------------------------------------
-            __syncthreads(); // the operands are used up
-            float *s_o = reinterpret_cast<float *>(smem + M::kO);
-            auto o_at = [](int t, int c) { return t * DV + (c ^ (((t >> 1) & 3) << 3)); };
+            // ---- o of both halves, [token][value column]; norm, gate and store follow behind the next barrier -----------------------
+            float4 *s_x = reinterpret_cast<float4 *>(smem + M::kX) + rb * 4 * 32 + lane;
+            if (half == 1) {
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s_o[half * (kTile * DV) + o_at(nt * 8 + 2 * q4 + (e & 1), rb * 16 + g + 8 * (e >> 1))] = o[nt][e];
+                for (int nt = 0; nt < 4; ++nt) {
+                    s_x[nt * 32] = make_float4(o[nt][0], o[nt][1], o[nt][2], o[nt][3]);
                 }
             }
-            cp_async_wait<0>(); // the gates
-            __syncthreads();
-            // a warp's tokens side by side: their sums and exponentials overlap
-            constexpr int kRows = kTile / kWarps;
-            using F = Pieces<float, kPer>; // (the swizzle moves whole groups of eight columns)
-            using P = Pieces<__nv_bfloat16, kPer>;
-            const int c = lane * kPer;
-            F v[kRows];
-            float ss[kRows];
+            named_barrier_sync(2 + rb, 64);
+            if (half == 0) {
 #pragma unroll
-            for (int u = 0; u < kRows; ++u) {
-                const int t = warp + u * kWarps;
-                v[u] = *reinterpret_cast<const F *>(s_o + o_at(t, c));
-                const F other = *reinterpret_cast<const F *>(s_o + kTile * DV + o_at(t, c));
-                ss[u] = 0.f;
-#pragma unroll
-                for (int e = 0; e < kPer; ++e) {
-                    v[u].v[e] += other.v[e];
-                    ss[u] = fmaf(v[u].v[e], v[u].v[e], ss[u]); // (columns past n_cols are zero)
-                }
-            }
-            if (dv_slices > 1) { // the norm runs over more columns than this CTA has: a kernel of its own finishes
-#pragma unroll
-                for (int u = 0; u < kRows; ++u) {
-                    const int t = warp + u * kWarps;
-                    if (t < n && c < n_cols) {
-                        *reinterpret_cast<F *>(a.scratch + at.raw + (int64_t(t0 + t) * a.heads + head) * a.dv + col0 + c) = v[u];
-                    }
-                }
-            } else {
-#pragma unroll
-                for (int o2 = 16; o2 > 0; o2 >>= 1) {
-#pragma unroll
-                    for (int u = 0; u < kRows; ++u) {
-                        ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o2);
-                    }
-                }
-#pragma unroll
-                for (int u = 0; u < kRows; ++u) {
-                    const int t = warp + u * kWarps;
-                    const float inv = rsqrtf(ss[u] / float(a.dv) + a.eps);
-                    const P gate = *reinterpret_cast<const P *>(smem + M::kG + (t * DV + c) * 2);
-                    P y;
-#pragma unroll
-                    for (int e = 0; e < kPer; ++e) {
-                        const float z = to_f32(gate.v[e]);
-                        y.v[e] = __float2bfloat16_rn(v[u].v[e] * inv * norm_w[e] * __fdividef(a.gate_silu ? z : 1.f, 1.f + ex2(fminf(z * -kLog2e, 120.f))));
-                    }
-                    if (t < n && c < n_cols) { // (n_cols is a multiple of 8)
-                        *reinterpret_cast<P *>(static_cast<__nv_bfloat16 *>(a.out) + int64_t(t0 + t) * a.out_stride + int64_t(head) * a.dv + c) = y;
-                    }
+                for (int nt = 0; nt < 4; ++nt) {
+                    const float4 other = s_x[nt * 32];
+                    const int t = nt * 8 + 2 * q4, c = rb * 16 + g;
+                    s_o[o_at(t, c)] = o[nt][0] + other.x;
+                    s_o[o_at(t + 1, c)] = o[nt][1] + other.y;
+                    s_o[o_at(t, c + 8)] = o[nt][2] + other.z;
+                    s_o[o_at(t + 1, c + 8)] = o[nt][3] + other.w;
                 }
             }
         }
+    }
+    if constexpr (!kStateOnly) {
+        cp_async_wait<0>(); // the last tile's gates
+        __syncthreads();
+        const int t0 = begin + (end - 1 - begin) / kTile * kTile;
+        outputs(t0, end - t0);
     }
 
     float *to = kStateOnly ? slot : (last ? state : nullptr);
@@ -790,62 +857,98 @@ __global__ void __launch_bounds__(DV * 4)
 }
 
 // Slots of a sequence hold what each segment does to the state, C [dk, dv] and M by columns; afterwards their first part holds
-// each segment's starting state. A CTA follows kScanCols value columns through all segments, state rows across threads.
-constexpr int kScanThreads = 256, kScanPer = 4; // columns per thread
+// each segment's starting state. A CTA follows kScanCols value columns through all segments, state rows across threads; the
+// segments' M arrive one ahead, through two buffers in shared memory.
+constexpr int kScanThreads = 256, kScanPer = 8; // columns per thread
 
 template <int DK>
 __global__ void __launch_bounds__(kScanThreads) gated_delta_scan_kernel(GatedDeltaArgs a, int segs, int seg_len) {
     constexpr int kGroups = kScanThreads / DK, kCols = kGroups * kScanPer;
-    __shared__ __align__(16) float s_s[DK][kCols];
+    using F = Pieces<float, kScanPer>; // (dv is a multiple of 8: a thread's columns are all there, or none)
+    extern __shared__ __align__(16) float s_m[]; // [2][dk][dk]
+    __shared__ __align__(32) float s_s[DK][kCols];
     const int head = int(blockIdx.x) % a.heads, i = int(blockIdx.x) / a.heads;
     const int len = a.q_starts[i + 1] - a.q_starts[i];
     if (len < 2) {
         return;
     }
     const int n = (len + seg_len - 1) / seg_len;
-    const int64_t size = int64_t(a.dk) * a.dv, stride = size + int64_t(a.dk) * a.dk;
-    float *slot = a.segments + (int64_t(i) * a.heads + head) * segs * stride;
+    const int64_t size = int64_t(a.dk) * a.dv, square = int64_t(a.dk) * a.dk, stride = size + square;
+    float *slots = a.segments + (int64_t(i) * a.heads + head) * segs * stride;
     const float *state = a.state + int64_t(a.seq_ids[i]) * a.slot_stride + int64_t(head) * size;
     const bool fresh = a.kv_lens[i] == len;
     const int d = int(threadIdx.x) % DK, c0 = int(threadIdx.x) / DK * kScanPer, col = int(blockIdx.y) * kCols + c0;
-    auto valid = [&](int e) { return d < a.dk && col + e < a.dv; };
-    float s[kScanPer];
-#pragma unroll
-    for (int e = 0; e < kScanPer; ++e) {
-        s[e] = !fresh && valid(e) ? state[int64_t(d) * a.dv + col + e] : 0.f;
-    }
-    for (int j = 0; j < n; ++j, slot += stride) {
-        float next[kScanPer];
-#pragma unroll
-        for (int e = 0; e < kScanPer; ++e) {
-            next[e] = valid(e) && j + 1 < n ? slot[int64_t(d) * a.dv + col + e] : 0.f;
-            if (valid(e)) {
-                slot[int64_t(d) * a.dv + col + e] = s[e];
+    const bool mine = d < a.dk && col < a.dv;
+    auto fetch = [&](int j) { // (dk is a multiple of 8: 16-byte pieces)
+        if (j + 1 < n) {
+            const float *m = slots + j * stride + size;
+            const uint32_t to = smem_u32(s_m + (j & 1) * square);
+            for (int u = int(threadIdx.x); u < int(square / 4); u += kScanThreads) {
+                cp_async_16(to + u * 16, m + u * 4, 16);
             }
-            s_s[d][c0 + e] = s[e];
         }
+        cp_async_commit();
+    };
+    auto load = [&](const float *p, bool there) {
+        F f;
+#pragma unroll
+        for (int e = 0; e < kScanPer; e += 4) {
+            const float4 x = there ? *reinterpret_cast<const float4 *>(p + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+            f.v[e] = x.x, f.v[e + 1] = x.y, f.v[e + 2] = x.z, f.v[e + 3] = x.w;
+        }
+        return f;
+    };
+    auto store = [&](float *p, const F &f) {
+#pragma unroll
+        for (int e = 0; e < kScanPer; e += 4) {
+            *reinterpret_cast<float4 *>(p + e) = make_float4(f.v[e], f.v[e + 1], f.v[e + 2], f.v[e + 3]);
+        }
+    };
+    const int64_t at = int64_t(d) * a.dv + col;
+    F s = load(state + at, mine && !fresh), next = load(slots + at, mine && n > 1);
+    fetch(0);
+    for (int j = 0; j < n; ++j) {
+        fetch(j + 1);
+        const F after = load(slots + (j + 1) * stride + at, mine && j + 2 < n); // C of the next segment
+        if (mine) {
+            store(slots + j * stride + at, s);
+        }
+        store(&s_s[d][c0], s);
         if (j + 1 == n) {
             break; // (nothing starts from what the last segment leaves)
         }
+        cp_async_wait<1>();
         __syncthreads();
-        const float *m = slot + size + d;
+        const float *m = s_m + (j & 1) * square + d;
         if (d < a.dk) {
 #pragma unroll 8
             for (int u = 0; u < a.dk; ++u) {
-                const float f = m[int64_t(u) * a.dk];
-                const float4 x = *reinterpret_cast<const float4 *>(&s_s[u][c0]);
-                next[0] = fmaf(f, x.x, next[0]);
-                next[1] = fmaf(f, x.y, next[1]);
-                next[2] = fmaf(f, x.z, next[2]);
-                next[3] = fmaf(f, x.w, next[3]);
+                const float f = m[u * a.dk];
+                const F x = *reinterpret_cast<const F *>(&s_s[u][c0]);
+#pragma unroll
+                for (int e = 0; e < kScanPer; ++e) {
+                    next.v[e] = fmaf(f, x.v[e], next.v[e]);
+                }
             }
         }
         __syncthreads();
-#pragma unroll
-        for (int e = 0; e < kScanPer; ++e) {
-            s[e] = next[e];
-        }
+        s = next;
+        next = after;
     }
+    cp_async_wait<0>();
+}
+
+template <int DK>
+void launch_scan(cudaStream_t s, const GatedDeltaArgs &a, int segs, int seg_len) {
+    static std::once_flag once[64];
+    int dev = 0;
+    LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
+    std::call_once(once[dev & 63], [] {
+        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(gated_delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * DK * DK * 4));
+    });
+    constexpr int kCols = kScanThreads / DK * kScanPer;
+    const dim3 grid(unsigned(a.n_seqs) * unsigned(a.heads), unsigned((a.dv + kCols - 1) / kCols));
+    gated_delta_scan_kernel<DK><<<grid, kScanThreads, 2 * size_t(a.dk) * a.dk * sizeof(float), s>>>(a, segs, seg_len);
 }
 
 template <int DK, int DV, bool kStateOnly>
@@ -854,15 +957,18 @@ void launch_tiles(cudaStream_t s, const GatedDeltaArgs &a, const DeltaScratch &a
     int dev = 0;
     LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
     constexpr int kFixed = DeltaSmem<DK, DV>::kZ;
-    constexpr int kMaxBytes = kFixed + kTile * kMaxRank * 2;
-    static_assert(kMaxBytes <= 227 * 1024, "shared memory of one CTA");
-    const int bytes = kFixed + (a.decay_w != nullptr ? kTile * ((a.rank + 15) / 16 * 16) * 2 : 0);
+    constexpr int kMaxBytes = 227 * 1024 - 1024; // (the static shared memory beside it)
+    static_assert(kFixed + kTile * kMaxRank * 2 <= kMaxBytes, "shared memory of one CTA");
+    const int rank = a.decay_w != nullptr ? (a.rank + 15) / 16 * 16 : 0;
+    const int without = kFixed + kTile * rank * 2, with = without + DK * rank * 2;
+    const bool weights_in_smem = rank > 0 && with <= kMaxBytes && (kFixed > 113 * 1024 || with <= 113 * 1024); // (or one CTA less per SM)
+    const int bytes = weights_in_smem ? with : without;
     std::call_once(once[dev & 63], [] {
         LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(gated_delta_tile_kernel<DK, DV, kStateOnly>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxBytes));
     });
     const int extra = kStateOnly ? (a.dk + DV - 1) / DV : 0;
     const dim3 grid(unsigned(a.n_seqs) * unsigned(a.heads) * unsigned(segs), unsigned(slices + extra));
-    gated_delta_tile_kernel<DK, DV, kStateOnly><<<grid, DV * 4, bytes, s>>>(a, at, segs, seg_len, slices);
+    gated_delta_tile_kernel<DK, DV, kStateOnly><<<grid, DV * 4, bytes, s>>>(a, at, segs, seg_len, slices, weights_in_smem ? 1 : 0);
 }
 
 } // namespace
@@ -904,13 +1010,7 @@ void gated_delta_tiles(stream_t stream, const GatedDeltaArgs &a) {
     };
     if (segs > 1) {
         run(std::true_type{});
-        const int cols = kScanThreads / (a.dk <= 64 ? 64 : 128) * kScanPer;
-        const dim3 grid(unsigned(pairs), unsigned((a.dv + cols - 1) / cols));
-        if (a.dk <= 64) {
-            gated_delta_scan_kernel<64><<<grid, kScanThreads, 0, s>>>(a, int(segs), seg_len);
-        } else {
-            gated_delta_scan_kernel<128><<<grid, kScanThreads, 0, s>>>(a, int(segs), seg_len);
-        }
+        a.dk <= 64 ? launch_scan<64>(s, a, int(segs), seg_len) : launch_scan<128>(s, a, int(segs), seg_len);
     }
     run(std::false_type{});
     check_launch("gated_delta_tiles");
