@@ -394,7 +394,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32, kTaps > 0 ? 4 : 2) gated_delt
             float sum = 0.f;
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
-                y.v[e] = from_f32<T>(std::is_same_v<T, float> ? silu(acc[e]) : __fdividef(acc[e], 1.f + __expf(fminf(-acc[e], 80.f))));
+                y.v[e] = from_f32<T>(std::is_same_v<T, float> ? silu(acc[e]) : __fdividef(acc[e], 1.f + __expf(-acc[e])));
                 sum = fmaf(to_f32(y.v[e]), to_f32(y.v[e]), sum);
             }
             *reinterpret_cast<P *>(conv + int64_t(row) * at.conv_stride + ch) = y;

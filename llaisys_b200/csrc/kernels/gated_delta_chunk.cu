@@ -86,6 +86,14 @@ __device__ __forceinline__ void cp_async_4(uint32_t dst, const void *src, int sr
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;\n" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
 }
 
+// log2(1 + e^x) = max(x, 0) log2 e + log2(1 + 2^(-|x| log2 e)). Its error, a few 2^-24 of absolute size, is that of rounding the
+// decay itself to f32.
+__device__ __forceinline__ float softplus_log2(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(1.f + ex2(fabsf(x) * -kLog2e)));
+    return fmaf(fmaxf(x, 0.f), kLog2e, y);
+}
+
 __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0,
                                      uint32_t bl1) {
     mma_bf16(d, ah, bh0, bh1);
@@ -230,7 +238,7 @@ __global__ void __launch_bounds__(DV * 4)
     }
     const bool fresh = a.kv_lens[i] == row1 - row0;
     float *state = a.state + int64_t(a.seq_ids[i]) * a.slot_stride + int64_t(head) * a.dk * a.dv;
-    float *slot = a.segments != nullptr ? a.segments + ((int64_t(i) * a.heads + head) * segs + seg) * (int64_t(a.dk) * a.dv + int64_t(a.dk) * a.dk)
+    float *slot = a.segments != nullptr ? a.segments + ((int64_t(i) * a.heads + head) * segs + seg) * (int64_t(a.dk) * a.dv + DK * DK)
                                         : nullptr;
 
     // ---- the state: s[nt] = S^T rows 16 rb + g (+ 8), channels d0 + 8 nt + 2 q4 (+ 1) -------------------------------------
@@ -283,10 +291,11 @@ __global__ void __launch_bounds__(DV * 4)
             s_norm[c] = c < n_cols ? to_f32(static_cast<const __nv_bfloat16 *>(a.norm_w)[c]) : 0.f;
         }
     }
-    const float to_log2 = per_channel ? expf(to_f32(static_cast<const __nv_bfloat16 *>(a.a_log)[head])) * kLog2e : kLog2e;
-    auto load_tile = [&](int t0, int buf) {
+    const float minus_a = per_channel ? -expf(to_f32(static_cast<const __nv_bfloat16 *>(a.a_log)[head])) : 0.f;
+    // inputs of a tile, by threads first, first + 1, .. of `threads`
+    auto load_tile = [&](int t0, int buf, int first, int threads) {
         constexpr int kPieces = DK / 8, kVPieces = DV / 8;
-        for (int u = tid; u < kTile * kPieces; u += kThreads) {
+        for (int u = first; u < kTile * kPieces; u += threads) {
             const int t = u / kPieces, c = u - t * kPieces;
             const int bytes = t0 + t < end && c * 8 < a.dk ? 16 : 0;
             const __nv_bfloat16 *src = bytes ? conv + int64_t(t0 + t) * at.conv_stride + int64_t(kvh) * a.dk + c * 8 : conv;
@@ -298,36 +307,36 @@ __global__ void __launch_bounds__(DV * 4)
         }
         if (per_channel) {
             const int z_pieces = rank_steps * 2;
-            for (int u = tid; u < kTile * z_pieces; u += kThreads) {
+            for (int u = first; u < kTile * z_pieces; u += threads) {
                 const int t = u / z_pieces, c = u - t * z_pieces;
                 const int bytes = t0 + t < end ? max(0, min(16, (a.rank - c * 8) * 2)) : 0;
                 cp_async_16(sm + z_at(t, c), bytes ? z_rows + int64_t(t0 + t) * a.row_stride + c * 8 : z_rows, bytes);
             }
         }
         if (!identity) {
-            for (int u = tid; u < kTile * kVPieces; u += kThreads) {
+            for (int u = first; u < kTile * kVPieces; u += threads) {
                 const int t = u / kVPieces, c = u - t * kVPieces;
                 const int bytes = t0 + t < end && c * 8 < n_cols ? 16 : 0;
                 cp_async_16(sm + M::kV + buf * (kTile * DV * 2) + swz(t, c, DV * 2),
                             bytes ? conv + int64_t(t0 + t) * at.conv_stride + 2 * nq + int64_t(head) * a.dv + col0 + c * 8 : conv, bytes);
             }
         }
-        if (tid < 4 * kTile) {
-            const int which = tid / kTile, t = tid - which * kTile;
+        if (first < 4 * kTile) {
+            const int which = first / kTile, t = first - which * kTile;
             const int64_t row = t0 + t;
             const int bytes = t0 + t < end ? 4 : 0;
             const float *src = which < 2 ? a.scratch + at.unit + row * 2 * a.kv_heads + which * a.kv_heads + kvh
                                          : a.scratch + (which == 2 ? at.beta : at.decay_log) + row * a.heads + head;
-            cp_async_4(sm + M::kScal + (buf * 4 * kTile + tid) * 4, bytes ? src : a.scratch, which == 3 && per_channel ? 0 : bytes);
+            cp_async_4(sm + M::kScal + (buf * 4 * kTile + first) * 4, bytes ? src : a.scratch, which == 3 && per_channel ? 0 : bytes);
         }
         cp_async_commit();
     };
     // the gates of the CURRENT tile, needed at its end: asked for together with the next tile's operands
-    auto load_gates = [&](int t0) {
+    auto load_gates = [&](int t0, int first, int threads) {
         if (!kStateOnly && dv_slices == 1) {
             constexpr int kPieces = DV / 8;
             const __nv_bfloat16 *gate = static_cast<const __nv_bfloat16 *>(a.gate);
-            for (int u = tid; u < kTile * kPieces; u += kThreads) {
+            for (int u = first; u < kTile * kPieces; u += threads) {
                 const int t = u / kPieces, c = u - t * kPieces;
                 const int bytes = t0 + t < end && c * 8 < n_cols ? 16 : 0;
                 cp_async_16(sm + M::kG + u * 16, bytes ? gate + int64_t(t0 + t) * a.gate_stride + int64_t(head) * a.dv + c * 8 : gate, bytes);
@@ -340,7 +349,7 @@ __global__ void __launch_bounds__(DV * 4)
             *reinterpret_cast<uint4 *>(smem + M::kV + u * 16) = make_uint4(0, 0, 0, 0);
         }
     }
-    load_tile(begin, 0);
+    load_tile(begin, 0, tid, kThreads);
 
     const int frag = rb * 3 * 2 * 512 + lane * 16; // this lane's place in the row block's fragments
     auto put_frag = [&](int which, const uint32_t (&hi)[4], const uint32_t (&lo)[4]) {
@@ -391,7 +400,7 @@ __global__ void __launch_bounds__(DV * 4)
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
                         const float x = acc[j >> 1][2 * (j & 1) + e] + (e == 0 ? bias.x : bias.y);
-                        v[j][e] = real ? fmaxf(log_sigmoid_fast(-x) * to_log2, -kMaxTokenDecay) : 0.f;
+                        v[j][e] = real ? fmaxf(softplus_log2(x) * minus_a, -kMaxTokenDecay) : 0.f;
                     }
                 }
             }
@@ -419,7 +428,7 @@ __global__ void __launch_bounds__(DV * 4)
                 }
             }
         } else {
-            float v = fmaxf(s_scal[3 * kTile + lane] * to_log2, -kMaxTokenDecay);
+            float v = fmaxf(s_scal[3 * kTile + lane] * kLog2e, -kMaxTokenDecay);
 #pragma unroll
             for (int off = 1; off < 32; off *= 2) {
                 const float up = __shfl_up_sync(0xffffffffu, v, off);
@@ -573,12 +582,6 @@ __global__ void __launch_bounds__(DV * 4)
                 }
                 __syncthreads();
             }
-            if (p1 == n) {
-                load_gates(t0);
-            }
-            if (p1 == n && t0 + kTile < end) {
-                load_tile(t0 + kTile, buf ^ 1); // q, k and z are used up; v and the scalars go to the other buffer
-            }
             // ---- the 16 x 16 blocks on and below the diagonal of k~ . k^ (a share of the channels per warp) and q^ . k^ -----------
             constexpr int kBlockTasks = 3 * kSplit;
             const int share_of = warp < kInvWarp ? warp : (warp == kInvWarp ? kBlockTasks : warp - 1);
@@ -720,6 +723,12 @@ __global__ void __launch_bounds__(DV * 4)
                     }
                     put_frag(0, rh[0], rl[0]);
                 }
+                if (half == 1 && p1 == n) { // half 1 waits for half 0 here: time to ask for what comes next
+                    load_gates(t0, tid - kThreads / 2, kThreads / 2);
+                    if (t0 + kTile < end) {
+                        load_tile(t0 + kTile, buf ^ 1, tid - kThreads / 2, kThreads / 2); // q, k and z are used up; v and the scalars
+                    }                                                                     // go to the other buffer
+                }
                 named_barrier_sync(2 + rb, 64); // the two warps of the row block
                 if (half == 1) {
                     get_frag(0, rh[0], rl[0]);
@@ -837,6 +846,28 @@ __global__ void __launch_bounds__(DV * 4)
         outputs(t0, end - t0);
     }
 
+    if (identity) { // M as A fragments (high, low), behind the segment's C: pairs along its columns, transposed across the warp
+        uint4 *m = reinterpret_cast<uint4 *>(slot + int64_t(a.dk) * a.dv) + lane;
+#pragma unroll
+        for (int u = 0; u < kNt / 2; ++u) {
+            uint32_t hi[4], lo[4];
+            split2(s[2 * u][0], s[2 * u][1], hi[0], lo[0]);
+            split2(s[2 * u + 1][0], s[2 * u + 1][1], hi[1], lo[1]);
+            split2(s[2 * u][2], s[2 * u][3], hi[2], lo[2]);
+            split2(s[2 * u + 1][2], s[2 * u + 1][3], hi[3], lo[3]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                hi[e] = movmatrix_trans(hi[e]);
+                lo[e] = movmatrix_trans(lo[e]);
+            }
+            const int at16 = ((half * (kNt / 2) + u) * (DK / 16) + col0 / 16 + rb) * 2; // 16 rows x 16 columns of M
+            if (col0 + rb * 16 < DK) {
+                m[at16 * 32] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                m[(at16 + 1) * 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+        }
+        return;
+    }
     float *to = kStateOnly ? slot : (last ? state : nullptr);
     if (to != nullptr) {
 #pragma unroll
@@ -845,111 +876,114 @@ __global__ void __launch_bounds__(DV * 4)
             for (int e = 0; e < 4; ++e) {
                 const int d = d0 + nt * 8 + 2 * q4 + (e & 1), c = rb * 16 + g + 8 * (e >> 1);
                 if (d < a.dk && c < n_cols) {
-                    if (identity) { // M by columns, behind the segment's C
-                        to[int64_t(a.dk) * a.dv + int64_t(col0 + c) * a.dk + d] = s[nt][e];
-                    } else {
-                        to[int64_t(d) * a.dv + col0 + c] = s[nt][e];
-                    }
+                    to[int64_t(d) * a.dv + col0 + c] = s[nt][e];
                 }
             }
         }
     }
 }
 
-// Slots of a sequence hold what each segment does to the state, C [dk, dv] and M by columns; afterwards their first part holds
-// each segment's starting state. A CTA follows kScanCols value columns through all segments, state rows across threads; the
-// segments' M arrive one ahead, through two buffers in shared memory.
-constexpr int kScanThreads = 256, kScanPer = 8; // columns per thread
-
+// Slots of a sequence hold what each segment does to the state, C [dk, dv] f32 and M as operand fragments; afterwards their first
+// part holds each segment's starting state. A CTA follows 16 value columns through all segments, a warp per 16 rows of the
+// state: S_{j+1} = M_j S_j + C_j with both factors as two bf16 numbers. A fragment of M is replaced by the next segment's as soon
+// as it has been used.
 template <int DK>
-__global__ void __launch_bounds__(kScanThreads) gated_delta_scan_kernel(GatedDeltaArgs a, int segs, int seg_len) {
-    constexpr int kGroups = kScanThreads / DK, kCols = kGroups * kScanPer;
-    using F = Pieces<float, kScanPer>; // (dv is a multiple of 8: a thread's columns are all there, or none)
-    extern __shared__ __align__(16) float s_m[]; // [2][dk][dk]
-    __shared__ __align__(32) float s_s[DK][kCols];
+__global__ void __launch_bounds__(DK * 2) gated_delta_scan_kernel(GatedDeltaArgs a, int segs, int seg_len) {
+    constexpr int kSteps = DK / 16;
+    __shared__ uint2 s_s[2][kSteps][2][2][32]; // S as B fragments: two buffers, [16 rows][8 columns][high, low][lane]
     const int head = int(blockIdx.x) % a.heads, i = int(blockIdx.x) / a.heads;
     const int len = a.q_starts[i + 1] - a.q_starts[i];
     if (len < 2) {
         return;
     }
     const int n = (len + seg_len - 1) / seg_len;
-    const int64_t size = int64_t(a.dk) * a.dv, square = int64_t(a.dk) * a.dk, stride = size + square;
+    const int64_t size = int64_t(a.dk) * a.dv, stride = size + DK * DK;
     float *slots = a.segments + (int64_t(i) * a.heads + head) * segs * stride;
     const float *state = a.state + int64_t(a.seq_ids[i]) * a.slot_stride + int64_t(head) * size;
     const bool fresh = a.kv_lens[i] == len;
-    const int d = int(threadIdx.x) % DK, c0 = int(threadIdx.x) / DK * kScanPer, col = int(blockIdx.y) * kCols + c0;
-    const bool mine = d < a.dk && col < a.dv;
-    auto fetch = [&](int j) { // (dk is a multiple of 8: 16-byte pieces)
-        if (j + 1 < n) {
-            const float *m = slots + j * stride + size;
-            const uint32_t to = smem_u32(s_m + (j & 1) * square);
-            for (int u = int(threadIdx.x); u < int(square / 4); u += kScanThreads) {
-                cp_async_16(to + u * 16, m + u * 4, 16);
+    const int warp = int(threadIdx.x) >> 5, lane = int(threadIdx.x) & 31, g = lane >> 2, q4 = lane & 3;
+    const int col = int(blockIdx.y) * 16 + 2 * q4;
+    // this lane's rows 16 warp + g (+ 8), columns col (+ 1) of both 8-column groups
+    auto each = [&](auto &&body) {
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int d = warp * 16 + g + 8 * h, c = col + nt * 8;
+                body(nt, h, int64_t(d) * a.dv + c, d < a.dk && c < a.dv);
             }
         }
-        cp_async_commit();
     };
-    auto load = [&](const float *p, bool there) {
-        F f;
+    auto load = [&](const float *p, bool there, float (&x)[2][4]) { // (dv is even: both columns are there, or neither)
+        each([&](int nt, int h, int64_t at, bool in) {
+            const float2 v = in && there ? *reinterpret_cast<const float2 *>(p + at) : make_float2(0.f, 0.f);
+            x[nt][2 * h] = v.x, x[nt][2 * h + 1] = v.y;
+        });
+    };
+    auto fragments = [&](int j, int ks) { return reinterpret_cast<const uint4 *>(slots + j * stride + size) + ((warp * kSteps + ks) * 2) * 32 + lane; };
+    float s[2][4], next[2][4];
+    load(state, !fresh, s);
+    load(slots, n > 1, next);
+    uint4 mh[kSteps], ml[kSteps];
 #pragma unroll
-        for (int e = 0; e < kScanPer; e += 4) {
-            const float4 x = there ? *reinterpret_cast<const float4 *>(p + e) : make_float4(0.f, 0.f, 0.f, 0.f);
-            f.v[e] = x.x, f.v[e + 1] = x.y, f.v[e + 2] = x.z, f.v[e + 3] = x.w;
-        }
-        return f;
-    };
-    auto store = [&](float *p, const F &f) {
-#pragma unroll
-        for (int e = 0; e < kScanPer; e += 4) {
-            *reinterpret_cast<float4 *>(p + e) = make_float4(f.v[e], f.v[e + 1], f.v[e + 2], f.v[e + 3]);
-        }
-    };
-    const int64_t at = int64_t(d) * a.dv + col;
-    F s = load(state + at, mine && !fresh), next = load(slots + at, mine && n > 1);
-    fetch(0);
+    for (int ks = 0; ks < kSteps; ++ks) {
+        mh[ks] = n > 1 ? fragments(0, ks)[0] : make_uint4(0, 0, 0, 0);
+        ml[ks] = n > 1 ? fragments(0, ks)[32] : make_uint4(0, 0, 0, 0);
+    }
     for (int j = 0; j < n; ++j) {
-        fetch(j + 1);
-        const F after = load(slots + (j + 1) * stride + at, mine && j + 2 < n); // C of the next segment
-        if (mine) {
-            store(slots + j * stride + at, s);
-        }
-        store(&s_s[d][c0], s);
+        each([&](int nt, int h, int64_t at, bool in) {
+            if (in) {
+                *reinterpret_cast<float2 *>(slots + j * stride + at) = make_float2(s[nt][2 * h], s[nt][2 * h + 1]);
+            }
+        });
         if (j + 1 == n) {
             break; // (nothing starts from what the last segment leaves)
         }
-        cp_async_wait<1>();
-        __syncthreads();
-        const float *m = s_m + (j & 1) * square + d;
-        if (d < a.dk) {
-#pragma unroll 8
-            for (int u = 0; u < a.dk; ++u) {
-                const float f = m[u * a.dk];
-                const F x = *reinterpret_cast<const F *>(&s_s[u][c0]);
 #pragma unroll
-                for (int e = 0; e < kScanPer; ++e) {
-                    next.v[e] = fmaf(f, x.v[e], next.v[e]);
-                }
+        for (int nt = 0; nt < 2; ++nt) { // rows of S become the summed dimension: transpose the pairs across the warp
+            uint32_t h0, l0, h1, l1;
+            split2(s[nt][0], s[nt][1], h0, l0);
+            split2(s[nt][2], s[nt][3], h1, l1);
+            s_s[j & 1][warp][nt][0][lane] = make_uint2(movmatrix_trans(h0), movmatrix_trans(h1));
+            s_s[j & 1][warp][nt][1][lane] = make_uint2(movmatrix_trans(l0), movmatrix_trans(l1));
+        }
+        float after[2][4];
+        load(slots + (j + 1) * stride, j + 2 < n, after); // C of the next segment
+        __syncthreads();
+        float low[2][4] = {}, high[2][4] = {};
+#pragma unroll
+        for (int ks = 0; ks < kSteps; ++ks) {
+            const uint32_t ah[4] = {mh[ks].x, mh[ks].y, mh[ks].z, mh[ks].w}, al[4] = {ml[ks].x, ml[ks].y, ml[ks].z, ml[ks].w};
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt) {
+                const uint2 bh = s_s[j & 1][ks][nt][0][lane], bl = s_s[j & 1][ks][nt][1][lane];
+                mma_bf16(next[nt], ah, bh.x, bh.y);
+                mma_bf16(low[nt], al, bh.x, bh.y);
+                mma_bf16(high[nt], ah, bl.x, bl.y);
+            }
+            if (j + 2 < n) {
+                mh[ks] = fragments(j + 1, ks)[0];
+                ml[ks] = fragments(j + 1, ks)[32];
             }
         }
-        __syncthreads();
-        s = next;
-        next = after;
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                s[nt][e] = next[nt][e] + (low[nt][e] + high[nt][e]);
+                next[nt][e] = after[nt][e];
+            }
+        }
     }
-    cp_async_wait<0>();
 }
 
 template <int DK>
 void launch_scan(cudaStream_t s, const GatedDeltaArgs &a, int segs, int seg_len) {
-    static std::once_flag once[64];
-    int dev = 0;
-    LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
-    std::call_once(once[dev & 63], [] {
-        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(gated_delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * DK * DK * 4));
-    });
-    constexpr int kCols = kScanThreads / DK * kScanPer;
-    const dim3 grid(unsigned(a.n_seqs) * unsigned(a.heads), unsigned((a.dv + kCols - 1) / kCols));
-    gated_delta_scan_kernel<DK><<<grid, kScanThreads, 2 * size_t(a.dk) * a.dk * sizeof(float), s>>>(a, segs, seg_len);
+    const dim3 grid(unsigned(a.n_seqs) * unsigned(a.heads), unsigned((a.dv + 15) / 16));
+    gated_delta_scan_kernel<DK><<<grid, DK * 2, 0, s>>>(a, segs, seg_len);
 }
+
+int64_t slot_floats(int64_t dk, int64_t dv) { return dk * dv + (dk <= 64 ? 64 * 64 : 128 * 128); }
 
 template <int DK, int DV, bool kStateOnly>
 void launch_tiles(cudaStream_t s, const GatedDeltaArgs &a, const DeltaScratch &at, int segs, int seg_len, int slices) {
@@ -977,7 +1011,7 @@ size_t gated_delta_segment_floats(llaisysDataType_t dtype, size_t heads, size_t 
     if (heads == 0 || !gated_delta_tiles_fit(dtype, int64_t(dk), int64_t(dv))) {
         return 0;
     }
-    return size_t(kMaxCtas) * (dk * dv + dk * dk); // pairs x segments of a launch that is cut never exceed kMaxCtas
+    return size_t(kMaxCtas) * size_t(slot_floats(int64_t(dk), int64_t(dv))); // pairs x segments of a launch that is cut never exceed kMaxCtas
 }
 
 void gated_delta_tiles(stream_t stream, const GatedDeltaArgs &a) {
@@ -990,7 +1024,7 @@ void gated_delta_tiles(stream_t stream, const GatedDeltaArgs &a) {
     const int slices = (a.dv + 127) / 128;
     const int64_t pairs = int64_t(a.n_seqs) * a.heads;
     int64_t segs = std::min<int64_t>(kMaxCtas / (pairs * slices), (a.max_q_len + kTile - 1) / kTile);
-    segs = a.segments == nullptr ? 1 : std::min(segs, int64_t(a.segment_floats) / ((int64_t(a.dk) * a.dv + int64_t(a.dk) * a.dk) * pairs));
+    segs = a.segments == nullptr ? 1 : std::min(segs, int64_t(a.segment_floats) / (slot_floats(a.dk, a.dv) * pairs));
     int seg_len = (a.max_q_len + kTile - 1) / kTile * kTile;
     if (segs >= kMinSegments) {
         seg_len = int((a.max_q_len + segs * kTile - 1) / (segs * kTile)) * kTile;

@@ -320,7 +320,8 @@ def test_delta_repeated_keys_written_in_full(cuda_device, dtype, rank):
 
 
 @pytest.mark.parametrize("dtype,heads,kv_heads,dk,dv,rank", [(torch.bfloat16, 1, 1, 128, 128, 16), (torch.bfloat16, 2, 1, 64, 96, 0),
-                                                             (torch.bfloat16, 1, 1, 96, 256, 0), (torch.float32, 1, 1, 64, 64, 8)])
+                                                             (torch.bfloat16, 1, 1, 96, 256, 0), (torch.bfloat16, 3, 3, 40, 24, 5),
+                                                             (torch.float32, 1, 1, 64, 64, 8)])
 def test_delta_long_runs(cuda_device, dtype, heads, kv_heads, dk, dv, rank):
     """Runs long enough to be cut into segments: the same outputs and states as uncut, from a fresh and from a carried state."""
     lens = [1500, 700, 3]
