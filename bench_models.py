@@ -51,7 +51,7 @@ def doderax_config(s: dict) -> dict:
     layers = [{"type": "channel_delta", "mixer": delta(s["gla_heads"]), "mlp": mlp},
               {"type": "parallel", "mixer": {"left": left, "right": delta(s["gla_heads"] // 2)}, "mlp": mlp}]
     return {"architecture": "Doderax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
-            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}, "layers": layers * (s["layers"] // 2)}
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 10007, "mul_cur": 257}}, "layers": layers * (s["layers"] // 2)}
 
 
 def attention_layers(family: str, s: dict) -> int:

@@ -43,7 +43,7 @@ constexpr float kMaxDecay = 80.f;       // log2 units
 constexpr float kMaxTokenDecay = 160.f; // log2: one token's decay is cut here, where it is zero in f32
 constexpr int kMaxRank = 512;
 constexpr int kMaxCtas = 148; // (pairs x segments) of a launch that is cut
-constexpr int kMinSegments = 3; // two passes over the state instead of one: fewer segments do not pay
+constexpr int kMinSegments = 3; // M and C cost a pass each: fewer segments do not pay
 constexpr int kAStride = 36;  // floats per column of A
 constexpr float kLog2e = 1.4426950408889634f;
 
