@@ -1,7 +1,8 @@
 /*
  * llaisys C ABI -- token mixers beyond plain causal attention, on device buffers and an explicit stream: caches whose
  * layers differ in shape, attention with a sliding window (that can keep a sequence's first tokens) and an output factor per
- * head, the norm / rotation + append in front of it, gated linear attention and the gated delta rule with recurrent state.
+ * head, attention without a softmax whose weights are mixed over the heads, the norm / rotation + append in front of them, and
+ * gated linear attention, the gated delta rule and minGRU with recurrent state.
  * NVIDIA devices. No counterpart in the reference.
  * Status codes as in paged_kv.h; as for every ...Dev call there: no host validation of index arrays, no staging copy.
  */
@@ -37,6 +38,12 @@ struct LlaisysNormAppend {
     const int32_t *seq_ids_dev, *positions_dev;
     size_t n_rows, nh, rot_dims;
     const float *rot_table; /* [n_rows, rot_dims / 2, 2] */
+    /* The row form (row_norm != 0; no rotation, no gate): bias, element by element of a row (NULL: none), is added to q, k and v;
+     * q_norm [nh, k_dim] and k_norm [nkvh, k_dim] follow ONE root mean square over the whole of q and of k; q is multiplied by
+     * 1 + temp_coef ln(floor((position + 1) / temp_every) + 1). */
+    int row_norm;
+    const void *bias;
+    float temp_coef, temp_every;
 };
 /* table[row, i] = (cos, sin)(positions[row] * freq[i]), i < half, all on the device */
 LLAISYS_API int llaisysRotaryTableDev(llaisysDeviceType_t device_type, int device_id, float *table, const int32_t *positions_dev,
@@ -53,6 +60,39 @@ LLAISYS_API int llaisysPagedAttentionOptDev(llaisysPagedKV_t kv, size_t layer, v
                                             size_t n_seqs, size_t total_q, size_t max_q_len, size_t max_kv_len, size_t nh,
                                             float scale, size_t window, size_t keep_first, const float *row_scale,
                                             size_t row_stride, llaisysStream_t stream);
+
+/* Attention without a softmax over the pages: head h gives key j <= i (with i - j < window, if window > 0) the weight
+ *     a_hij = sigmoid(s - slopes[h] * (i - j) + bias[h]),   s = softcap * tanh(scale <q, k> / softcap)   (softcap <= 0: scale <q, k>)
+ * and weighs the values of its own kv head with sum_g talk[h, g] a_gij. slopes [nh] f32, bias [nh] and talk [nh, nh] of the cache's
+ * dtype, all on the device; NULL: no distance term, no bias, no mixing. Other arguments as llaisysPagedAttentionOptDev. */
+struct LlaisysGates {
+    float softcap;
+    const float *slopes;
+    const void *bias, *talk;
+};
+LLAISYS_API int llaisysPagedAttentionGatesDev(llaisysPagedKV_t kv, size_t layer, void *out, const void *q, const int32_t *seq_ids_dev,
+                                              const int32_t *q_starts_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t total_q,
+                                              size_t max_q_len, size_t max_kv_len, size_t nh, float scale, size_t window,
+                                              const struct LlaisysGates *gates, size_t row_stride, llaisysStream_t stream);
+
+/* minGRU, element by element over `width` channels: with z_t = sigmoid(z + bias_z) and u_t = x + bias_x,
+ *     S_t = (1 - z_t) S_{t-1} + z_t g(u_t),   g(u) = u + 1/2 for u >= 0, sigmoid(u) below;   out_t = S_t silu(g)
+ * z, x and g are `width` elements each at z_at, x_at and g_at of a projection row; biases [width] of `dtype`; the state [width] f32
+ * of slot s at state + s * slot_stride. Sequences, rows, slots and `decode` as for LlaisysGatedLinear. */
+struct LlaisysMinGru {
+    const void *proj;
+    int64_t row_stride, z_at, x_at, g_at;
+    const void *bias_z, *bias_x;
+    size_t width;
+    float *state;
+    int64_t slot_stride;
+    const int32_t *seq_ids_dev, *q_starts_dev, *kv_lens_dev;
+    size_t n_seqs, n_rows, max_q_len;
+    void *out;
+    int64_t out_stride;
+};
+LLAISYS_API int llaisysMinGruDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype, const struct LlaisysMinGru *args,
+                                 int decode, llaisysStream_t stream);
 
 /* Gated linear attention. Per head, with state S [dk, dv] in f32 (row-major, slot s of the sequence in seq_ids at
  * state + s * slot_stride + head * dk * dv):

@@ -57,6 +57,8 @@ LLAISYS_API const char *llaisysGetLastError(void);
 #define LLAISYS_KERNEL_DECODE_TMA_FUSED 4 /* the same launch also appends the step's new K/V rows                 */
 #define LLAISYS_KERNEL_DECODE_CP_ASYNC 5  /* split-KV flash decoding over plain K/V tensors (legacy operator)     */
 #define LLAISYS_KERNEL_PREFILL_TC 6       /* causal chunk attention on tcgen05 tensor cores                       */
+#define LLAISYS_KERNEL_GATES 7            /* gated attention (mixers.h), any dtype / head_dim: one CTA per query  */
+#define LLAISYS_KERNEL_GATES_TILES 8      /* gated attention on the tensor cores, queries x keys x all heads      */
 /* Kernel of the calling thread's most recent attention call: any cache, or llaisysSelfAttention. */
 LLAISYS_API int llaisysLastAttentionKernel(void);
 

@@ -67,6 +67,10 @@ int llaisysPagedKVNormAppendDev(llaisysPagedKV_t kv, size_t layer, const Llaisys
         n.positions = a->positions_dev;
         n.n_rows = a->n_rows;
         n.nh = int32_t(a->nh);
+        n.row_norm = a->row_norm;
+        n.bias = a->bias;
+        n.temp_coef = a->temp_coef;
+        n.temp_every = a->temp_every;
         kv->impl.normAppendDev(layer, n, stream);
     });
 }
@@ -90,6 +94,76 @@ int llaisysPagedAttentionOptDev(llaisysPagedKV_t kv, size_t layer, void *out, co
             kv->impl.prefillDev(layer, out, q, seq_ids_dev, q_starts_dev, kv_lens_dev, n_seqs, total_q, max_q_len, max_kv_len, nh,
                                 scale, stream, opt);
         }
+    });
+}
+
+int llaisysPagedAttentionGatesDev(llaisysPagedKV_t kv, size_t layer, void *out, const void *q, const int32_t *seq_ids_dev,
+                                  const int32_t *q_starts_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t total_q,
+                                  size_t max_q_len, size_t max_kv_len, size_t nh, float scale, size_t window,
+                                  const LlaisysGates *gates, size_t row_stride, llaisysStream_t stream) {
+    if (kv == nullptr || gates == nullptr) {
+        return bad("gated attention: null argument");
+    }
+    return guarded([&] {
+        llaisys::kernels::GateArgs g;
+        g.softcap = gates->softcap;
+        g.slopes = gates->slopes;
+        g.bias = gates->bias;
+        g.talk = gates->talk;
+        llaisys::kv::AttnOptions opt;
+        opt.window = window;
+        opt.row_stride = row_stride;
+        opt.gates = &g;
+        if (q_starts_dev == nullptr) {
+            kv->impl.decodeDev(layer, out, nullptr, q, seq_ids_dev, kv_lens_dev, n_seqs, max_kv_len, nh, scale, stream, opt);
+        } else {
+            kv->impl.prefillDev(layer, out, q, seq_ids_dev, q_starts_dev, kv_lens_dev, n_seqs, total_q, max_q_len, max_kv_len, nh,
+                                scale, stream, opt);
+        }
+    });
+}
+
+int llaisysMinGruDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype, const LlaisysMinGru *a, int decode,
+                     llaisysStream_t stream) {
+    if (a == nullptr || a->proj == nullptr || a->bias_z == nullptr || a->bias_x == nullptr || a->state == nullptr ||
+        a->seq_ids_dev == nullptr || a->kv_lens_dev == nullptr || a->out == nullptr || (decode == 0 && a->q_starts_dev == nullptr)) {
+        return bad("minGRU: null argument");
+    }
+    if (device_type != LLAISYS_DEVICE_NVIDIA) {
+        llaisys::kernels::set_last_error("minGRU: NVIDIA devices only");
+        return LLAISYS_E_UNSUPPORTED;
+    }
+    return guarded([&] {
+#ifdef ENABLE_NVIDIA_API
+        llaisys::core::context().setDevice(device_type, device_id);
+        llaisys::kernels::MinGruArgs g;
+        g.proj = a->proj;
+        g.row_stride = a->row_stride;
+        g.z_at = a->z_at;
+        g.x_at = a->x_at;
+        g.g_at = a->g_at;
+        g.bias_z = a->bias_z;
+        g.bias_x = a->bias_x;
+        g.width = int32_t(a->width);
+        g.state = a->state;
+        g.slot_stride = a->slot_stride;
+        g.seq_ids = a->seq_ids_dev;
+        g.q_starts = a->q_starts_dev;
+        g.kv_lens = a->kv_lens_dev;
+        g.n_seqs = int32_t(a->n_seqs);
+        g.n_rows = int32_t(a->n_rows);
+        g.max_q_len = int32_t(a->max_q_len);
+        g.out = a->out;
+        g.out_stride = a->out_stride;
+        if (decode != 0) {
+            llaisys::kernels::min_gru_decode(stream, dtype, g);
+        } else {
+            llaisys::kernels::min_gru_chunk(stream, dtype, g);
+        }
+#else
+        (void)dtype, (void)device_id, (void)decode, (void)stream;
+        throw llaisys::kv::StatusError(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
+#endif
     });
 }
 

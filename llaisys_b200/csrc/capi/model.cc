@@ -1,5 +1,6 @@
 // extern "C" thunks of the generic model API and of the families that have no older ABI of their own.
 #include "llaisys/models/doderax.h"
+#include "llaisys/models/lilovik.h"
 #include "llaisys/models/model.h"
 #include "llaisys/models/vozozen.h"
 #include "llaisys/paged_kv.h"
@@ -98,6 +99,9 @@ LlaisysModel *llaisysVozozenModelCreate(const LlaisysVozozenMeta *meta, llaisysD
 }
 LlaisysModel *llaisysDoderaxModelCreate(const LlaisysDoderaxMeta *meta, llaisysDeviceType_t device, int device_id) {
     return create_model<llaisys::models::Doderax>("llaisysDoderaxModelCreate", meta, device, device_id);
+}
+LlaisysModel *llaisysLilovikModelCreate(const LlaisysLilovikMeta *meta, llaisysDeviceType_t device, int device_id) {
+    return create_model<llaisys::models::Lilovik>("llaisysLilovikModelCreate", meta, device, device_id);
 }
 
 int llaisysModelRecordStream(LlaisysModel *model, int enable) {

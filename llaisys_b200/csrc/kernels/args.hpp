@@ -85,6 +85,16 @@ struct AttnOut {
     const struct PeerSink *peers = nullptr; // decode over a page pool only: partial rows go to exchange slots instead
 };
 
+// Attention without a softmax: the weight of a visible key j for head h and the query at position i is
+//   a_hij = sigmoid(score - slopes_h (i - j) + bias_h),  score = softcap tanh(scale <q, k> / softcap), or scale <q, k> without a cap,
+// and head h weighs the values of its kv head with sum_g talk[h, g] a_gij. Nothing is normalised over the keys.
+struct GateArgs {
+    float softcap = 0.f;           // <= 0: none
+    const float *slopes = nullptr; // [nh] on the device; null: no distance term
+    const void *bias = nullptr;    // [nh], cache dtype; null: none
+    const void *talk = nullptr;    // [nh, nh], cache dtype; null: every head keeps its own weights
+};
+
 // Exchange buffers of a KV-range split across the GPUs of a node, as rank `rank` sees them: table[r] (an array in
 // device memory) is rank r's buffer, peer memory for r != rank, and `own` is table[rank]. A buffer holds 2 (step
 // parity) x world slots of slot_floats 8-byte words -- slot s of parity p is written by rank s; a word is a float and,
@@ -127,6 +137,12 @@ struct NormAppendArgs {
     const int32_t *seq_ids = nullptr, *positions = nullptr; // per row, on the device
     size_t n_rows = 0;
     int32_t nh = 0;
+    // The row form (row_norm != 0; no rotation, no gate): `bias` (element e belongs to element e of a row; null: none) is added
+    // to q, k and v; q_norm [nh * d] and k_norm [nkvh * d] go with ONE root mean square over the whole of q and of k; q is then
+    // multiplied by 1 + temp_coef ln(floor((position + 1) / temp_every) + 1)
+    int32_t row_norm = 0;
+    const void *bias = nullptr;
+    float temp_coef = 0.f, temp_every = 1.f;
 };
 
 // Gated linear attention over one packed projection (per head a state S [dk, dv], decayed per key channel):
@@ -194,6 +210,23 @@ struct GatedDeltaArgs {
     float *segments = nullptr; // see gated_delta_segment_floats; null: never cut
     size_t segment_floats = 0;
     LLAISYS_ARGS_FN int32_t channels() const { return 2 * kv_heads * dk + heads * dv; }
+};
+
+// minGRU over one packed projection, element by element: with z = sigmoid(z_at .. + bias_z) and u = x_at .. + bias_x,
+//   S_t = (1 - z_t) S_{t-1} + z_t g(u_t),  g(u) = u + 1/2 for u >= 0, sigmoid(u) for u < 0;   out_t = S_t silu(g_at ..)
+struct MinGruArgs {
+    const void *proj = nullptr; // [n_rows, row_stride], model dtype
+    int64_t row_stride = 0;
+    int64_t z_at = 0, x_at = 0, g_at = 0;
+    const void *bias_z = nullptr, *bias_x = nullptr; // [width]
+    int32_t width = 0;
+    float *state = nullptr; // slot s: state + s * slot_stride, [width]
+    int64_t slot_stride = 0;
+    // the batch, as in GatedLinearArgs
+    const int32_t *seq_ids = nullptr, *q_starts = nullptr, *kv_lens = nullptr;
+    int32_t n_seqs = 0, n_rows = 0, max_q_len = 0;
+    void *out = nullptr; // row r: out + r * out_stride, model dtype
+    int64_t out_stride = 0;
 };
 
 using stream_t = void *;

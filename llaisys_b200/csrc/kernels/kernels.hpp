@@ -47,6 +47,8 @@ bool linear_tc(stream_t stream, llaisysDataType_t dtype, void *out, const void *
 int linear_tc_status(stream_t stream);
 // out[r, i] = up * silu(gate) with gate = gu[r, i], up = gu[r, di + i]: the activation on a packed gate|up projection.
 void swiglu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate_up, size_t rows, size_t di);
+// out[r, i] = up * max(gate, 0), packed alike
+void relu_glu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate_up, size_t rows, size_t di);
 // Row-wise argmax with every row split over several CTAs (a vocabulary-sized row on one CTA leaves the GPU idle).
 // scratch: 12 * rows bytes, zero before the first call; the kernel leaves it zero again.
 void argmax_rows_split(stream_t stream, llaisysDataType_t dtype, int64_t *idx_out, const void *vals, size_t rows, size_t n,
@@ -97,6 +99,10 @@ size_t gated_delta_state_floats(size_t heads, size_t kv_heads, size_t dk, size_t
 size_t gated_delta_scratch_floats(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t kv_heads, size_t dk, size_t dv);
 size_t gated_delta_segment_floats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
 
+// minGRU (see MinGruArgs). decode: one token per sequence. chunk: ragged runs of tokens, one pass over their rows.
+void min_gru_decode(stream_t stream, llaisysDataType_t dtype, const MinGruArgs &args);
+void min_gru_chunk(stream_t stream, llaisysDataType_t dtype, const MinGruArgs &args);
+
 // Gated linear attention (see GatedLinearArgs). decode: one token per sequence, everything in one launch. chunk: ragged
 // runs of tokens.
 void gated_linear_decode(stream_t stream, llaisysDataType_t dtype, const GatedLinearArgs &args);
@@ -112,6 +118,9 @@ void embed_scaled(stream_t stream, llaisysDataType_t dtype, float *x, void *copy
 // prev[r] < 0 (no token before this one); pairs has buckets + 1 rows
 void embed_pairs(stream_t stream, llaisysDataType_t dtype, float *x, const int64_t *tokens, const int64_t *prev, const void *w,
                  const void *pairs, int64_t mul_prev, int64_t mul_cur, int64_t buckets, size_t rows, size_t d, size_t vocab);
+// x[r, :] = w[tokens[r], :] + (sin, cos, sin, cos, ..)(positions[r] * freq[i]) for columns 2 i and 2 i + 1; freq [(d + 1) / 2] f64
+void embed_positions(stream_t stream, llaisysDataType_t dtype, float *x, const int64_t *tokens, const int32_t *positions,
+                     const double *freq, const void *w, size_t rows, size_t d, size_t vocab);
 // out[r, :] = dtype(x[r, :]), row r at out + r * out_stride
 void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const float *x, size_t rows, size_t d);
 // out[i, :] = rms_norm(x[r, :]) * (offset + w) with r = row_index[i] (null: r = i), f32 arithmetic, one rounding. offset 1: a
@@ -126,10 +135,11 @@ void relu_squared(stream_t stream, llaisysDataType_t dtype, void *v, size_t n);
 // out = gelu(in), tanh form, [rows, n] each with its own row stride (elements)
 void gelu_tanh(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const void *in, int64_t in_stride,
                size_t rows, size_t n);
-// x += scale * (rms_norm(a) * wa + rms_norm(b) * wb), a and b f32 [rows, d] like x; h (may be null) = dtype(rms_norm(x) *
-// (offset + w)) of the new x, the norm that comes next
+// x += scale * (rms_norm(a) * (branch_offset + wa) + rms_norm(b) * (branch_offset + wb)), a and b f32 [rows, d] like x (b may be
+// null: one branch); h (may be null) = dtype(rms_norm(x) * (offset + w)) of the new x, the norm that comes next
 void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const float *a, const void *wa, const float *b,
-                       const void *wb, float scale, float eps, void *h, const void *w, float offset, size_t rows, size_t d);
+                       const void *wb, float scale, float eps, void *h, const void *w, float offset, size_t rows, size_t d,
+                       float branch_offset = 0.f);
 // table[r, i] = (cos, sin)(positions[r] * freq[i]), i < half
 void rotary_table(stream_t stream, float *table, const int32_t *positions, const float *freq, size_t rows, size_t half);
 // logits = cap * tanh(logits / cap) in place (cap <= 0: unchanged) and the row-wise argmax of the result, one launch;
@@ -145,6 +155,11 @@ void paged_gather(stream_t stream, size_t elem_size, const KVView &kv, int32_t s
 // operator for shapes they do not cover.
 void attention_generic(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch,
                        const void *q, float scale, const AttnOut &out, int32_t *error_flag);
+
+// Attention without a softmax whose weights are mixed over the heads (see GateArgs). Any dtype and sizes, windows but no kept
+// tokens, neither partial results nor output factors. The kernel behind shapes that attention_gates_tiles does not cover.
+void attention_gates(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch, const void *q, float scale,
+                     const GateArgs &gates, const AttnOut &out, int32_t *error_flag);
 
 // K2 (+ fused K3): split-KV flash decoding for 16-bit K/V, head_dim 128, page size 16, GQA group <= 8,
 // one query per sequence. Returns -1 if the shape is not covered.

@@ -228,8 +228,15 @@ __global__ void bias_add_kernel(T *__restrict__ out, const T *__restrict__ bias,
     }
 }
 
-template <typename T, int VEC>
-__global__ void swiglu_packed_kernel(T *__restrict__ out, const T *__restrict__ gu, size_t rows, size_t di) {
+struct SiluOf {
+    static __device__ __forceinline__ float of(float v) { return v / (1.f + expf(-v)); }
+};
+struct ReluOf {
+    static __device__ __forceinline__ float of(float v) { return fmaxf(v, 0.f); }
+};
+
+template <typename Act, typename T, int VEC>
+__global__ void glu_packed_kernel(T *__restrict__ out, const T *__restrict__ gu, size_t rows, size_t di) {
     grid_dependency_wait(); // (programmatic launch, as rms_norm_vec_kernel)
     grid_launch_dependents();
     struct alignas(sizeof(T) * VEC) P {
@@ -244,8 +251,7 @@ __global__ void swiglu_packed_kernel(T *__restrict__ out, const T *__restrict__ 
         P o;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            const float gv = to_f32(g.v[e]);
-            o.v[e] = from_f32<T>(to_f32(u.v[e]) * (gv / (1.f + expf(-gv))));
+            o.v[e] = from_f32<T>(to_f32(u.v[e]) * Act::of(to_f32(g.v[e])));
         }
         *reinterpret_cast<P *>(out + r * di + c) = o;
     }
@@ -395,7 +401,8 @@ void swiglu(stream_t stream, llaisysDataType_t dtype, void *out, const void *gat
     check_launch("swiglu");
 }
 
-void swiglu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate_up, size_t rows, size_t di) {
+template <typename Act>
+static void glu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate_up, size_t rows, size_t di) {
     if (rows == 0 || di == 0) {
         return;
     }
@@ -405,14 +412,23 @@ void swiglu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const vo
     LLAISYS_CUDA_DISPATCH_FLOAT(dtype, {
         constexpr int kVec = 16 / int(sizeof(T));
         if (ptrs_ok && di % kVec == 0) {
-            launch_programmatic(swiglu_packed_kernel<T, kVec>, unsigned(grid_for(rows * di / kVec, 256)), 256u, s,
+            launch_programmatic(glu_packed_kernel<Act, T, kVec>, unsigned(grid_for(rows * di / kVec, 256)), 256u, s,
                                 static_cast<T *>(out), static_cast<const T *>(gate_up), rows, di);
         } else {
-            launch_programmatic(swiglu_packed_kernel<T, 1>, unsigned(grid_for(rows * di, 256)), 256u, s, static_cast<T *>(out),
+            launch_programmatic(glu_packed_kernel<Act, T, 1>, unsigned(grid_for(rows * di, 256)), 256u, s, static_cast<T *>(out),
                                 static_cast<const T *>(gate_up), rows, di);
         }
     });
+}
+
+void swiglu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate_up, size_t rows, size_t di) {
+    glu_packed<SiluOf>(stream, dtype, out, gate_up, rows, di);
     check_launch("swiglu_packed");
+}
+
+void relu_glu_packed(stream_t stream, llaisysDataType_t dtype, void *out, const void *gate_up, size_t rows, size_t di) {
+    glu_packed<ReluOf>(stream, dtype, out, gate_up, rows, di);
+    check_launch("relu_glu_packed");
 }
 
 void argmax_rows_split(stream_t stream, llaisysDataType_t dtype, int64_t *idx_out, const void *vals, size_t rows, size_t n,

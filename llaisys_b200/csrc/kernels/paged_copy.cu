@@ -500,6 +500,127 @@ __global__ void __launch_bounds__(256)
     }
 }
 
+// The row form of NormAppendArgs: one CTA per row, because q and k are normed over all their heads at once. A row's pieces of
+// VEC elements lie in q, then k, then v; the first PER_THREAD of a thread stay in registers between the sums and the stores.
+template <typename T, int VEC, int PER_THREAD>
+__global__ void paged_row_norm_append_kernel(unsigned char *__restrict__ k_pool, unsigned char *__restrict__ v_pool, NormAppendArgs a,
+                                             const int32_t *__restrict__ table, CopyGeom g, int32_t d, int32_t dv,
+                                             int64_t v_head_stride_b, int64_t v_token_stride_b, int32_t max_blocks, int32_t *error_flag) {
+    using P = Pack<T, VEC>;
+    asm volatile("griddepcontrol.wait;\n" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    const int64_t row = blockIdx.x;
+    const int32_t nq = a.nh * d / VEC, nk = g.nkvh * d / VEC, n = nq + nk + g.nkvh * dv / VEC;
+    const T *proj = static_cast<const T *>(a.proj) + row * a.row_stride, *bias = static_cast<const T *>(a.bias);
+    struct Piece {
+        float v[VEC];
+    };
+    auto load = [&](int32_t i) {
+        const int64_t at = i < nq ? a.q_at + int64_t(i) * VEC : (i < nq + nk ? a.k_at + int64_t(i - nq) * VEC : a.v_at + int64_t(i - nq - nk) * VEC);
+        const P x = *reinterpret_cast<const P *>(proj + at);
+        Piece f;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            f.v[e] = to_f32(x.v[e]);
+        }
+        if (bias != nullptr) {
+            const P b = *reinterpret_cast<const P *>(bias + at);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                f.v[e] += to_f32(b.v[e]);
+            }
+        }
+        return f;
+    };
+    float sq = 0.f, sk = 0.f;
+    auto square = [&](int32_t i, const Piece &f) {
+        float s = 0.f;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            s = fmaf(f.v[e], f.v[e], s);
+        }
+        sq += i < nq ? s : 0.f;
+        sk += i >= nq && i < nq + nk ? s : 0.f;
+    };
+    Piece held[PER_THREAD];
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * int32_t(blockDim.x);
+        if (i < n) {
+            held[r] = load(i);
+            square(i, held[r]);
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * int32_t(blockDim.x); i < nq + nk; i += int32_t(blockDim.x)) {
+        square(i, load(i));
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    __shared__ float part_q[32], part_k[32];
+    if ((threadIdx.x & 31) == 0) {
+        part_q[threadIdx.x >> 5] = sq;
+        part_k[threadIdx.x >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int i = 0; i < int(blockDim.x >> 5); ++i) { // every thread sums the few partials in the same order
+        sq += part_q[i];
+        sk += part_k[i];
+    }
+    const int32_t pos = a.positions[row];
+    float inv_q = a.q_norm != nullptr ? rsqrtf(sq / float(a.nh * d) + a.eps) : 1.f;
+    const float inv_k = a.k_norm != nullptr ? rsqrtf(sk / float(g.nkvh * d) + a.eps) : 1.f;
+    if (a.temp_coef != 0.f) {
+        inv_q *= fmaf(a.temp_coef, logf(floorf(__fdiv_rn(float(pos + 1), a.temp_every)) + 1.f), 1.f);
+    }
+    int32_t page = 0, slot = 0;
+    const bool stores = resolve_slot(table, g, a.seq_ids[row], pos, max_blocks, error_flag, page, slot);
+    auto store = [&](int32_t i, const Piece &f) {
+        const bool is_q = i < nq, is_k = !is_q && i < nq + nk;
+        const int32_t at = (is_q ? i : (is_k ? i - nq : i - nq - nk)) * VEC;
+        const T *w = static_cast<const T *>(is_q ? a.q_norm : (is_k ? a.k_norm : nullptr));
+        const float inv = is_q ? inv_q : (is_k ? inv_k : 1.f);
+        P o;
+        if (w != nullptr) {
+            const P ww = *reinterpret_cast<const P *>(w + at);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                o.v[e] = from_f32<T>(f.v[e] * inv * to_f32(ww.v[e]));
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                o.v[e] = from_f32<T>(f.v[e] * inv);
+            }
+        }
+        if (is_q) {
+            *reinterpret_cast<P *>(static_cast<T *>(a.q_out) + row * a.nh * d + at) = o;
+            return;
+        }
+        if (!stores) {
+            return;
+        }
+        const int32_t len = is_k ? d : dv, head = at / len;
+        const int64_t off = int64_t(page) * g.page_stride_b + (at - head * len) * int64_t(sizeof(T)) +
+                            (is_k ? int64_t(head) * g.head_stride_b + int64_t(slot) * g.token_stride_b
+                                  : int64_t(head) * v_head_stride_b + int64_t(slot) * v_token_stride_b);
+        *reinterpret_cast<P *>((is_k ? k_pool : v_pool) + off) = o;
+    };
+#pragma unroll
+    for (int r = 0; r < PER_THREAD; ++r) {
+        const int32_t i = int32_t(threadIdx.x) + r * int32_t(blockDim.x);
+        if (i < n) {
+            store(i, held[r]);
+        }
+    }
+    for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * int32_t(blockDim.x); i < n; i += int32_t(blockDim.x)) {
+        store(i, load(i));
+    }
+}
+
 template <typename T>
 void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &a, int32_t max_blocks, int32_t *error_flag) {
     CopyGeom g{};
@@ -513,19 +634,36 @@ void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &
     constexpr int kVec = 4;
     auto aligned = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const int32_t d = kv.d, dv = kv.vDim();
-    const bool wide = d % kVec == 0 && dv % kVec == 0 && a.row_stride % kVec == 0 && a.q_at % kVec == 0 && a.k_at % kVec == 0 &&
-                      a.v_at % kVec == 0 && aligned(a.proj) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out) &&
-                      a.rot_dims / 2 % kVec == 0;
-    const int64_t warps = int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh);
     cudaLaunchConfig_t cfg{};
-    cfg.gridDim = dim3(unsigned((warps + 7) / 8));
-    cfg.blockDim = dim3(256);
     cfg.stream = s;
     cudaLaunchAttribute attr{};
     attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = 1;
+    if (a.row_norm != 0) {
+        CHECK_ARGUMENT(a.rot_dims == 0 && a.gate_at < 0 && a.row_scale == nullptr && a.temp_every > 0.f,
+                       "norm append: the row form takes neither a rotation nor a gate");
+        constexpr int kRow = 16 / int(sizeof(T));
+        const bool pieces = d % kRow == 0 && dv % kRow == 0 && a.row_stride % kRow == 0 && a.q_at % kRow == 0 && a.k_at % kRow == 0 &&
+                            a.v_at % kRow == 0 && aligned(a.proj) && aligned(a.bias) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out);
+        const int64_t n = (int64_t(a.nh) * d + int64_t(kv.nkvh) * (d + dv)) / (pieces ? kRow : 1);
+        CHECK_ARGUMENT(n < (int64_t(1) << 30), "norm append: row too long");
+        const int64_t threads = (n + 2) / 3 + 31;
+        cfg.gridDim = dim3(unsigned(a.n_rows));
+        cfg.blockDim = dim3(unsigned(threads < 64 ? 64 : (threads > 512 ? 512 : threads / 32 * 32)));
+        auto row_kernel = pieces ? paged_row_norm_append_kernel<T, kRow, 3> : paged_row_norm_append_kernel<T, 1, 3>;
+        LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, row_kernel, static_cast<unsigned char *>(kv.k_base), static_cast<unsigned char *>(kv.v_base),
+                                              NormAppendArgs(a), kv.block_table, g, d, dv, kv.vHeadStride() * int64_t(sizeof(T)),
+                                              kv.vTokenStride() * int64_t(sizeof(T)), max_blocks, error_flag));
+        return;
+    }
+    const bool wide = d % kVec == 0 && dv % kVec == 0 && a.row_stride % kVec == 0 && a.q_at % kVec == 0 && a.k_at % kVec == 0 &&
+                      a.v_at % kVec == 0 && aligned(a.proj) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out) &&
+                      a.rot_dims / 2 % kVec == 0;
+    const int64_t warps = int64_t(a.n_rows) * (a.nh + 2 * kv.nkvh);
+    cfg.gridDim = dim3(unsigned((warps + 7) / 8));
+    cfg.blockDim = dim3(256);
     constexpr int kPiece = 16 / int(sizeof(T));
     const int32_t longest = d > dv ? d : dv;
     // (small calls are latency-bound: there the kernel with a warp per head row has the shorter chain)

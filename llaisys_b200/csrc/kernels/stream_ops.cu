@@ -82,6 +82,28 @@ __global__ void embed_pairs_kernel(float *__restrict__ x, const int64_t *__restr
     }
 }
 
+// One thread per column pair (sine, cosine); the angle is reduced in f64, so that far positions lose nothing.
+template <typename T>
+__global__ void embed_positions_kernel(float *__restrict__ x, const int64_t *__restrict__ tokens, const int32_t *__restrict__ positions,
+                                       const double *__restrict__ freq, const T *__restrict__ w, int32_t d, int64_t vocab) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    int64_t tok = tokens[row];
+    tok = tok < 0 || tok >= vocab ? 0 : tok; // validated on the host; never read out of range here
+    const double pos = double(positions[row]);
+    constexpr double kTurn = 6.283185307179586;
+    for (int32_t i = int32_t(threadIdx.x); 2 * i < d; i += int32_t(blockDim.x)) {
+        const double angle = pos * freq[i];
+        float s, c;
+        sincosf(float(fma(-kTurn, rint(angle * (1.0 / kTurn)), angle)), &s, &c);
+        x[row * d + 2 * i] = to_f32(w[tok * d + 2 * i]) + s;
+        if (2 * i + 1 < d) {
+            x[row * d + 2 * i + 1] = to_f32(w[tok * d + 2 * i + 1]) + c;
+        }
+    }
+}
+
 template <typename T, int VEC>
 __global__ void stream_cast_kernel(T *__restrict__ out, int64_t out_stride, const float *__restrict__ x, int32_t d) {
     grid_dependency_wait();
@@ -183,12 +205,12 @@ __device__ __forceinline__ float block_sum(float v, float *part) {
     return tot;
 }
 
-// One CTA per row, like stream_rms_norm_kernel: two norms over the rows of a and b, their sum into the stream, and the norm
+// One CTA per row, like stream_rms_norm_kernel: norms over the rows of a and (TWO) b, their sum into the stream, and the norm
 // that follows. The first PER_THREAD pieces of a thread stay in registers.
-template <typename T, int VEC, int PER_THREAD>
+template <typename T, int VEC, int PER_THREAD, bool TWO>
 __global__ void stream_add_normed_kernel(float *__restrict__ x, const float *__restrict__ a, const T *__restrict__ wa,
                                          const float *__restrict__ b, const T *__restrict__ wb, float scale, float eps,
-                                         T *__restrict__ h, const T *__restrict__ w, float offset, int32_t d) {
+                                         T *__restrict__ h, const T *__restrict__ w, float offset, int32_t d, float branch_offset) {
     grid_dependency_wait();
     grid_launch_dependents();
     using F = Vec<float, VEC>;
@@ -209,23 +231,36 @@ __global__ void stream_add_normed_kernel(float *__restrict__ x, const float *__r
         const int32_t i = int32_t(threadIdx.x) + r * step;
         if (i < n_vec) {
             ha[r] = reinterpret_cast<const F *>(a + row)[i];
-            hb[r] = reinterpret_cast<const F *>(b + row)[i];
             square(ha[r], sa);
-            square(hb[r], sb);
+            if constexpr (TWO) {
+                hb[r] = reinterpret_cast<const F *>(b + row)[i];
+                square(hb[r], sb);
+            }
         }
     }
     for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * step; i < n_vec; i += step) {
         square(reinterpret_cast<const F *>(a + row)[i], sa);
-        square(reinterpret_cast<const F *>(b + row)[i], sb);
+        if constexpr (TWO) {
+            square(reinterpret_cast<const F *>(b + row)[i], sb);
+        }
     }
-    const float ia = rsqrtf(block_sum(sa, s_a) / float(d) + eps) * scale, ib = rsqrtf(block_sum(sb, s_b) / float(d) + eps) * scale;
+    const float ia = rsqrtf(block_sum(sa, s_a) / float(d) + eps) * scale;
+    const float ib = TWO ? rsqrtf(block_sum(sb, s_b) / float(d) + eps) * scale : 0.f;
     float sx = 0.f;
     auto add = [&](int32_t i, const F &fa, const F &fb) {
         F f = reinterpret_cast<const F *>(x + row)[i];
-        const W va = reinterpret_cast<const W *>(wa)[i], vb = reinterpret_cast<const W *>(wb)[i];
+        const W va = reinterpret_cast<const W *>(wa)[i];
+        W vb;
+        if constexpr (TWO) {
+            vb = reinterpret_cast<const W *>(wb)[i];
+        }
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            f.v[e] += fa.v[e] * ia * to_f32(va.v[e]) + fb.v[e] * ib * to_f32(vb.v[e]);
+            float more = fa.v[e] * ia * (branch_offset + to_f32(va.v[e]));
+            if constexpr (TWO) {
+                more += fb.v[e] * ib * (branch_offset + to_f32(vb.v[e]));
+            }
+            f.v[e] += more;
         }
         square(f, sx);
         reinterpret_cast<F *>(x + row)[i] = f;
@@ -239,7 +274,7 @@ __global__ void stream_add_normed_kernel(float *__restrict__ x, const float *__r
         }
     }
     for (int32_t i = int32_t(threadIdx.x) + PER_THREAD * step; i < n_vec; i += step) {
-        add(i, reinterpret_cast<const F *>(a + row)[i], reinterpret_cast<const F *>(b + row)[i]);
+        add(i, reinterpret_cast<const F *>(a + row)[i], TWO ? reinterpret_cast<const F *>(b + row)[i] : F{});
     }
     if (h == nullptr) {
         return;
@@ -432,6 +467,19 @@ void embed_pairs(stream_t stream, llaisysDataType_t dtype, float *x, const int64
     check_launch("embed_pairs");
 }
 
+void embed_positions(stream_t stream, llaisysDataType_t dtype, float *x, const int64_t *tokens, const int32_t *positions,
+                     const double *freq, const void *w, size_t rows, size_t d, size_t vocab) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        launch_programmatic(embed_positions_kernel<T>, dim3(unsigned(rows)), block_for((d + 1) / 2, 2), static_cast<cudaStream_t>(stream), x,
+                            tokens, positions, freq, static_cast<const T *>(w), int32_t(d), int64_t(vocab));
+    });
+    check_launch("embed_positions");
+}
+
 void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t out_stride, const float *x, size_t rows, size_t d) {
     if (rows == 0 || d == 0) {
         return;
@@ -464,7 +512,8 @@ void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const 
 }
 
 void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const float *a, const void *wa, const float *b,
-                       const void *wb, float scale, float eps, void *h, const void *w, float offset, size_t rows, size_t d) {
+                       const void *wb, float scale, float eps, void *h, const void *w, float offset, size_t rows, size_t d,
+                       float branch_offset) {
     if (rows == 0 || d == 0) {
         return;
     }
@@ -473,9 +522,11 @@ void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const
         using T = decltype(tag);
         const bool wide = d % 4 == 0 && aligned16(x) && aligned16(a) && aligned16(b) && aligned16(wa) && aligned16(wb) && aligned16(h) &&
                           aligned16(w);
-        auto kernel = wide ? stream_add_normed_kernel<T, 4, 3> : stream_add_normed_kernel<T, 1, 3>;
+        auto kernel = b != nullptr ? (wide ? stream_add_normed_kernel<T, 4, 3, true> : stream_add_normed_kernel<T, 1, 3, true>)
+                                   : (wide ? stream_add_normed_kernel<T, 4, 4, false> : stream_add_normed_kernel<T, 1, 4, false>);
         launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, x, a, static_cast<const T *>(wa), b,
-                            static_cast<const T *>(wb), scale, eps, static_cast<T *>(h), static_cast<const T *>(w), offset, int32_t(d));
+                            static_cast<const T *>(wb), scale, eps, static_cast<T *>(h), static_cast<const T *>(w), offset, int32_t(d),
+                            branch_offset);
     });
     check_launch("stream_add_normed");
 }

@@ -445,8 +445,25 @@ void PagedKV::requireEqualRows(size_t layer, const char *what) const {
 
 void PagedKV::requirePlain(size_t layer, const AttnOptions &opt) const {
     requireEqualRows(layer, "attention on the CPU");
-    KV_REQUIRE(opt.window == 0 && opt.row_scale == nullptr && opt.row_stride == 0, LLAISYS_E_UNSUPPORTED,
-               "paged attention: windows and output scales on NVIDIA caches only");
+    KV_REQUIRE(opt.window == 0 && opt.row_scale == nullptr && opt.row_stride == 0 && opt.gates == nullptr, LLAISYS_E_UNSUPPORTED,
+               "paged attention: windows, output scales and gated weights on NVIDIA caches only");
+}
+
+void PagedKV::requireGates(const AttnOptions &opt) const {
+    KV_REQUIRE(opt.gates == nullptr || (opt.keep_first == 0 && opt.row_scale == nullptr), LLAISYS_E_UNSUPPORTED,
+               "gated attention: neither kept tokens nor output factors");
+}
+
+int PagedKV::runGates(const kernels::KVView &v, const kernels::AttnBatch &b, const void *q, float scale, const kernels::GateArgs &gates,
+                      const kernels::AttnOut &o, llaisysStream_t stream) const {
+#ifdef ENABLE_NVIDIA_API
+    kernels::attention_gates(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch().error_flag);
+    noteAttentionKernel(LLAISYS_KERNEL_GATES);
+    return LLAISYS_KERNEL_GATES;
+#else
+    (void)v, (void)b, (void)q, (void)scale, (void)gates, (void)o, (void)stream;
+    fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
+#endif
 }
 
 std::byte *PagedKV::poolData(size_t layer) const {
@@ -642,8 +659,9 @@ void PagedKV::decodeDev(size_t layer, void *out, float *part, const void *q, con
     }
     KV_REQUIRE((out != nullptr) != (part != nullptr), LLAISYS_E_INVALID, "paged attention: exactly one output");
     KV_REQUIRE(q && seq_ids_dev && kv_lens_dev, LLAISYS_E_INVALID, "paged attention: null argument");
-    KV_REQUIRE(part == nullptr || (opt.row_scale == nullptr && opt.row_stride == 0), LLAISYS_E_INVALID,
-               "paged attention: partial results take neither an output scale nor a row stride");
+    KV_REQUIRE(part == nullptr || (opt.row_scale == nullptr && opt.row_stride == 0 && opt.gates == nullptr), LLAISYS_E_INVALID,
+               "paged attention: partial results take neither an output scale, a row stride nor gated weights");
+    requireGates(opt);
     launchDecode(layer, out, part, q, nullptr, nullptr, seq_ids_dev, kv_lens_dev, n_seqs, max_kv_len, nh, scale, stream,
                  _overlap, nullptr, nullptr, nullptr, opt);
 }
@@ -742,6 +760,8 @@ void PagedKV::launchDecode(size_t layer, void *out, float *part, const void *q, 
             }
             _last_kernel = LLAISYS_KERNEL_DECODE_TMA_FUSED;
             noteAttentionKernel(_last_kernel);
+        } else if (opt.gates != nullptr) {
+            _last_kernel = runGates(v, b, q_at, scale, *opt.gates, o, stream);
         } else {
             _last_kernel = run_attention_nvidia(stream, _cfg.dtype, v, b, q_at, scale, o, scratch());
         }
@@ -768,6 +788,7 @@ void PagedKV::prefillDev(size_t layer, void *out, const void *q, const int32_t *
     }
     KV_REQUIRE(out && q && seq_ids_dev && q_starts_dev && kv_lens_dev, LLAISYS_E_INVALID,
                "paged attention: null argument");
+    requireGates(opt);
     const kernels::KVView v = view(layer);
     kernels::AttnBatch b;
     b.seq_ids = seq_ids_dev;
@@ -793,7 +814,8 @@ void PagedKV::prefillDev(size_t layer, void *out, const void *q, const int32_t *
     }
 #ifdef ENABLE_NVIDIA_API
     enter();
-    _last_kernel = run_attention_nvidia(stream, _cfg.dtype, v, b, q, scale, o, scratch());
+    _last_kernel = opt.gates != nullptr ? runGates(v, b, q, scale, *opt.gates, o, stream)
+                                        : run_attention_nvidia(stream, _cfg.dtype, v, b, q, scale, o, scratch());
 #else
     (void)stream;
     fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");

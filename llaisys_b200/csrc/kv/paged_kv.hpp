@@ -34,6 +34,7 @@ struct AttnOptions {
     size_t keep_first = 0;             // with a window: the first tokens of a sequence that stay visible behind it
     const float *row_scale = nullptr;  // device, [rows, nh]: factor on every head's output
     size_t row_stride = 0;             // elements between output rows; 0 = packed
+    const kernels::GateArgs *gates = nullptr; // weights without a softmax, mixed over the heads; with neither kept tokens nor factors
 };
 
 struct PagedKVConfig {
@@ -157,6 +158,10 @@ private:
     void markDirty(int32_t seq, int32_t lo, int32_t hi);
     void checkLayer(size_t layer) const;
     void requireEqualRows(size_t layer, const char *what) const; // K and V rows of one length, unpadded
+    void requireGates(const AttnOptions &opt) const;
+    // gated attention of one batch: the tile kernel where the shape allows, the generic one otherwise -> LLAISYS_KERNEL_*
+    int runGates(const kernels::KVView &v, const kernels::AttnBatch &b, const void *q, float scale, const kernels::GateArgs &gates,
+                 const kernels::AttnOut &o, llaisysStream_t stream) const;
     void requirePlain(size_t layer, const AttnOptions &opt) const;
     kernels::KVView view(size_t layer) const;
     core::Runtime &enter() const;                   // make the cache's device current on this thread

@@ -159,12 +159,44 @@ class LlaisysDoderaxMeta(Structure):
                 ("pair_mul_cur", c_int64), ("eps", c_float), ("logit_scale", c_float), ("end_token", c_int64)]
 
 
+class LlaisysGatesAttentionMeta(Structure):
+    """struct LlaisysGatesAttentionMeta (include/llaisys/models/lilovik.h)."""
+    _fields_ = [("heads", c_size_t), ("kv_heads", c_size_t), ("dim", c_size_t), ("vdim", c_size_t), ("scale", c_float),
+                ("softcap", c_float), ("temp_coef", c_float), ("temp_every", c_float)]
+
+
+class LlaisysLilovikLayerMeta(Structure):
+    """struct LlaisysLilovikLayerMeta (include/llaisys/models/lilovik.h)."""
+    _fields_ = [("recurrent", c_int), ("attn", LlaisysGatesAttentionMeta), ("gru_width", c_size_t), ("ff", c_size_t)]
+
+
+class LlaisysLilovikMeta(Structure):
+    """struct LlaisysLilovikMeta (include/llaisys/models/lilovik.h)."""
+    _fields_ = [("dtype", llaisysDataType_t), ("nlayer", c_size_t), ("layers", POINTER(LlaisysLilovikLayerMeta)),
+                ("width", c_size_t), ("voc", c_size_t), ("maxseq", c_size_t), ("eps", c_float), ("logit_scale", c_float),
+                ("end_token", c_int64)]
+
+
 class LlaisysNormAppend(Structure):
     """struct LlaisysNormAppend (include/llaisys/mixers.h)."""
     _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("k_at", c_int64), ("v_at", c_int64),
                 ("gate_at", c_int64), ("q_norm", c_void_p), ("k_norm", c_void_p), ("eps", c_float), ("gate_scale", c_float),
                 ("q_out", c_void_p), ("row_scale", c_void_p), ("seq_ids_dev", c_void_p), ("positions_dev", c_void_p),
-                ("n_rows", c_size_t), ("nh", c_size_t), ("rot_dims", c_size_t), ("rot_table", c_void_p)]
+                ("n_rows", c_size_t), ("nh", c_size_t), ("rot_dims", c_size_t), ("rot_table", c_void_p), ("row_norm", c_int),
+                ("bias", c_void_p), ("temp_coef", c_float), ("temp_every", c_float)]
+
+
+class LlaisysGates(Structure):
+    """struct LlaisysGates (include/llaisys/mixers.h)."""
+    _fields_ = [("softcap", c_float), ("slopes", c_void_p), ("bias", c_void_p), ("talk", c_void_p)]
+
+
+class LlaisysMinGru(Structure):
+    """struct LlaisysMinGru (include/llaisys/mixers.h)."""
+    _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("z_at", c_int64), ("x_at", c_int64), ("g_at", c_int64),
+                ("bias_z", c_void_p), ("bias_x", c_void_p), ("width", c_size_t), ("state", c_void_p), ("slot_stride", c_int64),
+                ("seq_ids_dev", c_void_p), ("q_starts_dev", c_void_p), ("kv_lens_dev", c_void_p), ("n_seqs", c_size_t),
+                ("n_rows", c_size_t), ("max_q_len", c_size_t), ("out", c_void_p), ("out_stride", c_int64)]
 
 
 class LlaisysGatedDelta(Structure):
@@ -323,6 +355,10 @@ PROTOTYPES: dict[str, tuple] = {
     "llaisysPagedAttentionOptDev": (c_int, [_KV, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t,
                                             c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, c_size_t, c_void_p,
                                             c_size_t, llaisysStream_t]),
+    "llaisysPagedAttentionGatesDev": (c_int, [_KV, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t,
+                                              c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, POINTER(LlaisysGates),
+                                              c_size_t, llaisysStream_t]),
+    "llaisysMinGruDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysMinGru), c_int, llaisysStream_t]),
     "llaisysRotaryTableDev": (c_int, [llaisysDeviceType_t, c_int, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t,
                                       llaisysStream_t]),
     "llaisysGatedDeltaDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysGatedDelta), c_int,
@@ -352,6 +388,8 @@ PROTOTYPES: dict[str, tuple] = {
     "llaisysModelRecordStream": (c_int, [_MODEL, c_int]),
     "llaisysModelLayerStream": (c_int, [_MODEL, POINTER(c_float), c_size_t, POINTER(c_size_t)]),
     # include/llaisys/models/vozozen.h
+    # include/llaisys/models/lilovik.h
+    "llaisysLilovikModelCreate": (_MODEL, [POINTER(LlaisysLilovikMeta), llaisysDeviceType_t, c_int]),
     # include/llaisys/models/doderax.h
     "llaisysDoderaxModelCreate": (_MODEL, [POINTER(LlaisysDoderaxMeta), llaisysDeviceType_t, c_int]),
     "llaisysVozozenModelCreate": (_MODEL, [POINTER(LlaisysVozozenMeta), llaisysDeviceType_t, c_int]),
@@ -400,5 +438,6 @@ __all__ = [
     "llaisysDataType_t", "DataType", "llaisysDeviceType_t", "DeviceType", "llaisysMemcpyKind_t", "MemcpyKind",
     "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent",
     "LlaisysNormAppend", "LlaisysGatedLinear", "LlaisysGatedDelta", "LlaisysDoderaxMeta", "LlaisysDoderaxLayerMeta",
+    "LlaisysGates", "LlaisysMinGru", "LlaisysLilovikMeta", "LlaisysLilovikLayerMeta", "LlaisysGatesAttentionMeta",
     "LlaisysSinkAttentionMeta", "LlaisysDeltaMixerMeta", "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
 ]

@@ -14,8 +14,8 @@ from typing import Sequence
 
 import numpy as np
 
-from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysGatedDelta, LlaisysGatedLinear, LlaisysNormAppend, Status,
-                         llaisysPagedKV_t)
+from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysGatedDelta, LlaisysGatedLinear, LlaisysGates, LlaisysMinGru,
+                         LlaisysNormAppend, Status, llaisysPagedKV_t)
 from .runtime import _addr
 
 _I32P = ctypes.POINTER(c_int32)
@@ -30,6 +30,8 @@ class Kernel(IntEnum):
     DECODE_TMA_FUSED = 4
     DECODE_CP_ASYNC = 5
     PREFILL_TC = 6
+    GATES = 7
+    GATES_TILES = 8
 
 
 def last_attention_kernel() -> Kernel:
@@ -279,9 +281,9 @@ class PagedKVCache:
         return self
 
     def norm_append_dev(self, layer: int, stream, **fields) -> None:
-        """Per-head norm and rotation of q and k, append of k and v, gates to factors; fields of LlaisysNormAppend (buffers may be
+        """Norm (per head, or of the whole row) and rotation of q and k, append of k and v, gates to factors; fields of LlaisysNormAppend (buffers may be
         tensors)."""
-        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev", "rot_table"}
+        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev", "rot_table", "bias"}
         args = LlaisysNormAppend(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
         _check(LIB_LLAISYS.llaisysPagedKVNormAppendDev(self._kv, layer, byref(args), stream))
 
@@ -294,6 +296,25 @@ class PagedKVCache:
             self._kv, layer, _addr(out), _addr(q), _addr(seq_ids_dev), None if q_starts_dev is None else _addr(q_starts_dev),
             _addr(kv_lens_dev), n_seqs, total_q, max_q_len, max_kv_len, nh, scale, window,
             keep_first, None if row_scale is None else _addr(row_scale), row_stride, stream))
+
+
+    def gates_dev(self, layer: int, out, q, seq_ids_dev, q_starts_dev, kv_lens_dev, *, n_seqs: int, total_q: int, max_q_len: int,
+                  max_kv_len: int, nh: int, scale: float, stream, softcap: float = 0.0, slopes=None, bias=None, talk=None,
+                  window: int = 0, row_stride: int = 0) -> None:
+        """Attention without a softmax, weights mixed over the heads (llaisysPagedAttentionGatesDev): decode (q_starts_dev None) or
+        ragged chunks."""
+        gates = LlaisysGates(softcap=softcap, **{k: None if v is None else _addr(v) for k, v in
+                                                 (("slopes", slopes), ("bias", bias), ("talk", talk))})
+        _check(LIB_LLAISYS.llaisysPagedAttentionGatesDev(
+            self._kv, layer, _addr(out), _addr(q), _addr(seq_ids_dev), None if q_starts_dev is None else _addr(q_starts_dev),
+            _addr(kv_lens_dev), n_seqs, total_q, max_q_len, max_kv_len, nh, scale, window, byref(gates), row_stride, stream))
+
+
+def min_gru_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
+    """minGRU on device buffers; fields of LlaisysMinGru (include/llaisys/mixers.h), buffers may be tensors."""
+    pointers = {"proj", "bias_z", "bias_x", "state", "seq_ids_dev", "q_starts_dev", "kv_lens_dev", "out"}
+    args = LlaisysMinGru(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+    _check(LIB_LLAISYS.llaisysMinGruDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
 
 
 def gated_linear_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
