@@ -161,6 +161,12 @@ void attention_generic(stream_t stream, llaisysDataType_t dtype, const KVView &k
 void attention_gates(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch, const void *q, float scale,
                      const GateArgs &gates, const AttnOut &out, int32_t *error_flag);
 
+// The same on the tensor cores: bf16, rows of at most 128 in whole 16-element steps, 16-token pages, at most 64 heads. Returns -1 if
+// the view or shape is not covered, or the scratch is smaller than attention_gates_tiles_scratch asks for.
+int attention_gates_tiles(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch, const void *q, float scale,
+                          const GateArgs &gates, const AttnOut &out, const AttnScratch &scratch);
+void attention_gates_tiles_scratch(size_t longest_v_row, size_t *floats, size_t *counters);
+
 // K2 (+ fused K3): split-KV flash decoding for 16-bit K/V, head_dim 128, page size 16, GQA group <= 8,
 // one query per sequence. Returns -1 if the shape is not covered.
 int attention_decode_split(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch,

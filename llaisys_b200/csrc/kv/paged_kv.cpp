@@ -126,6 +126,18 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
             kernels::attention_prefill_tc_scratch(&f2, &c2);
             _partials_floats = std::max(floats, f2);
             _counters_len = std::max(counters, c2);
+        }
+        size_t longest_v = 0; // of the layers that the gated tile kernel can serve
+        for (const Layer &l : _layers) {
+            longest_v = std::max(longest_v, l.k_dim <= 128 && l.v_dim <= 128 ? l.v_dim : 0);
+        }
+        if (cfg.dtype == LLAISYS_DTYPE_BF16 && cfg.page_size == 16 && longest_v != 0) {
+            size_t floats = 0, counters = 0;
+            kernels::attention_gates_tiles_scratch(longest_v, &floats, &counters);
+            _partials_floats = std::max(_partials_floats, floats);
+            _counters_len = std::max(_counters_len, counters);
+        }
+        if (_partials_floats != 0) {
             _partials = rt.allocateDeviceStorage(_partials_floats * sizeof(float));
             _counters = rt.allocateDeviceStorage(_counters_len * sizeof(int32_t));
             kernels::fill_zero(rt.stream(), _counters->memory(), _counters->size());
@@ -457,9 +469,13 @@ void PagedKV::requireGates(const AttnOptions &opt) const {
 int PagedKV::runGates(const kernels::KVView &v, const kernels::AttnBatch &b, const void *q, float scale, const kernels::GateArgs &gates,
                       const kernels::AttnOut &o, llaisysStream_t stream) const {
 #ifdef ENABLE_NVIDIA_API
-    kernels::attention_gates(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch().error_flag);
-    noteAttentionKernel(LLAISYS_KERNEL_GATES);
-    return LLAISYS_KERNEL_GATES;
+    int used = LLAISYS_KERNEL_GATES_TILES;
+    if (kernels::attention_gates_tiles(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch()) != 0) {
+        kernels::attention_gates(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch().error_flag);
+        used = LLAISYS_KERNEL_GATES;
+    }
+    noteAttentionKernel(used);
+    return used;
 #else
     (void)v, (void)b, (void)q, (void)scale, (void)gates, (void)o, (void)stream;
     fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
