@@ -1,11 +1,12 @@
-"""bench.py --workload vozozen | doderax: a design beside its closest relative at equal size, one GPU -- Vozozen beside Qwen2,
-Doderax beside Vozozen.
+"""bench.py --workload vozozen | doderax | lilovik: a design beside its closest relative at equal size, one GPU -- Vozozen beside Qwen2,
+Doderax beside Vozozen, Lilovik beside Qwen2.
 
 Two parts, one JSON line:
   models   prefill and decode throughput of whole models with random weights. Equal size: the same width, query and kv heads,
            layers and vocabulary, and an MLP of as many parameters (two matrices have an inner size 1.5 times that of Qwen2's
            three). Vozozen's second mixer (gated linear attention) comes on top of Qwen2's attention; Doderax has as many heads of
-           the delta rule in every layer, and attention in every other one.
+           the delta rule in every layer, and attention in every other one. Lilovik has Qwen2's attention heads and MLP sizes, and in
+           every other layer a minGRU of as many parameters instead of the attention.
   kernels  every new kernel alone next to the like kernel of the relative, each as a fraction of its own roofline: CUDA graphs of
            launches over rotating buffers larger than L2, the median of the replays.
 """
@@ -54,8 +55,22 @@ def doderax_config(s: dict) -> dict:
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 10007, "mul_cur": 257}}, "layers": layers * (s["layers"] // 2)}
 
 
+def lilovik_config(s: dict) -> dict:
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 30.0,
+            "q_temp": {"coef": 0.1, "every": 1024}}
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    layers = [{"type": "attention", "mixer": attn, "mlp": mlp}, {"type": "mingru", "mixer": {"width": gru_width(s)}, "mlp": mlp}]
+    return {"architecture": "Lilovik", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": layers * (s["layers"] // 2)}
+
+
+def gru_width(s: dict) -> int:
+    """Channels of a minGRU with as many parameters as the attention."""
+    return (s["heads"] + s["kv_heads"]) * D // 2
+
+
 def attention_layers(family: str, s: dict) -> int:
-    return s["layers"] // 2 if family == "doderax" else s["layers"]
+    return s["layers"] // 2 if family in ("doderax", "lilovik") else s["layers"]
 
 
 def build_model(torch, llaisys, family: str, s: dict):
@@ -78,6 +93,11 @@ def build_model(torch, llaisys, family: str, s: dict):
 
         cfg = doderax_config(s)
         shapes = weight_shapes(cfg, [(LOW_RANK, LOW_RANK)] * s["layers"])
+    elif family == "lilovik":
+        from llaisys_b200.models.lilovik import weight_shapes
+
+        cfg = lilovik_config(s)
+        shapes = weight_shapes(cfg)
     else:
         from llaisys_b200.models.vozozen import weight_shapes
 
@@ -86,7 +106,9 @@ def build_model(torch, llaisys, family: str, s: dict):
     g = torch.Generator(device="cuda").manual_seed(4)
     weights, total, per_token = {}, 0, 0
     for name, shape in shapes.items():
-        if name.endswith(("norm", "norm1", "norm2", ".out")):
+        if family == "lilovik" and name.endswith(("talk", "pb", ".b")):
+            w = torch.eye(shape[0]) + 0.1 if name.endswith("talk") else torch.full(shape, -3.0 if name.endswith("pb") else 0.0)
+        elif name.endswith(("norm", "norm1", "norm2", "norm1b", "norm2b", ".out")):
             w = torch.ones(shape)
         elif name.endswith(("a2.b", "dt_bias")):
             w = torch.full(shape, 3.0 if family == "vozozen" else -5.0)
@@ -100,7 +122,7 @@ def build_model(torch, llaisys, family: str, s: dict):
         if name not in ("embed", "bigram"):
             total += w.numel() * 2
             per_token += w.numel() if w.ndim == 2 and name != "head" and not name.endswith(".conv") else 0
-    cls = llaisys.models.Doderax if family == "doderax" else llaisys.models.Vozozen
+    cls = getattr(llaisys.models, family.capitalize())
     model = cls(config=cfg, state_dict=weights, dtype=llaisys.DataType.BF16)
     return model, total, per_token
 
@@ -118,9 +140,9 @@ def visible(n: int, window: int | None, keep: int = 0) -> int:
 def prefill_flops(family: str, s: dict, lens: list[int], per_token: int) -> float:
     tokens = sum(lens)
     flops = 2.0 * tokens * per_token + 2.0 * len(lens) * s["vocab"] * s["width"]
-    window, keep = (None if family == "qwen2" else s["window"]), (KEEP_FIRST if family == "doderax" else 0)
+    window, keep = (None if family in ("qwen2", "lilovik") else s["window"]), (KEEP_FIRST if family == "doderax" else 0)
     flops += attention_layers(family, s) * s["heads"] * 4.0 * D * sum(visible(n, window, keep) for n in lens)
-    if family != "qwen2":  # state update and read-out, and the delta rule's correction
+    if family not in ("qwen2", "lilovik"):  # state update and read-out, and the delta rule's correction
         flops += s["layers"] * s["gla_heads"] * tokens * (6.0 if family == "doderax" else 4.0) * D * D
     return flops
 
@@ -158,10 +180,12 @@ def measure_model(torch, llaisys, stream, family: str, s: dict, repeats: int) ->
     model.decode_loop(seqs, nxt, DECODE_STEPS + 1)
     ms = model.last_loop_ms
     keys = DECODE_CTX + DECODE_STEPS // 2
-    if family != "qwen2":
+    if family not in ("qwen2", "lilovik"):
         keys = min(keys, s["window"] + (KEEP_FIRST if family == "doderax" else 0))
     kv = attention_layers(family, s) * DECODE_SEQS * keys * s["kv_heads"] * 2 * D * 2
-    state = 2 * s["layers"] * DECODE_SEQS * s["gla_heads"] * D * D * 4 if family != "qwen2" else 0
+    state = 2 * s["layers"] * DECODE_SEQS * s["gla_heads"] * D * D * 4 if family not in ("qwen2", "lilovik") else 0
+    if family == "lilovik":
+        state = 2 * (s["layers"] // 2) * DECODE_SEQS * gru_width(s) * 4
     moved = weight_bytes + kv + state
     rec["decode"] = {"tokens_per_s": DECODE_SEQS * 1e3 / ms, "ms_per_step": ms, "bytes": {"weights": weight_bytes, "kv": kv, "state": state},
                      "gb_per_s": moved / ms / 1e6, "frac_of_copy": moved / ms / 1e6 / hbm, "peak_kind": kind}
@@ -301,6 +325,70 @@ class Kernels:
                                              pos.data_ptr(), n, heads, 1e6, self.cs)
         assert rc == 0
 
+    def gates(self, heads: int, kv_heads: int, ctx: int = 2048, layers: int = 3) -> dict:
+        """Attention without a softmax beside Qwen2's on the same pages: decode over 64 sequences, one chunk of 8192 tokens, eight of
+        1024; the position-wise kernel in front of each."""
+        torch, ll = self.torch, self.ll
+        out = {}
+        n_seqs, rows = 64, 8192
+        cache = ll.PagedKVCache(max(n_seqs * ctx, rows) // 16, kv_heads, D, nlayer=layers, dtype=ll.DataType.BF16,
+                                device=ll.DeviceType.NVIDIA, max_seqs=n_seqs, max_pages_per_seq=max(ctx, rows) // 16)
+        cache.set_launch_overlap(True)
+        width = (heads + 2 * kv_heads) * D
+        opt = dict(softcap=30.0, slopes=torch.tensor([2.0 ** (-8 * (h + 1) / heads) for h in range(heads)], device="cuda"),
+                   bias=self.rand(heads) - 3, talk=(torch.eye(heads, device="cuda") + 0.1).bfloat16())
+        bias, qn, kn = self.rand(width), self.rand(heads * D), self.rand(kv_heads * D)
+        for what, lens, q_lens in (("decode", [ctx] * n_seqs, [1] * n_seqs), ("one chunk of 8192", [rows], [rows]),
+                                   ("eight chunks of 1024", [1024] * 8, [1024] * 8)):
+            seqs, n = [cache.add_seq() for _ in lens], sum(q_lens)
+            for q, length in zip(seqs, lens):
+                cache.reserve(q, length)
+            cache.flush()
+            for layer in range(layers):  # every page holds something
+                for q, length in zip(seqs, lens):
+                    k, v = self.rand(length, kv_heads, D), self.rand(length, kv_heads, D)
+                    cache.append_dev(layer, k, v, self.i32([q] * length), self.i32(list(range(length))), length, self.cs)
+                    self.stream.synchronize()
+            q, o = self.rand(n, heads, D), self.rand(n, heads, D)
+            ids, kv = self.i32(seqs), self.i32(lens)
+            starts = None if what == "decode" else self.i32([0, *np.cumsum(q_lens).tolist()])
+            common = dict(n_seqs=len(lens), total_q=n, max_q_len=max(q_lens), max_kv_len=max(lens), nh=heads, scale=D ** -0.5, stream=self.cs)
+            gates = self.time(lambda i: cache.gates_dev(i % layers, o, q, ids, starts, kv, **common, **opt))
+            soft = self.time(lambda i: cache.attention_dev(i % layers, o, q, ids, starts, kv, **common))
+            for name, us in (("gated attention, ", gates), ("softmax attention, Qwen2, ", soft)):
+                out[name + what] = self.memory(us, sum(lens) * kv_heads * 2 * D * 2 + 2 * n * heads * D * 2) if what == "decode" else \
+                    self.tensor(us, 4.0 * D * heads * sum(visible(x, None) for x in lens))
+            if what != "eight chunks of 1024":
+                ids_n = self.i32([s for s, c in zip(seqs, q_lens) for _ in range(c)])
+                pos_n = self.i32([length - c + t for length, c in zip(lens, q_lens) for t in range(c)])
+                proj = [self.rand(n, width) for _ in range(layers)]
+                us = self.time(lambda i: cache.norm_append_dev(
+                    i % layers, self.cs, proj=proj[i % layers], row_stride=width, q_at=0, k_at=heads * D, v_at=(heads + kv_heads) * D,
+                    gate_at=-1, q_norm=qn, k_norm=kn, eps=1e-6, gate_scale=1.0, q_out=q, row_scale=None, seq_ids_dev=ids_n,
+                    positions_dev=pos_n, n_rows=n, nh=heads, row_norm=1, bias=bias, temp_coef=0.1, temp_every=1024.0))
+                out[f"row norm + append, {n} rows"] = self.memory(us, n * 2 * width * 2)
+                us = self.time(lambda i: self._rope_append(cache, i % layers, q, proj[i % layers], bias, ids_n, pos_n, n, heads))
+                out[f"rope + append, Qwen2, {n} rows"] = self.memory(us, n * 2 * width * 2)
+            for s in seqs:
+                cache.free_seq(s)
+        cache.check()
+        cache.close()
+        return out
+
+    def min_gru(self, width: int, lens: list[int], copies: int = 6) -> dict:
+        torch, ll = self.torch, self.ll
+        rows = sum(lens)
+        copies = copies if rows * width * 6 < 30e6 else 3
+        proj = [self.rand(rows, 3 * width) for _ in range(copies)]
+        state = [torch.zeros(len(lens), width, device="cuda") for _ in range(copies)]
+        bz, bx, out = self.rand(width), self.rand(width), [self.rand(rows, width) for _ in range(copies)]
+        ids, starts, kv = self.i32(list(range(len(lens)))), self.i32([0, *np.cumsum(lens).tolist()]), self.i32([x + 100 for x in lens])
+        us = self.time(lambda i: ll.min_gru_dev(
+            ll.DataType.BF16, decode=max(lens) == 1, stream=self.cs, proj=proj[i % copies], row_stride=3 * width, z_at=0, x_at=width,
+            g_at=2 * width, bias_z=bz, bias_x=bx, width=width, state=state[i % copies], slot_stride=width, seq_ids_dev=ids,
+            q_starts_dev=starts, kv_lens_dev=kv, n_seqs=len(lens), n_rows=rows, max_q_len=max(lens), out=out[i % copies], out_stride=width))
+        return self.memory(us, rows * 4 * width * 2 + 2 * len(lens) * width * 4)
+
     def gated_linear(self, heads: int, lens: list[int], rank: int = 16, copies: int = 3) -> dict:
         torch, ll = self.torch, self.ll
         decode, rows, n = max(lens) == 1, sum(lens), heads * D
@@ -368,15 +456,21 @@ def run(args) -> None:
     stream = torch.cuda.ExternalStream(int(getattr(handle, "value", handle)))
     repeats = 10 if args.repeats == 100 else max(3, args.repeats)
     design = args.workload
-    relative = {"vozozen": "qwen2", "doderax": "vozozen"}[design]
+    relative = {"vozozen": "qwen2", "doderax": "vozozen", "lilovik": "qwen2"}[design]
     chunks = {"one run of 8192": [8192], "eight runs of 1024": [1024] * 8}
     models, kernels = {}, {}
     with ClockSampler(local_rank) as clocks:
         for name, s in SIZES.items():
             models[name] = {"size": s, **{f: measure_model(torch, llaisys, stream, f, s, repeats) for f in (design, relative)}}
             k = Kernels(torch, llaisys, stream, max(30, repeats))
-            kernels[name] = k.attention(s["heads"], s["kv_heads"], s["window"], design=design)
             h = s["gla_heads"]
+            if design == "lilovik":
+                kernels[name] = k.gates(s["heads"], s["kv_heads"])
+                kernels[name]["minGRU decode, 64 sequences"] = k.min_gru(gru_width(s), [1] * 64)
+                for what, lens in chunks.items():
+                    kernels[name]["minGRU chunk, " + what] = k.min_gru(gru_width(s), lens)
+            else:
+                kernels[name] = k.attention(s["heads"], s["kv_heads"], s["window"], design=design)
             kernels[name]["gated linear decode, 64 sequences"] = k.gated_linear(h, [1] * 64)
             if design == "doderax":
                 kernels[name]["gated delta decode, decay per channel, 64 sequences"] = k.gated_delta(h, h, [1] * 64, 16)
