@@ -1284,7 +1284,7 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=100, help="steps per timed graph replay (the graph is replayed >= 30 times)")
     ap.add_argument("--warmup", type=int, default=20)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="north_star", choices=["north_star", "config2", "config3", "config4", "config5", "copy", "vozozen", "doderax"])
+    ap.add_argument("--workload", default="north_star", choices=["north_star", "config2", "config3", "config4", "config5", "copy", "vozozen", "doderax", "lilovik"])
     ap.add_argument("--layers", type=int, default=4, help="pools to rotate over between steps (L2 flush)")
     ap.add_argument("--repeats", type=int, default=100, help="replays of the timed graph (at least 30)")
     ap.add_argument("--tp", action="store_true", help="config4 on several GPUs: tensor parallelism instead of sequence sharding")
@@ -1317,7 +1317,7 @@ def main() -> None:
     if args.workload == "copy":
         run_copy_workload(args)
         return
-    if args.workload in ("vozozen", "doderax"):
+    if args.workload in ("vozozen", "doderax", "lilovik"):
         import bench_models
 
         bench_models.run(args)
