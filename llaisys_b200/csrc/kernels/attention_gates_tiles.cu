@@ -10,8 +10,8 @@
 // Sums need no running maximum, so the tiles of all query blocks form one list that is cut into equal shares, one per SM; a block
 // that is cut leaves partial sums in the scratch, and the last of its CTAs to arrive adds them in a fixed order.
 //
-// K and V tiles come by cp.async through one buffer each: the next K tile is under way from the end of the scores, the next V tile
-// from the end of the values.
+// K and V tiles come by cp.async through two buffers each. Between two barriers a warp adds the values of tile t and scores tile t + 1,
+// while K of tile t + 2 and V of tile t + 1 are under way; between the next two it mixes tile t + 1.
 #include "kernels.hpp"
 #include "linear_tiles.cuh"
 
@@ -42,7 +42,8 @@ struct TileArgs {
 
 // Byte offsets of the parts of shared memory. Rows are padded by 16 bytes: ldmatrix then meets every bank once.
 struct TileSmem {
-    int k, v, w, m, t, row_of, prefix, total;
+    int k, v, w, m, t, row_of, pages, prefix, total, k_bytes, v_bytes; // k, v: two buffers
+
     __host__ __device__ TileSmem(const KVView &kv, int bq, int bk, int units_per_group, int hp, int n_seqs) {
         int at = 0;
         auto take = [&](int bytes) {
@@ -50,12 +51,15 @@ struct TileSmem {
             at += (bytes + 15) / 16 * 16;
             return here;
         };
-        k = take(kv.nkvh * bk * (kv.d + 8) * 2);
-        v = take(kv.nkvh * bk * (kv.vDim() + 8) * 2);
+        k_bytes = kv.nkvh * bk * (kv.d + 8) * 2;
+        v_bytes = kv.nkvh * bk * (kv.vDim() + 8) * 2;
+        k = take(2 * k_bytes);
+        v = take(2 * v_bytes);
         w = take(bq * bk * (hp + 8) * 2);
         m = take(kv.nkvh * units_per_group * 8 * (bk + 8) * 2);
         t = take(hp * (hp + 8) * 2);
         row_of = take(hp * 4);
+        pages = take(4 * bk / 16 * 4);
         prefix = take((n_seqs + 1) * 4);
         total = at;
     }
@@ -74,10 +78,10 @@ __device__ __forceinline__ float rcp(float x) {
     asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
 }
-// x_i <- unit / x_i for four numbers in [1, 2^31 + 1] with one reciprocal
-__device__ __forceinline__ void rcp4(float (&x)[4], float unit) {
+// 1 / x_i for four numbers in [1, 2^31 + 1] with one reciprocal, times unit, plus c_i
+__device__ __forceinline__ void rcp4(float (&x)[4], float unit, const float (&c)[4]) {
     const float p01 = x[0] * x[1], p23 = x[2] * x[3], r = rcp(p01 * p23) * unit, r01 = r * p23, r23 = r * p01;
-    const float y0 = r01 * x[1], y1 = r01 * x[0], y2 = r23 * x[3], y3 = r23 * x[2];
+    const float y0 = fmaf(r01, x[1], c[0]), y1 = fmaf(r01, x[0], c[1]), y2 = fmaf(r23, x[3], c[2]), y3 = fmaf(r23, x[2], c[3]);
     x[0] = y0;
     x[1] = y1;
     x[2] = y2;
@@ -103,39 +107,35 @@ __device__ __forceinline__ Block block_of(const TileArgs &a, int q_len, int kv_l
     return o;
 }
 
-// K or V rows of tile `tile`: a warp per (kv head, page). Keys from kv_end on become zero.
+// K or V rows of tile `tile`, its page ids in `ids`: a warp per (kv head, page). Keys from kv_end on become zero.
 template <int STEPS>
 __device__ __forceinline__ void load_tile(const TileArgs &a, const void *base, int64_t head_stride, int64_t token_stride, int width, uint32_t dst,
-                                          const int32_t *table, int tile, int kv_end) {
+                                          const int *ids, int tile, int kv_end) {
     const int warp = int(threadIdx.x) >> 5, lane = int(threadIdx.x) & 31, pages = a.bk / 16, row_bytes = (width + 8) * 2;
     const auto *src0 = static_cast<const __nv_bfloat16 *>(base);
     for (int item = warp; item < a.kv.nkvh * pages; item += kWarps) {
-        const int c = item / pages, first = tile * a.bk + (item - c * pages) * 16;
-        int page = -1;
-        if (first < kv_end) {
-            page = table[first / 16];
-            if (page < 0 || page >= a.kv.num_pages) {
-                if (lane == 0) {
-                    atomicOr(a.error_flag, kErrBadPage);
-                }
-                page = -1;
-            }
-        }
+        const int c = item / pages, p = item - c * pages, page = ids[p];
+        const int n = page < 0 ? 0 : min(16, kv_end - tile * a.bk - p * 16); // rows that exist
         const __nv_bfloat16 *src = src0 + int64_t(max(page, 0)) * a.kv.page_stride + c * head_stride;
-        const uint32_t rows = dst + uint32_t((c * a.bk + (item - c * pages) * 16) * row_bytes);
-        auto copy = [&](int r, int chunk) {
-            const bool ok = page >= 0 && first + r < kv_end;
-            cp_async_16(rows + uint32_t(r * row_bytes + chunk * 16), ok ? src + r * token_stride + chunk * 8 : src0, ok ? 16 : 0);
-        };
+        const uint32_t rows = dst + uint32_t((c * a.bk + p * 16) * row_bytes);
         if (width == STEPS * 16) {
-#pragma unroll 4
-            for (int i = lane; i < 16 * STEPS * 2; i += 32) {
-                copy(i / (STEPS * 2), i % (STEPS * 2));
+            constexpr int kChunks = STEPS * 2, kStride = 32 / kChunks;
+            const int r0 = lane / kChunks;
+            const __nv_bfloat16 *from = src + r0 * token_stride + lane % kChunks * 8;
+            uint32_t to = rows + uint32_t(r0 * row_bytes + lane % kChunks * 16);
+#pragma unroll
+            for (int r = 0; r < 16; r += kStride) {
+                const bool ok = r + r0 < n;
+                cp_async_16(to, ok ? from : src0, ok ? 16 : 0);
+                from += kStride * token_stride;
+                to += uint32_t(kStride * row_bytes);
             }
         } else {
             const int chunks = width / 8;
             for (int i = lane; i < 16 * chunks; i += 32) {
-                copy(i / chunks, i % chunks);
+                const int r = i / chunks, chunk = i - r * chunks;
+                const bool ok = r < n;
+                cp_async_16(rows + uint32_t(r * row_bytes + chunk * 16), ok ? src + r * token_stride + chunk * 8 : src0, ok ? 16 : 0);
             }
         }
     }
@@ -143,8 +143,8 @@ __device__ __forceinline__ void load_tile(const TileArgs &a, const void *base, i
 }
 
 // UNITS: per warp. SHARE: warps that share units -- they split a tile's keys for the scores and the value dims for the values.
-// STEPS: 16-element steps of a K row at most (4 or 8); V rows likewise.
-template <int UNITS, int SHARE, int STEPS>
+// STEPS: 16-element steps of a K row at most (4 or 8); V rows likewise. ONE: the units of a warp belong to one kv head.
+template <int UNITS, int SHARE, int STEPS, bool ONE>
 __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(const __grid_constant__ TileArgs a) {
     extern __shared__ __align__(16) unsigned char smem[];
     constexpr int kDims = (STEPS + SHARE - 1) / SHARE; // 16-dim blocks of V per warp
@@ -153,7 +153,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
     const uint32_t base = smem_u32(smem);
     const int warp = int(threadIdx.x) >> 5, lane = int(threadIdx.x) & 31;
     const int unit0 = warp / SHARE * UNITS, part = warp % SHARE, n_units = groups * a.units_per_group;
-    int *prefix = reinterpret_cast<int *>(smem + lay.prefix), *row_of = reinterpret_cast<int *>(smem + lay.row_of);
+    int *prefix = reinterpret_cast<int *>(smem + lay.prefix), *page_ids = reinterpret_cast<int *>(smem + lay.pages), *row_of = reinterpret_cast<int *>(smem + lay.row_of);
 
     // ---- the list of tiles, and this CTA's share of it ----
     for (int s = warp; s < a.batch.n_seqs; s += kWarps) {
@@ -267,8 +267,43 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         }
         const int32_t *table = a.kv.block_table + int64_t(a.batch.seq_ids != nullptr ? a.batch.seq_ids[seq] : seq) * a.kv.table_stride;
         const int64_t row0 = q_first(a.batch, seq) + blk.q0;
-        load_tile<STEPS>(a, a.kv.k_base, a.kv.head_stride, a.kv.token_stride, d, base + lay.k, table, blk.tile0 + from, blk.kv_end);
-        load_tile<STEPS>(a, a.kv.v_base, a.kv.vHeadStride(), a.kv.vTokenStride(), dv, base + lay.v, table, blk.tile0 + from, blk.kv_end);
+        const int pages = bk / 16;
+        auto page_id = [&](int tile, int p) { // -1: past the end, or out of range
+            const int at_block = tile * pages + p;
+            int id = -1;
+            if (at_block * 16 < blk.kv_end) {
+                id = table[at_block];
+                if (id < 0 || id >= a.kv.num_pages) {
+                    atomicOr(a.error_flag, kErrBadPage);
+                    id = -1;
+                }
+            }
+            return id;
+        };
+        auto load_k = [&](int t) {
+            if (t < upto) {
+                load_tile<STEPS>(a, a.kv.k_base, a.kv.head_stride, a.kv.token_stride, d, base + lay.k + (t & 1) * lay.k_bytes,
+                                 page_ids + (t & 3) * pages, blk.tile0 + t, blk.kv_end);
+            } else {
+                cp_async_commit(); // (an empty group keeps the count)
+            }
+        };
+        auto load_v = [&](int t) {
+            if (t < upto) {
+                load_tile<STEPS>(a, a.kv.v_base, a.kv.vHeadStride(), a.kv.vTokenStride(), dv, base + lay.v + (t & 1) * lay.v_bytes,
+                                 page_ids + (t & 3) * pages, blk.tile0 + t, blk.kv_end);
+            } else {
+                cp_async_commit();
+            }
+        };
+        if (int(threadIdx.x) < 3 * pages) {
+            const int t = from + int(threadIdx.x) / pages, p = int(threadIdx.x) % pages;
+            page_ids[(t & 3) * pages + p] = page_id(blk.tile0 + t, p);
+        }
+        __syncthreads();
+        load_k(from);
+        load_v(from);
+        load_k(from + 1);
 
         // queries, and what a column needs for its gate
         uint32_t qf[UNITS][STEPS][2];
@@ -309,56 +344,70 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         const bool pairs = share % 2 == 0; // the two columns of a thread are neighbouring heads of one query
         __half *w_s = reinterpret_cast<__half *>(smem + lay.w);
 
-        for (int t = from; t < upto; ++t) {
-            const int tile = blk.tile0 + t;
-            cp_async_wait<1>();
-            __syncthreads();
-            // ---- scores and gates ----
-            for (int kb = part; kb < bk / 16; kb += SHARE) {
-                float s[UNITS][4];
+        // scores and gates of NK blocks of 16 keys of tile t (kb0, kb0 + SHARE, ..); `edge`: some keys are out of sight
+        auto score = [&](auto nk, int t, int kb0, bool edge) {
+            constexpr int NK = decltype(nk)::value;
+            const uint32_t k_s = base + uint32_t(lay.k + (t & 1) * lay.k_bytes);
+            float s[NK][UNITS][4];
+#pragma unroll
+            for (int b = 0; b < NK; ++b) {
 #pragma unroll
                 for (int u = 0; u < UNITS; ++u) {
-                    s[u][0] = s[u][1] = s[u][2] = s[u][3] = 0.f;
+                    s[b][u][0] = s[b][u][1] = s[b][u][2] = s[b][u][3] = 0.f;
                 }
+            }
 #pragma unroll
-                for (int ks = 0; ks < STEPS; ++ks) {
-                    if (ks * 16 < d) {
+            for (int ks = 0; ks < STEPS; ++ks) {
+                if (ks * 16 < d) {
+#pragma unroll
+                    for (int b = 0; b < NK; ++b) {
                         uint32_t kf[4];
 #pragma unroll
                         for (int u = 0; u < UNITS; ++u) {
-                            if (u == 0 || group_of[u] != group_of[u - 1]) {
-                                ldmatrix_x4(kf, base + uint32_t(lay.k + ((group_of[u] * bk + kb * 16 + (lane & 15)) * (d + 8) + ks * 16 +
-                                                                         (lane >> 4) * 8) * 2));
+                            if (u == 0 || (!ONE && group_of[u] != group_of[u - 1])) {
+                                ldmatrix_x4(kf, k_s + uint32_t(((group_of[u] * bk + (kb0 + b * SHARE) * 16 + (lane & 15)) * (d + 8) + ks * 16 +
+                                                                (lane >> 4) * 8) * 2));
                             }
-                            mma_bf16(s[u], kf, qf[u][ks][0], qf[u][ks][1]);
+                            mma_bf16(s[b][u], kf, qf[u][ks][0], qf[u][ks][1]);
                         }
                     }
                 }
-                const int key = kb * 16 + (lane >> 2);
-                const float j = float(tile * bk + key);
+            }
+#pragma unroll
+            for (int b = 0; b < NK; ++b) {
+                const int key = (kb0 + b * SHARE) * 16 + (lane >> 2);
+                const float j = float((blk.tile0 + t) * bk + key);
 #pragma unroll
                 for (int u = 0; u < UNITS; ++u) {
-                    float x[4], ago[4]; // element i: key + 8 (i / 2), column i % 2
+                    float x[4], ago[4], c[4]; // element i: key + 8 (i / 2), column i % 2
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         ago[i] = q_pos[u][i & 1] - (j + float(i >> 1) * 8.f);
-                        x[i] = s[u][i] * to_exp;
+                        c[i] = fmaf(slope[u][i & 1], ago[i], shift[u][i & 1]);
                     }
                     if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
 #pragma unroll
                         for (int i = 0; i < 4; ++i) {
-                            x[i] = 1.f + ex2(fminf(x[i], 31.f));
+                            x[i] = 1.f + ex2(fminf(s[b][u][i] * to_exp, 31.f));
                         }
-                        rcp4(x, cap2);
+                        rcp4(x, cap2, c);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            x[i] = fmaf(s[b][u][i], to_exp, c[i]);
+                        }
                     }
+                    const float zero[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        x[i] = 1.f + ex2(fminf(x[i] + fmaf(slope[u][i & 1], ago[i], shift[u][i & 1]), 31.f));
+                        x[i] = 1.f + ex2(fminf(x[i], 31.f));
                     }
-                    rcp4(x, kWeightUnit);
+                    rcp4(x, kWeightUnit, zero);
+                    if (edge) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        x[i] = ago[i] >= 0.f && ago[i] < window ? x[i] : 0.f;
+                        for (int i = 0; i < 4; ++i) {
+                            x[i] = ago[i] >= 0.f && ago[i] < window ? x[i] : 0.f;
+                        }
                     }
 #pragma unroll
                     for (int r = 0; r < 2; ++r) {
@@ -378,39 +427,20 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
                     }
                 }
             }
-            __syncthreads();
-            if (t + 1 < upto) {
-                load_tile<STEPS>(a, a.kv.k_base, a.kv.head_stride, a.kv.token_stride, d, base + lay.k, table, tile + 1, blk.kv_end);
-            } else {
-                cp_async_commit(); // (an empty group keeps the count)
+        };
+        auto scores = [&](int t) {
+            const int first = (blk.tile0 + t) * bk;
+            const bool edge = first + bk > blk.pos0 + 1 || (a.batch.window > 0 && first + a.batch.window < blk.pos0 + blk.n_q);
+            int kb = part;
+            for (; kb + SHARE < bk / 16; kb += 2 * SHARE) {
+                score(std::integral_constant<int, 2>{}, t, kb, edge);
             }
-            // ---- mixing over the heads ----
-            for (int item = warp; item < blk.n_q * (bk / 16); item += kWarps) {
-                const int qi = item / (bk / 16), kb = item % (bk / 16);
-                for (int mt = 0; mt < a.hp / 16; ++mt) {
-                    float y0[4] = {0.f, 0.f, 0.f, 0.f}, y1[4] = {0.f, 0.f, 0.f, 0.f};
-                    for (int kt = 0; kt < a.hp / 16; ++kt) {
-                        uint32_t tf[4], wf[4];
-                        ldmatrix_x4(tf, base + uint32_t(lay.t + ((mt * 16 + (lane & 15)) * (a.hp + 8) + kt * 16 + (lane >> 4) * 8) * 2));
-                        ldmatrix_x4(wf, base + uint32_t(lay.w + (((qi * bk + kb * 16 + (lane & 7) + (lane >> 4) * 8) * (a.hp + 8)) + kt * 16 +
-                                                                 ((lane >> 3) & 1) * 8) * 2));
-                        mma_f16(y0, tf, wf[0], wf[1]);
-                        mma_f16(y1, tf, wf[2], wf[3]);
-                    }
-#pragma unroll
-                    for (int r = 0; r < 2; ++r) {
-                        const int row = row_of[mt * 16 + (lane >> 2) + 8 * r];
-                        if (row >= 0) {
-                            auto *dst = reinterpret_cast<uint32_t *>(smem + lay.m + ((row + qi * share) * (bk + 8) + kb * 16 + 2 * (lane & 3)) * 2);
-                            dst[0] = pack2<true>(y0[2 * r], y0[2 * r + 1]);
-                            dst[4] = pack2<true>(y1[2 * r], y1[2 * r + 1]);
-                        }
-                    }
-                }
+            if (kb < bk / 16) {
+                score(std::integral_constant<int, 1>{}, t, kb, edge);
             }
-            cp_async_wait<1>();
-            __syncthreads();
-            // ---- values ----
+        };
+        auto values = [&](int t) {
+            const uint32_t v_s = base + uint32_t(lay.v + (t & 1) * lay.v_bytes);
             for (int kb = 0; kb < bk / 16; ++kb) {
                 uint32_t mf[UNITS][2];
 #pragma unroll
@@ -425,20 +455,63 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
                         uint32_t vf[4];
 #pragma unroll
                         for (int u = 0; u < UNITS; ++u) {
-                            if (u == 0 || group_of[u] != group_of[u - 1]) {
-                                ldmatrix_x4_trans(vf, base + uint32_t(lay.v + ((group_of[u] * bk + kb * 16 + (lane & 7) + (lane >> 4) * 8) * (dv + 8) +
-                                                                               dim + ((lane >> 3) & 1) * 8) * 2));
+                            if (u == 0 || (!ONE && group_of[u] != group_of[u - 1])) {
+                                ldmatrix_x4_trans(vf, v_s + uint32_t(((group_of[u] * bk + kb * 16 + (lane & 7) + (lane >> 4) * 8) * (dv + 8) + dim +
+                                                                      ((lane >> 3) & 1) * 8) * 2));
                             }
                             mma_bf16(o[u][b], vf, mf[u][0], mf[u][1]);
                         }
                     }
                 }
             }
+        };
+        auto mix = [&]() { // a warp per (query, 16 keys, 16 heads)
+            const int tiles_h = a.hp / 16, per_q = pages * tiles_h;
+            for (int item = warp; item < blk.n_q * per_q; item += kWarps) {
+                const int qi = item / per_q, rest = item - qi * per_q, kb = rest / tiles_h, mt = rest - kb * tiles_h;
+                float y0[4] = {0.f, 0.f, 0.f, 0.f}, y1[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int kt = 0; kt < tiles_h; ++kt) {
+                    uint32_t tf[4], wf[4];
+                    ldmatrix_x4(tf, base + uint32_t(lay.t + ((mt * 16 + (lane & 15)) * (a.hp + 8) + kt * 16 + (lane >> 4) * 8) * 2));
+                    ldmatrix_x4(wf, base + uint32_t(lay.w + (((qi * bk + kb * 16 + (lane & 7) + (lane >> 4) * 8) * (a.hp + 8)) + kt * 16 +
+                                                             ((lane >> 3) & 1) * 8) * 2));
+                    mma_f16(y0, tf, wf[0], wf[1]);
+                    mma_f16(y1, tf, wf[2], wf[3]);
+                }
+#pragma unroll
+                for (int r = 0; r < 2; ++r) {
+                    const int row = row_of[mt * 16 + (lane >> 2) + 8 * r];
+                    if (row >= 0) {
+                        auto *dst = reinterpret_cast<uint32_t *>(smem + lay.m + ((row + qi * share) * (bk + 8) + kb * 16 + 2 * (lane & 3)) * 2);
+                        dst[0] = pack2<true>(y0[2 * r], y0[2 * r + 1]);
+                        dst[4] = pack2<true>(y1[2 * r], y1[2 * r + 1]);
+                    }
+                }
+            }
+        };
+
+        cp_async_wait<2>(); // K of the first tile
+        __syncthreads();
+        scores(from);
+        __syncthreads();
+        mix();
+        for (int t = from; t < upto; ++t) {
+            cp_async_wait<0>(); // V of tile t, K of tile t + 1
             __syncthreads();
+            int next_page = 0;
+            if (int(threadIdx.x) < pages) {
+                next_page = page_id(blk.tile0 + t + 3, int(threadIdx.x));
+            }
+            load_k(t + 2);
+            load_v(t + 1);
+            values(t);
             if (t + 1 < upto) {
-                load_tile<STEPS>(a, a.kv.v_base, a.kv.vHeadStride(), a.kv.vTokenStride(), dv, base + lay.v, table, tile + 1, blk.kv_end);
-            } else {
-                cp_async_commit();
+                scores(t + 1);
+                if (int(threadIdx.x) < pages) {
+                    page_ids[((t + 3) & 3) * pages + int(threadIdx.x)] = next_page;
+                }
+                __syncthreads();
+                mix();
             }
         }
 
@@ -527,7 +600,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
     }
 }
 
-constexpr int kMaxSmem = 220 * 1024;
+constexpr int kMaxSmem = 226 * 1024;
 
 int sm_count() {
     static int n = [] {
@@ -541,7 +614,8 @@ int sm_count() {
 
 template <int UNITS, int SHARE, int STEPS>
 void launch(cudaStream_t s, const TileArgs &args, size_t smem, int grid, bool overlap) {
-    auto kernel = attention_gates_tiles_kernel<UNITS, SHARE, STEPS>;
+    auto kernel = args.units_per_group % UNITS == 0 ? attention_gates_tiles_kernel<UNITS, SHARE, STEPS, true>
+                                                    : attention_gates_tiles_kernel<UNITS, SHARE, STEPS, UNITS == 1>;
     LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem));
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(unsigned(grid));
