@@ -1,0 +1,766 @@
+// Attention without a softmax (GateArgs) over chunks of queries, on the 5th-generation tensor cores (tcgen05 + TMEM): bf16, K and V
+// rows of 128, 16-token pages, at most 32 heads and 16 kv heads.
+//
+// Roofline: tensor; 4 * nh * 128 flops per visible (query, key) pair as for softmax attention. What bounds it is the multi-function
+// unit: a capped score and its sigmoid take two exponentials and half a reciprocal where a softmax takes one exponential.
+//
+// A CTA takes a block of bq queries with ALL heads, because the weights of all heads meet in every output, and visits its visible keys
+// 128 at a time (a TILE). A kv head's columns are the pairs (query, head of its group), padded to n_c, a multiple of 16; both products
+// are transposed, so that the long sides (keys, value dims) fill the 128 rows of an MMA and a kv head's few columns are its N:
+//   S_c[key, column]   = K_c q^T          A = K tile (K-major), B = queries in shared memory
+//   O_c[dim, column]  += V_c^T P_c        A = V tile (MN-major, as the pages hold it), B = P_c [column][key]
+// S_c and O_c of all kv heads live in TMEM (256 columns each).
+//
+//   warps 0-15   read S (lane = key), compute the weights, store them as f16 times 2^15 into the buffer that becomes P; when all heads
+//                are there, mix them IN PLACE: 16 keys of one query, all heads, are read as mma.sync operands, multiplied by the talk
+//                matrix (in registers) and stored as bf16 to the same places
+//   warp 16      TMA of K and V tiles into a ring of 32 KiB slots
+//   warp 17      one thread issues the MMAs: S of tile t + 1 kv head by kv head as the scores of tile t have been read, then O of tile t.
+//                Weights of tile t + 1 go where P_c of tile t was as soon as O_c has taken it.
+//
+// The tiles of all blocks form one line that is cut into equal shares, one per CTA; a block that is cut leaves partial sums in the
+// scratch (nothing is rescaled: sums add), and the last of its CTAs to arrive adds them in a fixed order.
+//
+// Every wait is bounded: one that runs out sets bit 8 of the error word and the CTA winds down. No cluster launch, no multicast.
+#include "kernels.hpp"
+#include "linear_tiles.cuh"
+#include "tcgen05_utils.cuh"
+
+#include <cuda.h>
+
+#include <algorithm>
+#include <cstring>
+
+namespace llaisys::kernels {
+
+namespace {
+
+constexpr int kD = 128, kBk = 128, kPages = kBk / 16;
+constexpr int kWorkers = 16, kProducer = 16, kIssuer = 17, kThreads = 18 * 32;
+constexpr int kSlot = kBk * kD * 2, kMaxStages = 6, kMaxColumns = 256, kMaxGroups = 16;
+constexpr int kSmemLimit = 227 * 1024, kErrTimeout = 8;
+constexpr float kLog2e = 1.4426950408889634f, kWeightUnit = 32768.f;
+
+struct Params {
+    AttnBatch batch;
+    GateArgs gates;
+    const __nv_bfloat16 *q;
+    __nv_bfloat16 *out;
+    int64_t out_stride;
+    float scale;
+    int64_t page0;
+    const int32_t *block_table;
+    int32_t table_stride, num_pages;
+    int32_t groups, share, bq, n_c, stages; // n_c: columns of a kv head, padded
+    float *partials; // [CTA][2][groups * n_c][128]
+    int32_t *counters;
+    int32_t *error_flag;
+};
+
+struct Block { // a block of queries
+    int q0, n_q;        // first query within its chunk, queries
+    int pos0, kv_end;   // position of the first query, keys that the last one sees
+    int tile0, n_tiles; // key tiles
+};
+
+__device__ __forceinline__ Block block_of(const Params &p, int q_len, int kv_len, int index) {
+    Block o;
+    o.q0 = index * p.bq;
+    o.n_q = min(p.bq, q_len - o.q0);
+    o.pos0 = kv_len - q_len + o.q0;
+    o.kv_end = o.n_q > 0 ? max(0, o.pos0 + o.n_q) : 0;
+    o.tile0 = p.batch.window > 0 ? max(0, o.pos0 - p.batch.window + 1) / kBk : 0;
+    o.n_tiles = o.n_q > 0 ? max(0, (o.kv_end + kBk - 1) / kBk - o.tile0) : 0;
+    return o;
+}
+
+// A CTA's walk over its share of the line: every role walks the same fragments.
+struct Walk {
+    int at, end, seq, index, block_begin;
+};
+struct Fragment {
+    Block block;
+    int seq, from, upto, block_begin; // tiles of the block
+    int64_t row0;                     // first query row
+};
+__device__ __forceinline__ bool next_fragment(const Params &p, Walk &w, Fragment &f) {
+    while (w.at < w.end) {
+        const int first = p.batch.q_starts[w.seq], q_len = p.batch.q_starts[w.seq + 1] - first;
+        f.block = block_of(p, q_len, p.batch.kv_lens[w.seq], w.index);
+        f.seq = w.seq;
+        f.block_begin = w.block_begin;
+        f.from = w.at - w.block_begin;
+        f.upto = min(f.block.n_tiles, w.end - w.block_begin);
+        f.row0 = first + f.block.q0;
+        w.block_begin += f.block.n_tiles;
+        w.index += 1;
+        if (w.index * p.bq >= q_len) {
+            w.index = 0;
+            w.seq += 1;
+        }
+        if (f.upto > f.from) {
+            w.at += f.upto - f.from;
+            return true;
+        }
+    }
+    return false;
+}
+
+__device__ __forceinline__ void tmem_ld8(uint32_t taddr, float (&v)[8]) {
+    uint32_t r[8];
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+                 : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        v[i] = __uint_as_float(r[i]);
+    }
+}
+__device__ __forceinline__ void mma_f16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+// unit / x_i + c_i for four numbers in [1, 2^31 + 1] with one reciprocal
+__device__ __forceinline__ void rcp4(float *x, float unit, const float *c) {
+    const float p01 = x[0] * x[1], p23 = x[2] * x[3], r = rcp(p01 * p23) * unit, r01 = r * p23, r23 = r * p01;
+    const float y0 = fmaf(r01, x[1], c[0]), y1 = fmaf(r01, x[0], c[1]), y2 = fmaf(r23, x[3], c[2]), y3 = fmaf(r23, x[2], c[3]);
+    x[0] = y0;
+    x[1] = y1;
+    x[2] = y2;
+    x[3] = y3;
+}
+__device__ __forceinline__ void store_u16(uint32_t addr, uint32_t v) {
+    asm volatile("st.shared.u16 [%0], %1;\n" ::"r"(addr), "h"(static_cast<unsigned short>(v)) : "memory");
+}
+__device__ __forceinline__ void store_u32(uint32_t addr, uint32_t v) { asm volatile("st.shared.u32 [%0], %1;\n" ::"r"(addr), "r"(v) : "memory"); }
+
+// Shared memory: ring | queries | weights (all 1024-byte aligned) | per-column constants | barriers | small words.
+struct Layout {
+    int q, w, columns, bars, misc, total;
+    __host__ __device__ Layout(int stages, int n_columns) {
+        q = stages * kSlot;
+        w = q + n_columns * kD * 2;
+        columns = w + n_columns * kBk * 2;
+        bars = columns + n_columns * 8;
+        misc = bars + (kMaxStages + 5 * kMaxGroups + 3) * 8;
+        misc = (misc + 15) / 16 * 16;
+        total = misc + 32; // [0, 16) zeros, then abort flag, TMEM base, `last`
+    }
+};
+// barriers
+constexpr int kBarFull = 0;                            // [stages] producer -> issuer: a tile has landed
+constexpr int kBarS = kBarFull + kMaxStages;           // [2][groups] S_c of a tile is written (and its K slot is free)
+constexpr int kBarPV = kBarS + 2 * kMaxGroups;         // [2][groups] O_c has taken a tile (its V slot and P_c are free)
+constexpr int kBarRead = kBarPV + 2 * kMaxGroups;      // [groups] workers -> issuer: S_c has been read
+constexpr int kBarP = kBarRead + kMaxGroups;           // workers -> issuer: P of a tile is complete
+constexpr int kBarQ = kBarP + 1;                       // workers -> issuer: queries of a fragment are in place
+constexpr int kBarO = kBarQ + 1;                       // workers -> issuer: O has been read
+
+template <int MT> // heads in whole 16s
+__global__ void __launch_bounds__(kThreads, 1)
+    attention_gates_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+                              const __grid_constant__ Params p) {
+    extern __shared__ __align__(1024) unsigned char smem[];
+    const int groups = p.groups, share = p.share, n_c = p.n_c, nh = p.batch.nh, n_columns = groups * n_c;
+    const Layout lay(p.stages, n_columns);
+    const uint32_t base = smem_u32(smem);
+    const int tid = int(threadIdx.x), warp = tid >> 5, lane = tid & 31;
+    int *misc = reinterpret_cast<int *>(smem + lay.misc);
+    volatile int *s_abort = misc + 4;
+    auto bar = [&](int which) { return base + uint32_t(lay.bars + which * 8); };
+    auto s_bar = [&](int n, int c) { return bar(kBarS + (n & 1) * kMaxGroups + c); };
+    auto pv_bar = [&](int n, int c) { return bar(kBarPV + (n & 1) * kMaxGroups + c); };
+    auto give_up = [&]() {
+        *s_abort = 1;
+        atomicOr(p.error_flag, kErrTimeout);
+    };
+
+    // ---- the line of tiles (its prefix sums lie in the ring, which nothing uses yet) ----
+    int *prefix = reinterpret_cast<int *>(smem);
+    for (int s = warp; s < p.batch.n_seqs; s += kThreads / 32) {
+        const int q_len = p.batch.q_starts[s + 1] - p.batch.q_starts[s], kv_len = p.batch.kv_lens[s], blocks = (q_len + p.bq - 1) / p.bq;
+        int sum = 0;
+        for (int b = lane; b < blocks; b += 32) {
+            sum += block_of(p, q_len, kv_len, b).n_tiles;
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        }
+        if (lane == 0) {
+            prefix[s + 1] = sum;
+        }
+    }
+    if (tid == 0) {
+        prefix[0] = 0;
+        for (int i = 0; i < kBarO + 1; ++i) {
+            mbar_init(bar(i), i >= kBarRead ? kWorkers : 1);
+        }
+        misc[0] = misc[1] = misc[2] = misc[3] = 0;
+        *s_abort = 0;
+        mbar_init_fence();
+    }
+    __syncthreads();
+    if (warp == 0) {
+        int carry = 0;
+        for (int s0 = 0; s0 < p.batch.n_seqs; s0 += 32) {
+            int v = s0 + lane < p.batch.n_seqs ? prefix[s0 + lane + 1] : 0;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, v, o);
+                v += lane >= o ? up : 0;
+            }
+            __syncwarp();
+            if (s0 + lane < p.batch.n_seqs) {
+                prefix[s0 + lane + 1] = carry + v;
+            }
+            carry += __shfl_sync(0xffffffffu, v, 31);
+        }
+    }
+    __syncthreads();
+    const int64_t total = prefix[p.batch.n_seqs], ctas = min(int64_t(gridDim.x), total); // (every share holds a tile)
+    grid_dependency_wait(); // (the index arrays above are older than the kernel before this one)
+    if (int64_t(blockIdx.x) >= ctas) {
+        return;
+    }
+    Walk walk{int(total * blockIdx.x / ctas), int(total * (blockIdx.x + 1) / ctas), 0, 0, 0};
+    {
+        int lo = 0, hi = p.batch.n_seqs - 1;
+        while (lo < hi) { // last sequence with prefix[seq] <= walk.at
+            const int mid = (lo + hi + 1) >> 1;
+            if (prefix[mid] <= walk.at) {
+                lo = mid;
+            } else {
+                hi = mid - 1;
+            }
+        }
+        walk.seq = lo;
+        walk.block_begin = prefix[lo];
+        const int q_len = p.batch.q_starts[lo + 1] - p.batch.q_starts[lo], kv_len = p.batch.kv_lens[lo], blocks = (q_len + p.bq - 1) / p.bq;
+        for (int b0 = 0; b0 < blocks; b0 += 32) { // every warp finds the same
+            const int mine = b0 + lane < blocks ? block_of(p, q_len, kv_len, b0 + lane).n_tiles : 0;
+            int v = mine;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, v, o);
+                v += lane >= o ? up : 0;
+            }
+            const unsigned past = __ballot_sync(0xffffffffu, walk.block_begin + v > walk.at);
+            if (past != 0u) {
+                const int at = __ffs(int(past)) - 1;
+                walk.block_begin += __shfl_sync(0xffffffffu, v - mine, at);
+                walk.index = b0 + at;
+                break;
+            }
+            walk.block_begin += __shfl_sync(0xffffffffu, v, 31);
+        }
+    }
+    __syncthreads(); // the prefix sums have been read
+    // rows of a tile past the last page keep what they held: their weights are zero, so they only have to be finite
+    for (int i = tid; i < p.stages * kSlot / 16; i += kThreads) {
+        reinterpret_cast<uint4 *>(smem)[i] = make_uint4(0, 0, 0, 0);
+    }
+    // what a column adds to the exponent of its gate at distance x from the block's first query: columns[].x * x + columns[].y
+    const bool capped = p.gates.softcap > 0.f;
+    float2 *columns = reinterpret_cast<float2 *>(smem + lay.columns);
+    for (int i = tid; i < n_columns; i += kThreads) {
+        const int c = i / n_c, r = i - c * n_c, qi = r / share, h = c * share + r - qi * share;
+        float2 v = make_float2(0.f, 0.f);
+        if (qi < p.bq) {
+            const float b = p.gates.bias != nullptr ? to_f32(static_cast<const __nv_bfloat16 *>(p.gates.bias)[h]) : 0.f;
+            v.x = p.gates.slopes != nullptr ? kLog2e * p.gates.slopes[h] : 0.f;
+            v.y = fmaf(v.x, float(qi), -kLog2e * (b + (capped ? p.gates.softcap : 0.f)));
+        }
+        columns[i] = v;
+    }
+    if (warp == kIssuer) {
+        tmem_alloc(base + uint32_t(lay.misc + 20), 512);
+        tmem_relinquish();
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = uint32_t(misc[5]), tmem_o = tmem + kMaxColumns;
+
+    if (warp == kProducer) {
+        // ================================ K and V tiles ==================================================
+        bool alive = true;
+        int op = 0, n = 0; // operands loaded, tiles before this fragment
+        uint32_t free_bar[kMaxStages];
+        int free_parity[kMaxStages];
+        Fragment f;
+        while (alive && next_fragment(p, walk, f)) {
+            const int32_t *table = p.block_table + int64_t(p.batch.seq_ids != nullptr ? p.batch.seq_ids[f.seq] : f.seq) * p.table_stride;
+            const int n_pages = (f.block.kv_end + 15) / 16, count = f.upto - f.from;
+            auto page_of = [&](int t) { // of lane's page in tile t of the block; -1: none
+                const int i = (f.block.tile0 + t) * kPages + (lane & (kPages - 1));
+                int page = t < f.upto && i < n_pages ? table[i] : -1;
+                if (t < f.upto && i < n_pages && (page < 0 || page >= p.num_pages)) {
+                    atomicOr(p.error_flag, kErrBadPage);
+                    page = 0;
+                }
+                return page;
+            };
+            // the operand of every kv head of one tile
+            auto load = [&](int page, int tile_no, bool is_v) {
+                const int here = __popc(__ballot_sync(0xffffffffu, lane < kPages && page >= 0));
+                const int c3 = int((p.page0 + max(page, 0)) * 2);
+                for (int c = 0; c < groups && alive; ++c, ++op) {
+                    const int slot = op % p.stages;
+                    if (op >= p.stages && !wait_or_abort(free_bar[slot], uint32_t(free_parity[slot]), s_abort)) {
+                        alive = false;
+                        break;
+                    }
+                    if (lane == 0) {
+                        mbar_arrive_expect_tx(bar(kBarFull + slot), uint32_t(here) * 4096);
+                    }
+                    __syncwarp();
+                    if (lane < kPages && page >= 0) {
+                        if (is_v) { // one box per page: [half of the dims][16 tokens][128 B]
+                            tma_load_5d(base + uint32_t(slot * kSlot + lane * 4096), &map_v, 0, 0, 0, c, c3 + 1, bar(kBarFull + slot));
+                        } else { // [half of the dims][128 tokens][128 B]
+                            const uint32_t dst = base + uint32_t(slot * kSlot + lane * 2048);
+                            tma_load_4d(dst, &map_k, 0, 0, c, c3, bar(kBarFull + slot));
+                            tma_load_4d(dst + kSlot / 2, &map_k, 64, 0, c, c3, bar(kBarFull + slot));
+                        }
+                    }
+                    free_bar[slot] = is_v ? pv_bar(tile_no, c) : s_bar(tile_no, c);
+                    free_parity[slot] = (tile_no >> 1) & 1;
+                }
+            };
+            int page = page_of(f.from), ahead = page_of(f.from + 1);
+            load(page, n, false);
+            for (int i = 0; i < count && alive; ++i) {
+                const int two_ahead = page_of(f.from + i + 2);
+                if (i + 1 < count) {
+                    load(ahead, n + i + 1, false);
+                }
+                load(page, n + i, true);
+                page = ahead;
+                ahead = two_ahead;
+            }
+            n += count;
+        }
+        if (!alive && lane == 0) {
+            give_up();
+        }
+    } else if (warp == kIssuer) {
+        // ================================ MMAs (one thread) ==============================================
+        if (lane == 0) {
+            const uint32_t idesc_s = make_idesc(true, false, kBk, n_c), idesc_o = make_idesc(true, false, kD, n_c) | (1u << 15); // A MN-major
+            bool ok = true;
+            int op = 0, n = 0, n_fragments = 0;
+            auto next_slot = [&]() { // waits for the operand
+                const int slot = op % p.stages;
+                ok = ok && wait_or_abort(bar(kBarFull + slot), uint32_t(op / p.stages) & 1u, s_abort);
+                ++op;
+                return base + uint32_t(slot * kSlot);
+            };
+            auto scores = [&](int tile_no, bool waits) { // S of tile tile_no; waits: until the tile before it has been read
+                for (int c = 0; c < groups && ok; ++c) {
+                    if (waits) {
+                        ok = wait_or_abort(bar(kBarRead + c), uint32_t(tile_no - 1) & 1u, s_abort);
+                    }
+                    const uint32_t k_s = next_slot();
+                    if (!ok) {
+                        break;
+                    }
+                    tc_fence_after();
+                    const uint32_t q_s = base + uint32_t(lay.q + c * n_c * kD * 2);
+#pragma unroll
+                    for (int ks = 0; ks < kD / 16; ++ks) {
+                        umma_f16(tmem + uint32_t(c * n_c), smem_desc_sw128(k_s + (ks >> 2) * (kSlot / 2) + (ks & 3) * 32, 0, 1024),
+                                 smem_desc_sw128(q_s + uint32_t((ks >> 2) * n_c * 128 + (ks & 3) * 32), 0, 1024), idesc_s, ks > 0 ? 1u : 0u);
+                    }
+                    umma_commit(s_bar(tile_no, c));
+                }
+            };
+            Fragment f;
+            for (; ok && next_fragment(p, walk, f); ++n_fragments) {
+                const int count = f.upto - f.from;
+                ok = wait_or_abort(bar(kBarQ), uint32_t(n_fragments) & 1u, s_abort);
+                scores(n, n > 0);
+                for (int i = 0; i < count && ok; ++i, ++n) {
+                    if (i + 1 < count) {
+                        scores(n + 1, true);
+                    }
+                    ok = ok && wait_or_abort(bar(kBarP), uint32_t(n) & 1u, s_abort);
+                    if (i == 0 && n_fragments > 0) {
+                        ok = ok && wait_or_abort(bar(kBarO), uint32_t(n_fragments - 1) & 1u, s_abort);
+                    }
+                    for (int c = 0; c < groups && ok; ++c) {
+                        const uint32_t v_s = next_slot();
+                        if (!ok) {
+                            break;
+                        }
+                        tc_fence_after();
+                        const uint32_t p_s = base + uint32_t(lay.w + c * n_c * kBk * 2);
+#pragma unroll
+                        for (int kk = 0; kk < kBk / 16; ++kk) { // 16 keys: one page
+                            umma_f16(tmem_o + uint32_t(c * n_c), smem_desc_sw128(v_s + kk * 4096, 2048, 1024),
+                                     smem_desc_sw128(p_s + uint32_t((kk >> 2) * n_c * 128 + (kk & 3) * 32), 0, 1024), idesc_o,
+                                     i > 0 || kk > 0 ? 1u : 0u);
+                        }
+                        umma_commit(pv_bar(n, c));
+                    }
+                }
+            }
+            if (!ok) {
+                give_up();
+            }
+        }
+        __syncwarp();
+    } else {
+        // ================================ weights, mixing, output ========================================
+        bool dead = false; // a thread whose wait ran out keeps walking, so that the named barriers see all of them
+        auto wait = [&](uint32_t at, int parity) {
+            if (!dead && !wait_or_abort(at, uint32_t(parity), s_abort)) {
+                dead = true;
+                give_up();
+            }
+            __syncwarp();
+        };
+        auto arrive = [&](int which) {
+            __syncwarp();
+            if (lane == 0) {
+                mbar_arrive(bar(which));
+            }
+        };
+        const int quarter = warp & 3, part = warp >> 2, units = n_c / 8; // lanes of TMEM, and which of every four 8-column units
+        const int key = quarter * 32 + lane;
+        const uint32_t lanes = uint32_t(quarter * 32) << 16;
+        const float to_exp = capped ? 2.f * kLog2e * p.scale / p.gates.softcap : -kLog2e * p.scale, cap2 = 2.f * kLog2e * p.gates.softcap;
+        const uint32_t w_s = base + uint32_t(lay.w);
+        // a weight of column r: row r, 16-byte chunk (key / 8) ^ (r mod 8) of the row's 64-key half
+        const uint32_t w_key = w_s + uint32_t((quarter >> 1) * n_c * 128 + (((quarter & 1) * 4 + (lane >> 3)) << 4) + (lane & 7) * 2);
+
+        // talk as mma operands, and where heads lie: byte offset of a head's kv head, and its place in the group
+        uint32_t talk[MT][MT][4];
+        int in_base[MT], in_at[MT], out_base[MT][2], out_at[MT][2];
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+#pragma unroll
+            for (int kt = 0; kt < MT; ++kt) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    float v[2];
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        const int h = mt * 16 + (lane >> 2) + (e & 1) * 8, g = kt * 16 + 2 * (lane & 3) + (e >> 1) * 8 + x;
+                        v[x] = 0.f;
+                        if (h < nh && g < nh) {
+                            v[x] = p.gates.talk != nullptr ? to_f32(static_cast<const __nv_bfloat16 *>(p.gates.talk)[h * nh + g]) : float(h == g);
+                        }
+                    }
+                    talk[mt][kt][e] = pack2<false>(v[0], v[1]);
+                }
+            }
+            const int hi = mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+            in_base[mt] = hi < nh ? hi / share * n_c * kBk * 2 : -1;
+            in_at[mt] = hi % share;
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const int ho = mt * 16 + (lane >> 2) + 8 * r;
+                out_base[mt][r] = ho < nh ? ho / share * n_c * kBk * 2 : -1;
+                out_at[mt][r] = ho % share;
+            }
+        }
+
+        auto load_q = [&](const Fragment &f) {
+            for (int i = tid; i < n_columns * 16; i += kWorkers * 32) {
+                const int col = i >> 4, cc = i & 15, c = col / n_c, r = col - c * n_c, qi = r / share, h = c * share + r - qi * share;
+                uint4 v = make_uint4(0, 0, 0, 0);
+                if (qi < f.block.n_q) {
+                    v = *reinterpret_cast<const uint4 *>(p.q + ((f.row0 + qi) * nh + h) * kD + cc * 8);
+                }
+                *reinterpret_cast<uint4 *>(smem + lay.q + c * n_c * kD * 2 + (cc >> 3) * n_c * 128 + r * 128 + (((cc & 7) ^ (r & 7)) << 4)) = v;
+            }
+            fence_proxy_async_smem();
+            arrive(kBarQ);
+        };
+
+        Fragment f, next;
+        bool more = next_fragment(p, walk, f);
+        if (more) {
+            load_q(f);
+        }
+        int n = 0;
+        while (more) {
+            const Block &blk = f.block;
+            for (int t = f.from; t < f.upto; ++t, ++n) {
+                const int first = (blk.tile0 + t) * kBk;
+                const bool edge = first + kBk > blk.pos0 + 1 || (p.batch.window > 0 && first + p.batch.window < blk.pos0 + blk.n_q);
+                const float ago0 = float(blk.pos0 - first - key); // from this thread's key to the block's first query
+                for (int c = 0; c < groups; ++c) {
+                    wait(s_bar(n, c), (n >> 1) & 1);
+                    tc_fence_after();
+                    const int shift = (part - c * units) & 3;
+                    bool first_store = true;
+                    for (int u = shift; u < units; u += 4) {
+                        const int col = c * n_c + u * 8;
+                        float x[8], a[8];
+                        tmem_ld8(tmem + lanes + uint32_t(col), x);
+#pragma unroll
+                        for (int i = 0; i < 8; i += 2) {
+                            const float4 k2 = *reinterpret_cast<const float4 *>(columns + col + i);
+                            a[i] = fmaf(k2.x, ago0, k2.y);
+                            a[i + 1] = fmaf(k2.z, ago0, k2.w);
+                        }
+                        if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) {
+                                x[i] = 1.f + ex2(fminf(x[i] * to_exp, 31.f));
+                            }
+                            rcp4(x, cap2, a);
+                            rcp4(x + 4, cap2, a + 4);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) {
+                                x[i] = fmaf(x[i], to_exp, a[i]);
+                            }
+                        }
+                        const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            x[i] = 1.f + ex2(fminf(x[i], 31.f));
+                        }
+                        rcp4(x, kWeightUnit, zero);
+                        rcp4(x + 4, kWeightUnit, zero);
+                        if (edge) {
+                            const float window = p.batch.window > 0 ? float(p.batch.window) : INFINITY;
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) {
+                                const float ago = ago0 + float((u * 8 + i) / share);
+                                x[i] = ago >= 0.f && ago < window ? x[i] : 0.f;
+                            }
+                        }
+                        if (first_store && n > 0) {
+                            wait(pv_bar(n - 1, c), ((n - 1) >> 1) & 1);
+                        }
+                        first_store = false;
+                        const uint32_t at = w_key + uint32_t(c * n_c * kBk * 2 + u * 8 * 128);
+#pragma unroll
+                        for (int i = 0; i < 8; i += 2) {
+                            const uint32_t two = pack2<false>(x[i], x[i + 1]);
+                            store_u16((at ^ uint32_t(i << 4)) + uint32_t(i * 128), two);
+                            store_u16((at ^ uint32_t((i + 1) << 4)) + uint32_t((i + 1) * 128), two >> 16);
+                        }
+                    }
+                    tc_fence_before();
+                    arrive(kBarRead + c);
+                }
+                named_barrier_sync(1, kWorkers * 32); // weights of all heads are in place
+                for (int item = warp; item < blk.n_q * kPages; item += kWorkers) {
+                    const int qi = item / kPages, kb = item % kPages, q_row = qi * share;
+                    const int half = (kb >> 2) * n_c * 128, chunk = (kb & 3) * 2;
+                    uint32_t in[MT][4];
+#pragma unroll
+                    for (int kt = 0; kt < MT; ++kt) {
+                        const int row = q_row + in_at[kt];
+                        const uint32_t at = in_base[kt] < 0 ? base + uint32_t(lay.misc)
+                                                            : w_s + uint32_t(in_base[kt] + half + row * 128 + (((chunk + (lane >> 4)) ^ (row & 7)) << 4));
+                        ldmatrix_x4_trans(in[kt], at);
+                    }
+                    __syncwarp();
+#pragma unroll
+                    for (int mt = 0; mt < MT; ++mt) {
+                        float y0[4] = {0.f, 0.f, 0.f, 0.f}, y1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                        for (int kt = 0; kt < MT; ++kt) {
+                            mma_f16(y0, talk[mt][kt], in[kt][0], in[kt][1]);
+                            mma_f16(y1, talk[mt][kt], in[kt][2], in[kt][3]);
+                        }
+#pragma unroll
+                        for (int r = 0; r < 2; ++r) {
+                            if (out_base[mt][r] >= 0) {
+                                const int row = q_row + out_at[mt][r];
+                                const uint32_t at = w_s + uint32_t(out_base[mt][r] + half + row * 128 + ((chunk ^ (row & 7)) << 4) + (lane & 3) * 4);
+                                store_u32(at, pack2<true>(y0[2 * r], y0[2 * r + 1]));
+                                store_u32(at ^ 16u, pack2<true>(y1[2 * r], y1[2 * r + 1])); // (chunk is even)
+                            }
+                        }
+                    }
+                }
+                fence_proxy_async_smem();
+                arrive(kBarP);
+            }
+            more = next_fragment(p, walk, next);
+            if (more) {
+                load_q(next); // every S of this fragment is done: its queries are free
+            }
+            // ---- the block's output, whole or in pieces ----
+            wait(pv_bar(n - 1, groups - 1), ((n - 1) >> 1) & 1);
+            tc_fence_after();
+            const bool whole = f.from == 0 && f.upto == blk.n_tiles;
+            const int64_t slot = int64_t(n_columns) * kD;
+            auto slot_of = [&](int cta, bool begins) { return p.partials + (int64_t(cta) * 2 + (begins ? 1 : 0)) * slot; };
+            auto each_unit = [&](auto &&body) {
+                for (int g = part; g < groups * units; g += 4) {
+                    body(g * 8);
+                }
+            };
+            auto store = [&](int col, const float (&v)[8]) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const int c = (col + i) / n_c, r = col + i - c * n_c, qi = r / share, h = c * share + r - qi * share;
+                    if (qi < blk.n_q) {
+                        p.out[(f.row0 + qi) * p.out_stride + int64_t(h) * kD + key] = __float2bfloat16_rn(v[i] * (1.f / kWeightUnit));
+                    }
+                }
+            };
+            if (whole) {
+                each_unit([&](int col) {
+                    float v[8];
+                    tmem_ld8(tmem_o + lanes + uint32_t(col), v);
+                    store(col, v);
+                });
+                tc_fence_before();
+                arrive(kBarO);
+            } else {
+                float *own = slot_of(int(blockIdx.x), f.from == 0);
+                each_unit([&](int col) {
+                    float v[8];
+                    tmem_ld8(tmem_o + lanes + uint32_t(col), v);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        own[int64_t(col + i) * kD + key] = v[i];
+                    }
+                });
+                tc_fence_before();
+                arrive(kBarO);
+                // CTAs whose shares touch the block: share c holds tile t iff c is the largest with c * total < (t + 1) * ctas
+                const int first_cta = int(((int64_t(f.block_begin) + 1) * ctas - 1) / total);
+                const int last_cta = int((int64_t(f.block_begin + blk.n_tiles) * ctas - 1) / total);
+                __threadfence();
+                named_barrier_sync(1, kWorkers * 32);
+                if (tid == 0) {
+                    misc[6] = atomicAdd(p.counters + first_cta, 1) == last_cta - first_cta;
+                    if (misc[6]) {
+                        p.counters[first_cta] = 0;
+                    }
+                }
+                named_barrier_sync(1, kWorkers * 32);
+                const bool last = misc[6] != 0;
+                if (last) {
+                    __threadfence();
+                    each_unit([&](int col) {
+                        float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+                        for (int cta = first_cta; cta <= last_cta; ++cta) {
+                            const float *from = slot_of(cta, cta == first_cta) + int64_t(col) * kD + key;
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) {
+                                v[i] += __ldcg(from + i * kD);
+                            }
+                        }
+                        store(col, v);
+                    });
+                }
+                named_barrier_sync(1, kWorkers * 32); // `last` has been read
+            }
+            f = next;
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == kIssuer) {
+        tmem_dealloc(tmem, 512);
+    }
+}
+
+int sm_count() {
+    static int n = [] {
+        int dev = 0, v = 0;
+        LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
+        LLAISYS_CUDA_CHECK(cudaDeviceGetAttribute(&v, cudaDevAttrMultiProcessorCount, dev));
+        return v;
+    }();
+    return n;
+}
+
+template <int MT>
+void launch(cudaStream_t s, const CUtensorMap &map_k, const CUtensorMap &map_v, const Params &p, size_t smem, int grid, bool overlap) {
+    auto kernel = attention_gates_tc_kernel<MT>;
+    LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit));
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(unsigned(grid));
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = overlap ? 1 : 0;
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, map_k, map_v, p));
+}
+
+} // namespace
+
+void attention_gates_tc_scratch(size_t *floats, size_t *counters) {
+    *floats = size_t(sm_count()) * 2 * kMaxColumns * kD;
+    *counters = size_t(sm_count());
+}
+
+int attention_gates_tc(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch, const void *q, float scale,
+                       const GateArgs &gates, const AttnOut &out, const AttnScratch &scratch) {
+    if (dtype != LLAISYS_DTYPE_BF16 || kv.d != kD || kv.vDim() != kD || kv.page_size != 16 || kv.block_table == nullptr ||
+        kv.tma_tile_desc == nullptr || batch.q_starts == nullptr || batch.kv_lens == nullptr || kv.nkvh <= 0 || kv.nkvh > kMaxGroups ||
+        batch.nh > 32 || batch.nh % kv.nkvh != 0 || batch.n_seqs <= 0 || batch.n_seqs > 8192 || batch.max_q_len < 8 || batch.keep_first != 0 ||
+        out.out == nullptr || out.part != nullptr || out.row_scale != nullptr || reinterpret_cast<uintptr_t>(q) % 16 != 0) {
+        return -1;
+    }
+    Params p{};
+    p.share = batch.nh / kv.nkvh;
+    auto padded = [&](int bq) { return (bq * p.share + 15) / 16 * 16; };
+    for (int bq = 1; bq <= std::min(batch.max_q_len, 64) && kv.nkvh * padded(bq) <= kMaxColumns; ++bq) {
+        p.bq = bq;
+    }
+    if (p.bq < 4) {
+        return -1;
+    }
+    p.groups = kv.nkvh;
+    p.n_c = padded(p.bq);
+    const int n_columns = p.groups * p.n_c;
+    // (a slot is handed over by the barrier of the operand that it held: that barrier must not run on before the slot is due)
+    p.stages = std::min(kMaxStages, 3 * p.groups);
+    while (p.stages > 2 && Layout(p.stages, n_columns).total > kSmemLimit) {
+        --p.stages;
+    }
+    const Layout lay(p.stages, n_columns);
+    const int grid = sm_count();
+    if (lay.total > kSmemLimit || scratch.partials == nullptr || scratch.counters == nullptr || scratch.error_flag == nullptr ||
+        scratch.partials_floats < size_t(grid) * 2 * size_t(n_columns) * kD || scratch.counters_len < size_t(grid)) {
+        return -1;
+    }
+    p.batch = batch;
+    p.gates = gates;
+    p.q = static_cast<const __nv_bfloat16 *>(q);
+    p.out = static_cast<__nv_bfloat16 *>(out.out);
+    p.out_stride = out.row_stride ? out.row_stride : int64_t(batch.nh) * kD;
+    p.scale = scale;
+    p.page0 = kv.tma_page0;
+    p.block_table = kv.block_table;
+    p.table_stride = kv.table_stride;
+    p.num_pages = kv.num_pages;
+    p.partials = scratch.partials;
+    p.counters = scratch.counters;
+    p.error_flag = scratch.error_flag;
+    CUtensorMap map_k, map_v;
+    std::memcpy(&map_k, kv.tma_tile_desc, sizeof(map_k));
+    std::memcpy(&map_v, static_cast<const unsigned char *>(kv.tma_tile_desc) + sizeof(map_k), sizeof(map_v));
+    auto s = static_cast<cudaStream_t>(stream);
+    batch.nh <= 16 ? launch<1>(s, map_k, map_v, p, size_t(lay.total), grid, kv.overlap_launch)
+                   : launch<2>(s, map_k, map_v, p, size_t(lay.total), grid, kv.overlap_launch);
+    check_launch("attention_gates_tc");
+    return 0;
+}
+
+} // namespace llaisys::kernels

@@ -11,7 +11,8 @@
 // that is cut leaves partial sums in the scratch, and the last of its CTAs to arrive adds them in a fixed order.
 //
 // K and V tiles come by cp.async through two buffers each. Between two barriers a warp adds the values of tile t and scores tile t + 1,
-// while K of tile t + 2 and V of tile t + 1 are under way; between the next two it mixes tile t + 1.
+// while K of tile t + 2 and V of tile t + 1 are under way; between the next two it mixes tile t + 1. Where two do not fit (many wide kv
+// heads) there is one buffer each, and both loads stand between the barriers of the mixing.
 #include "kernels.hpp"
 #include "linear_tiles.cuh"
 
@@ -33,6 +34,7 @@ struct TileArgs {
     GateArgs gates;
     float scale;
     int32_t bq, bk;          // queries of a block, keys of a tile
+    int32_t bufs;            // buffers per operand, 1 or 2
     int32_t units_per_group; // of one kv head
     int32_t hp;              // heads padded to 16
     float *partials;         // [CTA][2][units * 8 * dv]
@@ -42,9 +44,9 @@ struct TileArgs {
 
 // Byte offsets of the parts of shared memory. Rows are padded by 16 bytes: ldmatrix then meets every bank once.
 struct TileSmem {
-    int k, v, w, m, t, row_of, pages, prefix, total, k_bytes, v_bytes; // k, v: two buffers
+    int k, v, w, m, t, row_of, pages, prefix, total, k_bytes, v_bytes; // of one buffer
 
-    __host__ __device__ TileSmem(const KVView &kv, int bq, int bk, int units_per_group, int hp, int n_seqs) {
+    __host__ __device__ TileSmem(const KVView &kv, int bufs, int bq, int bk, int units_per_group, int hp, int n_seqs) {
         int at = 0;
         auto take = [&](int bytes) {
             const int here = at;
@@ -53,8 +55,8 @@ struct TileSmem {
         };
         k_bytes = kv.nkvh * bk * (kv.d + 8) * 2;
         v_bytes = kv.nkvh * bk * (kv.vDim() + 8) * 2;
-        k = take(2 * k_bytes);
-        v = take(2 * v_bytes);
+        k = take(bufs * k_bytes);
+        v = take(bufs * v_bytes);
         w = take(bq * bk * (hp + 8) * 2);
         m = take(kv.nkvh * units_per_group * 8 * (bk + 8) * 2);
         t = take(hp * (hp + 8) * 2);
@@ -149,7 +151,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
     extern __shared__ __align__(16) unsigned char smem[];
     constexpr int kDims = (STEPS + SHARE - 1) / SHARE; // 16-dim blocks of V per warp
     const int nh = a.batch.nh, groups = a.kv.nkvh, share = nh / groups, d = a.kv.d, dv = a.kv.vDim(), bk = a.bk;
-    const TileSmem lay(a.kv, a.bq, bk, a.units_per_group, a.hp, a.batch.n_seqs);
+    const TileSmem lay(a.kv, a.bufs, a.bq, bk, a.units_per_group, a.hp, a.batch.n_seqs);
     const uint32_t base = smem_u32(smem);
     const int warp = int(threadIdx.x) >> 5, lane = int(threadIdx.x) & 31;
     const int unit0 = warp / SHARE * UNITS, part = warp % SHARE, n_units = groups * a.units_per_group;
@@ -282,7 +284,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         };
         auto load_k = [&](int t) {
             if (t < upto) {
-                load_tile<STEPS>(a, a.kv.k_base, a.kv.head_stride, a.kv.token_stride, d, base + lay.k + (t & 1) * lay.k_bytes,
+                load_tile<STEPS>(a, a.kv.k_base, a.kv.head_stride, a.kv.token_stride, d, base + lay.k + (t & (a.bufs - 1)) * lay.k_bytes,
                                  page_ids + (t & 3) * pages, blk.tile0 + t, blk.kv_end);
             } else {
                 cp_async_commit(); // (an empty group keeps the count)
@@ -290,7 +292,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         };
         auto load_v = [&](int t) {
             if (t < upto) {
-                load_tile<STEPS>(a, a.kv.v_base, a.kv.vHeadStride(), a.kv.vTokenStride(), dv, base + lay.v + (t & 1) * lay.v_bytes,
+                load_tile<STEPS>(a, a.kv.v_base, a.kv.vHeadStride(), a.kv.vTokenStride(), dv, base + lay.v + (t & (a.bufs - 1)) * lay.v_bytes,
                                  page_ids + (t & 3) * pages, blk.tile0 + t, blk.kv_end);
             } else {
                 cp_async_commit();
@@ -303,7 +305,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         __syncthreads();
         load_k(from);
         load_v(from);
-        load_k(from + 1);
+        load_k(a.bufs == 2 ? from + 1 : upto); // (upto: an empty group)
 
         // queries, and what a column needs for its gate
         uint32_t qf[UNITS][STEPS][2];
@@ -347,7 +349,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         // scores and gates of NK blocks of 16 keys of tile t (kb0, kb0 + SHARE, ..); `edge`: some keys are out of sight
         auto score = [&](auto nk, int t, int kb0, bool edge) {
             constexpr int NK = decltype(nk)::value;
-            const uint32_t k_s = base + uint32_t(lay.k + (t & 1) * lay.k_bytes);
+            const uint32_t k_s = base + uint32_t(lay.k + (t & (a.bufs - 1)) * lay.k_bytes);
             float s[NK][UNITS][4];
 #pragma unroll
             for (int b = 0; b < NK; ++b) {
@@ -440,7 +442,7 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
             }
         };
         auto values = [&](int t) {
-            const uint32_t v_s = base + uint32_t(lay.v + (t & 1) * lay.v_bytes);
+            const uint32_t v_s = base + uint32_t(lay.v + (t & (a.bufs - 1)) * lay.v_bytes);
             for (int kb = 0; kb < bk / 16; ++kb) {
                 uint32_t mf[UNITS][2];
 #pragma unroll
@@ -494,6 +496,9 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
         __syncthreads();
         scores(from);
         __syncthreads();
+        if (a.bufs == 1) {
+            load_k(from + 1);
+        }
         mix();
         for (int t = from; t < upto; ++t) {
             cp_async_wait<0>(); // V of tile t, K of tile t + 1
@@ -502,8 +507,10 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
             if (int(threadIdx.x) < pages) {
                 next_page = page_id(blk.tile0 + t + 3, int(threadIdx.x));
             }
-            load_k(t + 2);
-            load_v(t + 1);
+            if (a.bufs == 2) {
+                load_k(t + 2);
+                load_v(t + 1);
+            }
             values(t);
             if (t + 1 < upto) {
                 scores(t + 1);
@@ -511,6 +518,10 @@ __global__ void __launch_bounds__(kThreads, 1) attention_gates_tiles_kernel(cons
                     page_ids[((t + 3) & 3) * pages + int(threadIdx.x)] = next_page;
                 }
                 __syncthreads();
+                if (a.bufs == 1) {
+                    load_k(t + 2);
+                    load_v(t + 1);
+                }
                 mix();
             }
         }
@@ -678,10 +689,11 @@ int attention_gates_tiles(stream_t stream, llaisysDataType_t dtype, const KVView
         return -1;
     }
     size_t smem = 0;
-    for (int bq = best; bq >= 1 && smem == 0; bq = bq > 1 ? bq / 2 : 0) {
+    for (int bufs = 2, bq = best; bufs >= 1 && smem == 0; bq > 1 ? bq /= 2 : (bq = best, --bufs)) {
         for (int bk = bq == 1 ? 128 : 64; bk >= 16; bk /= 2) {
-            const TileSmem lay(kv, bq, bk, units(bq), a.hp, batch.n_seqs);
+            const TileSmem lay(kv, bufs, bq, bk, units(bq), a.hp, batch.n_seqs);
             if (lay.total <= kMaxSmem) {
+                a.bufs = bufs;
                 a.bq = bq;
                 a.bk = bk;
                 a.units_per_group = units(bq);

@@ -167,6 +167,13 @@ int attention_gates_tiles(stream_t stream, llaisysDataType_t dtype, const KVView
                           const GateArgs &gates, const AttnOut &out, const AttnScratch &scratch);
 void attention_gates_tiles_scratch(size_t longest_v_row, size_t *floats, size_t *counters);
 
+// The same on tcgen05 for chunks over page pools that carry the half-tile tensor map (KVView::tma_tile_desc): bf16, K and V rows of 128,
+// at most 32 heads and 16 kv heads, chunks of 8 tokens or more among them. Returns -1 if the view or shape is not covered, or the
+// scratch (as above) is smaller than attention_gates_tc_scratch asks for.
+int attention_gates_tc(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch, const void *q, float scale,
+                       const GateArgs &gates, const AttnOut &out, const AttnScratch &scratch);
+void attention_gates_tc_scratch(size_t *floats, size_t *counters);
+
 // K2 (+ fused K3): split-KV flash decoding for 16-bit K/V, head_dim 128, page size 16, GQA group <= 8,
 // one query per sequence. Returns -1 if the shape is not covered.
 int attention_decode_split(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch,

@@ -136,6 +136,11 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
             kernels::attention_gates_tiles_scratch(longest_v, &floats, &counters);
             _partials_floats = std::max(_partials_floats, floats);
             _counters_len = std::max(_counters_len, counters);
+            if (any_tma) {
+                kernels::attention_gates_tc_scratch(&floats, &counters);
+                _partials_floats = std::max(_partials_floats, floats);
+                _counters_len = std::max(_counters_len, counters);
+            }
         }
         if (_partials_floats != 0) {
             _partials = rt.allocateDeviceStorage(_partials_floats * sizeof(float));
@@ -469,7 +474,12 @@ void PagedKV::requireGates(const AttnOptions &opt) const {
 int PagedKV::runGates(const kernels::KVView &v, const kernels::AttnBatch &b, const void *q, float scale, const kernels::GateArgs &gates,
                       const kernels::AttnOut &o, llaisysStream_t stream) const {
 #ifdef ENABLE_NVIDIA_API
-    int used = LLAISYS_KERNEL_GATES_TILES;
+    int used = LLAISYS_KERNEL_GATES_TC;
+    if (kernels::attention_gates_tc(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch()) == 0) {
+        noteAttentionKernel(used);
+        return used;
+    }
+    used = LLAISYS_KERNEL_GATES_TILES;
     if (kernels::attention_gates_tiles(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch()) != 0) {
         kernels::attention_gates(stream, _cfg.dtype, v, b, q, scale, gates, o, scratch().error_flag);
         used = LLAISYS_KERNEL_GATES;

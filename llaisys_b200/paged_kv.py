@@ -32,6 +32,7 @@ class Kernel(IntEnum):
     PREFILL_TC = 6
     GATES = 7
     GATES_TILES = 8
+    GATES_TC = 9
 
 
 def last_attention_kernel() -> Kernel:
