@@ -37,9 +37,18 @@ namespace {
 
 constexpr int kD = 128, kBk = 128, kPages = kBk / 16;
 constexpr int kWorkers = 16, kProducer = 16, kIssuer = 17, kThreads = 18 * 32;
+constexpr int kChunk = 32; // columns of one kv head that a warp turns into weights at a time
 constexpr int kSlot = kBk * kD * 2, kMaxStages = 6, kMaxColumns = 256, kMaxGroups = 16;
+// What a block costs besides its tiles (queries in, products drained, outputs out), in tiles. The line that is cut into equal shares
+// counts every block as this many units and then its tiles.
+constexpr int kBlockCost = 1;
 constexpr int kSmemLimit = 227 * 1024, kErrTimeout = 8;
 constexpr float kLog2e = 1.4426950408889634f, kWeightUnit = 32768.f;
+
+// A shared-memory descriptor that starts `bytes` further on (the address field counts 16-byte steps and does not overflow).
+__device__ __forceinline__ uint64_t desc_at(uint64_t desc, uint32_t bytes) {
+    return (desc & 0xffffffff00000000ull) | uint32_t(uint32_t(desc) + (bytes >> 4));
+}
 
 struct Params {
     AttnBatch batch;
@@ -61,6 +70,7 @@ struct Block { // a block of queries
     int q0, n_q;        // first query within its chunk, queries
     int pos0, kv_end;   // position of the first query, keys that the last one sees
     int tile0, n_tiles; // key tiles
+    __device__ __forceinline__ int units() const { return n_tiles > 0 ? kBlockCost + n_tiles : 0; }
 };
 
 __device__ __forceinline__ Block block_of(const Params &p, int q_len, int kv_len, int index) {
@@ -74,9 +84,9 @@ __device__ __forceinline__ Block block_of(const Params &p, int q_len, int kv_len
     return o;
 }
 
-// A CTA's walk over its share of the line: every role walks the same fragments.
+// A CTA's walk over its share [at, end) of the line: every role walks the same fragments.
 struct Walk {
-    int at, end, seq, index, block_begin;
+    int at, end, seq, index, block_begin; // (at: kept within the block at `index`)
 };
 struct Fragment {
     Block block;
@@ -89,17 +99,17 @@ __device__ __forceinline__ bool next_fragment(const Params &p, Walk &w, Fragment
         f.block = block_of(p, q_len, p.batch.kv_lens[w.seq], w.index);
         f.seq = w.seq;
         f.block_begin = w.block_begin;
-        f.from = w.at - w.block_begin;
-        f.upto = min(f.block.n_tiles, w.end - w.block_begin);
+        f.from = max(0, w.at - w.block_begin - kBlockCost);
+        f.upto = min(f.block.n_tiles, w.end - w.block_begin - kBlockCost);
         f.row0 = first + f.block.q0;
-        w.block_begin += f.block.n_tiles;
+        w.block_begin += f.block.units();
+        w.at = max(w.at, w.block_begin);
         w.index += 1;
         if (w.index * p.bq >= q_len) {
             w.index = 0;
             w.seq += 1;
         }
         if (f.upto > f.from) {
-            w.at += f.upto - f.from;
             return true;
         }
     }
@@ -127,19 +137,50 @@ __device__ __forceinline__ float rcp(float x) {
     asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
 }
-// unit / x_i + c_i for four numbers in [1, 2^31 + 1] with one reciprocal
-__device__ __forceinline__ void rcp4(float *x, float unit, const float *c) {
-    const float p01 = x[0] * x[1], p23 = x[2] * x[3], r = rcp(p01 * p23) * unit, r01 = r * p23, r23 = r * p01;
-    const float y0 = fmaf(r01, x[1], c[0]), y1 = fmaf(r01, x[0], c[1]), y2 = fmaf(r23, x[3], c[2]), y3 = fmaf(r23, x[2], c[3]);
-    x[0] = y0;
-    x[1] = y1;
-    x[2] = y2;
-    x[3] = y3;
+// Pairs of f32 in one register pair: two of these operations go out as one instruction.
+using Pair = unsigned long long;
+__device__ __forceinline__ Pair pair(float x, float y) {
+    Pair p;
+    asm("mov.b64 %0, {%1, %2};\n" : "=l"(p) : "f"(x), "f"(y));
+    return p;
 }
+__device__ __forceinline__ void unpair(Pair p, float &x, float &y) { asm("mov.b64 {%0, %1}, %2;\n" : "=f"(x), "=f"(y) : "l"(p)); }
+__device__ __forceinline__ Pair mul2(Pair a, Pair b) {
+    Pair d;
+    asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ Pair add2(Pair a, Pair b) {
+    Pair d;
+    asm("add.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ Pair fma2(Pair a, Pair b, Pair c) {
+    Pair d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+// 1 + 2^min(x, 31), element by element
+__device__ __forceinline__ Pair one_plus_ex2(Pair x, Pair ones) {
+    float a, b;
+    unpair(x, a, b);
+    return add2(ones, pair(ex2(fminf(a, 31.f)), ex2(fminf(b, 31.f))));
+}
+// (unit / the four numbers of x and y), which lie in [1, 2^31 + 1], with one reciprocal: p times y is for x, p times x for y
+__device__ __forceinline__ Pair rcp4(Pair x, Pair y, float unit) {
+    float a, b;
+    unpair(mul2(x, y), a, b);
+    const float r = rcp(a * b) * unit;
+    return pair(r * b, r * a);
+}
+// n / d for 0 <= n < 2^15, inv = 1 / d rounded
+__device__ __forceinline__ int small_div(int n, float inv) { return int((float(n) + 0.5f) * inv); }
 __device__ __forceinline__ void store_u16(uint32_t addr, uint32_t v) {
     asm volatile("st.shared.u16 [%0], %1;\n" ::"r"(addr), "h"(static_cast<unsigned short>(v)) : "memory");
 }
-__device__ __forceinline__ void store_u32(uint32_t addr, uint32_t v) { asm volatile("st.shared.u32 [%0], %1;\n" ::"r"(addr), "r"(v) : "memory"); }
+__device__ __forceinline__ void stmatrix_x4(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
+    asm volatile("stmatrix.sync.aligned.m8n8.x4.shared.b16 [%0], {%1, %2, %3, %4};\n" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
+}
 
 // Shared memory: ring | queries | weights (all 1024-byte aligned) | per-column constants | barriers | small words.
 struct Layout {
@@ -158,7 +199,7 @@ struct Layout {
 constexpr int kBarFull = 0;                            // [stages] producer -> issuer: a tile has landed
 constexpr int kBarS = kBarFull + kMaxStages;           // [2][groups] S_c of a tile is written (and its K slot is free)
 constexpr int kBarPV = kBarS + 2 * kMaxGroups;         // [2][groups] O_c has taken a tile (its V slot and P_c are free)
-constexpr int kBarRead = kBarPV + 2 * kMaxGroups;      // [groups] workers -> issuer: S_c has been read
+constexpr int kBarRead = kBarPV + 2 * kMaxGroups;      // [groups] workers -> issuer: S_c has been read (a warp per chunk and quarter)
 constexpr int kBarP = kBarRead + kMaxGroups;           // workers -> issuer: P of a tile is complete
 constexpr int kBarQ = kBarP + 1;                       // workers -> issuer: queries of a fragment are in place
 constexpr int kBarO = kBarQ + 1;                       // workers -> issuer: O has been read
@@ -188,7 +229,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const int q_len = p.batch.q_starts[s + 1] - p.batch.q_starts[s], kv_len = p.batch.kv_lens[s], blocks = (q_len + p.bq - 1) / p.bq;
         int sum = 0;
         for (int b = lane; b < blocks; b += 32) {
-            sum += block_of(p, q_len, kv_len, b).n_tiles;
+            sum += block_of(p, q_len, kv_len, b).units();
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -201,7 +242,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     if (tid == 0) {
         prefix[0] = 0;
         for (int i = 0; i < kBarO + 1; ++i) {
-            mbar_init(bar(i), i >= kBarRead ? kWorkers : 1);
+            mbar_init(bar(i), i < kBarRead ? 1 : (i < kBarP ? 4 * ((n_c + kChunk - 1) / kChunk) : kWorkers));
         }
         misc[0] = misc[1] = misc[2] = misc[3] = 0;
         *s_abort = 0;
@@ -225,7 +266,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         }
     }
     __syncthreads();
-    const int64_t total = prefix[p.batch.n_seqs], ctas = min(int64_t(gridDim.x), total); // (every share holds a tile)
+    const int64_t total = prefix[p.batch.n_seqs], ctas = min(int64_t(gridDim.x), total); // (every share holds a unit)
     grid_dependency_wait(); // (the index arrays above are older than the kernel before this one)
     if (int64_t(blockIdx.x) >= ctas) {
         return;
@@ -245,7 +286,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         walk.block_begin = prefix[lo];
         const int q_len = p.batch.q_starts[lo + 1] - p.batch.q_starts[lo], kv_len = p.batch.kv_lens[lo], blocks = (q_len + p.bq - 1) / p.bq;
         for (int b0 = 0; b0 < blocks; b0 += 32) { // every warp finds the same
-            const int mine = b0 + lane < blocks ? block_of(p, q_len, kv_len, b0 + lane).n_tiles : 0;
+            const int mine = b0 + lane < blocks ? block_of(p, q_len, kv_len, b0 + lane).units() : 0;
             int v = mine;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -267,9 +308,10 @@ __global__ void __launch_bounds__(kThreads, 1)
     for (int i = tid; i < p.stages * kSlot / 16; i += kThreads) {
         reinterpret_cast<uint4 *>(smem)[i] = make_uint4(0, 0, 0, 0);
     }
-    // what a column adds to the exponent of its gate at distance x from the block's first query: columns[].x * x + columns[].y
+    // what a column adds to the exponent of its gate at distance x from the block's first query, a * x + b: for a pair of columns a, a, b, b
     const bool capped = p.gates.softcap > 0.f;
-    float2 *columns = reinterpret_cast<float2 *>(smem + lay.columns);
+    float *columns = reinterpret_cast<float *>(smem + lay.columns);
+    const float inv_share = 1.f / float(share), inv_n_c = 1.f / float(n_c);
     for (int i = tid; i < n_columns; i += kThreads) {
         const int c = i / n_c, r = i - c * n_c, qi = r / share, h = c * share + r - qi * share;
         float2 v = make_float2(0.f, 0.f);
@@ -278,7 +320,8 @@ __global__ void __launch_bounds__(kThreads, 1)
             v.x = p.gates.slopes != nullptr ? kLog2e * p.gates.slopes[h] : 0.f;
             v.y = fmaf(v.x, float(qi), -kLog2e * (b + (capped ? p.gates.softcap : 0.f)));
         }
-        columns[i] = v;
+        columns[i / 2 * 4 + i % 2] = v.x;
+        columns[i / 2 * 4 + i % 2 + 2] = v.y;
     }
     if (warp == kIssuer) {
         tmem_alloc(base + uint32_t(lay.misc + 20), 512);
@@ -375,10 +418,11 @@ __global__ void __launch_bounds__(kThreads, 1)
                     }
                     tc_fence_after();
                     const uint32_t q_s = base + uint32_t(lay.q + c * n_c * kD * 2);
+                    const uint64_t da = smem_desc_sw128(k_s, 0, 1024), db = smem_desc_sw128(q_s, 0, 1024), db2 = desc_at(db, uint32_t(n_c * 128));
 #pragma unroll
                     for (int ks = 0; ks < kD / 16; ++ks) {
-                        umma_f16(tmem + uint32_t(c * n_c), smem_desc_sw128(k_s + (ks >> 2) * (kSlot / 2) + (ks & 3) * 32, 0, 1024),
-                                 smem_desc_sw128(q_s + uint32_t((ks >> 2) * n_c * 128 + (ks & 3) * 32), 0, 1024), idesc_s, ks > 0 ? 1u : 0u);
+                        umma_f16(tmem + uint32_t(c * n_c), desc_at(da, (ks >> 2) * (kSlot / 2) + (ks & 3) * 32),
+                                 desc_at(ks < 4 ? db : db2, (ks & 3) * 32), idesc_s, ks > 0 ? 1u : 0u);
                     }
                     umma_commit(s_bar(tile_no, c));
                 }
@@ -403,10 +447,11 @@ __global__ void __launch_bounds__(kThreads, 1)
                         }
                         tc_fence_after();
                         const uint32_t p_s = base + uint32_t(lay.w + c * n_c * kBk * 2);
+                        const uint64_t da = smem_desc_sw128(v_s, 2048, 1024), db = smem_desc_sw128(p_s, 0, 1024),
+                                       db2 = desc_at(db, uint32_t(n_c * 128));
 #pragma unroll
                         for (int kk = 0; kk < kBk / 16; ++kk) { // 16 keys: one page
-                            umma_f16(tmem_o + uint32_t(c * n_c), smem_desc_sw128(v_s + kk * 4096, 2048, 1024),
-                                     smem_desc_sw128(p_s + uint32_t((kk >> 2) * n_c * 128 + (kk & 3) * 32), 0, 1024), idesc_o,
+                            umma_f16(tmem_o + uint32_t(c * n_c), desc_at(da, kk * 4096), desc_at(kk < 4 ? db : db2, (kk & 3) * 32), idesc_o,
                                      i > 0 || kk > 0 ? 1u : 0u);
                         }
                         umma_commit(pv_bar(n, c));
@@ -434,17 +479,18 @@ __global__ void __launch_bounds__(kThreads, 1)
                 mbar_arrive(bar(which));
             }
         };
-        const int quarter = warp & 3, part = warp >> 2, units = n_c / 8; // lanes of TMEM, and which of every four 8-column units
+        const int quarter = warp & 3, part = warp >> 2, units = n_c / 8; // lanes of TMEM, and which of every four chunks or units
         const int key = quarter * 32 + lane;
         const uint32_t lanes = uint32_t(quarter * 32) << 16;
         const float to_exp = capped ? 2.f * kLog2e * p.scale / p.gates.softcap : -kLog2e * p.scale, cap2 = 2.f * kLog2e * p.gates.softcap;
+        const Pair to_exp2 = pair(to_exp, to_exp), ones = pair(1.f, 1.f);
         const uint32_t w_s = base + uint32_t(lay.w);
         // a weight of column r: row r, 16-byte chunk (key / 8) ^ (r mod 8) of the row's 64-key half
         const uint32_t w_key = w_s + uint32_t((quarter >> 1) * n_c * 128 + (((quarter & 1) * 4 + (lane >> 3)) << 4) + (lane & 7) * 2);
 
-        // talk as mma operands, and where heads lie: byte offset of a head's kv head, and its place in the group
+        // talk as mma operands, and the head whose row this lane addresses: byte offset of its kv head, place in the group
         uint32_t talk[MT][MT][4];
-        int in_base[MT], in_at[MT], out_base[MT][2], out_at[MT][2];
+        int head_base[MT], head_at[MT];
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
@@ -463,20 +509,14 @@ __global__ void __launch_bounds__(kThreads, 1)
                     talk[mt][kt][e] = pack2<false>(v[0], v[1]);
                 }
             }
-            const int hi = mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
-            in_base[mt] = hi < nh ? hi / share * n_c * kBk * 2 : -1;
-            in_at[mt] = hi % share;
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                const int ho = mt * 16 + (lane >> 2) + 8 * r;
-                out_base[mt][r] = ho < nh ? ho / share * n_c * kBk * 2 : -1;
-                out_at[mt][r] = ho % share;
-            }
+            const int head = mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+            head_base[mt] = head < nh ? head / share * n_c * kBk * 2 : -1;
+            head_at[mt] = head % share;
         }
 
         auto load_q = [&](const Fragment &f) {
             for (int i = tid; i < n_columns * 16; i += kWorkers * 32) {
-                const int col = i >> 4, cc = i & 15, c = col / n_c, r = col - c * n_c, qi = r / share, h = c * share + r - qi * share;
+                const int col = i >> 4, cc = i & 15, c = small_div(col, inv_n_c), r = col - c * n_c, qi = small_div(r, inv_share), h = c * share + r - qi * share;
                 uint4 v = make_uint4(0, 0, 0, 0);
                 if (qi < f.block.n_q) {
                     v = *reinterpret_cast<const uint4 *>(p.q + ((f.row0 + qi) * nh + h) * kD + cc * 8);
@@ -499,92 +539,124 @@ __global__ void __launch_bounds__(kThreads, 1)
                 const int first = (blk.tile0 + t) * kBk;
                 const bool edge = first + kBk > blk.pos0 + 1 || (p.batch.window > 0 && first + p.batch.window < blk.pos0 + blk.n_q);
                 const float ago0 = float(blk.pos0 - first - key); // from this thread's key to the block's first query
-                for (int c = 0; c < groups; ++c) {
-                    wait(s_bar(n, c), (n >> 1) & 1);
-                    tc_fence_after();
-                    const int shift = (part - c * units) & 3;
-                    bool first_store = true;
-                    for (int u = shift; u < units; u += 4) {
-                        const int col = c * n_c + u * 8;
-                        float x[8], a[8];
-                        tmem_ld8(tmem + lanes + uint32_t(col), x);
-#pragma unroll
-                        for (int i = 0; i < 8; i += 2) {
-                            const float4 k2 = *reinterpret_cast<const float4 *>(columns + col + i);
-                            a[i] = fmaf(k2.x, ago0, k2.y);
-                            a[i + 1] = fmaf(k2.z, ago0, k2.w);
+                const Pair ago2 = pair(ago0, ago0);
+                const int chunks = (n_c + kChunk - 1) / kChunk;
+                for (int c = 0, k = 0; c < groups; ++c) {
+                    for (int piece = 0; piece < chunks; ++piece, ++k) {
+                        if ((k & 3) != part) {
+                            continue;
                         }
-                        if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
-#pragma unroll
-                            for (int i = 0; i < 8; ++i) {
-                                x[i] = 1.f + ex2(fminf(x[i] * to_exp, 31.f));
-                            }
-                            rcp4(x, cap2, a);
-                            rcp4(x + 4, cap2, a + 4);
-                        } else {
-#pragma unroll
-                            for (int i = 0; i < 8; ++i) {
-                                x[i] = fmaf(x[i], to_exp, a[i]);
-                            }
-                        }
-                        const float zero[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-                        for (int i = 0; i < 8; ++i) {
-                            x[i] = 1.f + ex2(fminf(x[i], 31.f));
-                        }
-                        rcp4(x, kWeightUnit, zero);
-                        rcp4(x + 4, kWeightUnit, zero);
-                        if (edge) {
-                            const float window = p.batch.window > 0 ? float(p.batch.window) : INFINITY;
-#pragma unroll
-                            for (int i = 0; i < 8; ++i) {
-                                const float ago = ago0 + float((u * 8 + i) / share);
-                                x[i] = ago >= 0.f && ago < window ? x[i] : 0.f;
-                            }
-                        }
-                        if (first_store && n > 0) {
+                        const int col0 = c * n_c + piece * kChunk, n_units = min(kChunk, n_c - piece * kChunk) / 8;
+                        wait(s_bar(n, c), (n >> 1) & 1);
+                        tc_fence_after();
+                        uint32_t raw[kChunk]; // (columns past the chunk are S or O columns all the same, and go unused)
+                        tmem_ld32_nowait(tmem + lanes + uint32_t(col0), raw);
+                        tmem_wait_ld();
+                        tc_fence_before();
+                        arrive(kBarRead + c);
+                        if (n > 0) {
                             wait(pv_bar(n - 1, c), ((n - 1) >> 1) & 1);
                         }
-                        first_store = false;
-                        const uint32_t at = w_key + uint32_t(c * n_c * kBk * 2 + u * 8 * 128);
+                        uint32_t at[8];
 #pragma unroll
-                        for (int i = 0; i < 8; i += 2) {
-                            const uint32_t two = pack2<false>(x[i], x[i + 1]);
-                            store_u16((at ^ uint32_t(i << 4)) + uint32_t(i * 128), two);
-                            store_u16((at ^ uint32_t((i + 1) << 4)) + uint32_t((i + 1) * 128), two >> 16);
+                        for (int i = 0; i < 8; ++i) {
+                            at[i] = (w_key ^ uint32_t(i << 4)) + uint32_t(c * n_c * kBk * 2 + piece * kChunk * 128 + i * 128);
+                        }
+#pragma unroll
+                        for (int u = 0; u < kChunk / 8; ++u) {
+                            if (u >= n_units) {
+                                break;
+                            }
+                            Pair x[4], a[4];
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) {
+                                const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(columns + 2 * (col0 + u * 8) + 4 * i);
+                                a[i] = fma2(k2.x, ago2, k2.y);
+                                x[i] = pair(__uint_as_float(raw[u * 8 + 2 * i]), __uint_as_float(raw[u * 8 + 2 * i + 1]));
+                            }
+                            if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
+#pragma unroll
+                                for (int i = 0; i < 4; ++i) {
+                                    x[i] = one_plus_ex2(mul2(x[i], to_exp2), ones);
+                                }
+#pragma unroll
+                                for (int i = 0; i < 4; i += 2) {
+                                    const Pair r = rcp4(x[i], x[i + 1], cap2), first = fma2(r, x[i + 1], a[i]);
+                                    x[i + 1] = fma2(r, x[i], a[i + 1]);
+                                    x[i] = first;
+                                }
+                            } else {
+#pragma unroll
+                                for (int i = 0; i < 4; ++i) {
+                                    x[i] = fma2(x[i], to_exp2, a[i]);
+                                }
+                            }
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) {
+                                x[i] = one_plus_ex2(x[i], ones);
+                            }
+                            float w[8];
+#pragma unroll
+                            for (int i = 0; i < 4; i += 2) {
+                                const Pair r = rcp4(x[i], x[i + 1], kWeightUnit);
+                                unpair(mul2(r, x[i + 1]), w[2 * i], w[2 * i + 1]);
+                                unpair(mul2(r, x[i]), w[2 * i + 2], w[2 * i + 3]);
+                            }
+                            if (edge) {
+                                const float window = p.batch.window > 0 ? float(p.batch.window) : INFINITY;
+#pragma unroll
+                                for (int i = 0; i < 8; ++i) {
+                                    const float ago = ago0 + float(small_div(piece * kChunk + u * 8 + i, inv_share));
+                                    w[i] = ago >= 0.f && ago < window ? w[i] : 0.f;
+                                }
+                            }
+#pragma unroll
+                            for (int i = 0; i < 8; i += 2) {
+                                const uint32_t two = pack2<false>(w[i], w[i + 1]);
+                                store_u16(at[i] + uint32_t(u * 1024), two);
+                                store_u16(at[i + 1] + uint32_t(u * 1024), two >> 16);
+                            }
                         }
                     }
-                    tc_fence_before();
-                    arrive(kBarRead + c);
                 }
                 named_barrier_sync(1, kWorkers * 32); // weights of all heads are in place
-                for (int item = warp; item < blk.n_q * kPages; item += kWorkers) {
-                    const int qi = item / kPages, kb = item % kPages, q_row = qi * share;
-                    const int half = (kb >> 2) * n_c * 128, chunk = (kb & 3) * 2;
-                    uint32_t in[MT][4];
+                constexpr int kAtOnce = MT == 1 ? 4 : 2;
+                // a warp per query and half of the keys: 16 keys of all heads at a time, results in place of the operands
+                for (int item = warp; item < blk.n_q * 2; item += kWorkers) {
+                    const int half = (item & 1) * n_c * 128, q_row = (item >> 1) * share;
+                    uint32_t row_at[MT];
 #pragma unroll
                     for (int kt = 0; kt < MT; ++kt) {
-                        const int row = q_row + in_at[kt];
-                        const uint32_t at = in_base[kt] < 0 ? base + uint32_t(lay.misc)
-                                                            : w_s + uint32_t(in_base[kt] + half + row * 128 + (((chunk + (lane >> 4)) ^ (row & 7)) << 4));
-                        ldmatrix_x4_trans(in[kt], at);
+                        const int row = q_row + head_at[kt];
+                        row_at[kt] = w_s + uint32_t(head_base[kt] + half + row * 128 + (((lane >> 4) ^ (row & 7)) << 4));
                     }
-                    __syncwarp();
 #pragma unroll
-                    for (int mt = 0; mt < MT; ++mt) {
-                        float y0[4] = {0.f, 0.f, 0.f, 0.f}, y1[4] = {0.f, 0.f, 0.f, 0.f};
+                    for (int kb0 = 0; kb0 < 4; kb0 += kAtOnce) {
+                        uint32_t in[kAtOnce][MT][4], at[kAtOnce][MT];
 #pragma unroll
-                        for (int kt = 0; kt < MT; ++kt) {
-                            mma_f16(y0, talk[mt][kt], in[kt][0], in[kt][1]);
-                            mma_f16(y1, talk[mt][kt], in[kt][2], in[kt][3]);
+                        for (int b = 0; b < kAtOnce; ++b) {
+#pragma unroll
+                            for (int kt = 0; kt < MT; ++kt) {
+                                at[b][kt] = head_base[kt] < 0 ? base + uint32_t(lay.misc) : row_at[kt] ^ uint32_t((kb0 + b) << 5);
+                                ldmatrix_x4_trans(in[b][kt], at[b][kt]);
+                            }
                         }
+                        __syncwarp();
 #pragma unroll
-                        for (int r = 0; r < 2; ++r) {
-                            if (out_base[mt][r] >= 0) {
-                                const int row = q_row + out_at[mt][r];
-                                const uint32_t at = w_s + uint32_t(out_base[mt][r] + half + row * 128 + ((chunk ^ (row & 7)) << 4) + (lane & 3) * 4);
-                                store_u32(at, pack2<true>(y0[2 * r], y0[2 * r + 1]));
-                                store_u32(at ^ 16u, pack2<true>(y1[2 * r], y1[2 * r + 1])); // (chunk is even)
+                        for (int mt = 0; mt < MT; ++mt) {
+                            float y[kAtOnce][2][4] = {}; // [16 keys][8 of them]
+#pragma unroll
+                            for (int kt = 0; kt < MT; ++kt) {
+#pragma unroll
+                                for (int b = 0; b < kAtOnce; ++b) {
+                                    mma_f16(y[b][0], talk[mt][kt], in[b][kt][0], in[b][kt][1]);
+                                    mma_f16(y[b][1], talk[mt][kt], in[b][kt][2], in[b][kt][3]);
+                                }
+                            }
+#pragma unroll
+                            for (int b = 0; b < kAtOnce; ++b) { // (rows of padding heads: zeros, to where zeros lie)
+                                stmatrix_x4(at[b][mt], pack2<true>(y[b][0][0], y[b][0][1]), pack2<true>(y[b][0][2], y[b][0][3]),
+                                            pack2<true>(y[b][1][0], y[b][1][1]), pack2<true>(y[b][1][2], y[b][1][3]));
                             }
                         }
                     }
@@ -608,11 +680,19 @@ __global__ void __launch_bounds__(kThreads, 1)
                 }
             };
             auto store = [&](int col, const float (&v)[8]) {
+                const int c = small_div(col, inv_n_c), r = col - c * n_c;
+                int qi = small_div(r, inv_share), hl = r - qi * share;
+                __nv_bfloat16 *dst = p.out + (f.row0 + qi) * p.out_stride + int64_t(c * share + hl) * kD + key;
 #pragma unroll
                 for (int i = 0; i < 8; ++i) {
-                    const int c = (col + i) / n_c, r = col + i - c * n_c, qi = r / share, h = c * share + r - qi * share;
                     if (qi < blk.n_q) {
-                        p.out[(f.row0 + qi) * p.out_stride + int64_t(h) * kD + key] = __float2bfloat16_rn(v[i] * (1.f / kWeightUnit));
+                        *dst = __float2bfloat16_rn(v[i] * (1.f / kWeightUnit));
+                    }
+                    dst += kD;
+                    if (++hl == share) { // the next query's first head of the group
+                        hl = 0;
+                        ++qi;
+                        dst += p.out_stride - int64_t(share) * kD;
                     }
                 }
             };
@@ -636,9 +716,9 @@ __global__ void __launch_bounds__(kThreads, 1)
                 });
                 tc_fence_before();
                 arrive(kBarO);
-                // CTAs whose shares touch the block: share c holds tile t iff c is the largest with c * total < (t + 1) * ctas
-                const int first_cta = int(((int64_t(f.block_begin) + 1) * ctas - 1) / total);
-                const int last_cta = int((int64_t(f.block_begin + blk.n_tiles) * ctas - 1) / total);
+                // CTAs that hold tiles of the block: share c holds unit u iff c is the largest with c * total < (u + 1) * ctas
+                const int64_t unit0 = f.block_begin + kBlockCost;
+                const int first_cta = int(((unit0 + 1) * ctas - 1) / total), last_cta = int(((unit0 + blk.n_tiles) * ctas - 1) / total);
                 __threadfence();
                 named_barrier_sync(1, kWorkers * 32);
                 if (tid == 0) {
