@@ -381,12 +381,15 @@ class Kernels:
         copies = copies if rows * width * 6 < 30e6 else 3
         proj = [self.rand(rows, 3 * width) for _ in range(copies)]
         state = [torch.zeros(len(lens), width, device="cuda") for _ in range(copies)]
+        n_scratch = ll.min_gru_scratch_floats(rows, width)
+        scratch = torch.empty(n_scratch, device="cuda")
         bz, bx, out = self.rand(width), self.rand(width), [self.rand(rows, width) for _ in range(copies)]
         ids, starts, kv = self.i32(list(range(len(lens)))), self.i32([0, *np.cumsum(lens).tolist()]), self.i32([x + 100 for x in lens])
         us = self.time(lambda i: ll.min_gru_dev(
             ll.DataType.BF16, decode=max(lens) == 1, stream=self.cs, proj=proj[i % copies], row_stride=3 * width, z_at=0, x_at=width,
             g_at=2 * width, bias_z=bz, bias_x=bx, width=width, state=state[i % copies], slot_stride=width, seq_ids_dev=ids,
-            q_starts_dev=starts, kv_lens_dev=kv, n_seqs=len(lens), n_rows=rows, max_q_len=max(lens), out=out[i % copies], out_stride=width))
+            q_starts_dev=starts, kv_lens_dev=kv, n_seqs=len(lens), n_rows=rows, max_q_len=max(lens), out=out[i % copies], out_stride=width,
+            scratch=scratch, scratch_floats=n_scratch))
         return self.memory(us, rows * 4 * width * 2 + 2 * len(lens) * width * 4)
 
     def gated_linear(self, heads: int, lens: list[int], rank: int = 16, copies: int = 3) -> dict:

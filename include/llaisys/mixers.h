@@ -78,7 +78,8 @@ LLAISYS_API int llaisysPagedAttentionGatesDev(llaisysPagedKV_t kv, size_t layer,
 /* minGRU, element by element over `width` channels: with z_t = sigmoid(z + bias_z) and u_t = x + bias_x,
  *     S_t = (1 - z_t) S_{t-1} + z_t g(u_t),   g(u) = u + 1/2 for u >= 0, sigmoid(u) below;   out_t = S_t silu(g)
  * z, x and g are `width` elements each at z_at, x_at and g_at of a projection row; biases [width] of `dtype`; the state [width] f32
- * of slot s at state + s * slot_stride. Sequences, rows, slots and `decode` as for LlaisysGatedLinear. */
+ * of slot s at state + s * slot_stride. Sequences, rows, slots and `decode` as for LlaisysGatedLinear. Runs of more than 128 tokens
+ * need the scratch (llaisysMinGruScratchFloats floats). */
 struct LlaisysMinGru {
     const void *proj;
     int64_t row_stride, z_at, x_at, g_at;
@@ -90,7 +91,10 @@ struct LlaisysMinGru {
     size_t n_seqs, n_rows, max_q_len;
     void *out;
     int64_t out_stride;
+    float *scratch;
+    size_t scratch_floats;
 };
+LLAISYS_API size_t llaisysMinGruScratchFloats(size_t n_rows, size_t width);
 LLAISYS_API int llaisysMinGruDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype, const struct LlaisysMinGru *args,
                                  int decode, llaisysStream_t stream);
 

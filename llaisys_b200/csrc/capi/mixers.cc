@@ -123,6 +123,15 @@ int llaisysPagedAttentionGatesDev(llaisysPagedKV_t kv, size_t layer, void *out, 
     });
 }
 
+size_t llaisysMinGruScratchFloats(size_t n_rows, size_t width) {
+#ifdef ENABLE_NVIDIA_API
+    return llaisys::kernels::min_gru_scratch_floats(n_rows, width);
+#else
+    (void)n_rows, (void)width;
+    return 0;
+#endif
+}
+
 int llaisysMinGruDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype, const LlaisysMinGru *a, int decode,
                      llaisysStream_t stream) {
     if (a == nullptr || a->proj == nullptr || a->bias_z == nullptr || a->bias_x == nullptr || a->state == nullptr ||
@@ -155,6 +164,8 @@ int llaisysMinGruDev(llaisysDeviceType_t device_type, int device_id, llaisysData
         g.max_q_len = int32_t(a->max_q_len);
         g.out = a->out;
         g.out_stride = a->out_stride;
+        g.scratch = a->scratch;
+        g.scratch_floats = a->scratch_floats;
         if (decode != 0) {
             llaisys::kernels::min_gru_decode(stream, dtype, g);
         } else {

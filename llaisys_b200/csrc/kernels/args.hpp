@@ -227,6 +227,8 @@ struct MinGruArgs {
     int32_t n_seqs = 0, n_rows = 0, max_q_len = 0;
     void *out = nullptr; // row r: out + r * out_stride, model dtype
     int64_t out_stride = 0;
+    float *scratch = nullptr; // min_gru_scratch_floats, for runs of more than 128 tokens
+    size_t scratch_floats = 0;
 };
 
 using stream_t = void *;

@@ -99,9 +99,10 @@ size_t gated_delta_state_floats(size_t heads, size_t kv_heads, size_t dk, size_t
 size_t gated_delta_scratch_floats(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t kv_heads, size_t dk, size_t dv);
 size_t gated_delta_segment_floats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
 
-// minGRU (see MinGruArgs). decode: one token per sequence. chunk: ragged runs of tokens, one pass over their rows.
+// minGRU (see MinGruArgs). decode: one token per sequence. chunk: ragged runs of tokens.
 void min_gru_decode(stream_t stream, llaisysDataType_t dtype, const MinGruArgs &args);
 void min_gru_chunk(stream_t stream, llaisysDataType_t dtype, const MinGruArgs &args);
+size_t min_gru_scratch_floats(size_t n_rows, size_t width); // of MinGruArgs::scratch
 
 // Gated linear attention (see GatedLinearArgs). decode: one token per sequence, everything in one launch. chunk: ragged
 // runs of tokens.

@@ -1,25 +1,20 @@
 // minGRU (MinGruArgs): a gated recurrence per channel whose gates read the current token only, so a run of tokens is a chain of
 // affine maps S -> a S + b that compose in any grouping.
 //
-// Roofline: HBM (three projections read, one activation written, per token and channel). Decode: a thread per (sequence, VEC
-// channels). Runs: one pass over the rows. A cluster of up to 8 CTAs owns a slice of 8 x VEC channels of one sequence and walks
-// its tokens in tiles of 256 per CTA; a thread holds 8 tokens x VEC channels in registers, composes them, the CTA scans its 32
-// groups of tokens with shuffles, and the CTAs of the cluster hand their totals to one another through distributed shared memory.
-// State and gates are f32.
+// Roofline: HBM (three projections read, one activation written, per token and channel); six multi-function operations per element
+// come close to it. Decode: a thread per (sequence, VEC channels). Runs are cut into segments of 128 tokens, a thread per segment and
+// VEC channels: one launch composes the maps of every segment but a sequence's last into (a, b), a second starts each segment from
+// the state that those before it leave and writes the outputs. Runs of one segment take the second launch only. State and gates are
+// f32.
 #include "gated_linear.cuh"
 #include "kernels.hpp"
 #include "mma_utils.cuh"
-
-#include <cooperative_groups.h>
-
-namespace cg = cooperative_groups;
 
 namespace llaisys::kernels {
 
 namespace {
 
-constexpr int kThreads = 256, kLanes = 8 /* threads side by side over channels */, kGroups = kThreads / kLanes, kTokens = 8;
-constexpr int kTile = kGroups * kTokens, kMaxCluster = 8;
+constexpr int kThreads = 128, kSegment = 128, kAhead = 8;
 
 // 1 / (1 + e^-x); the 16-bit forms divide and exponentiate with the fast approximations (relative error near 2^-21)
 template <typename T>
@@ -69,126 +64,119 @@ __global__ void min_gru_decode_kernel(MinGruArgs a) {
     *reinterpret_cast<P *>(static_cast<T *>(a.out) + int64_t(seq) * a.out_stride + c) = o;
 }
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(kThreads, 2) min_gru_chunk_kernel(MinGruArgs a) {
+// Where the composed maps of a sequence lie in the scratch, [entry][width][2]. Only segments with one behind them have an entry, so
+// these are whole, and sequences' entries do not overlap. A sequence's first entry holds (state before the run, state after it).
+__device__ __forceinline__ float *first_entry(const MinGruArgs &a, int row0) { return a.scratch + int64_t(row0 / kSegment) * a.width * 2; }
+
+// OUT false: composes; true: outputs.
+template <typename T, int VEC, bool OUT>
+__global__ void __launch_bounds__(kThreads) min_gru_segment_kernel(MinGruArgs a) {
     grid_dependency_wait();
     grid_launch_dependents();
-    constexpr int kChannels = kLanes * VEC;
     using P = Pieces<T, VEC>;
-    __shared__ float s_a[kChannels][kGroups + 1], s_b[kChannels][kGroups + 1]; // a tile's groups, then what comes before each
-    __shared__ float s_all[2][kMaxCluster][2][kChannels];                      // [parity][CTA][a | b]: tile totals
-    const cg::cluster_group cluster = cg::this_cluster();
-    const int n_ctas = int(cluster.num_blocks()), rank = int(cluster.block_rank());
-    const int seq = blockIdx.y, slice = int(blockIdx.x) / n_ctas;
-    const int group = int(threadIdx.x) / kLanes, lc = int(threadIdx.x) % kLanes * VEC, c = slice * kChannels + lc;
-    const int warp = int(threadIdx.x) >> 5, lane = int(threadIdx.x) & 31;
-    const int64_t row0 = a.q_starts[seq];
-    const int len = a.q_starts[seq + 1] - int(row0);
-    const bool holds = c < a.width; // (VEC divides the width)
-    float *state = a.state + int64_t(a.seq_ids[seq]) * a.slot_stride + c;
-    float carry[VEC], bz[VEC], bx[VEC];
+    using S = Pieces<float, VEC>;
+    using M = Pieces<float, 2 * VEC>; // (a, b) of each channel
+    const int seq = blockIdx.z, segment = blockIdx.y, c = (int(blockIdx.x) * kThreads + int(threadIdx.x)) * VEC;
+    const int row0 = a.q_starts[seq], len = a.q_starts[seq + 1] - row0, t0 = segment * kSegment, n = min(kSegment, len - t0);
+    const bool last = t0 + kSegment >= len;
+    if (c >= a.width || n <= 0 || (!OUT && last)) {
+        return;
+    }
+    S *state = reinterpret_cast<S *>(a.state + int64_t(a.seq_ids[seq]) * a.slot_stride + c);
+    float *entry = first_entry(a, row0) + int64_t(c) * 2;
+    const int64_t entry_stride = int64_t(a.width) * 2;
+    const P bz = *reinterpret_cast<const P *>(static_cast<const T *>(a.bias_z) + c), bx = *reinterpret_cast<const P *>(static_cast<const T *>(a.bias_x) + c);
+    S s{}, whole; // the state (OUT, and a first segment), or b of the segment so far; a of the segment so far
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-        carry[e] = holds && a.kv_lens[seq] > len ? state[e] : 0.f;
-        bz[e] = holds ? to_f32(static_cast<const T *>(a.bias_z)[c + e]) : 0.f;
-        bx[e] = holds ? to_f32(static_cast<const T *>(a.bias_x)[c + e]) : 0.f;
+        whole.v[e] = 1.f;
     }
-    const T *proj = static_cast<const T *>(a.proj) + row0 * a.row_stride + c;
-    T *out = static_cast<T *>(a.out) + row0 * a.out_stride + c;
-    int parity = 0;
-    for (int base = 0; base < len; base += kTile * n_ctas, parity ^= 1) {
-        const int t0 = base + rank * kTile + group * kTokens;
-        P z[kTokens], u[kTokens], g[kTokens];
-#pragma unroll
-        for (int i = 0; i < kTokens; ++i) {
-            if (holds && t0 + i < len) {
-                const T *row = proj + int64_t(t0 + i) * a.row_stride;
-                z[i] = *reinterpret_cast<const P *>(row + a.z_at);
-                u[i] = *reinterpret_cast<const P *>(row + a.x_at);
-                g[i] = *reinterpret_cast<const P *>(row + a.g_at);
-            }
+    S before{};
+    if (segment == 0 && (!OUT || last)) {
+        if (a.kv_lens[seq] > len) {
+            s = *state;
         }
-        float keep[kTokens][VEC], add[kTokens][VEC];
+        before = s;
+    } else if (OUT) {
+        const M first = *reinterpret_cast<const M *>(entry);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            float ta = 1.f, tb = 0.f;
-#pragma unroll
-            for (int i = 0; i < kTokens; ++i) {
-                keep[i][e] = 1.f;
-                add[i][e] = 0.f;
-                if (holds && t0 + i < len) {
-                    affine<T>(to_f32(z[i].v[e]) + bz[e], to_f32(u[i].v[e]) + bx[e], keep[i][e], add[i][e]);
-                }
-                ta *= keep[i][e];
-                tb = fmaf(keep[i][e], tb, add[i][e]);
-            }
-            s_a[lc + e][group] = ta;
-            s_b[lc + e][group] = tb;
+            s.v[e] = segment == 0 ? first.v[2 * e] : first.v[2 * e + 1];
         }
-        __syncthreads();
+#pragma unroll 8
+        for (int k = 1; k < segment; ++k) {
+            const M m = *reinterpret_cast<const M *>(entry + k * entry_stride);
 #pragma unroll
-        for (int w = 0; w < kChannels / 8; ++w) { // a warp scans a channel's 32 groups
-            const int ch = warp + 8 * w;
-            float pa = s_a[ch][lane], pb = s_b[ch][lane];
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float qa = __shfl_up_sync(0xffffffffu, pa, o), qb = __shfl_up_sync(0xffffffffu, pb, o);
-                if (lane >= o) {
-                    pb = fmaf(pa, qb, pb);
-                    pa *= qa;
-                }
-            }
-            const float xa = __shfl_up_sync(0xffffffffu, pa, 1), xb = __shfl_up_sync(0xffffffffu, pb, 1);
-            s_a[ch][lane] = lane == 0 ? 1.f : xa;
-            s_b[ch][lane] = lane == 0 ? 0.f : xb;
-            const float all_a = __shfl_sync(0xffffffffu, pa, 31), all_b = __shfl_sync(0xffffffffu, pb, 31);
-            if (lane < n_ctas) {
-                float *slot = cluster.map_shared_rank(&s_all[parity][rank][0][ch], unsigned(lane));
-                slot[0] = all_a;
-                slot[kChannels] = all_b;
-            }
-        }
-        cluster.sync(); // (the other parity's slots have been read by every CTA before it arrives here)
-        P o[kTokens];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            float s = carry[e];
-            for (int r = 0; r < n_ctas; ++r) {
-                if (r == rank) {
-                    s = carry[e];
-                }
-                carry[e] = fmaf(s_all[parity][r][0][lc + e], carry[e], s_all[parity][r][1][lc + e]);
-            }
-            s = fmaf(s_a[lc + e][group], s, s_b[lc + e][group]);
-#pragma unroll
-            for (int i = 0; i < kTokens; ++i) {
-                s = fmaf(keep[i][e], s, add[i][e]);
-                const float gv = to_f32(g[i].v[e]);
-                o[i].v[e] = from_f32<T>(s * gv * sigmoid<T>(gv));
-            }
-        }
-        __syncthreads(); // s_a, s_b have been read
-#pragma unroll
-        for (int i = 0; i < kTokens; ++i) {
-            if (holds && t0 + i < len) {
-                *reinterpret_cast<P *>(out + int64_t(t0 + i) * a.out_stride) = o[i];
+            for (int e = 0; e < VEC; ++e) {
+                s.v[e] = fmaf(m.v[2 * e], s.v[e], m.v[2 * e + 1]);
             }
         }
     }
-    if (holds && rank == 0 && group == 0 && len > 0) {
+    const T *row = static_cast<const T *>(a.proj) + int64_t(row0 + t0) * a.row_stride + c;
+    T *out = static_cast<T *>(a.out) + int64_t(row0 + t0) * a.out_stride + c;
+    struct Group {
+        P z[kAhead], u[kAhead], g[OUT ? kAhead : 1];
+    };
+    auto load = [&](Group &x, int t) {
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            if (t + i < n) {
+                const T *at = row + int64_t(t + i) * a.row_stride;
+                x.z[i] = *reinterpret_cast<const P *>(at + a.z_at);
+                x.u[i] = *reinterpret_cast<const P *>(at + a.x_at);
+                if constexpr (OUT) {
+                    x.g[i] = *reinterpret_cast<const P *>(at + a.g_at);
+                }
+            }
+        }
+    };
+    Group now, next;
+    load(now, 0);
+    for (int t = 0; t < n; t += kAhead) {
+        load(next, t + kAhead);
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            if (t + i < n) {
+                P o;
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) {
+                    float keep, add;
+                    affine<T>(to_f32(now.z[i].v[e]) + to_f32(bz.v[e]), to_f32(now.u[i].v[e]) + to_f32(bx.v[e]), keep, add);
+                    s.v[e] = fmaf(keep, s.v[e], add);
+                    if constexpr (OUT) {
+                        const float gv = to_f32(now.g[i].v[e]);
+                        o.v[e] = from_f32<T>(s.v[e] * gv * sigmoid<T>(gv));
+                    } else {
+                        whole.v[e] *= keep;
+                    }
+                }
+                if constexpr (OUT) {
+                    *reinterpret_cast<P *>(out + int64_t(t + i) * a.out_stride) = o;
+                }
+            }
+        }
+        now = next;
+    }
+    if constexpr (OUT) {
+        if (last) {
+            *state = s;
+        }
+    } else {
+        M m;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            state[e] = carry[e];
+            m.v[2 * e] = segment == 0 ? before.v[e] : whole.v[e];
+            m.v[2 * e + 1] = s.v[e];
         }
+        *reinterpret_cast<M *>(entry + segment * entry_stride) = m;
     }
-    cluster.sync(); // no CTA leaves while another may still write into its shared memory
 }
 
-bool vec4_fits(const MinGruArgs &a) {
+bool vec_fits(const MinGruArgs &a, int vec) {
     auto aligned = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-    return a.width % 4 == 0 && a.row_stride % 4 == 0 && a.z_at % 4 == 0 && a.x_at % 4 == 0 && a.g_at % 4 == 0 && a.out_stride % 4 == 0 &&
-           a.slot_stride % 4 == 0 && aligned(a.proj) && aligned(a.bias_z) && aligned(a.bias_x) && aligned(a.state) &&
-           reinterpret_cast<uintptr_t>(a.out) % 16 == 0;
+    return a.width % vec == 0 && a.row_stride % vec == 0 && a.z_at % vec == 0 && a.x_at % vec == 0 && a.g_at % vec == 0 &&
+           a.out_stride % vec == 0 && a.slot_stride % vec == 0 && aligned(a.proj) && aligned(a.bias_z) && aligned(a.bias_x) &&
+           aligned(a.state) && aligned(a.out) && aligned(a.scratch);
 }
 
 template <typename F>
@@ -215,7 +203,7 @@ void min_gru_decode(stream_t stream, llaisysDataType_t dtype, const MinGruArgs &
         return;
     }
     CHECK_ARGUMENT(a.n_seqs <= 65535, "minGRU: too many sequences for one launch");
-    const bool wide = vec4_fits(a);
+    const bool wide = vec_fits(a, 4);
     const int pieces = wide ? a.width / 4 : a.width, block = pieces >= 1024 ? 128 : 64;
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(unsigned((pieces + block - 1) / block), unsigned(a.n_seqs));
@@ -237,32 +225,33 @@ void min_gru_chunk(stream_t stream, llaisysDataType_t dtype, const MinGruArgs &a
     if (a.n_seqs <= 0 || a.width <= 0 || a.max_q_len <= 0) {
         return;
     }
-    CHECK_ARGUMENT(a.n_seqs <= 65535, "minGRU: too many sequences for one launch");
-    const bool wide = vec4_fits(a);
-    const int channels = kLanes * (wide ? 4 : 1), slices = (a.width + channels - 1) / channels;
-    // enough CTAs to fill the GPU twice, as far as the longest run has tiles for them
-    int cluster = 1;
-    while (cluster < kMaxCluster && int64_t(slices) * a.n_seqs * cluster < 2 * 148 && cluster * kTile < a.max_q_len) {
-        cluster *= 2;
-    }
+    const int segments = (a.max_q_len + kSegment - 1) / kSegment;
+    CHECK_ARGUMENT(a.n_seqs <= 65535 && segments <= 65535, "minGRU: too many sequences or too long a run for one launch");
+    CHECK_ARGUMENT(segments == 1 || (a.scratch != nullptr && a.scratch_floats >= min_gru_scratch_floats(size_t(a.n_rows), size_t(a.width))),
+                   "minGRU: the scratch is too small");
+    const bool wide = vec_fits(a, 2);
+    const int block = kThreads * (wide ? 2 : 1);
     cudaLaunchConfig_t cfg{};
-    cfg.gridDim = dim3(unsigned(slices * cluster), unsigned(a.n_seqs));
+    cfg.gridDim = dim3(unsigned((a.width + block - 1) / block), unsigned(segments), unsigned(a.n_seqs));
     cfg.blockDim = dim3(kThreads);
     cfg.stream = static_cast<cudaStream_t>(stream);
-    cudaLaunchAttribute attrs[2] = {};
-    attrs[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attrs[0].val.programmaticStreamSerializationAllowed = 1;
-    attrs[1].id = cudaLaunchAttributeClusterDimension;
-    attrs[1].val.clusterDim.x = unsigned(cluster);
-    attrs[1].val.clusterDim.y = 1;
-    attrs[1].val.clusterDim.z = 1;
-    cfg.attrs = attrs;
-    cfg.numAttrs = 2;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = 1;
     dispatch(dtype, [&](auto tag) {
         using T = decltype(tag);
-        LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, wide ? min_gru_chunk_kernel<T, 4> : min_gru_chunk_kernel<T, 1>, MinGruArgs(a)));
+        if (segments > 1) {
+            --cfg.gridDim.y; // (no sequence's last segment is composed)
+            LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, wide ? min_gru_segment_kernel<T, 2, false> : min_gru_segment_kernel<T, 1, false>, MinGruArgs(a)));
+            ++cfg.gridDim.y;
+        }
+        LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, wide ? min_gru_segment_kernel<T, 2, true> : min_gru_segment_kernel<T, 1, true>, MinGruArgs(a)));
     });
     check_launch("min_gru_chunk");
 }
+
+size_t min_gru_scratch_floats(size_t n_rows, size_t width) { return (n_rows / kSegment + 1) * width * 2; }
 
 } // namespace llaisys::kernels

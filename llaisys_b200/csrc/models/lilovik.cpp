@@ -137,11 +137,14 @@ void Lilovik::ensureActivations(size_t n_tokens, size_t n_out) {
     const size_t W = _meta.width;
     if (n_tokens > _ws_tokens) {
         ++_generation;
-        size_t proj = 0, q = 0, mix = 0, ff = 0;
+        size_t proj = 0, q = 0, mix = 0, ff = 0, scratch = 0;
         for (const Layer &l : _layers) {
             proj = std::max({proj, l.n_proj, 2 * l.ff});
             mix = std::max(mix, l.n_mix);
             ff = std::max(ff, l.ff);
+#ifdef ENABLE_NVIDIA_API
+            scratch = std::max(scratch, l.meta.recurrent ? kernels::min_gru_scratch_floats(n_tokens, l.meta.gru_width) : 0);
+#endif
             q = std::max(q, l.meta.recurrent ? 0 : l.meta.attn.heads * l.meta.attn.dim);
         }
         auto block = [&](size_t bytes) { return bytes != 0 ? rt.allocateDeviceStorage(bytes) : core::storage_t{}; };
@@ -152,6 +155,7 @@ void Lilovik::ensureActivations(size_t n_tokens, size_t n_out) {
         _q = block(n_tokens * q * _elem);
         _mix = block(n_tokens * mix * _elem);
         _u = block(n_tokens * ff * _elem);
+        _scratch = block(scratch * sizeof(float));
 #ifdef ENABLE_NVIDIA_API
         // padding columns of the mix buffer meet zero weights: they only have to be finite
         kernels::fill_zero(rt.stream(), _mix->memory(), _mix->size());
@@ -228,6 +232,8 @@ void Lilovik::recurrence(const Layer &l, const StepArrays &a, const StepShape &s
     g.max_q_len = int32_t(s.max_q_len);
     g.out = _mix->memory();
     g.out_stride = int64_t(l.n_mix);
+    g.scratch = reinterpret_cast<float *>(_scratch->memory());
+    g.scratch_floats = _scratch->size() / sizeof(float);
     if (s.decode_only) {
         kernels::min_gru_decode(_stream, _dtype, g);
     } else {

@@ -47,7 +47,7 @@ private:
     std::byte *_embed = nullptr, *_final_norm = nullptr, *_head = nullptr;
     core::storage_t _freq; // f64, of the position vectors
 
-    core::storage_t _x, _y, _h, _proj, _q, _mix, _u, _h_out;
+    core::storage_t _x, _y, _h, _proj, _q, _mix, _u, _scratch, _h_out;
 };
 
 } // namespace llaisys::models

@@ -196,7 +196,8 @@ class LlaisysMinGru(Structure):
     _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("z_at", c_int64), ("x_at", c_int64), ("g_at", c_int64),
                 ("bias_z", c_void_p), ("bias_x", c_void_p), ("width", c_size_t), ("state", c_void_p), ("slot_stride", c_int64),
                 ("seq_ids_dev", c_void_p), ("q_starts_dev", c_void_p), ("kv_lens_dev", c_void_p), ("n_seqs", c_size_t),
-                ("n_rows", c_size_t), ("max_q_len", c_size_t), ("out", c_void_p), ("out_stride", c_int64)]
+                ("n_rows", c_size_t), ("max_q_len", c_size_t), ("out", c_void_p), ("out_stride", c_int64), ("scratch", c_void_p),
+                ("scratch_floats", c_size_t)]
 
 
 class LlaisysGatedDelta(Structure):
@@ -358,6 +359,7 @@ PROTOTYPES: dict[str, tuple] = {
     "llaisysPagedAttentionGatesDev": (c_int, [_KV, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t,
                                               c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, POINTER(LlaisysGates),
                                               c_size_t, llaisysStream_t]),
+    "llaisysMinGruScratchFloats": (c_size_t, [c_size_t, c_size_t]),
     "llaisysMinGruDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysMinGru), c_int, llaisysStream_t]),
     "llaisysRotaryTableDev": (c_int, [llaisysDeviceType_t, c_int, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t,
                                       llaisysStream_t]),

@@ -313,9 +313,14 @@ class PagedKVCache:
 
 def min_gru_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
     """minGRU on device buffers; fields of LlaisysMinGru (include/llaisys/mixers.h), buffers may be tensors."""
-    pointers = {"proj", "bias_z", "bias_x", "state", "seq_ids_dev", "q_starts_dev", "kv_lens_dev", "out"}
+    pointers = {"proj", "bias_z", "bias_x", "state", "seq_ids_dev", "q_starts_dev", "kv_lens_dev", "out", "scratch"}
     args = LlaisysMinGru(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
     _check(LIB_LLAISYS.llaisysMinGruDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
+
+
+def min_gru_scratch_floats(n_rows: int, width: int) -> int:
+    """Size of `scratch` for n_rows rows."""
+    return int(LIB_LLAISYS.llaisysMinGruScratchFloats(n_rows, width))
 
 
 def gated_linear_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:

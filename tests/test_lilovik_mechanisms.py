@@ -227,11 +227,14 @@ class Gru:
         q_lens = [hi[i] - lo[i] for i in live]
         out = torch.full((len(proj), self.pad + 8), 7.0, dtype=self.dtype, device="cuda")
         bz, bx = self.bz.cuda(), self.bx.cuda()
+        floats = llaisys.min_gru_scratch_floats(len(proj), self.width)
+        scratch = torch.full((floats + 8,), 3e3, device="cuda")
         llaisys.min_gru_dev(LL[self.dtype], decode=decode, stream=stream(), proj=proj, row_stride=3 * self.pad, z_at=0, x_at=self.pad,
                             g_at=2 * self.pad, bias_z=bz, bias_x=bx, width=self.width, state=self.state, slot_stride=self.stride,
                             seq_ids_dev=i32([int(self.slots[i]) for i in live]), q_starts_dev=i32([0, *np.cumsum(q_lens).tolist()]),
                             kv_lens_dev=i32([hi[i] for i in live]), n_seqs=len(live), n_rows=len(proj), max_q_len=max(q_lens), out=out,
-                            out_stride=self.pad + 8)
+                            out_stride=self.pad + 8, scratch=scratch, scratch_floats=floats)
+        assert torch.all(scratch[floats:] == 3e3)
         torch.cuda.synchronize()
         assert torch.all(out[:, self.width:] == 7.0)
         parts = out[:, :self.width].cpu().split(q_lens)
@@ -272,10 +275,13 @@ def test_min_gru_whole_and_in_portions(cuda_device, dtype, width, z_bias):
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
 def test_min_gru_long_runs_and_mixed_batches(cuda_device, dtype):
-    """Thousands of tokens over clusters of CTAs, beside single tokens and short runs, and a far write that lasts."""
+    """Thousands of tokens in many segments, beside single tokens and short runs, and a far write that lasts."""
     g = Gru(dtype, 40, [9000, 1, 2, 2049, 300, 4096], z_bias=-2.0)
     got = g.run([0] * 6, g.lens)
     g.check(got)
+    for width, lens in ((10, [127, 128, 129, 255, 256, 257, 1, 385]), (3, [300, 128, 512])):
+        g = Gru(dtype, width, lens, z_bias=-3.0)
+        g.check(g.run([0] * len(lens), lens), lens)
     g = Gru(dtype, 12, [6000], z_bias=-14.0)  # after the first token everything is kept
     g.x[0][0, :12] = 30.0
     g.x[0][0, g.pad:g.pad + 12] = 5.0
