@@ -14,7 +14,7 @@
 //   warps 0-15   read S (lane = key), compute the weights, store them as f16 times 2^15 into the buffer that becomes P; when all heads
 //                are there, mix them IN PLACE: 16 keys of one query, all heads, are read as mma.sync operands, multiplied by the talk
 //                matrix (in registers) and stored as bf16 to the same places
-//   warp 16      TMA of K and V tiles into a ring of 32 KiB slots
+//   warp 16      TMA of K and V tiles into a ring of 32 KiB slots (as warp 17, an elected lane)
 //   warp 17      issues the MMAs (the whole warp walks, an elected lane issues: descriptors then stay in uniform registers, which made
 //                a batch of eight small MMAs 3.7 times as fast as a loop run by one thread): S of tile t + 1 kv head by kv head as the scores of tile t have been read, then O of tile t.
 //                Weights of tile t + 1 go where P_c of tile t was as soon as O_c has taken it.
@@ -50,6 +50,20 @@ constexpr float kLog2e = 1.4426950408889634f, kWeightUnit = 32768.f;
 __device__ __forceinline__ uint64_t desc_at(uint64_t desc, uint32_t bytes) {
     return (desc & 0xffffffff00000000ull) | uint32_t(uint32_t(desc) + (bytes >> 4));
 }
+
+// A cursor over the ring: the next slot, and the parity of its barriers' phases in this round. (No division: the warps that hold one
+// run between busy ones, and every instruction of theirs counts.)
+struct Cursor {
+    int slot = 0;
+    uint32_t parity = 0;
+    __device__ __forceinline__ void next(int stages) {
+        ++slot;
+        if (slot == stages) {
+            slot = 0;
+            parity ^= 1u;
+        }
+    }
+};
 
 struct Params {
     AttnBatch batch;
@@ -201,15 +215,16 @@ struct Layout {
         w = q + n_columns * kD * 2;
         columns = w + n_columns * kBk * 2;
         bars = columns + n_columns * 8;
-        misc = bars + (kMaxStages + 5 * kMaxGroups + 3) * 8;
+        misc = bars + (2 * kMaxStages + 5 * kMaxGroups + 3) * 8;
         misc = (misc + 15) / 16 * 16;
         total = misc + 32; // [0, 16) zeros, then abort flag, TMEM base, `last`
     }
 };
 // barriers
 constexpr int kBarFull = 0;                            // [stages] producer -> issuer: a tile has landed
-constexpr int kBarS = kBarFull + kMaxStages;           // [2][groups] S_c of a tile is written (and its K slot is free)
-constexpr int kBarPV = kBarS + 2 * kMaxGroups;         // [2][groups] O_c has taken a tile (its V slot and P_c are free)
+constexpr int kBarFree = kBarFull + kMaxStages;        // [stages] MMAs -> producer: it has been used
+constexpr int kBarS = kBarFree + kMaxStages;           // [2][groups] S_c of a tile is written
+constexpr int kBarPV = kBarS + 2 * kMaxGroups;         // [2][groups] O_c has taken a tile (P_c is free)
 constexpr int kBarRead = kBarPV + 2 * kMaxGroups;      // [groups] workers -> issuer: S_c has been read (a warp per chunk and quarter)
 constexpr int kBarP = kBarRead + kMaxGroups;           // workers -> issuer: P of a tile is complete
 constexpr int kBarQ = kBarP + 1;                       // workers -> issuer: queries of a fragment are in place
@@ -347,9 +362,8 @@ __global__ void __launch_bounds__(kThreads, 1)
     if (warp == kProducer) {
         // ================================ K and V tiles ==================================================
         bool alive = true;
-        int op = 0, n = 0; // operands loaded, tiles before this fragment
-        uint32_t free_bar[kMaxStages];
-        int free_parity[kMaxStages];
+        Cursor at;
+        bool first_round = true; // nothing has used the slots yet
         Fragment f;
         while (alive && next_fragment(p, walk, f)) {
             const int32_t *table = p.block_table + int64_t(p.batch.seq_ids != nullptr ? p.batch.seq_ids[f.seq] : f.seq) * p.table_stride;
@@ -364,44 +378,49 @@ __global__ void __launch_bounds__(kThreads, 1)
                 return page;
             };
             // the operand of every kv head of one tile
-            auto load = [&](int page, int tile_no, bool is_v) {
-                const int here = __popc(__ballot_sync(0xffffffffu, lane < kPages && page >= 0));
-                const int c3 = int((p.page0 + max(page, 0)) * 2);
-                for (int c = 0; c < groups && alive; ++c, ++op) {
-                    const int slot = op % p.stages;
-                    if (op >= p.stages && !wait_or_abort(free_bar[slot], uint32_t(free_parity[slot]), s_abort)) {
+            auto load = [&](int page, bool is_v) {
+                const int here = __popc(__ballot_sync(0xffffffffu, lane < kPages && page >= 0)); // (the first ones)
+                int c3[kPages];
+#pragma unroll
+                for (int i = 0; i < kPages; ++i) {
+                    c3[i] = int((p.page0 + max(__shfl_sync(0xffffffffu, page, i), 0)) * 2) + (is_v ? 1 : 0);
+                }
+                for (int c = 0; c < groups && alive; ++c) {
+                    if (!first_round && !__all_sync(0xffffffffu, wait_or_abort(bar(kBarFree + at.slot), at.parity ^ 1u, s_abort))) {
                         alive = false;
                         break;
                     }
-                    if (lane == 0) {
-                        mbar_arrive_expect_tx(bar(kBarFull + slot), uint32_t(here) * 4096);
-                    }
-                    __syncwarp();
-                    if (lane < kPages && page >= 0) {
-                        if (is_v) { // one box per page: [half of the dims][16 tokens][128 B]
-                            tma_load_5d(base + uint32_t(slot * kSlot + lane * 4096), &map_v, 0, 0, 0, c, c3 + 1, bar(kBarFull + slot));
-                        } else { // [half of the dims][128 tokens][128 B]
-                            const uint32_t dst = base + uint32_t(slot * kSlot + lane * 2048);
-                            tma_load_4d(dst, &map_k, 0, 0, c, c3, bar(kBarFull + slot));
-                            tma_load_4d(dst + kSlot / 2, &map_k, 64, 0, c, c3, bar(kBarFull + slot));
+                    const uint32_t dst = base + uint32_t(at.slot * kSlot), full = bar(kBarFull + at.slot);
+                    if (elect_one()) {
+                        mbar_arrive_expect_tx(full, uint32_t(here) * 4096);
+#pragma unroll
+                        for (int i = 0; i < kPages; ++i) {
+                            if (i < here) {
+                                if (is_v) { // one box per page: [half of the dims][16 tokens][128 B]
+                                    tma_load_5d(dst + uint32_t(i * 4096), &map_v, 0, 0, 0, c, c3[i], full);
+                                } else { // [half of the dims][128 tokens][128 B]
+                                    tma_load_4d(dst + uint32_t(i * 2048), &map_k, 0, 0, c, c3[i], full);
+                                    tma_load_4d(dst + uint32_t(kSlot / 2 + i * 2048), &map_k, 64, 0, c, c3[i], full);
+                                }
+                            }
                         }
                     }
-                    free_bar[slot] = is_v ? pv_bar(tile_no, c) : s_bar(tile_no, c);
-                    free_parity[slot] = (tile_no >> 1) & 1;
+                    __syncwarp();
+                    at.next(p.stages);
+                    first_round = first_round && at.slot != 0;
                 }
             };
             int page = page_of(f.from), ahead = page_of(f.from + 1);
-            load(page, n, false);
+            load(page, false);
             for (int i = 0; i < count && alive; ++i) {
                 const int two_ahead = page_of(f.from + i + 2);
                 if (i + 1 < count) {
-                    load(ahead, n + i + 1, false);
+                    load(ahead, false);
                 }
-                load(page, n + i, true);
+                load(page, true);
                 page = ahead;
                 ahead = two_ahead;
             }
-            n += count;
         }
         if (!alive && lane == 0) {
             give_up();
@@ -409,78 +428,69 @@ __global__ void __launch_bounds__(kThreads, 1)
     } else if (warp == kIssuer) {
         // ================================ MMAs ===========================================================
         auto wait = [&](uint32_t at, int parity) { return __all_sync(0xffffffffu, wait_or_abort(at, uint32_t(parity), s_abort)) != 0; };
-        {
-            const uint32_t idesc_s = make_idesc(true, false, kBk, n_c), idesc_o = make_idesc(true, false, kD, n_c) | (1u << 15); // A MN-major
-            bool ok = true;
-            int op = 0, n = 0, n_fragments = 0;
-            auto next_slot = [&]() { // waits for the operand
-                const int slot = op % p.stages;
-                ok = ok && wait(bar(kBarFull + slot), (op / p.stages) & 1);
-                ++op;
-                return base + uint32_t(slot * kSlot);
-            };
-            auto scores = [&](int tile_no, bool waits) { // S of tile tile_no; waits: until the tile before it has been read
-                for (int c = 0; c < groups && ok; ++c) {
-                    if (waits) {
-                        ok = wait(bar(kBarRead + c), (tile_no - 1) & 1);
-                    }
-                    const uint32_t k_s = next_slot();
-                    if (!ok) {
-                        break;
-                    }
-                    tc_fence_after();
-                    const uint32_t q_s = base + uint32_t(lay.q + c * n_c * kD * 2);
-                    const uint64_t da = smem_desc_sw128(k_s, 0, 1024), db = smem_desc_sw128(q_s, 0, 1024), db2 = desc_at(db, uint32_t(n_c * 128));
-                    if (elect_one()) {
+        const uint32_t idesc_s = make_idesc(true, false, kBk, n_c), idesc_o = make_idesc(true, false, kD, n_c) | (1u << 15); // A MN-major
+        // low words of the operands' descriptors count 16-byte steps; the high words are the same for all
+        const uint64_t slots_k = smem_desc_sw128(base, 0, 1024), slots_v = smem_desc_sw128(base, 2048, 1024);
+        const uint64_t q_desc = smem_desc_sw128(base + uint32_t(lay.q), 0, 1024), p_desc = smem_desc_sw128(base + uint32_t(lay.w), 0, 1024);
+        const uint32_t group_bytes = uint32_t(n_c) * 256, half_bytes = uint32_t(n_c) * 128;
+        bool ok = true;
+        Cursor at;
+        int n = 0, n_fragments = 0;
+        auto scores = [&](int tile_no, bool waits) { // S of tile tile_no; waits: until the tile before it has been read
+            uint64_t b = q_desc;
+            uint32_t d = tmem, done = s_bar(tile_no, 0), read = bar(kBarRead);
+            for (int c = 0; c < groups && ok; ++c, b = desc_at(b, group_bytes), d += uint32_t(n_c), done += 8, read += 8) {
+                ok = (!waits || wait(read, (tile_no - 1) & 1)) && wait(bar(kBarFull + at.slot), int(at.parity));
+                tc_fence_after();
+                const uint64_t a = desc_at(slots_k, uint32_t(at.slot * kSlot)), b2 = desc_at(b, half_bytes);
+                if (ok && elect_one()) {
 #pragma unroll
-                        for (int ks = 0; ks < kD / 16; ++ks) {
-                            umma_f16(tmem + uint32_t(c * n_c), desc_at(da, (ks >> 2) * (kSlot / 2) + (ks & 3) * 32),
-                                     desc_at(ks < 4 ? db : db2, (ks & 3) * 32), idesc_s, ks > 0 ? 1u : 0u);
+                    for (int ks = 0; ks < kD / 16; ++ks) {
+                        umma_f16(d, desc_at(a, (ks >> 2) * (kSlot / 2) + (ks & 3) * 32), desc_at(ks < 4 ? b : b2, (ks & 3) * 32), idesc_s, ks > 0 ? 1u : 0u);
+                    }
+                    umma_commit(done);
+                    umma_commit(bar(kBarFree + at.slot));
+                }
+                __syncwarp();
+                at.next(p.stages);
+            }
+        };
+        Fragment f;
+        for (; ok && next_fragment(p, walk, f); ++n_fragments) {
+            const int count = f.upto - f.from;
+            ok = wait(bar(kBarQ), n_fragments & 1);
+            scores(n, n > 0);
+            for (int i = 0; i < count && ok; ++i, ++n) {
+                if (i + 1 < count) {
+                    scores(n + 1, true);
+                }
+                ok = ok && wait(bar(kBarP), n & 1);
+                if (i == 0 && n_fragments > 0) {
+                    ok = ok && wait(bar(kBarO), (n_fragments - 1) & 1);
+                }
+                uint64_t b = p_desc;
+                uint32_t d = tmem_o, done = pv_bar(n, 0);
+                for (int c = 0; c < groups && ok; ++c, b = desc_at(b, group_bytes), d += uint32_t(n_c), done += 8) {
+                    ok = wait(bar(kBarFull + at.slot), int(at.parity));
+                    tc_fence_after();
+                    const uint64_t a = desc_at(slots_v, uint32_t(at.slot * kSlot)), b2 = desc_at(b, half_bytes);
+                    if (ok && elect_one()) {
+#pragma unroll
+                        for (int kk = 0; kk < kBk / 16; ++kk) { // 16 keys: one page
+                            umma_f16(d, desc_at(a, kk * 4096), desc_at(kk < 4 ? b : b2, (kk & 3) * 32), idesc_o, i > 0 || kk > 0 ? 1u : 0u);
                         }
-                        umma_commit(s_bar(tile_no, c));
+                        umma_commit(done);
+                        umma_commit(bar(kBarFree + at.slot));
                     }
                     __syncwarp();
-                }
-            };
-            Fragment f;
-            for (; ok && next_fragment(p, walk, f); ++n_fragments) {
-                const int count = f.upto - f.from;
-                ok = wait(bar(kBarQ), n_fragments & 1);
-                scores(n, n > 0);
-                for (int i = 0; i < count && ok; ++i, ++n) {
-                    if (i + 1 < count) {
-                        scores(n + 1, true);
-                    }
-                    ok = ok && wait(bar(kBarP), n & 1);
-                    if (i == 0 && n_fragments > 0) {
-                        ok = ok && wait(bar(kBarO), (n_fragments - 1) & 1);
-                    }
-                    for (int c = 0; c < groups && ok; ++c) {
-                        const uint32_t v_s = next_slot();
-                        if (!ok) {
-                            break;
-                        }
-                        tc_fence_after();
-                        const uint32_t p_s = base + uint32_t(lay.w + c * n_c * kBk * 2);
-                        const uint64_t da = smem_desc_sw128(v_s, 2048, 1024), db = smem_desc_sw128(p_s, 0, 1024),
-                                       db2 = desc_at(db, uint32_t(n_c * 128));
-                        if (elect_one()) {
-#pragma unroll
-                            for (int kk = 0; kk < kBk / 16; ++kk) { // 16 keys: one page
-                                umma_f16(tmem_o + uint32_t(c * n_c), desc_at(da, kk * 4096), desc_at(kk < 4 ? db : db2, (kk & 3) * 32), idesc_o,
-                                         i > 0 || kk > 0 ? 1u : 0u);
-                            }
-                            umma_commit(pv_bar(n, c));
-                        }
-                        __syncwarp();
-                    }
+                    at.next(p.stages);
                 }
             }
-            if (!ok && lane == 0) {
-                give_up();
-            }
-            __syncwarp();
         }
+        if (!ok && lane == 0) {
+            give_up();
+        }
+        __syncwarp();
     } else {
         // ================================ weights, mixing, output ========================================
         bool dead = false; // a thread whose wait ran out keeps walking, so that the named barriers see all of them
@@ -833,8 +843,7 @@ int attention_gates_tc(stream_t stream, llaisysDataType_t dtype, const KVView &k
     p.groups = kv.nkvh;
     p.n_c = padded(p.bq);
     const int n_columns = p.groups * p.n_c;
-    // (a slot is handed over by the barrier of the operand that it held: that barrier must not run on before the slot is due)
-    p.stages = std::min(kMaxStages, 3 * p.groups);
+    p.stages = kMaxStages;
     while (p.stages > 2 && Layout(p.stages, n_columns).total > kSmemLimit) {
         --p.stages;
     }
