@@ -14,7 +14,8 @@
 //   warps 0-15   read S (lane = key), compute the weights, store them as f16 times 2^15 into the buffer that becomes P; when all heads
 //                are there, mix them IN PLACE: 16 keys of one query, all heads, are read as mma.sync operands, multiplied by the talk
 //                matrix (in registers) and stored as bf16 to the same places
-//   warp 16      TMA of K and V tiles into a ring of 32 KiB slots (as warp 17, an elected lane)
+//   warps 16, 18 TMA of K and V tiles into a ring of 32 KiB slots, half of a tile's pages each (as in warp 17, an elected lane issues:
+//                a warp between busy ones needs about 1000 clocks for a tile's 16 boxes)
 //   warp 17      issues the MMAs (the whole warp walks, an elected lane issues: descriptors then stay in uniform registers, which made
 //                a batch of eight small MMAs 3.7 times as fast as a loop run by one thread): S of tile t + 1 kv head by kv head as the scores of tile t have been read, then O of tile t.
 //                Weights of tile t + 1 go where P_c of tile t was as soon as O_c has taken it.
@@ -37,7 +38,7 @@ namespace llaisys::kernels {
 namespace {
 
 constexpr int kD = 128, kBk = 128, kPages = kBk / 16;
-constexpr int kWorkers = 16, kProducer = 16, kIssuer = 17, kThreads = 18 * 32;
+constexpr int kWorkers = 16, kProducer = 16, kIssuer = 17, kProducer2 = 18, kThreads = 19 * 32;
 constexpr int kChunk = 32; // columns of one kv head that a warp turns into weights at a time
 constexpr int kSlot = kBk * kD * 2, kMaxStages = 6, kMaxColumns = 256, kMaxGroups = 16;
 // What a block costs besides its tiles (queries in, products drained, outputs out), in tiles. The line that is cut into equal shares
@@ -221,8 +222,8 @@ struct Layout {
     }
 };
 // barriers
-constexpr int kBarFull = 0;                            // [stages] producer -> issuer: a tile has landed
-constexpr int kBarFree = kBarFull + kMaxStages;        // [stages] MMAs -> producer: it has been used
+constexpr int kBarFull = 0;                            // [stages] producers -> issuer: a tile has landed
+constexpr int kBarFree = kBarFull + kMaxStages;        // [stages] MMAs -> producers: it has been used
 constexpr int kBarS = kBarFree + kMaxStages;           // [2][groups] S_c of a tile is written
 constexpr int kBarPV = kBarS + 2 * kMaxGroups;         // [2][groups] O_c has taken a tile (P_c is free)
 constexpr int kBarRead = kBarPV + 2 * kMaxGroups;      // [groups] workers -> issuer: S_c has been read (a warp per chunk and quarter)
@@ -268,7 +269,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     if (tid == 0) {
         prefix[0] = 0;
         for (int i = 0; i < kBarO + 1; ++i) {
-            mbar_init(bar(i), i < kBarRead ? 1 : (i < kBarP ? 4 * ((n_c + kChunk - 1) / kChunk) : kWorkers));
+            mbar_init(bar(i), i < kBarFree ? 2 : i < kBarRead ? 1 : (i < kBarP ? 4 * ((n_c + kChunk - 1) / kChunk) : kWorkers));
         }
         misc[0] = misc[1] = misc[2] = misc[3] = 0;
         *s_abort = 0;
@@ -359,9 +360,10 @@ __global__ void __launch_bounds__(kThreads, 1)
     tc_fence_after();
     const uint32_t tmem = uint32_t(misc[5]), tmem_o = tmem + kMaxColumns;
 
-    if (warp == kProducer) {
+    if (warp == kProducer || warp == kProducer2) {
         // ================================ K and V tiles ==================================================
         bool alive = true;
+        const int page0 = warp == kProducer ? 0 : kPages / 2; // this warp's pages of a tile
         Cursor at;
         bool first_round = true; // nothing has used the slots yet
         Fragment f;
@@ -379,11 +381,11 @@ __global__ void __launch_bounds__(kThreads, 1)
             };
             // the operand of every kv head of one tile
             auto load = [&](int page, bool is_v) {
-                const int here = __popc(__ballot_sync(0xffffffffu, lane < kPages && page >= 0)); // (the first ones)
-                int c3[kPages];
+                const int here = min(max(__popc(__ballot_sync(0xffffffffu, lane < kPages && page >= 0)) - page0, 0), kPages / 2); // (the first ones)
+                int c3[kPages / 2];
 #pragma unroll
-                for (int i = 0; i < kPages; ++i) {
-                    c3[i] = int((p.page0 + max(__shfl_sync(0xffffffffu, page, i), 0)) * 2) + (is_v ? 1 : 0);
+                for (int i = 0; i < kPages / 2; ++i) {
+                    c3[i] = int((p.page0 + max(__shfl_sync(0xffffffffu, page, page0 + i), 0)) * 2) + (is_v ? 1 : 0);
                 }
                 for (int c = 0; c < groups && alive; ++c) {
                     if (!first_round && !__all_sync(0xffffffffu, wait_or_abort(bar(kBarFree + at.slot), at.parity ^ 1u, s_abort))) {
@@ -394,13 +396,13 @@ __global__ void __launch_bounds__(kThreads, 1)
                     if (elect_one()) {
                         mbar_arrive_expect_tx(full, uint32_t(here) * 4096);
 #pragma unroll
-                        for (int i = 0; i < kPages; ++i) {
+                        for (int i = 0; i < kPages / 2; ++i) {
                             if (i < here) {
                                 if (is_v) { // one box per page: [half of the dims][16 tokens][128 B]
-                                    tma_load_5d(dst + uint32_t(i * 4096), &map_v, 0, 0, 0, c, c3[i], full);
+                                    tma_load_5d(dst + uint32_t((page0 + i) * 4096), &map_v, 0, 0, 0, c, c3[i], full);
                                 } else { // [half of the dims][128 tokens][128 B]
-                                    tma_load_4d(dst + uint32_t(i * 2048), &map_k, 0, 0, c, c3[i], full);
-                                    tma_load_4d(dst + uint32_t(kSlot / 2 + i * 2048), &map_k, 64, 0, c, c3[i], full);
+                                    tma_load_4d(dst + uint32_t((page0 + i) * 2048), &map_k, 0, 0, c, c3[i], full);
+                                    tma_load_4d(dst + uint32_t(kSlot / 2 + (page0 + i) * 2048), &map_k, 64, 0, c, c3[i], full);
                                 }
                             }
                         }
