@@ -17,6 +17,7 @@ random permutation of a 16384-page pool):
   config5     one 131072-token sequence, 28 layers, KV range split over the GPUs, partial results exchanged and merged
   vozozen     the Vozozen design beside Qwen2 at equal size: whole models and single kernels (bench_models.py)
   doderax     the Doderax design beside Vozozen, in the same way
+  lilovik     the Lilovik design beside Qwen2, in the same way
 The default run (north_star) also measures config2 and config3 in the same process (N = 1: sub-records "config2",
 "config3") and, with N > 1, the KV-range split of config5 in the same process group (sub-record "kv_split"): the one
 mode of this path in which GPUs exchange data.

@@ -168,6 +168,21 @@ def test_greedy_generation_and_engine(cuda_device):
                                                                              temperature=0.9, seed=1)
 
 
+def test_pages_of_a_shared_beginning_are_reused_without_recurrent_layers(cuda_device):
+    """A model whose layers are all attention finds a published prefix; logits behind it are those of the whole sequence."""
+    cfg, w = cases.case("attention_only", seed=1)
+    model = make(cfg, w, "f32")
+    model.configure_cache(3, 96)
+    toks = cases.tokens(cfg, 60, seed=4)
+    a = model.add_seq()
+    model.step_rows([a], [toks[:50]], [])
+    b, covered = model.add_seq_with_prefix(toks)
+    assert covered == 48
+    check(model.step_rows([b], [toks[covered:]], range(60 - covered)), oracle.forward(cfg, w, toks)[0][covered:], "f32")
+    model.free_seq(a)
+    check(model.step_rows([b], [[7]], [0]), oracle.forward(cfg, w, toks + [7])[0][-1:], "f32")
+
+
 def test_loading_errors(cuda_device):
     cfg, w = cases.case("mixed")
     short = {k: v for k, v in w.items() if k != "l3.mix.talk"}

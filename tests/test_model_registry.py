@@ -11,13 +11,15 @@ import torch
 
 import llaisys_b200 as llaisys
 from llaisys_b200 import trace
-from llaisys_b200.models import Doderax, Qwen2, Vozozen, load_model, model_class
+from llaisys_b200.models import Doderax, Lilovik, Qwen2, Vozozen, load_model, model_class
 from llaisys_b200.models import doderax as dx
+from llaisys_b200.models import lilovik as lk
 from llaisys_b200.models import vozozen as vz
 from llaisys_b200.models.weights import SafetensorsFile, checkpoint_files
 from oracle import doderax as doderax_oracle
+from oracle import lilovik as lilovik_oracle
 from oracle import vozozen as oracle
-from tests import doderax_cases
+from tests import doderax_cases, lilovik_cases
 from tests import vozozen_cases as cases
 
 
@@ -34,6 +36,7 @@ def write_safetensors(path, tensors):
 def test_class_by_config():
     assert model_class({"architecture": "Vozozen"}) is Vozozen
     assert model_class({"architecture": "Doderax"}) is Doderax
+    assert model_class({"architecture": "Lilovik"}) is Lilovik
     assert model_class({"architectures": ["Qwen2ForCausalLM"], "model_type": "qwen2"}) is Qwen2
     assert model_class({"model_type": "qwen2"}) is Qwen2
     with pytest.raises(ValueError, match="Mamba"):
@@ -185,6 +188,73 @@ def test_doderax_oracle_mechanisms_agree_with_closed_forms():
     assert torch.allclose(doderax_oracle.short_conv(y, w), oracle.silu(y))
     assert doderax_oracle.pair_rows([3, 4, 3], {"buckets": 10, "mul_prev": 2, "mul_cur": 5}) == [10, 6, 3]
     assert torch.allclose(doderax_oracle.gelu(y), torch.nn.functional.gelu(y, approximate="tanh"))
+
+
+@pytest.mark.parametrize("name", sorted(lilovik_cases.CASES))
+def test_lilovik_configuration_reaches_the_library(name):
+    cfg, w = lilovik_cases.case(name)
+    assert set(w) == set(lk.weight_shapes(cfg)) and all(w[n].shape == s for n, s in lk.weight_shapes(cfg).items())
+    meta = lk.build_meta(cfg, llaisys.DataType.F32)
+    assert (meta.nlayer, meta.width, meta.voc, meta.end_token) == (len(cfg["layers"]), cfg["width"], cfg["vocab"], -1)
+    assert meta.eps == pytest.approx(cfg["norm"]["eps"]) and meta.logit_scale == pytest.approx(cfg["logit_scale"])
+    for i, entry in enumerate(cfg["layers"]):
+        got, m = meta.layers[i], entry["mixer"]
+        assert got.ff == (entry["mlp"]["ff"] if entry["mlp"] else 0) and got.recurrent == (entry["type"] == "mingru")
+        if got.recurrent:
+            assert got.gru_width == m["width"]
+            continue
+        temp = m.get("q_temp")
+        assert (got.attn.heads, got.attn.kv_heads, got.attn.dim, got.attn.vdim) == (m["heads"], m["kv_heads"], m["dim"], m["vdim"])
+        assert got.attn.scale == pytest.approx(m["scale"]) and got.attn.softcap == pytest.approx(m.get("softcap", 0.0))
+        assert got.attn.temp_coef == pytest.approx(temp["coef"] if temp else 0.0)
+        assert temp is None or got.attn.temp_every == temp["every"]
+
+
+def test_unknown_parts_of_a_lilovik_configuration_are_refused():
+    cfg, w = lilovik_cases.case("mixed")
+    cfg["layers"][0]["type"] = "serial"
+    with pytest.raises(ValueError, match="serial"):
+        lk.build_meta(cfg, llaisys.DataType.BF16)
+    cfg, w = lilovik_cases.case("mixed")
+    cfg["layers"][1]["mlp"]["kind"] = "experts"
+    with pytest.raises(ValueError, match="experts"):
+        lk.build_meta(cfg, llaisys.DataType.BF16)
+    with pytest.raises(RuntimeError, match="NVIDIA"):
+        Lilovik(config=lilovik_cases.case("mixed")[0], state_dict=w, device=llaisys.DeviceType.CPU)
+
+
+def test_lilovik_oracle_mechanisms_agree_with_closed_forms():
+    torch.manual_seed(2)
+    T, H, G, d, dv = 9, 4, 2, 6, 5
+    q, k, v = torch.randn(T, H, d).double(), torch.randn(T, G, d).double(), torch.randn(T, G, dv).double()
+    none, eye = torch.zeros(H).double(), torch.eye(H).double()
+    # slopes halve from head to head at eight heads; a query far behind its keys sees sigmoid(score - slope distance + bias)
+    assert torch.allclose(lilovik_oracle.slopes(8), 0.5 ** torch.arange(1, 9).double())
+    a = lilovik_oracle.gates(q, k, 0.3, None, none + 0.7)
+    assert torch.allclose(a[1, 5, 2], torch.sigmoid(0.3 * (q[5, 1] @ k[2, 0]) - 3 * 2.0 ** -4 + 0.7))
+    assert (torch.triu(a, 1) == 0).all() and torch.allclose(a[:, 4:6, :], lilovik_oracle.gates(q[4:6], k, 0.3, None, none + 0.7, first=4))
+    # a wide cap is none, and nothing passes a cap
+    assert torch.allclose(lilovik_oracle.gates(q, k, 0.3, 1e6, none), lilovik_oracle.gates(q, k, 0.3, None, none), atol=1e-9)
+    assert lilovik_oracle.gates(q, k, 50.0, 2.0, none)[:, range(T), range(T)].max() <= torch.sigmoid(torch.tensor(2.0).double())
+    # mixing with the identity changes nothing, with a permutation it moves heads; unweighted values add up
+    assert torch.allclose(lilovik_oracle.mix_heads(a, eye), a) and torch.allclose(lilovik_oracle.mix_heads(a, eye[[2, 0, 1, 3]]), a[[2, 0, 1, 3]])
+    ones = torch.tril(torch.ones(H, T, T)).double()
+    assert torch.allclose(lilovik_oracle.weigh_values(ones, v), v.cumsum(0).repeat_interleave(H // G, 1))
+    # the query factor steps where position + 1 reaches a multiple
+    f = lilovik_oracle.query_factors([0, 6, 7, 14, 15], {"coef": 0.5, "every": 8})
+    assert torch.allclose(f, 1 + 0.5 * torch.tensor([1.0, 1.0, 2.0, 2.0, 3.0]).double().log()) and (lilovik_oracle.query_factors([3], None) == 1).all()
+    # position 0 is (0, 1, 0, 1, ..); the pair's distance to another position depends on the difference only
+    p = lilovik_oracle.position_vectors([0, 3, 7, 10], 8)
+    assert torch.equal(p[0], torch.tensor([0.0, 1.0] * 4).double()) and torch.allclose(p[0] @ p[1], p[2] @ p[3])
+    # a closed gate keeps the state, an open one takes the candidate, which is continuous at zero
+    z, u, o = (torch.randn(T, 3).double() for _ in range(3))
+    start = torch.randn(3).double()
+    y, S = lilovik_oracle.min_gru(z * 0 - 1e3, u, o, start)
+    assert torch.allclose(S, start) and torch.allclose(y, start * lilovik_oracle.silu(o))
+    _, S = lilovik_oracle.min_gru(z * 0 + 1e3, u.abs(), o, start)
+    assert torch.allclose(S, u[-1].abs() + 0.5)
+    _, S = lilovik_oracle.min_gru(z * 0 + 1e3, torch.tensor([[0.0, -1e-9, -50.0]]).double().expand(T, 3), o, start)
+    assert torch.allclose(S, torch.tensor([0.5, 0.5, 0.0]).double())
 
 
 def test_no_host_stand_in():
