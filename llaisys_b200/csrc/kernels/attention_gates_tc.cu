@@ -11,7 +11,7 @@
 //   O_c[dim, column]  += V_c^T P_c        A = V tile (MN-major, as the pages hold it), B = P_c [column][key]
 // S_c and O_c of all kv heads live in TMEM (256 columns each).
 //
-//   warps 0-15   read S (lane = key), compute the weights, store them as f16 times 2^15 into the buffer that becomes P; when all heads
+//   warps 0-15   read S as mma fragments (a thread has four keys of two neighbouring columns in every eight), compute the weights, store them as f16 times 2^15 into the buffer that becomes P; when all heads
 //                are there, mix them IN PLACE: 16 keys of one query, all heads, are read as mma.sync operands, multiplied by the talk
 //                matrix (in registers) and stored as bf16 to the same places
 //   warps 16, 18 TMA of K and V tiles into a ring of 32 KiB slots, half of a tile's pages each (as in warp 17, an elected lane issues:
@@ -201,8 +201,15 @@ __device__ __forceinline__ Pair rcp4(Pair x, Pair y, float unit) {
 }
 // n / d for 0 <= n < 2^15, inv = 1 / d rounded
 __device__ __forceinline__ int small_div(int n, float inv) { return int((float(n) + 0.5f) * inv); }
-__device__ __forceinline__ void store_u16(uint32_t addr, uint32_t v) {
-    asm volatile("st.shared.u16 [%0], %1;\n" ::"r"(addr), "h"(static_cast<unsigned short>(v)) : "memory");
+// 32 columns of 16 lanes as m16n8 fragments: of columns 8 j + 2 (lane % 4) and the next, r[4 j ..] holds those of lane / 4, then those of lane / 4 + 8
+__device__ __forceinline__ void tmem_ld_fragments(uint32_t taddr, uint32_t (&r)[16]) {
+    asm volatile("tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
+                   "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+                 : "r"(taddr));
+}
+__device__ __forceinline__ void stmatrix_x4_trans(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
+    asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1, %2, %3, %4};\n" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
 }
 __device__ __forceinline__ void stmatrix_x4(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
     asm volatile("stmatrix.sync.aligned.m8n8.x4.shared.b16 [%0], {%1, %2, %3, %4};\n" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
@@ -515,8 +522,9 @@ __global__ void __launch_bounds__(kThreads, 1)
         const float to_exp = capped ? 2.f * kLog2e * p.scale / p.gates.softcap : -kLog2e * p.scale, cap2 = 2.f * kLog2e * p.gates.softcap;
         const Pair to_exp2 = pair(to_exp, to_exp), ones = pair(1.f, 1.f);
         const uint32_t w_s = base + uint32_t(lay.w);
-        // a weight of column r: row r, 16-byte chunk (key / 8) ^ (r mod 8) of the row's 64-key half
-        const uint32_t w_key = w_s + uint32_t((quarter >> 1) * n_c * 128 + (((quarter & 1) * 4 + (lane >> 3)) << 4) + (lane & 7) * 2);
+        // a weight of column r: row r, 16-byte chunk (key / 8) ^ (r mod 8) of the row's 64-key half; this lane addresses the row of column
+        // lane % 8 for keys 8 (lane / 8) .. of the warp's 32
+        const uint32_t w_lane = w_s + uint32_t((quarter >> 1) * n_c * 128 + (lane & 7) * 128 + ((((quarter & 1) * 4 + (lane >> 3)) ^ (lane & 7)) << 4));
 
         // talk as mma operands, and the head whose row this lane addresses: byte offset of its kv head, place in the group
         uint32_t talk[MT][MT][4];
@@ -568,8 +576,11 @@ __global__ void __launch_bounds__(kThreads, 1)
             for (int t = f.from; t < f.upto; ++t, ++n) {
                 const int first = (blk.tile0 + t) * kBk;
                 const bool edge = first + kBk > blk.pos0 + 1 || (p.batch.window > 0 && first + p.batch.window < blk.pos0 + blk.n_q);
-                const float ago0 = float(blk.pos0 - first - key); // from this thread's key to the block's first query
-                const Pair ago2 = pair(ago0, ago0);
+                float ago[4]; // from this thread's keys to the block's first query
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    ago[k] = float(blk.pos0 - first - quarter * 32 - (lane >> 2) - 8 * k);
+                }
                 const int chunks = (n_c + kChunk - 1) / kChunk;
                 for (int c = 0, k = 0; c < groups; ++c) {
                     for (int piece = 0; piece < chunks; ++piece, ++k) {
@@ -579,23 +590,24 @@ __global__ void __launch_bounds__(kThreads, 1)
                         const int col0 = c * n_c + piece * kChunk, n_units = min(kChunk, n_c - piece * kChunk) / 8;
                         wait(s_bar(n, c), (n >> 1) & 1);
                         tc_fence_after();
-                        uint32_t raw[kChunk]; // (columns past the chunk are S or O columns all the same, and go unused)
-                        tmem_ld32_nowait(tmem + lanes + uint32_t(col0), raw);
+                        uint32_t raw[2][kChunk / 2]; // 16 keys each (columns past the chunk are S or O columns all the same, and go unused)
+                        tmem_ld_fragments(tmem + lanes + uint32_t(col0), raw[0]);
+                        tmem_ld_fragments(tmem + lanes + (16u << 16) + uint32_t(col0), raw[1]);
                         tmem_wait_ld();
                         tc_fence_before();
                         arrive(kBarRead + c);
-                        uint32_t weights[kChunk / 2]; // as f16 pairs
+                        uint32_t weights[kChunk / 8][4]; // f16 pairs of four keys
 #pragma unroll
                         for (int u = 0; u < kChunk / 8; ++u) {
                             if (u >= n_units) {
                                 break;
                             }
                             Pair x[4], a[4];
+                            const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(columns + 2 * (col0 + u * 8) + 4 * (lane & 3));
 #pragma unroll
                             for (int i = 0; i < 4; ++i) {
-                                const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(columns + 2 * (col0 + u * 8) + 4 * i);
-                                a[i] = fma2(k2.x, ago2, k2.y);
-                                x[i] = pair(__uint_as_float(raw[u * 8 + 2 * i]), __uint_as_float(raw[u * 8 + 2 * i + 1]));
+                                a[i] = fma2(k2.x, pair(ago[i], ago[i]), k2.y);
+                                x[i] = pair(__uint_as_float(raw[i / 2][4 * u + 2 * (i % 2)]), __uint_as_float(raw[i / 2][4 * u + 2 * (i % 2) + 1]));
                             }
                             if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
 #pragma unroll
@@ -627,30 +639,27 @@ __global__ void __launch_bounds__(kThreads, 1)
                             }
                             if (edge) {
                                 const float window = p.batch.window > 0 ? float(p.batch.window) : INFINITY;
+                                const int r = piece * kChunk + u * 8 + 2 * (lane & 3);
+                                const float q0 = float(small_div(r, inv_share)), q1 = float(small_div(r + 1, inv_share));
 #pragma unroll
-                                for (int i = 0; i < 8; ++i) {
-                                    const float ago = ago0 + float(small_div(piece * kChunk + u * 8 + i, inv_share));
-                                    w[i] = ago >= 0.f && ago < window ? w[i] : 0.f;
+                                for (int i = 0; i < 4; ++i) {
+                                    w[2 * i] = ago[i] + q0 >= 0.f && ago[i] + q0 < window ? w[2 * i] : 0.f;
+                                    w[2 * i + 1] = ago[i] + q1 >= 0.f && ago[i] + q1 < window ? w[2 * i + 1] : 0.f;
                                 }
                             }
 #pragma unroll
                             for (int i = 0; i < 4; ++i) {
-                                weights[u * 4 + i] = pack2<false>(w[2 * i], w[2 * i + 1]);
+                                weights[u][i] = pack2<false>(w[2 * i], w[2 * i + 1]);
                             }
                         }
                         if (n > 0) {
                             wait(pv_bar(n - 1, c), ((n - 1) >> 1) & 1);
                         }
-                        const uint32_t at = w_key + uint32_t(c * n_c * kBk * 2 + piece * kChunk * 128);
+                        const uint32_t at = w_lane + uint32_t(c * n_c * kBk * 2 + piece * kChunk * 128);
 #pragma unroll
-                        for (int i = 0; i < 8; i += 2) {
-                            const uint32_t at0 = (at ^ uint32_t(i << 4)) + uint32_t(i * 128), at1 = (at ^ uint32_t((i + 1) << 4)) + uint32_t((i + 1) * 128);
-#pragma unroll
-                            for (int u = 0; u < kChunk / 8; ++u) {
-                                if (u < n_units) {
-                                    store_u16(at0 + uint32_t(u * 1024), weights[u * 4 + i / 2]);
-                                    store_u16(at1 + uint32_t(u * 1024), weights[u * 4 + i / 2] >> 16);
-                                }
+                        for (int u = 0; u < kChunk / 8; ++u) {
+                            if (u < n_units) {
+                                stmatrix_x4_trans(at + uint32_t(u * 1024), weights[u][0], weights[u][1], weights[u][2], weights[u][3]);
                             }
                         }
                     }
