@@ -590,66 +590,53 @@ __global__ void __launch_bounds__(kThreads, 1)
                         const int col0 = c * n_c + piece * kChunk, n_units = min(kChunk, n_c - piece * kChunk) / 8;
                         wait(s_bar(n, c), (n >> 1) & 1);
                         tc_fence_after();
-                        uint32_t raw[2][kChunk / 2]; // 16 keys each (columns past the chunk are S or O columns all the same, and go unused)
-                        tmem_ld_fragments(tmem + lanes + uint32_t(col0), raw[0]);
-                        tmem_ld_fragments(tmem + lanes + (16u << 16) + uint32_t(col0), raw[1]);
-                        tmem_wait_ld();
-                        tc_fence_before();
-                        arrive(kBarRead + c);
                         uint32_t weights[kChunk / 8][4]; // f16 pairs of four keys
 #pragma unroll
-                        for (int u = 0; u < kChunk / 8; ++u) {
-                            if (u >= n_units) {
-                                break;
+                        for (int half = 0; half < 2; ++half) { // 16 keys at a time, two of them this thread's
+                            uint32_t raw[16]; // (columns past the chunk are S or O columns all the same, and go unused)
+                            tmem_ld_fragments(tmem + lanes + (uint32_t(16 * half) << 16) + uint32_t(col0), raw);
+                            tmem_wait_ld();
+                            if (half == 1) {
+                                tc_fence_before();
+                                arrive(kBarRead + c);
                             }
-                            Pair x[4], a[4];
-                            const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(columns + 2 * (col0 + u * 8) + 4 * (lane & 3));
+                            const Pair ago_a = pair(ago[2 * half], ago[2 * half]), ago_b = pair(ago[2 * half + 1], ago[2 * half + 1]);
 #pragma unroll
-                            for (int i = 0; i < 4; ++i) {
-                                a[i] = fma2(k2.x, pair(ago[i], ago[i]), k2.y);
-                                x[i] = pair(__uint_as_float(raw[i / 2][4 * u + 2 * (i % 2)]), __uint_as_float(raw[i / 2][4 * u + 2 * (i % 2) + 1]));
-                            }
-                            if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
-#pragma unroll
-                                for (int i = 0; i < 4; ++i) {
-                                    x[i] = one_plus_ex2(mul2(x[i], to_exp2), ones);
+                            for (int u = 0; u < kChunk / 8; ++u) {
+                                if (u >= n_units) {
+                                    break;
                                 }
-#pragma unroll
-                                for (int i = 0; i < 4; i += 2) {
-                                    const Pair r = rcp4(x[i], x[i + 1], cap2), first = fma2(r, x[i + 1], a[i]);
-                                    x[i + 1] = fma2(r, x[i], a[i + 1]);
-                                    x[i] = first;
+                                const ulonglong2 k2 = *reinterpret_cast<const ulonglong2 *>(columns + 2 * (col0 + u * 8) + 4 * (lane & 3));
+                                Pair x = pair(__uint_as_float(raw[4 * u]), __uint_as_float(raw[4 * u + 1]));
+                                Pair y = pair(__uint_as_float(raw[4 * u + 2]), __uint_as_float(raw[4 * u + 3]));
+                                const Pair a = fma2(k2.x, ago_a, k2.y), b = fma2(k2.x, ago_b, k2.y);
+                                if (capped) { // softcap tanh(y) = softcap - 2 softcap / (1 + e^(2 y))
+                                    x = one_plus_ex2(mul2(x, to_exp2), ones);
+                                    y = one_plus_ex2(mul2(y, to_exp2), ones);
+                                    const Pair r = rcp4(x, y, cap2), first_key = fma2(r, y, a);
+                                    y = fma2(r, x, b);
+                                    x = first_key;
+                                } else {
+                                    x = fma2(x, to_exp2, a);
+                                    y = fma2(y, to_exp2, b);
                                 }
-                            } else {
+                                x = one_plus_ex2(x, ones);
+                                y = one_plus_ex2(y, ones);
+                                const Pair r = rcp4(x, y, kWeightUnit);
+                                float w[4];
+                                unpair(mul2(r, y), w[0], w[1]);
+                                unpair(mul2(r, x), w[2], w[3]);
+                                if (edge) {
+                                    const float window = p.batch.window > 0 ? float(p.batch.window) : INFINITY;
+                                    const int col = piece * kChunk + u * 8 + 2 * (lane & 3);
 #pragma unroll
-                                for (int i = 0; i < 4; ++i) {
-                                    x[i] = fma2(x[i], to_exp2, a[i]);
+                                    for (int i = 0; i < 4; ++i) {
+                                        const float far = ago[2 * half + i / 2] + float(small_div(col + i % 2, inv_share));
+                                        w[i] = far >= 0.f && far < window ? w[i] : 0.f;
+                                    }
                                 }
-                            }
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) {
-                                x[i] = one_plus_ex2(x[i], ones);
-                            }
-                            float w[8];
-#pragma unroll
-                            for (int i = 0; i < 4; i += 2) {
-                                const Pair r = rcp4(x[i], x[i + 1], kWeightUnit);
-                                unpair(mul2(r, x[i + 1]), w[2 * i], w[2 * i + 1]);
-                                unpair(mul2(r, x[i]), w[2 * i + 2], w[2 * i + 3]);
-                            }
-                            if (edge) {
-                                const float window = p.batch.window > 0 ? float(p.batch.window) : INFINITY;
-                                const int r = piece * kChunk + u * 8 + 2 * (lane & 3);
-                                const float q0 = float(small_div(r, inv_share)), q1 = float(small_div(r + 1, inv_share));
-#pragma unroll
-                                for (int i = 0; i < 4; ++i) {
-                                    w[2 * i] = ago[i] + q0 >= 0.f && ago[i] + q0 < window ? w[2 * i] : 0.f;
-                                    w[2 * i + 1] = ago[i] + q1 >= 0.f && ago[i] + q1 < window ? w[2 * i + 1] : 0.f;
-                                }
-                            }
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) {
-                                weights[u][i] = pack2<false>(w[2 * i], w[2 * i + 1]);
+                                weights[u][2 * half] = pack2<false>(w[0], w[1]);
+                                weights[u][2 * half + 1] = pack2<false>(w[2], w[3]);
                             }
                         }
                         if (n > 0) {
