@@ -71,8 +71,8 @@ def close(got, want, dtype, factor=1.0, what=""):
 
 
 # dtype, kv heads, heads, key size, value size; does the tile kernel serve it
-SHAPES = [(F32, 2, 6, 20, 12, False), (F32, 4, 4, 64, 64, False), (BF16, 3, 3, 40, 72, False), (BF16, 1, 5, 13, 9, False),
-          (BF16, 4, 4, 64, 64, True), (BF16, 2, 6, 64, 32, True), (BF16, 3, 3, 16, 48, True), (BF16, 1, 7, 32, 128, True),
+SHAPES = [(F32, 2, 6, 20, 12, False), (F32, 3, 3, 64, 64, False), (BF16, 3, 3, 40, 72, False), (BF16, 1, 5, 13, 9, False),
+          (BF16, 5, 5, 64, 64, True), (BF16, 2, 6, 64, 32, True), (BF16, 3, 3, 16, 48, True), (BF16, 1, 7, 32, 128, True),
           (BF16, 8, 32, 128, 128, True), (BF16, 2, 12, 128, 128, True), (BF16, 5, 20, 96, 112, True), (BF16, 1, 1, 128, 16, True),
           (BF16, 24, 24, 32, 32, True), (BF16, 2, 64, 48, 80, True), (BF16, 25, 25, 32, 32, False), (BF16, 1, 66, 32, 32, False),
           (BF16, 1, 5, 128, 128, True), (BF16, 4, 4, 128, 128, True), (BF16, 16, 32, 128, 128, True), (BF16, 3, 24, 128, 128, True)]
@@ -113,7 +113,7 @@ def test_one_key_far_away(cuda_device, dtype, nkvh, nh, d, dv, tiles):
     decoded; the query just before the key sees nothing."""
     n = 400
     for place in (0, 1, 15, 16, 31, 32, 63, 64, 127, 128, 255, n - 1):
-        g = Gates(dtype, nkvh, nh, d, dv, [n], softcap=20.0, slopes=[0.01 * (h + 1) / nh for h in range(nh)], seed=place)
+        g = Gates(dtype, nkvh, nh, d, dv, [n], softcap=15.0, slopes=[0.01 * (h + 1) / nh for h in range(nh)], seed=place)
         g.bias = torch.full((nh,), -14.0).to(dtype)
         g.pool.k[0] *= 0.02
         direction = torch.ones(d) / d ** 0.5
