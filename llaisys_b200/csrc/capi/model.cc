@@ -1,5 +1,6 @@
 // extern "C" thunks of the generic model API and of the families that have no older ABI of their own.
 #include "llaisys/models/doderax.h"
+#include "llaisys/models/folivik.h"
 #include "llaisys/models/lilovik.h"
 #include "llaisys/models/model.h"
 #include "llaisys/models/vozozen.h"
@@ -102,6 +103,10 @@ LlaisysModel *llaisysDoderaxModelCreate(const LlaisysDoderaxMeta *meta, llaisysD
 }
 LlaisysModel *llaisysLilovikModelCreate(const LlaisysLilovikMeta *meta, llaisysDeviceType_t device, int device_id) {
     return create_model<llaisys::models::Lilovik>("llaisysLilovikModelCreate", meta, device, device_id);
+}
+
+LlaisysModel *llaisysFolivikModelCreate(const LlaisysFolivikMeta *meta, llaisysDeviceType_t device, int device_id) {
+    return create_model<llaisys::models::Folivik>("llaisysFolivikModelCreate", meta, device, device_id);
 }
 
 int llaisysModelRecordStream(LlaisysModel *model, int enable) {

@@ -3,6 +3,7 @@
 #pragma once
 
 #include "../models/doderax.hpp"
+#include "../models/folivik.hpp"
 #include "../models/lilovik.hpp"
 #include "../models/qwen2.hpp"
 #include "../models/vozozen.hpp"

@@ -71,6 +71,9 @@ struct AttnBatch {
     int32_t nh = 0;
     int32_t window = 0; // > 0: a query at position i sees keys j with 0 <= i - j < window; 0: all earlier keys
     int32_t keep_first = 0; // with a window: keys j < keep_first stay visible behind it (j <= i)
+    // Distance penalty of the softmax kernels: fade_a[h] ln(1 + fade_b[h] (i - j)) is taken off head h's score (after the scale).
+    // f32 [nh] on the executing device; null: none. fade_b >= 0.
+    const float *fade_a = nullptr, *fade_b = nullptr;
 };
 
 // Output selection: `out` [total_q, nh, d] in the KV dtype, or `part` float [total_q, nh, d + 2] holding the
@@ -143,6 +146,81 @@ struct NormAppendArgs {
     int32_t row_norm = 0;
     const void *bias = nullptr;
     float temp_coef = 0.f, temp_every = 1.f;
+    const float *head_scale = nullptr; // [nh] f32, not the row form: factor on every query head after norm and rotation; null: none
+};
+
+// K1d: what enters attention over latents. Of a packed projection row [.. query latent | key latent, key part to turn | gates ..]: the
+// query latent normed -> q_latent; the key latent normed and, behind it, the other key dims turned by their position -> the
+// token's row of the cache (KVView of one kv head, K rows of rank + rot_dims); a gate per head -> factor of the attention's epilogue.
+struct LatentAppendArgs {
+    const void *proj = nullptr; // [n_rows, row_stride], cache dtype
+    int64_t row_stride = 0;
+    int64_t q_at = 0, kv_at = 0, gate_at = 0; // gate_at < 0: no gate
+    int32_t q_rank = 0, rank = 0, rot_dims = 0, nh = 0;
+    const void *q_norm = nullptr, *kv_norm = nullptr; // [q_rank], [rank]
+    float eps = 0.f;
+    const float *rot_table = nullptr; // [n_rows, rot_dims / 2, 2] (rotary_table): dims 2 i and 2 i + 1 turn
+    void *q_latent = nullptr;         // [n_rows, q_latent_stride]
+    int64_t q_latent_stride = 0;
+    float *row_scale = nullptr;       // [n_rows, nh] = sigmoid(gate)
+    const int32_t *seq_ids = nullptr, *positions = nullptr;
+    size_t n_rows = 0;
+};
+
+// Mamba-2 over one packed projection row [.. z | .. x, B, C .. | dt ..]: x (heads x dv), B and C (groups x dk each) follow one another at
+// x_at, pass a causal convolution of `taps` taps per channel with a bias, and silu. Per head a state S [dk, dv]; head h uses group
+// h / (heads / groups):
+//   dt = softplus(dt_t + dt_bias_h),  S_t = exp(-exp(a_log_h) dt) S_{t-1} + dt B_t x_t^T,  y_t = S_t^T C_t + d_skip_h x_t
+// out = norm_w * rms_norm(y * silu(z)), the norm in norm_groups equal parts of the heads' concatenated outputs.
+struct StateSpaceArgs {
+    const void *proj = nullptr; // [n_rows, row_stride], model dtype
+    int64_t row_stride = 0;
+    int64_t z_at = 0, x_at = 0, dt_at = 0;
+    const void *conv_w = nullptr, *conv_b = nullptr; // [channels, taps] (the last tap is the current token's), [channels]
+    const void *norm_w = nullptr;                    // [heads * dv]
+    const float *a_log = nullptr, *dt_bias = nullptr, *d_skip = nullptr; // [heads]
+    int32_t taps = 0, heads = 0, groups = 0, dk = 0, dv = 0, norm_groups = 1;
+    float eps = 0.f;
+    // slot s: the heads' matrices [heads][dk][dv], then convolution inputs [taps][channels]: position p at p mod taps
+    float *state = nullptr;
+    int64_t slot_stride = 0;
+    // the batch: sequence i owns rows [q_starts[i], q_starts[i + 1]) and state slot seq_ids[i]; kv_lens[i] tokens after the
+    // step (a sequence whose first token is in the step starts from zero)
+    const int32_t *seq_ids = nullptr, *q_starts = nullptr, *kv_lens = nullptr;
+    int32_t n_seqs = 0, n_rows = 0, max_q_len = 0;
+    void *out = nullptr; // row r: out + r * out_stride, [heads * dv], model dtype
+    int64_t out_stride = 0;
+    float *scratch = nullptr; // state_space_scratch_floats, 16-byte aligned
+    size_t scratch_floats = 0;
+    float *segments = nullptr; // state_space_segment_floats; null: runs are never cut
+    size_t segment_floats = 0;
+    LLAISYS_ARGS_FN int32_t inner() const { return heads * dv; }
+    LLAISYS_ARGS_FN int32_t channels() const { return heads * dv + 2 * groups * dk; }
+};
+
+// Mixture of experts over rows h [n_rows, width]. The router's logits become scores s = softmax over experts + identity outputs;
+// `top` of them are chosen by s + correction, among the best `keep` of `groups` equal groups (a group counts as much as its best
+// choice score); weight of a chosen one: scale * s / (sum of the chosen s + 1e-20). Expert e: down_e (silu(gate_e h) * up_e h);
+// outputs from `experts` on are identity experts: h itself.
+struct ExpertArgs {
+    int32_t experts = 0, identity = 0, top = 0, groups = 1, keep = 1;
+    float scale = 1.f;
+    int32_t width = 0, ff = 0;        // ff: padded rows per expert of `gate_up` halves, columns of `down`
+    const void *gate_up = nullptr;    // [experts][2 ff][width]: gate rows, then up rows
+    const void *down = nullptr;       // [experts][width][ff]
+    const float *correction = nullptr; // [experts + identity]
+    const float *logits = nullptr;    // [n_rows, experts + identity]
+    const void *h = nullptr;          // [n_rows, width], model dtype
+    int32_t n_rows = 0;
+    // routing (written by experts_route): per row `top` choices; rows of every expert in one line, expert after expert
+    int32_t *chosen = nullptr;  // [n_rows, top] expert
+    float *weights = nullptr;   // [n_rows, top]
+    int32_t *place = nullptr;   // [n_rows, top] row in the line (after experts_place); -1 for an identity expert
+    int32_t *counts = nullptr;  // [experts] rows of every expert, zero before experts_route
+    int32_t *line = nullptr;    // [n_rows * top] source row of every row in the line
+    void *rows = nullptr;       // [n_rows * top, width] the line's inputs (tensor-core form)
+    void *act = nullptr;        // [n_rows * top, ff]
+    void *out = nullptr;        // [n_rows * top, width]
 };
 
 // Gated linear attention over one packed projection (per head a state S [dk, dv], decayed per key channel):

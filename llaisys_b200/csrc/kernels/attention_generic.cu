@@ -1,4 +1,4 @@
-// Generic attention over a paged or contiguous K/V view: any of F32 / F16 / BF16, V rows of up to 256, any GQA
+// Generic attention over a paged or contiguous K/V view: any of F32 / F16 / BF16, V rows of up to 1024, any GQA
 // ratio, any page size, decode or ragged causal chunks.
 //
 // One CTA of four warps per (query row, query head). Keys are dealt to warps in blocks of 32; inside a warp
@@ -18,9 +18,9 @@ namespace llaisys::kernels {
 namespace {
 
 constexpr int kWarps = 4;
-constexpr int kMaxDimsPerLane = 8; // head_dim <= 256
+constexpr int kDimsPerLane = 8, kMostDimsPerLane = 32; // V rows of up to 256, and of up to 1024
 
-template <typename T>
+template <typename T, int kMaxDimsPerLane>
 __global__ void __launch_bounds__(kWarps * 32)
     attention_generic_kernel(KVView kv, AttnBatch batch, const T *__restrict__ q, float scale, T *__restrict__ out,
                              float *__restrict__ part, const float *__restrict__ row_scale, int64_t out_stride,
@@ -64,6 +64,7 @@ __global__ void __launch_bounds__(kWarps * 32)
     const int kept = min(batch.keep_first, first), gap = first - kept;
     const int seq_row = batch.seq_ids ? batch.seq_ids[seq] : seq;
     const int kvh = h / (batch.nh / kv.nkvh);
+    const float fade_a = batch.fade_a != nullptr ? batch.fade_a[h] : 0.f, fade_b = batch.fade_a != nullptr ? batch.fade_b[h] : 0.f;
 
     const T *q_row = q + (int64_t(row) * batch.nh + h) * d;
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
@@ -107,7 +108,7 @@ __global__ void __launch_bounds__(kWarps * 32)
             for (int i = 0; i < d; ++i) {
                 dot = fmaf(q_s[i], to_f32(k_row[i]), dot);
             }
-            s = dot;
+            s = fade_a == 0.f ? dot : dot - fade_a * log1pf(fade_b * float(visible - 1 - j));
         }
         float mx = s;
 #pragma unroll
@@ -201,10 +202,9 @@ void launch(cudaStream_t s, const KVView &kv, const AttnBatch &batch, const void
             int32_t *error_flag) {
     const dim3 grid(unsigned(batch.total_q), unsigned(batch.nh));
     const size_t smem = (size_t(kv.d) + size_t(kv.vDim()) * kWarps + 2 * kWarps) * sizeof(float);
-    attention_generic_kernel<T><<<grid, kWarps * 32, smem, s>>>(kv, batch, static_cast<const T *>(q), scale,
-                                                                static_cast<T *>(out.out), out.part, out.row_scale,
-                                                                out.row_stride ? out.row_stride : int64_t(batch.nh) * kv.vDim(),
-                                                                error_flag);
+    auto kernel = kv.vDim() <= 32 * kDimsPerLane ? attention_generic_kernel<T, kDimsPerLane> : attention_generic_kernel<T, kMostDimsPerLane>;
+    kernel<<<grid, kWarps * 32, smem, s>>>(kv, batch, static_cast<const T *>(q), scale, static_cast<T *>(out.out), out.part, out.row_scale,
+                                           out.row_stride ? out.row_stride : int64_t(batch.nh) * kv.vDim(), error_flag);
 }
 
 } // namespace
@@ -214,8 +214,8 @@ void attention_generic(stream_t stream, llaisysDataType_t dtype, const KVView &k
     if (batch.total_q <= 0 || batch.nh <= 0) {
         return;
     }
-    CHECK_ARGUMENT(kv.d > 0 && kv.d <= 8192 && kv.vDim() > 0 && kv.vDim() <= 32 * kMaxDimsPerLane,
-                   "attention: V rows must have 1 to 256 elements, K rows at most 8192");
+    CHECK_ARGUMENT(kv.d > 0 && kv.d <= 8192 && kv.vDim() > 0 && kv.vDim() <= 32 * kMostDimsPerLane,
+                   "attention: V rows must have 1 to 1024 elements, K rows at most 8192");
     CHECK_ARGUMENT(kv.nkvh > 0 && batch.nh % kv.nkvh == 0, "attention: nh must be a multiple of nkvh");
     CHECK_ARGUMENT(batch.nh <= 65535, "attention: too many heads for one launch");
     auto s = static_cast<cudaStream_t>(stream);

@@ -89,6 +89,36 @@ void paged_rope_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
 void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const NormAppendArgs &args,
                        int32_t max_blocks, int32_t *error_flag);
 
+// K1d (see LatentAppendArgs); same addressing and flags as K1.
+void latent_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const LatentAppendArgs &args, int32_t max_blocks,
+                   int32_t *error_flag);
+// The dims behind the first `dim` of every head of q [n_rows, nh, dim + rot_dims] turn by the row's position (dims 2 i and 2 i + 1 by
+// rot_table[row][i]) -> the same elements of out rows of out_dim behind the first out_at: out [n_rows, nh, out_dim]. out may be q.
+void rotate_pairs(stream_t stream, llaisysDataType_t dtype, void *out, size_t out_dim, size_t out_at, const void *q, size_t dim, size_t rot_dims,
+                  const float *rot_table, size_t n_rows, size_t nh);
+// nh products side by side: out[r, h, :n] = in[r, h, :k] . W_h^T, W_h [n, k] at weight + h * n * k (transposed = false) or W_h^T stored
+// [k, n] there (transposed = true). Strides in elements: between rows and between heads of `in` and `out`. f32 accumulation.
+void linear_heads(stream_t stream, llaisysDataType_t dtype, void *out, const void *in, const void *weight, size_t rows, size_t nh, size_t n,
+                  size_t k, bool transposed, size_t in_row, size_t in_head, size_t out_row, size_t out_head);
+
+// Mamba-2 (see StateSpaceArgs). decode: one token per sequence. chunk: ragged runs of tokens.
+void state_space_decode(stream_t stream, llaisysDataType_t dtype, const StateSpaceArgs &args);
+void state_space_chunk(stream_t stream, llaisysDataType_t dtype, const StateSpaceArgs &args);
+// Floats of one sequence's state, of StateSpaceArgs::scratch for n_rows rows and of StateSpaceArgs::segments (0: never cut).
+size_t state_space_state_floats(size_t heads, size_t groups, size_t dk, size_t dv, size_t taps);
+size_t state_space_scratch_floats(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t groups, size_t dk, size_t dv);
+size_t state_space_segment_floats(llaisysDataType_t dtype, size_t heads, size_t dk, size_t dv);
+
+// Mixture of experts (see ExpertArgs). route: scores, choice, weights, every choice's place among its expert's rows. apply: the
+// chosen experts' outputs, a row each, in args.out. combine: x[r, :] += the weighted sum of row r's choices; next (may be null): what
+// becomes dtype(rms_norm(x) * *gain) of the new x (args.h is a good place: rows are read before they are written).
+void experts_route(stream_t stream, llaisysDataType_t dtype, const ExpertArgs &args);
+void experts_apply(stream_t stream, llaisysDataType_t dtype, const ExpertArgs &args);
+void experts_combine(stream_t stream, llaisysDataType_t dtype, const ExpertArgs &args, float *x, void *next, const float *gain, float eps);
+// The tcgen05 form behind experts_apply: 16-bit, width and ff in whole 16-byte pieces.
+bool experts_tc_covers(llaisysDataType_t dtype, const ExpertArgs &args);
+void experts_tc(stream_t stream, llaisysDataType_t dtype, const ExpertArgs &args); // after experts_route and the placing of rows
+
 // Gated delta rule (see GatedDeltaArgs). decode: one token per sequence, everything in one launch. chunk: ragged runs of
 // tokens.
 void gated_delta_decode(stream_t stream, llaisysDataType_t dtype, const GatedDeltaArgs &args);
@@ -128,6 +158,9 @@ void stream_cast(stream_t stream, llaisysDataType_t dtype, void *out, int64_t ou
 // weight stored around zero
 void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
                      const void *w, float eps, size_t rows, size_t d, float offset = 0.f);
+// the same with one number (f32, on the device) for all columns: out[i, :] = rms_norm(x[r, :]) * *gain
+void stream_rms_norm_gain(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
+                          const float *gain, float eps, size_t rows, size_t d);
 // out (f32) = alpha * in . W^T (+ out when accumulate): a projection into the stream, or logits
 void linear_f32(stream_t stream, llaisysDataType_t dtype, float *out, const void *in, const void *weight, size_t m, size_t n,
                 size_t k, bool accumulate, float alpha = 1.f, size_t in_stride = 0);
@@ -143,6 +176,8 @@ void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const
                        float branch_offset = 0.f);
 // table[r, i] = (cos, sin)(positions[r] * freq[i]), i < half
 void rotary_table(stream_t stream, float *table, const int32_t *positions, const float *freq, size_t rows, size_t half);
+// the same with angles in f64, reduced to a turn before they are rounded
+void rotary_table(stream_t stream, float *table, const int32_t *positions, const double *freq, size_t rows, size_t half);
 // logits = cap * tanh(logits / cap) in place (cap <= 0: unchanged) and the row-wise argmax of the result, one launch;
 // scratch as argmax_rows_split
 void softcap_argmax(stream_t stream, float *logits, float cap, int64_t *idx_out, size_t rows, size_t n, void *scratch);

@@ -27,6 +27,9 @@ struct CublasApi {
     cublasStatus_t (*gemm_ex)(cublasHandle_t, cublasOperation_t, cublasOperation_t, int, int, int, const void *, const void *,
                               cudaDataType, int, const void *, cudaDataType, int, const void *, void *, cudaDataType, int,
                               cublasComputeType_t, cublasGemmAlgo_t) = nullptr;
+    cublasStatus_t (*gemm_strided)(cublasHandle_t, cublasOperation_t, cublasOperation_t, int, int, int, const void *, const void *, cudaDataType,
+                                   int, long long, const void *, cudaDataType, int, long long, const void *, void *, cudaDataType, int, long long,
+                                   int, cublasComputeType_t, cublasGemmAlgo_t) = nullptr;
     bool ok = false;
 };
 
@@ -46,7 +49,8 @@ const CublasApi &cublas_api() {
         a.create = reinterpret_cast<decltype(a.create)>(dlsym(lib, "cublasCreate_v2"));
         a.set_stream = reinterpret_cast<decltype(a.set_stream)>(dlsym(lib, "cublasSetStream_v2"));
         a.gemm_ex = reinterpret_cast<decltype(a.gemm_ex)>(dlsym(lib, "cublasGemmEx"));
-        a.ok = a.create != nullptr && a.set_stream != nullptr && a.gemm_ex != nullptr;
+        a.gemm_strided = reinterpret_cast<decltype(a.gemm_strided)>(dlsym(lib, "cublasGemmStridedBatchedEx"));
+        a.ok = a.create != nullptr && a.set_stream != nullptr && a.gemm_ex != nullptr && a.gemm_strided != nullptr;
         return a;
     }();
     return api;
@@ -143,6 +147,23 @@ void linear_f32(stream_t stream, llaisysDataType_t dtype, float *out, const void
         return;
     }
     gemm(stream, dtype, LLAISYS_DTYPE_F32, out, in, weight, m, n, k, in_stride == 0 ? k : in_stride, n, alpha, accumulate ? 1.f : 0.f);
+}
+
+void linear_heads(stream_t stream, llaisysDataType_t dtype, void *out, const void *in, const void *weight, size_t rows, size_t nh, size_t n,
+                  size_t k, bool transposed, size_t in_row, size_t in_head, size_t out_row, size_t out_head) {
+    if (rows == 0 || nh == 0 || n == 0) {
+        return;
+    }
+    ASSERT(cublas_api().ok, "linear on NVIDIA needs cuBLAS (libcublas.so.12 was not found)");
+    const cudaDataType type = cuda_type(dtype);
+    cublasHandle_t h = handle_for_current_device();
+    cublasStatus_t st = cublas_api().set_stream(h, static_cast<cudaStream_t>(stream));
+    ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasSetStream failed with status " << int(st));
+    const float alpha = 1.f, beta = 0.f;
+    st = cublas_api().gemm_strided(h, transposed ? CUBLAS_OP_N : CUBLAS_OP_T, CUBLAS_OP_N, int(n), int(rows), int(k), &alpha, weight, type,
+                                   int(transposed ? n : k), (long long)(n * k), in, type, int(in_row), (long long)in_head, &beta, out, type,
+                                   int(out_row), (long long)out_head, int(nh), CUBLAS_COMPUTE_32F, CUBLAS_GEMM_DEFAULT);
+    ASSERT(st == CUBLAS_STATUS_SUCCESS, "cublasGemmStridedBatchedEx failed with status " << int(st));
 }
 
 } // namespace llaisys::kernels

@@ -8,8 +8,7 @@
 //
 // Roofline: HBM. Algorithmic bytes per row = 2 * (2 * nkvh * d * elem_size) (read the new K and V row, write
 // them) + 8 (sequence id and position) + 4 (table entry).
-#include "device_utils.cuh"
-#include "kernels.hpp"
+#include "launch_utils.cuh"
 
 #include <algorithm>
 
@@ -308,15 +307,15 @@ __global__ void paged_rope_append_kernel(unsigned char *__restrict__ k_pool, uns
     }
 }
 
-// Elements [at, at + VEC) of a q or k head row after norm (inv, w; w null: none) and rotation: the partners across the rotated
+// Elements [at, at + VEC) of a q or k head row after norm (inv, w; w null: none), rotation and a factor: the partners across the rotated
 // range are read from the row itself. VEC divides rot_dims / 2, so a piece lies in one half.
 template <typename T, int VEC>
 __device__ __forceinline__ Pack<T, VEC> norm_rotate(Pack<T, VEC> x, const T *src, int32_t at, float inv, const T *w,
-                                                    const NormAppendArgs &a, int64_t row) {
+                                                    const NormAppendArgs &a, int64_t row, float factor) {
     using P = Pack<T, VEC>;
     const int32_t half = a.rot_dims / 2;
     const bool turns = at < a.rot_dims;
-    if (w == nullptr && !turns) {
+    if (w == nullptr && !turns && factor == 1.f) {
         return x;
     }
     float f[VEC];
@@ -348,7 +347,7 @@ __device__ __forceinline__ Pack<T, VEC> norm_rotate(Pack<T, VEC> x, const T *src
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-        x.v[e] = from_f32<T>(f[e]);
+        x.v[e] = from_f32<T>(f[e] * factor);
     }
     return x;
 }
@@ -416,7 +415,7 @@ __global__ void __launch_bounds__(256)
     for (int32_t i = lane * VEC; i < n; i += 32 * VEC) {
         P x = *reinterpret_cast<const P *>(src + i);
         if (!is_v) {
-            x = norm_rotate<T, VEC>(x, src, i, inv, w, a, row);
+            x = norm_rotate<T, VEC>(x, src, i, inv, w, a, row, is_q && a.head_scale != nullptr ? a.head_scale[head] : 1.f);
         }
         *reinterpret_cast<P *>(dst + i) = x;
     }
@@ -477,7 +476,7 @@ __global__ void __launch_bounds__(256)
             const T *src = static_cast<const T *>(a.proj) + int64_t(row[u]) * a.row_stride +
                            (is_q ? a.q_at + int64_t(head[u]) * d : a.k_at + int64_t(head[u] - a.nh) * d);
             x[u] = norm_rotate<T, VEC>(x[u], src, at, rsqrtf(ss[u] / float(d) + a.eps), static_cast<const T *>(is_q ? a.q_norm : a.k_norm), a,
-                                       row[u]);
+                                       row[u], is_q && a.head_scale != nullptr ? a.head_scale[head[u]] : 1.f);
         }
         if (is_q) {
             *reinterpret_cast<P *>(static_cast<T *>(a.q_out) + (int64_t(row[u]) * a.nh + head[u]) * d + at) = x[u];
@@ -621,6 +620,81 @@ __global__ void paged_row_norm_append_kernel(unsigned char *__restrict__ k_pool,
     }
 }
 
+// K1d: one CTA per row (see LatentAppendArgs).
+template <typename T>
+__global__ void __launch_bounds__(256) latent_append_kernel(T *__restrict__ k_pool, LatentAppendArgs a, const int32_t *__restrict__ table,
+                                                            CopyGeom g, int32_t max_blocks, int32_t *error_flag) {
+    asm volatile("griddepcontrol.wait;\n" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    const int64_t row = blockIdx.x;
+    const int32_t tid = int32_t(threadIdx.x), step = int32_t(blockDim.x);
+    const T *proj = static_cast<const T *>(a.proj) + row * a.row_stride;
+    const T *q = proj + a.q_at, *kv = proj + a.kv_at;
+    float sq = 0.f, sk = 0.f;
+    for (int32_t i = tid; i < a.q_rank; i += step) {
+        sq = fmaf(to_f32(q[i]), to_f32(q[i]), sq);
+    }
+    for (int32_t i = tid; i < a.rank; i += step) {
+        sk = fmaf(to_f32(kv[i]), to_f32(kv[i]), sk);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    __shared__ float part_q[8], part_k[8];
+    if ((tid & 31) == 0) {
+        part_q[tid >> 5] = sq;
+        part_k[tid >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int32_t i = 0; i < step >> 5; ++i) { // every thread sums the few partials in the same order
+        sq += part_q[i];
+        sk += part_k[i];
+    }
+    const float inv_q = rsqrtf(sq / float(a.q_rank) + a.eps), inv_k = rsqrtf(sk / float(a.rank) + a.eps);
+    const T *q_norm = static_cast<const T *>(a.q_norm), *kv_norm = static_cast<const T *>(a.kv_norm);
+    T *q_out = static_cast<T *>(a.q_latent) + row * a.q_latent_stride;
+    for (int32_t i = tid; i < a.q_rank; i += step) {
+        q_out[i] = from_f32<T>(to_f32(q[i]) * inv_q * to_f32(q_norm[i]));
+    }
+    if (a.row_scale != nullptr) {
+        for (int32_t h = tid; h < a.nh; h += step) {
+            a.row_scale[row * a.nh + h] = a.gate_at < 0 ? 1.f : 1.f / (1.f + expf(-to_f32(proj[a.gate_at + h])));
+        }
+    }
+    int32_t page, slot;
+    if (!resolve_slot(table, g, a.seq_ids[row], a.positions[row], max_blocks, error_flag, page, slot)) {
+        return;
+    }
+    T *dst = k_pool + int64_t(page) * (g.page_stride_b / int64_t(sizeof(T))) + int64_t(slot) * (g.token_stride_b / int64_t(sizeof(T)));
+    for (int32_t i = tid; i < a.rank; i += step) {
+        dst[i] = from_f32<T>(to_f32(kv[i]) * inv_k * to_f32(kv_norm[i]));
+    }
+    const float2 *turn = reinterpret_cast<const float2 *>(a.rot_table) + row * (a.rot_dims / 2);
+    for (int32_t i = tid; i < a.rot_dims / 2; i += step) {
+        const float u = to_f32(kv[a.rank + 2 * i]), v = to_f32(kv[a.rank + 2 * i + 1]);
+        const float2 t = turn[i];
+        dst[a.rank + 2 * i] = from_f32<T>(u * t.x - v * t.y);
+        dst[a.rank + 2 * i + 1] = from_f32<T>(v * t.x + u * t.y);
+    }
+}
+
+template <typename T>
+void launch_latent_append(cudaStream_t s, const KVView &kv, const LatentAppendArgs &a, int32_t max_blocks, int32_t *error_flag) {
+    CopyGeom g{};
+    g.page_stride_b = kv.page_stride * int64_t(sizeof(T));
+    g.token_stride_b = kv.token_stride * int64_t(sizeof(T));
+    g.nkvh = 1;
+    g.page_size = kv.page_size;
+    g.num_pages = kv.num_pages;
+    g.table_stride = kv.table_stride;
+    const int32_t longest = std::max(a.q_rank, a.rank);
+    launch_programmatic(latent_append_kernel<T>, dim3(unsigned(a.n_rows)), longest <= 256 ? 64u : (longest <= 1024 ? 128u : 256u), s,
+                        static_cast<T *>(kv.k_base), a, kv.block_table, g, max_blocks, error_flag);
+}
+
 template <typename T>
 void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &a, int32_t max_blocks, int32_t *error_flag) {
     CopyGeom g{};
@@ -642,8 +716,8 @@ void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &
     cfg.attrs = &attr;
     cfg.numAttrs = 1;
     if (a.row_norm != 0) {
-        CHECK_ARGUMENT(a.rot_dims == 0 && a.gate_at < 0 && a.row_scale == nullptr && a.temp_every > 0.f,
-                       "norm append: the row form takes neither a rotation nor a gate");
+        CHECK_ARGUMENT(a.rot_dims == 0 && a.gate_at < 0 && a.row_scale == nullptr && a.head_scale == nullptr && a.temp_every > 0.f,
+                       "norm append: the row form takes neither a rotation, a gate nor factors per head");
         constexpr int kRow = 16 / int(sizeof(T));
         const bool pieces = d % kRow == 0 && dv % kRow == 0 && a.row_stride % kRow == 0 && a.q_at % kRow == 0 && a.k_at % kRow == 0 &&
                             a.v_at % kRow == 0 && aligned(a.proj) && aligned(a.bias) && aligned(a.q_norm) && aligned(a.k_norm) && aligned(a.q_out);
@@ -853,6 +927,16 @@ void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
         EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
     }
     check_launch("paged_norm_append");
+}
+
+void latent_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const LatentAppendArgs &args, int32_t max_blocks,
+                   int32_t *error_flag) {
+    if (args.n_rows == 0) {
+        return;
+    }
+    CHECK_ARGUMENT(args.q_rank > 0 && args.rank > 0 && args.rot_dims % 2 == 0 && kv.nkvh == 1, "latent append: bad sizes");
+    dispatch(dtype, [&](auto tag) { launch_latent_append<decltype(tag)>(static_cast<cudaStream_t>(stream), kv, args, max_blocks, error_flag); });
+    check_launch("latent_append");
 }
 
 } // namespace llaisys::kernels

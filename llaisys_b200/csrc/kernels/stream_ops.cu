@@ -1,11 +1,8 @@
 // Operators of a decoder whose residual stream stays in f32 between layers: the embedding with its scale, the norm that
 // turns stream rows into activations, the cast that feeds the stream to a projection, the squared-relu activation and the
 // soft cap of the logits with the greedy choice behind it. All HBM-bound, one pass over their data.
-#include "device_utils.cuh"
-#include "kernels.hpp"
+#include "launch_utils.cuh"
 #include "mma_utils.cuh"
-
-#include <utility>
 
 namespace llaisys::kernels {
 
@@ -15,22 +12,6 @@ template <typename T, int N>
 struct alignas(sizeof(T) * N) Vec {
     T v[N];
 };
-
-// Programmatic launch: every kernel below waits for its predecessor before it touches anything, then lets its successor be
-// scheduled, so that a launch hides under the kernel before it (see rms_norm_vec_kernel).
-template <typename... KArgs, typename... Args>
-void launch_programmatic(void (*kernel)(KArgs...), dim3 grid, unsigned block, cudaStream_t s, Args &&...args) {
-    cudaLaunchConfig_t cfg{};
-    cfg.gridDim = grid;
-    cfg.blockDim = dim3(block);
-    cfg.stream = s;
-    cudaLaunchAttribute attr{};
-    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr.val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = &attr;
-    cfg.numAttrs = 1;
-    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, KArgs(std::forward<Args>(args))...));
-}
 
 template <typename T, int VEC>
 __global__ void embed_scaled_kernel(float *__restrict__ x, T *__restrict__ copy, int64_t copy_stride,
@@ -124,7 +105,7 @@ __global__ void stream_cast_kernel(T *__restrict__ out, int64_t out_stride, cons
 // has beyond them is read again.
 template <typename T, int VEC, int PER_THREAD>
 __global__ void stream_rms_norm_kernel(T *__restrict__ out, const float *__restrict__ x, const int64_t *__restrict__ row_index,
-                                       const T *__restrict__ w, float eps, int32_t d, float offset) {
+                                       const T *__restrict__ w, const float *__restrict__ gain, float eps, int32_t d, float offset) {
     grid_dependency_wait();
     grid_launch_dependents();
     using F = Vec<float, VEC>;
@@ -164,14 +145,21 @@ __global__ void stream_rms_norm_kernel(T *__restrict__ out, const float *__restr
     for (int i = 0; i < int(blockDim.x >> 5); ++i) {
         tot += s_part[i]; // every thread sums the few partials in the same order
     }
-    const float inv = rsqrtf(tot / float(d) + eps);
+    const float inv = rsqrtf(tot / float(d) + eps) * (w == nullptr ? *gain : 1.f);
     T *dst = out + int64_t(blockIdx.x) * d;
     auto store = [&](int32_t i, const F &f) {
-        const Vec<T, VEC> ww = *reinterpret_cast<const Vec<T, VEC> *>(w + int64_t(i) * VEC);
         Vec<T, VEC> o;
+        if (w == nullptr) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            o.v[e] = from_f32<T>(f.v[e] * inv * (offset + to_f32(ww.v[e])));
+            for (int e = 0; e < VEC; ++e) {
+                o.v[e] = from_f32<T>(f.v[e] * inv);
+            }
+        } else {
+            const Vec<T, VEC> ww = *reinterpret_cast<const Vec<T, VEC> *>(w + int64_t(i) * VEC);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                o.v[e] = from_f32<T>(f.v[e] * inv * (offset + to_f32(ww.v[e])));
+            }
         }
         *reinterpret_cast<Vec<T, VEC> *>(dst + int64_t(i) * VEC) = o;
     };
@@ -342,6 +330,42 @@ __global__ void rotary_table_kernel(float2 *__restrict__ table, const int32_t *_
     }
 }
 
+// The angle in f64, reduced there, so that far positions lose nothing.
+__global__ void rotary_table_wide_kernel(float2 *__restrict__ table, const int32_t *__restrict__ positions, const double *__restrict__ freq,
+                                         int32_t half, int64_t total) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    constexpr double kTurn = 6.283185307179586;
+    const int64_t at = int64_t(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (at < total) {
+        const int64_t row = at / half;
+        const double angle = double(positions[row]) * freq[at - row * half];
+        float s, c;
+        sincosf(float(fma(-kTurn, rint(angle * (1.0 / kTurn)), angle)), &s, &c);
+        table[at] = make_float2(c, s);
+    }
+}
+
+// One thread per pair of a head
+template <typename T>
+__global__ void rotate_pairs_kernel(T *out, int64_t out_dim, int64_t out_at, const T *q, int32_t dim, int32_t half,
+                                    const float2 *__restrict__ table, int32_t nh, int64_t total) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t at = int64_t(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (at >= total) {
+        return;
+    }
+    const int64_t head = at / half, row = head / nh; // head: of all rows
+    const int32_t i = int32_t(at - head * half);
+    const T *src = q + head * (dim + 2 * half) + dim + 2 * i;
+    const float u = to_f32(src[0]), v = to_f32(src[1]);
+    const float2 t = table[row * half + i];
+    T *dst = out + head * out_dim + out_at + 2 * i;
+    dst[0] = from_f32<T>(u * t.x - v * t.y);
+    dst[1] = from_f32<T>(v * t.x + u * t.y);
+}
+
 template <typename T, int VEC>
 __global__ void relu_squared_kernel(T *__restrict__ v, size_t n_vec) {
     grid_dependency_wait();
@@ -412,25 +436,6 @@ unsigned block_for(size_t n_vec, size_t per_thread) {
     const size_t block = (want + 31) / 32 * 32;
     return unsigned(block < 64 ? 64 : (block > 1024 ? 1024 : block));
 }
-bool aligned16(const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
-
-template <typename F>
-void dispatch(llaisysDataType_t dtype, F &&body) {
-    switch (dtype) {
-    case LLAISYS_DTYPE_F32:
-        body(float{});
-        break;
-    case LLAISYS_DTYPE_F16:
-        body(__half{});
-        break;
-    case LLAISYS_DTYPE_BF16:
-        body(__nv_bfloat16{});
-        break;
-    default:
-        EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
-    }
-}
-
 } // namespace
 
 void embed_scaled(stream_t stream, llaisysDataType_t dtype, float *x, void *copy, int64_t copy_stride, const int64_t *tokens,
@@ -506,9 +511,25 @@ void stream_rms_norm(stream_t stream, llaisysDataType_t dtype, void *out, const 
         const bool wide = d % 4 == 0 && aligned16(x) && aligned16(out) && aligned16(w);
         auto kernel = wide ? stream_rms_norm_kernel<T, 4, 4> : stream_rms_norm_kernel<T, 1, 4>;
         launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, static_cast<T *>(out), x, row_index,
-                            static_cast<const T *>(w), eps, int32_t(d), offset);
+                            static_cast<const T *>(w), nullptr, eps, int32_t(d), offset);
     });
     check_launch("stream_rms_norm");
+}
+
+void stream_rms_norm_gain(stream_t stream, llaisysDataType_t dtype, void *out, const float *x, const int64_t *row_index,
+                          const float *gain, float eps, size_t rows, size_t d) {
+    if (rows == 0 || d == 0) {
+        return;
+    }
+    auto s = static_cast<cudaStream_t>(stream);
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        const bool wide = d % 4 == 0 && aligned16(x) && aligned16(out);
+        auto kernel = wide ? stream_rms_norm_kernel<T, 4, 4> : stream_rms_norm_kernel<T, 1, 4>;
+        launch_programmatic(kernel, dim3(unsigned(rows)), block_for(wide ? d / 4 : d, 2), s, static_cast<T *>(out), x, row_index,
+                            nullptr, gain, eps, int32_t(d), 0.f);
+    });
+    check_launch("stream_rms_norm_gain");
 }
 
 void stream_add_normed(stream_t stream, llaisysDataType_t dtype, float *x, const float *a, const void *wa, const float *b,
@@ -562,6 +583,31 @@ void rotary_table(stream_t stream, float *table, const int32_t *positions, const
     launch_programmatic(rotary_table_kernel, dim3(unsigned((total + 255) / 256)), 256u, static_cast<cudaStream_t>(stream),
                         reinterpret_cast<float2 *>(table), positions, freq, int32_t(half), total);
     check_launch("rotary_table");
+}
+
+void rotary_table(stream_t stream, float *table, const int32_t *positions, const double *freq, size_t rows, size_t half) {
+    if (rows == 0 || half == 0) {
+        return;
+    }
+    const int64_t total = int64_t(rows) * int64_t(half);
+    launch_programmatic(rotary_table_wide_kernel, dim3(unsigned((total + 255) / 256)), 256u, static_cast<cudaStream_t>(stream),
+                        reinterpret_cast<float2 *>(table), positions, freq, int32_t(half), total);
+    check_launch("rotary_table");
+}
+
+void rotate_pairs(stream_t stream, llaisysDataType_t dtype, void *out, size_t out_dim, size_t out_at, const void *q, size_t dim, size_t rot_dims,
+                  const float *rot_table, size_t n_rows, size_t nh) {
+    const int64_t half = int64_t(rot_dims / 2), total = int64_t(n_rows) * int64_t(nh) * half;
+    if (total == 0) {
+        return;
+    }
+    dispatch(dtype, [&](auto tag) {
+        using T = decltype(tag);
+        launch_programmatic(rotate_pairs_kernel<T>, dim3(unsigned((total + 255) / 256)), 256u, static_cast<cudaStream_t>(stream),
+                            static_cast<T *>(out), int64_t(out_dim), int64_t(out_at), static_cast<const T *>(q), int32_t(dim), int32_t(half),
+                            reinterpret_cast<const float2 *>(rot_table), int32_t(nh), total);
+    });
+    check_launch("rotate_pairs");
 }
 
 void relu_squared(stream_t stream, llaisysDataType_t dtype, void *v, size_t n) {

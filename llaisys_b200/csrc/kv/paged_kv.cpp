@@ -39,6 +39,8 @@ void setWindow(kernels::AttnBatch &b, const PagedKVConfig &cfg, const AttnOption
     const size_t longest = cfg.page_size * cfg.max_pages_per_seq;
     b.window = int32_t(std::min(opt.window, longest));
     b.keep_first = opt.window != 0 ? int32_t(std::min(opt.keep_first, longest)) : 0;
+    b.fade_a = opt.fade_a;
+    b.fade_b = opt.fade_b;
 }
 constexpr size_t kMaxDecodeSeqs = 1024; // sequences per launch of the TMA decode kernel
 
@@ -65,12 +67,13 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
     size_t pool_bytes = 0, max_kvh = 0;
     for (const KVLayerShape &shape : _cfg.layers) {
         KV_REQUIRE(shape.nkvh > 0 && shape.k_dim > 0 && shape.v_dim > 0, LLAISYS_E_INVALID, "paged KV: every size must be positive");
+        KV_REQUIRE(!shape.v_in_k || shape.v_dim <= shape.k_dim, LLAISYS_E_INVALID, "paged KV: V rows inside K rows cannot be longer");
         Layer l;
         l.nkvh = shape.nkvh;
         l.k_dim = shape.k_dim;
         l.v_dim = shape.v_dim;
         l.k_row = (l.k_dim + align - 1) / align * align;
-        l.v_row = (l.v_dim + align - 1) / align * align;
+        l.v_row = shape.v_in_k ? 0 : (l.v_dim + align - 1) / align * align;
         l.page_elems = l.nkvh * cfg.page_size * (l.k_row + l.v_row);
         l.offset = pool_bytes;
         l.bytes = cfg.num_pages * l.page_elems * _elem;
@@ -101,7 +104,7 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
         rt.synchronize();
         bool any_tma = false;
         for (Layer &l : _layers) {
-            if (_elem != 2 || l.k_dim != 128 || l.v_dim != 128 || cfg.page_size != 16) {
+            if (_elem != 2 || l.k_dim != 128 || l.v_dim != 128 || l.v_row == 0 || cfg.page_size != 16) {
                 continue;
             }
             // one row of 128 elements per (page, K|V, kv-head, slot)
@@ -456,19 +459,20 @@ void PagedKV::checkLayer(size_t layer) const {
 }
 
 void PagedKV::requireEqualRows(size_t layer, const char *what) const {
-    KV_REQUIRE(_layers[layer].k_dim == _layers[layer].v_dim && _layers[layer].k_dim == _layers[layer].k_row, LLAISYS_E_UNSUPPORTED,
+    KV_REQUIRE(_layers[layer].k_dim == _layers[layer].v_dim && _layers[layer].k_dim == _layers[layer].k_row && _layers[layer].v_row != 0, LLAISYS_E_UNSUPPORTED,
                "paged KV ", what, ": this layer's K and V rows differ in length or are padded");
 }
 
 void PagedKV::requirePlain(size_t layer, const AttnOptions &opt) const {
     requireEqualRows(layer, "attention on the CPU");
-    KV_REQUIRE(opt.window == 0 && opt.row_scale == nullptr && opt.row_stride == 0 && opt.gates == nullptr, LLAISYS_E_UNSUPPORTED,
-               "paged attention: windows, output scales and gated weights on NVIDIA caches only");
+    KV_REQUIRE(opt.window == 0 && opt.row_scale == nullptr && opt.row_stride == 0 && opt.gates == nullptr && opt.fade_a == nullptr, LLAISYS_E_UNSUPPORTED,
+               "paged attention: windows, penalties, output scales and gated weights on NVIDIA caches only");
 }
 
 void PagedKV::requireGates(const AttnOptions &opt) const {
-    KV_REQUIRE(opt.gates == nullptr || (opt.keep_first == 0 && opt.row_scale == nullptr), LLAISYS_E_UNSUPPORTED,
-               "gated attention: neither kept tokens nor output factors");
+    KV_REQUIRE(opt.gates == nullptr || (opt.keep_first == 0 && opt.row_scale == nullptr && opt.fade_a == nullptr), LLAISYS_E_UNSUPPORTED,
+               "gated attention: neither kept tokens, output factors nor a distance penalty");
+    KV_REQUIRE((opt.fade_a != nullptr) == (opt.fade_b != nullptr), LLAISYS_E_INVALID, "paged attention: a distance penalty has two factors");
 }
 
 int PagedKV::runGates(const kernels::KVView &v, const kernels::AttnBatch &b, const void *q, float scale, const kernels::GateArgs &gates,
@@ -511,7 +515,12 @@ kernels::KVView PagedKV::view(size_t layer) const {
     v.num_pages = int32_t(_cfg.num_pages);
     v.nkvh = int32_t(l.nkvh);
     v.d = int32_t(l.k_dim);
-    if (l.v_dim != l.k_dim) {
+    if (l.v_row == 0) {
+        v.v_base = v.k_base;
+        v.v_d = int32_t(l.v_dim);
+        v.v_head_stride = v.head_stride;
+        v.v_token_stride = v.token_stride;
+    } else if (l.v_dim != l.k_dim) {
         v.v_d = int32_t(l.v_dim);
         v.v_head_stride = int64_t(_cfg.page_size * l.v_row);
         v.v_token_stride = int64_t(l.v_row);
@@ -666,6 +675,25 @@ void PagedKV::normAppendDev(size_t layer, const kernels::NormAppendArgs &args, l
     enter();
     kernels::paged_norm_append(stream, _cfg.dtype, view(layer), args, int32_t(_cfg.max_pages_per_seq),
                                reinterpret_cast<int32_t *>(_error_dev->memory()));
+#else
+    (void)stream;
+    fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
+#endif
+}
+
+void PagedKV::latentAppendDev(size_t layer, const kernels::LatentAppendArgs &args, llaisysStream_t stream) {
+    checkLayer(layer);
+    const Layer &l = _layers[layer];
+    KV_REQUIRE(args.n_rows <= kMaxInt32 && l.v_row == 0 && l.nkvh == 1 && args.rank > 0 && args.rot_dims >= 0 && args.rot_dims % 2 == 0 &&
+                   size_t(args.rank) == l.v_dim && size_t(args.rank + args.rot_dims) == l.k_dim,
+               LLAISYS_E_INVALID, "paged KV latent append: this layer's rows hold no latents of this size");
+    if (args.n_rows == 0) {
+        return;
+    }
+    KV_REQUIRE(onDevice(), LLAISYS_E_UNSUPPORTED, "paged KV latent append: NVIDIA caches only");
+#ifdef ENABLE_NVIDIA_API
+    enter();
+    kernels::latent_append(stream, _cfg.dtype, view(layer), args, int32_t(_cfg.max_pages_per_seq), reinterpret_cast<int32_t *>(_error_dev->memory()));
 #else
     (void)stream;
     fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
@@ -1110,7 +1138,7 @@ int run_attention_nvidia(llaisysStream_t stream, llaisysDataType_t dtype, const 
                          const kernels::AttnBatch &batch, const void *q, float scale, const kernels::AttnOut &out,
                          const kernels::AttnScratch &scratch) {
     const bool one_query_each = batch.q_starts == nullptr && batch.const_q_len == 1;
-    const bool fast = fast_shape(dtype, view, batch);
+    const bool fast = fast_shape(dtype, view, batch) && batch.fade_a == nullptr;
     int used = LLAISYS_KERNEL_GENERIC;
     if (fast && one_query_each && view.block_table != nullptr && batch.kv_lens != nullptr) {
         // a page pool: the TMA kernel, or nothing

@@ -26,6 +26,7 @@ struct StatusError : std::runtime_error {
 // Geometry of one layer's K/V rows.
 struct KVLayerShape {
     size_t nkvh = 0, k_dim = 0, v_dim = 0;
+    bool v_in_k = false; // a V row is the first v_dim elements of its K row (one row per token serves as both)
 };
 
 // What a layer's attention adds to plain causal attention.
@@ -34,6 +35,7 @@ struct AttnOptions {
     size_t keep_first = 0;             // with a window: the first tokens of a sequence that stay visible behind it
     const float *row_scale = nullptr;  // device, [rows, nh]: factor on every head's output
     size_t row_stride = 0;             // elements between output rows; 0 = packed
+    const float *fade_a = nullptr, *fade_b = nullptr; // device, [nh]: distance penalty (see AttnBatch); softmax attention only
     const kernels::GateArgs *gates = nullptr; // weights without a softmax, mixed over the heads; with neither kept tokens nor factors
 };
 
@@ -131,6 +133,8 @@ public:
                     size_t nh, float scale, llaisysStream_t stream, const AttnOptions &opt = {});
     // Per-head RMS norm of q and k, then append: see kernels::paged_norm_append. Device caches only.
     void normAppendDev(size_t layer, const kernels::NormAppendArgs &args, llaisysStream_t stream);
+    // The same for latents: see kernels::latent_append. Layers with v_in_k and one kv head.
+    void latentAppendDev(size_t layer, const kernels::LatentAppendArgs &args, llaisysStream_t stream);
 
 private:
     struct Seq {
@@ -180,7 +184,7 @@ private:
     size_t _elem = 0;
     // Geometry of one layer in the pool. Rows are padded to whole 16-byte pieces (k_row, v_row elements).
     struct Layer {
-        size_t nkvh = 0, k_dim = 0, v_dim = 0, k_row = 0, v_row = 0;
+        size_t nkvh = 0, k_dim = 0, v_dim = 0, k_row = 0, v_row = 0; // v_row = 0: V rows lie in K rows
         size_t page_elems = 0; // K and V of one page
         size_t offset = 0, bytes = 0; // of the layer's pages in the pool
         // TMA view of the layer's pages (NVIDIA, 16-bit, K and V rows of 128, page 16 only)

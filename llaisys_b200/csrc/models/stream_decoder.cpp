@@ -30,7 +30,7 @@ std::byte *StreamDecoder::matrix(size_t rows, size_t cols) {
 
 void StreamDecoder::place(const std::string &name, std::byte *base, size_t row, size_t col, size_t rows, size_t cols, size_t ld,
                     size_t ndim) {
-    _slots.emplace(name, Slot{base, row, col, rows, cols, ld, ndim});
+    _slots.emplace(name, Slot{base, row, col, rows, cols, ld, ndim, _dtype});
 }
 
 std::byte *StreamDecoder::vector(const std::string &name, size_t n) {
@@ -39,24 +39,33 @@ std::byte *StreamDecoder::vector(const std::string &name, size_t n) {
     return p;
 }
 
+float *StreamDecoder::floats(const std::string &name, size_t n) {
+    auto &rt = enter();
+    const size_t rows = std::max<size_t>(n, 1);
+    _weight_blocks.push_back(rt.allocateDeviceStorage(rows * sizeof(float)));
+    std::byte *p = _weight_blocks.back()->memory();
+    _slots.emplace(name, Slot{p, 0, 0, rows, 1, 1, n == 0 ? size_t(0) : size_t(1), LLAISYS_DTYPE_F32});
+    return reinterpret_cast<float *>(p);
+}
+
 bool StreamDecoder::loadTensor(const std::string &name, llaisysDataType_t dtype, const std::vector<size_t> &shape, const void *data) {
     auto it = _slots.find(name);
     if (it == _slots.end()) {
         return false;
     }
     Slot &slot = it->second;
-    const bool fits = shape.size() == slot.ndim && shape[0] == slot.rows && (slot.ndim == 1 || shape[1] == slot.cols);
+    const bool fits = shape.size() == slot.ndim && (slot.ndim < 1 || shape[0] == slot.rows) && (slot.ndim < 2 || shape[1] == slot.cols);
     if (!fits) {
         failModel(LLAISYS_E_INVALID, "tensor " + name + " has another shape than the configuration gives it");
     }
     if (dtype != LLAISYS_DTYPE_F32 && dtype != LLAISYS_DTYPE_BF16 && dtype != LLAISYS_DTYPE_F16) {
         failModel(LLAISYS_E_INVALID, "tensor " + name + ": F32, F16 or BF16 expected");
     }
-    const size_t n = slot.rows * slot.cols;
+    const size_t n = slot.rows * slot.cols, elem = utils::dsize(slot.dtype);
     std::vector<std::byte> converted;
     const std::byte *src = static_cast<const std::byte *>(data);
-    if (dtype != _dtype) {
-        converted.resize(n * _elem);
+    if (dtype != slot.dtype) {
+        converted.resize(n * elem);
         for (size_t i = 0; i < n; ++i) {
             float v = 0.f;
             switch (dtype) {
@@ -70,7 +79,7 @@ bool StreamDecoder::loadTensor(const std::string &name, llaisysDataType_t dtype,
                 v = utils::cast<float>(static_cast<const bf16_t *>(data)[i]);
                 break;
             }
-            switch (_dtype) {
+            switch (slot.dtype) {
             case LLAISYS_DTYPE_F32:
                 reinterpret_cast<float *>(converted.data())[i] = v;
                 break;
@@ -86,12 +95,12 @@ bool StreamDecoder::loadTensor(const std::string &name, llaisysDataType_t dtype,
     }
     auto &rt = enter();
     rt.synchronize(); // the zero fill of the packed matrix comes first
-    std::byte *dst = slot.base + (slot.row * slot.ld + slot.col) * _elem;
+    std::byte *dst = slot.base + (slot.row * slot.ld + slot.col) * elem;
     if (slot.cols == slot.ld) {
-        rt.api()->memcpy_sync(dst, src, n * _elem, LLAISYS_MEMCPY_H2D);
+        rt.api()->memcpy_sync(dst, src, n * elem, LLAISYS_MEMCPY_H2D);
     } else {
         for (size_t r = 0; r < slot.rows; ++r) {
-            rt.api()->memcpy_sync(dst + r * slot.ld * _elem, src + r * slot.cols * _elem, slot.cols * _elem, LLAISYS_MEMCPY_H2D);
+            rt.api()->memcpy_sync(dst + r * slot.ld * elem, src + r * slot.cols * elem, slot.cols * elem, LLAISYS_MEMCPY_H2D);
         }
     }
     slot.loaded = true;

@@ -28,6 +28,8 @@ protected:
     // checkpoint tensor (1: a vector of `rows`, cols == 1).
     void place(const std::string &name, std::byte *base, size_t row, size_t col, size_t rows, size_t cols, size_t ld, size_t ndim = 2);
     std::byte *vector(const std::string &name, size_t n);
+    // n numbers kept in f32 whatever the model's dtype; n == 0: one number, a tensor without dimensions
+    float *floats(const std::string &name, size_t n);
 
     void beginRecord() { _recorded.clear(); }
     void recordLayer(const float *stream, size_t n); // n floats on the device; nothing unless recording is on
@@ -37,6 +39,7 @@ private:
         std::byte *base;
         size_t row, col, rows, cols, ld;
         size_t ndim;
+        llaisysDataType_t dtype;
         bool loaded = false;
     };
     std::map<std::string, Slot> _slots;

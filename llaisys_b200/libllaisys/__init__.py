@@ -177,6 +177,42 @@ class LlaisysLilovikMeta(Structure):
                 ("end_token", c_int64)]
 
 
+class LlaisysLatentAttentionMeta(Structure):
+    """struct LlaisysLatentAttentionMeta (include/llaisys/models/folivik.h)."""
+    _fields_ = [("heads", c_size_t), ("dim", c_size_t), ("rot_dim", c_size_t), ("vdim", c_size_t), ("q_rank", c_size_t),
+                ("kv_rank", c_size_t), ("rot_base", c_double), ("scale", c_float)]
+
+
+class LlaisysFadingAttentionMeta(Structure):
+    """struct LlaisysFadingAttentionMeta (include/llaisys/models/folivik.h)."""
+    _fields_ = [("heads", c_size_t), ("kv_heads", c_size_t), ("dim", c_size_t), ("vdim", c_size_t), ("window", c_size_t),
+                ("scale", c_float)]
+
+
+class LlaisysStateSpaceMixerMeta(Structure):
+    """struct LlaisysStateSpaceMixerMeta (include/llaisys/models/folivik.h)."""
+    _fields_ = [("heads", c_size_t), ("groups", c_size_t), ("state", c_size_t), ("vdim", c_size_t), ("taps", c_size_t),
+                ("norm_groups", c_size_t)]
+
+
+class LlaisysExpertLayerMeta(Structure):
+    """struct LlaisysExpertLayerMeta (include/llaisys/models/folivik.h)."""
+    _fields_ = [("experts", c_size_t), ("identity", c_size_t), ("top", c_size_t), ("groups", c_size_t), ("keep", c_size_t),
+                ("ff", c_size_t), ("shared_ff", c_size_t), ("scale", c_float)]
+
+
+class LlaisysFolivikLayerMeta(Structure):
+    """struct LlaisysFolivikLayerMeta (include/llaisys/models/folivik.h)."""
+    _fields_ = [("mixer", c_int), ("latent", LlaisysLatentAttentionMeta), ("attn", LlaisysFadingAttentionMeta),
+                ("ssm", LlaisysStateSpaceMixerMeta), ("mlp", LlaisysExpertLayerMeta)]
+
+
+class LlaisysFolivikMeta(Structure):
+    """struct LlaisysFolivikMeta (include/llaisys/models/folivik.h)."""
+    _fields_ = [("dtype", llaisysDataType_t), ("nlayer", c_size_t), ("layers", POINTER(LlaisysFolivikLayerMeta)),
+                ("width", c_size_t), ("voc", c_size_t), ("maxseq", c_size_t), ("eps", c_float), ("end_token", c_int64)]
+
+
 class LlaisysNormAppend(Structure):
     """struct LlaisysNormAppend (include/llaisys/mixers.h)."""
     _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("k_at", c_int64), ("v_at", c_int64),
@@ -392,6 +428,8 @@ PROTOTYPES: dict[str, tuple] = {
     # include/llaisys/models/vozozen.h
     # include/llaisys/models/lilovik.h
     "llaisysLilovikModelCreate": (_MODEL, [POINTER(LlaisysLilovikMeta), llaisysDeviceType_t, c_int]),
+    # include/llaisys/models/folivik.h
+    "llaisysFolivikModelCreate": (_MODEL, [POINTER(LlaisysFolivikMeta), llaisysDeviceType_t, c_int]),
     # include/llaisys/models/doderax.h
     "llaisysDoderaxModelCreate": (_MODEL, [POINTER(LlaisysDoderaxMeta), llaisysDeviceType_t, c_int]),
     "llaisysVozozenModelCreate": (_MODEL, [POINTER(LlaisysVozozenMeta), llaisysDeviceType_t, c_int]),
@@ -441,5 +479,7 @@ __all__ = [
     "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent",
     "LlaisysNormAppend", "LlaisysGatedLinear", "LlaisysGatedDelta", "LlaisysDoderaxMeta", "LlaisysDoderaxLayerMeta",
     "LlaisysGates", "LlaisysMinGru", "LlaisysLilovikMeta", "LlaisysLilovikLayerMeta", "LlaisysGatesAttentionMeta",
+    "LlaisysFolivikMeta", "LlaisysFolivikLayerMeta", "LlaisysLatentAttentionMeta", "LlaisysFadingAttentionMeta",
+    "LlaisysStateSpaceMixerMeta", "LlaisysExpertLayerMeta",
     "LlaisysSinkAttentionMeta", "LlaisysDeltaMixerMeta", "LlaisysVozozenMeta", "LlaisysVozozenLayerMeta", "LlaisysWindowAttentionMeta", "LlaisysGatedLinearMeta", "ALL_REDUCE_FN",
 ]

@@ -226,11 +226,11 @@ class NamedWeightsLM(CausalLM):
         self._load(name, value, kind)
 
     def _load(self, name: str, array: np.ndarray, kind: DataType) -> None:
-        array = np.ascontiguousarray(array)
-        shape = (c_size_t * array.ndim)(*array.shape)
+        ndim, shape = array.ndim, (c_size_t * array.ndim)(*array.shape)
+        array = np.ascontiguousarray(array)  # (gives a single number a dimension)
         known = c_int(0)
         try:
-            _check(LIB_LLAISYS.llaisysModelLoadTensor(self._model, name.encode(), int(kind), shape, array.ndim,
+            _check(LIB_LLAISYS.llaisysModelLoadTensor(self._model, name.encode(), int(kind), shape, ndim,
                                                       array.ctypes.data, ctypes.byref(known)))
         except LlaisysError as err:
             raise ValueError(str(err)) from err

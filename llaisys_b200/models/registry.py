@@ -7,13 +7,15 @@ from typing import Mapping
 
 from .base import CausalLM
 from .doderax import Doderax
+from .folivik import Folivik
 from .lilovik import Lilovik
 from .qwen2 import Qwen2
 from .vozozen import Vozozen
 
 # architecture name (config "architecture", an entry of "architectures", or "model_type") -> class
 MODELS: dict[str, type[CausalLM]] = {"qwen2": Qwen2, "Qwen2ForCausalLM": Qwen2, "Vozozen": Vozozen, "vozozen": Vozozen,
-                                   "Doderax": Doderax, "doderax": Doderax, "Lilovik": Lilovik, "lilovik": Lilovik}
+                                   "Doderax": Doderax, "doderax": Doderax, "Lilovik": Lilovik, "lilovik": Lilovik,
+                                   "Folivik": Folivik, "folivik": Folivik}
 
 
 def model_class(config: Mapping) -> type[CausalLM]:
