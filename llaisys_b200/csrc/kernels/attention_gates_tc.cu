@@ -132,16 +132,6 @@ __device__ __forceinline__ bool next_fragment(const Params &p, Walk &w, Fragment
     return false;
 }
 
-__device__ __forceinline__ bool elect_one() { // one lane of a converged warp
-    uint32_t leader;
-    asm volatile("{\n"
-                 ".reg .pred p;\n"
-                 "elect.sync _|p, 0xffffffff;\n"
-                 "selp.u32 %0, 1, 0, p;\n"
-                 "}\n"
-                 : "=r"(leader));
-    return leader != 0;
-}
 __device__ __forceinline__ void tmem_ld8(uint32_t taddr, float (&v)[8]) {
     uint32_t r[8];
     asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];\n"

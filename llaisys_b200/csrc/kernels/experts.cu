@@ -1,6 +1,7 @@
 // Mixture of experts (see ExpertArgs): the choice of experts, the line of rows sorted by expert, the plain form of the experts'
 // products (any dtype and sizes, f32 accumulation), and the sum into the stream with the norm that follows. The tensor-core form
 // of the products is experts_tc.cu; it serves 16-bit models whose rows are whole 16-byte pieces.
+#include "experts.cuh"
 #include "launch_utils.cuh"
 #include "mma_utils.cuh"
 
@@ -190,37 +191,6 @@ __global__ void __launch_bounds__(256) experts_place_kernel(ExpertArgs a) {
                 reinterpret_cast<Piece *>(static_cast<T *>(a.rows) + int64_t(s_place[k]) * a.width)[i] = p;
             }
         }
-    }
-}
-
-// Row tile `tile` of the line: the experts' rows are cut into tiles of `per_tile`, expert after expert. -> expert, first row, rows
-// (0: there is no such tile). For whole warps.
-__device__ __forceinline__ void find_tile(const int32_t *counts, int experts, int per_tile, int tile, int &expert, int &first, int &rows) {
-    const int lane = int(threadIdx.x) & 31;
-    int tiles = 0, before = 0;
-    rows = 0;
-    for (int base = 0; base < experts; base += 32) {
-        const int c = base + lane < experts ? counts[base + lane] : 0;
-        const int t = (c + per_tile - 1) / per_tile;
-        int t_sum = t, c_sum = c; // inclusive scans
-#pragma unroll
-        for (int o = 1; o < 32; o *= 2) {
-            const int tv = __shfl_up_sync(0xffffffffu, t_sum, o), cv = __shfl_up_sync(0xffffffffu, c_sum, o);
-            t_sum += lane >= o ? tv : 0;
-            c_sum += lane >= o ? cv : 0;
-        }
-        const unsigned hit = __ballot_sync(0xffffffffu, tile < tiles + t_sum);
-        if (hit != 0) {
-            const int l = __ffs(int(hit)) - 1;
-            const int t_before = tiles + __shfl_sync(0xffffffffu, t_sum - t, l), c_before = before + __shfl_sync(0xffffffffu, c_sum - c, l);
-            const int here = __shfl_sync(0xffffffffu, c, l), off = (tile - t_before) * per_tile;
-            expert = base + l;
-            first = c_before + off;
-            rows = min(per_tile, here - off);
-            return;
-        }
-        tiles += __shfl_sync(0xffffffffu, t_sum, 31);
-        before += __shfl_sync(0xffffffffu, c_sum, 31);
     }
 }
 
@@ -434,8 +404,7 @@ void experts_apply(stream_t stream, llaisysDataType_t dtype, const ExpertArgs &a
             experts_tc(stream, dtype, a);
             return;
         }
-        // no more tiles than this, whatever the routing
-        const int64_t total = int64_t(a.n_rows) * a.top, tiles = total / 32 + (total < a.experts ? total : int64_t(a.experts));
+        const int64_t tiles = expert_tiles_bound(a, 32);
         CHECK_ARGUMENT(tiles <= 65535, "experts: too many rows for the plain form");
         launch_programmatic(experts_plain_kernel<T, true>, dim3(unsigned((a.ff + 63) / 64), unsigned(tiles)), 256u, s, a, static_cast<const T *>(a.h),
                             a.line, static_cast<const T *>(a.gate_up), static_cast<T *>(a.act), a.ff, a.width);

@@ -22,9 +22,8 @@
 // Every mbarrier wait is bounded; a wait that runs out sets the error word and the CTA skips its stores but still
 // takes part in both cluster barriers and frees its TMEM.
 #include "kernels.hpp"
+#include "matrix_map.cuh"
 #include "tcgen05_utils.cuh"
-
-#include <cuda.h>
 
 #include <cstdlib>
 #include <cstring>
@@ -43,7 +42,6 @@ constexpr int kWStageBytes = kBF * 128; // 16 KiB
 constexpr int kMaxStages = 10;
 constexpr int kMaxSplit = 8;            // portable cluster size
 constexpr int kRingBudget = 196 * 1024; // bytes of shared memory given to the stage ring
-constexpr int kErrGemmTimeout = 16;
 constexpr int kNumBars = 2 * kMaxStages + 1;
 
 struct GemmParams {
@@ -300,8 +298,8 @@ EncodeTiledFn gemm_encode_fn() {
     return fn;
 }
 
-// Row-major [rows, k] 16-bit matrix -> 2-D map with a box of 64 elements x box_rows rows, 128-byte swizzle. Maps are
-// cached: a decode loop asks for the same handful of (pointer, shape) pairs every step.
+} // namespace
+
 bool matrix_map(CUtensorMap *out, const void *ptr, uint64_t rows, uint64_t k, uint32_t box_rows, bool bf16) {
     using Key = std::tuple<const void *, uint64_t, uint64_t, uint32_t, bool, int>;
     static std::mutex mu;
@@ -357,6 +355,8 @@ int32_t *gemm_error_word() {
     words.emplace(dev, w);
     return w;
 }
+
+namespace {
 
 template <bool kBf16>
 void launch_gemm(cudaStream_t s, const CUtensorMap &tx, const CUtensorMap &tw, const GemmParams &p, int tiles, int split,
