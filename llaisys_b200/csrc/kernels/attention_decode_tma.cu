@@ -91,6 +91,7 @@ struct TmaDecodeParams {
     int32_t window, keep_first;
     long long out_stride;
     const float *row_scale;
+    const float *fade_a, *fade_b; // [nh], with a distance penalty
     // KV-range split across GPUs (exchange instantiation; out null, part = PeerSink::rows): a pair's finished rows
     // (o, m, l) are written locally like any partial output, and the epilogue warp of the CTA that finished them then
     // stores every value, together with the step number, as one 8-byte word into slot `rank` of EVERY rank's exchange
@@ -226,13 +227,15 @@ __device__ __forceinline__ bool wait_or_abort(uint32_t bar, uint32_t parity, vol
 // kShare: launches with few pairs for their grid, whose pairs can be in many pieces, carry the shared merge (all five
 // warps of the last-arriving CTA); the others do not even contain its code -- this kernel's timing moves by a
 // microsecond with what is compiled around its hot loop.
-// kWin: sliding window, output row stride and output factor per head -- an instantiation of its own for the same reason.
+// kExtra 1: sliding window, output row stride and output factor per head -- an instantiation of its own for the same reason. 2: the
+// same with a distance penalty.
 // The pages between a sequence's kept first tokens and its window are not part of the line at all: page indices of a segment
 // count without them.
-template <bool kBf16, bool kXchg, bool kShare, bool kWin>
+template <bool kBf16, bool kXchg, bool kShare, int kExtra>
 __global__ void __launch_bounds__(kThreads, kCtasPerSm)
     paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ InlineIndex ix,
                             TmaDecodeParams p) {
+    constexpr bool kWin = kExtra >= 1, kFade = kExtra == 2;
     extern __shared__ unsigned char smem_raw[];
     // the 128-byte swizzle is a function of the shared-memory address: slots must start on 1 KiB boundaries
     const uint32_t raw_u32 = smem_u32(smem_raw);
@@ -591,6 +594,14 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
                 qf[ks][1] = g < p.group ? q_row[ks * 8 + 4 + q4] : 0u;
             }
         }
+        float fade_a0 = 0.f, fade_a1 = 0.f, fade_b0 = 0.f, fade_b1 = 0.f; // of this thread's two heads (those past the group: any)
+        if constexpr (kFade) {
+            const int h0 = sg.kvh * p.group + min(2 * q4, p.group - 1), h1 = sg.kvh * p.group + min(2 * q4 + 1, p.group - 1);
+            fade_a0 = p.fade_a[h0];
+            fade_a1 = p.fade_a[h1];
+            fade_b0 = p.fade_b[h0];
+            fade_b1 = p.fade_b[h1];
+        }
         // fused step: index in this segment of the pair's last page, which receives the new row; the warp that will
         // take that page fetches the row (K: lanes 0-15, V: lanes 16-31, 16 bytes each) and the page index now
         const int kept = kWin ? kept_pages(p) : 0, gap = kWin ? gap_pages(p, sg.kv_len) : 0;
@@ -669,10 +680,18 @@ __global__ void __launch_bounds__(kThreads, kCtasPerSm)
             // online softmax in the log2 domain; this thread holds tokens g, g + 8 for heads 2*q4, 2*q4 + 1
             const bool ok_lo = g < n_valid && (!kWin || g >= n_before || g < n_kept);
             const bool ok_hi = g + 8 < n_valid && (!kWin || g + 8 >= n_before || g + 8 < n_kept);
-            const float t0 = ok_lo ? sc[0] * p.scale_log2 : -INFINITY;
-            const float t1 = ok_lo ? sc[1] * p.scale_log2 : -INFINITY;
-            const float t2 = ok_hi ? sc[2] * p.scale_log2 : -INFINITY;
-            const float t3 = ok_hi ? sc[3] * p.scale_log2 : -INFINITY;
+            float less[4] = {0.f, 0.f, 0.f, 0.f};
+            if constexpr (kFade) {
+                const float d_lo = float(max(sg.kv_len - 1 - token0 - g, 0)), d_hi = float(max(sg.kv_len - 1 - token0 - g - 8, 0));
+                less[0] = fade_a0 * fast_log2(fmaf(fade_b0, d_lo, 1.f));
+                less[1] = fade_a1 * fast_log2(fmaf(fade_b1, d_lo, 1.f));
+                less[2] = fade_a0 * fast_log2(fmaf(fade_b0, d_hi, 1.f));
+                less[3] = fade_a1 * fast_log2(fmaf(fade_b1, d_hi, 1.f));
+            }
+            const float t0 = ok_lo ? (kFade ? fmaf(sc[0], p.scale_log2, -less[0]) : sc[0] * p.scale_log2) : -INFINITY;
+            const float t1 = ok_lo ? (kFade ? fmaf(sc[1], p.scale_log2, -less[1]) : sc[1] * p.scale_log2) : -INFINITY;
+            const float t2 = ok_hi ? (kFade ? fmaf(sc[2], p.scale_log2, -less[2]) : sc[2] * p.scale_log2) : -INFINITY;
+            const float t3 = ok_hi ? (kFade ? fmaf(sc[3], p.scale_log2, -less[3]) : sc[3] * p.scale_log2) : -INFINITY;
             float mx0 = fmaxf(t0, t2), mx1 = fmaxf(t1, t3);
 #pragma unroll
             for (int o = 4; o < 32; o <<= 1) {
@@ -855,7 +874,7 @@ size_t smem_bytes(int group, int n_seqs) {
            size_t(2 * n_seqs + 1) * sizeof(int) + 16 + size_t(kConsumerWarps) * kStageBytes;
 }
 
-template <bool kBf16, bool kXchg, bool kShare, bool kWin>
+template <bool kBf16, bool kXchg, bool kShare, int kExtra>
 void launch(cudaStream_t s, const CUtensorMap &tmap, const InlineIndex &ix, const TmaDecodeParams &p, int grid, size_t smem,
             bool overlap) {
     static std::once_flag once[64];
@@ -865,8 +884,8 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const InlineIndex &ix, cons
         int optin = 0;
         LLAISYS_CUDA_CHECK(cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev));
         cudaFuncAttributes attr{};
-        LLAISYS_CUDA_CHECK(cudaFuncGetAttributes(&attr, paged_decode_tma_kernel<kBf16, kXchg, kShare, kWin>));
-        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tma_kernel<kBf16, kXchg, kShare, kWin>,
+        LLAISYS_CUDA_CHECK(cudaFuncGetAttributes(&attr, paged_decode_tma_kernel<kBf16, kXchg, kShare, kExtra>));
+        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tma_kernel<kBf16, kXchg, kShare, kExtra>,
                                                 cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                 optin - int(attr.sharedSizeBytes)));
     });
@@ -880,7 +899,7 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const InlineIndex &ix, cons
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = overlap ? 1 : 0;
-    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_decode_tma_kernel<kBf16, kXchg, kShare, kWin>, tmap, ix, p));
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_decode_tma_kernel<kBf16, kXchg, kShare, kExtra>, tmap, ix, p));
 }
 
 } // namespace
@@ -950,9 +969,10 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
         return -1;
     }
     const int group = batch.nh / kv.nkvh;
-    const bool windowed = batch.window > 0 || out.row_scale != nullptr || out.row_stride != 0;
+    const bool fading = batch.fade_a != nullptr;
+    const bool windowed = batch.window > 0 || out.row_scale != nullptr || out.row_stride != 0 || fading;
     if (windowed && (out.out == nullptr || out.peers != nullptr || k_new != nullptr)) {
-        reason = "a window or an output scale goes with plain decode into an output tensor only";
+        reason = "a window, a distance penalty or an output scale goes with plain decode into an output tensor only";
         return -1;
     }
     // (a window reaches at most window + page - 1 tokens' worth of pages, the kept tokens keep_first + page - 1)
@@ -1006,6 +1026,8 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
     p.keep_first = batch.window > 0 ? batch.keep_first : 0;
     p.out_stride = out.row_stride != 0 ? out.row_stride : (long long)batch.nh * kD;
     p.row_scale = out.row_scale;
+    p.fade_a = batch.fade_a;
+    p.fade_b = batch.fade_b;
     p.xchg = PeerSink{};
     if (out.peers != nullptr) {
         p.xchg = *out.peers;
@@ -1033,11 +1055,13 @@ int attention_decode_tma(stream_t stream, llaisysDataType_t dtype, const KVView 
     };
     auto pick_xchg = [&](auto bf) {
         if (xchg) {
-            pick_share(bf, std::true_type{}, std::false_type{});
+            pick_share(bf, std::true_type{}, std::integral_constant<int, 0>{});
+        } else if (fading) {
+            pick_share(bf, std::false_type{}, std::integral_constant<int, 2>{});
         } else if (windowed) {
-            pick_share(bf, std::false_type{}, std::true_type{});
+            pick_share(bf, std::false_type{}, std::integral_constant<int, 1>{});
         } else {
-            pick_share(bf, std::false_type{}, std::false_type{});
+            pick_share(bf, std::false_type{}, std::integral_constant<int, 0>{});
         }
     };
     bf16 ? pick_xchg(std::true_type{}) : pick_xchg(std::false_type{});

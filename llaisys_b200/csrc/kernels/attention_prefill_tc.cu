@@ -55,6 +55,7 @@
 #include <cstring>
 #include <mutex>
 #include <string>
+#include <type_traits>
 
 namespace llaisys::kernels {
 
@@ -132,6 +133,8 @@ struct PrefillParams {
     int32_t window, keep_first;
     long long out_stride;
     const float *row_scale;
+    // fading instantiation: fade_a[h] log2(1 + fade_b[h] (distance)) is taken off the scores in the log2 domain
+    const float *fade_a, *fade_b;
     int32_t out_wide;  // out is 32-byte aligned: rows are stored 32 bytes (a whole sector) per instruction
 };
 
@@ -284,12 +287,18 @@ __device__ __forceinline__ void add2(float &s0, float &s1, float a0, float a1) {
         : "f"(a0), "f"(a1));
 }
 
-// kWin: sliding window, output row stride and output factor; a separate instantiation, so that the plain kernel's loops
-// carry nothing of it.
-template <bool kBf16, bool kWin>
+// What an instantiation of the kernel adds to plain causal attention; the plain kernel's loops carry nothing of it.
+enum Form {
+    kPlain,
+    kWindowed, // sliding window, output row stride and output factor
+    kFading,   // the same with a distance penalty
+};
+
+template <bool kBf16, int kForm>
 __global__ void __launch_bounds__(kThreads, 2)
     paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ CUtensorMap tmap_v,
                             PrefillParams p) {
+    constexpr bool kWin = kForm != kPlain, kFade = kForm == kFading;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     const uint32_t raw_u32 = smem_u32(smem_raw);
     const uint32_t base_u32 = (raw_u32 + 1023u) & ~1023u; // swizzled operands need 1 KiB alignment
@@ -632,6 +641,8 @@ __global__ void __launch_bounds__(kThreads, 2)
             const int t = f.qb * kBlockM + row;        // query index inside the chunk
             const int last_visible = t + g.off;        // keys j <= last_visible (and < kv_len) take part
             float m_used = -INFINITY, l = 0.f;
+            const float fade_a = kFade ? p.fade_a[f.h] : 0.f, fade_b = kFade ? p.fade_b[f.h] : 0.f;
+            const float to_log2 = kFade ? 1.f : p.scale_log2; // what the scores still have to be multiplied by
             for (int i = 0; i < n && !dead; ++i) {
                 const int gi = done + i, buf = gi & 1;
                 if (!wait_or_abort(bar(kBarQKDone + buf), uint32_t(gi >> 1) & 1u, s_abort)) {
@@ -650,10 +661,25 @@ __global__ void __launch_bounds__(kThreads, 2)
                     tmem_ld32_nowait(tmem_s + c * 32, sr[c]);
                 }
                 tmem_wait_ld();
+                if constexpr (kFade) {
+                    // (distances are exact; those of hidden keys may be negative, whatever comes of them is masked below)
+                    const float d0 = float(last_visible - j0);
+#pragma unroll
+                    for (int c = 0; c < kBlockN / 32; ++c) {
+#pragma unroll
+                        for (int k = 0; k < 32; k += 2) {
+                            float a0, a1, x0, x1;
+                            fma2(a0, a1, d0 - float(c * 32 + k), d0 - float(c * 32 + k + 1), fade_b, 1.f);
+                            fma2(x0, x1, __uint_as_float(sr[c][k]), __uint_as_float(sr[c][k + 1]), p.scale_log2, 0.f);
+                            sr[c][k] = __float_as_uint(fmaf(-fade_a, fast_log2(a0), x0));
+                            sr[c][k + 1] = __float_as_uint(fmaf(-fade_a, fast_log2(a1), x1));
+                        }
+                    }
+                }
                 // Most blocks lie wholly below the diagonal: the whole warp then skips the mask (warp-uniform choice).
                 // Otherwise the hidden scores become -inf and take the same path: 2^(-inf * scale - m) = 0. (A scale
                 // that is not positive takes the slow path further down.)
-                const bool plain = p.scale_log2 > 0.f;
+                const bool plain = kFade || p.scale_log2 > 0.f;
                 if (plain && !__all_sync(0xffffffffu, n_ok >= kBlockN && (!kWin || n_lo <= 0 || n_kept >= kBlockN))) {
 #pragma unroll
                     for (int c = 0; c < kBlockN / 32; ++c) {
@@ -684,7 +710,7 @@ __global__ void __launch_bounds__(kThreads, 2)
 #pragma unroll
                         for (int k = 0; k < 32; ++k) {
                             if (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo || c * 32 + k < n_kept)) {
-                                mx8[k & 7] = fmaxf(mx8[k & 7], __uint_as_float(sr[c][k]) * p.scale_log2);
+                                mx8[k & 7] = fmaxf(mx8[k & 7], __uint_as_float(sr[c][k]) * to_log2);
                             }
                         }
                     }
@@ -692,7 +718,7 @@ __global__ void __launch_bounds__(kThreads, 2)
                 float mx = fmaxf(fmaxf(fmaxf(mx8[0], mx8[1]), fmaxf(mx8[2], mx8[3])),
                                  fmaxf(fmaxf(mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7])));
                 if (plain) {
-                    mx *= p.scale_log2;
+                    mx *= to_log2;
                 }
                 // The running max only moves when it grew by more than 2^8: P and the row sum both use m_used, so the
                 // result is exact either way, and O is rescaled rarely.
@@ -714,7 +740,7 @@ __global__ void __launch_bounds__(kThreads, 2)
 #pragma unroll
                         for (int k = 0; k < 32; k += 2) {
                             float x0, x1;
-                            fma2(x0, x1, __uint_as_float(sr[c][k]), __uint_as_float(sr[c][k + 1]), p.scale_log2, neg_m);
+                            fma2(x0, x1, __uint_as_float(sr[c][k]), __uint_as_float(sr[c][k + 1]), to_log2, neg_m);
                             const float p0 = fast_exp2(x0);
                             const float p1 = fast_exp2(x1);
                             if (k & 2) {
@@ -731,9 +757,9 @@ __global__ void __launch_bounds__(kThreads, 2)
 #pragma unroll
                         for (int k = 0; k < 32; k += 2) {
                             const float p0 =
-                                (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo || c * 32 + k < n_kept)) ? fast_exp2(fmaf(__uint_as_float(sr[c][k]), p.scale_log2, neg_m)) : 0.f;
+                                (c * 32 + k < n_ok && (!kWin || c * 32 + k >= n_lo || c * 32 + k < n_kept)) ? fast_exp2(fmaf(__uint_as_float(sr[c][k]), to_log2, neg_m)) : 0.f;
                             const float p1 = (c * 32 + k + 1 < n_ok && (!kWin || c * 32 + k + 1 >= n_lo || c * 32 + k + 1 < n_kept))
-                                                 ? fast_exp2(fmaf(__uint_as_float(sr[c][k + 1]), p.scale_log2, neg_m))
+                                                 ? fast_exp2(fmaf(__uint_as_float(sr[c][k + 1]), to_log2, neg_m))
                                                  : 0.f;
                             l0 += p0;
                             l1 += p1;
@@ -1108,13 +1134,13 @@ int prefill_slots() {
     return n;
 }
 
-template <bool kBf16, bool kWin>
+template <bool kBf16, int kForm>
 void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, const PrefillParams &p, int grid, bool overlap) {
     static std::once_flag once[64];
     int dev = 0;
     LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
     std::call_once(once[dev & 63], [] {
-        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_prefill_tc_kernel<kBf16, kWin>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        LLAISYS_CUDA_CHECK(cudaFuncSetAttribute(paged_prefill_tc_kernel<kBf16, kForm>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                 int(kSmemBytes)));
     });
     cudaLaunchConfig_t cfg{};
@@ -1127,7 +1153,7 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, 
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = overlap ? 1 : 0;
-    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_prefill_tc_kernel<kBf16, kWin>, tmap, tmap_v, p));
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_prefill_tc_kernel<kBf16, kForm>, tmap, tmap_v, p));
 }
 
 } // namespace
@@ -1268,7 +1294,7 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
         reinterpret_cast<uintptr_t>(scratch.partials) % 16 != 0) {
         return -1;
     }
-    const bool windowed = batch.window > 0 || out.row_scale != nullptr || out.row_stride != 0;
+    const bool fading = batch.fade_a != nullptr, windowed = batch.window > 0 || out.row_scale != nullptr || out.row_stride != 0 || fading;
     if ((windowed && !paged) || out.row_stride % 8 != 0) {
         return -1;
     }
@@ -1276,6 +1302,8 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
     p.keep_first = batch.window > 0 ? batch.keep_first : 0;
     p.out_stride = out.row_stride != 0 ? out.row_stride : (long long)batch.nh * kD;
     p.row_scale = out.row_scale;
+    p.fade_a = batch.fade_a;
+    p.fade_b = batch.fade_b;
     p.out_wide = reinterpret_cast<uintptr_t>(out.out) % 32 == 0 && p.out_stride % 16 == 0 ? 1 : 0;
     p.partials = scratch.partials;
     p.counters = scratch.counters;
@@ -1288,12 +1316,16 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
         return -1;
     }
     auto s = static_cast<cudaStream_t>(stream);
-    if (windowed) {
-        bf16 ? launch<true, true>(s, tmap, tmap_v, p, grid, kv.overlap_launch)
-             : launch<false, true>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
+    auto run = [&](auto form) {
+        constexpr int kForm = decltype(form)::value;
+        bf16 ? launch<true, kForm>(s, tmap, tmap_v, p, grid, kv.overlap_launch) : launch<false, kForm>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
+    };
+    if (fading) {
+        run(std::integral_constant<int, kFading>{});
+    } else if (windowed) {
+        run(std::integral_constant<int, kWindowed>{});
     } else {
-        bf16 ? launch<true, false>(s, tmap, tmap_v, p, grid, kv.overlap_launch)
-             : launch<false, false>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
+        run(std::integral_constant<int, kPlain>{});
     }
     check_launch("paged_prefill_tc");
     return 0;

@@ -1130,7 +1130,7 @@ namespace {
 // call to the generic kernel behind the caller's back.
 bool fast_shape(llaisysDataType_t dtype, const kernels::KVView &view, const kernels::AttnBatch &batch) {
     return (dtype == LLAISYS_DTYPE_BF16 || dtype == LLAISYS_DTYPE_F16) && view.d == 128 && view.page_size == 16 &&
-           view.vDim() == 128 && view.nkvh > 0 && batch.nh % view.nkvh == 0 && batch.nh / view.nkvh <= 8;
+           view.vDim() == 128 && view.v_base != view.k_base && view.nkvh > 0 && batch.nh % view.nkvh == 0 && batch.nh / view.nkvh <= 8;
 }
 } // namespace
 
@@ -1138,7 +1138,7 @@ int run_attention_nvidia(llaisysStream_t stream, llaisysDataType_t dtype, const 
                          const kernels::AttnBatch &batch, const void *q, float scale, const kernels::AttnOut &out,
                          const kernels::AttnScratch &scratch) {
     const bool one_query_each = batch.q_starts == nullptr && batch.const_q_len == 1;
-    const bool fast = fast_shape(dtype, view, batch) && batch.fade_a == nullptr;
+    const bool fast = fast_shape(dtype, view, batch);
     int used = LLAISYS_KERNEL_GENERIC;
     if (fast && one_query_each && view.block_table != nullptr && batch.kv_lens != nullptr) {
         // a page pool: the TMA kernel, or nothing
