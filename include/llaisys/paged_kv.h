@@ -60,6 +60,8 @@ LLAISYS_API const char *llaisysGetLastError(void);
 #define LLAISYS_KERNEL_GATES 7            /* gated attention (mixers.h), any dtype / head_dim: one CTA per query  */
 #define LLAISYS_KERNEL_GATES_TILES 8      /* gated attention on the tensor cores, queries x keys x all heads      */
 #define LLAISYS_KERNEL_GATES_TC 9         /* gated attention of chunks on tcgen05 tensor cores                    */
+#define LLAISYS_KERNEL_LATENT_TC 10       /* attention over pages of latents (mixers.h) on tcgen05 tensor cores   */
+#define LLAISYS_KERNEL_EXPANDED_TC 11     /* chunk attention over keys and values made from latents, tcgen05      */
 /* Kernel of the calling thread's most recent attention call: any cache, or llaisysSelfAttention. */
 LLAISYS_API int llaisysLastAttentionKernel(void);
 

@@ -167,6 +167,25 @@ struct LatentAppendArgs {
     size_t n_rows = 0;
 };
 
+// Causal attention of ragged chunks over plain K and V tensors of a whole batch, the keys of a head being `dim` dims of their own and
+// rot_dim dims that all heads share. Sequence i's keys are rows 16 page_starts[i] .. + kv_lens[i] (page_starts[i] < 0: left out); rows up
+// to the next multiple of 64 may be read and must be finite.
+struct ExpandedArgs {
+    const void *q = nullptr;        // [rows, nh, dim + rot_dim]
+    const void *k = nullptr;        // [tokens, nh, dim]
+    const void *k_shared = nullptr; // row t at k_shared + t * shared_stride, [rot_dim]
+    int64_t shared_stride = 0;
+    const void *v = nullptr;        // [tokens, nh, vdim]
+    int64_t tokens = 0;
+    int32_t nh = 0, dim = 0, rot_dim = 0, vdim = 0;
+    const int32_t *page_starts = nullptr, *q_starts = nullptr, *kv_lens = nullptr; // [n_seqs], [n_seqs + 1], [n_seqs] on the device
+    int32_t n_seqs = 0;
+    float scale = 1.f;
+    void *out = nullptr; // row r, head h: out + r * out_stride + h * vdim, times row_scale[r * nh + h] (null: 1)
+    int64_t out_stride = 0;
+    const float *row_scale = nullptr;
+};
+
 // Mamba-2 over one packed projection row [.. z | .. x, B, C .. | dt ..]: x (heads x dv), B and C (groups x dk each) follow one another at
 // x_at, pass a causal convolution of `taps` taps per channel with a bias, and silu. Per head a state S [dk, dv]; head h uses group
 // h / (heads / groups):

@@ -72,7 +72,6 @@ constexpr int kProducerWarp = 4, kMmaWarp = 5;
 constexpr int kThreads = 192;
 // Every operand is stored as 64-element (128-byte) column halves of [rows][128 B], 128-byte swizzled.
 constexpr int kQHalfBytes = kBlockM * 128;       // Q: 128 rows x 64 dims, 16 KiB; two of them
-constexpr int kQBytes = 2 * kQHalfBytes;
 constexpr int kKvHalfBytes = kBlockN * 128;      // K (or V): kBlockN keys x 64 dims; two of them per operand
 constexpr int kKvOperandBytes = 2 * kKvHalfBytes;
 constexpr int kStageBytes = 2 * kKvOperandBytes; // K block + V block
@@ -135,6 +134,10 @@ struct PrefillParams {
     const float *row_scale;
     // fading instantiation: fade_a[h] log2(1 + fade_b[h] (distance)) is taken off the scores in the log2 domain
     const float *fade_a, *fade_b;
+    // expanded instantiation: sequence a's keys are rows 16 page_starts[a] .. of plain tensors (page_starts[a] < 0: not part of the call); a
+    // key is nope_halves 64-dim pieces of its own head (from `dim` dims) and one that all heads share (`rot` dims); V rows of dv
+    const int32_t *page_starts;
+    int32_t dim, rot, dv, nope_halves;
     int32_t out_wide;  // out is 32-byte aligned: rows are stored 32 bytes (a whole sector) per instruction
 };
 
@@ -154,7 +157,7 @@ __device__ __forceinline__ SeqGeom seq_geom(const PrefillParams &p, int a) {
         g.kv_len = max(p.const_kv_len, g.q_len);
     } else {
         g.q_start = p.q_starts[a];
-        g.q_len = p.q_starts[a + 1] - g.q_start;
+        g.q_len = p.page_starts != nullptr && p.page_starts[a] < 0 ? 0 : p.q_starts[a + 1] - g.q_start;
         g.kv_len = min(max(p.kv_lens[a], g.q_len), p.table_stride * kPage);
     }
     g.q_len = min(g.q_len, g.kv_len); // (a chunk longer than the tables can hold: flagged elsewhere, never off the end here)
@@ -292,13 +295,20 @@ enum Form {
     kPlain,
     kWindowed, // sliding window, output row stride and output factor
     kFading,   // the same with a distance penalty
+    kExpanded, // output row stride and factor; K and V in plain tensors of the whole batch, K rows of up to 192 in three pieces of 64 dims
 };
 
 template <bool kBf16, int kForm>
 __global__ void __launch_bounds__(kThreads, 2)
     paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ CUtensorMap tmap_v,
-                            PrefillParams p) {
-    constexpr bool kWin = kForm != kPlain, kFade = kForm == kFading;
+                            const __grid_constant__ CUtensorMap tmap_r, PrefillParams p) {
+    constexpr bool kWin = kForm == kWindowed || kForm == kFading, kFade = kForm == kFading, kWide = kForm == kExpanded, kRows = kForm != kPlain;
+    constexpr int kPieces = kWide ? 3 : 2; // of a Q or K row
+    constexpr int kQBytes = kPieces * kQHalfBytes;
+    // K and V of a stage side by side; expanded: two K stages, then ONE stage of V (so that two CTAs fit an SM)
+    constexpr int kKStride = kWide ? kPieces * kKvHalfBytes : kStageBytes;
+    constexpr int kVAt = kWide ? 2 * kKStride : kKvOperandBytes, kVStride = kWide ? 0 : kStageBytes;
+    static_assert(!kWide || kVAt + kKvOperandBytes == kStages * kStageBytes, "the same ring");
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     const uint32_t raw_u32 = smem_u32(smem_raw);
     const uint32_t base_u32 = (raw_u32 + 1023u) & ~1023u; // swizzled operands need 1 KiB alignment
@@ -409,6 +419,34 @@ __global__ void __launch_bounds__(kThreads, 2)
         // the stores are volatile asm, which no load may pass, and one round trip per 16 bytes made a fragment
         // boundary cost six blocks' time.
         const char *q_base = static_cast<const char *>(p.q);
+        if constexpr (kWide) {
+            constexpr int kRow = kPieces * 8, kAtOnce = 8;
+            const int dim = p.dim, head = dim + p.rot;
+            for (int u0 = first; u0 < kBlockM * kRow; u0 += kAtOnce * stride) {
+                uint4 vals[kAtOnce];
+#pragma unroll
+                for (int it = 0; it < kAtOnce; ++it) {
+                    const int idx = u0 + it * stride, r = idx / kRow, cc = idx - r * kRow, t = f.qb * kBlockM + r;
+                    const int piece = cc >> 3, e = (cc & 7) * 8, last = p.nope_halves;
+                    const int at = piece == last ? dim + e : piece * 64 + e, end = piece == last ? head : dim;
+                    vals[it] = make_uint4(0u, 0u, 0u, 0u);
+                    if (idx < kBlockM * kRow && t < g.q_len && piece <= last && at < end) {
+                        vals[it] = *reinterpret_cast<const uint4 *>(q_base + (((long long)(g.q_start + t) * p.nh + f.h) * head + at) * 2);
+                    }
+                }
+#pragma unroll
+                for (int it = 0; it < kAtOnce; ++it) {
+                    const int idx = u0 + it * stride, r = idx / kRow, cc = idx - r * kRow;
+                    if (idx < kBlockM * kRow) {
+                        const uint32_t dst = q_u32 + (cc >> 3) * kQHalfBytes + r * 128 + (((cc & 7) ^ (r & 7)) << 4);
+                        asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};\n" ::"r"(dst), "r"(vals[it].x), "r"(vals[it].y),
+                                     "r"(vals[it].z), "r"(vals[it].w)
+                                     : "memory");
+                    }
+                }
+            }
+            return;
+        }
         constexpr int kMaxIter = kBlockM * 16 / kSoftmaxThreads; // the fewest threads that call this
         uint4 vals[kMaxIter];
 #pragma unroll
@@ -472,7 +510,55 @@ __global__ void __launch_bounds__(kThreads, 2)
         atomicOr(p.error_flag, kErrTimeout);
     };
 
-    if (warp == kProducerWarp) {
+    if (kWide && warp == kProducerWarp) {
+        // ================================ producer, plain tensors ================================================
+        // K runs one block ahead of V: its stage is free as soon as the scores of two blocks before are there, the one stage of V
+        // when the product of the block before is done.
+        bool alive = true;
+        int done = 0;
+        const uint32_t k_bytes = uint32_t(p.nope_halves + 1) * kKvHalfBytes;
+        for (int pos = piece_begin; alive;) {
+            Fragment f;
+            if (!locate(p, walker, pos, piece_end, f)) {
+                break;
+            }
+            const int n = f.b1 - f.b0, token0 = p.page_starts[f.a] * kPage + f.b0 * kBlockN;
+            auto load_k = [&](int i) {
+                const int gi = done + i, st = gi & 1;
+                if (gi >= kStages && !__all_sync(0xffffffffu, wait_or_abort(bar(kBarQKDone + st), uint32_t((gi >> 1) - 1) & 1u, s_abort))) {
+                    return false;
+                }
+                if (elect_one()) {
+                    const uint32_t dst = kv_u32 + st * kKStride, full = bar(kBarKFull + st);
+                    mbar_arrive_expect_tx(full, k_bytes);
+                    for (int piece = 0; piece < p.nope_halves; ++piece) {
+                        tma_load_3d(dst + piece * kKvHalfBytes, &tmap, piece * 64, f.h, token0 + i * kBlockN, full);
+                    }
+                    tma_load_2d(dst + p.nope_halves * kKvHalfBytes, &tmap_r, 0, token0 + i * kBlockN, full);
+                }
+                __syncwarp();
+                return true;
+            };
+            alive = load_k(0);
+            for (int i = 0; i < n && alive; ++i) {
+                alive = i + 1 >= n || load_k(i + 1);
+                const int gi = done + i;
+                if (alive && gi >= 1) {
+                    alive = __all_sync(0xffffffffu, wait_or_abort(bar(kBarPVDone + ((gi - 1) & 1)), uint32_t((gi - 1) >> 1) & 1u, s_abort));
+                }
+                if (alive && elect_one()) {
+                    mbar_arrive_expect_tx(bar(kBarVFull), kKvOperandBytes);
+                    tma_load_4d(kv_u32 + kVAt, &tmap_v, 0, token0 + i * kBlockN, 0, f.h, bar(kBarVFull));
+                }
+                __syncwarp();
+            }
+            pos += n;
+            done += n;
+        }
+        if (!alive && lane == 0) {
+            give_up();
+        }
+    } else if (warp == kProducerWarp) {
         // ================================ producer: TMA tiles of K and V =========================================
         bool alive = true;
         int done = 0; // blocks of earlier fragments: ring stage and parity run on across fragments
@@ -566,17 +652,18 @@ __global__ void __launch_bounds__(kThreads, 2)
             bool ok = true;
             auto issue_pv = [&](int gj, bool first_of_fragment) { // O (+)= P . V of the CTA's gj-th block
                 if (!wait_or_abort(bar(kBarPFull), uint32_t(gj) & 1u, s_abort) ||
-                    !wait_or_abort(bar(kBarVFull + (gj & 1)), uint32_t(gj >> 1) & 1u, s_abort)) {
+                    !wait_or_abort(bar(kBarVFull + (kWide ? 0 : gj & 1)), uint32_t(kWide ? gj : gj >> 1) & 1u, s_abort)) {
                     return false;
                 }
                 tc_fence_after();
-                const uint32_t v_u32 = kv_u32 + (gj & 1) * kStageBytes + kKvOperandBytes;
+                const uint32_t v_u32 = kv_u32 + (gj & 1) * kVStride + kVAt;
 #pragma unroll
                 for (int kk = 0; kk < kBlockN / 16; ++kk) {
                     // B = 16 keys (one page) x 128 dims of V, MN-major: 8-key groups 1 KiB apart, the page's two
                     // 64-dim halves 2 KiB apart, pages 4 KiB apart. A = P rows x 16 keys from tensor memory: 8 columns
                     // of packed pairs per step, in S buffer gj & 1
-                    const uint64_t b = smem_desc_sw128(v_u32 + kk * (2 * 2048), 2048, 1024);
+                    // (plain tensors: the block's two halves 8 KiB apart, 16 keys 2 KiB)
+                    const uint64_t b = kWide ? smem_desc_sw128(v_u32 + kk * 2048, kKvHalfBytes, 1024) : smem_desc_sw128(v_u32 + kk * (2 * 2048), 2048, 1024);
                     umma_f16_ts(tmem_o, tmem_base + kColS + (gj & 1) * kBlockN + kk * 8, b, idesc_pv,
                                 (!first_of_fragment || kk > 0) ? 1u : 0u);
                 }
@@ -600,9 +687,12 @@ __global__ void __launch_bounds__(kThreads, 2)
                         break;
                     }
                     tc_fence_after();
-                    const uint32_t k_u32 = kv_u32 + st * kStageBytes;
+                    const uint32_t k_u32 = kv_u32 + st * kKStride;
 #pragma unroll
-                    for (int ks = 0; ks < kD / 16; ++ks) {
+                    for (int ks = 0; ks < kPieces * 4; ++ks) {
+                        if (kWide && (ks >> 2) > p.nope_halves) {
+                            break;
+                        }
                         const uint64_t a = smem_desc_sw128(q_u32 + (ks >> 2) * kQHalfBytes + (ks & 3) * 32, 0, 1024);
                         const uint64_t b = smem_desc_sw128(k_u32 + (ks >> 2) * kKvHalfBytes + (ks & 3) * 32, 0, 1024);
                         umma_f16(tmem_base + kColS + buf * kBlockN, a, b, idesc_qk, ks > 0 ? 1u : 0u);
@@ -821,7 +911,7 @@ __global__ void __launch_bounds__(kThreads, 2)
             }
             tc_fence_after();
             const bool whole = f.b0 == 0 && f.b1 == f.tile_nblk;
-            char *out_row = static_cast<char *>(p.out) + (kWin ? (long long)(g.q_start + t) * p.out_stride * 2 + f.h * (kD * 2)
+            char *out_row = static_cast<char *>(p.out) + (kRows ? (long long)(g.q_start + t) * p.out_stride * 2 + f.h * ((kWide ? p.dv : kD) * 2)
                                                                : ((long long)(g.q_start + t) * p.nh + f.h) * (kD * 2));
             bool store_rows = whole, staged = false;
             float w_own = 1.f, l_all = l, m_all = m_used;
@@ -951,7 +1041,7 @@ __global__ void __launch_bounds__(kThreads, 2)
             }
             if (store_rows && (staged || !dead)) {
                 float inv = l_all > 0.f ? 1.f / l_all : 0.f;
-                if (kWin && p.row_scale != nullptr && t < g.q_len) {
+                if (kRows && p.row_scale != nullptr && t < g.q_len) {
                     inv *= p.row_scale[(long long)(g.q_start + t) * p.nh + f.h];
                 }
 #pragma unroll
@@ -1049,6 +1139,9 @@ __global__ void __launch_bounds__(kThreads, 2)
                             }
                         }
                     }
+                    if (kWide && c4 * 32 >= p.dv) {
+                        continue; // (V rows of 64: the other columns are nothing)
+                    }
                     if (t < g.q_len && p.out_wide) {
                         // a thread owns a row: a 16-byte store fills half a 32-byte sector and the other half comes
                         // with the next instruction; 32-byte stores halve the write transactions of the epilogue
@@ -1118,7 +1211,10 @@ EncodeTiledFn prefill_encode_fn() {
 
 // operands + barriers + TMEM-address / abort words + scheduling words; kAlignSlack bytes for the 1 KiB alignment of the
 // operand area (the dynamic window itself starts aligned when the kernel has no static shared memory)
-constexpr size_t kSmemBytes = kAlignSlack + kQBytes + kStages * kStageBytes + kNumBars * sizeof(uint64_t) + 8 + 16 * sizeof(int);
+constexpr size_t smem_bytes(int pieces) {
+    return size_t(kAlignSlack) + size_t(pieces) * kQHalfBytes + kStages * kStageBytes + kNumBars * sizeof(uint64_t) + 8 + 16 * sizeof(int);
+}
+static_assert(2 * (smem_bytes(3) + 1024) <= 228 * 1024, "two CTAs per SM");
 
 // CTAs of the fixed grid: two per SM
 int prefill_slots() {
@@ -1135,7 +1231,9 @@ int prefill_slots() {
 }
 
 template <bool kBf16, int kForm>
-void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, const PrefillParams &p, int grid, bool overlap) {
+void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, const CUtensorMap &tmap_r, const PrefillParams &p, int grid,
+            bool overlap) {
+    constexpr size_t kSmemBytes = smem_bytes(kForm == kExpanded ? 3 : 2);
     static std::once_flag once[64];
     int dev = 0;
     LLAISYS_CUDA_CHECK(cudaGetDevice(&dev));
@@ -1153,7 +1251,7 @@ void launch(cudaStream_t s, const CUtensorMap &tmap, const CUtensorMap &tmap_v, 
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = overlap ? 1 : 0;
-    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_prefill_tc_kernel<kBf16, kForm>, tmap, tmap_v, p));
+    LLAISYS_CUDA_CHECK(cudaLaunchKernelEx(&cfg, paged_prefill_tc_kernel<kBf16, kForm>, tmap, tmap_v, tmap_r, p));
 }
 
 } // namespace
@@ -1268,7 +1366,7 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
     if (!paged && !contiguous) {
         return -1;
     }
-    PrefillParams p;
+    PrefillParams p{};
     p.page0 = paged ? kv.tma_page0 : 0;
     p.block_table = kv.block_table;
     p.table_stride = kv.table_stride;
@@ -1318,7 +1416,8 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
     auto s = static_cast<cudaStream_t>(stream);
     auto run = [&](auto form) {
         constexpr int kForm = decltype(form)::value;
-        bf16 ? launch<true, kForm>(s, tmap, tmap_v, p, grid, kv.overlap_launch) : launch<false, kForm>(s, tmap, tmap_v, p, grid, kv.overlap_launch);
+        bf16 ? launch<true, kForm>(s, tmap, tmap_v, tmap, p, grid, kv.overlap_launch)
+             : launch<false, kForm>(s, tmap, tmap_v, tmap, p, grid, kv.overlap_launch);
     };
     if (fading) {
         run(std::integral_constant<int, kFading>{});
@@ -1328,6 +1427,76 @@ int attention_prefill_tc(stream_t stream, llaisysDataType_t dtype, const KVView 
         run(std::integral_constant<int, kPlain>{});
     }
     check_launch("paged_prefill_tc");
+    return 0;
+}
+
+bool attention_expanded_covers(llaisysDataType_t dtype, size_t dim, size_t rot_dim, size_t vdim) {
+    return (dtype == LLAISYS_DTYPE_BF16 || dtype == LLAISYS_DTYPE_F16) && dim != 0 && dim <= kD && dim % 8 == 0 && rot_dim != 0 && rot_dim <= 64 &&
+           rot_dim % 8 == 0 && (vdim == 64 || vdim == kD);
+}
+
+int attention_expanded_tc(stream_t stream, llaisysDataType_t dtype, const ExpandedArgs &a, const AttnScratch &scratch) {
+    const bool bf16 = dtype == LLAISYS_DTYPE_BF16;
+    const int grid = prefill_slots();
+    if (!attention_expanded_covers(dtype, size_t(a.dim), size_t(a.rot_dim), size_t(a.vdim)) || a.n_seqs <= 0 || a.tokens <= 0 ||
+        a.tokens >= (int64_t(1) << 31) || a.shared_stride % 8 != 0 || a.out_stride % 8 != 0 || scratch.error_flag == nullptr ||
+        scratch.partials == nullptr || scratch.counters == nullptr || scratch.partials_floats < 2 * size_t(grid) * size_t(kPartialFloats) ||
+        scratch.counters_len < size_t(grid)) {
+        return -1;
+    }
+    for (const void *ptr : {a.q, a.k, a.k_shared, a.v, static_cast<const void *>(a.out), static_cast<const void *>(scratch.partials)}) {
+        if (reinterpret_cast<uintptr_t>(ptr) % 16 != 0) {
+            return -1;
+        }
+    }
+    EncodeTiledFn encode = prefill_encode_fn();
+    if (encode == nullptr) {
+        return -1;
+    }
+    const CUtensorMapDataType type = bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
+    auto map = [&](CUtensorMap *out, const void *base, int rank, const cuuint64_t *dims, const cuuint64_t *strides, const cuuint32_t *box) {
+        const cuuint32_t one[4] = {1, 1, 1, 1};
+        return encode(out, type, cuuint32_t(rank), const_cast<void *>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                      CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+    };
+    const cuuint64_t heads = cuuint64_t(a.nh), tokens = cuuint64_t(a.tokens), dim = cuuint64_t(a.dim), dv = cuuint64_t(a.vdim);
+    // K: 64 dims x 1 head x 64 tokens (dims past `dim` read as zero); what all heads share: 64 dims x 64 tokens; V: a block as its two halves
+    const cuuint64_t k_dims[3] = {dim, heads, tokens}, k_strides[2] = {dim * 2, heads * dim * 2};
+    const cuuint32_t k_box[3] = {64, 1, kBlockN};
+    const cuuint64_t r_dims[2] = {cuuint64_t(a.rot_dim), tokens}, r_strides[1] = {cuuint64_t(a.shared_stride) * 2};
+    const cuuint32_t r_box[2] = {64, kBlockN};
+    const cuuint64_t v_dims[4] = {64, tokens, dv / 64, heads}, v_strides[3] = {heads * dv * 2, 128, dv * 2};
+    const cuuint32_t v_box[4] = {64, kBlockN, 2, 1};
+    CUtensorMap tmap, tmap_v, tmap_r;
+    if (!map(&tmap, a.k, 3, k_dims, k_strides, k_box) || !map(&tmap_v, a.v, 4, v_dims, v_strides, v_box) ||
+        !map(&tmap_r, a.k_shared, 2, r_dims, r_strides, r_box)) {
+        return -1;
+    }
+    PrefillParams p{};
+    p.table_stride = (1 << 30) / kPage; // (no table bounds a sequence)
+    p.kv_lens = a.kv_lens;
+    p.q_starts = a.q_starts;
+    p.page_starts = a.page_starts;
+    p.n_seqs = a.n_seqs;
+    p.nkvh = a.nh;
+    p.group = 1;
+    p.nh = a.nh;
+    p.q = a.q;
+    p.out = a.out;
+    p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.error_flag = scratch.error_flag;
+    p.partials = scratch.partials;
+    p.counters = scratch.counters;
+    p.out_stride = a.out_stride;
+    p.row_scale = a.row_scale;
+    p.dim = a.dim;
+    p.rot = a.rot_dim;
+    p.dv = a.vdim;
+    p.nope_halves = (a.dim + 63) / 64;
+    p.out_wide = reinterpret_cast<uintptr_t>(a.out) % 32 == 0 && p.out_stride % 16 == 0 ? 1 : 0;
+    auto s = static_cast<cudaStream_t>(stream);
+    bf16 ? launch<true, kExpanded>(s, tmap, tmap_v, tmap_r, p, grid, false) : launch<false, kExpanded>(s, tmap, tmap_v, tmap_r, p, grid, false);
+    check_launch("attention_expanded_tc");
     return 0;
 }
 

@@ -244,6 +244,25 @@ void attention_prefill_tc_scratch(size_t *floats, size_t *counters);
 int make_kv_tile_tensor_map(void *out_256_bytes, void *pool_base, uint64_t total_rows, uint32_t nkvh,
                             llaisysDataType_t dtype);
 
+// Decode and short chunks over pages of latents (views whose V rows lie in their K rows) on tcgen05: 16-bit, 16-token pages, V parts of up
+// to 512 elements, rows of whole 16-byte pieces of which at most one 64-element piece lies behind the V part's last 128. batch.q_starts may
+// begin anywhere in q and out (rows are absolute; total_q: rows of this call). Returns -1 if the view or shape is not covered, or the
+// scratch (attention_latent_scratch floats) is too small.
+bool attention_latent_covers(llaisysDataType_t dtype, size_t nh, size_t rank, size_t dim);
+size_t attention_latent_scratch(size_t rank);
+int attention_latent_tc(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch, const void *q, float scale,
+                        const AttnOut &out, const AttnScratch &scratch);
+
+// K4 over plain tensors with keys in two parts (see ExpandedArgs): 16-bit, own parts of up to 128 dims and shared ones of up to 64 in steps
+// of 8, V rows of 64 or 128. Returns -1 if the sizes or the scratch (as attention_prefill_tc) do not fit.
+bool attention_expanded_covers(llaisysDataType_t dtype, size_t dim, size_t rot_dim, size_t vdim);
+int attention_expanded_tc(stream_t stream, llaisysDataType_t dtype, const ExpandedArgs &args, const AttnScratch &scratch);
+
+// Rows [0, kv_lens[i]) of the sequences with page_starts[i] >= 0 (layers whose V rows lie in their K rows) -> out rows 16 page_starts[i] ..,
+// kv.d elements each, out_stride apart, zeros up to the next multiple of 16 rows. max_kv_len: of those sequences.
+void latent_gather(stream_t stream, size_t elem_size, const KVView &kv, void *out, int64_t out_stride, const int32_t *seq_ids,
+                   const int32_t *page_starts, const int32_t *kv_lens, int32_t n_seqs, int32_t max_kv_len, int32_t *error_flag);
+
 // K3: out[r, :] = sum_p w_p o_p[r, :] / sum_p w_p, w_p = l_p exp(m_p - max_p m_p), over n_parts partials laid out
 // float [n_parts][n_rows][d + 2].
 void lse_merge(stream_t stream, llaisysDataType_t dtype, void *out, const float *parts, int32_t n_parts,

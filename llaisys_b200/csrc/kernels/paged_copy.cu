@@ -695,6 +695,34 @@ void launch_latent_append(cudaStream_t s, const KVView &kv, const LatentAppendAr
                         static_cast<T *>(kv.k_base), a, kv.block_table, g, max_blocks, error_flag);
 }
 
+// One CTA per (page, sequence); P: the widest piece that divides a row.
+template <typename P>
+__global__ void __launch_bounds__(128) latent_gather_kernel(const unsigned char *__restrict__ pool, const int32_t *__restrict__ table, CopyGeom g,
+                                                            P *__restrict__ out, int64_t out_pieces, int32_t row_pieces,
+                                                            const int32_t *__restrict__ seq_ids, const int32_t *__restrict__ page_starts,
+                                                            const int32_t *__restrict__ kv_lens, int32_t *error_flag) {
+    asm volatile("griddepcontrol.wait;\n" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    const int32_t i = int32_t(blockIdx.y), blk = int32_t(blockIdx.x), len = kv_lens[i], start = page_starts[i];
+    if (start < 0 || blk * g.page_size >= len) {
+        return;
+    }
+    int32_t page, slot;
+    if (!resolve_slot(table, g, seq_ids[i], blk * g.page_size, g.table_stride, error_flag, page, slot)) {
+        return;
+    }
+    const unsigned char *src = pool + int64_t(page) * g.page_stride_b;
+    P *dst = out + int64_t(start + blk) * g.page_size * out_pieces;
+    for (int32_t u = int32_t(threadIdx.x); u < g.page_size * row_pieces; u += 128) {
+        const int32_t t = u / row_pieces, c = u - t * row_pieces;
+        P v{};
+        if (blk * g.page_size + t < len) {
+            v = reinterpret_cast<const P *>(src + int64_t(t) * g.token_stride_b)[c];
+        }
+        dst[int64_t(t) * out_pieces + c] = v;
+    }
+}
+
 template <typename T>
 void launch_norm_append(cudaStream_t s, const KVView &kv, const NormAppendArgs &a, int32_t max_blocks, int32_t *error_flag) {
     CopyGeom g{};
@@ -927,6 +955,26 @@ void paged_norm_append(stream_t stream, llaisysDataType_t dtype, const KVView &k
         EXCEPTION_UNSUPPORTED_DATATYPE(dtype);
     }
     check_launch("paged_norm_append");
+}
+
+void latent_gather(stream_t stream, size_t elem_size, const KVView &kv, void *out, int64_t out_stride, const int32_t *seq_ids,
+                   const int32_t *page_starts, const int32_t *kv_lens, int32_t n_seqs, int32_t max_kv_len, int32_t *error_flag) {
+    if (n_seqs == 0 || max_kv_len == 0) {
+        return;
+    }
+    const size_t row = size_t(kv.d) * elem_size, step = size_t(out_stride) * elem_size;
+    CHECK_ARGUMENT(row % 16 == 0 && step % 16 == 0 && aligned16(out) && n_seqs <= 65535, "latent gather: rows of whole 16-byte pieces");
+    CopyGeom g{};
+    g.page_stride_b = kv.page_stride * int64_t(elem_size);
+    g.token_stride_b = kv.token_stride * int64_t(elem_size);
+    g.nkvh = 1;
+    g.page_size = kv.page_size;
+    g.num_pages = kv.num_pages;
+    g.table_stride = kv.table_stride;
+    launch_programmatic(latent_gather_kernel<uint4>, dim3(unsigned((max_kv_len + kv.page_size - 1) / kv.page_size), unsigned(n_seqs)), 128u,
+                        static_cast<cudaStream_t>(stream), static_cast<const unsigned char *>(kv.k_base), kv.block_table, g,
+                        static_cast<uint4 *>(out), int64_t(step / 16), int32_t(row / 16), seq_ids, page_starts, kv_lens, error_flag);
+    check_launch("latent_gather");
 }
 
 void latent_append(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const LatentAppendArgs &args, int32_t max_blocks,

@@ -130,6 +130,14 @@ PagedKV::PagedKV(const PagedKVConfig &cfg) : _cfg(cfg) {
             _partials_floats = std::max(floats, f2);
             _counters_len = std::max(counters, c2);
         }
+        for (const Layer &l : _layers) { // layers whose V rows lie in their K rows
+            if (l.v_row == 0 && l.nkvh == 1 && cfg.page_size == 16 && kernels::attention_latent_covers(cfg.dtype, 1, l.v_dim, l.k_dim)) {
+                size_t f2 = 0, c2 = 0;
+                kernels::attention_prefill_tc_scratch(&f2, &c2);
+                _partials_floats = std::max({_partials_floats, kernels::attention_latent_scratch(l.v_dim), f2});
+                _counters_len = std::max(_counters_len, c2);
+            }
+        }
         size_t longest_v = 0; // of the layers that the gated tile kernel can serve
         for (const Layer &l : _layers) {
             longest_v = std::max(longest_v, l.k_dim <= 128 && l.v_dim <= 128 ? l.v_dim : 0);
@@ -700,6 +708,56 @@ void PagedKV::latentAppendDev(size_t layer, const kernels::LatentAppendArgs &arg
 #endif
 }
 
+bool PagedKV::latentTc(size_t layer, size_t nh) const {
+#ifdef ENABLE_NVIDIA_API
+    const Layer &l = _layers.at(layer);
+    return onDevice() && l.v_row == 0 && l.nkvh == 1 && _cfg.page_size == 16 && l.k_row == l.k_dim &&
+           kernels::attention_latent_covers(_cfg.dtype, nh, l.v_dim, l.k_dim);
+#else
+    (void)layer, (void)nh;
+    return false;
+#endif
+}
+
+bool PagedKV::canExpand(size_t layer, size_t dim, size_t rot_dim, size_t vdim) const {
+#ifdef ENABLE_NVIDIA_API
+    return latentTc(layer, 1) && kernels::attention_expanded_covers(_cfg.dtype, dim, rot_dim, vdim);
+#else
+    (void)layer, (void)dim, (void)rot_dim, (void)vdim;
+    return false;
+#endif
+}
+
+void PagedKV::latentGatherDev(size_t layer, void *out, int64_t out_stride, const int32_t *seq_ids_dev, const int32_t *page_starts_dev,
+                              const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len, llaisysStream_t stream) {
+    checkLayer(layer);
+    KV_REQUIRE(onDevice() && _layers[layer].v_row == 0 && out_stride >= int64_t(_layers[layer].k_dim), LLAISYS_E_INVALID,
+               "paged KV latent gather: this layer holds no latents of this size");
+    KV_REQUIRE(max_kv_len <= _cfg.page_size * _cfg.max_pages_per_seq, LLAISYS_E_INVALID, "paged KV latent gather: context too large for this cache");
+#ifdef ENABLE_NVIDIA_API
+    enter();
+    kernels::latent_gather(stream, _elem, view(layer), out, out_stride, seq_ids_dev, page_starts_dev, kv_lens_dev, int32_t(n_seqs),
+                           int32_t(max_kv_len), reinterpret_cast<int32_t *>(_error_dev->memory()));
+#else
+    (void)out, (void)seq_ids_dev, (void)page_starts_dev, (void)kv_lens_dev, (void)n_seqs, (void)stream;
+#endif
+}
+
+void PagedKV::expandedDev(const kernels::ExpandedArgs &args, llaisysStream_t stream) {
+#ifdef ENABLE_NVIDIA_API
+    KV_REQUIRE(onDevice(), LLAISYS_E_UNSUPPORTED, "expanded attention: NVIDIA caches only");
+    enter();
+    if (kernels::attention_expanded_tc(stream, _cfg.dtype, args, scratch()) != 0) {
+        fail(LLAISYS_E_UNSUPPORTED, "expanded attention (tcgen05 kernel): sizes or alignment not covered, or the workspace is missing");
+    }
+    _last_kernel = LLAISYS_KERNEL_EXPANDED_TC;
+    noteAttentionKernel(_last_kernel);
+#else
+    (void)args, (void)stream;
+    fail(LLAISYS_E_UNSUPPORTED, "this build has no NVIDIA backend");
+#endif
+}
+
 void PagedKV::decodeDev(size_t layer, void *out, float *part, const void *q, const int32_t *seq_ids_dev,
                         const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len, size_t nh, float scale,
                         llaisysStream_t stream, const AttnOptions &opt) {
@@ -1140,7 +1198,9 @@ int run_attention_nvidia(llaisysStream_t stream, llaisysDataType_t dtype, const 
     const bool one_query_each = batch.q_starts == nullptr && batch.const_q_len == 1;
     const bool fast = fast_shape(dtype, view, batch);
     int used = LLAISYS_KERNEL_GENERIC;
-    if (fast && one_query_each && view.block_table != nullptr && batch.kv_lens != nullptr) {
+    if (kernels::attention_latent_tc(stream, dtype, view, batch, q, scale, out, scratch) == 0) { // (V rows inside K rows)
+        used = LLAISYS_KERNEL_LATENT_TC;
+    } else if (fast && one_query_each && view.block_table != nullptr && batch.kv_lens != nullptr) {
         // a page pool: the TMA kernel, or nothing
         const char *why = nullptr;
         if (kernels::attention_decode_tma(stream, dtype, view, batch, q, scale, out, scratch, nullptr, nullptr, &why) != 0) {

@@ -135,6 +135,15 @@ public:
     void normAppendDev(size_t layer, const kernels::NormAppendArgs &args, llaisysStream_t stream);
     // The same for latents: see kernels::latent_append. Layers with v_in_k and one kv head.
     void latentAppendDev(size_t layer, const kernels::LatentAppendArgs &args, llaisysStream_t stream);
+    // Long chunks over latents: the rows of chosen sequences side by side (see kernels::latent_gather), and attention over the keys
+    // and values a model makes of them, with this cache's workspace. canExpand: whether the kernels take these sizes.
+    bool canExpand(size_t layer, size_t dim, size_t rot_dim, size_t vdim) const;
+    void latentGatherDev(size_t layer, void *out, int64_t out_stride, const int32_t *seq_ids_dev, const int32_t *page_starts_dev,
+                         const int32_t *kv_lens_dev, size_t n_seqs, size_t max_kv_len, llaisysStream_t stream);
+    void expandedDev(const kernels::ExpandedArgs &args, llaisysStream_t stream);
+    // Decode and short chunks over latents run on the tensor-core kernel (which takes calls over a part of a batch: q_starts may begin
+    // anywhere in q and out)
+    bool latentTc(size_t layer, size_t nh) const;
 
 private:
     struct Seq {

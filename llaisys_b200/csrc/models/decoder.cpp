@@ -352,6 +352,10 @@ void Decoder::stepRows(const int32_t *seq_ids, const int32_t *n_tokens, size_t n
     shape.max_kv_len = max_kv;
     shape.decode_only = decode_only;
     shape.out_is_all = out_is_all;
+    if (!decode_only) {
+        shape.host_q_starts = host(a.q_starts);
+        shape.host_kv_lens = host(a.kv_lens);
+    }
     copyToDevice(dev0, host0, _meta_bytes);
     _cache->flush();
     bool replayed = false;

@@ -93,6 +93,8 @@ protected:
         size_t max_q_len = 0, max_kv_len = 0;
         bool decode_only = false;   // one token per sequence
         bool out_is_all = false;    // logits are wanted for every row, in order (no gather needed)
+        // the same as StepArrays::q_starts and kv_lens in host memory, valid during forward(); null in decode steps
+        const int32_t *host_q_starts = nullptr, *host_kv_lens = nullptr;
     };
 
     // ---- what a model supplies ----

@@ -12,6 +12,12 @@
 
 namespace llaisys::models {
 
+namespace {
+constexpr size_t kExpandFrom = 128;    // tokens of a chunk from which keys and values of its context are made
+constexpr size_t kPassTokens = 65536;  // context rows that are expanded together (one sequence alone may have more)
+constexpr size_t kTailRows = 64;       // zero rows behind the last context: key blocks of 64 may reach into them
+} // namespace
+
 // ---- construction -------------------------------------------------------------------------------------------------------
 
 Folivik::Folivik(const LlaisysFolivikMeta &meta, llaisysDeviceType_t device, int device_id)
@@ -276,10 +282,7 @@ void Folivik::ensureActivations(size_t n_tokens, size_t n_out) {
 void Folivik::latentAttention(const Layer &l, const StepArrays &a, const StepShape &s) {
 #ifdef ENABLE_NVIDIA_API
     const LlaisysLatentAttentionMeta &m = l.meta.latent;
-    const size_t T = s.n_tokens, H = m.heads, row = m.kv_rank + m.rot_dim, dim = m.dim + m.rot_dim;
-    const float *table = m.rot_dim != 0 ? reinterpret_cast<const float *>(_rotary[l.rotary].table->memory()) : nullptr;
-    std::byte *q = _q->memory(), *wide = _q_wide->memory(), *out = wide + T * H * row * _elem;
-    float *scale = reinterpret_cast<float *>(_scale->memory());
+    const size_t T = s.n_tokens, H = m.heads;
     kernels::LatentAppendArgs n;
     n.proj = _proj->memory();
     n.row_stride = int64_t(l.n_proj);
@@ -293,29 +296,143 @@ void Folivik::latentAttention(const Layer &l, const StepArrays &a, const StepSha
     n.q_norm = l.q_norm;
     n.kv_norm = l.k_norm;
     n.eps = _meta.eps;
-    n.rot_table = table;
+    n.rot_table = m.rot_dim != 0 ? reinterpret_cast<const float *>(_rotary[l.rotary].table->memory()) : nullptr;
     n.q_latent = _latent->memory();
     n.q_latent_stride = int64_t(l.q_rank);
-    n.row_scale = scale;
+    n.row_scale = reinterpret_cast<float *>(_scale->memory());
     n.seq_ids = a.seq32;
     n.positions = a.pos32;
     n.n_rows = T;
     _cache->latentAppendDev(l.index, n, _stream);
-    kernels::linear(_stream, _dtype, q, _latent->memory(), l.uq, nullptr, T, H * dim, l.q_rank);
-    kernels::linear_heads(_stream, _dtype, wide, q, l.uk, T, H, m.kv_rank, m.dim, true, H * dim, dim, H * row, row);
-    kernels::rotate_pairs(_stream, _dtype, wide, row, m.kv_rank, q, m.dim, m.rot_dim, table, T, H);
-    kv::AttnOptions opt;
-    opt.row_scale = scale;
-    if (s.decode_only) {
-        _cache->decodeDev(l.index, out, nullptr, wide, a.seq_list, a.kv_lens, s.n_seqs, s.max_kv_len, H, m.scale, _stream, opt);
-    } else {
-        _cache->prefillDev(l.index, out, wide, a.seq_list, a.q_starts, a.kv_lens, s.n_seqs, T, s.max_q_len, s.max_kv_len, H, m.scale, _stream,
-                           opt);
+    kernels::linear(_stream, _dtype, _q->memory(), _latent->memory(), l.uq, nullptr, T, H * (m.dim + m.rot_dim), l.q_rank);
+    if (s.decode_only || !_cache->latentTc(l.index, H) || !_cache->canExpand(l.index, m.dim, m.rot_dim, m.vdim)) {
+        latentRange(l, a, s, LatentRange{false, 0, s.n_seqs, 0, T, s.max_q_len, s.max_kv_len, 0});
+        return;
     }
-    kernels::linear_heads(_stream, _dtype, _mix->memory(), out, l.uv, T, H, m.vdim, m.kv_rank, false, H * m.kv_rank, m.kv_rank, l.n_mix, m.vdim);
+    for (const LatentRange &r : _ranges) {
+        r.expanded ? expandedRange(l, a, s, r) : latentRange(l, a, s, r);
+    }
 #else
     (void)l, (void)a, (void)s;
 #endif
+}
+
+// Sequences whose queries are multiplied into the latents' space
+void Folivik::latentRange(const Layer &l, const StepArrays &a, const StepShape &s, const LatentRange &r) {
+#ifdef ENABLE_NVIDIA_API
+    const LlaisysLatentAttentionMeta &m = l.meta.latent;
+    const size_t T = s.n_tokens, H = m.heads, row = m.kv_rank + m.rot_dim, dim = m.dim + m.rot_dim;
+    const float *table = m.rot_dim != 0 ? reinterpret_cast<const float *>(_rotary[l.rotary].table->memory()) + r.row * m.rot_dim : nullptr;
+    std::byte *wide = _q_wide->memory(), *out = wide + T * H * row * _elem; // (whole steps: the attention kernels take absolute rows)
+    const std::byte *q = _q->memory() + r.row * H * dim * _elem;
+    std::byte *q_rows = wide + r.row * H * row * _elem;
+    kernels::linear_heads(_stream, _dtype, q_rows, q, l.uk, r.n_rows, H, m.kv_rank, m.dim, true, H * dim, dim, H * row, row);
+    kernels::rotate_pairs(_stream, _dtype, q_rows, row, m.kv_rank, q, m.dim, m.rot_dim, table, r.n_rows, H);
+    kv::AttnOptions opt;
+    opt.row_scale = reinterpret_cast<const float *>(_scale->memory());
+    const size_t n = r.to - r.from;
+    if (s.decode_only) {
+        _cache->decodeDev(l.index, out, nullptr, wide, a.seq_list, a.kv_lens, n, s.max_kv_len, H, m.scale, _stream, opt);
+    } else {
+        _cache->prefillDev(l.index, out, wide, a.seq_list + r.from, a.q_starts + r.from, a.kv_lens + r.from, n, r.n_rows, r.max_q_len,
+                           r.max_kv_len, H, m.scale, _stream, opt);
+    }
+    kernels::linear_heads(_stream, _dtype, _mix->memory() + r.row * l.n_mix * _elem, out + r.row * H * m.kv_rank * _elem, l.uv, r.n_rows, H,
+                          m.vdim, m.kv_rank, false, H * m.kv_rank, m.kv_rank, l.n_mix, m.vdim);
+#else
+    (void)l, (void)a, (void)s, (void)r;
+#endif
+}
+
+// Sequences whose contexts' rows become keys and values
+void Folivik::expandedRange(const Layer &l, const StepArrays &a, const StepShape &s, const LatentRange &r) {
+#ifdef ENABLE_NVIDIA_API
+    (void)s;
+    const LlaisysLatentAttentionMeta &m = l.meta.latent;
+    const size_t H = m.heads, row = m.kv_rank + m.rot_dim, dim = m.dim + m.rot_dim, n = r.to - r.from;
+    const int32_t *starts = reinterpret_cast<const int32_t *>(_page_starts->memory()) + r.from;
+    const float *table = reinterpret_cast<const float *>(_rotary[l.rotary].table->memory()) + r.row * m.rot_dim;
+    std::byte *context = _context->memory(), *q = _q->memory() + r.row * H * dim * _elem;
+    _cache->latentGatherDev(l.index, context, int64_t(row), a.seq_list + r.from, starts, a.kv_lens + r.from, n, r.max_kv_len, _stream);
+    kernels::fill_zero(_stream, context + (r.tokens - kTailRows) * row * _elem, kTailRows * row * _elem);
+    kernels::linear(_stream, _dtype, _keys->memory(), context, l.uk, nullptr, r.tokens, H * m.dim, m.kv_rank, false, row);
+    kernels::linear(_stream, _dtype, _values->memory(), context, l.uv, nullptr, r.tokens, H * m.vdim, m.kv_rank, false, row);
+    kernels::rotate_pairs(_stream, _dtype, q, dim, m.dim, q, m.dim, m.rot_dim, table, r.n_rows, H);
+    kernels::ExpandedArgs e;
+    e.q = _q->memory();
+    e.k = _keys->memory();
+    e.k_shared = context + m.kv_rank * _elem;
+    e.shared_stride = int64_t(row);
+    e.v = _values->memory();
+    e.tokens = int64_t(r.tokens);
+    e.nh = int32_t(H);
+    e.dim = int32_t(m.dim);
+    e.rot_dim = int32_t(m.rot_dim);
+    e.vdim = int32_t(m.vdim);
+    e.page_starts = starts;
+    e.q_starts = a.q_starts + r.from;
+    e.kv_lens = a.kv_lens + r.from;
+    e.n_seqs = int32_t(n);
+    e.scale = m.scale;
+    e.out = _mix->memory();
+    e.out_stride = int64_t(l.n_mix);
+    e.row_scale = reinterpret_cast<const float *>(_scale->memory());
+    _cache->expandedDev(e, _stream);
+#else
+    (void)l, (void)a, (void)s, (void)r;
+#endif
+}
+
+// Cuts a step's sequences into ranges, and makes room for the contexts of those that are expanded.
+void Folivik::planLatents(const StepShape &s) {
+    _ranges.clear();
+    size_t row = 0, keys = 0, values = 0, tokens = 0;
+    for (const Layer &l : _layers) {
+        const LlaisysLatentAttentionMeta &m = l.meta.latent;
+        if (l.meta.mixer == LLAISYS_FOLIVIK_LATENT && _cache->canExpand(l.index, m.dim, m.rot_dim, m.vdim)) {
+            row = std::max(row, m.kv_rank + m.rot_dim);
+            keys = std::max(keys, m.heads * m.dim);
+            values = std::max(values, m.heads * m.vdim);
+        }
+    }
+    if (row == 0 || s.decode_only) {
+        return;
+    }
+    _page_starts_host.assign(s.n_seqs, -1);
+    bool any = false;
+    for (size_t i = 0; i < s.n_seqs; ++i) {
+        const size_t first = size_t(s.host_q_starts[i]), n = size_t(s.host_q_starts[i + 1]) - first, len = size_t(s.host_kv_lens[i]);
+        const size_t padded = (len + 15) / 16 * 16;
+        const bool expanded = n >= kExpandFrom;
+        if (_ranges.empty() || _ranges.back().expanded != expanded || (expanded && _ranges.back().tokens + padded > kPassTokens)) {
+            _ranges.push_back(LatentRange{expanded, i, i, first, 0, 0, 0, expanded ? kTailRows : 0});
+        }
+        LatentRange &r = _ranges.back();
+        if (expanded) {
+            _page_starts_host[i] = int32_t((r.tokens - kTailRows) / 16);
+            r.tokens += padded;
+            any = true;
+        }
+        r.to = i + 1;
+        r.n_rows += n;
+        r.max_q_len = std::max(r.max_q_len, n);
+        r.max_kv_len = std::max(r.max_kv_len, len);
+        tokens = std::max(tokens, r.tokens);
+    }
+    if (!any) {
+        return;
+    }
+    auto &rt = enter();
+    auto grow = [&](core::storage_t &block, size_t bytes) {
+        if (!block || block->size() < bytes) {
+            block = rt.allocateDeviceStorage(bytes);
+        }
+    };
+    grow(_page_starts, s.n_seqs * sizeof(int32_t));
+    grow(_context, tokens * row * _elem);
+    grow(_keys, tokens * keys * _elem);
+    grow(_values, tokens * values * _elem);
+    copyToDevice(_page_starts->memory(), _page_starts_host.data(), s.n_seqs * sizeof(int32_t));
 }
 
 void Folivik::windowAttention(const Layer &l, const StepArrays &a, const StepShape &s) {
@@ -459,6 +576,7 @@ void Folivik::forward(const StepArrays &a, const StepShape &s) {
         kernels::rotary_table(_stream, reinterpret_cast<float *>(r.table->memory()), a.pos32, reinterpret_cast<const double *>(r.freq->memory()),
                               T, r.dims / 2);
     }
+    planLatents(s);
     bool normed = false; // h holds the norm of x that the coming layer reads
     for (size_t i = 0; i < _layers.size(); ++i) {
         const Layer &l = _layers[i];

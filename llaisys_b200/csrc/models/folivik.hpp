@@ -6,7 +6,9 @@
 // into the stream), and one kernel for the weighted sum, the residual and the norm of the next layer.
 //
 // Latent attention caches one row per token, [latent | turned key part], for all heads. The unrotated query is multiplied into the
-// latent's space (W_uk of its head), attention runs over the rows as they are, and W_uv of each head follows.
+// latent's space (W_uk of its head), attention runs over the rows as they are, and W_uv of each head follows. For long chunks that
+// is more arithmetic than making keys and values of the contexts' rows once and running ordinary attention over them: chunks of at
+// least kExpandFrom tokens do so, a pass over neighbouring sequences at a time.
 #pragma once
 
 #include "llaisys/models/folivik.h"
@@ -49,11 +51,20 @@ private:
         core::storage_t table; // of the step's rows
     };
 
+    // Neighbouring sequences [from, to) of a step that are served alike, their rows, and for expanded ones the rows of their contexts
+    struct LatentRange {
+        bool expanded;
+        size_t from, to, row, n_rows, max_q_len, max_kv_len, tokens;
+    };
+
     kv::PagedKVConfig cacheShape() const override;
     std::vector<size_t> stateShape() const override;
     void ensureActivations(size_t n_tokens, size_t n_out) override;
     void forward(const StepArrays &a, const StepShape &s) override;
     void latentAttention(const Layer &l, const StepArrays &a, const StepShape &s);
+    void latentRange(const Layer &l, const StepArrays &a, const StepShape &s, const LatentRange &r);
+    void expandedRange(const Layer &l, const StepArrays &a, const StepShape &s, const LatentRange &r);
+    void planLatents(const StepShape &s);
     void windowAttention(const Layer &l, const StepArrays &a, const StepShape &s);
     void stateSpace(const Layer &l, const StepArrays &a, const StepShape &s);
     void experts(const Layer &l, const StepShape &s, const float *next_gain);
@@ -66,6 +77,9 @@ private:
     float *_final_norm = nullptr;
 
     core::storage_t _x, _h, _proj, _q, _q_wide, _latent, _scale, _mix, _scratch, _segments, _h_out;
+    std::vector<LatentRange> _ranges; // of the current step
+    std::vector<int32_t> _page_starts_host;
+    core::storage_t _page_starts, _context, _keys, _values; // expanded: context rows, keys and values made of them
     core::storage_t _logits_e, _choice, _counts, _rows, _act, _expert_out, _shared; // experts
 };
 

@@ -33,6 +33,8 @@ class Kernel(IntEnum):
     GATES = 7
     GATES_TILES = 8
     GATES_TC = 9
+    LATENT_TC = 10
+    EXPANDED_TC = 11
 
 
 def last_attention_kernel() -> Kernel:
