@@ -1,8 +1,9 @@
 /*
  * llaisys C ABI -- token mixers beyond plain causal attention, on device buffers and an explicit stream: caches whose
  * layers differ in shape, attention with a sliding window (that can keep a sequence's first tokens) and an output factor per
- * head, attention without a softmax whose weights are mixed over the heads, the norm / rotation + append in front of them, and
- * gated linear attention, the gated delta rule and minGRU with recurrent state.
+ * head or a penalty on distance, attention over latents, attention without a softmax whose weights are mixed over the heads, the norm /
+ * rotation + append in front of them, gated linear attention, the gated delta rule, minGRU and the Mamba-2 state space with recurrent
+ * state, and mixtures of experts.
  * NVIDIA devices. No counterpart in the reference.
  * Status codes as in paged_kv.h; as for every ...Dev call there: no host validation of index arrays, no staging copy.
  */
@@ -44,10 +45,14 @@ struct LlaisysNormAppend {
     int row_norm;
     const void *bias;
     float temp_coef, temp_every;
+    const float *head_scale; /* [nh] f32, not the row form: factor on every query head after norm and rotation (NULL: none) */
 };
 /* table[row, i] = (cos, sin)(positions[row] * freq[i]), i < half, all on the device */
 LLAISYS_API int llaisysRotaryTableDev(llaisysDeviceType_t device_type, int device_id, float *table, const int32_t *positions_dev,
                                       const float *freq_dev, size_t n_rows, size_t half, llaisysStream_t stream);
+/* the same with angles formed and reduced in f64 */
+LLAISYS_API int llaisysRotaryTableWideDev(llaisysDeviceType_t device_type, int device_id, float *table, const int32_t *positions_dev,
+                                          const double *freq_dev, size_t n_rows, size_t half, llaisysStream_t stream);
 LLAISYS_API int llaisysPagedKVNormAppendDev(llaisysPagedKV_t kv, size_t layer, const struct LlaisysNormAppend *args,
                                             llaisysStream_t stream);
 
@@ -60,6 +65,66 @@ LLAISYS_API int llaisysPagedAttentionOptDev(llaisysPagedKV_t kv, size_t layer, v
                                             size_t n_seqs, size_t total_q, size_t max_q_len, size_t max_kv_len, size_t nh,
                                             float scale, size_t window, size_t keep_first, const float *row_scale,
                                             size_t row_stride, llaisysStream_t stream);
+
+/* The same without kept tokens and factors, with a penalty on distance: fade_a[h] ln(1 + fade_b[h] (i - j)) is taken off head h's score of
+ * key j for the query at position i, after the scale. fade_a, fade_b [nh] f32 on the device, fade_b >= 0. */
+LLAISYS_API int llaisysPagedAttentionFadeDev(llaisysPagedKV_t kv, size_t layer, void *out, const void *q, const int32_t *seq_ids_dev,
+                                             const int32_t *q_starts_dev, const int32_t *kv_lens_dev, size_t n_seqs, size_t total_q,
+                                             size_t max_q_len, size_t max_kv_len, size_t nh, float scale, size_t window,
+                                             const float *fade_a, const float *fade_b, size_t row_stride, llaisysStream_t stream);
+
+/* ---- latents ----
+ * A cache whose layers hold ONE row of rank[l] + rot_dim[l] elements per token: keys are whole rows, values their first rank elements, for
+ * all heads. llaisysPagedAttentionOptDev runs over it with queries [rows, nh, rank + rot_dim] and outputs [rows, nh, rank]. */
+LLAISYS_API int llaisysPagedKVCreateLatents(llaisysPagedKV_t *kv_out, llaisysDeviceType_t device_type, int device_id,
+                                            llaisysDataType_t dtype, size_t nlayer, const size_t *rank, const size_t *rot_dim,
+                                            size_t num_pages, size_t page_size, size_t max_seqs, size_t max_pages_per_seq);
+
+/* Of a projection row: the q_rank elements at q_at, divided by their root mean square (eps inside the root) and weighted with q_norm, go to
+ * q_latent (rows q_latent_stride apart); the rank elements at kv_at, treated alike with kv_norm, and behind them the next rot_dims
+ * elements, dims 2 i and 2 i + 1 turned by the angle whose cosine and sine are rot_table[row][i], go to token positions[i] of sequence
+ * seq_ids[i]; row_scale [n_rows, nh] (NULL: none) becomes the sigmoid of the nh elements at gate_at (< 0: 1). */
+struct LlaisysLatentAppend {
+    const void *proj;
+    int64_t row_stride, q_at, kv_at, gate_at;
+    size_t q_rank, rank, rot_dims, nh;
+    const void *q_norm, *kv_norm;
+    float eps;
+    const float *rot_table;
+    void *q_latent;
+    int64_t q_latent_stride;
+    float *row_scale;
+    const int32_t *seq_ids_dev, *positions_dev;
+    size_t n_rows;
+};
+LLAISYS_API int llaisysPagedKVLatentAppendDev(llaisysPagedKV_t kv, size_t layer, const struct LlaisysLatentAppend *args,
+                                              llaisysStream_t stream);
+/* out[r, h, out_at ..] = the rot_dims elements of q [n_rows, nh, dim + rot_dims] behind the first dim, turned as above; out rows of heads
+ * out_dim apart; out may be q (out_dim = dim + rot_dims, out_at = dim) */
+LLAISYS_API int llaisysRotatePairsDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype, void *out, size_t out_dim,
+                                      size_t out_at, const void *q, size_t dim, size_t rot_dims, const float *rot_table, size_t n_rows,
+                                      size_t nh, llaisysStream_t stream);
+/* Rows of the sequences with page_starts[i] >= 0, side by side: token t of sequence i -> row 16 page_starts[i] + t of out (rows out_stride
+ * elements apart), zero rows up to the next multiple of 16. max_kv_len: of those sequences. */
+LLAISYS_API int llaisysPagedKVLatentGatherDev(llaisysPagedKV_t kv, size_t layer, void *out, int64_t out_stride,
+                                              const int32_t *seq_ids_dev, const int32_t *page_starts_dev, const int32_t *kv_lens_dev,
+                                              size_t n_seqs, size_t max_kv_len, llaisysStream_t stream);
+/* Causal attention of ragged chunks over plain keys and values, 16-bit, on tcgen05: a head's key is its own `dim` elements of k [tokens,
+ * nh, dim] and rot_dim elements that all heads share (row t at k_shared + t * shared_stride); v [tokens, nh, vdim], vdim 64 or 128. Sequence
+ * i's keys begin at row 16 page_starts[i] (< 0: left out); key blocks of 64 may read past a sequence's end, so rows up to the next multiple of
+ * 64 must exist and be finite. out: row r, head h at r * out_stride + h * vdim, times row_scale[r, h] (NULL: 1). Uses kv's workspace. */
+struct LlaisysExpandedAttention {
+    const void *q, *k, *k_shared, *v;
+    int64_t shared_stride;
+    size_t tokens, nh, dim, rot_dim, vdim;
+    const int32_t *page_starts_dev, *q_starts_dev, *kv_lens_dev;
+    size_t n_seqs;
+    float scale;
+    void *out;
+    int64_t out_stride;
+    const float *row_scale;
+};
+LLAISYS_API int llaisysPagedAttentionExpandedDev(llaisysPagedKV_t kv, const struct LlaisysExpandedAttention *args, llaisysStream_t stream);
 
 /* Attention without a softmax over the pages: head h gives key j <= i (with i - j < window, if window > 0) the weight
  *     a_hij = sigmoid(s - slopes[h] * (i - j) + bias[h]),   s = softcap * tanh(scale <q, k> / softcap)   (softcap <= 0: scale <q, k>)
@@ -170,6 +235,61 @@ LLAISYS_API int llaisysGatedDeltaDev(llaisysDeviceType_t device_type, int device
 /* Floats of a sequence's state, of `scratch` for n_rows rows and of `scratch_segments` (any pointer may be NULL). */
 LLAISYS_API void llaisysGatedDeltaSizes(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t kv_heads, size_t dk, size_t dv,
                                         size_t taps, size_t *state_floats, size_t *scratch_floats, size_t *segment_floats);
+
+/* Mamba-2 state space. x (heads x dv), B and C (groups x dk each) follow one another at x_at of a projection row; each channel passes a
+ * causal convolution over time of `taps` taps (conv_w [channels, taps], the last tap is the current token's, zeros before a sequence's
+ * start; conv_b [channels]) and silu. Per head, with state S [dk, dv] in f32 (head h uses group h / (heads / groups)):
+ *     dt = softplus(dt_t + dt_bias_h),  S_t = exp(-exp(a_log_h) dt) S_{t-1} + dt B_t x_t^T,  y_t = S_t^T C_t + d_skip_h x_t
+ * out = norm_w * u / sqrt(mean(u^2) + eps), u = y * silu(z), the mean over each of norm_groups equal parts of the heads x dv outputs. dt_t:
+ * heads numbers at dt_at; z: heads x dv at z_at. a_log, dt_bias, d_skip [heads] f32; all else of `dtype` but state and scratch. state: slot s of
+ * a sequence holds [heads][dk][dv], then the convolutions' inputs [taps][channels] (position p at p mod taps). Sequences, rows and
+ * `decode` as for LlaisysGatedLinear. scratch is 16-byte aligned; with scratch_segments long runs are cut into segments that start in parallel. */
+struct LlaisysStateSpace {
+    const void *proj;
+    int64_t row_stride, z_at, x_at, dt_at;
+    const void *conv_w, *conv_b, *norm_w;
+    const float *a_log, *dt_bias, *d_skip;
+    size_t taps, heads, groups, dk, dv, norm_groups;
+    float eps;
+    float *state;
+    int64_t slot_stride;
+    const int32_t *seq_ids_dev, *q_starts_dev, *kv_lens_dev;
+    size_t n_seqs, n_rows, max_q_len;
+    void *out;
+    int64_t out_stride;
+    float *scratch;
+    size_t scratch_floats;
+    float *scratch_segments;
+    size_t scratch_segment_floats;
+};
+LLAISYS_API int llaisysStateSpaceDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype,
+                                     const struct LlaisysStateSpace *args, int decode, llaisysStream_t stream);
+/* Floats of a sequence's state, of `scratch` for n_rows rows and of `scratch_segments` (any pointer may be NULL). */
+LLAISYS_API void llaisysStateSpaceSizes(llaisysDataType_t dtype, size_t n_rows, size_t heads, size_t groups, size_t dk, size_t dv, size_t taps,
+                                        size_t *state_floats, size_t *scratch_floats, size_t *segment_floats);
+
+/* Mixture of experts over rows h [n_rows, width]. Scores s = softmax(logits) over experts + identity outputs; the `top` largest of
+ * s + correction are chosen, among the best `keep` of `groups` equal groups of neighbours (a group counts as much as its best); weight of a
+ * chosen one: scale * s / (sum of the chosen s + 1e-20). Expert e: down_e (silu(gate_e h) * up_e h), gate_up [experts][gate rows, up rows][width]
+ * with ff rows each, down [experts][width][ff]; outputs from `experts` on are h itself. x [n_rows, width] f32 += the weighted sum;
+ * next (NULL: none) = x / sqrt(mean(x^2) + eps) * *gain of the new x, and may be h. chosen and weights [n_rows, top] are results too.
+ * place, line [n_rows, top], rows and out [n_rows, top, width], act [n_rows, top, ff]: scratch; counts [experts] zero before the first
+ * call (left zero). */
+struct LlaisysExperts {
+    size_t experts, identity, top, groups, keep, width, ff, n_rows;
+    float scale, eps;
+    const void *gate_up, *down;
+    const float *correction, *logits, *gain;
+    const void *h;
+    int32_t *chosen;
+    float *weights;
+    int32_t *place, *counts, *line;
+    void *rows, *act, *out;
+    float *x;
+    void *next;
+};
+LLAISYS_API int llaisysExpertsDev(llaisysDeviceType_t device_type, int device_id, llaisysDataType_t dtype, const struct LlaisysExperts *args,
+                                  llaisysStream_t stream);
 
 #ifdef __cplusplus
 }

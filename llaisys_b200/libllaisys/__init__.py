@@ -219,7 +219,43 @@ class LlaisysNormAppend(Structure):
                 ("gate_at", c_int64), ("q_norm", c_void_p), ("k_norm", c_void_p), ("eps", c_float), ("gate_scale", c_float),
                 ("q_out", c_void_p), ("row_scale", c_void_p), ("seq_ids_dev", c_void_p), ("positions_dev", c_void_p),
                 ("n_rows", c_size_t), ("nh", c_size_t), ("rot_dims", c_size_t), ("rot_table", c_void_p), ("row_norm", c_int),
-                ("bias", c_void_p), ("temp_coef", c_float), ("temp_every", c_float)]
+                ("bias", c_void_p), ("temp_coef", c_float), ("temp_every", c_float), ("head_scale", c_void_p)]
+
+
+class LlaisysLatentAppend(Structure):
+    """struct LlaisysLatentAppend (include/llaisys/mixers.h)."""
+    _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("q_at", c_int64), ("kv_at", c_int64), ("gate_at", c_int64),
+                ("q_rank", c_size_t), ("rank", c_size_t), ("rot_dims", c_size_t), ("nh", c_size_t), ("q_norm", c_void_p),
+                ("kv_norm", c_void_p), ("eps", c_float), ("rot_table", c_void_p), ("q_latent", c_void_p), ("q_latent_stride", c_int64),
+                ("row_scale", c_void_p), ("seq_ids_dev", c_void_p), ("positions_dev", c_void_p), ("n_rows", c_size_t)]
+
+
+class LlaisysExpandedAttention(Structure):
+    """struct LlaisysExpandedAttention (include/llaisys/mixers.h)."""
+    _fields_ = [("q", c_void_p), ("k", c_void_p), ("k_shared", c_void_p), ("v", c_void_p), ("shared_stride", c_int64), ("tokens", c_size_t),
+                ("nh", c_size_t), ("dim", c_size_t), ("rot_dim", c_size_t), ("vdim", c_size_t), ("page_starts_dev", c_void_p),
+                ("q_starts_dev", c_void_p), ("kv_lens_dev", c_void_p), ("n_seqs", c_size_t), ("scale", c_float), ("out", c_void_p),
+                ("out_stride", c_int64), ("row_scale", c_void_p)]
+
+
+class LlaisysStateSpace(Structure):
+    """struct LlaisysStateSpace (include/llaisys/mixers.h)."""
+    _fields_ = [("proj", c_void_p), ("row_stride", c_int64), ("z_at", c_int64), ("x_at", c_int64), ("dt_at", c_int64),
+                ("conv_w", c_void_p), ("conv_b", c_void_p), ("norm_w", c_void_p), ("a_log", c_void_p), ("dt_bias", c_void_p),
+                ("d_skip", c_void_p), ("taps", c_size_t), ("heads", c_size_t), ("groups", c_size_t), ("dk", c_size_t), ("dv", c_size_t),
+                ("norm_groups", c_size_t), ("eps", c_float), ("state", c_void_p), ("slot_stride", c_int64), ("seq_ids_dev", c_void_p),
+                ("q_starts_dev", c_void_p), ("kv_lens_dev", c_void_p), ("n_seqs", c_size_t), ("n_rows", c_size_t),
+                ("max_q_len", c_size_t), ("out", c_void_p), ("out_stride", c_int64), ("scratch", c_void_p), ("scratch_floats", c_size_t),
+                ("scratch_segments", c_void_p), ("scratch_segment_floats", c_size_t)]
+
+
+class LlaisysExperts(Structure):
+    """struct LlaisysExperts (include/llaisys/mixers.h)."""
+    _fields_ = [("experts", c_size_t), ("identity", c_size_t), ("top", c_size_t), ("groups", c_size_t), ("keep", c_size_t),
+                ("width", c_size_t), ("ff", c_size_t), ("n_rows", c_size_t), ("scale", c_float), ("eps", c_float), ("gate_up", c_void_p),
+                ("down", c_void_p), ("correction", c_void_p), ("logits", c_void_p), ("gain", c_void_p), ("h", c_void_p),
+                ("chosen", c_void_p), ("weights", c_void_p), ("place", c_void_p), ("counts", c_void_p), ("line", c_void_p),
+                ("rows", c_void_p), ("act", c_void_p), ("out", c_void_p), ("x", c_void_p), ("next", c_void_p)]
 
 
 class LlaisysGates(Structure):
@@ -396,6 +432,21 @@ PROTOTYPES: dict[str, tuple] = {
                                               c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_size_t, POINTER(LlaisysGates),
                                               c_size_t, llaisysStream_t]),
     "llaisysMinGruScratchFloats": (c_size_t, [c_size_t, c_size_t]),
+    "llaisysRotaryTableWideDev": (c_int, [llaisysDeviceType_t, c_int, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t, llaisysStream_t]),
+    "llaisysPagedAttentionFadeDev": (c_int, [_KV, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t, c_size_t,
+                                             c_size_t, c_size_t, c_float, c_size_t, c_void_p, c_void_p, c_size_t, llaisysStream_t]),
+    "llaisysPagedKVCreateLatents": (c_int, [POINTER(_KV), llaisysDeviceType_t, c_int, llaisysDataType_t, c_size_t, POINTER(c_size_t),
+                                            POINTER(c_size_t), c_size_t, c_size_t, c_size_t, c_size_t]),
+    "llaisysPagedKVLatentAppendDev": (c_int, [_KV, c_size_t, POINTER(LlaisysLatentAppend), llaisysStream_t]),
+    "llaisysRotatePairsDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, c_void_p, c_size_t, c_size_t, c_void_p, c_size_t, c_size_t,
+                                      c_void_p, c_size_t, c_size_t, llaisysStream_t]),
+    "llaisysPagedKVLatentGatherDev": (c_int, [_KV, c_size_t, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t,
+                                              llaisysStream_t]),
+    "llaisysPagedAttentionExpandedDev": (c_int, [_KV, POINTER(LlaisysExpandedAttention), llaisysStream_t]),
+    "llaisysStateSpaceDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysStateSpace), c_int, llaisysStream_t]),
+    "llaisysStateSpaceSizes": (None, [llaisysDataType_t, c_size_t, c_size_t, c_size_t, c_size_t, c_size_t, c_size_t, POINTER(c_size_t),
+                                      POINTER(c_size_t), POINTER(c_size_t)]),
+    "llaisysExpertsDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysExperts), llaisysStream_t]),
     "llaisysMinGruDev": (c_int, [llaisysDeviceType_t, c_int, llaisysDataType_t, POINTER(LlaisysMinGru), c_int, llaisysStream_t]),
     "llaisysRotaryTableDev": (c_int, [llaisysDeviceType_t, c_int, c_void_p, c_void_p, c_void_p, c_size_t, c_size_t,
                                       llaisysStream_t]),
@@ -478,6 +529,7 @@ __all__ = [
     "llaisysDataType_t", "DataType", "llaisysDeviceType_t", "DeviceType", "llaisysMemcpyKind_t", "MemcpyKind",
     "Status", "library_path", "LlaisysQwen2Meta", "LlaisysQwen2Weights", "LlaisysEngineEvent",
     "LlaisysNormAppend", "LlaisysGatedLinear", "LlaisysGatedDelta", "LlaisysDoderaxMeta", "LlaisysDoderaxLayerMeta",
+    "LlaisysLatentAppend", "LlaisysExpandedAttention", "LlaisysStateSpace", "LlaisysExperts",
     "LlaisysGates", "LlaisysMinGru", "LlaisysLilovikMeta", "LlaisysLilovikLayerMeta", "LlaisysGatesAttentionMeta",
     "LlaisysFolivikMeta", "LlaisysFolivikLayerMeta", "LlaisysLatentAttentionMeta", "LlaisysFadingAttentionMeta",
     "LlaisysStateSpaceMixerMeta", "LlaisysExpertLayerMeta",

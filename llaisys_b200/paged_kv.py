@@ -14,8 +14,8 @@ from typing import Sequence
 
 import numpy as np
 
-from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysGatedDelta, LlaisysGatedLinear, LlaisysGates, LlaisysMinGru,
-                         LlaisysNormAppend, Status, llaisysPagedKV_t)
+from .libllaisys import (LIB_LLAISYS, DataType, DeviceType, LlaisysExpandedAttention, LlaisysExperts, LlaisysGatedDelta, LlaisysGatedLinear,
+                         LlaisysGates, LlaisysLatentAppend, LlaisysMinGru, LlaisysNormAppend, LlaisysStateSpace, Status, llaisysPagedKV_t)
 from .runtime import _addr
 
 _I32P = ctypes.POINTER(c_int32)
@@ -283,10 +283,50 @@ class PagedKVCache:
         self._kv = handle
         return self
 
+    @classmethod
+    def with_latents(cls, num_pages: int, layers: Sequence[tuple[int, int]], *, page_size: int = 16, dtype: DataType = DataType.BF16,
+                     device: DeviceType = DeviceType.NVIDIA, device_id: int = 0, max_seqs: int = 64,
+                     max_pages_per_seq: int | None = None) -> "PagedKVCache":
+        """Cache with one row of rank + rot_dim elements per token, for all heads; one (rank, rot_dim) per layer."""
+        self = cls.__new__(cls)
+        self._kv = None
+        self.max_pages_per_seq = max_pages_per_seq or num_pages
+        handle = llaisysPagedKV_t()
+        cols = [(ctypes.c_size_t * len(layers))(*[layer[i] for layer in layers]) for i in range(2)]
+        _check(LIB_LLAISYS.llaisysPagedKVCreateLatents(byref(handle), int(device), device_id, int(dtype), len(layers), *cols,
+                                                       num_pages, page_size, max_seqs, self.max_pages_per_seq))
+        self._kv = handle
+        return self
+
+    def latent_append_dev(self, layer: int, stream, **fields) -> None:
+        """Norms of both latents, rotation of the shared key part, append, gates to factors; fields of LlaisysLatentAppend."""
+        pointers = {"proj", "q_norm", "kv_norm", "rot_table", "q_latent", "row_scale", "seq_ids_dev", "positions_dev"}
+        args = LlaisysLatentAppend(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+        _check(LIB_LLAISYS.llaisysPagedKVLatentAppendDev(self._kv, layer, byref(args), stream))
+
+    def latent_gather_dev(self, layer: int, out, out_stride: int, seq_ids_dev, page_starts_dev, kv_lens_dev, n_seqs: int,
+                          max_kv_len: int, stream) -> None:
+        """Rows of chosen sequences (page_starts >= 0) side by side."""
+        _check(LIB_LLAISYS.llaisysPagedKVLatentGatherDev(self._kv, layer, _addr(out), out_stride, _addr(seq_ids_dev), _addr(page_starts_dev),
+                                                         _addr(kv_lens_dev), n_seqs, max_kv_len, stream))
+
+    def expanded_dev(self, stream, **fields) -> None:
+        """Chunk attention over plain keys (own and shared parts) and values; fields of LlaisysExpandedAttention."""
+        pointers = {"q", "k", "k_shared", "v", "page_starts_dev", "q_starts_dev", "kv_lens_dev", "out", "row_scale"}
+        args = LlaisysExpandedAttention(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+        _check(LIB_LLAISYS.llaisysPagedAttentionExpandedDev(self._kv, byref(args), stream))
+
+    def fade_dev(self, layer: int, out, q, seq_ids_dev, q_starts_dev, kv_lens_dev, *, n_seqs: int, total_q: int, max_q_len: int,
+                 max_kv_len: int, nh: int, scale: float, stream, fade_a, fade_b, window: int = 0, row_stride: int = 0) -> None:
+        """Decode (q_starts_dev None) or ragged chunks with a logarithmic penalty on distance, and a sliding window."""
+        _check(LIB_LLAISYS.llaisysPagedAttentionFadeDev(
+            self._kv, layer, _addr(out), _addr(q), _addr(seq_ids_dev), None if q_starts_dev is None else _addr(q_starts_dev),
+            _addr(kv_lens_dev), n_seqs, total_q, max_q_len, max_kv_len, nh, scale, window, _addr(fade_a), _addr(fade_b), row_stride, stream))
+
     def norm_append_dev(self, layer: int, stream, **fields) -> None:
         """Norm (per head, or of the whole row) and rotation of q and k, append of k and v, gates to factors; fields of LlaisysNormAppend (buffers may be
         tensors)."""
-        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev", "rot_table", "bias"}
+        pointers = {"proj", "q_norm", "k_norm", "q_out", "row_scale", "seq_ids_dev", "positions_dev", "rot_table", "bias", "head_scale"}
         args = LlaisysNormAppend(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
         _check(LIB_LLAISYS.llaisysPagedKVNormAppendDev(self._kv, layer, byref(args), stream))
 
@@ -353,6 +393,42 @@ def rotary_table_dev(table, positions_dev, freq_dev, n_rows: int, half: int, *, 
     """table [n_rows, half, 2] = (cos, sin)(position * freq), f32, on the device."""
     _check(LIB_LLAISYS.llaisysRotaryTableDev(int(DeviceType.NVIDIA), device_id, _addr(table), _addr(positions_dev), _addr(freq_dev),
                                              n_rows, half, stream))
+
+
+def rotary_table_wide_dev(table, positions_dev, freq_dev, n_rows: int, half: int, *, stream, device_id: int = 0) -> None:
+    """The same with freq f64 and angles formed and reduced in f64."""
+    _check(LIB_LLAISYS.llaisysRotaryTableWideDev(int(DeviceType.NVIDIA), device_id, _addr(table), _addr(positions_dev), _addr(freq_dev),
+                                                 n_rows, half, stream))
+
+
+def rotate_pairs_dev(dtype: DataType, out, out_dim: int, out_at: int, q, dim: int, rot_dims: int, rot_table, n_rows: int, nh: int, *,
+                     stream, device_id: int = 0) -> None:
+    """The dims of q [n_rows, nh, dim + rot_dims] behind the first dim, neighbours turned by their row's angles -> out [n_rows, nh, out_dim]
+    behind the first out_at."""
+    _check(LIB_LLAISYS.llaisysRotatePairsDev(int(DeviceType.NVIDIA), device_id, int(dtype), _addr(out), out_dim, out_at, _addr(q), dim, rot_dims,
+                                             _addr(rot_table), n_rows, nh, stream))
+
+
+def state_space_dev(dtype: DataType, *, decode: bool, stream, device_id: int = 0, **fields) -> None:
+    """Mamba-2 state space on device buffers; fields of LlaisysStateSpace (include/llaisys/mixers.h), buffers may be tensors."""
+    pointers = {"proj", "conv_w", "conv_b", "norm_w", "a_log", "dt_bias", "d_skip", "state", "seq_ids_dev", "q_starts_dev", "kv_lens_dev",
+                "out", "scratch", "scratch_segments"}
+    args = LlaisysStateSpace(**{k: (_addr(v) if k in pointers and v is not None else v) for k, v in fields.items()})
+    _check(LIB_LLAISYS.llaisysStateSpaceDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), int(decode), stream))
+
+
+def state_space_sizes(dtype: DataType, n_rows: int, heads: int, groups: int, dk: int, dv: int, taps: int) -> tuple[int, int, int]:
+    """Floats of a sequence's state, of `scratch` for n_rows rows and of `scratch_segments`."""
+    sizes = [c_size_t(0) for _ in range(3)]
+    LIB_LLAISYS.llaisysStateSpaceSizes(int(dtype), n_rows, heads, groups, dk, dv, taps, *[byref(s) for s in sizes])
+    return tuple(int(s.value) for s in sizes)
+
+
+def experts_dev(dtype: DataType, *, stream, device_id: int = 0, **fields) -> None:
+    """Mixture of experts on device buffers, added to x; fields of LlaisysExperts (include/llaisys/mixers.h), buffers may be tensors."""
+    numbers = {"experts", "identity", "top", "groups", "keep", "width", "ff", "n_rows", "scale", "eps"}
+    args = LlaisysExperts(**{k: (v if k in numbers or v is None else _addr(v)) for k, v in fields.items()})
+    _check(LIB_LLAISYS.llaisysExpertsDev(int(DeviceType.NVIDIA), device_id, int(dtype), byref(args), stream))
 
 
 def gated_linear_segment_floats(dtype: DataType, heads: int, dk: int, dv: int) -> int:

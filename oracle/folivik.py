@@ -48,18 +48,19 @@ def softmax_attention(q, k, v, scale, *, first=0, window=None, temp=None, bias=N
     bias: (a, b) per head, a ln(1 + b distance) is taken off the scores."""
     N, H = q.shape[:2]
     T, share = k.shape[0], H // k.shape[1]
+    k, v = k.repeat_interleave(share, 1), v.repeat_interleave(share, 1)
     out = torch.zeros(N, H, v.shape[2], dtype=torch.float64)
     for i in range(N):
         lo = 0 if window is None else max(0, first + i - window + 1)
-        keys = torch.arange(lo, first + i + 1)
-        assert keys[-1] < T
-        for h in range(H):
-            s = k[keys, h // share] @ q[i, h] * scale
-            if temp is not None:
-                s = s * temp[h]
-            if bias is not None:
-                s = s - bias[0][h] * torch.log(1 + bias[1][h] * (first + i - keys))
-            out[i, h] = torch.softmax(s, 0) @ v[keys, h // share]
+        hi = first + i + 1
+        assert hi <= T
+        s = torch.einsum("jhd,hd->hj", k[lo:hi], q[i]) * scale
+        if temp is not None:
+            s = s * temp.unsqueeze(1)
+        if bias is not None:
+            distance = first + i - torch.arange(lo, hi)
+            s = s - bias[0].unsqueeze(1) * torch.log(1 + bias[1].unsqueeze(1) * distance)
+        out[i] = torch.einsum("hj,jhd->hd", torch.softmax(s, 1), v[lo:hi])
     return out
 
 

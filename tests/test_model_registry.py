@@ -11,15 +11,17 @@ import torch
 
 import llaisys_b200 as llaisys
 from llaisys_b200 import trace
-from llaisys_b200.models import Doderax, Lilovik, Qwen2, Vozozen, load_model, model_class
+from llaisys_b200.models import Doderax, Folivik, Lilovik, Qwen2, Vozozen, load_model, model_class
 from llaisys_b200.models import doderax as dx
+from llaisys_b200.models import folivik as fk
 from llaisys_b200.models import lilovik as lk
 from llaisys_b200.models import vozozen as vz
 from llaisys_b200.models.weights import SafetensorsFile, checkpoint_files
 from oracle import doderax as doderax_oracle
+from oracle import folivik as folivik_oracle
 from oracle import lilovik as lilovik_oracle
 from oracle import vozozen as oracle
-from tests import doderax_cases, lilovik_cases
+from tests import doderax_cases, folivik_cases, lilovik_cases
 from tests import vozozen_cases as cases
 
 
@@ -37,6 +39,7 @@ def test_class_by_config():
     assert model_class({"architecture": "Vozozen"}) is Vozozen
     assert model_class({"architecture": "Doderax"}) is Doderax
     assert model_class({"architecture": "Lilovik"}) is Lilovik
+    assert model_class({"architecture": "Folivik"}) is Folivik
     assert model_class({"architectures": ["Qwen2ForCausalLM"], "model_type": "qwen2"}) is Qwen2
     assert model_class({"model_type": "qwen2"}) is Qwen2
     with pytest.raises(ValueError, match="Mamba"):
@@ -255,6 +258,110 @@ def test_lilovik_oracle_mechanisms_agree_with_closed_forms():
     assert torch.allclose(S, u[-1].abs() + 0.5)
     _, S = lilovik_oracle.min_gru(z * 0 + 1e3, torch.tensor([[0.0, -1e-9, -50.0]]).double().expand(T, 3), o, start)
     assert torch.allclose(S, torch.tensor([0.5, 0.5, 0.0]).double())
+
+
+@pytest.mark.parametrize("name", sorted(folivik_cases.CASES))
+def test_folivik_configuration_becomes_the_c_description(name):
+    cfg = folivik_cases.CASES[name]
+    meta = fk.build_meta(cfg, llaisys.DataType.BF16, 77)
+    assert (meta.nlayer, meta.width, meta.voc, meta.maxseq, meta.end_token) == (len(cfg["layers"]), cfg["width"], cfg["vocab"], 77, -1)
+    assert meta.eps == pytest.approx(cfg["norm"]["eps"])
+    for got, entry in zip(meta._layers, cfg["layers"]):
+        m, mlp = entry["mixer"], entry["mlp"]
+        part = {"latent_attention": got.latent, "attention": got.attn, "mamba2": got.ssm}[entry["type"]]
+        assert got.mixer == fk.LAYER_TYPES.index(entry["type"]) and part.heads == m["heads"] and part.vdim == m["vdim"]
+        if entry["type"] == "latent_attention":
+            assert (part.dim, part.rot_dim, part.q_rank, part.kv_rank) == (m["dim"], m["rot_dim"], m["q_rank"], m["kv_rank"])
+            assert part.rot_base == m["rot"]["base"] and part.scale == pytest.approx(m["scale"])
+        elif entry["type"] == "attention":
+            assert (part.kv_heads, part.dim, part.window) == (m["kv_heads"], m["dim"], m["mask"]["size"])
+        else:
+            assert (part.groups, part.state, part.taps, part.norm_groups) == (m["groups"], m["state"], m["conv"], m["norm_groups"])
+        if mlp is None:
+            assert got.mlp.top == 0
+            continue
+        r, groups = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
+        assert (got.mlp.experts, got.mlp.identity, got.mlp.top) == (r["experts"], r["identity"], r["top"])
+        assert (got.mlp.groups, got.mlp.keep, got.mlp.ff) == (groups["count"], groups["keep"], mlp["expert"]["ff"])
+        assert got.mlp.shared_ff == (mlp["shared"]["ff"] if mlp.get("shared") else 0) and got.mlp.scale == pytest.approx(r["scale"])
+    shapes = fk.weight_shapes(cfg)
+    assert shapes["l0.norm1"] == () and shapes["head"] == (cfg["vocab"], cfg["width"])
+
+
+def test_unknown_parts_of_a_folivik_configuration_are_refused():
+    def broken(change):
+        cfg = folivik_cases.case("mixed")[0]
+        change(cfg["layers"])
+        return cfg
+
+    for change, words in ((lambda l: l[0].update(type="serial"), "serial"), (lambda l: l[1]["mlp"].update(kind="dense"), "dense"),
+                          (lambda l: l[1]["mixer"]["rot"].update(dims=8), "rotated part"),
+                          (lambda l: l[0]["mlp"]["router"].update(groups={"count": 3, "keep": 1}), "do not fit"),
+                          (lambda l: l[0]["mlp"]["router"].update(top=7), "do not fit"),
+                          (lambda l: l[0]["mlp"]["router"].update(groups={"count": 4, "keep": 5}), "do not fit")):
+        with pytest.raises(ValueError, match=words):
+            fk.build_meta(broken(change), llaisys.DataType.BF16)
+    cfg, w = folivik_cases.case("recurrence_only")
+    with pytest.raises(RuntimeError, match="NVIDIA"):
+        Folivik(config=cfg, state_dict=w, device=llaisys.DeviceType.CPU)
+
+
+def test_folivik_oracle_mechanisms_agree_with_closed_forms():
+    torch.manual_seed(3)
+    o = folivik_oracle
+    T, H, G, d, dv = 9, 4, 2, 6, 5
+    q, k, v = torch.randn(T, H, d).double(), torch.randn(T, G, d).double(), torch.randn(T, G, dv).double()
+    ones, none = torch.ones(H).double(), torch.zeros(H).double()
+    full = o.softmax_attention(q, k, v, 0.3)
+    # a window of one token returns its value; a wide one is none; a penalty of zero and a factor of one change nothing
+    assert torch.allclose(o.softmax_attention(q, k, v, 0.3, window=1), v.repeat_interleave(2, 1))
+    assert torch.allclose(o.softmax_attention(q, k, v, 0.3, window=T, temp=ones, bias=(none, ones)), full)
+    assert torch.allclose(o.softmax_attention(q[4:], k, v, 0.3, first=4), full[4:])
+    # with equal scores the penalty leaves weights (1 + b distance)^(-a)
+    w = (1 + 0.5 * torch.arange(T - 1, -1, -1).double()) ** -2.0
+    got = o.softmax_attention(q, k * 0, v, 0.3, bias=(2 * ones, 0.5 * ones))[-1, 0]
+    assert torch.allclose(got, (w / w.sum()) @ v[:, 0])
+    # a turn keeps lengths, depends on the difference of positions in products, and is none at position 0
+    a, b = torch.randn(2, 1, 8).double()
+    at = lambda x, p: o.turn_pairs(x, [p], 100.0)[0]  # noqa: E731
+    assert torch.allclose(at(a, 0), a[0]) and torch.allclose(at(a, 5).norm(), a.norm())
+    assert torch.allclose(at(a, 7) @ at(b, 3), at(a, 14) @ at(b, 10))
+    # queries multiplied into the latents' space score like expanded keys
+    c, z, uk, uv = torch.randn(T, 7).double(), torch.randn(T, 2).double(), torch.randn(H * d, 7).double(), torch.randn(H * dv, 7).double()
+    kk, vv = o.latent_keys_values(c, z, uk, uv, H)
+    qq = torch.randn(T, H, d + 2).double()
+    wide = torch.cat([torch.einsum("thd,hdr->thr", qq[..., :d], uk.view(H, d, 7)), qq[..., d:]], dim=-1)
+    rows = torch.cat([c, z], dim=1).unsqueeze(1)
+    over = o.softmax_attention(wide, rows, c.unsqueeze(1), 0.4)
+    assert torch.allclose(torch.einsum("thr,hvr->thv", over, uv.view(H, dv, 7)), o.softmax_attention(qq, kk, vv, 0.4))
+    # a convolution whose only tap is the current token's; the inputs ahead of a portion stand in for its beginning
+    x, taps, bias = torch.randn(T, 3).double(), torch.randn(3, 4).double(), torch.randn(3).double()
+    last = torch.cat([torch.zeros(3, 3), torch.ones(3, 1)], dim=1).double()
+    assert torch.allclose(o.convolve(x, last, bias), o.silu(x + bias))
+    assert torch.allclose(o.convolve(x[5:], taps, bias, before=x[2:5]), o.convolve(x, taps, bias)[5:])
+    # no decay sums everything written; total decay keeps the newest token alone; a state carries over
+    xs, B, C, dt = torch.randn(T, 2, 4).double(), torch.randn(T, 1, 3).double(), torch.randn(T, 1, 3).double(), torch.rand(T, 2).double()
+    D = torch.randn(2).double()
+    _, S = o.state_space(xs, B, C, dt, torch.full((2,), -60.0).double(), D)
+    assert torch.allclose(S, torch.einsum("th,tn,thp->hnp", dt, B[:, 0], xs))
+    y, _ = o.state_space(xs, B, C, dt + 1, torch.full((2,), 8.0).double(), D)
+    assert torch.allclose(y[-1], ((B[-1, 0] @ C[-1, 0]) * (dt[-1] + 1) + D).unsqueeze(1) * xs[-1])
+    A = torch.randn(2).double()
+    y, S = o.state_space(xs, B, C, dt, A, D)
+    _, S5 = o.state_space(xs[:5], B[:5], C[:5], dt[:5], A, D)
+    y2, S2 = o.state_space(xs[5:], B[5:], C[5:], dt[5:], A, D, S5)
+    assert torch.allclose(y2, y[5:]) and torch.allclose(S2, S)
+    # parts of a norm are normed on their own
+    n = o.gated_parts_norm(torch.randn(2, 8).double() * torch.tensor([1.0] * 4 + [100.0] * 4).double(), torch.ones(2, 8).double(),
+                           torch.ones(8).double(), 2, 0.0)
+    assert torch.allclose(n.view(2, 2, 4).pow(2).mean(-1), torch.ones(2, 2).double())
+    # routing: the correction moves the choice and not the weights; refused groups stay out however low the others are
+    router = {"top": 2, "scale": 3.0, "groups": {"count": 2, "keep": 1}}
+    logits = torch.tensor([3.0, 2.0, 1.0, 0.0]).double()
+    chosen, weight = o.route(logits, torch.tensor([0.0, 0.0, -9.0, 1.0]).double(), router)
+    assert sorted(chosen.tolist()) == [2, 3] and weight.sum() == pytest.approx(3.0)
+    s = torch.softmax(logits, 0)
+    assert float(weight[chosen.tolist().index(2)]) == pytest.approx(float(3 * s[2] / (s[2] + s[3])))
 
 
 def test_no_host_stand_in():
