@@ -18,6 +18,7 @@ random permutation of a 16384-page pool):
   vozozen     the Vozozen design beside Qwen2 at equal size: whole models and single kernels (bench_models.py)
   doderax     the Doderax design beside Vozozen, in the same way
   lilovik     the Lilovik design beside Qwen2, in the same way
+  folivik     the Folivik design beside Vozozen, in the same way
 The default run (north_star) also measures config2 and config3 in the same process (N = 1: sub-records "config2",
 "config3") and, with N > 1, the KV-range split of config5 in the same process group (sub-record "kv_split"): the one
 mode of this path in which GPUs exchange data.
@@ -1285,7 +1286,7 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=100, help="steps per timed graph replay (the graph is replayed >= 30 times)")
     ap.add_argument("--warmup", type=int, default=20)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="north_star", choices=["north_star", "config2", "config3", "config4", "config5", "copy", "vozozen", "doderax", "lilovik"])
+    ap.add_argument("--workload", default="north_star", choices=["north_star", "config2", "config3", "config4", "config5", "copy", "vozozen", "doderax", "lilovik", "folivik"])
     ap.add_argument("--layers", type=int, default=4, help="pools to rotate over between steps (L2 flush)")
     ap.add_argument("--repeats", type=int, default=100, help="replays of the timed graph (at least 30)")
     ap.add_argument("--tp", action="store_true", help="config4 on several GPUs: tensor parallelism instead of sequence sharding")
@@ -1318,7 +1319,7 @@ def main() -> None:
     if args.workload == "copy":
         run_copy_workload(args)
         return
-    if args.workload in ("vozozen", "doderax", "lilovik"):
+    if args.workload in ("vozozen", "doderax", "lilovik", "folivik"):
         import bench_models
 
         bench_models.run(args)
