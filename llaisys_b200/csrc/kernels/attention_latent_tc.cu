@@ -84,10 +84,16 @@ __device__ __forceinline__ SeqGeom seq_geom(const Params &p, int a) {
     return g;
 }
 
-// Length of the line, and (kFind) the sequence that holds position `at` with the position of its beginning. For whole CTAs of whole
-// warps; s_scan: 34 ints of shared memory.
+// Length of the line, and (kFind) the sequence that holds position `at` with the position of its beginning; at < 0: the first position
+// of piece -1 - at of n_pieces, found by the same pass where every thread has at most one sequence. For whole CTAs of whole warps;
+// s_scan: 34 ints of shared memory.
+__device__ __forceinline__ int piece_length(int line, int n_pieces) {
+    const int even = (line + n_pieces - 1) / n_pieces;
+    return even < kMinPiece ? kMinPiece : even;
+}
+
 template <bool kFind>
-__device__ __forceinline__ int scan_line(const Params &p, int at, int *s_scan, int &seq, int &seq_begin) {
+__device__ __forceinline__ int scan_line(const Params &p, int at, int n_pieces, int *s_scan, int &seq, int &seq_begin) {
     const int tid = int(threadIdx.x), lane = tid & 31, warp = tid >> 5, n_warps = int(blockDim.x) >> 5;
     int before = 0;
     for (int base = 0; base < p.n_seqs; base += int(blockDim.x)) {
@@ -109,6 +115,9 @@ __device__ __forceinline__ int scan_line(const Params &p, int at, int *s_scan, i
             total += s_scan[w];
         }
         const int begin = before + warps_before + incl - len;
+        if (kFind && at < 0) { // (a single round: the total is known)
+            at = (-1 - at) * piece_length(total, n_pieces);
+        }
         if (kFind && len > 0 && begin <= at && at < begin + len) {
             s_scan[32] = base + tid;
             s_scan[33] = begin;
@@ -121,11 +130,6 @@ __device__ __forceinline__ int scan_line(const Params &p, int at, int *s_scan, i
         seq_begin = s_scan[33];
     }
     return before;
-}
-
-__device__ __forceinline__ int piece_length(int line, int n_pieces) {
-    const int even = (line + n_pieces - 1) / n_pieces;
-    return even < kMinPiece ? kMinPiece : even;
 }
 
 struct Walker {
@@ -223,15 +227,18 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
     Walker walker;
     int line;
     {
-        int a, begin;
-        line = scan_line<false>(p, 0, s_scan, a, begin);
+        const bool one_round = p.n_seqs <= kThreads;
+        line = one_round ? scan_line<true>(p, -1 - int(blockIdx.x), int(gridDim.x), s_scan, walker.a, walker.seq_begin)
+                         : scan_line<false>(p, 0, 0, s_scan, walker.a, walker.seq_begin);
         const int piece = piece_length(line, int(gridDim.x));
         if (int(blockIdx.x) * piece >= line) {
             grid_dependency_wait();
             grid_launch_dependents();
             return;
         }
-        scan_line<true>(p, int(blockIdx.x) * piece, s_scan, walker.a, walker.seq_begin);
+        if (!one_round) {
+            scan_line<true>(p, int(blockIdx.x) * piece, 0, s_scan, walker.a, walker.seq_begin);
+        }
         walker.g = seq_geom(p, walker.a);
     }
     const int piece = piece_length(line, int(gridDim.x)), piece_begin = int(blockIdx.x) * piece, piece_end = min(line, piece_begin + piece);
@@ -250,11 +257,6 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
         tmem_alloc(smem_u32(&s_tmem), kCols);
         tmem_relinquish();
     }
-    // rows that no page fills enter the products with weight zero: they only have to be finite
-    for (uint32_t at = base + uint32_t(tid) * 16; at < q_u32; at += kThreads * 16) {
-        asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};\n" ::"r"(at), "r"(0u) : "memory");
-    }
-    fence_proxy_async_smem();
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -275,14 +277,11 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
         for (int pos = piece_begin; ok && locate(p, walker, pos, piece_end, f); pos += f.t1 - f.t0) {
             const int n_pages = (walker.g.kv_len + kPage - 1) / kPage;
             const int32_t *table = p.block_table + (long long)(p.seq_ids != nullptr ? p.seq_ids[walker.a] : walker.a) * p.table_stride;
-            auto entry = [&](int t) {
-                const int at = t * kPagesPerTile + half * 4 + lane;
-                return lane < 4 && t < f.t1 && at < n_pages ? table[at] : 0;
-            };
+            // (behind the last page: that page again -- its rows enter the products with weight zero and only have to be finite)
+            auto entry = [&](int t) { return lane < 4 && t < f.t1 ? table[min(t * kPagesPerTile + half * 4 + lane, n_pages - 1)] : 0; };
             int pages = entry(f.t0);
             for (int t = f.t0; t < f.t1 && ok; ++t, ++tile_no) {
-                const int here = min(max(n_pages - t * kPagesPerTile - half * 4, 0), 4);
-                if (lane < here && (pages < 0 || pages >= p.num_pages)) {
+                if ((pages < 0 || pages >= p.num_pages)) {
                     atomicOr(p.error_flag, kErrBadPage);
                     pages = 0;
                 }
@@ -299,12 +298,12 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
                     const int n = min(p.chunks - 2 * pair, 2);
                     if (ok && elect_one()) {
                         const uint32_t dst = ring_u32 + uint32_t(slot) * kPairBytes + uint32_t(half) * (4 * 2048);
-                        mbar_arrive_expect_tx(bar(kBarFull + slot), uint32_t(here * n) * 2048u);
+                        mbar_arrive_expect_tx(bar(kBarFull + slot), uint32_t(4 * n) * 2048u);
 #pragma unroll
                         for (int c = 0; c < 2; ++c) {
 #pragma unroll
                             for (int i = 0; i < 4; ++i) {
-                                if (c < n && i < here) {
+                                if (c < n) {
                                     tma_load_2d(dst + uint32_t(c * kChunkBytes + i * 2048), &tmap, (2 * pair + c) * 64, row[i], bar(kBarFull + slot));
                                 }
                             }
@@ -321,12 +320,10 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
                         ok = wait(kBarS, tile_no - 1);
                     }
                     if (ok && elect_one()) {
-                        mbar_arrive_expect_tx(bar(kBarTail), uint32_t(here) * 2048u);
+                        mbar_arrive_expect_tx(bar(kBarTail), 4u * 2048u);
 #pragma unroll
                         for (int i = 0; i < 4; ++i) {
-                            if (i < here) {
-                                tma_load_2d(tail_u32 + uint32_t(half) * (4 * 2048) + uint32_t(i * 2048), &tmap, 2 * p.pairs * 64, row[i], bar(kBarTail));
-                            }
+                            tma_load_2d(tail_u32 + uint32_t(half) * (4 * 2048) + uint32_t(i * 2048), &tmap, 2 * p.pairs * 64, row[i], bar(kBarTail));
                         }
                     }
                     __syncwarp();
@@ -417,25 +414,27 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
             heads = min(p.group, p.nh - h0);
             first = block * p.block; // query of the chunk
         };
+        // kLanes neighbouring threads per row; a row's pieces in two batches, every load of a batch in flight
+        constexpr int kLanes = 128 / N, kBatch = (2 * kMaxPairs + 1) * 8 / kLanes / 2 + 1;
         auto load_q = [&](const SeqGeom &g, const Fragment &f) {
             int h0, heads, first;
             unit_at(g, f, h0, heads, first);
-            const int pieces = p.chunks * 8; // 16-byte pieces of a row, padded
-            const unsigned char *src = static_cast<const unsigned char *>(p.q);
-            for (int u0 = tid; u0 < N * pieces; u0 += 8 * 128) {
-                uint4 vals[8];
+            const int c = tid / kLanes, e0 = tid % kLanes, t = c / p.group, h = c - t * p.group, pieces = p.chunks * 8;
+            const bool holds = t < p.block && h < heads && first + t < g.q_len;
+            const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const unsigned char *>(p.q) +
+                                                               ((long long)(g.q_start + first + t) * p.nh + h0 + h) * p.dim * 2);
+            const int n = holds ? p.dim / 8 : 0;
+            for (int b = e0; b < pieces; b += kBatch * kLanes) {
+                uint4 vals[kBatch];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const int u = u0 + i * 128, c = u / pieces, e = u - c * pieces, t = c / p.group, h = c - t * p.group;
-                    vals[i] = make_uint4(0u, 0u, 0u, 0u);
-                    if (u < N * pieces && t < p.block && h < heads && first + t < g.q_len && e * 8 < p.dim) {
-                        vals[i] = *reinterpret_cast<const uint4 *>(src + (((long long)(g.q_start + first + t) * p.nh + h0 + h) * p.dim + e * 8) * 2);
-                    }
+                for (int i = 0; i < kBatch; ++i) {
+                    const int e = b + i * kLanes;
+                    vals[i] = e < n ? src[e] : make_uint4(0u, 0u, 0u, 0u);
                 }
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const int u = u0 + i * 128, c = u / pieces, e = u - c * pieces;
-                    if (u < N * pieces) {
+                for (int i = 0; i < kBatch; ++i) {
+                    const int e = b + i * kLanes;
+                    if (e < pieces) {
                         const uint32_t dst = q_u32 + uint32_t((e >> 3) * (N * 128) + c * 128 + (((e & 7) ^ (c & 7)) << 4));
                         asm volatile("st.shared.v4.u32 [%0], {%1, %2, %3, %4};\n" ::"r"(dst), "r"(vals[i].x), "r"(vals[i].y), "r"(vals[i].z), "r"(vals[i].w)
                                      : "memory");
@@ -575,25 +574,33 @@ __global__ void __launch_bounds__(kThreads, 1) attention_latent_kernel(const __g
             }
             if (cur.t0 == 0 && cur.t1 == g.tiles) {
                 const int t_col = col / p.group, h_col = col - t_col * p.group, row_col = g.q_start + first + t_col;
+                const bool holds = t_col < p.block && h_col < heads && first + t_col < g.q_len;
+                const unsigned columns = __ballot_sync(0xffffffffu, holds);
                 float factor = sum > 0.f ? 1.f / sum : 0.f;
-                if (p.row_scale != nullptr && t_col < p.block && h_col < heads && first + t_col < g.q_len) {
+                if (p.row_scale != nullptr && holds) {
                     factor *= p.row_scale[(long long)row_col * p.nh + h0 + h_col];
                 }
-                for (int pair = 0; pair < p.pairs; ++pair) {
+                float factors[N];
+#pragma unroll
+                for (int c = 0; c < N; ++c) {
+                    factors[c] = __shfl_sync(0xffffffffu, factor, c);
+                }
+                uint16_t *out = static_cast<uint16_t *>(p.out) + (long long)(g.q_start + first) * p.out_stride + (long long)h0 * p.rank + tid;
+                const long long next_query = p.out_stride - (long long)(p.group - 1) * p.rank;
+                for (int pair = 0; pair < p.pairs; ++pair, out += 128) {
                     float o[N];
                     load_columns<N>(lane_base + uint32_t(kColO + pair * N), o);
-                    const int dim = pair * 128 + tid;
-                    int tq = 0, h = 0;
+                    uint16_t *at = out;
+                    int left = p.group;
 #pragma unroll
                     for (int c = 0; c < N; ++c) {
-                        const float v = o[c] * __shfl_sync(0xffffffffu, factor, c);
-                        if (tq < p.block && h < heads && first + tq < g.q_len && dim < p.rank) {
-                            store_out<kBf16>(p.out, (long long)(g.q_start + first + tq) * p.out_stride + (long long)(h0 + h) * p.rank + dim, v);
+                        if ((columns >> c & 1u) != 0 && pair * 128 + tid < p.rank) {
+                            const float v = o[c] * factors[c];
+                            *at = kBf16 ? __bfloat16_as_ushort(__float2bfloat16_rn(v)) : __half_as_ushort(__float2half_rn(v));
                         }
-                        if (++h == p.group) {
-                            h = 0;
-                            ++tq;
-                        }
+                        --left;
+                        at += left != 0 ? (long long)p.rank : next_query;
+                        left = left != 0 ? left : p.group;
                     }
                 }
             } else {
@@ -667,7 +674,7 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(Params p, int n_piece
         __syncthreads();
     }
     int dummy_seq, dummy_begin;
-    const int line = scan_line<false>(p, 0, s_scan, dummy_seq, dummy_begin), piece = piece_length(line, n_pieces);
+    const int line = scan_line<false>(p, 0, 0, s_scan, dummy_seq, dummy_begin), piece = piece_length(line, n_pieces);
     if (h >= p.nh) {
         return;
     }

@@ -620,22 +620,62 @@ __global__ void paged_row_norm_append_kernel(unsigned char *__restrict__ k_pool,
     }
 }
 
-// K1d: one CTA per row (see LatentAppendArgs).
-template <typename T>
+// K1d: one CTA per row (see LatentAppendArgs). Pieces of VEC elements; the first kHeld of a thread of either latent stay in registers
+// between the sums and the stores, and the token's slot is looked up under the sums.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_append_kernel(T *__restrict__ k_pool, LatentAppendArgs a, const int32_t *__restrict__ table,
                                                             CopyGeom g, int32_t max_blocks, int32_t *error_flag) {
+    using P = Pack<T, VEC>;
+    constexpr int kHeld = 2;
     asm volatile("griddepcontrol.wait;\n" ::: "memory");
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     const int64_t row = blockIdx.x;
-    const int32_t tid = int32_t(threadIdx.x), step = int32_t(blockDim.x);
+    const int32_t tid = int32_t(threadIdx.x), step = int32_t(blockDim.x), nq = a.q_rank / VEC, nk = a.rank / VEC;
     const T *proj = static_cast<const T *>(a.proj) + row * a.row_stride;
-    const T *q = proj + a.q_at, *kv = proj + a.kv_at;
+    const P *q = reinterpret_cast<const P *>(proj + a.q_at), *kv = reinterpret_cast<const P *>(proj + a.kv_at);
+    const int32_t seq = a.seq_ids[row], pos = a.positions[row];
+    P hq[kHeld], hk[kHeld];
     float sq = 0.f, sk = 0.f;
-    for (int32_t i = tid; i < a.q_rank; i += step) {
-        sq = fmaf(to_f32(q[i]), to_f32(q[i]), sq);
+    auto square = [](const P &x, float &s) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            s = fmaf(to_f32(x.v[e]), to_f32(x.v[e]), s);
+        }
+    };
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+        if (tid + u * step < nq) {
+            hq[u] = q[tid + u * step];
+        }
+        if (tid + u * step < nk) {
+            hk[u] = kv[tid + u * step];
+        }
     }
-    for (int32_t i = tid; i < a.rank; i += step) {
-        sk = fmaf(to_f32(kv[i]), to_f32(kv[i]), sk);
+    const float2 *turn = reinterpret_cast<const float2 *>(a.rot_table) + row * (a.rot_dims / 2);
+    float2 t0 = make_float2(1.f, 0.f);
+    float u0 = 0.f, v0 = 0.f; // this thread's first pair to turn
+    const T *z = proj + a.kv_at + a.rank;
+    if (tid < a.rot_dims / 2) {
+        t0 = turn[tid];
+        u0 = to_f32(z[2 * tid]);
+        v0 = to_f32(z[2 * tid + 1]);
+    }
+    int32_t page, slot;
+    const bool stores = resolve_slot(table, g, seq, pos, max_blocks, error_flag, page, slot);
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+        if (tid + u * step < nq) {
+            square(hq[u], sq);
+        }
+        if (tid + u * step < nk) {
+            square(hk[u], sk);
+        }
+    }
+    for (int32_t i = tid + kHeld * step; i < nq; i += step) {
+        square(q[i], sq);
+    }
+    for (int32_t i = tid + kHeld * step; i < nk; i += step) {
+        square(kv[i], sk);
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -647,6 +687,11 @@ __global__ void __launch_bounds__(256) latent_append_kernel(T *__restrict__ k_po
         part_q[tid >> 5] = sq;
         part_k[tid >> 5] = sk;
     }
+    if (a.row_scale != nullptr) {
+        for (int32_t h = tid; h < a.nh; h += step) {
+            a.row_scale[row * a.nh + h] = a.gate_at < 0 ? 1.f : 1.f / (1.f + expf(-to_f32(proj[a.gate_at + h])));
+        }
+    }
     __syncthreads();
     sq = sk = 0.f;
     for (int32_t i = 0; i < step >> 5; ++i) { // every thread sums the few partials in the same order
@@ -654,28 +699,41 @@ __global__ void __launch_bounds__(256) latent_append_kernel(T *__restrict__ k_po
         sk += part_k[i];
     }
     const float inv_q = rsqrtf(sq / float(a.q_rank) + a.eps), inv_k = rsqrtf(sk / float(a.rank) + a.eps);
-    const T *q_norm = static_cast<const T *>(a.q_norm), *kv_norm = static_cast<const T *>(a.kv_norm);
-    T *q_out = static_cast<T *>(a.q_latent) + row * a.q_latent_stride;
-    for (int32_t i = tid; i < a.q_rank; i += step) {
-        q_out[i] = from_f32<T>(to_f32(q[i]) * inv_q * to_f32(q_norm[i]));
-    }
-    if (a.row_scale != nullptr) {
-        for (int32_t h = tid; h < a.nh; h += step) {
-            a.row_scale[row * a.nh + h] = a.gate_at < 0 ? 1.f : 1.f / (1.f + expf(-to_f32(proj[a.gate_at + h])));
+    auto normed = [](const P &x, const P &w, float inv) {
+        P y;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            y.v[e] = from_f32<T>(to_f32(x.v[e]) * inv * to_f32(w.v[e]));
+        }
+        return y;
+    };
+    const P *q_norm = static_cast<const P *>(a.q_norm), *kv_norm = static_cast<const P *>(a.kv_norm);
+    P *q_out = reinterpret_cast<P *>(static_cast<T *>(a.q_latent) + row * a.q_latent_stride);
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+        if (tid + u * step < nq) {
+            q_out[tid + u * step] = normed(hq[u], q_norm[tid + u * step], inv_q);
         }
     }
-    int32_t page, slot;
-    if (!resolve_slot(table, g, a.seq_ids[row], a.positions[row], max_blocks, error_flag, page, slot)) {
+    for (int32_t i = tid + kHeld * step; i < nq; i += step) {
+        q_out[i] = normed(q[i], q_norm[i], inv_q);
+    }
+    if (!stores) {
         return;
     }
     T *dst = k_pool + int64_t(page) * (g.page_stride_b / int64_t(sizeof(T))) + int64_t(slot) * (g.token_stride_b / int64_t(sizeof(T)));
-    for (int32_t i = tid; i < a.rank; i += step) {
-        dst[i] = from_f32<T>(to_f32(kv[i]) * inv_k * to_f32(kv_norm[i]));
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+        if (tid + u * step < nk) {
+            reinterpret_cast<P *>(dst)[tid + u * step] = normed(hk[u], kv_norm[tid + u * step], inv_k);
+        }
     }
-    const float2 *turn = reinterpret_cast<const float2 *>(a.rot_table) + row * (a.rot_dims / 2);
+    for (int32_t i = tid + kHeld * step; i < nk; i += step) {
+        reinterpret_cast<P *>(dst)[i] = normed(kv[i], kv_norm[i], inv_k);
+    }
     for (int32_t i = tid; i < a.rot_dims / 2; i += step) {
-        const float u = to_f32(kv[a.rank + 2 * i]), v = to_f32(kv[a.rank + 2 * i + 1]);
-        const float2 t = turn[i];
+        const float u = i == tid ? u0 : to_f32(z[2 * i]), v = i == tid ? v0 : to_f32(z[2 * i + 1]);
+        const float2 t = i == tid ? t0 : turn[i];
         dst[a.rank + 2 * i] = from_f32<T>(u * t.x - v * t.y);
         dst[a.rank + 2 * i + 1] = from_f32<T>(v * t.x + u * t.y);
     }
@@ -690,9 +748,14 @@ void launch_latent_append(cudaStream_t s, const KVView &kv, const LatentAppendAr
     g.page_size = kv.page_size;
     g.num_pages = kv.num_pages;
     g.table_stride = kv.table_stride;
-    const int32_t longest = std::max(a.q_rank, a.rank);
-    launch_programmatic(latent_append_kernel<T>, dim3(unsigned(a.n_rows)), longest <= 256 ? 64u : (longest <= 1024 ? 128u : 256u), s,
-                        static_cast<T *>(kv.k_base), a, kv.block_table, g, max_blocks, error_flag);
+    constexpr int kVec = 16 / int(sizeof(T));
+    const bool wide = a.q_rank % kVec == 0 && a.rank % kVec == 0 && a.row_stride % kVec == 0 && a.q_at % kVec == 0 && a.kv_at % kVec == 0 &&
+                      a.q_latent_stride % kVec == 0 && kv.token_stride % kVec == 0 && aligned16(a.proj) && aligned16(a.q_norm) &&
+                      aligned16(a.kv_norm) && aligned16(a.q_latent) && aligned16(kv.k_base);
+    const int32_t pieces = std::max(a.q_rank, a.rank) / (wide ? kVec : 1);
+    auto kernel = wide ? latent_append_kernel<T, kVec> : latent_append_kernel<T, 1>;
+    launch_programmatic(kernel, dim3(unsigned(a.n_rows)), pieces <= 128 ? 64u : (pieces <= 512 ? 128u : 256u), s, static_cast<T *>(kv.k_base), a,
+                        kv.block_table, g, max_blocks, error_flag);
 }
 
 // One CTA per (page, sequence); P: the widest piece that divides a row.
