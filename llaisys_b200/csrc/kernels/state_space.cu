@@ -17,8 +17,8 @@ namespace llaisys::kernels {
 
 namespace {
 
-constexpr int kDecodeThreads = 256;
-constexpr int kConvRows = 4; // rows of a thread of the preparing kernel
+constexpr int kDecodeThreads = 128;
+constexpr int kConvRows = 8, kConvRowsAny = 4; // rows of a thread of the preparing kernel: with a known number of taps, without
 
 template <int VEC>
 struct alignas(4 * VEC) Floats {
@@ -27,7 +27,7 @@ struct alignas(4 * VEC) Floats {
 
 // thread = (VEC columns, every row_groups-th of the dk rows)
 template <typename T, int VEC, int NR>
-__global__ void __launch_bounds__(kDecodeThreads, 3) state_decode_kernel(StateSpaceArgs a, int64_t y_stride, int col_groups) {
+__global__ void __launch_bounds__(kDecodeThreads, 10) state_decode_kernel(StateSpaceArgs a, int64_t y_stride, int col_groups) {
     using F = Floats<VEC>;
     extern __shared__ __align__(16) float smem[];
     auto up4 = [](int n) { return (n + 3) / 4 * 4; };
@@ -148,17 +148,47 @@ __global__ void __launch_bounds__(kDecodeThreads, 3) state_decode_kernel(StateSp
     }
 }
 
-// CTA: kConvRows rows, thread: VEC channels of them; the last CTAs of a row in x compute step sizes.
-template <typename T, int VEC>
+// The activation behind the convolutions of runs, rounded to the model dtype
+template <typename T>
+__device__ __forceinline__ T conv_out(float v) {
+    if constexpr (sizeof(T) == 4) {
+        return silu_of(v);
+    } else {
+        return from_f32<T>(__fdividef(v, 1.f + __expf(-v)));
+    }
+}
+
+// CTA: ROWS rows, thread: VEC channels of them; the last CTAs of a row in x compute step sizes. TAPS > 0: weights and the rows' inputs are
+// fetched once, all together; TAPS == 0: any number, tap by tap.
+template <typename T, int VEC, int TAPS, int ROWS>
 __global__ void __launch_bounds__(128) state_prepare_kernel(StateSpaceArgs a, StateScratch sc) {
     struct alignas(sizeof(T) * VEC) Piece {
         T v[VEC];
     };
     grid_dependency_wait();
     grid_launch_dependents();
-    __shared__ int s_first[kConvRows], s_pos[kConvRows], s_slot[kConvRows];
-    const int row0 = int(blockIdx.y) * kConvRows;
-    if (threadIdx.x < kConvRows && row0 + int(threadIdx.x) < a.n_rows) {
+    __shared__ int s_first[ROWS], s_pos[ROWS], s_slot[ROWS];
+    const int row0 = int(blockIdx.y) * ROWS, channels = a.channels(), ch = (int(blockIdx.x) * int(blockDim.x) + int(threadIdx.x)) * VEC;
+    const T *proj = static_cast<const T *>(a.proj);
+    const bool convolves = ch < channels;
+    constexpr int kIn = ROWS + TAPS - 1;
+    Piece in[TAPS > 0 ? kIn : 1], weight[TAPS > 0 ? TAPS : 1]; // weight: VEC channels x TAPS, as they lie in memory
+    if constexpr (TAPS > 0) {
+        if (convolves) {
+#pragma unroll
+            for (int i = 0; i < kIn; ++i) {
+                const int row = row0 - (TAPS - 1) + i;
+                if (row >= 0 && row < a.n_rows) { // (of whatever sequence: the first rows of a run do not use it)
+                    in[i] = *reinterpret_cast<const Piece *>(proj + int64_t(row) * a.row_stride + a.x_at + ch);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < TAPS; ++i) {
+                weight[i] = reinterpret_cast<const Piece *>(static_cast<const T *>(a.conv_w) + int64_t(ch) * TAPS)[i];
+            }
+        }
+    }
+    if (threadIdx.x < ROWS && row0 + int(threadIdx.x) < a.n_rows) {
         const int row = row0 + int(threadIdx.x);
         int lo = 0, hi = a.n_seqs - 1;
         while (lo < hi) { // last sequence whose first row is not behind this one
@@ -174,13 +204,11 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateSpaceArgs a, St
         s_slot[threadIdx.x] = a.seq_ids[lo];
     }
     __syncthreads();
-    const int channels = a.channels(), ch = (int(blockIdx.x) * int(blockDim.x) + int(threadIdx.x)) * VEC;
-    const T *proj = static_cast<const T *>(a.proj);
-    if (ch >= channels) {
+    if (!convolves) {
         float *dt = a.scratch + sc.dt;
         const int head = ch / VEC - (channels + VEC - 1) / VEC;
         if (head < a.heads) {
-            for (int u = 0; u < kConvRows && row0 + u < a.n_rows; ++u) {
+            for (int u = 0; u < ROWS && row0 + u < a.n_rows; ++u) {
                 dt[int64_t(row0 + u) * a.heads + head] =
                     softplus_of(to_f32(proj[int64_t(row0 + u) * a.row_stride + a.dt_at + head]) + a.dt_bias[head]);
             }
@@ -188,52 +216,73 @@ __global__ void __launch_bounds__(128) state_prepare_kernel(StateSpaceArgs a, St
         return;
     }
     const T *w = static_cast<const T *>(a.conv_w) + int64_t(ch) * a.taps, *bias = static_cast<const T *>(a.conv_b) + ch;
-    float acc[kConvRows][VEC];
-#pragma unroll
-    for (int u = 0; u < kConvRows; ++u) {
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            acc[u][e] = to_f32(bias[e]);
-        }
-    }
-    for (int tap = 0; tap < a.taps; ++tap) {
-        const int back = a.taps - 1 - tap;
-        float ww[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            ww[e] = to_f32(w[e * a.taps + tap]);
-        }
-#pragma unroll
-        for (int u = 0; u < kConvRows; ++u) {
-            const int row = row0 + u;
-            if (row >= a.n_rows) {
-                continue;
-            }
-            if (row - back >= s_first[u]) {
-                const Piece p = *reinterpret_cast<const Piece *>(proj + int64_t(row - back) * a.row_stride + a.x_at + ch);
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) {
-                    acc[u][e] = fmaf(ww[e], to_f32(p.v[e]), acc[u][e]);
-                }
-            } else if (s_pos[u] >= back) {
-                const float *ring = state_ring(a, s_slot[u]) + int64_t((s_pos[u] - back) % a.taps) * channels + ch;
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) {
-                    acc[u][e] = fmaf(ww[e], ring[e], acc[u][e]);
-                }
-            }
-        }
-    }
     T *conv = reinterpret_cast<T *>(a.scratch + sc.conv);
+    const int taps = TAPS > 0 ? TAPS : a.taps;
+    auto earlier = [&](int u, int back) { return state_ring(a, s_slot[u]) + int64_t((s_pos[u] - back) % taps) * channels + ch; };
+    auto store = [&](int u, const float (&acc)[VEC]) {
+        Piece p;
 #pragma unroll
-    for (int u = 0; u < kConvRows; ++u) {
-        if (row0 + u < a.n_rows) {
-            Piece p;
+        for (int e = 0; e < VEC; ++e) {
+            p.v[e] = conv_out<T>(acc[e]);
+        }
+        *reinterpret_cast<Piece *>(conv + int64_t(row0 + u) * sc.conv_stride + ch) = p;
+    };
+    if constexpr (TAPS > 0) {
+        float ww[TAPS][VEC], bb[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            bb[e] = to_f32(bias[e]);
+#pragma unroll
+            for (int tap = 0; tap < TAPS; ++tap) {
+                ww[tap][e] = to_f32(weight[(e * TAPS + tap) / VEC].v[(e * TAPS + tap) % VEC]);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < ROWS; ++u) {
+            if (row0 + u >= a.n_rows) {
+                break;
+            }
+            float acc[VEC];
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
-                p.v[e] = from_f32<T>(silu_of(acc[u][e]));
+                acc[e] = bb[e];
             }
-            *reinterpret_cast<Piece *>(conv + int64_t(row0 + u) * sc.conv_stride + ch) = p;
+#pragma unroll
+            for (int tap = 0; tap < TAPS; ++tap) {
+                const int back = TAPS - 1 - tap;
+                if (row0 + u - back >= s_first[u]) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        acc[e] = fmaf(ww[tap][e], to_f32(in[u + tap].v[e]), acc[e]);
+                    }
+                } else if (s_pos[u] >= back) {
+                    const float *ring = earlier(u, back);
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        acc[e] = fmaf(ww[tap][e], ring[e], acc[e]);
+                    }
+                }
+            }
+            store(u, acc);
+        }
+    } else {
+        for (int u = 0; u < ROWS && row0 + u < a.n_rows; ++u) {
+            float acc[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                acc[e] = to_f32(bias[e]);
+            }
+            for (int back = min(taps - 1, s_pos[u]); back >= 0; --back) {
+                const int tap = taps - 1 - back;
+                const bool here = row0 + u - back >= s_first[u];
+                const T *now = proj + int64_t(row0 + u - back) * a.row_stride + a.x_at + ch;
+                const float *ring = earlier(u, back);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) {
+                    acc[e] = fmaf(to_f32(w[e * taps + tap]), here ? to_f32(now[e]) : ring[e], acc[e]);
+                }
+            }
+            store(u, acc);
         }
     }
 }
@@ -406,7 +455,7 @@ void run_decode(cudaStream_t s, const StateSpaceArgs &a, const StateScratch &sc)
     const int vec = wide ? 4 : 1, col_groups = std::min((a.dv + vec - 1) / vec, kDecodeThreads), row_groups = kDecodeThreads / col_groups;
     auto up4 = [](int n) { return (n + 3) / 4 * 4; };
     const size_t smem = size_t(up4(a.dv) + 2 * up4(a.dk) + row_groups * col_groups * vec) * sizeof(float);
-    auto kernel = wide ? state_decode_kernel<T, 4, 8> : state_decode_kernel<T, 1, 8>;
+    auto kernel = wide ? state_decode_kernel<T, 4, 4> : state_decode_kernel<T, 1, 4>;
     launch_programmatic_smem(kernel, dim3(unsigned(a.n_seqs) * unsigned(a.heads)), kDecodeThreads, smem, s, a, sc.y_stride, col_groups);
     check_launch("state_space decode");
 }
@@ -428,9 +477,14 @@ template <typename T>
 void run_prepare(cudaStream_t s, const StateSpaceArgs &a, const StateScratch &sc) {
     constexpr int kVec = sizeof(T) == 2 ? 8 : 4;
     const bool wide = a.channels() % kVec == 0 && a.row_stride % kVec == 0 && a.x_at % kVec == 0 && aligned16(a.proj);
-    const int vec = wide ? kVec : 1, items = (a.channels() + vec - 1) / vec + a.heads;
-    auto kernel = wide ? state_prepare_kernel<T, kVec> : state_prepare_kernel<T, 1>;
-    const int64_t tiles = (a.n_rows + kConvRows - 1) / kConvRows;
+    const bool known = wide && a.taps >= 2 && a.taps <= 4 && aligned16(a.conv_w);
+    const int vec = wide ? kVec : 1, items = (a.channels() + vec - 1) / vec + a.heads, rows = known ? kConvRows : kConvRowsAny;
+    auto kernel = !wide           ? state_prepare_kernel<T, 1, 0, kConvRowsAny>
+                  : !known        ? state_prepare_kernel<T, kVec, 0, kConvRowsAny>
+                  : a.taps == 4   ? state_prepare_kernel<T, kVec, 4, kConvRows>
+                  : a.taps == 3   ? state_prepare_kernel<T, kVec, 3, kConvRows>
+                                  : state_prepare_kernel<T, kVec, 2, kConvRows>;
+    const int64_t tiles = (a.n_rows + rows - 1) / rows;
     CHECK_ARGUMENT(tiles <= 65535, "state space: too many rows in one call");
     launch_programmatic(kernel, dim3(unsigned((items + 127) / 128), unsigned(tiles)), 128u, s, a, sc);
     check_launch("state_space prepare");

@@ -34,6 +34,7 @@ constexpr int kWantedCtas = 148 * 6; // what a call is cut for
 struct Cut {
     int segment; // tokens of a segment, whole tiles; larger than any run: not cut
     float *states; // [segment of the call][heads][dk][dv]
+    float *decays; // [segment of the call][heads]: log of what is left of a state behind the segment
 };
 
 // Segment `index` of the batch, run after run; runs of one token have none. -> run, segment of the run, segments of the run (0: there
@@ -153,6 +154,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 3 : 1) state_tiles_ke
         __syncthreads();
     };
 
+    float decay = 0.f;
     constexpr float kLog2e = 1.4426950408889634f;
     const int lm_row = (lane & 7) + ((lane >> 3) & 1) * 8, lm_chunk = lane >> 4;  // rows 0 - 15 of two 8-column chunks
     const int lt_row = (lane & 7) + (lane >> 4) * 8, lt_chunk = (lane >> 3) & 1;  // the other order of the four matrices
@@ -273,6 +275,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 3 : 1) state_tiles_ke
         }
         // the state
         const float end = s_end, keep = ex2(end * kLog2e);
+        decay += end;
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
 #pragma unroll
@@ -311,6 +314,9 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 3 : 1) state_tiles_ke
                 *at = s;
             }
         });
+        if (tid == 0 && blockIdx.y == 0) {
+            cut.decays[int64_t(index) * a.heads + head] = decay;
+        }
     } else if (seg == segs - 1) {
         each_state(slot_state, [](float &s, float *at, bool holds) {
             if (holds) {
@@ -320,13 +326,14 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 3 : 1) state_tiles_ke
     }
 }
 
-// What segments add -> the states in front of them, run by run: thread = one element of a (run, head).
-__global__ void __launch_bounds__(256) state_scan_kernel(StateSpaceArgs a, StateScratch sc, Cut cut) {
+// What segments add -> the states in front of them, run by run: thread = one element of a (run, head); kAhead segments are fetched
+// together.
+__global__ void __launch_bounds__(256) state_scan_kernel(StateSpaceArgs a, Cut cut) {
+    constexpr int kAhead = 4;
     grid_dependency_wait();
     grid_launch_dependents();
-    __shared__ float s_sum;
     const int head = int(blockIdx.x) % a.heads, run = int(blockIdx.x) / a.heads, size = a.dk * a.dv;
-    const int first = a.q_starts[run], n_new = a.q_starts[run + 1] - first;
+    const int n_new = a.q_starts[run + 1] - a.q_starts[run];
     const int segs = n_new > 1 ? (n_new + cut.segment - 1) / cut.segment : 0;
     if (segs <= 1) {
         return;
@@ -349,40 +356,27 @@ __global__ void __launch_bounds__(256) state_scan_kernel(StateSpaceArgs a, State
     for (int w = 0; w < 8; ++w) {
         index += s_index[w];
     }
-    const float rate = -expf(a.a_log[head]);
-    const float *dts = a.scratch + sc.dt;
-    const bool fresh = a.kv_lens[run] == n_new;
-    const float *slot_state = a.state + int64_t(a.seq_ids[run]) * a.slot_stride + int64_t(head) * size;
     const int at = int(blockIdx.y) * 256 + int(threadIdx.x);
-    float s = at < size && !fresh ? slot_state[at] : 0.f;
-    for (int k = 0; k < segs; ++k) {
-        float *place = cut.states + (int64_t(index + k) * a.heads + head) * size + at;
-        float sum = 0.f;
-        for (int t = k * cut.segment + int(threadIdx.x); t < min(n_new, (k + 1) * cut.segment); t += 256) {
-            sum += dts[int64_t(first + t) * a.heads + head];
+    if (at >= size) {
+        return;
+    }
+    const bool fresh = a.kv_lens[run] == n_new;
+    float s = fresh ? 0.f : a.state[int64_t(a.seq_ids[run]) * a.slot_stride + int64_t(head) * size + at];
+    auto place = [&](int k) { return cut.states + (int64_t(index + k) * a.heads + head) * size + at; };
+    for (int k0 = 0; k0 < segs; k0 += kAhead) {
+        float added[kAhead], keep[kAhead];
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            const bool more = k0 + i + 1 < segs; // (behind the last segment nothing starts)
+            added[i] = more ? *place(k0 + i) : 0.f;
+            keep[i] = more ? cut.decays[int64_t(index + k0 + i) * a.heads + head] : 0.f;
         }
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        }
-        __shared__ float s_part[8];
-        __syncthreads();
-        if ((threadIdx.x & 31) == 0) {
-            s_part[threadIdx.x >> 5] = sum;
-        }
-        __syncthreads();
-        if (threadIdx.x == 0) {
-            float total = 0.f;
-            for (int w = 0; w < 8; ++w) {
-                total += s_part[w];
+        for (int i = 0; i < kAhead; ++i) {
+            if (k0 + i < segs) {
+                *place(k0 + i) = s;
+                s = fmaf(s, expf(keep[i]), added[i]);
             }
-            s_sum = total;
-        }
-        __syncthreads();
-        if (at < size) {
-            const float added = k + 1 < segs ? *place : 0.f;
-            *place = s;
-            s = fmaf(s, expf(rate * s_sum), added);
         }
     }
 }
@@ -393,15 +387,17 @@ void run_tiles(cudaStream_t s, const StateSpaceArgs &a, const StateScratch &sc) 
     constexpr size_t smem = 128 + size_t(kTile) * (kXB + 2 * kNB + 2 * 128);
     const int blocks = (a.dv + WARPS * 16 - 1) / (WARPS * 16);
     // segments: as many as fill the GPU a few times over, if the scratch holds their states
-    Cut cut{1 << 30, a.segments};
+    Cut cut{1 << 30, a.segments, nullptr};
     int segments = a.n_seqs;
     const int64_t tiles = (a.n_rows + kTile - 1) / kTile + a.n_seqs; // at most
     if (a.segments != nullptr && int64_t(a.n_seqs) * a.heads * blocks < kWantedCtas / 2) {
         const int64_t wanted = std::max<int64_t>(1, kWantedCtas / (int64_t(a.heads) * blocks));
         const int per = int(std::max<int64_t>(2, (tiles + wanted - 1) / wanted)) * kTile;
         const int64_t bound = a.n_rows / per + a.n_seqs;
-        if (per < a.max_q_len && size_t(bound) * a.heads * a.dk * a.dv <= a.segment_floats) {
+        const size_t floats = size_t(bound) * a.heads * a.dk * a.dv;
+        if (per < a.max_q_len && floats + size_t(bound) * a.heads <= a.segment_floats) {
             cut.segment = per;
+            cut.decays = a.segments + floats;
             segments = int(bound);
         }
     }
@@ -414,7 +410,7 @@ void run_tiles(cudaStream_t s, const StateSpaceArgs &a, const StateScratch &sc) 
     };
     if (cut.segment < (1 << 30)) {
         launch_programmatic_smem(prepare(state_tiles_kernel<NT, WARPS, true>), grid, WARPS * 32, smem, s, a, sc, cut);
-        launch_programmatic(state_scan_kernel, dim3(unsigned(a.n_seqs) * unsigned(a.heads), unsigned((a.dk * a.dv + 255) / 256)), 256u, s, a, sc, cut);
+        launch_programmatic(state_scan_kernel, dim3(unsigned(a.n_seqs) * unsigned(a.heads), unsigned((a.dk * a.dv + 255) / 256)), 256u, s, a, cut);
     }
     launch_programmatic_smem(prepare(state_tiles_kernel<NT, WARPS, false>), grid, WARPS * 32, smem, s, a, sc, cut);
     check_launch("state_space tiles");
@@ -430,7 +426,7 @@ size_t state_space_segment_floats(llaisysDataType_t dtype, size_t heads, size_t 
     if (dtype != LLAISYS_DTYPE_BF16 || dk > 128 || heads == 0) {
         return 0;
     }
-    return std::max<size_t>(kMaxPairs / heads, 1) * heads * dk * dv;
+    return std::max<size_t>(kMaxPairs / heads, 1) * heads * (dk * dv + 1);
 }
 
 void state_space_tiles(stream_t stream, const StateSpaceArgs &a) {
