@@ -186,7 +186,7 @@ void softcap_argmax(stream_t stream, float *logits, float cap, int64_t *idx_out,
 void paged_gather(stream_t stream, size_t elem_size, const KVView &kv, int32_t seq_row, int32_t n_tokens,
                   void *k_out, void *v_out, int32_t *error_flag);
 
-// Any dtype, head_dim <= 256, any GQA ratio, any page size: one CTA per (query row, query head), online
+// Any dtype, V rows of up to 1024, any GQA ratio, any page size, windows, kept tokens, distance penalties: one CTA per (query row, query head), online
 // softmax in f32. The correctness baseline for the specialised kernels and the kernel behind the legacy
 // operator for shapes they do not cover.
 void attention_generic(stream_t stream, llaisysDataType_t dtype, const KVView &kv, const AttnBatch &batch,

@@ -217,7 +217,7 @@ class Latents:
 
 
 # dtype, heads, rank, turned dims
-LATENT_SHAPES = [(torch.float32, 3, 40, 16), (torch.bfloat16, 4, 96, 32), (torch.bfloat16, 16, 512, 64), (torch.bfloat16, 5, 64, 64),
+LATENT_SHAPES = [(torch.float32, 3, 40, 16), (torch.bfloat16, 6, 88, 40), (torch.bfloat16, 16, 512, 64), (torch.bfloat16, 5, 64, 64),
                  (torch.bfloat16, 40, 256, 64), (torch.bfloat16, 1, 128, 0), (torch.float16, 12, 384, 24), (torch.bfloat16, 3, 13, 6),
                  (torch.bfloat16, 32, 200, 8), (torch.bfloat16, 7, 72, 56)]
 LATENT_TOL = {torch.float32: 2e-5, torch.bfloat16: 2e-2, torch.float16: 3e-3}
